@@ -1,0 +1,437 @@
+// Row kernels of the hybrid decoder: everything between its matrix products that works on one token at a time.
+//
+//   residual_step      the fp32 residual stream across a sublayer boundary, one pass:
+//                        x = x + mult * RMSNorm(y) w_post          (or x = RMSNorm(table[token]) w_post at the input)
+//                        depth average: x <- sum_j weight[j] X_j over the results X_j of all layers so far
+//                        h = RMSNorm(x) w_next                     (operand of the next matrix product)
+//   norm_shift_mix     h = RMSNorm(x) w; the inputs h + (h' - h) mu_s of a token-shifted mixer, h' being the h of the
+//                      token before (from the sequence's state at the start of a portion)
+//   poly_norm          a N(z) + b N(z^2) + c N(z^3) + e, N(v) = v / rms(v)
+//   split_tanh         tanh(z) as a bf16 pair (high part, remainder), so that a product with it loses no 16-bit digits
+//   head_norm          per-head RMSNorm of a mixer's fp32 output, with an optional silu gate
+//   gather_norm        RMSNorm of chosen rows (inputs of the LM head)
+//
+// The residual stream, its history, norms and states are fp32; GEMM operands are written as bf16 (or fp32 in the 32-bit
+// mode).  Widths are padded to a multiple of 8 with zero weights, so padding columns stay zero; means divide by the real
+// width.
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math.h>
+#include <stdint.h>
+
+#include "bounds_check.cuh"
+#include "host_utils.h"
+#include "row_io.cuh"
+
+namespace artb {
+
+struct ResidualArgs {
+  const int64_t* tokens;   // embedding lookup instead of y when set
+  const void* table;       // T [vocab, ldt]
+  int ldt;
+  long vocab;
+  void* y;                 // sublayer output, kind y_kind
+  int ldy, y_kind;
+  const float* x_in;
+  float* x_out;            // may alias x_in
+  int ldx;
+  const float* w_post;     // fp32 [dp]
+  float mult;
+  float* hist;             // fp32 [.., rows, ldx] results of the layers, or null
+  long hist_stride;
+  int hist_n;              // earlier results 0 .. hist_n - 1 are in hist; this one is stored as hist_n
+  const float* avg;        // fp32 [hist_n + 1], or null: store without averaging
+  const float* w_next;     // fp32 [dp], or null
+  void* h;                 // T [rows, ldh]
+  int ldh;
+  int d, dp;
+  float eps;
+  int* status;
+};
+
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, nv = a.dp >> 2;
+  float4 y[MAXV];
+  float ss = 0.f;
+  long tok = 0;
+  if (a.tokens) {
+    tok = a.tokens[row];
+    if (!index_ok(tok, a.vocab, a.status)) tok = 0;
+  }
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (v < nv) {
+      y[i] = a.tokens ? ld4(reinterpret_cast<const T*>(a.table) + static_cast<size_t>(tok) * a.ldt + v * 4)
+                      : take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, a.y_kind);
+      ss += sq4(y[i]);
+    }
+  }
+  ss = cta_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / a.d + a.eps);
+  const size_t xo = static_cast<size_t>(row) * a.ldx;
+  ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nv) {
+      const float4 w = ld4(a.w_post + v * 4);
+      float4 x = make_float4(y[i].x * r * w.x, y[i].y * r * w.y, y[i].z * r * w.z, y[i].w * r * w.w);
+      if (!a.tokens) {
+        const float4 x0 = ld4(a.x_in + xo + v * 4);
+        x = make_float4(fmaf(a.mult, x.x, x0.x), fmaf(a.mult, x.y, x0.y), fmaf(a.mult, x.z, x0.z), fmaf(a.mult, x.w, x0.w));
+      }
+      if (a.hist) {
+        float* hp = a.hist + xo + v * 4;
+        st4(hp + a.hist_n * a.hist_stride, x);
+        if (a.avg) {
+          const float wl = __ldg(a.avg + a.hist_n);
+          float4 s = make_float4(wl * x.x, wl * x.y, wl * x.z, wl * x.w);
+#pragma unroll 4
+          for (int j = 0; j < a.hist_n; ++j) {
+            const float wj = __ldg(a.avg + j);
+            const float4 q = ld4(hp + j * a.hist_stride);
+            s.x = fmaf(wj, q.x, s.x);
+            s.y = fmaf(wj, q.y, s.y);
+            s.z = fmaf(wj, q.z, s.z);
+            s.w = fmaf(wj, q.w, s.w);
+          }
+          x = s;
+        }
+      }
+      st4(a.x_out + xo + v * 4, x);
+      y[i] = x;
+      ss += sq4(x);
+    }
+  }
+  if (!a.w_next) return;       // uniform for the grid
+  ss = cta_sum(ss, red);
+  const float r2 = 1.f / sqrtf(ss / a.d + a.eps);
+  T* h = reinterpret_cast<T*>(a.h) + static_cast<size_t>(row) * a.ldh;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nv) {
+      const float4 w = ld4(a.w_next + v * 4);
+      st4(h + v * 4, make_float4(y[i].x * r2 * w.x, y[i].y * r2 * w.y, y[i].z * r2 * w.z, y[i].w * r2 * w.w));
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- token shift
+struct ShiftArgs {
+  const float* x;
+  int ldx;
+  const float* w;            // norm weight [dp]
+  const float* mu;           // [n_mix, dp]
+  int n_mix;
+  void* out;                 // T [n_mix][pitch rows][ldo]
+  long out_batch;            // elements between two mixes
+  int ldo;
+  float* state;              // [slots, dp]: h of the last token seen
+  long num_slots;
+  const int* row_seq;        // sequence of every row
+  const int* cu_q;           // first row of every sequence [n + 1]
+  const int* ctx;            // tokens of every sequence after this step
+  const int* state_slot;     // < 0: padding row
+  int d, dp;
+  float eps;
+  int* status;
+};
+
+// RMSNorm of row `x` (with weight) into v[]; contains block barriers
+template <int MAXV>
+__device__ __forceinline__ void norm_row(const float* x, const float* w, int nv, int d, float eps, float* red, float4 (&v)[MAXV]) {
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    v[i] = c < nv ? ld4(x + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += sq4(v[i]);
+  }
+  ss = cta_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / d + eps);
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < nv) {
+      const float4 g = ld4(w + c * 4);
+      v[i] = make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w);
+    }
+  }
+}
+
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(256) norm_shift_mix_kernel(const ShiftArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, nv = a.dp >> 2;
+  const int seq = a.row_seq[row];
+  const int r0 = a.cu_q[seq], rl = a.cu_q[seq + 1] - 1;
+  int slot = a.state_slot[seq];
+  if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
+  float4 h[MAXV], p[MAXV];
+  norm_row<MAXV>(a.x + static_cast<size_t>(row) * a.ldx, a.w, nv, a.d, a.eps, red, h);
+  const bool first = row == r0;
+  const bool start = first && a.ctx[seq] == rl - r0 + 1;      // the portion starts the sequence
+  if (first) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      p[i] = (start || slot < 0 || c >= nv) ? make_float4(0.f, 0.f, 0.f, 0.f)
+                                            : ld4(a.state + static_cast<size_t>(slot) * a.dp + c * 4);
+    }
+  } else {
+    norm_row<MAXV>(a.x + static_cast<size_t>(row - 1) * a.ldx, a.w, nv, a.d, a.eps, red, p);
+  }
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < nv) {
+      const float4 dlt = make_float4(p[i].x - h[i].x, p[i].y - h[i].y, p[i].z - h[i].z, p[i].w - h[i].w);
+      for (int s = 0; s < a.n_mix; ++s) {
+        const float4 m = ld4(a.mu + static_cast<size_t>(s) * a.dp + c * 4);
+        st4(reinterpret_cast<T*>(a.out) + s * a.out_batch + static_cast<size_t>(row) * a.ldo + c * 4,
+            make_float4(fmaf(dlt.x, m.x, h[i].x), fmaf(dlt.y, m.y, h[i].y), fmaf(dlt.z, m.z, h[i].z), fmaf(dlt.w, m.w, h[i].w)));
+      }
+    }
+  }
+  // The CTA of a portion's first row replaces the state: it is the only one that reads it, so no other CTA can see the
+  // new value too early.
+  if (first && slot >= 0) {
+    if (rl != r0) norm_row<MAXV>(a.x + static_cast<size_t>(rl) * a.ldx, a.w, nv, a.d, a.eps, red, h);
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int c = threadIdx.x + i * blockDim.x;
+      if (c < nv) st4(a.state + static_cast<size_t>(slot) * a.dp + c * 4, h[i]);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ PolyNorm
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(512)
+poly_norm_kernel(void* z, int ldz, int kind, const float* __restrict__ act, T* out, int ldo, int n, int np, float eps) {
+  __shared__ float red[3][16];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, nv = np >> 2;
+  float4 v[MAXV];
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < nv) {
+      v[i] = take4(z, static_cast<size_t>(row) * ldz + c * 4, kind);
+      const float* e = &v[i].x;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float q = e[j] * e[j], q2 = q * q;
+        s1 += q;
+        s2 += q2;
+        s3 = fmaf(q2, q, s3);
+      }
+    }
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  s1 = lane_sum(s1);
+  s2 = lane_sum(s2);
+  s3 = lane_sum(s3);
+  if (lane == 0) red[0][warp] = s1, red[1][warp] = s2, red[2][warp] = s3;
+  __syncthreads();
+  s1 = lane_sum(lane < nw ? red[0][lane] : 0.f);
+  s2 = lane_sum(lane < nw ? red[1][lane] : 0.f);
+  s3 = lane_sum(lane < nw ? red[2][lane] : 0.f);
+  const float a = act[0] / sqrtf(s1 / n + eps), b = act[1] / sqrtf(s2 / n + eps), c3 = act[2] / sqrtf(s3 / n + eps);
+  const float e0 = act[3];
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < nv) {
+      float4 o;
+      const float* x = &v[i].x;
+      float* y = &o.x;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] = c * 4 + j < n ? fmaf(fmaf(fmaf(c3, x[j], b), x[j], a), x[j], e0) : 0.f;
+      st4(out + static_cast<size_t>(row) * ldo + c * 4, o);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------- tanh for a low-rank decay
+// bf16: out[row] = [ hi(tanh z) | tanh z - hi ], r_p columns each; fp32: out[row] = tanh z
+template <typename T>
+__global__ void split_tanh_kernel(void* z, int ldz, int kind, T* out, int ldo, int M, int r, int rp) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= M * rp) return;
+  const int m = i / rp, c = i % rp;
+  const float t = c < r ? tanhf(take1(z, static_cast<size_t>(m) * ldz + c, kind)) : 0.f;
+  T* o = out + static_cast<size_t>(m) * ldo + c;
+  st1(o, t);
+  if (sizeof(T) == 2) st1(o + rp, t - __bfloat162float(__float2bfloat16(t)));
+}
+
+// --------------------------------------------------------------------------------------------- per-head norm
+// one warp per (row, head): out[row, h * vp + j] = rms(o[row, h, :])_j * w  (* silu(gate)), padding columns zero
+template <typename T>
+__global__ void __launch_bounds__(256)
+head_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__ w, int w_per_head, void* gate, int ldg,
+                 int gate_kind, T* out, int ldo, int M, int H, int vdim, int vp, float eps) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int u = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (u >= M * H) return;
+  const int m = u / H, h = u % H;
+  const float* x = o + static_cast<size_t>(m) * ldi + h * vdim;
+  float ss = 0.f;
+  for (int j = lane; j < vdim; j += 32) ss += x[j] * x[j];
+  const float r = 1.f / sqrtf(lane_sum(ss) / vdim + eps);
+  for (int j = lane; j < vp; j += 32) {
+    float v = 0.f;
+    if (j < vdim) {
+      v = x[j] * r * w[w_per_head ? h * vdim + j : j];
+      if (gate) v *= silu_f(take1(gate, static_cast<size_t>(m) * ldg + h * vdim + j, gate_kind));
+    }
+    st1(out + static_cast<size_t>(m) * ldo + h * vp + j, v);
+  }
+}
+
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(256)
+gather_norm_kernel(const float* __restrict__ x, int ldx, const int64_t* __restrict__ rows, const float* __restrict__ w, T* h,
+                   int ldh, int d, int dp, float eps, long n_rows, int* status) {
+  __shared__ float red[32];
+  float4 v[MAXV];
+  long r = rows[blockIdx.x];
+  if (!index_ok(r, n_rows, status)) r = 0;
+  norm_row<MAXV>(x + static_cast<size_t>(r) * ldx, w, dp >> 2, d, eps, red, v);
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c < (dp >> 2)) st4(h + static_cast<size_t>(blockIdx.x) * ldh + c * 4, v[i]);
+  }
+}
+
+static int row_threads(int dp) { return dp <= 512 ? 128 : 256; }
+// vectors of four per thread, rounded up to the instantiated counts; 0: too wide
+static int row_vecs(int dp, int threads) {
+  const int per = (dp / 4 + threads - 1) / threads;
+  return per <= 1 ? 1 : per <= 2 ? 2 : per <= 4 ? 4 : per <= 8 ? 8 : per <= 16 ? 16 : 0;
+}
+
+}  // namespace artb
+
+using namespace artb;
+
+#define ARTB_BY_VECS(V, CALL) \
+  switch (V) {                \
+    case 1: CALL(1); break;   \
+    case 2: CALL(2); break;   \
+    case 4: CALL(4); break;   \
+    case 8: CALL(8); break;   \
+    case 16: CALL(16); break; \
+    default: return ERR_TOO_LARGE; \
+  }
+
+// f32: operands (table, h) are fp32 instead of bf16.  See ResidualArgs; y_kind is a RowKind.
+ARTB_EXPORT int artb_residual_step(int f32, const int64_t* tokens, const void* table, int ldt, long vocab, void* y, int ldy,
+                                   int y_kind, const float* x_in, float* x_out, int ldx, const float* w_post, float mult,
+                                   float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
+                                   int ldh, int M, int d, int dp, float eps, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || !w_post || !x_out) return ERR_BAD_SHAPE;
+  if (!tokens && (!y || !x_in)) return ERR_BAD_SHAPE;
+  const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, hist, hist_stride, hist_n,
+                       avg, w_next, h, ldh, d, dp, eps, status};
+  const int th = row_threads(dp);
+  cudaError_t e = cudaSuccess;
+#define ARTB_RS(V)                                                                                                     \
+  e = f32 ? launch_kernel(residual_step_kernel<float, V>, dim3(M), dim3(th), 0, st, a)                                  \
+          : launch_kernel(residual_step_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, a)
+  ARTB_BY_VECS(row_vecs(dp, th), ARTB_RS)
+#undef ARTB_RS
+  return static_cast<int>(e);
+}
+
+ARTB_EXPORT int artb_norm_shift_mix(int f32, const float* x, int ldx, const float* w, const float* mu, int n_mix, void* out,
+                                    long out_batch, int ldo, float* state, long num_slots, const int* row_seq,
+                                    const int* cu_q, const int* ctx, const int* state_slot, int M, int d, int dp, float eps,
+                                    int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if ((dp & 3) || dp < d || (ldx & 3) || (ldo & 3) || (out_batch & 3) || n_mix < 1) return ERR_BAD_SHAPE;
+  const ShiftArgs a{x, ldx, w, mu, n_mix, out, out_batch, ldo, state, num_slots, row_seq, cu_q, ctx, state_slot, d, dp, eps,
+                    status};
+  const int th = row_threads(dp);
+  cudaError_t e = cudaSuccess;
+#define ARTB_SM(V)                                                                                                      \
+  e = f32 ? launch_kernel(norm_shift_mix_kernel<float, V>, dim3(M), dim3(th), 0, st, a)                                  \
+          : launch_kernel(norm_shift_mix_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, a)
+  ARTB_BY_VECS(row_vecs(dp, th), ARTB_SM)
+#undef ARTB_SM
+  return static_cast<int>(e);
+}
+
+// act: fp32 {a, b, c, e}; n real width, np padded width (columns n .. np - 1 of out are zero)
+ARTB_EXPORT int artb_poly_norm(int f32, void* z, int ldz, int kind, const float* act, void* out, int ldo, int M, int n, int np,
+                               float eps, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if ((np & 3) || np < n || (ldz & 3) || (ldo & 3)) return ERR_BAD_SHAPE;
+  const int th = np <= 1024 ? 128 : np <= 4096 ? 256 : 512;
+  cudaError_t e = cudaSuccess;
+#define ARTB_PN(V)                                                                                                       \
+  e = f32 ? launch_kernel(poly_norm_kernel<float, V>, dim3(M), dim3(th), 0, st, z, ldz, kind, act,                        \
+                          reinterpret_cast<float*>(out), ldo, n, np, eps)                                                 \
+          : launch_kernel(poly_norm_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, z, ldz, kind, act,                \
+                          reinterpret_cast<__nv_bfloat16*>(out), ldo, n, np, eps)
+  ARTB_BY_VECS(row_vecs(np, th), ARTB_PN)
+#undef ARTB_PN
+  return static_cast<int>(e);
+}
+
+ARTB_EXPORT int artb_split_tanh(int f32, void* z, int ldz, int kind, void* out, int ldo, int M, int r, int rp, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (rp < r || ldo < (f32 ? rp : 2 * rp)) return ERR_BAD_SHAPE;
+  const dim3 grid((M * rp + 255) / 256);
+  return static_cast<int>(f32 ? launch_kernel(split_tanh_kernel<float>, grid, dim3(256), 0, st, z, ldz, kind,
+                                              reinterpret_cast<float*>(out), ldo, M, r, rp)
+                              : launch_kernel(split_tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, z, ldz, kind,
+                                              reinterpret_cast<__nv_bfloat16*>(out), ldo, M, r, rp));
+}
+
+// o fp32 [M, H * vdim]; w [vdim] or, with w_per_head, [H * vdim]; gate [M, H * vdim] of kind gate_kind or null
+ARTB_EXPORT int artb_head_norm(int f32, const float* o, int ldi, const float* w, int w_per_head, void* gate, int ldg,
+                               int gate_kind, void* out, int ldo, int M, int H, int vdim, int vp, float eps, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (H <= 0 || vdim <= 0 || vp < vdim || ldo < H * vp) return ERR_BAD_SHAPE;
+  const dim3 grid(static_cast<unsigned>((static_cast<long>(M) * H + 7) / 8));
+  return static_cast<int>(f32 ? launch_kernel(head_norm_kernel<float>, grid, dim3(256), 0, st, o, ldi, w, w_per_head, gate, ldg,
+                                              gate_kind, reinterpret_cast<float*>(out), ldo, M, H, vdim, vp, eps)
+                              : launch_kernel(head_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, ldi, w, w_per_head,
+                                              gate, ldg, gate_kind, reinterpret_cast<__nv_bfloat16*>(out), ldo, M, H, vdim, vp,
+                                              eps));
+}
+
+ARTB_EXPORT int artb_gather_norm(int f32, const float* x, int ldx, const int64_t* rows, int n, const float* w, void* h, int ldh,
+                                 int d, int dp, float eps, long n_rows, int* status, cudaStream_t st) {
+  if (n <= 0) return 0;
+  if ((dp & 3) || dp < d || (ldx & 3) || (ldh & 3)) return ERR_BAD_SHAPE;
+  const int th = row_threads(dp);
+#define ARTB_GN(V)                                                                                                        \
+  if (f32)                                                                                                                \
+    gather_norm_kernel<float, V><<<n, th, 0, st>>>(x, ldx, rows, w, reinterpret_cast<float*>(h), ldh, d, dp, eps, n_rows, status); \
+  else                                                                                                                    \
+    gather_norm_kernel<__nv_bfloat16, V><<<n, th, 0, st>>>(x, ldx, rows, w, reinterpret_cast<__nv_bfloat16*>(h), ldh, d, dp, eps, \
+                                                           n_rows, status)
+  ARTB_BY_VECS(row_vecs(dp, th), ARTB_GN)
+#undef ARTB_GN
+  return static_cast<int>(cudaGetLastError());
+}

@@ -1,0 +1,225 @@
+// Latent attention over a paged cache of latents.
+//
+// A token's cache row is [ c: rank_p | rotated key part: rot_p ] (both padded to a multiple of 16 with zeros): the latent
+// that every head expands into its keys and values, and one rotated key part that all heads share.  Position i sees the
+// keys j with 0 <= i - j < window.
+//
+//   latent_finish_kernel   what follows the q | latent projection, one CTA per token: RMSNorm of the latent, interleaved
+//                          rotation of the shared key part and of every head's rotated query part, cache write, and the
+//                          queries in the layout the attention form of the row reads
+//   latent_attend_kernel   attention in latent space ("absorbed" form): q~ = W_uk^T q per head is taken against the cached
+//                          latents themselves, the weighted latents are expanded by W_uv afterwards.  Scalar fp32
+//                          arithmetic for any sizes and both number formats (the 32-bit mode runs on it).
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math.h>
+#include <stdint.h>
+
+#include "bounds_check.cuh"
+#include "host_utils.h"
+#include "row_io.cuh"
+
+namespace artb {
+
+struct LatentFinish {
+  void* p;                  // [M, ldp] of kind `kind`: q (H heads of dim | rot) | latent (rank) | rotated part (rot)
+  int ldp, kind;
+  const float* w;           // latent norm weight [rank]
+  const float* inv_freq;    // [rot / 2]
+  const int* pos;
+  const int* slot;          // cache row of every token, < 0: not written
+  void* cache;              // T [num_slots, ldc]
+  int ldc;
+  long num_slots;
+  int n_abs;                // rows below n_abs go to the absorbed layout
+  void* qn;                 // T [H][pitch][dim_p]
+  void* qr;                 // T [H][pitch][rot_p]
+  int pitch;
+  void* qe;                 // T [M - n_abs][ldqe], heads of (dim + rot)
+  int ldqe;
+  int H, dim, dim_p, rot, rot_p, rank, rank_p;
+  float eps;
+  int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a) {
+  __shared__ float red[32];
+  extern __shared__ float cs[];            // cos, sin of rot / 2 angles
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, tid = threadIdx.x, hp = a.rot >> 1, hq = a.dim + a.rot;
+  float *cc = cs, *sn = cs + hp;
+  const size_t row = static_cast<size_t>(m) * a.ldp;
+  for (int i = tid; i < hp; i += blockDim.x) sincosf(static_cast<float>(a.pos[m]) * a.inv_freq[i], &sn[i], &cc[i]);
+  int slot = a.slot[m];
+  if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
+  T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
+  // latent: two passes over the row (the second finds it in L1 / L2; a taken workspace is only cleared then)
+  const int c0 = a.H * hq, rkind = a.kind == ROW_F32_TAKE ? ROW_F32 : a.kind;
+  float ss = 0.f;
+  for (int i = tid; i < a.rank; i += blockDim.x) {
+    const float x = take1(a.p, row + c0 + i, rkind);
+    ss += x * x;
+  }
+  const float r = 1.f / sqrtf(cta_sum(ss, red) / a.rank + a.eps);      // also the barrier behind cos / sin
+  for (int i = tid; i < a.rank; i += blockDim.x) {
+    const float x = take1(a.p, row + c0 + i, a.kind);
+    if (slot >= 0) st1(crow + i, x * r * a.w[i]);
+  }
+  for (int i = tid; i < hp; i += blockDim.x) {
+    const float u = take1(a.p, row + c0 + a.rank + 2 * i, a.kind), v = take1(a.p, row + c0 + a.rank + 2 * i + 1, a.kind);
+    if (slot >= 0) {
+      st1(crow + a.rank_p + 2 * i, u * cc[i] - v * sn[i]);
+      st1(crow + a.rank_p + 2 * i + 1, v * cc[i] + u * sn[i]);
+    }
+  }
+  const bool absorbed = m < a.n_abs;
+  for (int j = tid; j < a.H * a.dim; j += blockDim.x) {
+    const int h = j / a.dim, i = j - h * a.dim;
+    const float x = take1(a.p, row + h * hq + i, a.kind);
+    if (absorbed) st1(reinterpret_cast<T*>(a.qn) + (static_cast<size_t>(h) * a.pitch + m) * a.dim_p + i, x);
+    else st1(reinterpret_cast<T*>(a.qe) + static_cast<size_t>(m - a.n_abs) * a.ldqe + h * hq + i, x);
+  }
+  for (int j = tid; j < a.H * hp; j += blockDim.x) {
+    const int h = j / hp, i = j - h * hp;
+    const size_t o = row + h * hq + a.dim + 2 * i;
+    const float u = take1(a.p, o, a.kind), v = take1(a.p, o + 1, a.kind);
+    const float x = u * cc[i] - v * sn[i], y = v * cc[i] + u * sn[i];
+    T* d = absorbed ? reinterpret_cast<T*>(a.qr) + (static_cast<size_t>(h) * a.pitch + m) * a.rot_p + 2 * i
+                    : reinterpret_cast<T*>(a.qe) + static_cast<size_t>(m - a.n_abs) * a.ldqe + h * hq + a.dim + 2 * i;
+    st1(d, x);
+    st1(d + 1, y);
+  }
+}
+
+struct LatentAttend {
+  const void* ql;           // T [H][pitch][rank_p]   queries in latent space
+  const void* qr;           // T [H][pitch][rot_p]
+  int pitch;
+  const void* cache;        // T [num_blocks * block_size, ldc]
+  int ldc;
+  const int* block_table;
+  int max_blocks, block_size;
+  long num_blocks;
+  const int* row_seq;
+  const int* pos;           // position of the row's token
+  const int* ctx;           // tokens of the sequence; 0: padding sequence
+  int window;               // <= 0: every earlier key
+  float scale;
+  void* o;                  // T [H][pitch][rank_p]   weighted latents
+  int rank_p, rot_p;
+  int* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_attend_kernel(const LatentAttend a) {
+  constexpr int KT = 128;
+  extern __shared__ float la_s[];
+  float* sq = la_s;                          // [rank_p + rot_p]
+  __shared__ float sp[KT];
+  __shared__ long srow[KT];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int D = a.rank_p + a.rot_p;
+  const int seq = a.row_seq[m], p = a.pos[m];
+  const int len = a.ctx[seq] > 0 ? p + 1 : 0;
+  const int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  const size_t qo = static_cast<size_t>(h) * a.pitch + m;
+  for (int i = tid; i < a.rank_p; i += 128) sq[i] = take1(const_cast<void*>(a.ql), qo * a.rank_p + i, sizeof(T) == 2 ? ROW_BF16 : ROW_F32);
+  for (int i = tid; i < a.rot_p; i += 128) sq[a.rank_p + i] = take1(const_cast<void*>(a.qr), qo * a.rot_p + i, sizeof(T) == 2 ? ROW_BF16 : ROW_F32);
+  constexpr int OV = 8;                      // up to 1024 latent dimensions
+  float acc[OV];
+#pragma unroll
+  for (int i = 0; i < OV; ++i) acc[i] = 0.f;
+  float mx = -INFINITY, sum = 0.f;
+  const T* cache = reinterpret_cast<const T*>(a.cache);
+  for (int k0 = lo; k0 < len; k0 += KT) {
+    __syncthreads();
+    const int j = k0 + tid;
+    float s = -INFINITY;
+    long cr = -1;
+    if (j < len) {
+      const int blk = a.block_table[static_cast<size_t>(seq) * a.max_blocks + j / a.block_size];
+      if (index_ok(blk, a.num_blocks, a.status)) {
+        cr = static_cast<long>(blk) * a.block_size + j % a.block_size;
+        const T* c = cache + cr * a.ldc;
+        float t = 0.f;
+        for (int i = 0; i < D; i += 4) {
+          const float4 x = ld4(c + i);
+          t = fmaf(x.x, sq[i], t);
+          t = fmaf(x.y, sq[i + 1], t);
+          t = fmaf(x.z, sq[i + 2], t);
+          t = fmaf(x.w, sq[i + 3], t);
+        }
+        s = t * a.scale;
+      }
+    }
+    float tm = s;
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, x));
+    if ((tid & 31) == 0) red[tid >> 5] = tm;
+    __syncthreads();
+    tm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+    const float mn = fmaxf(mx, tm);
+    if (mn == -INFINITY) continue;           // uniform: no usable key so far
+    const float corr = mx == -INFINITY ? 0.f : expf(mx - mn);
+    const float e = s == -INFINITY ? 0.f : expf(s - mn);
+    mx = mn;
+    sp[tid] = e;
+    srow[tid] = cr;
+    sum = sum * corr + cta_sum(e, red);      // barriers publish sp / srow
+    const int nk = min(KT, len - k0);
+#pragma unroll
+    for (int i = 0; i < OV; ++i) {
+      const int dcol = tid + i * 128;
+      if (dcol < a.rank_p) {
+        float t = acc[i] * corr;
+        for (int k = 0; k < nk; ++k)
+          if (srow[k] >= 0) t = fmaf(sp[k], take1(const_cast<void*>(a.cache), srow[k] * a.ldc + dcol, sizeof(T) == 2 ? ROW_BF16 : ROW_F32), t);
+        acc[i] = t;
+      }
+    }
+  }
+  const float inv = sum > 0.f ? 1.f / sum : 0.f;
+#pragma unroll
+  for (int i = 0; i < OV; ++i) {
+    const int dcol = tid + i * 128;
+    if (dcol < a.rank_p) st1(reinterpret_cast<T*>(const_cast<void*>(static_cast<const void*>(a.o))) + qo * a.rank_p + dcol, acc[i] * inv);
+  }
+}
+
+}  // namespace artb
+
+using namespace artb;
+
+ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const float* w, const float* inv_freq, const int* pos,
+                                   const int* slot, void* cache, int ldc, long num_slots, int n_abs, void* qn, void* qr, int pitch,
+                                   void* qe, int ldqe, int M, int H, int dim, int dim_p, int rot, int rot_p, int rank, int rank_p,
+                                   float eps, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (H <= 0 || (rot & 1) || dim_p < dim || rot_p < rot || rank_p < rank || ldc < rank_p + rot_p) return ERR_BAD_SHAPE;
+  if ((n_abs > 0 && (!qn || !qr || pitch < n_abs)) || (n_abs < M && (!qe || ldqe < H * (dim + rot)))) return ERR_BAD_SHAPE;
+  const LatentFinish a{p, ldp, kind, w, inv_freq, pos, slot, cache, ldc, num_slots, n_abs, qn, qr, pitch, qe, ldqe, H, dim, dim_p,
+                       rot, rot_p, rank, rank_p, eps, status};
+  const size_t smem = static_cast<size_t>(rot) * 4;
+  return static_cast<int>(f32 ? launch_kernel(latent_finish_kernel<float>, dim3(M), dim3(256), smem, st, a)
+                              : launch_kernel(latent_finish_kernel<__nv_bfloat16>, dim3(M), dim3(256), smem, st, a));
+}
+
+ARTB_EXPORT int artb_latent_attend(int f32, const void* ql, const void* qr, int pitch, const void* cache, int ldc,
+                                   const int* block_table, int max_blocks, int block_size, long num_blocks, const int* row_seq,
+                                   const int* pos, const int* ctx, int window, float scale, void* o, int M, int H, int rank_p,
+                                   int rot_p, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (H <= 0 || H > 65535 || rank_p > 1024 || (rank_p & 3) || (rot_p & 3) || (ldc & 3) || ldc < rank_p + rot_p || pitch < M ||
+      block_size <= 0)
+    return ERR_BAD_SHAPE;
+  const LatentAttend a{ql, qr, pitch, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, window, scale,
+                       o, rank_p, rot_p, status};
+  const size_t smem = static_cast<size_t>(rank_p + rot_p) * 4;
+  return static_cast<int>(f32 ? launch_kernel(latent_attend_kernel<float>, dim3(M, H), dim3(128), smem, st, a)
+                              : launch_kernel(latent_attend_kernel<__nv_bfloat16>, dim3(M, H), dim3(128), smem, st, a));
+}

@@ -86,6 +86,7 @@ class Sequence:
         self.params = params
         self.adapter = adapter
         self.blocks: list[int] = []
+        self.state_slot = -1                  # row of the recurrent-state buffers, for models that carry one
         self.num_cached = 0
         self.prefix_hit_tokens = 0            # prompt tokens served from the prefix cache at (the last) admission
         self.salt: int | None = None          # prefix-cache salt (adapter slot + version) the KV was computed under
@@ -112,7 +113,8 @@ class Sequence:
 
     def view(self) -> SeqView:
         return SeqView(self.tokens, self.num_cached, self.blocks, self.adapter, self.params.temperature, self.seed,
-                       len(self.output_ids), self.params.top_p, self.params.top_k, self.params.min_p, self.proc)
+                       len(self.output_ids), self.params.top_p, self.params.top_k, self.params.min_p, self.proc,
+                       state_slot=self.state_slot)
 
 
 def _deliver(per_queue: dict) -> None:
@@ -146,6 +148,9 @@ class Engine:
         time (its KV accumulates in its blocks; the token is sampled after the last chunk), so a long prompt neither
         waits for an empty step nor builds one oversized forward pass; without it such a prompt runs alone, whole."""
         self.runner, self.bm, self.kv = runner, block_manager, kv_cache
+        # models with recurrent layers: a sequence also holds a state slot, and cached blocks of another sequence are of
+        # no use to it (the state behind them is gone), so nothing is committed to or matched in the prefix cache
+        self.state_slots = getattr(kv_cache, "state_slots", None)
         self.log_stats_interval = log_stats_interval     # seconds between throughput lines in the log; None: no lines
         self._stats_mark = (time.monotonic(), 0, 0, 0, 0)   # time, prompt tokens, generated tokens, cache queries, hits
         self.chunked = enable_chunked_prefill
@@ -254,8 +259,8 @@ class Engine:
             self.kv.discard()
             with self._lock:   # KV of in-flight sequences is gone: recompute them from their tokens
                 for s in self.running + self.prefilling:
-                    self.bm.free(s.blocks)
-                    s.blocks, s.num_cached = [], 0
+                    self._drop_memory(s)
+                    s.num_cached = 0
                     self.waiting.appendleft(s)
                 self.running, self.prefilling = [], []
 
@@ -432,14 +437,22 @@ class Engine:
             except RuntimeError:
                 pass        # that client's event loop is closed: nobody is left to read its events; the others go on
 
+    def _drop_memory(self, seq: Sequence) -> None:
+        """Give back the blocks and the state slot a sequence holds."""
+        if seq.blocks:
+            self.bm.free(seq.blocks)
+            seq.blocks = []
+        if seq.state_slot >= 0:
+            self.state_slots.free(seq.state_slot)
+            seq.state_slot = -1
+
     def _release(self, seq: Sequence) -> None:
         if seq.blocks:
             toks = seq.tokens
             # KV computed (even partly) under weights that were replaced since admission must not become reusable
-            if seq.salt is not None and seq.salt == self._salt(seq.adapter):
+            if self.state_slots is None and seq.salt is not None and seq.salt == self._salt(seq.adapter):
                 self.bm.commit(seq.blocks, toks[: len(toks) - 1], seq.salt)
-            self.bm.free(seq.blocks)
-            seq.blocks = []
+        self._drop_memory(seq)
         seq.done_event.set()
 
     def _blocks_needed(self, n_tokens: int) -> int:
@@ -483,7 +496,10 @@ class Engine:
                     continue
                 toks = seq.tokens
                 salt = self._salt(seq.adapter)
-                cached = self.bm.match_prefix(toks[:-1], salt)   # always recompute the last token
+                if self.state_slots is not None and self.state_slots.num_free == 0:
+                    break
+                # always recompute the last token
+                cached = self.bm.match_prefix(toks[:-1], salt) if self.state_slots is None else []
                 n_new = len(toks) - len(cached) * bs
                 take = chunk(n_new)
                 if take <= 0 or (picked and len(cached) * bs + take > att_budget):
@@ -495,6 +511,8 @@ class Engine:
                     self.bm.free(cached)
                     break
                 self.waiting.popleft()
+                if self.state_slots is not None:
+                    seq.state_slot = self.state_slots.alloc()
                 seq.blocks = cached + fresh
                 seq.num_cached = len(cached) * bs
                 seq.prefix_hit_tokens = min(seq.num_cached, len(seq.prompt_ids))
@@ -522,8 +540,8 @@ class Engine:
                 steps = 1
                 continue
             victim = self.running.pop()   # newest: recompute later
-            self.bm.free(victim.blocks)
-            victim.blocks, victim.num_cached = [], 0
+            self._drop_memory(victim)
+            victim.num_cached = 0
             with self._lock:
                 self.waiting.appendleft(victim)
             self.stats.preemptions += 1
@@ -547,7 +565,7 @@ class Engine:
             with self._lock:
                 toks, n_prompt, adapter, loop, fut = self.score_queue.popleft()
             try:
-                res = self.runner.score(toks, n_prompt, adapter)
+                res = self._score(toks, n_prompt, adapter)
                 reply = lambda f=fut, r=res: f.done() or f.set_result(r)      # noqa: E731
             except BaseException as e:  # noqa: BLE001
                 reply = lambda f=fut, e=e: f.done() or f.set_exception(e)     # noqa: E731
@@ -559,8 +577,7 @@ class Engine:
             s.finished, s.finish_reason = True, "abort"
         for s in [s for s in self.prefilling if s.finished]:    # aborted half-way through its prompt
             self.prefilling.remove(s)
-            self.bm.free(s.blocks)
-            s.blocks = []
+            self._drop_memory(s)
             s.done_event.set()
         done = [s for s in self.running if s.finished]
         if done:
@@ -576,6 +593,15 @@ class Engine:
                 v = s.view()
                 v.upto = upto
                 views.append(v)
+            # a runner that takes mixed batches advances the running sequences by one token in the same step, so that
+            # they do not stall while prompts are computed
+            riders: list[Sequence] = []
+            if getattr(self.runner, "mixed_steps", False) and self.running and self._ensure_decode_blocks(1):
+                riders = list(self.running)
+                for s in riders:
+                    v = s.view()
+                    v.num_cached, v.upto = len(s.tokens) - 1, len(s.tokens)
+                    views.append(v)
             t0 = time.monotonic()
             self._inflight = [s for s, _ in work]       # out of the queues while the runner works: told if it fails
             toks, lps = self.runner.prefill(views)
@@ -596,6 +622,9 @@ class Engine:
                 s.num_cached = 0
                 self._emit(s, t, lps[i], tops[0][i] if tops else None)
                 self.running.append(s)
+            for i, s in enumerate(riders, len(work)):
+                t = s.forced.popleft() if s.forced else toks[i]
+                self._emit(s, t, lps[i], tops[0][i] if tops else None)
             return True
         if not self.running:
             return False
@@ -619,6 +648,20 @@ class Engine:
                     t = s.forced.popleft()
                 self._emit(s, t, lps[k][i], tops[k][i] if tops else None)
         return True
+
+    def _score(self, toks: list[int], n_prompt: int, adapter: int) -> list[float]:
+        if self.state_slots is None:
+            return self.runner.score(toks, n_prompt, adapter)
+        # a recurrent model scores through the cache and the state like any prompt: lend it blocks and a slot
+        seq = Sequence(toks, SamplingParams(), adapter, None)
+        blocks, slot = self.bm.alloc(self._blocks_needed(len(toks))), self.state_slots.alloc()
+        seq.blocks, seq.state_slot = blocks or [], -1 if slot is None else slot
+        try:
+            if blocks is None or slot is None:
+                raise RuntimeError("no cache blocks or state slot free to score a sequence")
+            return self.runner.score_view(seq.view(), n_prompt)
+        finally:
+            self._drop_memory(seq)
 
     def _traced_step(self) -> bool:
         """``step()``; with ``ARTB_TRACE_FILE`` set every iteration becomes a span of a Chrome trace plus counters
@@ -709,9 +752,7 @@ class Engine:
             self.waiting.clear()
             self.running, self.prefilling = [], []
         for s in dead:
-            if s.blocks:
-                self.bm.free(s.blocks)
-                s.blocks = []
+            self._drop_memory(s)
         self.bm.reset_prefix_cache()
         self._outbox = {}
         drop = getattr(self.runner, "drop_graphs", None)

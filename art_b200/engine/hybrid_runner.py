@@ -1,0 +1,304 @@
+"""Execution of hybrid decoders (``models/hybrid.py``) for the rollout engine.
+
+One batch is ragged: every sequence brings its next tokens, whether one decoded token or a portion of its prompt, and all
+of them go through the layers together.  ``Ragged`` describes it to the kernels: rows of the sequences one after another
+(``cu_q``), positions, cache rows, block tables, state slots.  Sequences with one new token come first, so that a row range
+tells which form of attention a row takes.
+
+Every sublayer is ``norm -> mixer or feed-forward -> norm -> residual``; the step from one to the next (post-norm, residual
+multiplier, depth average, next input norm) is one kernel over the fp32 residual stream (``ops.hybrid.residual_step``).
+Operands of the matrix products are bf16; with ``dtype=torch.float32`` everything is fp32, products included, through the
+same layer code.
+
+Decoding several tokens per call, CUDA graphs, sampling and logit processing come from
+:class:`~art_b200.engine.runner.DeviceRunner`.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from ..models.hybrid import SHIFT_MIXES, HybridConfig, check_weights
+from ..ops import hybrid as hy
+from ..ops.hybrid import Out, as_out, pad
+from .runner import DeviceRunner, SeqView
+
+
+@dataclass
+class Ragged:
+    """A batch on the device.  ``single``: every sequence brings exactly one token (row m = sequence m)."""
+    M: int
+    n_seqs: int
+    tokens: torch.Tensor        # int64 [M]
+    pos: torch.Tensor           # int32 [M]
+    slot: torch.Tensor          # int32 [M]   cache row of the token, -1: not written
+    row_seq: torch.Tensor       # int32 [M]
+    cu_q: torch.Tensor          # int32 [n_seqs + 1]
+    ctx: torch.Tensor           # int32 [n_seqs]  tokens after this step; 0: padding
+    state_slot: torch.Tensor    # int32 [n_seqs]
+    bt: torch.Tensor            # int32 [n_seqs, max_blocks]
+    single: bool
+
+
+class HybridRunner(DeviceRunner):
+    mixed_steps = True
+
+    def __init__(self, cfg: HybridConfig, kv, base: dict[str, torch.Tensor], *, device="cuda", dtype: torch.dtype = torch.bfloat16,
+                 max_loras: int = 0):
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"hybrid models run in bfloat16 or float32, not {dtype}")
+        check_weights(cfg, base)
+        self.cfg, self.kv, self.device, self.dtype = cfg, kv, torch.device(device), dtype
+        self.exact32 = dtype == torch.float32
+        self.max_loras = max_loras
+        self.dp = pad(cfg.hidden_size)
+        self._load(base)
+        self._buf: dict = {}
+
+    # -- weights ------------------------------------------------------------------------------------
+    def _mat(self, w: torch.Tensor, rows: int | None = None, cols: int | None = None) -> torch.Tensor:
+        """A matrix as GEMM operand: operand dtype, rows and columns padded with zeros (default: to multiples of 8)."""
+        out = torch.zeros(rows or pad(w.shape[0]), cols or pad(w.shape[1]), dtype=self.dtype, device=self.device)
+        out[:w.shape[0], :w.shape[1]] = w.to(self.device)
+        return out
+
+    def _vec(self, w: torch.Tensor, n: int | None = None) -> torch.Tensor:
+        w = w.reshape(-1).to(self.device, torch.float32)
+        out = torch.zeros(n or w.numel(), dtype=torch.float32, device=self.device)
+        out[:w.numel()] = w
+        return out
+
+    def _heads_in(self, w: torch.Tensor, heads: int, vdim: int) -> torch.Tensor:
+        """An output projection whose input keeps every head's ``vdim`` values at a pitch of ``pad(vdim)``."""
+        d, vp = w.shape[0], pad(vdim)
+        out = torch.zeros(self.dp, heads, vp, dtype=self.dtype, device=self.device)
+        out[:d, :, :vdim] = w.to(self.device).view(d, heads, vdim)
+        return out.view(self.dp, heads * vp)
+
+    def _load(self, base: dict[str, torch.Tensor]) -> None:
+        cfg, dp = self.cfg, self.dp
+        V = cfg.vocab_size
+        self._head = self._mat(base["embed"], pad(V), dp)          # embedding and output table are one
+        self.embed = self.lm_head = self._head[:V]
+        self.embed_norm, self.final_norm = self._vec(base["embed.norm"], dp), self._vec(base["final.norm"], dp)
+        self.layers = []
+        for i, s in enumerate(cfg.layers):
+            w = {k[len(f"l{i}."):]: t for k, t in base.items() if k.startswith(f"l{i}.")}
+            m = {k[4:]: t for k, t in w.items() if k.startswith("mix.")}
+            L: dict = {"norm1": self._vec(w["norm1"], dp), "norm1b": self._vec(w["norm1b"], dp), "dwa": self._vec(w["dwa"])}
+            if s.type == "latent_attention":
+                rank_p = pad(s.kv_rank, 16)
+                L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, dp)
+                L["c_norm"] = self._vec(m["dkv.norm"])
+                uk, uv = m["uk"].view(s.heads, s.dim, s.kv_rank), m["uv"].view(s.heads, s.vdim, s.kv_rank)
+                L["uk_t"] = torch.zeros(s.heads, rank_p, pad(s.dim, 16), dtype=self.dtype, device=self.device)
+                L["uk_t"][:, :s.kv_rank, :s.dim] = uk.transpose(1, 2).to(self.device)
+                L["uv"] = torch.zeros(s.heads, pad(s.vdim), rank_p, dtype=self.dtype, device=self.device)
+                L["uv"][:, :s.vdim, :s.kv_rank] = uv.to(self.device)
+                L["inv_freq"] = torch.tensor([s.rope_base ** (-2.0 * j / s.rot_dim) for j in range(s.rot_dim // 2)], dtype=torch.float64
+                                             ).to(self.device, torch.float32)
+            elif s.type == "hgrn2":
+                L["qv"] = self._mat(torch.cat([m["q"], m["v"]], 0), None, dp)
+                L["f"], L["f_b"], L["lower"] = self._mat(m["f"], None, dp), self._vec(m["f.b"]), self._vec(m["lower"])
+                L["o_norm"] = self._vec(m["norm"])
+            else:
+                n = pad(s.heads * s.dim)
+                L["mu"] = torch.stack([self._vec(m["mu." + x], dp) for x in SHIFT_MIXES])
+                L["rkvg"] = torch.stack([self._mat(m[x], n, dp) for x in "rkvg"])
+                rp = pad(s.decay_rank)
+                L["w1"] = self._mat(m["w1"], rp, dp)
+                w2 = self._mat(m["w2"], n, rp)
+                # bf16: tanh arrives as a pair (high part, remainder), both halves against the same matrix
+                L["w2"] = w2 if self.exact32 else torch.cat([w2, w2], 1).contiguous()
+                L["w0"], L["u"], L["o_norm"] = self._vec(m["w0"]), self._vec(m["u"]), self._vec(m["norm"])
+            L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
+            if s.ff:
+                L["norm2"], L["norm2b"] = self._vec(w["norm2"], dp), self._vec(w["norm2b"], dp)
+                L["up"], L["down"] = self._mat(w["mlp.up"], None, dp), self._mat(w["mlp.down"], dp, pad(s.ff))
+                L["act"] = self._vec(w["mlp.act"])
+            self.layers.append(L)
+
+    def set_adapter(self, slot: int, state) -> None:
+        if state is not None:
+            raise ValueError(f"{self.cfg.name}: adapters are not supported for hybrid models")
+
+    # -- products and buffers -------------------------------------------------------------------------
+    def _mm(self, x, W, f32: bool = False) -> Out:
+        if self.exact32:
+            return as_out(hy.gemm_f32(x, W))
+        from ..ops.gemm import gemm_tn
+
+        return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16))
+
+    def _logits(self, hidden) -> torch.Tensor:
+        y = self._mm(hidden, self._head, f32=True).t
+        return y[:, :self.cfg.vocab_size]
+
+    def _heads_buf(self, name: str, batch: int, b: Ragged, width: int) -> torch.Tensor:
+        """A head-major operand ``[batch, pitch, width]``, row pitch a multiple of 128.  Rows past M are never read back
+        but a tile loads them, so the storage starts as zeros and later holds old finite values.  Batches of single
+        tokens have buffers of their own size, which stay where they are: captured graphs hold their addresses."""
+        pitch = pad(b.M, 128)
+        n = batch * pitch * width
+        # one width per buffer: the padding columns of a row are written by nobody
+        key = (name, width, n) if b.single else (name, width)
+        t = self._buf.get(key)
+        if t is None or t.numel() < n or t.device != self.device:
+            t = self._buf[key] = torch.zeros(n, dtype=self.dtype, device=self.device)
+        return t[:n].view(batch, pitch, width)
+
+    # -- batches ------------------------------------------------------------------------------------------
+    def _pack(self, seqs: list[SeqView]) -> tuple[Ragged, list[tuple[int, int]]]:
+        """The batch of the sequences' not-yet-cached tokens and, per sequence, its row range."""
+        bs, dev = self.kv.shape[1], self.device
+        end = [len(s.tokens) if s.upto is None else min(s.upto, len(s.tokens)) for s in seqs]
+        order = sorted(range(len(seqs)), key=lambda i: end[i] - seqs[i].num_cached > 1)      # single tokens first
+        tok, pos, slot, row_seq, cu, ranges = [], [], [], [], [0], [(0, 0)] * len(seqs)
+        for j, i in enumerate(order):
+            s = seqs[i]
+            n0, n1 = s.num_cached, end[i]
+            if n1 <= n0:
+                raise ValueError("a scheduled sequence brings at least one token")
+            tok += s.tokens[n0:n1]
+            pos += range(n0, n1)
+            slot += [s.blocks[t // bs] * bs + t % bs for t in range(n0, n1)]
+            row_seq += [j] * (n1 - n0)
+            ranges[i] = (cu[-1], cu[-1] + n1 - n0)
+            cu.append(cu[-1] + n1 - n0)
+        width = max(len(s.blocks) for s in seqs)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
+        b = Ragged(cu[-1], len(seqs), torch.tensor(tok, dtype=torch.int64, device=dev), i32(pos), i32(slot), i32(row_seq), i32(cu),
+                   i32([end[i] for i in order]), i32([seqs[i].state_slot for i in order]),
+                   i32([seqs[i].blocks + [0] * (width - len(seqs[i].blocks)) for i in order]), cu[-1] == len(seqs))
+        return b, ranges
+
+    # -- layers ---------------------------------------------------------------------------------------------
+    def _forward(self, b: Ragged, capture: list | None = None, want_hidden: bool = False):
+        """The residual stream ``x`` fp32 [M, dp] behind the last layer and, with ``want_hidden``, its final norm in the
+        operand dtype.  ``capture``: receives a copy of the stream after every layer."""
+        cfg, dp, d, eps, m = self.cfg, self.dp, self.cfg.hidden_size, self.cfg.norm_eps, self.cfg.residual_mult
+        M, dev = b.M, self.device
+        x = torch.empty((M, dp), dtype=torch.float32, device=dev)
+        h = torch.empty((M, dp), dtype=self.dtype, device=dev)
+        hist = torch.empty((len(self.layers) + 1, M, dp), dtype=torch.float32, device=dev)
+        first_norm = lambda i: (self.layers[i]["norm1"] if cfg.layers[i].type != "wkv" else None) if i < len(self.layers) \
+            else (self.final_norm if want_hidden else None)      # noqa: E731  (a token-shift mixer norms its own input)
+        hy.residual_step(x, self.embed_norm, d, eps, tokens=b.tokens, table=self.embed, hist=hist, hist_n=0, w_next=first_norm(0), h=h)
+        for i, (s, L) in enumerate(zip(cfg.layers, self.layers)):
+            y = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b)
+            post = L["norm1b"]
+            if s.ff:
+                hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
+                z = self._mm(h, L["up"])
+                a = torch.empty((M, pad(s.ff)), dtype=self.dtype, device=dev)
+                y = self._mm(hy.poly_norm(z, L["act"], a, s.ff, eps), L["down"])
+                post = L["norm2b"]
+            hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
+            if capture is not None:
+                capture.append(x[:, :d].clone())
+        return x, h
+
+    def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Out:
+        M, H = b.M, s.heads
+        cache = self.kv.layers[i]["latent"]
+        p = self._mm(h, L["qkv"])
+        rank_p, rot_p = pad(s.kv_rank, 16), pad(s.rot_dim, 16)
+        qn = self._heads_buf("qn", H, b, pad(s.dim, 16))
+        qr = self._heads_buf("qr", H, b, rot_p)
+        hy.latent_finish(p, L["c_norm"], L["inv_freq"], b.pos, b.slot, cache, M, qn, qr, None, H, s.dim, s.rot_dim, s.kv_rank,
+                         self.cfg.norm_eps)
+        ql = self._heads_buf("ql", H, b, rank_p)
+        hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), M, c_batch=ql.stride(0))
+        ol = self._heads_buf("ol", H, b, rank_p)
+        hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, M)
+        vp = pad(s.vdim)
+        o = torch.empty((M, H * vp), dtype=self.dtype, device=self.device)
+        hy.gemm_batched(ol, L["uv"], o, M, c_batch=vp)
+        return self._mm(o, L["o"])
+
+    def _scan(self, mode, i, s, L, q, k, v, g, aux, bias, gate, b: Ragged) -> Out:
+        """Recurrence, per-head norm and gate, output projection."""
+        M, H, vp, eps = b.M, s.heads, pad(s.vdim), self.cfg.norm_eps
+        state = self.kv.layers[i]["state"]
+        per_head = gate is not None
+        out = torch.empty((M, H * vp), dtype=self.dtype, device=self.device)
+        if b.single:
+            hy.linear_decode(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, H, s.dim, s.vdim, L["o_norm"], per_head,
+                             gate, out, vp, eps)
+        else:
+            o = torch.empty((M, H * s.vdim), dtype=torch.float32, device=self.device)
+            hy.linear_scan(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, H, s.dim, s.vdim, o)
+            hy.head_norm(o, L["o_norm"], per_head, H, s.vdim, vp, out, eps, gate)
+        return self._mm(out, L["o"])
+
+    def _mix_hgrn2(self, i, s, L, x, h, b: Ragged) -> Out:
+        qv = self._mm(h, L["qv"])
+        g = self._mm(h, L["f"], f32=True)
+        return self._scan(hy.SCAN_HGRN2, i, s, L, qv, None, qv.col(s.heads * s.dim), g, L["lower"], L["f_b"], None, b)
+
+    def _mix_wkv(self, i, s, L, x, h, b: Ragged) -> Out:
+        M, n = b.M, L["rkvg"].shape[1]
+        mixes = self._heads_buf("mix", len(SHIFT_MIXES), b, self.dp)
+        hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
+                          self.cfg.hidden_size, self.cfg.norm_eps)
+        y = torch.empty((M, 4 * n), dtype=self.dtype, device=self.device)
+        hy.gemm_batched(mixes[:4], L["rkvg"], y, M, c_batch=n)
+        rp = L["w1"].shape[0]
+        z = self._mm(mixes[4, :M], L["w1"], f32=True)
+        t = torch.empty((M, L["w2"].shape[1]), dtype=self.dtype, device=self.device)
+        g = self._mm(hy.split_tanh(z, s.decay_rank, rp, t), L["w2"], f32=True)
+        y = as_out(y)
+        return self._scan(hy.SCAN_WKV, i, s, L, y, y.col(n), y.col(2 * n), g, L["u"], L["w0"], y.col(3 * n), b)
+
+    # -- the shared loops' hooks ------------------------------------------------------------------------------
+    def _prompt_forward(self, seqs: list[SeqView], write_kv: bool = True):
+        b, ranges = self._pack(seqs)
+        return self._forward(b)[0], ranges
+
+    def layer_outputs(self, seqs: list[SeqView]) -> list[torch.Tensor]:
+        """Residual stream after every layer for the sequences' new tokens (rows in batch order); advances their state."""
+        out: list[torch.Tensor] = []
+        self._forward(self._pack(seqs)[0], capture=out)
+        return out
+
+    def _hidden_rows(self, x, rows):
+        h = torch.empty((rows.numel(), self.dp), dtype=self.dtype, device=self.device)
+        return hy.gather_norm(x, rows, self.final_norm, h, self.cfg.hidden_size, self.cfg.norm_eps)
+
+    def score_view(self, view: SeqView, n_prompt: int) -> list[float]:
+        """Log-probabilities of ``view.tokens[n_prompt:]``; the view's blocks and state slot are used as scratch."""
+        x, _ = self._prompt_forward([view])
+        rows = torch.arange(n_prompt - 1, len(view.tokens) - 1, dtype=torch.int64, device=self.device)
+        tgt = torch.tensor(view.tokens[n_prompt:], dtype=torch.int32, device=self.device)
+        h = self._hidden_rows(x, rows)
+        if self.exact32:
+            lp = torch.log_softmax(self._logits(h), -1)
+            return lp.gather(-1, tgt.long().unsqueeze(-1)).squeeze(-1).tolist()
+        from ..ops import logprob_loss as lpl
+
+        return lpl.grpo_tokens(lpl.partials(h, self.lm_head, tgt)[0]).logprobs.tolist()
+
+    def _decode_buffers(self, nb: int) -> dict:
+        dev = self.device
+        return {"row_seq": torch.arange(nb, dtype=torch.int32, device=dev), "cu_q": torch.arange(nb + 1, dtype=torch.int32, device=dev),
+                "state_slot": torch.full((nb,), -1, dtype=torch.int32, device=dev)}
+
+    def _stage_sequences(self, st, seqs, nb: int) -> None:
+        st["state_slot"].copy_(torch.tensor([s.state_slot for s in seqs] + [-1] * (nb - len(seqs)), dtype=torch.int32), non_blocking=True)
+
+    def _attn_splits(self, nb: int, max_ctx: int) -> int:
+        return 1
+
+    def _decode_steps(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool, procs) -> None:
+        from ..ops import paged
+
+        nb = st["tokens"].shape[0]
+        b = Ragged(nb, nb, st["tokens"], st["pos"], st["slot"], st["row_seq"], st["cu_q"], st["ctx"], st["state_slot"], st["bt"], True)
+        for k in range(n_steps):
+            _, hidden = self._forward(b, want_hidden=True)
+            t, lp = self._sample(hidden, st["inv_t"], st["seeds"][k], restricted, st["top_k"], st["top_p"], st["min_p"], procs=procs)
+            st["out_t"][k].copy_(t)
+            st["out_l"][k].copy_(lp)
+            if k + 1 < n_steps:
+                paged.decode_advance(t, st["tokens"], st["pos"], st["ctx"], st["slot"], st["bt"], self.kv.shape[1], st["active"])

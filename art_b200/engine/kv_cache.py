@@ -246,3 +246,108 @@ class KVCache:
         self.k = [k.to(self.device, non_blocking=True) for k, _ in self._host]
         self.v = [v.to(self.device, non_blocking=True) for _, v in self._host]
         self._host = None
+
+
+class StateSlots:
+    """Rows of the recurrent-state buffers: one per admitted sequence, given back when it ends or is preempted.  A row
+    need not be cleared: a portion that starts a sequence ignores what its slot holds."""
+
+    def __init__(self, n: int):
+        self.n = n
+        self._free = list(range(n - 1, -1, -1))
+
+    @property
+    def num_free(self) -> int:
+        return len(self._free)
+
+    def alloc(self) -> int | None:
+        return self._free.pop() if self._free else None
+
+    def free(self, slot: int) -> None:
+        if not 0 <= slot < self.n or slot in self._free:
+            raise ValueError(f"state slot {slot} is not in use")
+        self._free.append(slot)
+
+
+class HybridCache:
+    """Per-layer sequence memory of a hybrid decoder (``models/hybrid.py``), behind the interface of :class:`KVCache`.
+
+    ``layers[i]`` is a dict of tensors by mixer type:
+
+    * latent attention: ``latent`` ``[num_blocks, block_size, rank_p + rot_p]``, paged, in the operand dtype; a row is the
+      normed latent and the rotated key part, each padded with zeros to a multiple of 16;
+    * recurrent mixers: ``state`` fp32 ``[num_slots, heads, vdim, dim padded to 4]`` (a value column's channels are
+      contiguous), and for token-shift mixers ``shift`` fp32 ``[num_slots, width padded to 8]``, the last token's input.
+
+    ``state_slots`` hands out the slots; ``None`` for a model without recurrent layers.
+    """
+
+    arena = None
+
+    def __init__(self, cfg, num_blocks: int, block_size: int, num_slots: int, device: torch.device,
+                 dtype: torch.dtype = torch.bfloat16):
+        self.cfg, self.device, self.dtype = cfg, torch.device(device), dtype
+        self.shape = (num_blocks, block_size)
+        self.num_slots, self.num_layers = num_slots, cfg.num_layers
+        self.state_slots = StateSlots(num_slots) if cfg.recurrent else None
+        self.layers: list[dict[str, torch.Tensor]] = []
+        self._host: list[dict[str, torch.Tensor]] | None = None
+        self._allocate()
+
+    @staticmethod
+    def layer_shapes(cfg, spec, num_blocks: int, block_size: int, num_slots: int, dtype) -> dict[str, tuple[tuple[int, ...], torch.dtype]]:
+        up = lambda n, m: (n + m - 1) // m * m      # noqa: E731
+        if spec.type == "latent_attention":
+            return {"latent": ((num_blocks, block_size, up(spec.kv_rank, 16) + up(spec.rot_dim, 16)), dtype)}
+        out = {"state": ((num_slots, spec.heads, spec.vdim, up(spec.dim, 4)), torch.float32)}
+        if spec.type == "wkv":
+            out["shift"] = ((num_slots, up(cfg.hidden_size, 8)), torch.float32)
+        return out
+
+    @classmethod
+    def bytes_per_block(cls, cfg, block_size: int, elem: int = 2) -> int:
+        return sum(block_size * shape[2] * elem for s in cfg.layers if not s.recurrent
+                   for shape, _ in cls.layer_shapes(cfg, s, 1, block_size, 1, None).values())
+
+    @classmethod
+    def bytes_per_slot(cls, cfg) -> int:
+        n = 0
+        for s in cfg.layers:
+            if s.recurrent:
+                for shape, _ in cls.layer_shapes(cfg, s, 1, 1, 1, None).values():
+                    k = 4
+                    for d in shape:
+                        k *= d
+                    n += k
+        return n
+
+    def _allocate(self) -> None:
+        nb, bs = self.shape
+        self.layers = [{k: torch.zeros(shape, dtype=dt, device=self.device)
+                        for k, (shape, dt) in self.layer_shapes(self.cfg, s, nb, bs, self.num_slots, self.dtype).items()}
+                       for s in self.cfg.layers]
+
+    @property
+    def resident(self) -> bool:
+        return bool(self.layers)
+
+    def discard(self) -> None:
+        self.layers, self._host = [], None
+        if self.device.type == "cuda":
+            torch.cuda.empty_cache()
+
+    def offload(self) -> None:
+        pin = self.device.type == "cuda"
+        self._host = [{k: t.to("cpu").pin_memory() if pin else t.clone() for k, t in L.items()} for L in self.layers]
+        self.layers = []
+        if pin:
+            torch.cuda.empty_cache()
+
+    def restore(self) -> None:
+        if self.resident:
+            return
+        if self._host is None:
+            self._allocate()
+            return
+        self.layers = [{k: t.to(self.device, non_blocking=True) for k, t in L.items()} for L in self._host]
+        self._host = None

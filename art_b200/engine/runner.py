@@ -8,6 +8,7 @@
                     a batch that mixes adapters and the base model), writes K/V into the paged
                     cache, and samples with the fused LM-head sampler.  Decode runs several steps
                     back to back on the device before the host looks at the tokens.
+``DeviceRunner``    what NativeRunner shares with the runners of other model families (hybrid_runner.py).
 ``ReferenceRunner`` plain PyTorch, no KV cache (recomputes the prefix); used for CPU tests of
                     the scheduler / server / backend and as a numerical oracle.
 
@@ -79,6 +80,7 @@ class SeqView:
     min_p: float = 0.0         # keep tokens at least min_p times as likely as the most likely one (<= 0: off)
     proc: LogitProc | None = None   # penalties / logit_bias / top_logprobs: the step materialises fp32 logits
     upto: int | None = None    # chunked prefill: compute KV for tokens[num_cached:upto] only and sample nothing
+    state_slot: int = -1       # row of the recurrent-state buffers (models that carry one), -1: none
 
     @property
     def partial(self) -> bool:
@@ -187,7 +189,7 @@ class ReferenceRunner:
         return toks, lps
 
 
-# ---------------------------------------------------------------------------------- native
+# ---------------------------------------------------------------------------------- device
 # CTA-pair GEMMs at decode time: "1" = every projection, "wide" = only the unsplit (gate|up) ones, "0" = none
 _TWO_CTA_MODE = os.environ.get("ARTB_DECODE_2CTA", "1")
 TWO_CTA_DECODE = _TWO_CTA_MODE != "0"
@@ -344,7 +346,275 @@ class EngineLinear:
         return gemm_tn(T, self.B_all, residual=y_ext[:, :N], swiglu_out=swiglu_out)
 
 
-class NativeRunner:
+class DeviceRunner:
+    """What every device-side runner shares: sampling from hidden rows, prompt steps, and the multi-step decode on
+    persistent buffers with CUDA graphs.  A model family supplies
+
+    ``_prompt_forward(seqs, write_kv=True)``  residual rows of the not-yet-cached tokens and each sequence's row range
+    ``_hidden_rows(x, rows)``                 final norm of chosen rows
+    ``_decode_steps(st, ...)``                n decode steps on the staged buffers
+    ``_decode_buffers / _stage_sequences``    further per-sequence buffers of a decode batch and how they are filled
+    ``_attn_splits / _attn_workspace``        split-KV plan of the decode attention
+    """
+
+    tp, tp_group, tp_rank = 1, None, 0
+    exact32 = False            # operands are fp32 (no bf16 anywhere)
+    mixed_steps = False        # prompt portions and single decoded tokens may share one batch
+    table_width: int | None = None
+
+    def _decode_buffers(self, nb: int) -> dict:
+        return {}
+
+    def _stage_sequences(self, st, seqs, nb: int) -> None:
+        pass
+
+    def close(self) -> None:
+        """Drop the captured decode graphs and their buffers.  A tensor-parallel runner must be closed before its
+        process group is destroyed: NCCL does not finish tearing down a communicator while CUDA graphs that captured
+        its collectives are alive."""
+        self.drop_graphs()
+
+    def drop_graphs(self) -> None:
+        """Forget every captured decode graph (and its buffers); the next decode of each shape runs eagerly and is
+        captured again.  Needed whenever an address baked into the graphs changes, e.g. a KV cache that was freed and
+        re-allocated around a training step."""
+        if self.device.type == "cuda":
+            torch.cuda.synchronize(self.device)
+        if hasattr(self, "_dgraphs"):
+            self._dgraphs.clear()
+            self._dstate.clear()
+            self._dseen.clear()
+
+    def _logits(self, hidden) -> torch.Tensor:
+        """fp32 logits [M, vocab] (unit inner stride) of normed hidden rows."""
+        from ..ops.gemm import gemm_tn
+
+        local = gemm_tn(hidden, self.lm_head, out_dtype=torch.float32)          # [M, V / T]
+        if self.tp == 1:
+            return local
+        allv = torch.empty((self.tp,) + tuple(local.shape), dtype=local.dtype, device=local.device)
+        torch.distributed.all_gather_into_tensor(allv, local, group=self.tp_group)
+        return allv.permute(1, 0, 2).reshape(local.shape[0], -1).contiguous()
+
+    def _sample(self, hidden, inv_t, seeds, restricted: bool, top_k=None, top_p=None, min_p=None, procs=None):
+        """``procs``: per-row ``(LogitProc, tokens)`` or None entries; any entry sends the step through fp32 logits
+        (one GEMM), the sparse logit-edit kernel, the restricted sampler and, if asked, the top-logprobs kernel."""
+        from ..ops import paged
+
+        self._step_top = None
+        if procs is not None and any(p is not None for p in procs):
+            logits = self._logits(hidden)
+            n = len(procs)
+            paged.logit_adjust_(logits, paged.build_logit_edits([p if p is not None and p[0].edits else None for p in procs]))
+            grammars = [p[0].grammar if p is not None else None for p in procs]
+            if any(g is not None for g in grammars):
+                apply_token_mask(logits, grammars + [None] * (logits.shape[0] - len(grammars)))
+            kmax = max((p[0].top_logprobs for p in procs if p is not None), default=0)
+            if kmax > 0:
+                ti, tl = paged.top_logprobs(logits, inv_t, kmax)
+                ti, tl = ti[:n].tolist(), tl[:n].tolist()
+                self._step_top = [None if p is None or p[0].top_logprobs <= 0 else
+                                  list(zip(ti[i][:p[0].top_logprobs], tl[i][:p[0].top_logprobs])) for i, p in enumerate(procs)]
+            return paged.sample_from_logits(logits, inv_t, seeds, top_k, top_p, min_p)
+        if self.exact32:        # no fused sampler over fp32 operands: logits, then the sampling half alone
+            M = hidden.shape[0]
+            if not restricted:
+                top_k = torch.zeros(M, dtype=torch.int32, device=hidden.device)
+                top_p = torch.ones(M, dtype=torch.float32, device=hidden.device)
+            return paged.sample_from_logits(self._logits(hidden), inv_t, seeds, top_k, top_p, min_p)
+        if self.tp == 1:
+            if restricted:
+                return paged.sample_restricted(hidden, self.lm_head, inv_t, seeds, top_k, top_p, min_p)
+            return paged.sample(hidden, self.lm_head, inv_t, seeds)
+        dist = torch.distributed
+        if restricted:
+            return paged.sample_from_logits(self._logits(hidden), inv_t, seeds, top_k, top_p, min_p)
+        part = paged.sample_partials(hidden, self.lm_head, inv_t, seeds, self.vocab_offset)    # [splits, M, 8]
+        allp = torch.empty((self.tp * part.shape[0],) + tuple(part.shape[1:]), dtype=part.dtype, device=part.device)
+        dist.all_gather_into_tensor(allp, part, group=self.tp_group)
+        return paged.sample_merge(allp)
+
+    def prefill(self, seqs: list[SeqView]) -> tuple[list[int], list[float]]:
+        x, ranges = self._prompt_forward(seqs, write_kv=True)
+        if any(s.partial for s in seqs):
+            # chunks that do not reach the end of their prompt only fill the cache; sample for the others
+            done = [i for i, s in enumerate(seqs) if not s.partial]
+            toks: list = [None] * len(seqs)
+            lps: list = [None] * len(seqs)
+            self.last_top_logprobs = None
+            if done:
+                t, lp, tops = self._sample_rows(x, [ranges[i] for i in done], [seqs[i] for i in done])
+                for j, i in enumerate(done):
+                    toks[i], lps[i] = t[j], lp[j]
+                if tops is not None:
+                    full = [None] * len(seqs)
+                    for j, i in enumerate(done):
+                        full[i] = tops[j]
+                    self.last_top_logprobs = [full]
+            return toks, lps
+        t, lp, tops = self._sample_rows(x, ranges, seqs)
+        self.last_top_logprobs = [tops] if tops is not None else None
+        return t, lp
+
+    def _sample_rows(self, x, ranges, seqs):
+        """Sample the next token of every sequence from the last row of its range in ``x``."""
+        dev = self.device
+        hidden = self._hidden_rows(x, torch.tensor([r1 - 1 for _, r1 in ranges], dtype=torch.int64, device=dev))
+        inv_t = torch.tensor([0.0 if s.temperature <= 0 else 1.0 / s.temperature for s in seqs], dtype=torch.float32, device=dev)
+        seeds = torch.tensor([_mix_seed(s.seed, s.step) for s in seqs], dtype=torch.int64, device=dev).to(torch.int32)
+        procs = [(s.proc, s.tokens) if s.proc is not None else None for s in seqs]
+        if any(s.restricted or s.proc is not None for s in seqs):
+            tk = torch.tensor([s.top_k for s in seqs], dtype=torch.int32, device=dev)
+            tp = torch.tensor([s.top_p for s in seqs], dtype=torch.float32, device=dev)
+            mp = torch.tensor([s.min_p for s in seqs], dtype=torch.float32, device=dev)
+            t, lp = self._sample(hidden, inv_t, seeds, True, tk, tp, mp, procs=procs)
+        else:
+            t, lp = self._sample(hidden, inv_t, seeds, False)
+        return t.tolist(), lp.tolist(), self._step_top
+
+    def step_logits(self, seqs: list[SeqView], want: list[list[int]]) -> torch.Tensor:
+        """One batch step that samples nothing: computes ``tokens[num_cached:upto]`` of every sequence from what earlier
+        steps left in its cache and state, and returns the fp32 logits ``[sum(len(w)), vocab]`` at the places ``want[i]``
+        among sequence ``i``'s new tokens."""
+        x, ranges = self._prompt_forward(seqs)
+        rows = [r0 + j for (r0, _), w in zip(ranges, want) for j in w]
+        if not rows:
+            return torch.empty((0, self.cfg.vocab_size), dtype=torch.float32, device=self.device)
+        return self._logits(self._hidden_rows(x, torch.tensor(rows, dtype=torch.int64, device=self.device)))
+
+    # -- decode -------------------------------------------------------------------------------------
+    # The multi-step decode runs on persistent device buffers (one set per batch-size bucket) so that
+    # the whole run of n_steps x (all layers + sampler + state advance) can be captured in a CUDA
+    # graph and replayed: a decode step is ~500 small launches, which the host cannot issue as fast
+    # as the GPU retires them.  The first use of a (bucket, n_steps, lora, splits, table width) key
+    # runs eagerly, the second captures, later ones replay.
+    BUCKETS = (8, 16, 32, 64, 128, 256, 512, 1024)
+
+    def _decode_state(self, nb: int, max_blocks: int, n_steps: int):
+        key = (nb, max_blocks, n_steps)
+        st = self._dstate.get(key) if hasattr(self, "_dstate") else None
+        if st is None:
+            if not hasattr(self, "_dstate"):
+                self._dstate, self._dgraphs, self._dseen = {}, {}, set()
+            dev = self.device
+            st = {
+                "tokens": torch.zeros(nb, dtype=torch.int64, device=dev), "pos": torch.zeros(nb, dtype=torch.int32, device=dev),
+                "ctx": torch.zeros(nb, dtype=torch.int32, device=dev), "slot": torch.full((nb,), -1, dtype=torch.int32, device=dev),
+                "ad": torch.full((nb,), -1, dtype=torch.int32, device=dev), "active": torch.zeros(nb, dtype=torch.int32, device=dev),
+                "inv_t": torch.zeros(nb, dtype=torch.float32, device=dev),
+                "top_k": torch.zeros(nb, dtype=torch.int32, device=dev), "top_p": torch.ones(nb, dtype=torch.float32, device=dev),
+                "min_p": torch.zeros(nb, dtype=torch.float32, device=dev),
+                "seeds": torch.zeros((n_steps, nb), dtype=torch.int32, device=dev),
+                "bt": torch.zeros((nb, max_blocks), dtype=torch.int32, device=dev),
+                "out_t": torch.zeros((n_steps, nb), dtype=torch.int32, device=dev),
+                "out_l": torch.zeros((n_steps, nb), dtype=torch.float32, device=dev),
+            }
+            st.update(self._decode_buffers(nb))
+            self._dstate[key] = st
+        return st
+
+    def _decode_body(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool = False, procs=None):
+        from ..ops import paged
+
+        prev_pdl = paged.set_pdl(os.environ.get("ARTB_PDL", "1") != "0")
+        try:
+            self._decode_steps(st, n_steps, any_lora, splits, ws, restricted, procs)
+        finally:
+            paged.set_pdl(prev_pdl)
+
+    def decode(self, seqs: list[SeqView], n_steps: int, use_graph: bool = True) -> tuple[list[list[int]], list[list[float]]]:
+        bs = self.kv.shape[1]
+        n = len(seqs)
+        nb = next((b for b in self.BUCKETS if b >= n), (n + 255) // 256 * 256)
+        need_blocks = max(len(s.blocks) for s in seqs)
+        max_blocks = self.table_width or 64
+        while max_blocks < need_blocks:
+            max_blocks *= 2
+        st = self._decode_state(nb, max_blocks, n_steps)
+        import numpy as np
+
+        lens = [len(s.tokens) for s in seqs]
+        pad = nb - n
+        # host-side staging with numpy: one array per input instead of one small tensor per sequence
+        bt = np.zeros((nb, max_blocks), dtype=np.int32)
+        for i, s in enumerate(seqs):
+            bt[i, :len(s.blocks)] = s.blocks
+        la = np.zeros(nb, dtype=np.int64)
+        la[:n] = lens
+        last = np.zeros(nb, dtype=np.int64)
+        last[:n] = [s.tokens[-1] for s in seqs]
+        slot = np.full(nb, -1, dtype=np.int32)
+        rows = np.arange(n)
+        slot[:n] = bt[rows, (la[:n] - 1) // bs] * bs + (la[:n] - 1) % bs
+        ad = np.full(nb, -1, dtype=np.int32)
+        ad[:n] = [s.adapter for s in seqs]
+        act = np.zeros(nb, dtype=np.int32)
+        act[:n] = 1
+        inv_t = np.zeros(nb, dtype=np.float32)
+        inv_t[:n] = [0.0 if s.temperature <= 0 else 1.0 / s.temperature for s in seqs]
+        # _mix_seed(seed, step + k) for every sequence and step, in 64-bit arithmetic
+        sd = np.zeros((1, nb), dtype=np.uint64)
+        sd[0, :n] = [s.seed & 0xFFFFFFFF for s in seqs]
+        stp = np.zeros((1, nb), dtype=np.uint64)
+        stp[0, :n] = [s.step for s in seqs]
+        ks = np.arange(n_steps, dtype=np.uint64)[:, None]
+        seeds = (sd * np.uint64(0x9E3779B1) + (stp + ks) * np.uint64(0x85EBCA77) + np.uint64(0x165667B1)) & np.uint64(0xFFFFFFFF)
+        seeds[:, n:] = 0
+        st["bt"].copy_(torch.from_numpy(bt), non_blocking=True)
+        st["tokens"].copy_(torch.from_numpy(last), non_blocking=True)
+        st["pos"].copy_(torch.from_numpy((la - 1).clip(min=0).astype(np.int32)), non_blocking=True)
+        st["ctx"].copy_(torch.from_numpy(la.astype(np.int32)), non_blocking=True)
+        st["slot"].copy_(torch.from_numpy(slot), non_blocking=True)
+        st["ad"].copy_(torch.from_numpy(ad), non_blocking=True)
+        st["active"].copy_(torch.from_numpy(act), non_blocking=True)
+        st["inv_t"].copy_(torch.from_numpy(inv_t), non_blocking=True)
+        st["seeds"].copy_(torch.from_numpy(seeds.astype(np.int64)).to(torch.int32), non_blocking=True)
+        self._stage_sequences(st, seqs, nb)
+        any_lora = any(s.adapter >= 0 for s in seqs)
+        self._moe_mixed = any_lora and (pad > 0 or any(s.adapter < 0 for s in seqs))
+        procs = None
+        if any(s.proc is not None for s in seqs):
+            # logit edits depend on every token sampled so far: one step at a time, outside the captured graphs
+            if n_steps != 1:
+                raise ValueError("sequences with penalties, logit_bias or top_logprobs decode one step per call")
+            procs = [(s.proc, s.tokens) if s.proc is not None else None for s in seqs] + [None] * pad
+            use_graph = False
+        restricted = any(s.restricted for s in seqs) or procs is not None
+        if restricted:
+            st["top_k"].copy_(torch.tensor([s.top_k for s in seqs] + [0] * pad, dtype=torch.int32), non_blocking=True)
+            st["top_p"].copy_(torch.tensor([s.top_p for s in seqs] + [1.0] * pad, dtype=torch.float32), non_blocking=True)
+            st["min_p"].copy_(torch.tensor([s.min_p for s in seqs] + [0.0] * pad, dtype=torch.float32), non_blocking=True)
+        max_ctx = max(lens) + n_steps
+        splits = self._attn_splits(nb, max_ctx)
+        key = (nb, max_blocks, n_steps, any_lora, splits, restricted, self._moe_mixed)
+        ws = None
+        if splits > 1:
+            ws = st.get(("ws", splits))
+            if ws is None:
+                ws = st[("ws", splits)] = self._attn_workspace(nb, splits)
+        graph = self._dgraphs.get(key) if procs is None else None
+        self.last_top_logprobs = None
+        if procs is not None:
+            self._decode_body(st, 1, any_lora, splits, ws, True, procs=procs)
+            self.last_top_logprobs = [self._step_top] if self._step_top is not None else None
+        elif graph is not None:
+            graph.replay()
+        elif use_graph and key in self._dseen and not os.environ.get("ARTB_DECODE_NO_GRAPH"):
+            torch.cuda.synchronize()
+            graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(graph):
+                self._decode_body(st, n_steps, any_lora, splits, ws, restricted)
+            self._dgraphs[key] = graph
+            graph.replay()
+        else:
+            self._dseen.add(key)
+            self._decode_body(st, n_steps, any_lora, splits, ws, restricted)
+        out_t = st["out_t"][:, :n].tolist()
+        out_l = st["out_l"][:, :n].tolist()
+        return out_t, out_l
+
+
+class NativeRunner(DeviceRunner):
     def __init__(self, cfg: ModelConfig, lora_cfg: LoraConfig, kv, *, decoder=None, base: dict | None = None,
                  max_loras: int = 4, device="cuda", tp_group=None):
         """``decoder``: a trainer-side NativeDecoder whose frozen weights are shared; else ``base`` weights.
@@ -474,23 +744,6 @@ class NativeRunner:
         self.slot_loaded = [False] * max_loras
         self.table_width: int | None = None    # fixed block-table width (else grown by doubling, which adds graph keys)
 
-    def close(self) -> None:
-        """Drop the captured decode graphs and their buffers.  A tensor-parallel runner must be closed before its
-        process group is destroyed: NCCL does not finish tearing down a communicator while CUDA graphs that captured
-        its collectives are alive."""
-        self.drop_graphs()
-
-    def drop_graphs(self) -> None:
-        """Forget every captured decode graph (and its buffers); the next decode of each shape runs eagerly and is
-        captured again.  Needed whenever an address baked into the graphs changes, e.g. a KV cache that was freed and
-        re-allocated around a training step."""
-        if self.device.type == "cuda":
-            torch.cuda.synchronize(self.device)
-        if hasattr(self, "_dgraphs"):
-            self._dgraphs.clear()
-            self._dstate.clear()
-            self._dseen.clear()
-
     # -- tensor parallel ------------------------------------------------------------------------
     def _reduce(self, x: torch.Tensor) -> torch.Tensor:
         """Sum the row-parallel partial products over the replica (in place; a no-op on one GPU)."""
@@ -501,50 +754,6 @@ class NativeRunner:
     def _res(self, x: torch.Tensor):
         """The residual enters a row-parallel projection on one rank only: the all-reduce then adds it once."""
         return x if self.tp_rank == 0 else None
-
-    def _sample(self, hidden, inv_t, seeds, restricted: bool, top_k=None, top_p=None, min_p=None, procs=None):
-        """``procs``: per-row ``(LogitProc, tokens)`` or None entries; any entry sends the step through fp32 logits
-        (one GEMM), the sparse logit-edit kernel, the restricted sampler and, if asked, the top-logprobs kernel."""
-        from ..ops import paged
-
-        self._step_top = None
-        if procs is not None and any(p is not None for p in procs):
-            from ..ops.gemm import gemm_tn
-
-            logits = gemm_tn(hidden, self.lm_head, out_dtype=torch.float32)
-            if self.tp > 1:
-                allv = torch.empty((self.tp,) + tuple(logits.shape), dtype=logits.dtype, device=logits.device)
-                torch.distributed.all_gather_into_tensor(allv, logits, group=self.tp_group)
-                logits = allv.permute(1, 0, 2).reshape(logits.shape[0], -1).contiguous()
-            n = len(procs)
-            paged.logit_adjust_(logits, paged.build_logit_edits([p if p is not None and p[0].edits else None for p in procs]))
-            grammars = [p[0].grammar if p is not None else None for p in procs]
-            if any(g is not None for g in grammars):
-                apply_token_mask(logits, grammars + [None] * (logits.shape[0] - len(grammars)))
-            kmax = max((p[0].top_logprobs for p in procs if p is not None), default=0)
-            if kmax > 0:
-                ti, tl = paged.top_logprobs(logits, inv_t, kmax)
-                ti, tl = ti[:n].tolist(), tl[:n].tolist()
-                self._step_top = [None if p is None or p[0].top_logprobs <= 0 else
-                                  list(zip(ti[i][:p[0].top_logprobs], tl[i][:p[0].top_logprobs])) for i, p in enumerate(procs)]
-            return paged.sample_from_logits(logits, inv_t, seeds, top_k, top_p, min_p)
-        if self.tp == 1:
-            if restricted:
-                return paged.sample_restricted(hidden, self.lm_head, inv_t, seeds, top_k, top_p, min_p)
-            return paged.sample(hidden, self.lm_head, inv_t, seeds)
-        dist = torch.distributed
-        if restricted:
-            from ..ops.gemm import gemm_tn
-
-            local = gemm_tn(hidden, self.lm_head, out_dtype=torch.float32)          # [M, V / T]
-            allv = torch.empty((self.tp,) + tuple(local.shape), dtype=local.dtype, device=local.device)
-            dist.all_gather_into_tensor(allv, local, group=self.tp_group)
-            logits = allv.permute(1, 0, 2).reshape(local.shape[0], -1).contiguous()
-            return paged.sample_from_logits(logits, inv_t, seeds, top_k, top_p, min_p)
-        part = paged.sample_partials(hidden, self.lm_head, inv_t, seeds, self.vocab_offset)    # [splits, M, 8]
-        allp = torch.empty((self.tp * part.shape[0],) + tuple(part.shape[1:]), dtype=part.dtype, device=part.device)
-        dist.all_gather_into_tensor(allp, part, group=self.tp_group)
-        return paged.sample_merge(allp)
 
     # -- adapters -----------------------------------------------------------------------------
     def set_adapter(self, slot: int, state: dict[str, torch.Tensor] | None) -> None:
@@ -671,52 +880,6 @@ class NativeRunner:
             x = self._mlp(L, x2, t_ad, any_lora)
         return x, row_ranges
 
-    def prefill(self, seqs: list[SeqView]) -> tuple[list[int], list[float]]:
-        from ..ops import elementwise as ew
-        from ..ops import paged
-
-        cfg, dev = self.cfg, self.device
-        x, ranges = self._prompt_forward(seqs, write_kv=True)
-        if any(s.partial for s in seqs):
-            # chunks that do not reach the end of their prompt only fill the cache; sample for the others
-            done = [i for i, s in enumerate(seqs) if not s.partial]
-            toks: list = [None] * len(seqs)
-            lps: list = [None] * len(seqs)
-            self.last_top_logprobs = None
-            if done:
-                t, lp, tops = self._sample_rows(x, [ranges[i] for i in done], [seqs[i] for i in done])
-                for j, i in enumerate(done):
-                    toks[i], lps[i] = t[j], lp[j]
-                if tops is not None:
-                    full = [None] * len(seqs)
-                    for j, i in enumerate(done):
-                        full[i] = tops[j]
-                    self.last_top_logprobs = [full]
-            return toks, lps
-        t, lp, tops = self._sample_rows(x, ranges, seqs)
-        self.last_top_logprobs = [tops] if tops is not None else None
-        return t, lp
-
-    def _sample_rows(self, x, ranges, seqs):
-        """Sample the next token of every sequence from the last row of its range in ``x``."""
-        from ..ops import elementwise as ew
-
-        cfg, dev = self.cfg, self.device
-        t_last = torch.tensor([r1 - 1 for _, r1 in ranges], dtype=torch.int64, device=dev)
-        hl = ew.gather_rows(x, t_last)
-        hidden, _ = ew.rmsnorm_fwd(hl, self.final_norm, cfg.rms_norm_eps, want_rstd=False)
-        inv_t = torch.tensor([0.0 if s.temperature <= 0 else 1.0 / s.temperature for s in seqs], dtype=torch.float32, device=dev)
-        seeds = torch.tensor([_mix_seed(s.seed, s.step) for s in seqs], dtype=torch.int64, device=dev).to(torch.int32)
-        procs = [(s.proc, s.tokens) if s.proc is not None else None for s in seqs]
-        if any(s.restricted or s.proc is not None for s in seqs):
-            tk = torch.tensor([s.top_k for s in seqs], dtype=torch.int32, device=dev)
-            tp = torch.tensor([s.top_p for s in seqs], dtype=torch.float32, device=dev)
-            mp = torch.tensor([s.min_p for s in seqs], dtype=torch.float32, device=dev)
-            t, lp = self._sample(hidden, inv_t, seeds, True, tk, tp, mp, procs=procs)
-        else:
-            t, lp = self._sample(hidden, inv_t, seeds, False)
-        return t.tolist(), lp.tolist(), self._step_top
-
     def score(self, tokens: list[int], n_prompt: int, adapter: int) -> list[float]:
         """Log-probabilities of ``tokens[n_prompt:]`` given what precedes them (no KV is written)."""
         from ..ops import elementwise as ew
@@ -737,48 +900,6 @@ class NativeRunner:
             return lp.gather(-1, tgt.long().unsqueeze(-1)).squeeze(-1).tolist()
         part, _ = lpl.partials(h, self.lm_head, tgt)
         return lpl.grpo_tokens(part).logprobs.tolist()
-
-    # -- decode -------------------------------------------------------------------------------------
-    # The multi-step decode runs on persistent device buffers (one set per batch-size bucket) so that
-    # the whole run of n_steps x (all layers + sampler + state advance) can be captured in a CUDA
-    # graph and replayed: a decode step is ~500 small launches, which the host cannot issue as fast
-    # as the GPU retires them.  The first use of a (bucket, n_steps, lora, splits, table width) key
-    # runs eagerly, the second captures, later ones replay.
-    BUCKETS = (8, 16, 32, 64, 128, 256, 512, 1024)
-
-    def _decode_state(self, nb: int, max_blocks: int, n_steps: int):
-        key = (nb, max_blocks, n_steps)
-        st = self._dstate.get(key) if hasattr(self, "_dstate") else None
-        if st is None:
-            if not hasattr(self, "_dstate"):
-                self._dstate, self._dgraphs, self._dseen = {}, {}, set()
-            dev, cfg = self.device, self.cfg
-            st = {
-                "tokens": torch.zeros(nb, dtype=torch.int64, device=dev), "pos": torch.zeros(nb, dtype=torch.int32, device=dev),
-                "ctx": torch.zeros(nb, dtype=torch.int32, device=dev), "slot": torch.full((nb,), -1, dtype=torch.int32, device=dev),
-                "ad": torch.full((nb,), -1, dtype=torch.int32, device=dev), "active": torch.zeros(nb, dtype=torch.int32, device=dev),
-                "inv_t": torch.zeros(nb, dtype=torch.float32, device=dev),
-                "top_k": torch.zeros(nb, dtype=torch.int32, device=dev), "top_p": torch.ones(nb, dtype=torch.float32, device=dev),
-                "min_p": torch.zeros(nb, dtype=torch.float32, device=dev),
-                "seeds": torch.zeros((n_steps, nb), dtype=torch.int32, device=dev),
-                "bt": torch.zeros((nb, max_blocks), dtype=torch.int32, device=dev),
-                "out_t": torch.zeros((n_steps, nb), dtype=torch.int32, device=dev),
-                "out_l": torch.zeros((n_steps, nb), dtype=torch.float32, device=dev),
-                "attn_out": torch.zeros((nb, cfg.q_size), dtype=torch.bfloat16, device=dev),
-                "q": torch.zeros((nb, cfg.q_size), dtype=torch.bfloat16, device=dev),
-            }
-            self._dstate[key] = st
-        return st
-
-    def _decode_body(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool = False, procs=None):
-        from ..ops import elementwise as ew
-        from ..ops import paged
-
-        prev_pdl = paged.set_pdl(os.environ.get("ARTB_PDL", "1") != "0")
-        try:
-            self._decode_steps(st, n_steps, any_lora, splits, ws, restricted, procs)
-        finally:
-            paged.set_pdl(prev_pdl)
 
     def _decode_steps(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool, procs) -> None:
         from ..ops import elementwise as ew
@@ -851,92 +972,19 @@ class NativeRunner:
                                    eps=cfg.rms_norm_eps, h_out=h3)
         return x3, h3
 
-    def decode(self, seqs: list[SeqView], n_steps: int, use_graph: bool = True) -> tuple[list[list[int]], list[list[float]]]:
-        cfg, dev, bs = self.cfg, self.device, self.kv.shape[1]
-        n = len(seqs)
-        nb = next((b for b in self.BUCKETS if b >= n), (n + 255) // 256 * 256)
-        need_blocks = max(len(s.blocks) for s in seqs)
-        max_blocks = self.table_width or 64
-        while max_blocks < need_blocks:
-            max_blocks *= 2
-        st = self._decode_state(nb, max_blocks, n_steps)
-        import numpy as np
+    # -- hooks of the shared decode loop ----------------------------------------------------------
+    def _hidden_rows(self, x, rows):
+        from ..ops import elementwise as ew
 
-        lens = [len(s.tokens) for s in seqs]
-        pad = nb - n
-        # host-side staging with numpy: one array per input instead of one small tensor per sequence
-        bt = np.zeros((nb, max_blocks), dtype=np.int32)
-        for i, s in enumerate(seqs):
-            bt[i, :len(s.blocks)] = s.blocks
-        la = np.zeros(nb, dtype=np.int64)
-        la[:n] = lens
-        last = np.zeros(nb, dtype=np.int64)
-        last[:n] = [s.tokens[-1] for s in seqs]
-        slot = np.full(nb, -1, dtype=np.int32)
-        rows = np.arange(n)
-        slot[:n] = bt[rows, (la[:n] - 1) // bs] * bs + (la[:n] - 1) % bs
-        ad = np.full(nb, -1, dtype=np.int32)
-        ad[:n] = [s.adapter for s in seqs]
-        act = np.zeros(nb, dtype=np.int32)
-        act[:n] = 1
-        inv_t = np.zeros(nb, dtype=np.float32)
-        inv_t[:n] = [0.0 if s.temperature <= 0 else 1.0 / s.temperature for s in seqs]
-        # _mix_seed(seed, step + k) for every sequence and step, in 64-bit arithmetic
-        sd = np.zeros((1, nb), dtype=np.uint64)
-        sd[0, :n] = [s.seed & 0xFFFFFFFF for s in seqs]
-        stp = np.zeros((1, nb), dtype=np.uint64)
-        stp[0, :n] = [s.step for s in seqs]
-        ks = np.arange(n_steps, dtype=np.uint64)[:, None]
-        seeds = (sd * np.uint64(0x9E3779B1) + (stp + ks) * np.uint64(0x85EBCA77) + np.uint64(0x165667B1)) & np.uint64(0xFFFFFFFF)
-        seeds[:, n:] = 0
-        st["bt"].copy_(torch.from_numpy(bt), non_blocking=True)
-        st["tokens"].copy_(torch.from_numpy(last), non_blocking=True)
-        st["pos"].copy_(torch.from_numpy((la - 1).clip(min=0).astype(np.int32)), non_blocking=True)
-        st["ctx"].copy_(torch.from_numpy(la.astype(np.int32)), non_blocking=True)
-        st["slot"].copy_(torch.from_numpy(slot), non_blocking=True)
-        st["ad"].copy_(torch.from_numpy(ad), non_blocking=True)
-        st["active"].copy_(torch.from_numpy(act), non_blocking=True)
-        st["inv_t"].copy_(torch.from_numpy(inv_t), non_blocking=True)
-        st["seeds"].copy_(torch.from_numpy(seeds.astype(np.int64)).to(torch.int32), non_blocking=True)
-        any_lora = any(s.adapter >= 0 for s in seqs)
-        self._moe_mixed = any_lora and (pad > 0 or any(s.adapter < 0 for s in seqs))
-        procs = None
-        if any(s.proc is not None for s in seqs):
-            # logit edits depend on every token sampled so far: one step at a time, outside the captured graphs
-            if n_steps != 1:
-                raise ValueError("sequences with penalties, logit_bias or top_logprobs decode one step per call")
-            procs = [(s.proc, s.tokens) if s.proc is not None else None for s in seqs] + [None] * pad
-            use_graph = False
-        restricted = any(s.restricted for s in seqs) or procs is not None
-        if restricted:
-            st["top_k"].copy_(torch.tensor([s.top_k for s in seqs] + [0] * pad, dtype=torch.int32), non_blocking=True)
-            st["top_p"].copy_(torch.tensor([s.top_p for s in seqs] + [1.0] * pad, dtype=torch.float32), non_blocking=True)
-            st["min_p"].copy_(torch.tensor([s.min_p for s in seqs] + [0.0] * pad, dtype=torch.float32), non_blocking=True)
-        max_ctx = max(lens) + n_steps
-        splits = 1 if nb * cfg.num_kv_heads >= 128 else min(8, max(1, 1 << (max(1, max_ctx // 512).bit_length() - 1)))
-        key = (nb, max_blocks, n_steps, any_lora, splits, restricted, self._moe_mixed)
-        ws = None
-        if splits > 1:
-            ws = st.get(("ws", splits))
-            if ws is None:
-                ws = st[("ws", splits)] = torch.empty(nb * cfg.num_heads * splits * (cfg.head_dim + 2), dtype=torch.float32, device=dev)
-        graph = self._dgraphs.get(key) if procs is None else None
-        self.last_top_logprobs = None
-        if procs is not None:
-            self._decode_body(st, 1, any_lora, splits, ws, True, procs=procs)
-            self.last_top_logprobs = [self._step_top] if self._step_top is not None else None
-        elif graph is not None:
-            graph.replay()
-        elif use_graph and key in self._dseen and not os.environ.get("ARTB_DECODE_NO_GRAPH"):
-            torch.cuda.synchronize()
-            graph = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(graph):
-                self._decode_body(st, n_steps, any_lora, splits, ws, restricted)
-            self._dgraphs[key] = graph
-            graph.replay()
-        else:
-            self._dseen.add(key)
-            self._decode_body(st, n_steps, any_lora, splits, ws, restricted)
-        out_t = st["out_t"][:, :n].tolist()
-        out_l = st["out_l"][:, :n].tolist()
-        return out_t, out_l
+        return ew.rmsnorm_fwd(ew.gather_rows(x, rows), self.final_norm, self.cfg.rms_norm_eps, want_rstd=False)[0]
+
+    def _decode_buffers(self, nb: int) -> dict:
+        cfg = self.cfg
+        return {"attn_out": torch.zeros((nb, cfg.q_size), dtype=torch.bfloat16, device=self.device),
+                "q": torch.zeros((nb, cfg.q_size), dtype=torch.bfloat16, device=self.device)}
+
+    def _attn_splits(self, nb: int, max_ctx: int) -> int:
+        return 1 if nb * self.cfg.num_kv_heads >= 128 else min(8, max(1, 1 << (max(1, max_ctx // 512).bit_length() - 1)))
+
+    def _attn_workspace(self, nb: int, splits: int) -> torch.Tensor:
+        return torch.empty(nb * self.cfg.num_heads * splits * (self.cfg.head_dim + 2), dtype=torch.float32, device=self.device)

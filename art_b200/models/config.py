@@ -4,12 +4,17 @@ Dense Qwen2 / Qwen2.5 / Llama-style decoders (RMSNorm, RoPE, GQA, SwiGLU, option
 bias) and Qwen3-MoE-style sparse decoders (per-head q/k RMSNorm, softmax top-k router,
 SwiGLU experts).  ``ModelConfig.from_hf_dict`` reads a Hugging Face ``config.json``;
 ``PRESETS`` holds the shapes used by the benchmarks, instantiated with random weights.
+Designs of this package's own (hybrid decoders) are described in ``models/hybrid.py`` and
+reached through the same entry points.
 """
 from __future__ import annotations
 
+import copy
 import json
 import os
 from dataclasses import asdict, dataclass, field
+
+from .hybrid import ARCHITECTURES, HYBRID_PRESETS, HybridConfig
 
 
 @dataclass
@@ -187,9 +192,12 @@ class ModelConfig:
         )
 
     @classmethod
-    def from_pretrained_dir(cls, path: str) -> "ModelConfig":
+    def from_pretrained_dir(cls, path: str) -> "ModelConfig | HybridConfig":
+        """Reads ``config.json``: an ``architecture`` key names one of this package's own designs (``models/hybrid.py``),
+        anything else is a Hugging Face configuration."""
         with open(os.path.join(path, "config.json")) as f:
-            return cls.from_hf_dict(json.load(f), name=os.path.basename(path.rstrip("/")))
+            d = json.load(f)
+        return config_from_dict(d, name=os.path.basename(path.rstrip("/")))
 
 
 PRESETS: dict[str, ModelConfig] = {
@@ -232,13 +240,25 @@ PRESETS: dict[str, ModelConfig] = {
 }
 
 
-def resolve_config(base_model: str, architecture: dict | None = None) -> ModelConfig:
+def config_from_dict(d: dict, name: str = "hf") -> "ModelConfig | HybridConfig":
+    """The configuration class a ``config.json`` asks for."""
+    if "architecture" in d:
+        make = ARCHITECTURES.get(d["architecture"])
+        if make is None:
+            raise ValueError(f"architecture {d['architecture']!r} is not supported (supported: {', '.join(ARCHITECTURES)})")
+        return make(d, name)
+    return ModelConfig.from_hf_dict(d, name)
+
+
+def resolve_config(base_model: str, architecture: dict | None = None) -> "ModelConfig | HybridConfig":
     """``architecture`` dict > local directory with config.json > preset by (fuzzy) name."""
     if architecture:
-        return ModelConfig(**architecture)
+        return config_from_dict(architecture, base_model) if "architecture" in architecture else ModelConfig(**architecture)
     if os.path.isdir(base_model) and os.path.exists(os.path.join(base_model, "config.json")):
         return ModelConfig.from_pretrained_dir(base_model)
     key = base_model.lower().removeprefix("random:").split("/")[-1].replace("-instruct", "")
+    if key in HYBRID_PRESETS:
+        return copy.deepcopy(HYBRID_PRESETS[key])
     if key in PRESETS:
         return PRESETS[key]
     for name, cfg in PRESETS.items():

@@ -15,6 +15,7 @@ from dataclasses import dataclass, field
 import torch
 
 from .config import ModelConfig
+from .hybrid import HybridConfig, check_weights, init_hybrid_weights
 
 ATTN_TARGETS = ("q_proj", "k_proj", "v_proj", "o_proj")
 MLP_TARGETS = ("gate_proj", "up_proj", "down_proj")
@@ -48,6 +49,8 @@ def init_base_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torc
     with ``std / sqrt(2 * num_layers)``, the usual depth-scaled initialisation.  Without it the residual of a deep
     random model is dominated by a component common to all tokens, and a random router then sends almost every
     token to the same few experts, which no trained mixture-of-experts model does."""
+    if isinstance(cfg, HybridConfig):
+        return init_hybrid_weights(cfg, seed=seed, dtype=dtype, device=device)
     g = torch.Generator(device=device).manual_seed(seed)
     out_scale = (2 * cfg.num_layers) ** -0.5 if scale_residual_out else 1.0
 
@@ -77,7 +80,7 @@ def init_base_weights(cfg: ModelConfig, seed: int = 0, dtype: torch.dtype = torc
 
 def load_base_weights(path: str, cfg: ModelConfig, dtype: torch.dtype = torch.bfloat16,
                       device: str | torch.device = "cpu") -> dict[str, torch.Tensor]:
-    """Read every ``*.safetensors`` shard in ``path`` (HF layout)."""
+    """Read every ``*.safetensors`` shard in ``path`` (HF layout, or the tensor names of a hybrid design)."""
     from safetensors import safe_open
 
     w: dict[str, torch.Tensor] = {}
@@ -87,7 +90,11 @@ def load_base_weights(path: str, cfg: ModelConfig, dtype: torch.dtype = torch.bf
     for fpath in files:
         with safe_open(fpath, framework="pt", device=str(device)) as f:
             for k in f.keys():
-                w[k] = f.get_tensor(k).to(dtype)
+                t = f.get_tensor(k)
+                w[k] = t.to(dtype) if t.is_floating_point() else t
+    if isinstance(cfg, HybridConfig):
+        check_weights(cfg, w)
+        return w
     if "lm_head.weight" not in w:
         w["lm_head.weight"] = w["model.embed_tokens.weight"]
     return w

@@ -1,0 +1,205 @@
+"""Front-ends of the hybrid decoder's kernels (``csrc/kernels/hybrid_rows.cu``, ``linear_scan.cu``, ``latent_attn*.cu``,
+``gemm_batched.cu``, ``gemm_f32.cu``).
+
+GEMM operands are bf16, or fp32 in the 32-bit mode; the residual stream, norms, gates and states are fp32 in both.  A
+projection's output reaches its consumer as bf16, as fp32, or as the fp32 workspace of a split-K GEMM that the consumer
+leaves zero: ``Out`` carries the tensor together with that kind.
+"""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+
+import torch
+
+from . import _lib
+
+vp, ci, cl, cf = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
+SCAN_HGRN2, SCAN_WKV = 0, 1
+KIND_BF16, KIND_F32, KIND_TAKE = 0, 1, 2
+_sigs = {
+    "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, cl, ci, vp, vp, vp, ci, ci, ci, ci, cf, vp, vp],
+    "artb_norm_shift_mix": [ci, vp, ci, vp, vp, ci, vp, cl, ci, vp, cl, vp, vp, vp, vp, ci, ci, ci, cf, vp, vp],
+    "artb_poly_norm": [ci, vp, ci, ci, vp, vp, ci, ci, ci, ci, cf, vp],
+    "artb_split_tanh": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
+    "artb_head_norm": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, cf, vp],
+    "artb_gather_norm": [ci, vp, ci, vp, ci, vp, vp, ci, ci, ci, cf, cl, vp, vp],
+    "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, vp, vp],
+    "artb_linear_decode": [ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci,
+                           vp, ci, ci, vp, ci, ci, cf, vp, vp],
+    "artb_latent_finish": [ci, vp, ci, ci, vp, vp, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
+                           vp],
+    "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
+    "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gemm_f32_tn": [vp, ci, cl, vp, ci, cl, vp, ci, cl, ci, ci, ci, ci, vp],
+}
+_bound: dict[str, object] = {}
+
+
+def _f(name: str):
+    fn = _bound.get(name)
+    if fn is None:
+        fn = getattr(_lib.kernels(), name)
+        fn.argtypes, fn.restype = _sigs[name], ci
+        _bound[name] = fn
+    return fn
+
+
+def pad(n: int, m: int = 8) -> int:
+    return (n + m - 1) // m * m
+
+
+@dataclass
+class Out:
+    """A projection's output as its consumer finds it: ``t`` [M, N] with unit inner stride and its kind."""
+    t: torch.Tensor
+    kind: int
+
+    def col(self, c: int) -> "Out":
+        return Out(self.t[:, c:], self.kind)
+
+
+def as_out(t: torch.Tensor) -> Out:
+    return Out(t, KIND_BF16 if t.dtype == torch.bfloat16 else KIND_F32)
+
+
+def _is32(t: torch.Tensor) -> int:
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def _st(t: torch.Tensor):
+    return _lib.ptr(_lib.status_word(t.device))
+
+
+def residual_step(x_out: torch.Tensor, w_post: torch.Tensor, d: int, eps: float, *, y: Out | None = None, x_in=None,
+                  mult: float = 1.0, tokens=None, table=None, hist=None, hist_n: int = 0, avg=None, w_next=None, h=None) -> None:
+    """One sublayer boundary of the fp32 residual stream ``[M, dp]``; ``y`` is the sublayer's output, or ``tokens`` /
+    ``table`` the embedding.  ``hist`` fp32 ``[layers + 1, M, dp]``: the result is stored at ``hist_n`` and, with ``avg``,
+    replaced by the weighted average of entries ``0 .. hist_n``.  ``w_next`` / ``h``: the next sublayer's input norm."""
+    M, dp = x_out.shape
+    f32 = _is32(table if table is not None else h) if (table is not None or h is not None) else 0
+    _lib.check_rc(_f("artb_residual_step")(
+        f32, _lib.ptr(tokens), _lib.ptr(table), table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0,
+        _lib.ptr(y.t if y is not None else None), y.t.stride(0) if y is not None else 0, y.kind if y is not None else 0,
+        _lib.ptr(x_in), _lib.ptr(x_out), x_out.stride(0), _lib.ptr(w_post), mult, _lib.ptr(hist),
+        hist.stride(0) if hist is not None else 0, hist_n, _lib.ptr(avg), _lib.ptr(w_next), _lib.ptr(h),
+        h.stride(0) if h is not None else 0, M, d, dp, eps, _st(x_out), _lib.stream_ptr()), "residual_step")
+
+
+def norm_shift_mix(x, w, mu, out, state, row_seq, cu_q, ctx, state_slot, d: int, eps: float) -> None:
+    """``out[s, m] = h + (h' - h) mu[s]`` with ``h`` the normed row and ``h'`` that of the token before it; ``out`` is
+    ``[n_mix, pitch, dp]``, ``state`` fp32 ``[slots, dp]``."""
+    M, dp = x.shape
+    _lib.check_rc(_f("artb_norm_shift_mix")(
+        _is32(out), _lib.ptr(x), x.stride(0), _lib.ptr(w), _lib.ptr(mu), mu.shape[0], _lib.ptr(out), out.stride(0), out.stride(1),
+        _lib.ptr(state), state.shape[0], _lib.ptr(row_seq), _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), M, d, dp, eps,
+        _st(x), _lib.stream_ptr()), "norm_shift_mix")
+
+
+def poly_norm(z: Out, act, out, n: int, eps: float) -> torch.Tensor:
+    _lib.check_rc(_f("artb_poly_norm")(_is32(out), _lib.ptr(z.t), z.t.stride(0), z.kind, _lib.ptr(act), _lib.ptr(out), out.stride(0),
+                                       out.shape[0], n, out.shape[1], eps, _lib.stream_ptr()), "poly_norm")
+    return out
+
+
+def split_tanh(z: Out, r: int, rp: int, out) -> torch.Tensor:
+    """bf16 ``[M, 2 rp]``: tanh of the first ``r`` columns as a pair of bf16 values; fp32 ``[M, rp]``: tanh."""
+    _lib.check_rc(_f("artb_split_tanh")(_is32(out), _lib.ptr(z.t), z.t.stride(0), z.kind, _lib.ptr(out), out.stride(0), out.shape[0],
+                                        r, rp, _lib.stream_ptr()), "split_tanh")
+    return out
+
+
+def head_norm(o, w, w_per_head: bool, H: int, vdim: int, vpad: int, out, eps: float, gate: Out | None = None) -> torch.Tensor:
+    """Per-head RMSNorm of ``o`` fp32 [M, H * vdim]; ``w`` [vdim], or [H * vdim] with ``w_per_head``; silu ``gate``."""
+    _lib.check_rc(_f("artb_head_norm")(
+        _is32(out), _lib.ptr(o), o.stride(0), _lib.ptr(w), 1 if w_per_head else 0,
+        _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0, _lib.ptr(out), out.stride(0),
+        out.shape[0], H, vdim, vpad, eps, _lib.stream_ptr()), "head_norm")
+    return out
+
+
+def gather_norm(x, rows, w, h, d: int, eps: float) -> torch.Tensor:
+    _lib.check_rc(_f("artb_gather_norm")(_is32(h), _lib.ptr(x), x.stride(0), _lib.ptr(rows), rows.numel(), _lib.ptr(w), _lib.ptr(h),
+                                         h.stride(0), d, x.shape[1], eps, x.shape[0], _st(x), _lib.stream_ptr()), "gather_norm")
+    return h
+
+
+def _scan_in(mode, q: Out, k: Out | None, v: Out, g: Out):
+    if q.kind != v.kind or (k is not None and k.kind != q.kind):
+        raise ValueError("q, k and v come from one projection and share their kind")
+    return (_lib.ptr(q.t), q.t.stride(0), _lib.ptr(k.t if k else None), k.t.stride(0) if k else 0, _lib.ptr(v.t), v.t.stride(0), q.kind,
+            _lib.ptr(g.t), g.t.stride(0), g.kind)
+
+
+def linear_scan(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, state, cu_q, ctx, state_slot, n_seqs: int, H: int,
+                dim: int, vdim: int, o) -> torch.Tensor:
+    """Portions of ``n_seqs`` sequences through the recurrence; ``state`` fp32 ``[slots, H, vdim, ld]``; ``o`` fp32."""
+    _lib.check_rc(_f("artb_linear_scan")(
+        mode, *_scan_in(mode, q, k, v, g), _lib.ptr(bias), _lib.ptr(aux), _lib.ptr(state), state.stride(0), state.shape[3],
+        state.shape[0], _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, H, dim, vdim, _lib.ptr(o), o.stride(0), _st(o),
+        _lib.stream_ptr()), "linear_scan")
+    return o
+
+
+def linear_decode(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, state, cu_q, ctx, state_slot, H: int, dim: int,
+                  vdim: int, w, w_per_head: bool, gate: Out | None, out, vpad: int, eps: float) -> torch.Tensor:
+    """One token of each sequence (row m = sequence m): recurrence, per-head norm, optional gate."""
+    M = out.shape[0]
+    _lib.check_rc(_f("artb_linear_decode")(
+        _is32(out), mode, *_scan_in(mode, q, k, v, g), _lib.ptr(bias), _lib.ptr(aux), _lib.ptr(state), state.stride(0),
+        state.shape[3], state.shape[0], _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), M, H, dim, vdim, _lib.ptr(w),
+        1 if w_per_head else 0, _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0,
+        _lib.ptr(out), out.stride(0), vpad, eps, _st(out), _lib.stream_ptr()), "linear_decode")
+    return out
+
+
+def latent_finish(p: Out, w, inv_freq, pos, slot, cache, n_abs: int, qn, qr, qe, H: int, dim: int, rot: int, rank: int,
+                  eps: float) -> None:
+    """Norm, rotation and cache write behind the q | latent projection.  Rows below ``n_abs`` leave their queries in
+    ``qn`` [H, pitch, dim_p] / ``qr`` [H, pitch, rot_p], the others in ``qe`` [M - n_abs, H * (dim + rot)]."""
+    M = pos.numel()
+    rank_p, rot_p = pad(rank, 16), pad(rot, 16)
+    _lib.check_rc(_f("artb_latent_finish")(
+        _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(w), _lib.ptr(inv_freq), _lib.ptr(pos), _lib.ptr(slot),
+        _lib.ptr(cache), cache.shape[-1], cache.shape[0] * cache.shape[1], n_abs, _lib.ptr(qn), _lib.ptr(qr),
+        qn.shape[1] if qn is not None else 0, _lib.ptr(qe), qe.stride(0) if qe is not None else 0, M, H, dim,
+        qn.shape[2] if qn is not None else dim, rot, rot_p, rank, rank_p, eps, _st(cache), _lib.stream_ptr()), "latent_finish")
+
+
+def latent_attend(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int) -> torch.Tensor:
+    """Windowed attention in latent space over the paged cache, scalar fp32 form; everything head-major [H, pitch, .]."""
+    H, pitch, rank_p = ql.shape
+    _lib.check_rc(_f("artb_latent_attend")(
+        _is32(cache), _lib.ptr(ql), _lib.ptr(qr), pitch, _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table),
+        block_table.stride(0), cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale,
+        _lib.ptr(o), M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_attend")
+    return o
+
+
+def gemm_batched(a, b, out, M: int, *, c_batch: int) -> torch.Tensor:
+    """``out_b[m, n] = a[b, m, :] . b[b, n, :]``; ``a`` [batch, pitch, K], ``b`` [batch, N, K]; ``out`` is a 2-D tensor whose
+    storage receives member ``b`` from element ``b * c_batch`` on (leading dimension ``out.stride(0)``)."""
+    batch, pitch, K = a.shape
+    N = b.shape[1]
+    if a.dtype == torch.float32:
+        _lib.check_rc(_f("artb_gemm_f32_tn")(_lib.ptr(a), a.stride(1), a.stride(0), _lib.ptr(b), b.stride(1), b.stride(0), _lib.ptr(out),
+                                             out.stride(0), c_batch, batch, M, N, K, _lib.stream_ptr()), "gemm_f32")
+        return out
+    if not (a.is_contiguous() and b.is_contiguous()):
+        raise ValueError("batched operands must be contiguous")
+    _lib.check_rc(_f("artb_gemm_batched_bf16_tn")(_lib.ptr(a), a.stride(1), pitch, _lib.ptr(b), b.stride(1), _lib.ptr(out), out.stride(0),
+                                                  c_batch, _is32(out), batch, M, N, K, _st(a), _lib.stream_ptr()), "gemm_batched")
+    return out
+
+
+def gemm_f32(a, b, out=None) -> torch.Tensor:
+    """``out[M, N] = a[M, K] @ b[N, K].T`` in fp32 multiply-adds (no reduced-precision mode)."""
+    if a.dtype != torch.float32 or b.dtype != torch.float32 or a.stride(1) != 1 or b.stride(1) != 1:
+        raise ValueError("gemm_f32: fp32 operands with unit inner stride")
+    M, K = a.shape
+    N = b.shape[0]
+    if out is None:
+        out = torch.empty((M, N), dtype=torch.float32, device=a.device)
+    _lib.check_rc(_f("artb_gemm_f32_tn")(_lib.ptr(a), a.stride(0), 0, _lib.ptr(b), b.stride(0), 0, _lib.ptr(out), out.stride(0), 0, 1, M, N,
+                                         K, _lib.stream_ptr()), "gemm_f32")
+    return out
