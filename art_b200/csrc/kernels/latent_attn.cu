@@ -9,7 +9,7 @@
 //                          queries in the layout the attention form of the row reads
 //   latent_attend_kernel   attention in latent space ("absorbed" form): q~ = W_uk^T q per head is taken against the cached
 //                          latents themselves, the weighted latents are expanded by W_uv afterwards.  Scalar fp32
-//                          arithmetic for any sizes and both number formats (the 32-bit mode runs on it).
+//                          arithmetic: the 32-bit mode runs on it (bf16: latent_decode.cu, latent_prefill.cu).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -35,7 +35,7 @@ struct LatentFinish {
   void* qn;                 // T [H][pitch][dim_p]
   void* qr;                 // T [H][pitch][rot_p]
   int pitch;
-  void* qe;                 // T [M - n_abs][ldqe], heads of (dim + rot)
+  void* qe;                 // T [M - n_abs][ldqe], heads of (dim_p + rot_p), padding zero
   int ldqe;
   int H, dim, dim_p, rot, rot_p, rank, rank_p;
   float eps;
@@ -75,11 +75,20 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
     }
   }
   const bool absorbed = m < a.n_abs;
+  const int he = a.dim_p + a.rot_p;
+  T* erow = reinterpret_cast<T*>(a.qe) + static_cast<size_t>(absorbed ? 0 : m - a.n_abs) * a.ldqe;
   for (int j = tid; j < a.H * a.dim; j += blockDim.x) {
     const int h = j / a.dim, i = j - h * a.dim;
     const float x = take1(a.p, row + h * hq + i, a.kind);
     if (absorbed) st1(reinterpret_cast<T*>(a.qn) + (static_cast<size_t>(h) * a.pitch + m) * a.dim_p + i, x);
-    else st1(reinterpret_cast<T*>(a.qe) + static_cast<size_t>(m - a.n_abs) * a.ldqe + h * hq + i, x);
+    else st1(erow + h * he + i, x);
+  }
+  if (!absorbed) {
+    const int np = he - a.dim - a.rot;       // padding columns of a head: behind the first part, behind the rotated part
+    for (int j = tid; j < a.H * np; j += blockDim.x) {
+      const int h = j / np, i = j - h * np;
+      st1(erow + h * he + (i < a.dim_p - a.dim ? a.dim + i : a.dim + i + a.rot), 0.f);
+    }
   }
   for (int j = tid; j < a.H * hp; j += blockDim.x) {
     const int h = j / hp, i = j - h * hp;
@@ -87,7 +96,7 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
     const float u = take1(a.p, o, a.kind), v = take1(a.p, o + 1, a.kind);
     const float x = u * cc[i] - v * sn[i], y = v * cc[i] + u * sn[i];
     T* d = absorbed ? reinterpret_cast<T*>(a.qr) + (static_cast<size_t>(h) * a.pitch + m) * a.rot_p + 2 * i
-                    : reinterpret_cast<T*>(a.qe) + static_cast<size_t>(m - a.n_abs) * a.ldqe + h * hq + a.dim + 2 * i;
+                    : erow + h * he + a.dim_p + 2 * i;
     st1(d, x);
     st1(d + 1, y);
   }
@@ -201,7 +210,7 @@ ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const fl
                                    float eps, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   if (H <= 0 || (rot & 1) || dim_p < dim || rot_p < rot || rank_p < rank || ldc < rank_p + rot_p) return ERR_BAD_SHAPE;
-  if ((n_abs > 0 && (!qn || !qr || pitch < n_abs)) || (n_abs < M && (!qe || ldqe < H * (dim + rot)))) return ERR_BAD_SHAPE;
+  if ((n_abs > 0 && (!qn || !qr || pitch < n_abs)) || (n_abs < M && (!qe || ldqe < H * (dim_p + rot_p)))) return ERR_BAD_SHAPE;
   const LatentFinish a{p, ldp, kind, w, inv_freq, pos, slot, cache, ldc, num_slots, n_abs, qn, qr, pitch, qe, ldqe, H, dim, dim_p,
                        rot, rot_p, rank, rank_p, eps, status};
   const size_t smem = static_cast<size_t>(rot) * 4;

@@ -23,8 +23,8 @@ def measure_decode(cfg, device, seqs: int = 256, prompt_len: int = 512, new_toke
     from ..models.weights import LoraConfig, init_base_weights, init_lora
     from ..ops import _lib
     from .engine import Engine, SamplingParams
-    from .kv_cache import BlockManager, KVCache
-    from .runner import NativeRunner
+    from .factory import build_runner
+    from .kv_cache import BlockManager
 
     dev = torch.device(device)
     tp = 1 if tp_group is None else torch.distributed.get_world_size(tp_group)
@@ -34,8 +34,8 @@ def measure_decode(cfg, device, seqs: int = 256, prompt_len: int = 512, new_toke
     bs = 16
     p_hi = max(prompt_len, prompt_len_max)
     nblocks = seqs * ((p_hi + new_tokens) // bs + 2)
-    kv = KVCache(cfg.num_layers, nblocks, bs, cfg.num_kv_heads // tp, cfg.head_dim, dev)
-    runner = NativeRunner(cfg, lcfg, kv, base=base, max_loras=max(1, loras), device=dev, tp_group=tp_group)
+    runner, kv = build_runner(cfg, base, num_blocks=nblocks, block_size=bs, num_slots=seqs, device=dev, lora_cfg=lcfg,
+                              max_loras=max(1, loras), tp_group=tp_group)
     width = 64
     while width < (p_hi + new_tokens) // bs + 2:
         width *= 2
@@ -104,7 +104,7 @@ def measure_decode(cfg, device, seqs: int = 256, prompt_len: int = 512, new_toke
 
 
 def main() -> None:
-    from ..models.config import PRESETS
+    from ..models.config import resolve_config
 
     ap = argparse.ArgumentParser()
     ap.add_argument("--model", default="qwen2.5-7b")
@@ -127,7 +127,7 @@ def main() -> None:
         if dist.get_world_size() != a.tp:
             raise SystemExit("--tp must equal the number of launched ranks")
         group = dist.group.WORLD
-    res = measure_decode(PRESETS[a.model], dev, a.seqs, a.prompt_len, a.new_tokens, a.loras, a.runs, tp_group=group,
+    res = measure_decode(resolve_config(a.model), dev, a.seqs, a.prompt_len, a.new_tokens, a.loras, a.runs, tp_group=group,
                          prompt_len_max=a.prompt_len_max)
     if rank == 0:
         print(json.dumps(res))

@@ -2,8 +2,12 @@
 
 One batch is ragged: every sequence brings its next tokens, whether one decoded token or a portion of its prompt, and all
 of them go through the layers together.  ``Ragged`` describes it to the kernels: rows of the sequences one after another
-(``cu_q``), positions, cache rows, block tables, state slots.  Sequences with one new token come first, so that a row range
-tells which form of attention a row takes.
+(``cu_q``), positions, cache rows, block tables, state slots.  Sequences with few new tokens come first, so that a row
+range tells which form of attention a row takes: short ones attend to the cached latents themselves (absorbed form), longer
+portions to keys and values expanded for their window.
+
+A batch of single tokens (decoding) leaves its projections as split-K partial sums in fp32 workspaces, which the kernel
+that follows finishes and clears, as the engine's other models do.
 
 Every sublayer is ``norm -> mixer or feed-forward -> norm -> residual``; the step from one to the next (post-norm, residual
 multiplier, depth average, next input norm) is one kernel over the fp32 residual stream (``ops.hybrid.residual_step``).
@@ -15,7 +19,7 @@ Decoding several tokens per call, CUDA graphs, sampling and logit processing com
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 import torch
 
@@ -39,6 +43,22 @@ class Ragged:
     state_slot: torch.Tensor    # int32 [n_seqs]
     bt: torch.Tensor            # int32 [n_seqs, max_blocks]
     single: bool
+    # portions longer than ABSORB_MAX tokens, in row order behind n_abs shorter rows: (sequence, tokens before, tokens)
+    portions: list[tuple[int, int, int]] = field(default_factory=list)
+    n_abs: int = 0
+    reach: int = 0              # upper bound of the tokens a short row may attend to
+    plans: dict = field(default_factory=dict)
+
+    def plan(self, window: int) -> hy.PrefillPlan:
+        p = self.plans.get(window)
+        if p is None:
+            p = self.plans[window] = hy.plan_prefill(self.portions, window, self.tokens.device)
+        return p
+
+
+# Portions up to this many tokens attend in latent space: expanding a window's keys and values for them would cost more
+# than the wider products of the absorbed form.
+ABSORB_MAX = 16
 
 
 class HybridRunner(DeviceRunner):
@@ -90,17 +110,25 @@ class HybridRunner(DeviceRunner):
             if s.type == "latent_attention":
                 rank_p = pad(s.kv_rank, 16)
                 L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, dp)
+                dk, dv = pad(s.dim, 16), pad(s.vdim, 16)
                 L["c_norm"] = self._vec(m["dkv.norm"])
                 uk, uv = m["uk"].view(s.heads, s.dim, s.kv_rank), m["uv"].view(s.heads, s.vdim, s.kv_rank)
                 L["uk_t"] = torch.zeros(s.heads, rank_p, pad(s.dim, 16), dtype=self.dtype, device=self.device)
                 L["uk_t"][:, :s.kv_rank, :s.dim] = uk.transpose(1, 2).to(self.device)
                 L["uv"] = torch.zeros(s.heads, pad(s.vdim), rank_p, dtype=self.dtype, device=self.device)
                 L["uv"][:, :s.vdim, :s.kv_rank] = uv.to(self.device)
+                if not self.exact32:       # keys of all heads, then values of all heads, from a latent
+                    kv = torch.zeros(s.heads * (dk + dv), rank_p, dtype=self.dtype, device=self.device)
+                    kv[:s.heads * dk].view(s.heads, dk, rank_p)[:, :s.dim, :s.kv_rank] = uk.to(self.device)
+                    kv[s.heads * dk:].view(s.heads, dv, rank_p)[:, :s.vdim, :s.kv_rank] = uv.to(self.device)
+                    L["ukv"] = kv
                 L["inv_freq"] = torch.tensor([s.rope_base ** (-2.0 * j / s.rot_dim) for j in range(s.rot_dim // 2)], dtype=torch.float64
                                              ).to(self.device, torch.float32)
             elif s.type == "hgrn2":
-                L["qv"] = self._mat(torch.cat([m["q"], m["v"]], 0), None, dp)
-                L["f"], L["f_b"], L["lower"] = self._mat(m["f"], None, dp), self._vec(m["f.b"]), self._vec(m["lower"])
+                qv, f = self._mat(torch.cat([m["q"], m["v"]], 0), None, dp), self._mat(m["f"], None, dp)
+                L["qvf"] = torch.cat([qv, f], 0)
+                L["qv"], L["f"] = L["qvf"][:qv.shape[0]], L["qvf"][qv.shape[0]:]
+                L["f_b"], L["lower"] = self._vec(m["f.b"]), self._vec(m["lower"])
                 L["o_norm"] = self._vec(m["norm"])
             else:
                 n = pad(s.heads * s.dim)
@@ -131,15 +159,35 @@ class HybridRunner(DeviceRunner):
 
         return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16))
 
+    def _mm_take(self, b: Ragged, name: str, x, W, f32: bool = False) -> Out:
+        """``x W^T`` for a consumer that accepts a split-K workspace: with few rows the product streams the weights from
+        all SMs and adds partial sums into the fp32 workspace ``name``, which the consumer reads once and leaves zero."""
+        from ..ops.gemm import gemm_splitk_, gemm_tn, plan_small_m
+
+        M, N, K = b.M, W.shape[0], W.shape[1]
+        if not b.single or self.exact32 or M > 512:
+            return self._mm(x, W, f32)
+        pair = M % 256 == 0 and N >= 256
+        bn, splits = plan_small_m(M, N, K, pair=pair)
+        if splits == 1:
+            return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16, bn=0 if pair else bn, two_cta=pair))
+        rows = next(n for n in self.BUCKETS if n >= M)
+        key = ("ws", name, N, rows)
+        ws = self._buf.get(key)
+        if ws is None:
+            ws = self._buf[key] = torch.zeros((rows, N), dtype=torch.float32, device=self.device)
+        gemm_splitk_(ws, x, W, bn, splits, two_cta=pair)
+        return Out(ws[:M], hy.KIND_TAKE)
+
     def _logits(self, hidden) -> torch.Tensor:
         y = self._mm(hidden, self._head, f32=True).t
         return y[:, :self.cfg.vocab_size]
 
-    def _heads_buf(self, name: str, batch: int, b: Ragged, width: int) -> torch.Tensor:
+    def _heads_buf(self, name: str, batch: int, M: int, b: Ragged, width: int) -> torch.Tensor:
         """A head-major operand ``[batch, pitch, width]``, row pitch a multiple of 128.  Rows past M are never read back
         but a tile loads them, so the storage starts as zeros and later holds old finite values.  Batches of single
         tokens have buffers of their own size, which stay where they are: captured graphs hold their addresses."""
-        pitch = pad(b.M, 128)
+        pitch = pad(M, 128)
         n = batch * pitch * width
         # one width per buffer: the padding columns of a row are written by nobody
         key = (name, width, n) if b.single else (name, width)
@@ -153,13 +201,18 @@ class HybridRunner(DeviceRunner):
         """The batch of the sequences' not-yet-cached tokens and, per sequence, its row range."""
         bs, dev = self.kv.shape[1], self.device
         end = [len(s.tokens) if s.upto is None else min(s.upto, len(s.tokens)) for s in seqs]
-        order = sorted(range(len(seqs)), key=lambda i: end[i] - seqs[i].num_cached > 1)      # single tokens first
+        order = sorted(range(len(seqs)), key=lambda i: end[i] - seqs[i].num_cached > ABSORB_MAX)
+        portions, n_abs, reach = [], 0, 0
         tok, pos, slot, row_seq, cu, ranges = [], [], [], [], [0], [(0, 0)] * len(seqs)
         for j, i in enumerate(order):
             s = seqs[i]
             n0, n1 = s.num_cached, end[i]
             if n1 <= n0:
                 raise ValueError("a scheduled sequence brings at least one token")
+            if n1 - n0 <= ABSORB_MAX or self.exact32:
+                n_abs, reach = n_abs + n1 - n0, max(reach, n1)
+            else:
+                portions.append((j, n0, n1 - n0))
             tok += s.tokens[n0:n1]
             pos += range(n0, n1)
             slot += [s.blocks[t // bs] * bs + t % bs for t in range(n0, n1)]
@@ -170,7 +223,7 @@ class HybridRunner(DeviceRunner):
         i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
         b = Ragged(cu[-1], len(seqs), torch.tensor(tok, dtype=torch.int64, device=dev), i32(pos), i32(slot), i32(row_seq), i32(cu),
                    i32([end[i] for i in order]), i32([seqs[i].state_slot for i in order]),
-                   i32([seqs[i].blocks + [0] * (width - len(seqs[i].blocks)) for i in order]), cu[-1] == len(seqs))
+                   i32([seqs[i].blocks + [0] * (width - len(seqs[i].blocks)) for i in order]), cu[-1] == len(seqs), portions, n_abs, reach)
         return b, ranges
 
     # -- layers ---------------------------------------------------------------------------------------------
@@ -190,9 +243,9 @@ class HybridRunner(DeviceRunner):
             post = L["norm1b"]
             if s.ff:
                 hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
-                z = self._mm(h, L["up"])
+                z = self._mm_take(b, "up", h, L["up"])
                 a = torch.empty((M, pad(s.ff)), dtype=self.dtype, device=dev)
-                y = self._mm(hy.poly_norm(z, L["act"], a, s.ff, eps), L["down"])
+                y = self._mm_take(b, "down", hy.poly_norm(z, L["act"], a, s.ff, eps), L["down"])
                 post = L["norm2b"]
             hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
             if capture is not None:
@@ -200,22 +253,34 @@ class HybridRunner(DeviceRunner):
         return x, h
 
     def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Out:
-        M, H = b.M, s.heads
+        M, H, n_abs = b.M, s.heads, b.n_abs
         cache = self.kv.layers[i]["latent"]
-        p = self._mm(h, L["qkv"])
-        rank_p, rot_p = pad(s.kv_rank, 16), pad(s.rot_dim, 16)
-        qn = self._heads_buf("qn", H, b, pad(s.dim, 16))
-        qr = self._heads_buf("qr", H, b, rot_p)
-        hy.latent_finish(p, L["c_norm"], L["inv_freq"], b.pos, b.slot, cache, M, qn, qr, None, H, s.dim, s.rot_dim, s.kv_rank,
+        p = self._mm_take(b, "qkv", h, L["qkv"])
+        rank_p, rot_p, dk, dv, vp = pad(s.kv_rank, 16), pad(s.rot_dim, 16), pad(s.dim, 16), pad(s.vdim, 16), pad(s.vdim)
+        qn = qr = qe = None
+        if n_abs:
+            qn, qr = self._heads_buf("qn", H, n_abs, b, dk), self._heads_buf("qr", H, n_abs, b, rot_p)
+        if n_abs < M:
+            qe = torch.empty((M - n_abs, H * (dk + rot_p)), dtype=self.dtype, device=self.device)
+        hy.latent_finish(p, L["c_norm"], L["inv_freq"], b.pos, b.slot, cache, n_abs, qn, qr, qe, H, s.dim, s.rot_dim, s.kv_rank,
                          self.cfg.norm_eps)
-        ql = self._heads_buf("ql", H, b, rank_p)
-        hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), M, c_batch=ql.stride(0))
-        ol = self._heads_buf("ol", H, b, rank_p)
-        hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, M)
-        vp = pad(s.vdim)
         o = torch.empty((M, H * vp), dtype=self.dtype, device=self.device)
-        hy.gemm_batched(ol, L["uv"], o, M, c_batch=vp)
-        return self._mm(o, L["o"])
+        if n_abs:
+            ql, ol = self._heads_buf("ql", H, n_abs, b, rank_p), self._heads_buf("ol", H, n_abs, b, rank_p)
+            hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), n_abs, c_batch=ql.stride(0))
+            if self.exact32:
+                hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs)
+            else:
+                keys = min(b.reach, s.window) if s.window > 0 else b.reach
+                hy.latent_decode(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs,
+                                 hy.latent_decode_splits(n_abs, H, keys))
+            hy.gemm_batched(ol, L["uv"], o, n_abs, c_batch=vp)
+        if n_abs < M:
+            plan = b.plan(s.window)
+            c = hy.latent_gather(cache, b.bt, plan)
+            kv = self._mm(c[:, :rank_p], L["ukv"]).t
+            hy.latent_prefill(qe, kv, c, plan, s.window, s.scale, o[n_abs:], H, dk, dv, rank_p, rot_p, s.vdim)
+        return self._mm_take(b, "o", o, L["o"])
 
     def _scan(self, mode, i, s, L, q, k, v, g, aux, bias, gate, b: Ragged) -> Out:
         """Recurrence, per-head norm and gate, output projection."""
@@ -230,22 +295,25 @@ class HybridRunner(DeviceRunner):
             o = torch.empty((M, H * s.vdim), dtype=torch.float32, device=self.device)
             hy.linear_scan(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, H, s.dim, s.vdim, o)
             hy.head_norm(o, L["o_norm"], per_head, H, s.vdim, vp, out, eps, gate)
-        return self._mm(out, L["o"])
+        return self._mm_take(b, "o", out, L["o"])
 
     def _mix_hgrn2(self, i, s, L, x, h, b: Ragged) -> Out:
-        qv = self._mm(h, L["qv"])
-        g = self._mm(h, L["f"], f32=True)
+        if b.single:        # one product, its outputs are taken where they lie
+            p = self._mm_take(b, "qvf", h, L["qvf"], f32=True)
+            qv, g = p, p.col(L["qv"].shape[0])
+        else:
+            qv, g = self._mm(h, L["qv"]), self._mm(h, L["f"], f32=True)
         return self._scan(hy.SCAN_HGRN2, i, s, L, qv, None, qv.col(s.heads * s.dim), g, L["lower"], L["f_b"], None, b)
 
     def _mix_wkv(self, i, s, L, x, h, b: Ragged) -> Out:
         M, n = b.M, L["rkvg"].shape[1]
-        mixes = self._heads_buf("mix", len(SHIFT_MIXES), b, self.dp)
+        mixes = self._heads_buf("mix", len(SHIFT_MIXES), M, b, self.dp)
         hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
                           self.cfg.hidden_size, self.cfg.norm_eps)
         y = torch.empty((M, 4 * n), dtype=self.dtype, device=self.device)
         hy.gemm_batched(mixes[:4], L["rkvg"], y, M, c_batch=n)
         rp = L["w1"].shape[0]
-        z = self._mm(mixes[4, :M], L["w1"], f32=True)
+        z = self._mm_take(b, "w1", mixes[4, :M], L["w1"], f32=True)
         t = torch.empty((M, L["w2"].shape[1]), dtype=self.dtype, device=self.device)
         g = self._mm(hy.split_tanh(z, s.decay_rank, rp, t), L["w2"], f32=True)
         y = as_out(y)
@@ -288,13 +356,27 @@ class HybridRunner(DeviceRunner):
         st["state_slot"].copy_(torch.tensor([s.state_slot for s in seqs] + [-1] * (nb - len(seqs)), dtype=torch.int32), non_blocking=True)
 
     def _attn_splits(self, nb: int, max_ctx: int) -> int:
-        return 1
+        """Stands for how far the batch's tokens reach back (a power of two): the latent layers plan their splits by it.
+        Contexts beyond every window change nothing, so that they share one captured graph."""
+        windows = [s.window for s in self.cfg.layers if s.type == "latent_attention"]
+        if not windows:
+            return 1
+        bound = max_ctx if any(w <= 0 for w in windows) else min(max_ctx, max(windows))
+        return 1 << max(0, bound - 1).bit_length()
+
+    def _attn_workspace(self, nb: int, splits: int) -> None:
+        return None
+
+    def drop_graphs(self) -> None:
+        super().drop_graphs()
+        self._buf.clear()         # workspaces of an interrupted step may hold partial sums
 
     def _decode_steps(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool, procs) -> None:
         from ..ops import paged
 
         nb = st["tokens"].shape[0]
-        b = Ragged(nb, nb, st["tokens"], st["pos"], st["slot"], st["row_seq"], st["cu_q"], st["ctx"], st["state_slot"], st["bt"], True)
+        b = Ragged(nb, nb, st["tokens"], st["pos"], st["slot"], st["row_seq"], st["cu_q"], st["ctx"], st["state_slot"], st["bt"], True,
+                   n_abs=nb, reach=splits)
         for k in range(n_steps):
             _, hidden = self._forward(b, want_hidden=True)
             t, lp = self._sample(hidden, st["inv_t"], st["seeds"][k], restricted, st["top_k"], st["top_p"], st["min_p"], procs=procs)

@@ -30,6 +30,9 @@ _sigs = {
     "artb_latent_finish": [ci, vp, ci, ci, vp, vp, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
                            vp],
     "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
+    "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, ci, vp, vp],
+    "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, vp, ci, vp, vp],
+    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, ci, ci, ci, vp],
     "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
     "artb_gemm_f32_tn": [vp, ci, cl, vp, ci, cl, vp, ci, cl, ci, ci, ci, ci, vp],
 }
@@ -156,14 +159,13 @@ def linear_decode(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, s
 def latent_finish(p: Out, w, inv_freq, pos, slot, cache, n_abs: int, qn, qr, qe, H: int, dim: int, rot: int, rank: int,
                   eps: float) -> None:
     """Norm, rotation and cache write behind the q | latent projection.  Rows below ``n_abs`` leave their queries in
-    ``qn`` [H, pitch, dim_p] / ``qr`` [H, pitch, rot_p], the others in ``qe`` [M - n_abs, H * (dim + rot)]."""
+    ``qn`` [H, pitch, dim_p] / ``qr`` [H, pitch, rot_p], the others in ``qe`` [M - n_abs, H * (dim_p + rot_p)]."""
     M = pos.numel()
-    rank_p, rot_p = pad(rank, 16), pad(rot, 16)
     _lib.check_rc(_f("artb_latent_finish")(
         _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(w), _lib.ptr(inv_freq), _lib.ptr(pos), _lib.ptr(slot),
         _lib.ptr(cache), cache.shape[-1], cache.shape[0] * cache.shape[1], n_abs, _lib.ptr(qn), _lib.ptr(qr),
-        qn.shape[1] if qn is not None else 0, _lib.ptr(qe), qe.stride(0) if qe is not None else 0, M, H, dim,
-        qn.shape[2] if qn is not None else dim, rot, rot_p, rank, rank_p, eps, _st(cache), _lib.stream_ptr()), "latent_finish")
+        qn.shape[1] if qn is not None else 0, _lib.ptr(qe), qe.stride(0) if qe is not None else 0, M, H, dim, pad(dim, 16), rot,
+        pad(rot, 16), rank, pad(rank, 16), eps, _st(cache), _lib.stream_ptr()), "latent_finish")
 
 
 def latent_attend(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int) -> torch.Tensor:
@@ -173,6 +175,87 @@ def latent_attend(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, sc
         _is32(cache), _lib.ptr(ql), _lib.ptr(qr), pitch, _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table),
         block_table.stride(0), cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale,
         _lib.ptr(o), M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_attend")
+    return o
+
+
+LATENT_TILE = 64        # keys per tile of the decode kernel: the unit its splits are made of
+PREFILL_ROWS = 128      # query rows per CTA of the prefill kernel
+
+
+def latent_decode_splits(M: int, H: int, keys: int, sms: int = 148) -> int:
+    """How many CTAs share a token's window: enough to cover the machine, two tiles each at least."""
+    ctas = M * ((H + 31) // 32 if H > 16 else 1)
+    return max(1, min(sms // max(1, ctas), (keys + LATENT_TILE - 1) // LATENT_TILE // 2, 32))
+
+
+def latent_decode(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int, splits: int = 1,
+                  ws=None) -> torch.Tensor:
+    """Tensor-core form of :func:`latent_attend` for rows ``0 .. M - 1`` (bf16)."""
+    H, pitch, rank_p = ql.shape
+    if splits > 1 and ws is None:
+        ws = torch.empty(M * H * splits * (rank_p + 2), dtype=torch.float32, device=o.device)
+    _lib.check_rc(_f("artb_latent_decode")(
+        _lib.ptr(ql), _lib.ptr(qr), pitch, _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0),
+        cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale, _lib.ptr(o), _lib.ptr(ws), splits,
+        M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_decode")
+    return o
+
+
+@dataclass
+class PrefillPlan:
+    """Query tiles and gathered key ranges of the portions of one batch under one window (int32, on the device).  Row
+    numbers count from the first portion row of the batch."""
+    n_keys: int
+    n_tiles: int
+    n_seqs: int
+    seq_of: torch.Tensor
+    key_off: torch.Tensor
+    key_pos0: torch.Tensor
+    row_end: torch.Tensor
+    row_pos0: torch.Tensor
+    tile_seq: torch.Tensor
+    tile_row: torch.Tensor
+
+
+def plan_prefill(portions: list[tuple[int, int, int]], window: int, device) -> PrefillPlan:
+    """``portions``: ``(sequence, tokens before the portion, tokens of the portion)`` in row order."""
+    seq_of, key_off, key_pos0, row_end, row_pos0, tile_seq, tile_row = [], [], [], [], [], [], []
+    row = keys = 0
+    for i, (seq, n0, n) in enumerate(portions):
+        first = max(0, n0 - window + 1) if window > 0 else 0
+        seq_of.append(seq)
+        key_off.append(keys)
+        key_pos0.append(first)
+        keys += n0 + n - first
+        row_pos0.append(n0 - row)
+        for r in range(row, row + n, PREFILL_ROWS):
+            tile_seq.append(i)
+            tile_row.append(r)
+        row += n
+        row_end.append(row)
+    t = lambda v: torch.tensor(v, dtype=torch.int32, device=device)      # noqa: E731
+    return PrefillPlan(keys, len(tile_seq), len(portions), t(seq_of), t(key_off), t(key_pos0), t(row_end), t(row_pos0), t(tile_seq), t(tile_row))
+
+
+def latent_gather(cache, block_table, plan: PrefillPlan) -> torch.Tensor:
+    """The cache rows the portions' windows reach, contiguous: ``[n_keys, rank_p + rot_p]``."""
+    out = torch.empty((plan.n_keys, cache.shape[-1]), dtype=cache.dtype, device=cache.device)
+    _lib.check_rc(_f("artb_latent_gather")(
+        _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1], cache.shape[0],
+        _lib.ptr(plan.seq_of), _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), plan.n_seqs, _lib.ptr(out), plan.n_keys, _st(cache),
+        _lib.stream_ptr()), "latent_gather")
+    return out
+
+
+def latent_prefill(q, kv, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
+                   vdim: int) -> torch.Tensor:
+    """Windowed attention of the portions: ``q`` [rows, H * (dk + rot_p)], ``kv`` [n_keys, H * dk + H * dv] the expanded
+    keys and values, ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)]."""
+    _lib.check_rc(_f("artb_latent_prefill")(
+        _lib.ptr(q), q.stride(0), _lib.ptr(kv), kv.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(plan.tile_seq),
+        _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0), _lib.ptr(plan.key_off),
+        _lib.ptr(plan.key_pos0), window, scale, _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, dk, dv, rot_p, _lib.stream_ptr()),
+        "latent_prefill")
     return o
 
 
