@@ -24,6 +24,8 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
   *reinterpret_cast<__nv_bfloat162*>(&r.y) = __floats2bfloat162_rn(v.z, v.w);
   *reinterpret_cast<uint2*>(p) = r;
 }
+__device__ __forceinline__ float ld1(const float* p) { return *p; }
+__device__ __forceinline__ float ld1(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void st1(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
@@ -34,6 +36,33 @@ __device__ __forceinline__ float4 take4(void* p, size_t off, int kind) {
   const float4 v = ld4(f);
   if (kind == ROW_F32_TAKE) st4(f, make_float4(0.f, 0.f, 0.f, 0.f));
   return v;
+}
+// eight elements (16-byte aligned)
+__device__ __forceinline__ void take8(void* p, size_t off, int kind, float (&f)[8]) {
+  if (kind == ROW_BF16) {
+    const uint4 r = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p) + off);
+    const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&r);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 v = __bfloat1622float2(b[i]);
+      f[2 * i] = v.x;
+      f[2 * i + 1] = v.y;
+    }
+    return;
+  }
+  const float4 a = take4(p, off, kind), c = take4(p, off + 4, kind);
+  f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = c.x, f[5] = c.y, f[6] = c.z, f[7] = c.w;
+}
+__device__ __forceinline__ void put8(float* p, const float (&f)[8]) {
+  st4(p, make_float4(f[0], f[1], f[2], f[3]));
+  st4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+__device__ __forceinline__ void put8(__nv_bfloat16* p, const float (&f)[8]) {
+  uint4 r;
+  __nv_bfloat162* b = reinterpret_cast<__nv_bfloat162*>(&r);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) b[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+  *reinterpret_cast<uint4*>(p) = r;
 }
 __device__ __forceinline__ float take1(void* p, size_t off, int kind) {
   if (kind == ROW_BF16) return __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p)[off]);

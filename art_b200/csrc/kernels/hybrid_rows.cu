@@ -215,31 +215,32 @@ __global__ void __launch_bounds__(256) norm_shift_mix_kernel(const ShiftArgs a) 
 }
 
 // ------------------------------------------------------------------------------------------------ PolyNorm
+// vectors of eight elements (16 bytes of bf16); np is a multiple of 8
 template <typename T, int MAXV>
 __global__ void __launch_bounds__(512)
 poly_norm_kernel(void* z, int ldz, int kind, const float* __restrict__ act, T* out, int ldo, int n, int np, float eps) {
   __shared__ float red[3][16];
   pdl_wait();
   pdl_launch_dependents();
-  const int row = blockIdx.x, nv = np >> 2;
-  float4 v[MAXV];
+  const int row = blockIdx.x, nv = np >> 3;
+  float v[MAXV][8];
   float s1 = 0.f, s2 = 0.f, s3 = 0.f;
 #pragma unroll
   for (int i = 0; i < MAXV; ++i) {
     const int c = threadIdx.x + i * blockDim.x;
-    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < nv) {
-      v[i] = take4(z, static_cast<size_t>(row) * ldz + c * 4, kind);
-      const float* e = &v[i].x;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float q = e[j] * e[j], q2 = q * q;
-        s1 += q;
-        s2 += q2;
-        s3 = fmaf(q2, q, s3);
-      }
-    }
+    for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
+    if (c < nv) take8(z, static_cast<size_t>(row) * ldz + c * 8, kind, v[i]);
   }
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float q = v[i][j] * v[i][j], q2 = q * q;
+      s1 += q;
+      s2 += q2;
+      s3 = fmaf(q2, q, s3);
+    }
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   s1 = lane_sum(s1);
   s2 = lane_sum(s2);
@@ -255,12 +256,12 @@ poly_norm_kernel(void* z, int ldz, int kind, const float* __restrict__ act, T* o
   for (int i = 0; i < MAXV; ++i) {
     const int c = threadIdx.x + i * blockDim.x;
     if (c < nv) {
-      float4 o;
-      const float* x = &v[i].x;
-      float* y = &o.x;
 #pragma unroll
-      for (int j = 0; j < 4; ++j) y[j] = c * 4 + j < n ? fmaf(fmaf(fmaf(c3, x[j], b), x[j], a), x[j], e0) : 0.f;
-      st4(out + static_cast<size_t>(row) * ldo + c * 4, o);
+      for (int j = 0; j < 8; ++j) {
+        const float x = v[i][j];
+        v[i][j] = c * 8 + j < n ? fmaf(fmaf(fmaf(c3, x, b), x, a), x, e0) : 0.f;
+      }
+      put8(out + static_cast<size_t>(row) * ldo + c * 8, v[i]);
     }
   }
 }
@@ -281,27 +282,55 @@ __global__ void split_tanh_kernel(void* z, int ldz, int kind, T* out, int ldo, i
 }
 
 // --------------------------------------------------------------------------------------------- per-head norm
-// one warp per (row, head): out[row, h * vp + j] = rms(o[row, h, :])_j * w  (* silu(gate)), padding columns zero
-template <typename T>
+// out[row, h * vp + j] = rms(o[row, h, :])_j * w  (* silu(gate)), padding columns zero.  LPH lanes share a (row, head);
+// with V4 a lane handles four neighbouring elements (vdim, vp and all strides multiples of 4).
+template <typename T, int LPH, bool V4>
 __global__ void __launch_bounds__(256)
 head_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__ w, int w_per_head, void* gate, int ldg,
                  int gate_kind, T* out, int ldo, int M, int H, int vdim, int vp, float eps) {
   pdl_wait();
   pdl_launch_dependents();
-  const int u = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (u >= M * H) return;
-  const int m = u / H, h = u % H;
+  const int u = static_cast<int>(blockIdx.x * (256u / LPH) + threadIdx.x / LPH);     // M * H < 2^31
+  const int lane = threadIdx.x % LPH;
+  const bool live = u < M * H;
+  const int m = live ? u / H : 0, h = live ? u % H : 0;
   const float* x = o + static_cast<size_t>(m) * ldi + h * vdim;
   float ss = 0.f;
-  for (int j = lane; j < vdim; j += 32) ss += x[j] * x[j];
-  const float r = 1.f / sqrtf(lane_sum(ss) / vdim + eps);
-  for (int j = lane; j < vp; j += 32) {
-    float v = 0.f;
-    if (j < vdim) {
-      v = x[j] * r * w[w_per_head ? h * vdim + j : j];
-      if (gate) v *= silu_f(take1(gate, static_cast<size_t>(m) * ldg + h * vdim + j, gate_kind));
+  if (live) {
+    if (V4)
+      for (int j = lane * 4; j < vdim; j += LPH * 4) ss += sq4(ld4(x + j));
+    else
+      for (int j = lane; j < vdim; j += LPH) ss += x[j] * x[j];
+  }
+#pragma unroll
+  for (int s = LPH / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!live) return;
+  const float r = 1.f / sqrtf(ss / vdim + eps);
+  const float* wh = w + (w_per_head ? h * vdim : 0);
+  T* y = out + static_cast<size_t>(m) * ldo + h * vp;
+  const size_t go = static_cast<size_t>(m) * ldg + h * vdim;
+  if (V4) {
+    for (int j = lane * 4; j < vp; j += LPH * 4) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (j < vdim) {
+        const float4 a = ld4(x + j), b = ld4(wh + j);
+        v = make_float4(a.x * r * b.x, a.y * r * b.y, a.z * r * b.z, a.w * r * b.w);
+        if (gate) {
+          const float4 g = take4(gate, go + j, gate_kind);
+          v = make_float4(v.x * silu_f(g.x), v.y * silu_f(g.y), v.z * silu_f(g.z), v.w * silu_f(g.w));
+        }
+      }
+      st4(y + j, v);
     }
-    st1(out + static_cast<size_t>(m) * ldo + h * vp + j, v);
+  } else {
+    for (int j = lane; j < vp; j += LPH) {
+      float v = 0.f;
+      if (j < vdim) {
+        v = x[j] * r * wh[j];
+        if (gate) v *= silu_f(take1(gate, go + j, gate_kind));
+      }
+      st1(y + j, v);
+    }
   }
 }
 
@@ -339,6 +368,15 @@ using namespace artb;
     case 4: CALL(4); break;   \
     case 8: CALL(8); break;   \
     case 16: CALL(16); break; \
+    default: return ERR_TOO_LARGE; \
+  }
+
+#define ARTB_BY_VECS8(V, CALL) \
+  switch (V) {                 \
+    case 1: CALL(1); break;    \
+    case 2: CALL(2); break;    \
+    case 4: CALL(4); break;    \
+    case 8: CALL(8); break;    \
     default: return ERR_TOO_LARGE; \
   }
 
@@ -384,15 +422,15 @@ ARTB_EXPORT int artb_norm_shift_mix(int f32, const float* x, int ldx, const floa
 ARTB_EXPORT int artb_poly_norm(int f32, void* z, int ldz, int kind, const float* act, void* out, int ldo, int M, int n, int np,
                                float eps, cudaStream_t st) {
   if (M <= 0) return 0;
-  if ((np & 3) || np < n || (ldz & 3) || (ldo & 3)) return ERR_BAD_SHAPE;
-  const int th = np <= 1024 ? 128 : np <= 4096 ? 256 : 512;
+  if ((np & 7) || np < n || (ldz & 7) || (ldo & 7)) return ERR_BAD_SHAPE;
+  const int th = np <= 2048 ? 128 : np <= 8192 ? 256 : 512;
   cudaError_t e = cudaSuccess;
 #define ARTB_PN(V)                                                                                                       \
   e = f32 ? launch_kernel(poly_norm_kernel<float, V>, dim3(M), dim3(th), 0, st, z, ldz, kind, act,                        \
                           reinterpret_cast<float*>(out), ldo, n, np, eps)                                                 \
           : launch_kernel(poly_norm_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, z, ldz, kind, act,                \
                           reinterpret_cast<__nv_bfloat16*>(out), ldo, n, np, eps)
-  ARTB_BY_VECS(row_vecs(np, th), ARTB_PN)
+  ARTB_BY_VECS8(row_vecs(np / 2, th), ARTB_PN)
 #undef ARTB_PN
   return static_cast<int>(e);
 }
@@ -411,13 +449,24 @@ ARTB_EXPORT int artb_split_tanh(int f32, void* z, int ldz, int kind, void* out, 
 ARTB_EXPORT int artb_head_norm(int f32, const float* o, int ldi, const float* w, int w_per_head, void* gate, int ldg,
                                int gate_kind, void* out, int ldo, int M, int H, int vdim, int vp, float eps, cudaStream_t st) {
   if (M <= 0) return 0;
-  if (H <= 0 || vdim <= 0 || vp < vdim || ldo < H * vp) return ERR_BAD_SHAPE;
-  const dim3 grid(static_cast<unsigned>((static_cast<long>(M) * H + 7) / 8));
-  return static_cast<int>(f32 ? launch_kernel(head_norm_kernel<float>, grid, dim3(256), 0, st, o, ldi, w, w_per_head, gate, ldg,
-                                              gate_kind, reinterpret_cast<float*>(out), ldo, M, H, vdim, vp, eps)
-                              : launch_kernel(head_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, ldi, w, w_per_head,
-                                              gate, ldg, gate_kind, reinterpret_cast<__nv_bfloat16*>(out), ldo, M, H, vdim, vp,
-                                              eps));
+  if (H <= 0 || vdim <= 0 || vp < vdim || ldo < H * vp || static_cast<long>(M) * H >= (1L << 31)) return ERR_BAD_SHAPE;
+  const bool v4 = !((vdim | vp | ldi | ldo | (gate ? ldg : 0)) & 3) && !(reinterpret_cast<uintptr_t>(gate) & 15);
+  const int lph = !v4 ? 32 : vdim <= 16 ? 4 : vdim <= 64 ? 16 : 32;
+  const dim3 grid(static_cast<unsigned>((static_cast<long>(M) * H * lph + 255) / 256));
+#define ARTB_HN(T_, L_, V_)                                                                                             \
+  return static_cast<int>(launch_kernel(head_norm_kernel<T_, L_, V_>, grid, dim3(256), 0, st, o, ldi, w, w_per_head, gate, ldg, \
+                                        gate_kind, reinterpret_cast<T_*>(out), ldo, M, H, vdim, vp, eps))
+  if (f32) {
+    if (lph == 4) ARTB_HN(float, 4, true);
+    if (lph == 16) ARTB_HN(float, 16, true);
+    if (v4) ARTB_HN(float, 32, true);
+    ARTB_HN(float, 32, false);
+  }
+  if (lph == 4) ARTB_HN(__nv_bfloat16, 4, true);
+  if (lph == 16) ARTB_HN(__nv_bfloat16, 16, true);
+  if (v4) ARTB_HN(__nv_bfloat16, 32, true);
+  ARTB_HN(__nv_bfloat16, 32, false);
+#undef ARTB_HN
 }
 
 ARTB_EXPORT int artb_gather_norm(int f32, const float* x, int ldx, const int64_t* rows, int n, const float* w, void* h, int ldh,

@@ -9,12 +9,13 @@
 //
 // Two kernels share the state layout [slot][head][vdim][ld_dim] (a column of S is contiguous):
 //
-//   linear_scan_kernel     portions of prompts.  A CTA owns (sequence, head, a slice of CW value columns) and walks over
-//                          the portion.  The state lives in registers: eight threads share a column, each with NR of its
-//                          rows (interleaved in groups of four, so that operands are 16-byte shared-memory reads without
-//                          bank conflicts).  Four extra warps load the next 16 tokens and apply decay / gate functions
-//                          while the others work on the current 16; the eight partial sums of eight tokens are reduced
-//                          by a seven-step exchange instead of 24 shuffles.
+//   linear_scan_kernel     portions of prompts.  A CTA owns (sequence, head, a slice of 16, 32 or 64 value columns) and
+//                          walks over the portion.  The state lives in registers: eight threads share one to four
+//                          columns, each with NR of their rows (interleaved in groups of four, so that operands are
+//                          16-byte shared-memory reads without bank conflicts).  Four extra warps load the
+//                          next 16 tokens and apply decay / gate functions while the others work on the current
+//                          16; the partial sums of four tokens over eight threads are reduced by four exchanges
+//                          instead of twelve.
 //   linear_decode_kernel   one new token per sequence.  A CTA owns (sequence, head), streams the state through registers
 //                          once (read, update, write) and finishes the head: RMSNorm over its vdim outputs, norm weight,
 //                          optional silu gate, bf16 store.
@@ -67,8 +68,6 @@ struct DecodeOut {
   float eps;
 };
 
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
-
 // packed fp32 pairs (one instruction per two multiply-adds)
 __device__ __forceinline__ uint64_t pack2(float a, float b) {
   uint64_t r;
@@ -110,177 +109,228 @@ constexpr int scan_smem(int DP, int cw) {
   return 2 * SCAN_TC * (scan_arrays<MODE>() * DP + 2 * cw + 1) * 4;
 }
 
-// decay, gate and raw values of channel i of one token; channels past dim leave the state at zero
+// decay, gate and bonus of one channel from the raw projections; k of hgrn2 is 1 - f
 template <int MODE>
-__device__ __forceinline__ void scan_channel(const ScanArgs& a, int m, int h, int i, float& q, float& f, float& k, float& bonus) {
-  q = 0.f;
-  k = 0.f;
-  bonus = 0.f;
-  f = MODE == SCAN_HGRN2 ? 1.f : 0.f;
-  if (i >= a.dim) return;
-  const int c = h * a.dim + i;
-  const float qr = take1(a.q, static_cast<size_t>(m) * a.ldq + c, a.qkv_kind);
-  const float g = take1(a.g, static_cast<size_t>(m) * a.ldg + c, a.g_kind) + a.bias[c];
+__device__ __forceinline__ void scan_gates(float qr, float kr, float g, float aux, float& q, float& f, float& k, float& bonus) {
   if (MODE == SCAN_HGRN2) {
-    const float l = a.aux[c];
-    q = silu_f(qr);
-    f = l + (1.f - l) * sigmoid_f(g);
+    q = __fdividef(qr, 1.f + expf(-qr));
+    f = aux + (1.f - aux) * __fdividef(1.f, 1.f + expf(-g));
+    k = 1.f - f;
+    bonus = 0.f;
   } else {
     q = qr;
     f = expf(-expf(g));
-    k = take1(a.k, static_cast<size_t>(m) * a.ldk + c, a.qkv_kind);
-    bonus = q * a.aux[c] * k;
+    k = kr;
+    bonus = qr * aux * kr;
   }
 }
 
-template <int NR, int MODE>
-__global__ void __launch_bounds__(SCAN_RG * 32 + SCAN_LOADERS)
-linear_scan_kernel(const ScanArgs a, const ScanOut so, int cw) {
-  constexpr int DP = SCAN_RG * NR;
+// all compute and loader warps; a named barrier because the two roles wait at different places of the code
+__device__ __forceinline__ void stage_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(SCAN_RG * 16 + SCAN_LOADERS) : "memory"); }
+
+// A CTA's column slice is CW = 16 * CPT wide: thread (rg, cg) holds rows {4 rg + 32 i} of columns {cg + 16 j}.
+template <int NR, int MODE, int CPT, typename T>
+__global__ void __launch_bounds__(SCAN_RG * 16 + SCAN_LOADERS, CPT * NR <= 64 ? 2 : 1)
+linear_scan_kernel(const ScanArgs a, const ScanOut so) {
+  constexpr int DP = SCAN_RG * NR, CW = 16 * CPT, COMP = SCAN_RG * 16, CH = DP / 32;
   extern __shared__ __align__(16) float scan_s[];
   float* sq = scan_s;                                   // [2][TC][DP]
   float* sf = sq + 2 * SCAN_TC * DP;
   float* sk = sf + 2 * SCAN_TC * DP;                    // wkv only
-  float* sv = sk + (MODE == SCAN_WKV ? 2 * SCAN_TC * DP : 0);   // [2][TC][cw]
-  float* sout = sv + 2 * SCAN_TC * cw;                  // [2][TC][cw]
-  float* sb = sout + 2 * SCAN_TC * cw;                  // [2][TC] bonus
+  float* sv = sk + (MODE == SCAN_WKV ? 2 * SCAN_TC * DP : 0);   // [2][TC][CW]
+  float* sout = sv + 2 * SCAN_TC * CW;                  // [2][TC][CW]
+  float* sb = sout + 2 * SCAN_TC * CW;                  // [2][TC] bonus
   pdl_wait();
   pdl_launch_dependents();
-  const int seq = blockIdx.y, h = blockIdx.x % a.H, c0 = (blockIdx.x / a.H) * cw;
-  const int row0 = a.cu_q[seq], T = a.cu_q[seq + 1] - row0;
-  if (T <= 0) return;
+  const int seq = blockIdx.y, h = blockIdx.x % a.H, c0 = (blockIdx.x / a.H) * CW;
+  const int row0 = a.cu_q[seq], len = a.cu_q[seq + 1] - row0;
+  if (len <= 0) return;
   int slot = a.state_slot[seq];
   if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
-  const int n_comp = SCAN_RG * cw;
-  const bool comp = static_cast<int>(threadIdx.x) < n_comp;
-  const int lt = static_cast<int>(threadIdx.x) - n_comp, lane = threadIdx.x & 31;
+  const bool comp = static_cast<int>(threadIdx.x) < COMP;
+  const int chunks = (len + SCAN_TC - 1) / SCAN_TC;
 
-  auto load = [&](int chunk, int buf) {       // loader warps: one token per warp at a time
-    const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, T - t0);
-    for (int t = lt >> 5; t < nt; t += SCAN_LOADERS / 32) {
-      const int m = row0 + t0 + t, at = buf * SCAN_TC + t;
-      float bsum = 0.f;
+  if (!comp) {
+    // ---------------------------------------------------------------- loader warps: one token per warp at a time
+    const int lt = static_cast<int>(threadIdx.x) - COMP, lane = lt & 31, lw = lt >> 5;
+    constexpr int TB = DP <= 96 ? 4 : 2;                // tokens whose raw values are in flight together
+    constexpr int PER = SCAN_TC / (SCAN_LOADERS / 32);  // tokens per warp and stage
+    float bias[CH], aux[CH];
 #pragma unroll
-      for (int i0 = 0; i0 < DP; i0 += 32) {
-        float q, f, k, b;
-        const int i = i0 + lane;
-        if (DP % 32 == 0 || i < DP) {
-          scan_channel<MODE>(a, m, h, i, q, f, k, b);
-          sq[at * DP + i] = q;
-          sf[at * DP + i] = f;
-          if (MODE == SCAN_WKV) {
-            sk[at * DP + i] = k;
-            bsum += b;
+    for (int i = 0; i < CH; ++i) {
+      const int c = i * 32 + lane;
+      bias[i] = c < a.dim ? a.bias[h * a.dim + c] : 0.f;
+      aux[i] = c < a.dim ? a.aux[h * a.dim + c] : 0.f;
+    }
+    const T* __restrict__ gq = reinterpret_cast<const T*>(a.q) + h * a.dim;
+    const T* __restrict__ gk = reinterpret_cast<const T*>(a.k) + h * a.dim;
+    const T* __restrict__ gv = reinterpret_cast<const T*>(a.v) + h * a.vdim + c0;
+    const float* __restrict__ gg = reinterpret_cast<const float*>(a.g) + h * a.dim;
+    auto load = [&](int chunk, int buf) {
+      const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, len - t0);
+#pragma unroll 1
+      for (int p = 0; p < PER; p += TB) {
+        float rq[TB][CH], rg_[TB][CH], rk[TB][CH], rv[TB][(CW + 31) / 32];
+#pragma unroll
+        for (int b = 0; b < TB; ++b) {
+          const int t = lw + (p + b) * (SCAN_LOADERS / 32);
+          const size_t m = static_cast<size_t>(row0 + t0 + t);
+#pragma unroll
+          for (int i = 0; i < CH; ++i) {
+            const int c = i * 32 + lane;
+            const bool ok = t < nt && c < a.dim;
+            rq[b][i] = ok ? ld1(gq + m * a.ldq + c) : 0.f;
+            rg_[b][i] = ok ? ld1(gg + m * a.ldg + c) : 0.f;
+            if (MODE == SCAN_WKV) rk[b][i] = ok ? ld1(gk + m * a.ldk + c) : 0.f;
+          }
+#pragma unroll
+          for (int i = 0; i < (CW + 31) / 32; ++i) {
+            const int c = i * 32 + lane;
+            rv[b][i] = t < nt && c < CW && c0 + c < a.vdim ? ld1(gv + m * a.ldv + c) : 0.f;
           }
         }
-      }
-      if (MODE == SCAN_WKV) {
-        bsum = lane_sum(bsum);
-        if (lane == 0) sb[at] = bsum;
-      }
-      for (int c = lane; c < cw; c += 32)
-        sv[at * cw + c] = c0 + c < a.vdim ? take1(a.v, static_cast<size_t>(m) * a.ldv + h * a.vdim + c0 + c, a.qkv_kind) : 0.f;
-    }
-  };
-  auto flush = [&](int chunk, int buf) {      // outputs of a finished stage -> global memory
-    const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, T - t0);
-    for (int i = lt; i < nt * cw; i += SCAN_LOADERS) {
-      const int t = i / cw, c = i - t * cw;
-      if (c0 + c < a.vdim)
-        so.o[static_cast<size_t>(row0 + t0 + t) * so.ldo + h * a.vdim + c0 + c] = sout[(buf * SCAN_TC + t) * cw + c];
-    }
-  };
-
-  const int rg = threadIdx.x & (SCAN_RG - 1), col = threadIdx.x >> 3;
-  const bool live = comp && c0 + col < a.vdim;
-  float* sp = a.state + static_cast<size_t>(slot < 0 ? 0 : slot) * a.slot_stride +
-              (static_cast<size_t>(h) * a.vdim + c0 + col) * a.ld_dim;
-  uint64_t S[NR / 2];
 #pragma unroll
-  for (int i = 0; i < NR / 2; ++i) S[i] = 0ull;
-  if (live && slot >= 0 && a.ctx[seq] != T) {
+        for (int b = 0; b < TB; ++b) {
+          const int t = lw + (p + b) * (SCAN_LOADERS / 32), at = buf * SCAN_TC + t;
+          float bsum = 0.f;
 #pragma unroll
-    for (int i = 0; i < NR / 4; ++i) {
-      const int r = i * 32 + rg * 4;
-      if (r < a.ld_dim) {
-        const Pair2 p = *reinterpret_cast<const Pair2*>(sp + r);
-        S[2 * i] = p.lo;
-        S[2 * i + 1] = p.hi;
+          for (int i = 0; i < CH; ++i) {
+            const int c = i * 32 + lane;
+            float q, f, k, bo;
+            scan_gates<MODE>(rq[b][i], MODE == SCAN_WKV ? rk[b][i] : 0.f, rg_[b][i] + bias[i], aux[i], q, f, k, bo);
+            const bool ok = c < a.dim;                  // channels past dim leave the state at zero
+            sq[at * DP + c] = ok ? q : 0.f;
+            sf[at * DP + c] = ok ? f : (MODE == SCAN_HGRN2 ? 1.f : 0.f);
+            if (MODE == SCAN_WKV) {
+              sk[at * DP + c] = ok ? k : 0.f;
+              bsum += ok ? bo : 0.f;
+            }
+          }
+          if (MODE == SCAN_WKV) {
+            bsum = lane_sum(bsum);
+            if (lane == 0) sb[at] = bsum;
+          }
+#pragma unroll
+          for (int i = 0; i < (CW + 31) / 32; ++i)
+            if (i * 32 + lane < CW) sv[at * CW + i * 32 + lane] = rv[b][i];
+        }
       }
+    };
+    auto flush = [&](int chunk, int buf) {      // outputs of a finished stage -> global memory
+      const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, len - t0);
+      for (int i = lt; i < nt * CW; i += SCAN_LOADERS) {
+        const int t = i / CW, c = i % CW;
+        if (c0 + c < a.vdim)
+          so.o[static_cast<size_t>(row0 + t0 + t) * so.ldo + h * a.vdim + c0 + c] = sout[(buf * SCAN_TC + t) * CW + c];
+      }
+    };
+    load(0, 0);
+    stage_barrier();
+    for (int ch = 0; ch < chunks; ++ch) {
+      if (ch + 1 < chunks) load(ch + 1, (ch + 1) & 1);
+      if (ch > 0) flush(ch - 1, (ch - 1) & 1);
+      stage_barrier();
     }
+    flush(chunks - 1, (chunks - 1) & 1);
+    return;
   }
 
-  const int chunks = (T + SCAN_TC - 1) / SCAN_TC;
-  if (!comp) load(0, 0);
-  __syncthreads();
+  // ------------------------------------------------------------------ compute warps
+  const int rg = threadIdx.x & (SCAN_RG - 1), cg = threadIdx.x >> 3;
+  float* sp = a.state + static_cast<size_t>(slot < 0 ? 0 : slot) * a.slot_stride + static_cast<size_t>(h) * a.vdim * a.ld_dim;
+  const bool resume = slot >= 0 && a.ctx[seq] != len;
+  const uint64_t minus1 = pack2(-1.f, -1.f);
+  uint64_t S[CPT][NR / 2];
+#pragma unroll
+  for (int j = 0; j < CPT; ++j)
+#pragma unroll
+    for (int i = 0; i < NR / 4; ++i) {
+      const int r = i * 32 + rg * 4, c = c0 + cg + 16 * j;
+      Pair2 p{0ull, 0ull};
+      if (resume && r < a.ld_dim && c < a.vdim) p = *reinterpret_cast<const Pair2*>(sp + static_cast<size_t>(c) * a.ld_dim + r);
+      S[j][2 * i] = p.lo;
+      S[j][2 * i + 1] = p.hi;
+    }
+  stage_barrier();
   for (int ch = 0; ch < chunks; ++ch) {
-    const int buf = ch & 1;
-    if (comp) {
-      const int nt = min(SCAN_TC, T - ch * SCAN_TC);
+    const int buf = ch & 1, nt = min(SCAN_TC, len - ch * SCAN_TC);
 #pragma unroll 1
-      for (int t8 = 0; t8 < nt; t8 += 8) {
-        float part[8];
+    for (int t4 = 0; t4 < nt; t4 += 4) {
+      float part[CPT][4];
 #pragma unroll
-        for (int t = 0; t < 8; ++t) {
-          part[t] = 0.f;
-          if (t8 + t < nt) {                       // uniform for the CTA
-            const int at = buf * SCAN_TC + t8 + t;
-            const float v = sv[at * cw + col];
-            const float* qp = sq + at * DP + rg * 4;
-            const float* fp = sf + at * DP + rg * 4;
-            const float* kp = sk + at * DP + rg * 4;
-            const uint64_t v2 = pack2(v, v);
-            uint64_t o0 = 0ull, o1 = 0ull;
+      for (int t = 0; t < 4; ++t) {
 #pragma unroll
-            for (int i = 0; i < NR / 4; ++i) {
-              const Pair2 q = *reinterpret_cast<const Pair2*>(qp + i * 32);
-              const Pair2 f = *reinterpret_cast<const Pair2*>(fp + i * 32);
+        for (int j = 0; j < CPT; ++j) part[j][t] = 0.f;
+        if (t4 + t < nt) {                       // uniform for the CTA
+          const int at = buf * SCAN_TC + t4 + t;
+          const float* qp = sq + at * DP + rg * 4;
+          const float* fp = sf + at * DP + rg * 4;
+          const float* kp = sk + at * DP + rg * 4;
+          uint64_t v2[CPT], o0[CPT], o1[CPT];
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            const float v = sv[at * CW + cg + 16 * j];
+            v2[j] = pack2(v, v);
+            o0[j] = o1[j] = 0ull;
+          }
+#pragma unroll
+          for (int i = 0; i < NR / 4; ++i) {
+            const Pair2 q = *reinterpret_cast<const Pair2*>(qp + i * 32);
+            const Pair2 f = *reinterpret_cast<const Pair2*>(fp + i * 32);
+            Pair2 k{0ull, 0ull};
+            if (MODE == SCAN_WKV) k = *reinterpret_cast<const Pair2*>(kp + i * 32);
+#pragma unroll
+            for (int j = 0; j < CPT; ++j) {
               if (MODE == SCAN_HGRN2) {            // f S + (1 - f) v  =  f (S - v) + v
-                const uint64_t n2 = pack2(-v, -v);
-                S[2 * i] = fma2(f.lo, add2(S[2 * i], n2), v2);
-                S[2 * i + 1] = fma2(f.hi, add2(S[2 * i + 1], n2), v2);
-                o0 = fma2(q.lo, S[2 * i], o0);
-                o1 = fma2(q.hi, S[2 * i + 1], o1);
+                S[j][2 * i] = fma2(f.lo, fma2(v2[j], minus1, S[j][2 * i]), v2[j]);
+                S[j][2 * i + 1] = fma2(f.hi, fma2(v2[j], minus1, S[j][2 * i + 1]), v2[j]);
+                o0[j] = fma2(q.lo, S[j][2 * i], o0[j]);
+                o1[j] = fma2(q.hi, S[j][2 * i + 1], o1[j]);
               } else {
-                const Pair2 k = *reinterpret_cast<const Pair2*>(kp + i * 32);
-                o0 = fma2(q.lo, S[2 * i], o0);
-                o1 = fma2(q.hi, S[2 * i + 1], o1);
-                S[2 * i] = fma2(f.lo, S[2 * i], mul2(k.lo, v2));
-                S[2 * i + 1] = fma2(f.hi, S[2 * i + 1], mul2(k.hi, v2));
+                o0[j] = fma2(q.lo, S[j][2 * i], o0[j]);
+                o1[j] = fma2(q.hi, S[j][2 * i + 1], o1[j]);
+                S[j][2 * i] = fma2(f.lo, S[j][2 * i], mul2(k.lo, v2[j]));
+                S[j][2 * i + 1] = fma2(f.hi, S[j][2 * i + 1], mul2(k.hi, v2[j]));
               }
             }
-            const float2 s = unpack2(add2(o0, o1));
-            part[t] = s.x + s.y;
-            if (MODE == SCAN_WKV && rg == 0) part[t] = fmaf(v, sb[at], part[t]);
+          }
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) {
+            const float2 s = unpack2(add2(o0[j], o1[j]));
+            part[j][t] = s.x + s.y;
+            if (MODE == SCAN_WKV && rg == 0) part[j][t] = fmaf(unpack2(v2[j]).x, sb[at], part[j][t]);
           }
         }
-        // eight partial sums of eight tokens over the eight threads of a column: thread rg ends with token t8 + rg
+      }
+      // four partial sums of four tokens over the eight threads of a column: thread rg ends with token t4 + (rg & 3)
 #pragma unroll
-        for (int half = 4; half >= 1; half >>= 1) {
+      for (int j = 0; j < CPT; ++j) {
+#pragma unroll
+        for (int half = 2; half >= 1; half >>= 1) {
           const bool up = rg & half;
 #pragma unroll
-          for (int j = 0; j < 4; ++j)
-            if (j < half) {
-              const float send = up ? part[j] : part[j + half];
-              const float keep = up ? part[j + half] : part[j];
-              part[j] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+          for (int x = 0; x < 2; ++x)
+            if (x < half) {
+              const float send = up ? part[j][x] : part[j][x + half];
+              const float keep = up ? part[j][x + half] : part[j][x];
+              part[j][x] = keep + __shfl_xor_sync(0xffffffffu, send, half);
             }
         }
-        if (t8 + rg < nt) sout[(buf * SCAN_TC + t8 + rg) * cw + col] = part[0];
+        part[j][0] += __shfl_xor_sync(0xffffffffu, part[j][0], 4);
+        if (rg < 4 && t4 + rg < nt) sout[(buf * SCAN_TC + t4 + rg) * CW + cg + 16 * j] = part[j][0];
       }
-    } else {
-      if (ch + 1 < chunks) load(ch + 1, buf ^ 1);
-      if (ch > 0) flush(ch - 1, buf ^ 1);
     }
-    __syncthreads();
+    stage_barrier();
   }
-  if (!comp) flush(chunks - 1, (chunks - 1) & 1);
-  if (live && slot >= 0) {
+  if (slot >= 0) {
 #pragma unroll
-    for (int i = 0; i < NR / 4; ++i) {
-      const int r = i * 32 + rg * 4;
-      if (r < a.ld_dim) *reinterpret_cast<Pair2*>(sp + r) = Pair2{S[2 * i], S[2 * i + 1]};
-    }
+    for (int j = 0; j < CPT; ++j)
+#pragma unroll
+      for (int i = 0; i < NR / 4; ++i) {
+        const int r = i * 32 + rg * 4, c = c0 + cg + 16 * j;
+        if (r < a.ld_dim && c < a.vdim)
+          *reinterpret_cast<Pair2*>(sp + static_cast<size_t>(c) * a.ld_dim + r) = Pair2{S[j][2 * i], S[j][2 * i + 1]};
+      }
   }
 }
 
@@ -302,11 +352,17 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
   float* base = a.state + static_cast<size_t>(slot < 0 ? 0 : slot) * a.slot_stride + static_cast<size_t>(h) * a.vdim * a.ld_dim;
   float bpart = 0.f;
   for (int i = threadIdx.x; i < DP; i += 256) {
-    float q, f, k, b;
-    scan_channel<MODE>(a, m, h, i, q, f, k, b);
+    float q = 0.f, f = 1.f, k = 0.f, b = 0.f;           // channels past dim leave the state at zero
+    if (i < a.dim) {
+      const int c = h * a.dim + i;
+      const float qr = take1(a.q, static_cast<size_t>(m) * a.ldq + c, a.qkv_kind);
+      const float g = take1(a.g, static_cast<size_t>(m) * a.ldg + c, a.g_kind) + a.bias[c];
+      const float kr = MODE == SCAN_WKV ? take1(a.k, static_cast<size_t>(m) * a.ldk + c, a.qkv_kind) : 0.f;
+      scan_gates<MODE>(qr, kr, g, a.aux[c], q, f, k, b);
+    }
     sq[i] = q;
     sf[i] = f;
-    sk[i] = MODE == SCAN_WKV ? k : (i < a.dim ? 1.f - f : 0.f);
+    sk[i] = k;
     bpart += b;
   }
   for (int j = threadIdx.x; j < a.vdim; j += 256) sv[j] = take1(a.v, static_cast<size_t>(m) * a.ldv + h * a.vdim + j, a.qkv_kind);
@@ -359,19 +415,29 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
 // rows per thread for a head of `dim` channels: instantiated multiples of four; 0: too large
 static int scan_rows(int dim) { return dim <= 32 ? 4 : dim <= 64 ? 8 : dim <= 96 ? 12 : dim <= 128 ? 16 : dim <= 192 ? 24 : dim <= 256 ? 32 : 0; }
 
-template <int NR, int MODE>
-static int launch_scan(const ScanArgs& a, const ScanOut& o, int n_seqs, int cw, cudaStream_t st) {
-  const int smem = scan_smem<MODE>(SCAN_RG * NR, cw);
-  static int configured[64] = {0};
+template <int NR, int MODE, int CPT, typename T>
+static int launch_scan_cpt(const ScanArgs& a, const ScanOut& o, int n_seqs, cudaStream_t st) {
+  const int smem = scan_smem<MODE>(SCAN_RG * NR, 16 * CPT);
+  static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (configured[dev & 63] < smem) {
-    cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<NR, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (!configured[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<NR, MODE, CPT, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
-    configured[dev & 63] = smem;
+    configured[dev & 63] = true;
   }
-  const dim3 grid(a.H * ((a.vdim + cw - 1) / cw), n_seqs);
-  return static_cast<int>(launch_kernel(linear_scan_kernel<NR, MODE>, grid, dim3(SCAN_RG * cw + SCAN_LOADERS), smem, st, a, o, cw));
+  const dim3 grid(a.H * ((a.vdim + 16 * CPT - 1) / (16 * CPT)), n_seqs);
+  return static_cast<int>(launch_kernel(linear_scan_kernel<NR, MODE, CPT, T>, grid, dim3(SCAN_RG * 16 + SCAN_LOADERS), smem, st, a, o));
+}
+
+// Columns per thread: wide slices share operand reads and the loaders' work, narrow ones give a small batch more CTAs.
+template <int NR, int MODE>
+static int launch_scan(const ScanArgs& a, const ScanOut& o, int n_seqs, cudaStream_t st) {
+  if (a.qkv_kind == ROW_F32) return launch_scan_cpt<NR, MODE, 1, float>(a, o, n_seqs, st);      // the 32-bit mode
+  const long units = static_cast<long>(n_seqs) * a.H, sms = sm_count();
+  if (a.vdim > 32 && units * ((a.vdim + 63) / 64) >= sms) return launch_scan_cpt<NR, MODE, 4, __nv_bfloat16>(a, o, n_seqs, st);
+  if (a.vdim > 16 && units * ((a.vdim + 31) / 32) >= sms / 2) return launch_scan_cpt<NR, MODE, 2, __nv_bfloat16>(a, o, n_seqs, st);
+  return launch_scan_cpt<NR, MODE, 1, __nv_bfloat16>(a, o, n_seqs, st);
 }
 
 }  // namespace artb
@@ -396,7 +462,7 @@ static bool scan_args_ok(const ScanArgs& a, int mode) {
 }
 
 // Portions of n_seqs sequences (rows cu_q[i] .. cu_q[i + 1] - 1); o fp32 [M, ldo] gets H * vdim columns.
-// Inputs must not be of kind ROW_F32_TAKE (several CTAs read them).
+// q, k, v bf16 or fp32, g fp32; not ROW_F32_TAKE (several CTAs read them).
 ARTB_EXPORT int artb_linear_scan(int mode, void* q, int ldq, void* k, int ldk, void* v, int ldv, int qkv_kind, void* g, int ldg,
                                  int g_kind, const float* bias, const float* aux, float* state, long slot_stride, int ld_dim,
                                  long num_slots, const int* cu_q, const int* ctx, const int* state_slot, int n_seqs, int H,
@@ -404,14 +470,11 @@ ARTB_EXPORT int artb_linear_scan(int mode, void* q, int ldq, void* k, int ldk, v
   if (n_seqs <= 0) return 0;
   const ScanArgs a{q, k, v, g, ldq, ldk, ldv, ldg, qkv_kind, g_kind, bias, aux, state, slot_stride, ld_dim, num_slots, cu_q, ctx,
                    state_slot, H, dim, vdim, status};
-  if (!scan_args_ok(a, mode) || qkv_kind == ROW_F32_TAKE || g_kind == ROW_F32_TAKE || n_seqs > 65535 || ldo < H * vdim)
+  if (!scan_args_ok(a, mode) || qkv_kind == ROW_F32_TAKE || g_kind != ROW_F32 || n_seqs > 65535 || ldo < H * vdim)
     return ERR_BAD_SHAPE;
   const ScanOut so{o, ldo};
-  // column slices: as wide as 32 (the loaders' work is shared by more columns), narrower while CTAs are scarce
-  int cw = vdim <= 8 ? 8 : vdim <= 16 ? 16 : 32;
-  while (cw > 8 && static_cast<long>(n_seqs) * H * ((vdim + cw - 1) / cw) < sm_count() / 2) cw >>= 1;
   const int nr = scan_rows(dim);
-#define ARTB_SC(NR_) return mode == SCAN_WKV ? launch_scan<NR_, SCAN_WKV>(a, so, n_seqs, cw, st) : launch_scan<NR_, SCAN_HGRN2>(a, so, n_seqs, cw, st)
+#define ARTB_SC(NR_) return mode == SCAN_WKV ? launch_scan<NR_, SCAN_WKV>(a, so, n_seqs, st) : launch_scan<NR_, SCAN_HGRN2>(a, so, n_seqs, st)
   ARTB_BY_ROWS(nr, ARTB_SC)
 #undef ARTB_SC
   return 0;

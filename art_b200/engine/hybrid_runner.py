@@ -43,7 +43,7 @@ class Ragged:
     state_slot: torch.Tensor    # int32 [n_seqs]
     bt: torch.Tensor            # int32 [n_seqs, max_blocks]
     single: bool
-    # portions longer than ABSORB_MAX tokens, in row order behind n_abs shorter rows: (sequence, tokens before, tokens)
+    # portions that attend in the expanded form, in row order behind n_abs shorter rows: (sequence, tokens before, tokens)
     portions: list[tuple[int, int, int]] = field(default_factory=list)
     n_abs: int = 0
     reach: int = 0              # upper bound of the tokens a short row may attend to
@@ -59,6 +59,9 @@ class Ragged:
 # Portions up to this many tokens attend in latent space: expanding a window's keys and values for them would cost more
 # than the wider products of the absorbed form.
 ABSORB_MAX = 16
+# Sizes the tensor-core kernels hold in shared memory and registers; beyond them the scalar absorbed form serves.
+LATENT_TC_MAX = 768         # cached row: latent + rotated part
+PREFILL_VALUE_MAX, PREFILL_KEY_MAX = 128, 320
 
 
 class HybridRunner(DeviceRunner):
@@ -73,6 +76,9 @@ class HybridRunner(DeviceRunner):
         self.exact32 = dtype == torch.float32
         self.max_loras = max_loras
         self.dp = pad(cfg.hidden_size)
+        wide = any(s.type == "latent_attention" and (s.vdim > PREFILL_VALUE_MAX or pad(s.dim, 16) + pad(s.rot_dim, 16) > PREFILL_KEY_MAX)
+                   for s in cfg.layers)
+        self.absorb_max = 1 << 30 if self.exact32 or wide else ABSORB_MAX
         self._load(base)
         self._buf: dict = {}
 
@@ -201,7 +207,7 @@ class HybridRunner(DeviceRunner):
         """The batch of the sequences' not-yet-cached tokens and, per sequence, its row range."""
         bs, dev = self.kv.shape[1], self.device
         end = [len(s.tokens) if s.upto is None else min(s.upto, len(s.tokens)) for s in seqs]
-        order = sorted(range(len(seqs)), key=lambda i: end[i] - seqs[i].num_cached > ABSORB_MAX)
+        order = sorted(range(len(seqs)), key=lambda i: end[i] - seqs[i].num_cached > self.absorb_max)
         portions, n_abs, reach = [], 0, 0
         tok, pos, slot, row_seq, cu, ranges = [], [], [], [], [0], [(0, 0)] * len(seqs)
         for j, i in enumerate(order):
@@ -209,7 +215,7 @@ class HybridRunner(DeviceRunner):
             n0, n1 = s.num_cached, end[i]
             if n1 <= n0:
                 raise ValueError("a scheduled sequence brings at least one token")
-            if n1 - n0 <= ABSORB_MAX or self.exact32:
+            if n1 - n0 <= self.absorb_max:
                 n_abs, reach = n_abs + n1 - n0, max(reach, n1)
             else:
                 portions.append((j, n0, n1 - n0))
@@ -268,7 +274,7 @@ class HybridRunner(DeviceRunner):
         if n_abs:
             ql, ol = self._heads_buf("ql", H, n_abs, b, rank_p), self._heads_buf("ol", H, n_abs, b, rank_p)
             hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), n_abs, c_batch=ql.stride(0))
-            if self.exact32:
+            if self.exact32 or rank_p + rot_p > LATENT_TC_MAX:
                 hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs)
             else:
                 keys = min(b.reach, s.window) if s.window > 0 else b.reach
@@ -311,7 +317,13 @@ class HybridRunner(DeviceRunner):
         hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
                           self.cfg.hidden_size, self.cfg.norm_eps)
         y = torch.empty((M, 4 * n), dtype=self.dtype, device=self.device)
-        hy.gemm_batched(mixes[:4], L["rkvg"], y, M, c_batch=n)
+        if M >= 1024 and not self.exact32:      # four products that each fill the machine: CTA-pair tiles
+            from ..ops.gemm import gemm_tn
+
+            for j in range(4):
+                gemm_tn(mixes[j, :M], L["rkvg"][j], out=y[:, j * n:(j + 1) * n])
+        else:
+            hy.gemm_batched(mixes[:4], L["rkvg"], y, M, c_batch=n)
         rp = L["w1"].shape[0]
         z = self._mm_take(b, "w1", mixes[4, :M], L["w1"], f32=True)
         t = torch.empty((M, L["w2"].shape[1]), dtype=self.dtype, device=self.device)
