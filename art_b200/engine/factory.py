@@ -23,6 +23,8 @@ def build_runner(cfg, base: dict[str, torch.Tensor] | None, *, num_blocks: int, 
                  max_loras: int = 4, tp_group=None, decoder=None, use_arena: bool = False):
     """``(runner, cache)`` on ``device``.  ``num_slots`` bounds the sequences that hold recurrent state at once."""
     dev = torch.device(device)
+    if dev.type == "cuda" and dev.index is None:       # the engine's stepping thread selects it by number
+        dev = torch.device("cuda", torch.cuda.current_device())
     if isinstance(cfg, HybridConfig):
         from .hybrid_runner import HybridRunner
 

@@ -5,6 +5,8 @@ Launch one process per GPU of the replica:
     python -m torch.distributed.run --nnodes=1 --nproc-per-node 8 --master-addr 127.0.0.1 \
         -m art_b200.engine.serve_replica --model qwen2.5-32b [--weights /path/to/hf_dir] --port 8000
 
+A hybrid design (``--weights`` with its ``config.json``, or a preset such as ``nikelix-7b``) runs with one process.
+
 Rank 0 runs the HTTP server on a :class:`~art_b200.engine.replica.ReplicaEngine`; the other ranks mirror
 it (``follow()``).  Collectives of the model run over NCCL, the control traffic of the replica over a
 gloo group of the same ranks.  ``--reference`` swaps in the PyTorch reference runner on CPU (gloo only),
@@ -25,36 +27,34 @@ import torch.distributed as dist
 
 def build_replica(args):
     from ..local.tokenizer import load_tokenizer
-    from ..models.config import PRESETS, ModelConfig
+    from ..models.config import ModelConfig, resolve_config
+    from ..models.hybrid import HybridConfig
     from ..models.weights import LoraConfig, init_base_weights, load_base_weights
-    from .kv_cache import BlockManager, KVCache
+    from .factory import build_runner
+    from .kv_cache import BlockManager
     from .replica import ReplicaEngine
 
     rank, world = dist.get_rank(), dist.get_world_size()
-    if args.weights:
-        cfg = ModelConfig.from_hf_dict(__import__("json").load(open(os.path.join(args.weights, "config.json"))),
-                                       name=args.model)
-    else:
-        cfg = PRESETS[args.model]
+    cfg = ModelConfig.from_pretrained_dir(args.weights) if args.weights else resolve_config(args.model)
     lcfg = LoraConfig()
     ctrl = dist.new_group(list(range(world)), backend="gloo")
     bs = args.block_size
     if args.reference:
         from .runner import ReferenceRunner
 
+        if isinstance(cfg, HybridConfig):
+            raise ValueError("hybrid models have no PyTorch reference runner: they are served on a GPU")
         dev = torch.device("cpu")
         base = (load_base_weights(args.weights, cfg, dtype=torch.float32, device=dev) if args.weights
                 else init_base_weights(cfg, seed=args.seed))
         runner, kv = ReferenceRunner(cfg, base, lcfg, max_loras=args.max_loras), None
     else:
-        from .runner import NativeRunner
-
         dev = torch.device("cuda", int(os.environ.get("LOCAL_RANK", rank)))
         base = (load_base_weights(args.weights, cfg, device=dev) if args.weights
                 else init_base_weights(cfg, seed=args.seed, dtype=torch.bfloat16, device=dev))
-        kv = KVCache(cfg.num_layers, args.num_blocks, bs, cfg.num_kv_heads // world, cfg.head_dim, dev)
-        runner = NativeRunner(cfg, lcfg, kv, base=base, max_loras=args.max_loras, device=dev,
-                              tp_group=dist.group.WORLD if world > 1 else None)
+        runner, kv = build_runner(cfg, base, num_blocks=args.num_blocks, block_size=bs, num_slots=args.max_num_seqs, device=dev,
+                                  dtype=getattr(torch, args.dtype), lora_cfg=lcfg, max_loras=args.max_loras,
+                                  tp_group=dist.group.WORLD if world > 1 else None)
         del base
         torch.cuda.empty_cache()
     tok = load_tokenizer(args.tokenizer or args.weights or f"byte-chat:{args.model}", cfg.vocab_size)
@@ -83,8 +83,9 @@ async def _lead(eng, tok, args, dev) -> None:
 
 def main(argv=None) -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("--model", default="qwen2.5-7b", help="architecture preset (or a name for --weights)")
-    ap.add_argument("--weights", default=None, help="Hugging Face directory with config.json and *.safetensors")
+    ap.add_argument("--model", default="qwen2.5-7b", help="architecture preset, hybrid presets included (or a name for --weights)")
+    ap.add_argument("--weights", default=None, help="directory with config.json and *.safetensors (Hugging Face layout or a hybrid design)")
+    ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"], help="float32: hybrid models only")
     ap.add_argument("--tokenizer", default=None)
     ap.add_argument("--served-model-name", default=None)
     ap.add_argument("--lora", action="append", help="name=adapter_dir, repeatable")

@@ -28,6 +28,7 @@ import torch
 
 from .. import dev, types
 from ..models.config import resolve_config
+from ..models.hybrid import HybridConfig
 from ..models.peft_io import is_adapter_dir, load_adapter, save_adapter
 from ..models.weights import LoraConfig, init_base_weights, init_lora, load_base_weights
 from ..utils.get_model_step import get_step_from_dir
@@ -99,7 +100,7 @@ class ModelState:
     def __init__(self, base_model: str, config: dev.InternalModelConfig, output_dir: str, rank: int = 0, world: int = 1,
                  tp: int = 1, master_port: int = 0):
         from ..engine.engine import Engine
-        from ..engine.kv_cache import BlockManager, KVCache
+        from ..engine.kv_cache import BlockManager
         from ..trainer.trainer import Trainer
 
         init_args = config.get("init_args", {})
@@ -147,6 +148,9 @@ class ModelState:
         elif self.group_kind == "pp":    # ... or to hold consecutive blocks of layers
             tp_group, pp_group = None, tp_group
         self.cfg = resolve_config(base_model, init_args.get("architecture"))
+        if isinstance(self.cfg, HybridConfig):
+            raise ValueError(f"{base_model}: hybrid models are served, not trained (python -m art_b200.engine.serve_replica); "
+                             "a model service needs a trainable family")
         self.lora_cfg = LoraConfig(r=int(peft_args.get("r", 8)), alpha=float(peft_args.get("lora_alpha", 16)),
                                    target_modules=tuple(peft_args.get("target_modules", LoraConfig().target_modules)),
                                    use_rslora=bool(peft_args.get("use_rslora", False)))
@@ -195,27 +199,21 @@ class ModelState:
         max_loras = int(engine_args.get("max_loras", 4))
         max_len = int(engine_args.get("max_model_len") or init_args.get("max_seq_length", 32768))
         if self.device.type == "cuda":
-            from ..engine.runner import NativeRunner
+            from ..engine.factory import build_runner, cache_bytes
 
             free, total = torch.cuda.mem_get_info(self.device)
             util = float(engine_args.get("gpu_memory_utilization", init_args.get("gpu_memory_utilization", 0.5)))
-            per_block = KVCache.bytes_per_block(self.cfg.num_layers, block_size, self.cfg.num_kv_heads, self.cfg.head_dim)
+            per_block, _ = cache_bytes(self.cfg, block_size)
             budget = min(free * 0.6, total * util * 0.5)   # leave room for training activations
             num_blocks = int(engine_args.get("num_gpu_blocks_override") or max(64, int(budget // per_block)))
             # sleep mode frees the cache while the trainer runs: the virtual-memory arena keeps every address stable, so
-            # decode graphs captured before a training step stay valid after it
-            sleep_mode = bool(engine_args.get("enable_sleep_mode", False))
-            try:
-                self.kv = KVCache(self.cfg.num_layers, num_blocks, block_size, self.cfg.num_kv_heads, self.cfg.head_dim,
-                                  self.device, use_arena=sleep_mode)
-            except RuntimeError:   # no VMM support: plain tensors; Engine.sleep() then drops the captured graphs
-                self.kv = KVCache(self.cfg.num_layers, num_blocks, block_size, self.cfg.num_kv_heads, self.cfg.head_dim,
-                                  self.device)
-            if tp_group is not None or pp_group is not None:      # the trainer holds a part of the weights: the replica keeps its own full copy
-                runner = NativeRunner(self.cfg, self.lora_cfg, self.kv, base=base, max_loras=max_loras, device=self.device)
-            else:           # trainer and engine share the frozen weights
-                runner = NativeRunner(self.cfg, self.lora_cfg, self.kv, decoder=self.trainer.model, max_loras=max_loras,
-                                      device=self.device)
+            # decode graphs captured before a training step stay valid after it.  The engine shares the trainer's frozen
+            # weights, unless the trainer holds a part of them only: the replica then keeps its own full copy.
+            shared = tp_group is None and pp_group is None
+            runner, self.kv = build_runner(self.cfg, None if shared else base, num_blocks=num_blocks, block_size=block_size,
+                                           device=self.device, lora_cfg=self.lora_cfg, max_loras=max_loras,
+                                           decoder=self.trainer.model if shared else None,
+                                           use_arena=bool(engine_args.get("enable_sleep_mode", False)))
         else:
             from ..engine.runner import ReferenceRunner
 

@@ -182,8 +182,6 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
             w[k] = uni(*shape)
         elif leaf in ("u", "f.b"):
             w[k] = rnd(*shape, std=0.5)
-        elif k == "embed":
-            w[k] = rnd(*shape)
         else:
             w[k] = rnd(*shape, std=shape[-1] ** -0.5)
     return w

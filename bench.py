@@ -66,6 +66,12 @@ def parse_args():
                     help="end-to-end number through the model service (default) or through Trainer.step on pinned rows")
     ap.add_argument("--extra-dp", type=int, default=0,
                     help="after a tensor-parallel run also measure plain data parallelism on the same GPUs (reported as `extra`)")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the headline benchmark: prefill / decode throughput and per-kernel timings of the hybrid "
+                         "decoders beside a dense model of equal size, one JSON line per measurement (one GPU)")
+    ap.add_argument("--hybrid-models", default="nikelix-1b,nikelix-7b")
+    ap.add_argument("--hybrid-batches", default="1,64,256")
+    ap.add_argument("--hybrid-layers", type=int, default=8, help="layers of each preset to run (0: all)")
     return ap.parse_args()
 
 
@@ -166,6 +172,13 @@ def main():
         print(json.dumps({"impl": "reference", "unavailable":
                           "pip install of the reference fails offline: build backend hatchling and the pinned "
                           "unsloth/trl/peft/bitsandbytes/vllm==0.8.5.post1 stack are not in the image or wheelhouse"}))
+        return 0
+
+    if args.hybrid:
+        from art_b200.engine.bench_hybrid import report
+
+        for row in report(args.hybrid_models.split(","), [int(b) for b in args.hybrid_batches.split(",")], args.hybrid_layers):
+            print(json.dumps(row), flush=True)
         return 0
 
     import torch

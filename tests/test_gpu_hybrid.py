@@ -444,3 +444,42 @@ def test_trace_command_line(tmp_path):
             check(got, ref[rows], F32 if dtype == "float32" else BF16)
             (tmp_path / f"{step}.f32").unlink()
     assert sys.executable
+
+
+def test_completion_server_over_a_hybrid_model():
+    """The OpenAI server on the preset engine: chat, logit processing, structured output; adapters are refused."""
+    import asyncio
+
+    import httpx
+
+    from art_b200.engine.factory import build_engine
+    from art_b200.engine.server import OpenAIServer
+    from art_b200.local.tokenizer import ByteChatTokenizer
+    from art_b200.models.config import resolve_config
+    from art_b200.models.weights import init_base_weights
+
+    cfg = resolve_config("nikelix-tiny")
+    tok = ByteChatTokenizer(cfg.vocab_size)
+    eng = build_engine(cfg, init_base_weights(cfg, dtype=BF16, device=DEV), num_blocks=64, max_num_seqs=4, eos_token_id=tok.eos_token_id)
+    eng.start()
+    srv = OpenAIServer(eng, tok, "nikelix-tiny")
+
+    async def main():
+        async with httpx.AsyncClient(transport=httpx.ASGITransport(app=srv.app), base_url="http://t", headers={"Authorization": "Bearer default"}) as c:
+            body = {"model": "nikelix-tiny", "messages": [{"role": "user", "content": "hi"}], "max_tokens": 6, "n": 3, "seed": 1}
+            r = await c.post("/v1/chat/completions", json=body)
+            assert r.status_code == 200 and len(r.json()["choices"]) == 3
+            r = await c.post("/v1/chat/completions", json={**body, "n": 1, "frequency_penalty": 0.5, "top_p": 0.8})
+            assert r.status_code == 200
+            r = await c.post("/v1/chat/completions", json={**body, "n": 1, "guided_choice": ["yes", "no"]})
+            assert r.json()["choices"][0]["message"]["content"] in ("yes", "no")
+
+    try:
+        asyncio.run(asyncio.wait_for(main(), 30))
+        assert eng.error is None
+        with pytest.raises(ValueError, match="adapters"):
+            eng.runner.set_adapter(0, {})
+        assert eng.state_slots.num_free + len(eng.running) == 4
+    finally:
+        eng.shutdown()
+        eng.runner.close()
