@@ -2,7 +2,7 @@
 //
 //   latent_gather_kernel    the cache rows a portion's window reaches, page by page, into one contiguous row range per
 //                           sequence (a GEMM then expands their latents into every head's keys and values)
-//   latent_prefill_kernel   windowed flash attention; a head's key is [ expanded part: dk | rotated part: rot_p ], the
+//   latent_prefill_kernel   windowed flash attention for any sizes (whole 64-column blocks: latent_prefill_tc.cu); a head's key is [ expanded part: dk | rotated part: rot_p ], the
 //                           rotated part coming from the gathered rows all heads share
 //
 // A CTA owns 128 query rows of one sequence and one head: four warps with 32 rows each, key tiles of 32, keys and values
@@ -20,7 +20,8 @@ constexpr int LP_BM = 128, LP_BN = 32, LP_WARPS = 4;
 
 __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, int ldc, const int* __restrict__ block_table, int max_blocks,
                                      int block_size, long num_blocks, const int* __restrict__ seq_of, const int* __restrict__ key_off,
-                                     const int* __restrict__ key_pos0, int n_seqs, __nv_bfloat16* __restrict__ out, int n_keys, int* status) {
+                                     const int* __restrict__ key_pos0, const int* __restrict__ key_cnt, int n_seqs, __nv_bfloat16* __restrict__ out,
+                                     int n_keys, int* status) {
   const int vec = ldc >> 3;
   const long total = static_cast<long>(n_keys) * vec;
   for (long i = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; i < total; i += static_cast<long>(gridDim.x) * blockDim.x) {
@@ -30,6 +31,10 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ cache, in
       const int mid = (lo + hi + 1) >> 1;
       if (key_off[mid] <= r) lo = mid;
       else hi = mid - 1;
+    }
+    if (r - key_off[lo] >= key_cnt[lo]) {      // rows between two sequences
+      *reinterpret_cast<uint4*>(out + static_cast<size_t>(r) * ldc + c) = make_uint4(0, 0, 0, 0);
+      continue;
     }
     const int j = key_pos0[lo] + r - key_off[lo];
     const int blk = block_table[static_cast<size_t>(seq_of[lo]) * max_blocks + j / block_size];
@@ -243,17 +248,17 @@ static int launch_latent_prefill(const LatentPrefill& a, int n_tiles, cudaStream
 using namespace artb;
 typedef __nv_bfloat16 bf16;
 
-// Gathered row r of sequence i (key_off[i] <= r < key_off[i + 1]) is position key_pos0[i] + r - key_off[i] of the
-// sequence seq_of[i] of the block table.
+// Gathered row r of sequence i (key_off[i] <= r < key_off[i] + key_cnt[i]) is position key_pos0[i] + r - key_off[i] of the
+// sequence seq_of[i] of the block table; rows up to the next sequence (or n_keys) are zero.
 ARTB_EXPORT int artb_latent_gather(const void* cache, int ldc, const int* block_table, int max_blocks, int block_size, long num_blocks,
-                                   const int* seq_of, const int* key_off, const int* key_pos0, int n_seqs, void* out, int n_keys,
+                                   const int* seq_of, const int* key_off, const int* key_pos0, const int* key_cnt, int n_seqs, void* out, int n_keys,
                                    int* status, cudaStream_t st) {
   if (n_keys <= 0 || n_seqs <= 0) return 0;
   if ((ldc & 7) || block_size <= 0) return ERR_BAD_SHAPE;
   long blocks = (static_cast<long>(n_keys) * (ldc / 8) + 255) / 256;
   if (blocks > 148L * 16) blocks = 148L * 16;
   latent_gather_kernel<<<static_cast<unsigned>(blocks), 256, 0, st>>>((const bf16*)cache, ldc, block_table, max_blocks, block_size, num_blocks,
-                                                                  seq_of, key_off, key_pos0, n_seqs, (bf16*)out, n_keys, status);
+                                                                  seq_of, key_off, key_pos0, key_cnt, n_seqs, (bf16*)out, n_keys, status);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -194,7 +194,10 @@ def kernel_rows(width: int = 4096, ff: int = 16384, prefill: int = 8192, decode:
             add("latent_gather", phase, lambda: hy.latent_gather(cache, bt, plan), plan.n_keys * ldc * 4)
             kv, o = rnd(plan.n_keys, H * (dk + dv)), torch.empty(M, H * dv, dtype=bf, device=dev)
             pairs = n_seqs * sum(min(i + 1, window) for i in range(2048))
-            add(f"latent_prefill window {window}", phase, lambda: hy.latent_prefill(qe, kv, c, plan, window, 0.07, o, H, dk, dv, rank, rot, dv),
+            k, vt = rnd(plan.n_keys, H * dk), rnd(H * dv, plan.n_keys)
+            add(f"latent_prefill_tc window {window}", phase, lambda: hy.latent_prefill_tc(qe, k, vt, c, plan, window, 0.07, o, H, dk, dv, rank, rot, dv),
+                (qe.numel() + kv.numel() + o.numel()) * 2, 2.0 * H * pairs * (dk + rot + dv))
+            add(f"latent_prefill (any sizes) window {window}", phase, lambda: hy.latent_prefill(qe, kv, c, plan, window, 0.07, o, H, dk, dv, rank, rot, dv),
                 (qe.numel() + kv.numel() + o.numel()) * 2, 2.0 * H * pairs * (dk + rot + dv))
             ids = torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(2048)
             ap = attn_ops.make_plan(ids, ids, M, "native")

@@ -116,7 +116,8 @@ class HybridRunner(DeviceRunner):
             if s.type == "latent_attention":
                 rank_p = pad(s.kv_rank, 16)
                 L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, dp)
-                dk, dv = pad(s.dim, 16), pad(s.vdim, 16)
+                L["tc_dv"] = hy.prefill_tc_values(s.dim, s.rot_dim, s.vdim, s.scale)
+                dk, dv = pad(s.dim, 16), L["tc_dv"] or pad(s.vdim, 16)
                 L["c_norm"] = self._vec(m["dkv.norm"])
                 uk, uv = m["uk"].view(s.heads, s.dim, s.kv_rank), m["uv"].view(s.heads, s.vdim, s.kv_rank)
                 L["uk_t"] = torch.zeros(s.heads, rank_p, pad(s.dim, 16), dtype=self.dtype, device=self.device)
@@ -284,6 +285,10 @@ class HybridRunner(DeviceRunner):
         if n_abs < M:
             plan = b.plan(s.window)
             c = hy.latent_gather(cache, b.bt, plan)
+            if L["tc_dv"]:
+                k, vt = self._mm(c[:, :rank_p], L["ukv"][:H * dk]).t, self._mm(L["ukv"][H * dk:], c[:, :rank_p]).t
+                hy.latent_prefill_tc(qe, k, vt, c, plan, s.window, s.scale, o[n_abs:], H, dk, L["tc_dv"], rank_p, rot_p, s.vdim)
+                return self._mm_take(b, "o", o, L["o"])
             kv = self._mm(c[:, :rank_p], L["ukv"]).t
             hy.latent_prefill(qe, kv, c, plan, s.window, s.scale, o[n_abs:], H, dk, dv, rank_p, rot_p, s.vdim)
         return self._mm_take(b, "o", o, L["o"])

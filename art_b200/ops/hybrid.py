@@ -31,7 +31,9 @@ _sigs = {
                            vp],
     "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
     "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, ci, vp, vp],
-    "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, vp, ci, vp, vp],
+    "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, vp, ci, vp, vp],
+    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, ci, ci,
+                               vp, vp],
     "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, ci, ci, ci, vp],
     "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
     "artb_gemm_f32_tn": [vp, ci, cl, vp, ci, cl, vp, ci, cl, ci, ci, ci, ci, vp],
@@ -211,6 +213,7 @@ class PrefillPlan:
     seq_of: torch.Tensor
     key_off: torch.Tensor
     key_pos0: torch.Tensor
+    key_cnt: torch.Tensor
     row_end: torch.Tensor
     row_pos0: torch.Tensor
     tile_seq: torch.Tensor
@@ -218,15 +221,17 @@ class PrefillPlan:
 
 
 def plan_prefill(portions: list[tuple[int, int, int]], window: int, device) -> PrefillPlan:
-    """``portions``: ``(sequence, tokens before the portion, tokens of the portion)`` in row order."""
-    seq_of, key_off, key_pos0, row_end, row_pos0, tile_seq, tile_row = [], [], [], [], [], [], []
+    """``portions``: ``(sequence, tokens before the portion, tokens of the portion)`` in row order.  Every sequence's
+    gathered keys start at a multiple of 8 rows."""
+    seq_of, key_off, key_pos0, key_cnt, row_end, row_pos0, tile_seq, tile_row = [], [], [], [], [], [], [], []
     row = keys = 0
     for i, (seq, n0, n) in enumerate(portions):
         first = max(0, n0 - window + 1) if window > 0 else 0
         seq_of.append(seq)
         key_off.append(keys)
         key_pos0.append(first)
-        keys += n0 + n - first
+        key_cnt.append(n0 + n - first)
+        keys += pad(n0 + n - first)
         row_pos0.append(n0 - row)
         for r in range(row, row + n, PREFILL_ROWS):
             tile_seq.append(i)
@@ -234,7 +239,7 @@ def plan_prefill(portions: list[tuple[int, int, int]], window: int, device) -> P
         row += n
         row_end.append(row)
     t = lambda v: torch.tensor(v, dtype=torch.int32, device=device)      # noqa: E731
-    return PrefillPlan(keys, len(tile_seq), len(portions), t(seq_of), t(key_off), t(key_pos0), t(row_end), t(row_pos0), t(tile_seq), t(tile_row))
+    return PrefillPlan(keys, len(tile_seq), len(portions), t(seq_of), t(key_off), t(key_pos0), t(key_cnt), t(row_end), t(row_pos0), t(tile_seq), t(tile_row))
 
 
 def latent_gather(cache, block_table, plan: PrefillPlan) -> torch.Tensor:
@@ -242,7 +247,7 @@ def latent_gather(cache, block_table, plan: PrefillPlan) -> torch.Tensor:
     out = torch.empty((plan.n_keys, cache.shape[-1]), dtype=cache.dtype, device=cache.device)
     _lib.check_rc(_f("artb_latent_gather")(
         _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1], cache.shape[0],
-        _lib.ptr(plan.seq_of), _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), plan.n_seqs, _lib.ptr(out), plan.n_keys, _st(cache),
+        _lib.ptr(plan.seq_of), _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), _lib.ptr(plan.key_cnt), plan.n_seqs, _lib.ptr(out), plan.n_keys, _st(cache),
         _lib.stream_ptr()), "latent_gather")
     return out
 
@@ -256,6 +261,24 @@ def latent_prefill(q, kv, c, plan: PrefillPlan, window: int, scale: float, o, H:
         _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0), _lib.ptr(plan.key_off),
         _lib.ptr(plan.key_pos0), window, scale, _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, dk, dv, rot_p, _lib.stream_ptr()),
         "latent_prefill")
+    return o
+
+
+def prefill_tc_values(dim: int, rot: int, vdim: int, scale: float) -> int:
+    """Value columns per head the tcgen05 prefill kernel would use (0: the sizes do not suit it)."""
+    if dim % 64 or rot % 64 or dim + rot > 192 or vdim > 128 or scale <= 0:
+        return 0
+    return 64 if vdim <= 64 else 128
+
+
+def latent_prefill_tc(q, k, vt, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
+                      vdim: int) -> torch.Tensor:
+    """:func:`latent_prefill` on tcgen05: ``k`` [n_keys, H * dk], values transposed ``vt`` [H * dv, n_keys]."""
+    _lib.check_rc(_f("artb_latent_prefill_tc")(
+        _lib.ptr(q), q.stride(0), q.shape[0], _lib.ptr(k), k.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(vt), vt.stride(0),
+        plan.n_keys, _lib.ptr(plan.tile_seq), _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0),
+        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, scale, _lib.ptr(o), o.stride(0), pad(vdim), H, dk, dv, rot_p, _st(o),
+        _lib.stream_ptr()), "latent_prefill_tc")
     return o
 
 

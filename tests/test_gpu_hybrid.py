@@ -82,7 +82,7 @@ def check(got, want, dtype, scale=1.0):
 
 
 LAYERS = {"latent": latent(), "latent-one": latent(heads=1, dim=8, rot=2, rank=8, vdim=8, window=1), "latent-wide": latent(heads=17, dim=40, rot=16, rank=144, vdim=136),
-          "latent-full": latent(heads=2, window=0), "hgrn2": hgrn2(), "hgrn2-one": hgrn2(heads=1, dim=1, vdim=1), "hgrn2-wide": hgrn2(heads=2, dim=130, vdim=100),
+          "latent-blocks": latent(heads=2, dim=64, rot=64, rank=80, vdim=72, window=33), "latent-full": latent(heads=2, window=0), "hgrn2": hgrn2(), "hgrn2-one": hgrn2(heads=1, dim=1, vdim=5), "hgrn2-wide": hgrn2(heads=2, dim=130, vdim=100),
           "wkv": wkv(), "wkv-one": wkv(heads=1, dim=4), "wkv-wide": wkv(heads=2, dim=200), "no-mlp": wkv(ff=0)}
 
 
@@ -90,13 +90,13 @@ LAYERS = {"latent": latent(), "latent-one": latent(heads=1, dim=8, rot=2, rank=8
 @pytest.mark.parametrize("name", list(LAYERS))
 def test_one_layer_prompts_portions_and_decoding(name, dtype):
     d = single_layer(LAYERS[name])
-    toks = tokens(75, 97, 1)
+    toks = tokens(75 if name != "latent-blocks" else 290, 97, 1)
     if name == "latent-full":      # the oracle reads the same dictionary: a window longer than the sequence stands for none
         want = oracle.forward(single_layer(latent(heads=2, window=10 ** 6)), model(d)[1], toks, torch.float64).float()
     else:
         want = want_logits(d, toks)
     rep = session(d, dtype)
-    for cuts in ([75], [1], [40, 1], [2], [17, 2, 33, 3]):
+    for cuts in ([300], [1], [40, 1], [2], [17, 2, 33, 3]):
         check(feed(rep, toks, cuts), want, dtype)
     assert rep.bm.num_free == 64
 
@@ -230,36 +230,49 @@ def test_window_edges_and_page_borders_of_every_attention_form(form, window):
             assert float(err) < (1e-5 if dt == F32 else 2e-2), (p, inside, float(err))
 
 
-def test_prefill_attention_tiles_against_plain_softmax():
-    """Several query tiles, sequences that continue a cached prefix, ragged ends, values narrower than the tile."""
+@pytest.mark.parametrize("H,dk,rot,rank,vdim,window", [(2, 48, 16, 32, 40, 100), (1, 128, 64, 64, 128, 300), (3, 16, 16, 16, 8, 1), (2, 64, 32, 48, 96, 0),
+                                                       (2, 128, 64, 96, 128, 129), (3, 64, 64, 32, 56, 1), (2, 64, 0, 32, 128, 0), (1, 128, 0, 16, 72, 500),
+                                                       (2, 128, 64, 64, 64, 250)])
+def test_prefill_attention_tiles_against_plain_softmax(H, dk, rot, rank, vdim, window):
+    """Several query tiles, sequences that continue a cached prefix, ragged ends, values narrower than the tile; both forms
+    of the kernel where the sizes suit both."""
     from art_b200.ops import hybrid as hy
 
     g = torch.Generator(device=DEV).manual_seed(0)
-    for H, dk, rot, rank, vdim, window in ((2, 48, 16, 32, 40, 100), (1, 128, 64, 64, 128, 300), (3, 16, 16, 16, 8, 1), (2, 64, 32, 48, 96, 0)):
-        dv = hy.pad(vdim, 16)
-        portions = [(1, 0, 130), (0, 77, 257), (2, 300, 20)]
-        plan = hy.plan_prefill(portions, window, DEV)
-        rows = sum(n for _, _, n in portions)
-        rnd = lambda *s: torch.randn(*s, device=DEV, generator=g).to(BF16)      # noqa: E731
-        q, kv, c = rnd(rows, H * (dk + rot)), rnd(plan.n_keys, H * (dk + dv)), rnd(plan.n_keys, rank + rot)
+    dv = hy.pad(vdim, 16)
+    portions = [(1, 0, 130), (0, 77, 257), (2, 300, 20), (3, 1, 17)]
+    plan = hy.plan_prefill(portions, window, DEV)
+    rows = sum(n for _, _, n in portions)
+    rnd = lambda *s: torch.randn(*s, device=DEV, generator=g).to(BF16)      # noqa: E731
+    q, kv, c = 1.5 * rnd(rows, H * (dk + rot)), rnd(plan.n_keys, H * (dk + dv)), rnd(plan.n_keys, rank + rot)
+    outs = []
+    if rot:
         o = torch.zeros(rows, H * hy.pad(vdim), dtype=BF16, device=DEV)
-        hy.latent_prefill(q, kv, c, plan, window, 0.11, o, H, dk, dv, rank, rot, vdim)
-        r0 = 0
-        for i, (_, n0, n) in enumerate(portions):
-            k0, kp = int(plan.key_off[i]), int(plan.key_pos0[i])
-            nk = n0 + n - kp
-            pos, kpos = torch.arange(n0, n0 + n, device=DEV), torch.arange(kp, kp + nk, device=DEV)
-            vis = kpos[None] <= pos[:, None]
-            if window:
-                vis &= kpos[None] > pos[:, None] - window
-            for h in range(H):
-                Q = q[r0:r0 + n, h * (dk + rot):(h + 1) * (dk + rot)].float()
-                K = torch.cat([kv[k0:k0 + nk, h * dk:(h + 1) * dk], c[k0:k0 + nk, rank:]], 1).float()
-                V = kv[k0:k0 + nk, H * dk + h * dv:H * dk + h * dv + vdim].float()
-                ref = torch.softmax((Q @ K.T * 0.11).masked_fill(~vis, float("-inf")), -1) @ V
+        outs.append(hy.latent_prefill(q, kv, c, plan, window, 0.11, o, H, dk, dv, rank, rot, vdim))
+    tdv = hy.prefill_tc_values(dk, rot, vdim, 0.11)
+    assert bool(tdv) == (dk % 64 == 0 and rot % 64 == 0)
+    if tdv:
+        v = torch.zeros(H, tdv, plan.n_keys, dtype=BF16, device=DEV)
+        v[:, :dv] = kv[:, H * dk:].reshape(-1, H, dv).permute(1, 2, 0)
+        o = torch.zeros(rows, H * hy.pad(vdim), dtype=BF16, device=DEV)
+        outs.append(hy.latent_prefill_tc(q, kv[:, :H * dk].contiguous(), v.view(H * tdv, -1), c, plan, window, 0.11, o, H, dk, tdv, rank, rot, vdim))
+    r0 = 0
+    for i, (_, n0, n) in enumerate(portions):
+        k0, kp = int(plan.key_off[i]), int(plan.key_pos0[i])
+        nk = n0 + n - kp
+        pos, kpos = torch.arange(n0, n0 + n, device=DEV), torch.arange(kp, kp + nk, device=DEV)
+        vis = kpos[None] <= pos[:, None]
+        if window:
+            vis &= kpos[None] > pos[:, None] - window
+        for h in range(H):
+            Q = q[r0:r0 + n, h * (dk + rot):(h + 1) * (dk + rot)].float()
+            K = torch.cat([kv[k0:k0 + nk, h * dk:(h + 1) * dk], c[k0:k0 + nk, rank:]], 1).float()
+            V = kv[k0:k0 + nk, H * dk + h * dv:H * dk + h * dv + vdim].float()
+            ref = torch.softmax((Q @ K.T * 0.11).masked_fill(~vis, float("-inf")), -1) @ V
+            for o in outs:
                 got = o[r0:r0 + n, h * hy.pad(vdim):h * hy.pad(vdim) + vdim].float()
-                assert ((got - ref).norm() / ref.norm()).item() < 1e-2
-            r0 += n
+                assert ((got - ref).norm(dim=-1) / ref.norm(dim=-1)).max().item() < 2e-2
+        r0 += n
 
 
 @pytest.mark.parametrize("mode", ["hgrn2", "wkv"])

@@ -271,7 +271,8 @@ def test_prefill_plan_covers_every_row_and_window():
     portions = [(0, 0, 5), (2, 100, 300), (3, 7, 129)]
     plan = plan_prefill(portions, window=33, device="cpu")
     assert plan.key_pos0.tolist() == [0, 68, 0]
-    assert plan.key_off.tolist() == [0, 5, 5 + 332] and plan.n_keys == 5 + 332 + 136
+    assert plan.key_cnt.tolist() == [5, 332, 136]
+    assert plan.key_off.tolist() == [0, 8, 8 + 336] and plan.n_keys == 8 + 336 + 136          # starts at multiples of 8
     assert plan.row_end.tolist() == [5, 305, 434] and plan.row_pos0.tolist() == [0, 95, -298]
     rows = []
     for s, r in zip(plan.tile_seq.tolist(), plan.tile_row.tolist()):
