@@ -42,7 +42,29 @@ struct LatentFinish {
   int* status;
 };
 
-template <typename T>
+// V neighbouring elements at a time (V = 4 when every size and offset allows it)
+template <int V>
+__device__ __forceinline__ void take_v(void* p, size_t off, int kind, float (&f)[V]) {
+  if (V == 4) {
+    const float4 v = take4(p, off, kind);
+    f[0] = v.x, f[1 % V] = v.y, f[2 % V] = v.z, f[3 % V] = v.w;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] = take1(p, off + i, kind);
+  }
+}
+template <typename T, int V>
+__device__ __forceinline__ void put_v(T* p, const float (&f)[V]) {
+  if (V == 4) {
+    st4(p, make_float4(f[0], f[1 % V], f[2 % V], f[3 % V]));
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) st1(p + i, f[i]);
+  }
+}
+
+// W: elements per access of the unrotated parts; RW: of the rotated parts (whole pairs)
+template <typename T, int W, int RW>
 __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a) {
   __shared__ float red[32];
   extern __shared__ float cs[];            // cos, sin of rot / 2 angles
@@ -55,33 +77,50 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
   int slot = a.slot[m];
   if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
   T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
-  // latent: two passes over the row (the second finds it in L1 / L2; a taken workspace is only cleared then)
-  const int c0 = a.H * hq, rkind = a.kind == ROW_F32_TAKE ? ROW_F32 : a.kind;
-  float ss = 0.f;
-  for (int i = tid; i < a.rank; i += blockDim.x) {
-    const float x = take1(a.p, row + c0 + i, rkind);
-    ss += x * x;
-  }
-  const float r = 1.f / sqrtf(cta_sum(ss, red) / a.rank + a.eps);      // also the barrier behind cos / sin
-  for (int i = tid; i < a.rank; i += blockDim.x) {
-    const float x = take1(a.p, row + c0 + i, a.kind);
-    if (slot >= 0) st1(crow + i, x * r * a.w[i]);
-  }
-  for (int i = tid; i < hp; i += blockDim.x) {
-    const float u = take1(a.p, row + c0 + a.rank + 2 * i, a.kind), v = take1(a.p, row + c0 + a.rank + 2 * i + 1, a.kind);
-    if (slot >= 0) {
-      st1(crow + a.rank_p + 2 * i, u * cc[i] - v * sn[i]);
-      st1(crow + a.rank_p + 2 * i + 1, v * cc[i] + u * sn[i]);
-    }
-  }
   const bool absorbed = m < a.n_abs;
   const int he = a.dim_p + a.rot_p;
   T* erow = reinterpret_cast<T*>(a.qe) + static_cast<size_t>(absorbed ? 0 : m - a.n_abs) * a.ldqe;
-  for (int j = tid; j < a.H * a.dim; j += blockDim.x) {
-    const int h = j / a.dim, i = j - h * a.dim;
-    const float x = take1(a.p, row + h * hq + i, a.kind);
-    if (absorbed) st1(reinterpret_cast<T*>(a.qn) + (static_cast<size_t>(h) * a.pitch + m) * a.dim_p + i, x);
-    else st1(erow + h * he + i, x);
+  T* qn = reinterpret_cast<T*>(a.qn) + static_cast<size_t>(m) * a.dim_p;
+  T* qr = reinterpret_cast<T*>(a.qr) + static_cast<size_t>(m) * a.rot_p;
+  // unrotated query parts first: they wait for nothing
+  const int du = a.dim / W;
+  for (int j = tid; j < a.H * du; j += blockDim.x) {
+    const int h = j / du, i = (j - h * du) * W;
+    float x[W];
+    take_v<W>(a.p, row + h * hq + i, a.kind, x);
+    put_v(absorbed ? qn + static_cast<size_t>(h) * a.pitch * a.dim_p + i : erow + h * he + i, x);
+  }
+  // latent: two passes over the row (the second finds it in L1 / L2; a taken workspace is only cleared then)
+  const int c0 = a.H * hq, rkind = a.kind == ROW_F32_TAKE ? ROW_F32 : a.kind;
+  float ss = 0.f;
+  for (int i = tid * W; i < a.rank; i += blockDim.x * W) {
+    float x[W];
+    take_v<W>(a.p, row + c0 + i, rkind, x);
+#pragma unroll
+    for (int e = 0; e < W; ++e) ss += x[e] * x[e];
+  }
+  const float r = 1.f / sqrtf(cta_sum(ss, red) / a.rank + a.eps);      // also the barrier behind cos / sin
+  for (int i = tid * W; i < a.rank; i += blockDim.x * W) {
+    float x[W];
+    take_v<W>(a.p, row + c0 + i, a.kind, x);
+#pragma unroll
+    for (int e = 0; e < W; ++e) x[e] = x[e] * r * a.w[i + e];
+    if (slot >= 0) put_v(crow + i, x);
+  }
+  // rotated parts: heads 0 .. H - 1 of the query, then the shared key part as "head" H
+  const int ru = a.rot / RW;
+  for (int j = tid; j < (a.H + 1) * ru; j += blockDim.x) {
+    const int h = j / ru, i = (j - h * ru) * RW;
+    float x[RW], y[RW];
+    take_v<RW>(a.p, row + (h < a.H ? h * hq + a.dim : c0 + a.rank) + i, a.kind, x);
+#pragma unroll
+    for (int e = 0; e < RW; e += 2) {
+      const float c = cc[(i + e) >> 1], s = sn[(i + e) >> 1];
+      y[e] = x[e] * c - x[e + 1] * s;
+      y[e + 1] = x[e + 1] * c + x[e] * s;
+    }
+    if (h < a.H) put_v(absorbed ? qr + static_cast<size_t>(h) * a.pitch * a.rot_p + i : erow + h * he + a.dim_p + i, y);
+    else if (slot >= 0) put_v(crow + a.rank_p + i, y);
   }
   if (!absorbed) {
     const int np = he - a.dim - a.rot;       // padding columns of a head: behind the first part, behind the rotated part
@@ -89,16 +128,6 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
       const int h = j / np, i = j - h * np;
       st1(erow + h * he + (i < a.dim_p - a.dim ? a.dim + i : a.dim + i + a.rot), 0.f);
     }
-  }
-  for (int j = tid; j < a.H * hp; j += blockDim.x) {
-    const int h = j / hp, i = j - h * hp;
-    const size_t o = row + h * hq + a.dim + 2 * i;
-    const float u = take1(a.p, o, a.kind), v = take1(a.p, o + 1, a.kind);
-    const float x = u * cc[i] - v * sn[i], y = v * cc[i] + u * sn[i];
-    T* d = absorbed ? reinterpret_cast<T*>(a.qr) + (static_cast<size_t>(h) * a.pitch + m) * a.rot_p + 2 * i
-                    : erow + h * he + a.dim_p + 2 * i;
-    st1(d, x);
-    st1(d + 1, y);
   }
 }
 
@@ -214,8 +243,15 @@ ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const fl
   const LatentFinish a{p, ldp, kind, w, inv_freq, pos, slot, cache, ldc, num_slots, n_abs, qn, qr, pitch, qe, ldqe, H, dim, dim_p,
                        rot, rot_p, rank, rank_p, eps, status};
   const size_t smem = static_cast<size_t>(rot) * 4;
-  return static_cast<int>(f32 ? launch_kernel(latent_finish_kernel<float>, dim3(M), dim3(256), smem, st, a)
-                              : launch_kernel(latent_finish_kernel<__nv_bfloat16>, dim3(M), dim3(256), smem, st, a));
+  const bool v4 = !((dim | rot | rank | ldp) & 3) && !(reinterpret_cast<uintptr_t>(p) & 15);
+#define ARTB_LF(T_, W_, R_) return static_cast<int>(launch_kernel(latent_finish_kernel<T_, W_, R_>, dim3(M), dim3(256), smem, st, a))
+  if (f32) {
+    if (v4) ARTB_LF(float, 4, 4);
+    ARTB_LF(float, 1, 2);
+  }
+  if (v4) ARTB_LF(__nv_bfloat16, 4, 4);
+  ARTB_LF(__nv_bfloat16, 1, 2);
+#undef ARTB_LF
 }
 
 ARTB_EXPORT int artb_latent_attend(int f32, const void* ql, const void* qr, int pitch, const void* cache, int ldc,

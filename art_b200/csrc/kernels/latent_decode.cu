@@ -1,7 +1,7 @@
 // Latent attention of single tokens on tensor cores: the absorbed form over the paged latent cache.
 //
 // All heads of a token read the same cache rows [ c: rank_p | rotated part: rot_p ], so the heads are the rows of the
-// matrix products:  S = [q~ | q_rot] [c | k_rot]^T  and  O = P c  per tile of 64 keys, one load of the tile serving both.
+// matrix products:  S = [q~ | q_rot] [c | k_rot]^T  and  O = P c  per tile of 32 or 64 keys, one load serving both.
 // A CTA owns (token, up to 16 * MT heads, a part of the window) and has eight warps.  In the score product a warp takes
 // half of the tile's keys and a quarter of the D channels, so that its query fragments stay in registers and every key
 // element is read from shared memory once; the four partial scores are added in the softmax step, where a warp owns
@@ -18,7 +18,6 @@
 
 namespace artb {
 
-constexpr int LD_KT = 64;          // keys per tile
 constexpr int LD_WARPS = 8;
 
 struct LatentDecode {
@@ -41,12 +40,13 @@ struct LatentDecode {
   int* status;
 };
 
-// NP: pairs of 8-column tiles per warp (128 * NP >= rank_p); KS: 16-channel steps per quarter (64 * KS >= D)
-template <int MT, int NP, int KS>
-__global__ void __launch_bounds__(32 * LD_WARPS, 1) latent_decode_kernel(const LatentDecode a) {
+// NP: pairs of 8-column tiles per warp (128 * NP >= rank_p); KS: 16-channel steps per quarter (64 * KS >= D); LD_KT: keys
+// per tile (32 or 64)
+template <int MT, int NP, int KS, int LD_KT>
+__global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1) latent_decode_kernel(const LatentDecode a) {
   extern __shared__ __align__(16) uint8_t ld_smem[];
   const int D = a.rank_p + a.rot_p, LD = D + 8;
-  constexpr int R = 16 * MT, LP = LD_KT + 8, RPW = R / LD_WARPS;
+  constexpr int R = 16 * MT, LP = LD_KT + 8, RPW = R / LD_WARPS, NK = LD_KT / 32, RT = LD_KT / LD_WARPS;
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(ld_smem);        // [2][KT][LD]
   __nv_bfloat16* sP = sK + 2 * LD_KT * LD;                                // [R][LP]
   float* sS = reinterpret_cast<float*>(sP + R * LP);                      // [4][R][LP]  partial scores
@@ -56,7 +56,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, 1) latent_decode_kernel(const L
 
   pdl_wait();
   pdl_launch_dependents();
-  const int m = blockIdx.x, h0 = blockIdx.y * R, split = blockIdx.z;
+  const int m = blockIdx.y, h0 = blockIdx.x * R, split = blockIdx.z;      // head groups of a token run side by side
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3, jm = lane >> 3, rr = lane & 7;
   const int dq = warp & 3, kh = warp >> 2;
@@ -71,19 +71,21 @@ __global__ void __launch_bounds__(32 * LD_WARPS, 1) latent_decode_kernel(const L
 
   auto load_tile = [&](int tile, int buf) {
     const int k0 = lo + tile * LD_KT;
-#pragma unroll 2
-    for (int i = warp; i < LD_KT; i += LD_WARPS) {       // a warp copies a key's row
-      const int j = k0 + i;
-      bool ok = j < len;
-      size_t s = 0;
-      if (ok) {
+    // the rows of the warp's RT keys, looked up by one lane each
+    int mine = -1;
+    if (lane < RT) {
+      const int j = k0 + warp + lane * LD_WARPS;
+      if (j < len) {
         const int blk = bt[j / a.block_size];
-        ok = index_ok(blk, a.num_blocks, a.status);
-        s = static_cast<size_t>(blk) * a.block_size + j % a.block_size;
+        if (index_ok(blk, a.num_blocks, a.status)) mine = blk * a.block_size + j % a.block_size;
       }
-      const __nv_bfloat16* src = a.cache + (ok ? s * a.ldc : 0);
-      __nv_bfloat16* dst = sK + (buf * LD_KT + i) * LD;
-      for (int c = lane; c < vec; c += 32) copy16_async(dst + c * 8, src + c * 8, ok);
+    }
+#pragma unroll
+    for (int i = 0; i < RT; ++i) {                       // a warp copies a key's row
+      const int row = __shfl_sync(0xffffffffu, mine, i);
+      const __nv_bfloat16* src = a.cache + static_cast<size_t>(max(row, 0)) * a.ldc;
+      __nv_bfloat16* dst = sK + (buf * LD_KT + warp + i * LD_WARPS) * LD;
+      for (int c = lane; c < vec; c += 32) copy16_async(dst + c * 8, src + c * 8, row >= 0);
     }
     copy_commit();
   };
@@ -125,17 +127,17 @@ __global__ void __launch_bounds__(32 * LD_WARPS, 1) latent_decode_kernel(const L
     __syncthreads();                   // the tile has landed and everyone is done with the other buffer
     if (tile + 1 < t_hi) load_tile(tile + 1, buf ^ 1);
     const __nv_bfloat16* K = sK + buf * LD_KT * LD;
-    float s[MT][4][4];
+    float s[MT][2 * NK][4];
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.f;
-    const __nv_bfloat16* kp = K + (kh * 32 + (jm >> 1) * 8 + rr) * LD + ks0 * 16 + (jm & 1) * 8;
+      for (int j = 0; j < 2 * NK; ++j) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.f;
+    const __nv_bfloat16* kp = K + (kh * 16 * NK + (jm >> 1) * 8 + rr) * LD + ks0 * 16 + (jm & 1) * 8;
 #pragma unroll
     for (int k = 0; k < KS; ++k)
       if (k < ks_n) {
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
+        for (int n = 0; n < NK; ++n) {
           uint32_t b[4];
           ldmat_x4(b, kp + n * 16 * LD + k * 16);
 #pragma unroll
@@ -148,36 +150,39 @@ __global__ void __launch_bounds__(32 * LD_WARPS, 1) latent_decode_kernel(const L
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
-      for (int n = 0; n < 4; ++n)
+      for (int n = 0; n < 2 * NK; ++n)
 #pragma unroll
         for (int e = 0; e < 2; ++e)
-          *reinterpret_cast<float2*>(sS + (dq * R + i * 16 + g + 8 * e) * LP + kh * 32 + n * 8 + 2 * t) =
+          *reinterpret_cast<float2*>(sS + (dq * R + i * 16 + g + 8 * e) * LP + kh * 16 * NK + n * 8 + 2 * t) =
               make_float2(s[i][n][2 * e], s[i][n][2 * e + 1]);
     __syncthreads();
 #pragma unroll
     for (int j = 0; j < RPW; ++j) {
       const int row = warp * RPW + j;
-      float2 x = make_float2(0.f, 0.f);
+      float x[NK], mx = mrow[j];
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float2 y = *reinterpret_cast<const float2*>(sS + (q * R + row) * LP + 2 * lane);
-        x.x += y.x;
-        x.y += y.y;
+      for (int k = 0; k < NK; ++k) {
+        const int c = k * 32 + lane;
+        const float* y = sS + row * LP + c;
+        x[k] = ((y[0] + y[R * LP]) + (y[2 * R * LP] + y[3 * R * LP])) * a.scale_log2;
+        if (k0 + c >= len) x[k] = -INFINITY;
+        mx = fmaxf(mx, x[k]);
       }
-      x.x = k0 + 2 * lane < len ? x.x * a.scale_log2 : -INFINITY;
-      x.y = k0 + 2 * lane + 1 < len ? x.y * a.scale_log2 : -INFINITY;
-      float mx = fmaxf(x.x, x.y);
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      mx = fmaxf(mx, mrow[j]);         // finite: a visited tile has at least one key
+      // finite from here on: a visited tile has at least one key
       const float corr = exp2f(mrow[j] - mx);
-      const float p0 = exp2f(x.x - mx), p1 = exp2f(x.y - mx);
-      float sum = p0 + p1;
+      float sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        const float p = exp2f(x[k] - mx);
+        sum += p;
+        sP[row * LP + k * 32 + lane] = __float2bfloat16(p);
+      }
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
       mrow[j] = mx;
       lrow[j] = lrow[j] * corr + sum;
-      *reinterpret_cast<uint32_t*>(sP + row * LP + 2 * lane) = pair_bf16(p0, p1);
       if (lane == 0) sCorr[row] = corr;
     }
     __syncthreads();
@@ -277,23 +282,23 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentDecode a)
   }
 }
 
-static size_t latent_decode_smem(int R, int D) {
-  return 2ull * LD_KT * (D + 8) * 2 + static_cast<size_t>(R) * (LD_KT + 8) * 2 + 4ull * R * (LD_KT + 8) * 4 + 3ull * R * 4;
+static size_t latent_decode_smem(int R, int D, int kt) {
+  return 2ull * kt * (D + 8) * 2 + static_cast<size_t>(R) * (kt + 8) * 2 + 4ull * R * (kt + 8) * 4 + 3ull * R * 4;
 }
 
-template <int MT, int NP, int KS>
+template <int MT, int NP, int KS, int KT>
 static int launch_latent_decode(const LatentDecode& a, int M, cudaStream_t st) {
-  const size_t smem = latent_decode_smem(16 * MT, a.rank_p + a.rot_p);
+  const size_t smem = latent_decode_smem(16 * MT, a.rank_p + a.rot_p, KT);
   if (smem > 226 * 1024) return ERR_TOO_LARGE;
   static size_t configured[64] = {0};
   int dev = 0;
   cudaGetDevice(&dev);
   if (configured[dev & 63] < smem) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, NP, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, NP, KS, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = smem;
   }
-  return static_cast<int>(launch_kernel(latent_decode_kernel<MT, NP, KS>, dim3(M, (a.H + 16 * MT - 1) / (16 * MT), a.splits),
+  return static_cast<int>(launch_kernel(latent_decode_kernel<MT, NP, KS, KT>, dim3((a.H + 16 * MT - 1) / (16 * MT), M, a.splits),
                                         dim3(32 * LD_WARPS), smem, st, a));
 }
 
@@ -317,12 +322,13 @@ ARTB_EXPORT int artb_latent_decode(const void* ql, const void* qr, int pitch, co
                        ctx, window, scale * 1.4426950408889634f, reinterpret_cast<__nv_bfloat16*>(o), ws, splits, H, rank_p, rot_p,
                        status};
   const int D = rank_p + rot_p;
-  const bool wide = H > 16;
+  if (M > 65535) return ERR_BAD_SHAPE;
   int e;
-  if (rank_p <= 128 && D <= 192) e = wide ? launch_latent_decode<2, 1, 3>(a, M, st) : launch_latent_decode<1, 1, 3>(a, M, st);
-  else if (rank_p <= 256 && D <= 320) e = wide ? launch_latent_decode<2, 2, 5>(a, M, st) : launch_latent_decode<1, 2, 5>(a, M, st);
-  else if (rank_p <= 512 && D <= 576) e = wide ? launch_latent_decode<2, 4, 9>(a, M, st) : launch_latent_decode<1, 4, 9>(a, M, st);
-  else if (D <= 1088) e = launch_latent_decode<1, 8, 17>(a, M, st);
+  if (rank_p <= 128 && D <= 192) e = launch_latent_decode<1, 1, 3, 32>(a, M, st);
+  else if (rank_p <= 256 && D <= 320) e = launch_latent_decode<1, 2, 5, 32>(a, M, st);
+  else if (rank_p <= 512 && D <= 576) 
+    e = H > 16 ? launch_latent_decode<2, 4, 9, 64>(a, M, st) : launch_latent_decode<1, 4, 9, 32>(a, M, st);
+  else if (D <= 1088) e = launch_latent_decode<1, 8, 17, 32>(a, M, st);
   else return ERR_TOO_LARGE;
   if (e || splits == 1) return e;
   return static_cast<int>(launch_kernel(latent_merge_kernel, dim3(M, H), dim3(128), 0, st, a));
