@@ -159,12 +159,18 @@ class HybridRunner(DeviceRunner):
             raise ValueError(f"{self.cfg.name}: adapters are not supported for hybrid models")
 
     # -- products and buffers -------------------------------------------------------------------------
+    def _new(self, M: int, n: int, dtype: torch.dtype | None = None) -> torch.Tensor:
+        """An uninitialised [M, n] activation.  The storage of a large batch has its row count rounded up, so that batches
+        of nearly the same size ask the allocator for the same blocks."""
+        return torch.empty((M if M <= 1024 else pad(M, 1024), n), dtype=dtype or self.dtype, device=self.device)[:M]
+
     def _mm(self, x, W, f32: bool = False) -> Out:
+        out = self._new(x.shape[0], W.shape[0], torch.float32 if f32 else None)
         if self.exact32:
-            return as_out(hy.gemm_f32(x, W))
+            return as_out(hy.gemm_f32(x, W, out))
         from ..ops.gemm import gemm_tn
 
-        return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16))
+        return as_out(gemm_tn(x, W, out=out, out_dtype=out.dtype))
 
     def _mm_take(self, b: Ragged, name: str, x, W, f32: bool = False) -> Out:
         """``x W^T`` for a consumer that accepts a split-K workspace: with few rows the product streams the weights from
@@ -239,9 +245,8 @@ class HybridRunner(DeviceRunner):
         operand dtype.  ``capture``: receives a copy of the stream after every layer."""
         cfg, dp, d, eps, m = self.cfg, self.dp, self.cfg.hidden_size, self.cfg.norm_eps, self.cfg.residual_mult
         M, dev = b.M, self.device
-        x = torch.empty((M, dp), dtype=torch.float32, device=dev)
-        h = torch.empty((M, dp), dtype=self.dtype, device=dev)
-        hist = torch.empty((len(self.layers) + 1, M, dp), dtype=torch.float32, device=dev)
+        x, h = self._new(M, dp, torch.float32), self._new(M, dp)
+        hist = torch.empty((len(self.layers) + 1, M if M <= 1024 else pad(M, 1024), dp), dtype=torch.float32, device=dev)
         first_norm = lambda i: (self.layers[i]["norm1"] if cfg.layers[i].type != "wkv" else None) if i < len(self.layers) \
             else (self.final_norm if want_hidden else None)      # noqa: E731  (a token-shift mixer norms its own input)
         hy.residual_step(x, self.embed_norm, d, eps, tokens=b.tokens, table=self.embed, hist=hist, hist_n=0, w_next=first_norm(0), h=h)
@@ -251,7 +256,7 @@ class HybridRunner(DeviceRunner):
             if s.ff:
                 hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
                 z = self._mm_take(b, "up", h, L["up"])
-                a = torch.empty((M, pad(s.ff)), dtype=self.dtype, device=dev)
+                a = self._new(M, pad(s.ff))
                 y = self._mm_take(b, "down", hy.poly_norm(z, L["act"], a, s.ff, eps), L["down"])
                 post = L["norm2b"]
             hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
@@ -268,10 +273,10 @@ class HybridRunner(DeviceRunner):
         if n_abs:
             qn, qr = self._heads_buf("qn", H, n_abs, b, dk), self._heads_buf("qr", H, n_abs, b, rot_p)
         if n_abs < M:
-            qe = torch.empty((M - n_abs, H * (dk + rot_p)), dtype=self.dtype, device=self.device)
+            qe = self._new(M - n_abs, H * (dk + rot_p))
         hy.latent_finish(p, L["c_norm"], L["inv_freq"], b.pos, b.slot, cache, n_abs, qn, qr, qe, H, s.dim, s.rot_dim, s.kv_rank,
                          self.cfg.norm_eps)
-        o = torch.empty((M, H * vp), dtype=self.dtype, device=self.device)
+        o = self._new(M, H * vp)
         if n_abs:
             ql, ol = self._heads_buf("ql", H, n_abs, b, rank_p), self._heads_buf("ol", H, n_abs, b, rank_p)
             hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), n_abs, c_batch=ql.stride(0))
@@ -298,12 +303,12 @@ class HybridRunner(DeviceRunner):
         M, H, vp, eps = b.M, s.heads, pad(s.vdim), self.cfg.norm_eps
         state = self.kv.layers[i]["state"]
         per_head = gate is not None
-        out = torch.empty((M, H * vp), dtype=self.dtype, device=self.device)
+        out = self._new(M, H * vp)
         if b.single:
             hy.linear_decode(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, H, s.dim, s.vdim, L["o_norm"], per_head,
                              gate, out, vp, eps)
         else:
-            o = torch.empty((M, H * s.vdim), dtype=torch.float32, device=self.device)
+            o = self._new(M, H * s.vdim, torch.float32)
             hy.linear_scan(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, H, s.dim, s.vdim, o)
             hy.head_norm(o, L["o_norm"], per_head, H, s.vdim, vp, out, eps, gate)
         return self._mm_take(b, "o", out, L["o"])
@@ -321,7 +326,7 @@ class HybridRunner(DeviceRunner):
         mixes = self._heads_buf("mix", len(SHIFT_MIXES), M, b, self.dp)
         hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
                           self.cfg.hidden_size, self.cfg.norm_eps)
-        y = torch.empty((M, 4 * n), dtype=self.dtype, device=self.device)
+        y = self._new(M, 4 * n)
         if M >= 1024 and not self.exact32:      # four products that each fill the machine: CTA-pair tiles
             from ..ops.gemm import gemm_tn
 
@@ -331,7 +336,7 @@ class HybridRunner(DeviceRunner):
             hy.gemm_batched(mixes[:4], L["rkvg"], y, M, c_batch=n)
         rp = L["w1"].shape[0]
         z = self._mm_take(b, "w1", mixes[4, :M], L["w1"], f32=True)
-        t = torch.empty((M, L["w2"].shape[1]), dtype=self.dtype, device=self.device)
+        t = self._new(M, L["w2"].shape[1])
         g = self._mm(hy.split_tanh(z, s.decay_rank, rp, t), L["w2"], f32=True)
         y = as_out(y)
         return self._scan(hy.SCAN_WKV, i, s, L, y, y.col(n), y.col(2 * n), g, L["u"], L["w0"], y.col(3 * n), b)
@@ -348,7 +353,7 @@ class HybridRunner(DeviceRunner):
         return out
 
     def _hidden_rows(self, x, rows):
-        h = torch.empty((rows.numel(), self.dp), dtype=self.dtype, device=self.device)
+        h = self._new(rows.numel(), self.dp)
         return hy.gather_norm(x, rows, self.final_norm, h, self.cfg.hidden_size, self.cfg.norm_eps)
 
     def score_view(self, view: SeqView, n_prompt: int) -> list[float]:
