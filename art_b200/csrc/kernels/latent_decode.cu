@@ -41,11 +41,13 @@ struct LatentDecode {
 };
 
 // NP: pairs of 8-column tiles per warp (128 * NP >= rank_p); KS: 16-channel steps per quarter (64 * KS >= D); LD_KT: keys
-// per tile (32 or 64)
-template <int MT, int NP, int KS, int LD_KT>
+// per tile (32 or 64); RANK, ROT: the sizes when they are known at compile time (addresses then fold into immediates: with
+// runtime sizes the address arithmetic outnumbers the other instructions), 0: runtime
+template <int MT, int NP, int KS, int LD_KT, int RANK, int ROT>
 __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1) latent_decode_kernel(const LatentDecode a) {
   extern __shared__ __align__(16) uint8_t ld_smem[];
-  const int D = a.rank_p + a.rot_p, LD = D + 8;
+  const int rank_p = RANK ? RANK : a.rank_p, rot_p = RANK ? ROT : a.rot_p;
+  const int D = rank_p + rot_p, LD = D + 8;
   constexpr int R = 16 * MT, LP = LD_KT + 8, RPW = R / LD_WARPS, NK = LD_KT / 32, RT = LD_KT / LD_WARPS;
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(ld_smem);        // [2][KT][LD]
   __nv_bfloat16* sP = sK + 2 * LD_KT * LD;                                // [R][LP]
@@ -85,6 +87,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
       const int row = __shfl_sync(0xffffffffu, mine, i);
       const __nv_bfloat16* src = a.cache + static_cast<size_t>(max(row, 0)) * a.ldc;
       __nv_bfloat16* dst = sK + (buf * LD_KT + warp + i * LD_WARPS) * LD;
+#pragma unroll
       for (int c = lane; c < vec; c += 32) copy16_async(dst + c * 8, src + c * 8, row >= 0);
     }
     copy_commit();
@@ -104,8 +107,8 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
         uint32_t v = 0;
         if (k < ks_n && h < a.H) {
           const size_t row = static_cast<size_t>(h) * a.pitch + m;
-          v = c < a.rank_p ? *reinterpret_cast<const uint32_t*>(a.ql + row * a.rank_p + c)
-                           : *reinterpret_cast<const uint32_t*>(a.qr + row * a.rot_p + (c - a.rank_p));
+          v = c < rank_p ? *reinterpret_cast<const uint32_t*>(a.ql + row * rank_p + c)
+                           : *reinterpret_cast<const uint32_t*>(a.qr + row * rot_p + (c - rank_p));
         }
         qf[i][k][e] = v;
       }
@@ -189,6 +192,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
       const float c0 = sCorr[i * 16 + g], c1 = sCorr[i * 16 + g + 8];
+      if (!__all_sync(0xffffffffu, c0 == 1.f && c1 == 1.f))      // most tiles raise no row's maximum
 #pragma unroll
       for (int j = 0; j < 2 * NP; ++j) {
         acc[i][j][0] *= c0;
@@ -205,7 +209,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
 #pragma unroll
       for (int n = 0; n < NP; ++n) {
         const int col = (warp + n * LD_WARPS) * 16;
-        if (col < a.rank_p) {           // uniform for the warp
+        if (col < rank_p) {           // uniform for the warp
           uint32_t b[4];
           ldmat_x4_t(b, K + (ks * 16 + (jm & 1) * 8 + rr) * LD + col + (jm >> 1) * 8);
 #pragma unroll
@@ -232,12 +236,12 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
       const int r = i * 16 + g + 8 * e, h = h0 + r;
       if (h >= a.H) continue;
       const float l = sL[r], inv = l > 0.f ? 1.f / l : 0.f;
-      float* w = a.ws + ((static_cast<size_t>(m) * a.H + h) * a.splits + split) * (a.rank_p + 2);
-      __nv_bfloat16* o = a.o + (static_cast<size_t>(h) * a.pitch + m) * a.rank_p;
+      float* w = a.ws + ((static_cast<size_t>(m) * a.H + h) * a.splits + split) * (rank_p + 2);
+      __nv_bfloat16* o = a.o + (static_cast<size_t>(h) * a.pitch + m) * rank_p;
 #pragma unroll
       for (int n = 0; n < NP; ++n) {
         const int col = (warp + n * LD_WARPS) * 16;
-        if (col < a.rank_p) {
+        if (col < rank_p) {
 #pragma unroll
           for (int k = 0; k < 2; ++k) {
             const int d = col + k * 8 + 2 * t;
@@ -251,8 +255,8 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
         }
       }
       if (a.splits > 1 && warp == 0 && t == 0) {
-        w[a.rank_p] = sM[r];
-        w[a.rank_p + 1] = l;
+        w[rank_p] = sM[r];
+        w[rank_p + 1] = l;
       }
     }
 }
@@ -286,7 +290,7 @@ static size_t latent_decode_smem(int R, int D, int kt) {
   return 2ull * kt * (D + 8) * 2 + static_cast<size_t>(R) * (kt + 8) * 2 + 4ull * R * (kt + 8) * 4 + 3ull * R * 4;
 }
 
-template <int MT, int NP, int KS, int KT>
+template <int MT, int NP, int KS, int KT, int RANK = 0, int ROT = 0>
 static int launch_latent_decode(const LatentDecode& a, int M, cudaStream_t st) {
   const size_t smem = latent_decode_smem(16 * MT, a.rank_p + a.rot_p, KT);
   if (smem > 226 * 1024) return ERR_TOO_LARGE;
@@ -294,11 +298,11 @@ static int launch_latent_decode(const LatentDecode& a, int M, cudaStream_t st) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (configured[dev & 63] < smem) {
-    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, NP, KS, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<MT, NP, KS, KT, RANK, ROT>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = smem;
   }
-  return static_cast<int>(launch_kernel(latent_decode_kernel<MT, NP, KS, KT>, dim3((a.H + 16 * MT - 1) / (16 * MT), M, a.splits),
+  return static_cast<int>(launch_kernel(latent_decode_kernel<MT, NP, KS, KT, RANK, ROT>, dim3((a.H + 16 * MT - 1) / (16 * MT), M, a.splits),
                                         dim3(32 * LD_WARPS), smem, st, a));
 }
 
@@ -324,7 +328,9 @@ ARTB_EXPORT int artb_latent_decode(const void* ql, const void* qr, int pitch, co
   const int D = rank_p + rot_p;
   if (M > 65535) return ERR_BAD_SHAPE;
   int e;
-  if (rank_p <= 128 && D <= 192) e = launch_latent_decode<1, 1, 3, 32>(a, M, st);
+  if (rank_p == 512 && rot_p == 64)
+    e = H > 16 ? launch_latent_decode<2, 4, 9, 64, 512, 64>(a, M, st) : launch_latent_decode<1, 4, 9, 32, 512, 64>(a, M, st);
+  else if (rank_p <= 128 && D <= 192) e = launch_latent_decode<1, 1, 3, 32>(a, M, st);
   else if (rank_p <= 256 && D <= 320) e = launch_latent_decode<1, 2, 5, 32>(a, M, st);
   else if (rank_p <= 512 && D <= 576) 
     e = H > 16 ? launch_latent_decode<2, 4, 9, 64>(a, M, st) : launch_latent_decode<1, 4, 9, 32>(a, M, st);

@@ -9,7 +9,7 @@
 //
 // Two kernels share the state layout [slot][head][vdim][ld_dim] (a column of S is contiguous):
 //
-//   linear_scan_kernel     portions of prompts.  A CTA owns (sequence, head, a slice of 16, 32 or 64 value columns) and
+//   linear_scan_kernel     portions of prompts.  A CTA owns (sequence, head, a slice of 16 to 128 value columns) and
 //                          walks over the portion.  The state lives in registers: eight threads share one to four
 //                          columns, each with NR of their rows (interleaved in groups of four, so that operands are
 //                          16-byte shared-memory reads without bank conflicts).  Four extra warps load the
@@ -126,13 +126,14 @@ __device__ __forceinline__ void scan_gates(float qr, float kr, float g, float au
 }
 
 // all compute and loader warps; a named barrier because the two roles wait at different places of the code
-__device__ __forceinline__ void stage_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(SCAN_RG * 16 + SCAN_LOADERS) : "memory"); }
+template <int THREADS>
+__device__ __forceinline__ void stage_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
 
-// A CTA's column slice is CW = 16 * CPT wide: thread (rg, cg) holds rows {4 rg + 32 i} of columns {cg + 16 j}.
-template <int NR, int MODE, int CPT, typename T>
-__global__ void __launch_bounds__(SCAN_RG * 16 + SCAN_LOADERS, CPT * NR <= 64 ? 2 : 1)
+// A CTA's column slice is CW = NC * CPT wide: thread (rg, cg) holds rows {4 rg + 32 i} of columns {cg + NC j}.
+template <int NR, int MODE, int CPT, int NC, typename T>
+__global__ void __launch_bounds__(SCAN_RG * NC + SCAN_LOADERS, CPT * NR <= 64 && NC == 16 ? 2 : 1)
 linear_scan_kernel(const ScanArgs a, const ScanOut so) {
-  constexpr int DP = SCAN_RG * NR, CW = 16 * CPT, COMP = SCAN_RG * 16, CH = DP / 32;
+  constexpr int DP = SCAN_RG * NR, CW = NC * CPT, COMP = SCAN_RG * NC, CH = DP / 32;
   extern __shared__ __align__(16) float scan_s[];
   float* sq = scan_s;                                   // [2][TC][DP]
   float* sf = sq + 2 * SCAN_TC * DP;
@@ -153,8 +154,9 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
   if (!comp) {
     // ---------------------------------------------------------------- loader warps: one token per warp at a time
     const int lt = static_cast<int>(threadIdx.x) - COMP, lane = lt & 31, lw = lt >> 5;
-    constexpr int TB = DP <= 96 ? 4 : 2;                // tokens whose raw values are in flight together
+    constexpr int TB = 2;                               // tokens of a warp whose raw values are in flight together
     constexpr int PER = SCAN_TC / (SCAN_LOADERS / 32);  // tokens per warp and stage
+    constexpr int CV = (CW + 31) / 32;
     float bias[CH], aux[CH];
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
@@ -166,55 +168,67 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
     const T* __restrict__ gk = reinterpret_cast<const T*>(a.k) + h * a.dim;
     const T* __restrict__ gv = reinterpret_cast<const T*>(a.v) + h * a.vdim + c0;
     const float* __restrict__ gg = reinterpret_cast<const float*>(a.g) + h * a.dim;
-    auto load = [&](int chunk, int buf) {
+    struct Raw {       // as loaded: converting them here would make the warp wait for them here
+      T q[TB][CH], k[TB][MODE == SCAN_WKV ? CH : 1], v[TB][CV];
+      float g[TB][CH];
+    };
+    const T zero = T(0.f);
+    auto fetch = [&](Raw& r, int chunk, int p) {        // raw values of tokens p, p + 1 of the warp's share of a stage
       const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, len - t0);
-#pragma unroll 1
-      for (int p = 0; p < PER; p += TB) {
-        float rq[TB][CH], rg_[TB][CH], rk[TB][CH], rv[TB][(CW + 31) / 32];
 #pragma unroll
-        for (int b = 0; b < TB; ++b) {
-          const int t = lw + (p + b) * (SCAN_LOADERS / 32);
-          const size_t m = static_cast<size_t>(row0 + t0 + t);
+      for (int b = 0; b < TB; ++b) {
+        const int t = lw + (p + b) * (SCAN_LOADERS / 32);
+        const size_t m = static_cast<size_t>(row0 + t0 + t);
 #pragma unroll
-          for (int i = 0; i < CH; ++i) {
-            const int c = i * 32 + lane;
-            const bool ok = t < nt && c < a.dim;
-            rq[b][i] = ok ? ld1(gq + m * a.ldq + c) : 0.f;
-            rg_[b][i] = ok ? ld1(gg + m * a.ldg + c) : 0.f;
-            if (MODE == SCAN_WKV) rk[b][i] = ok ? ld1(gk + m * a.ldk + c) : 0.f;
-          }
-#pragma unroll
-          for (int i = 0; i < (CW + 31) / 32; ++i) {
-            const int c = i * 32 + lane;
-            rv[b][i] = t < nt && c < CW && c0 + c < a.vdim ? ld1(gv + m * a.ldv + c) : 0.f;
-          }
+        for (int i = 0; i < CH; ++i) {
+          const int c = i * 32 + lane;
+          const bool ok = t < nt && c < a.dim;
+          r.q[b][i] = ok ? gq[m * a.ldq + c] : zero;
+          r.g[b][i] = ok ? gg[m * a.ldg + c] : 0.f;
+          if (MODE == SCAN_WKV) r.k[b][MODE == SCAN_WKV ? i : 0] = ok ? gk[m * a.ldk + c] : zero;
         }
 #pragma unroll
-        for (int b = 0; b < TB; ++b) {
-          const int t = lw + (p + b) * (SCAN_LOADERS / 32), at = buf * SCAN_TC + t;
-          float bsum = 0.f;
-#pragma unroll
-          for (int i = 0; i < CH; ++i) {
-            const int c = i * 32 + lane;
-            float q, f, k, bo;
-            scan_gates<MODE>(rq[b][i], MODE == SCAN_WKV ? rk[b][i] : 0.f, rg_[b][i] + bias[i], aux[i], q, f, k, bo);
-            const bool ok = c < a.dim;                  // channels past dim leave the state at zero
-            sq[at * DP + c] = ok ? q : 0.f;
-            sf[at * DP + c] = ok ? f : (MODE == SCAN_HGRN2 ? 1.f : 0.f);
-            if (MODE == SCAN_WKV) {
-              sk[at * DP + c] = ok ? k : 0.f;
-              bsum += ok ? bo : 0.f;
-            }
-          }
-          if (MODE == SCAN_WKV) {
-            bsum = lane_sum(bsum);
-            if (lane == 0) sb[at] = bsum;
-          }
-#pragma unroll
-          for (int i = 0; i < (CW + 31) / 32; ++i)
-            if (i * 32 + lane < CW) sv[at * CW + i * 32 + lane] = rv[b][i];
+        for (int i = 0; i < CV; ++i) {
+          const int c = i * 32 + lane;
+          r.v[b][i] = t < nt && c < CW && c0 + c < a.vdim ? gv[m * a.ldv + c] : zero;
         }
       }
+    };
+    auto stage = [&](const Raw& r, int buf, int p) {    // gates of those tokens -> shared memory
+#pragma unroll
+      for (int b = 0; b < TB; ++b) {
+        const int at = buf * SCAN_TC + lw + (p + b) * (SCAN_LOADERS / 32);
+        float bsum = 0.f;
+#pragma unroll
+        for (int i = 0; i < CH; ++i) {
+          const int c = i * 32 + lane;
+          float q, f, k, bo;
+          scan_gates<MODE>(ld1(&r.q[b][i]), ld1(&r.k[b][MODE == SCAN_WKV ? i : 0]), r.g[b][i] + bias[i], aux[i], q, f, k, bo);
+          const bool ok = c < a.dim;                    // channels past dim leave the state at zero
+          sq[at * DP + c] = ok ? q : 0.f;
+          sf[at * DP + c] = ok ? f : (MODE == SCAN_HGRN2 ? 1.f : 0.f);
+          if (MODE == SCAN_WKV) {
+            sk[at * DP + c] = ok ? k : 0.f;
+            bsum += ok ? bo : 0.f;
+          }
+        }
+        if (MODE == SCAN_WKV) {
+          bsum = lane_sum(bsum);
+          if (lane == 0) sb[at] = bsum;
+        }
+#pragma unroll
+        for (int i = 0; i < CV; ++i)
+          if (i * 32 + lane < CW) sv[at * CW + i * 32 + lane] = ld1(&r.v[b][i]);
+      }
+    };
+    // two register sets: the next tokens are on their way while the current ones go through their gates
+    Raw ra, rb;
+    auto load = [&](int chunk, int buf) {
+      static_assert(PER == 2 * TB, "two batches per stage");
+      fetch(rb, chunk, TB);
+      stage(ra, buf, 0);
+      if (chunk + 1 < chunks) fetch(ra, chunk + 1, 0);
+      stage(rb, buf, TB);
     };
     auto flush = [&](int chunk, int buf) {      // outputs of a finished stage -> global memory
       const int t0 = chunk * SCAN_TC, nt = min(SCAN_TC, len - t0);
@@ -224,12 +238,13 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
           so.o[static_cast<size_t>(row0 + t0 + t) * so.ldo + h * a.vdim + c0 + c] = sout[(buf * SCAN_TC + t) * CW + c];
       }
     };
+    fetch(ra, 0, 0);
     load(0, 0);
-    stage_barrier();
+    stage_barrier<COMP + SCAN_LOADERS>();
     for (int ch = 0; ch < chunks; ++ch) {
       if (ch + 1 < chunks) load(ch + 1, (ch + 1) & 1);
       if (ch > 0) flush(ch - 1, (ch - 1) & 1);
-      stage_barrier();
+      stage_barrier<COMP + SCAN_LOADERS>();
     }
     flush(chunks - 1, (chunks - 1) & 1);
     return;
@@ -245,13 +260,13 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
   for (int j = 0; j < CPT; ++j)
 #pragma unroll
     for (int i = 0; i < NR / 4; ++i) {
-      const int r = i * 32 + rg * 4, c = c0 + cg + 16 * j;
+      const int r = i * 32 + rg * 4, c = c0 + cg + NC * j;
       Pair2 p{0ull, 0ull};
       if (resume && r < a.ld_dim && c < a.vdim) p = *reinterpret_cast<const Pair2*>(sp + static_cast<size_t>(c) * a.ld_dim + r);
       S[j][2 * i] = p.lo;
       S[j][2 * i + 1] = p.hi;
     }
-  stage_barrier();
+  stage_barrier<COMP + SCAN_LOADERS>();
   for (int ch = 0; ch < chunks; ++ch) {
     const int buf = ch & 1, nt = min(SCAN_TC, len - ch * SCAN_TC);
 #pragma unroll 1
@@ -269,7 +284,7 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
           uint64_t v2[CPT], o0[CPT], o1[CPT];
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
-            const float v = sv[at * CW + cg + 16 * j];
+            const float v = sv[at * CW + cg + NC * j];
             v2[j] = pack2(v, v);
             o0[j] = o1[j] = 0ull;
           }
@@ -317,17 +332,17 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
             }
         }
         part[j][0] += __shfl_xor_sync(0xffffffffu, part[j][0], 4);
-        if (rg < 4 && t4 + rg < nt) sout[(buf * SCAN_TC + t4 + rg) * CW + cg + 16 * j] = part[j][0];
+        if (rg < 4 && t4 + rg < nt) sout[(buf * SCAN_TC + t4 + rg) * CW + cg + NC * j] = part[j][0];
       }
     }
-    stage_barrier();
+    stage_barrier<COMP + SCAN_LOADERS>();
   }
   if (slot >= 0) {
 #pragma unroll
     for (int j = 0; j < CPT; ++j)
 #pragma unroll
       for (int i = 0; i < NR / 4; ++i) {
-        const int r = i * 32 + rg * 4, c = c0 + cg + 16 * j;
+        const int r = i * 32 + rg * 4, c = c0 + cg + NC * j;
         if (r < a.ld_dim && c < a.vdim)
           *reinterpret_cast<Pair2*>(sp + static_cast<size_t>(c) * a.ld_dim + r) = Pair2{S[j][2 * i], S[j][2 * i + 1]};
       }
@@ -415,29 +430,32 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
 // rows per thread for a head of `dim` channels: instantiated multiples of four; 0: too large
 static int scan_rows(int dim) { return dim <= 32 ? 4 : dim <= 64 ? 8 : dim <= 96 ? 12 : dim <= 128 ? 16 : dim <= 192 ? 24 : dim <= 256 ? 32 : 0; }
 
-template <int NR, int MODE, int CPT, typename T>
-static int launch_scan_cpt(const ScanArgs& a, const ScanOut& o, int n_seqs, cudaStream_t st) {
-  const int smem = scan_smem<MODE>(SCAN_RG * NR, 16 * CPT);
+template <int NR, int MODE, int CPT, int NC, typename T>
+static int launch_scan_slices(const ScanArgs& a, const ScanOut& o, int n_seqs, cudaStream_t st) {
+  constexpr int CW = NC * CPT;
+  const int smem = scan_smem<MODE>(SCAN_RG * NR, CW);
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<NR, MODE, CPT, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(linear_scan_kernel<NR, MODE, CPT, NC, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = true;
   }
-  const dim3 grid(a.H * ((a.vdim + 16 * CPT - 1) / (16 * CPT)), n_seqs);
-  return static_cast<int>(launch_kernel(linear_scan_kernel<NR, MODE, CPT, T>, grid, dim3(SCAN_RG * 16 + SCAN_LOADERS), smem, st, a, o));
+  const dim3 grid(a.H * ((a.vdim + CW - 1) / CW), n_seqs);
+  return static_cast<int>(launch_kernel(linear_scan_kernel<NR, MODE, CPT, NC, T>, grid, dim3(SCAN_RG * NC + SCAN_LOADERS), smem, st, a, o));
 }
 
-// Columns per thread: wide slices share operand reads and the loaders' work, narrow ones give a small batch more CTAs.
+// Width of the column slices: wide ones share operand reads and the loaders' work, narrow ones give a small batch more CTAs.
 template <int NR, int MODE>
 static int launch_scan(const ScanArgs& a, const ScanOut& o, int n_seqs, cudaStream_t st) {
-  if (a.qkv_kind == ROW_F32) return launch_scan_cpt<NR, MODE, 1, float>(a, o, n_seqs, st);      // the 32-bit mode
+  if (a.qkv_kind == ROW_F32) return launch_scan_slices<NR, MODE, 1, 16, float>(a, o, n_seqs, st);      // the 32-bit mode
   const long units = static_cast<long>(n_seqs) * a.H, sms = sm_count();
-  if (a.vdim > 32 && units * ((a.vdim + 63) / 64) >= sms) return launch_scan_cpt<NR, MODE, 4, __nv_bfloat16>(a, o, n_seqs, st);
-  if (a.vdim > 16 && units * ((a.vdim + 31) / 32) >= sms / 2) return launch_scan_cpt<NR, MODE, 2, __nv_bfloat16>(a, o, n_seqs, st);
-  return launch_scan_cpt<NR, MODE, 1, __nv_bfloat16>(a, o, n_seqs, st);
+  if (NR <= 16 && a.vdim > 64 && units * ((a.vdim + 127) / 128) >= sms * 3 / 4)
+    return launch_scan_slices<(NR <= 16 ? NR : 16), MODE, 4, 32, __nv_bfloat16>(a, o, n_seqs, st);
+  if (a.vdim > 32 && units * ((a.vdim + 63) / 64) >= sms) return launch_scan_slices<NR, MODE, 4, 16, __nv_bfloat16>(a, o, n_seqs, st);
+  if (a.vdim > 16 && units * ((a.vdim + 31) / 32) >= sms / 2) return launch_scan_slices<NR, MODE, 2, 16, __nv_bfloat16>(a, o, n_seqs, st);
+  return launch_scan_slices<NR, MODE, 1, 16, __nv_bfloat16>(a, o, n_seqs, st);
 }
 
 }  // namespace artb
