@@ -15,6 +15,14 @@ __device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_gr
 template <int N>
 __device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+// bytes global -> shared (both 16-byte aligned, a multiple of 16), completion counted on an mbarrier
+__device__ __forceinline__ void bulk_load(void* smem, const void* gmem, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                   static_cast<uint32_t>(__cvta_generic_to_shared(smem))),
+               "l"(gmem), "r"(bytes), "r"(static_cast<uint32_t>(__cvta_generic_to_shared(bar)))
+               : "memory");
+}
+
 __device__ __forceinline__ void ldmat_x4(uint32_t (&r)[4], const void* p) {
   const uint32_t s = static_cast<uint32_t>(__cvta_generic_to_shared(p));
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(s));

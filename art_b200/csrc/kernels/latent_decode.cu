@@ -6,7 +6,7 @@
 // half of the tile's keys and a quarter of the D channels, so that its query fragments stay in registers and every key
 // element is read from shared memory once; the four partial scores are added in the softmax step, where a warp owns
 // 2 * MT rows.  In the value product a warp takes a share of the latent columns (16 at a time, strided by eight warps).
-// Tiles are double-buffered with asynchronous copies; scores, softmax and accumulators are fp32.
+// Tiles are double-buffered with bulk copies (one per key row); scores, softmax and accumulators are fp32.
 //
 // With several splits the partial (output, max, sum) triples go to a workspace and latent_merge_kernel combines them: a
 // small batch then still covers the machine, although a window has few tiles.
@@ -48,13 +48,14 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
   extern __shared__ __align__(16) uint8_t ld_smem[];
   const int rank_p = RANK ? RANK : a.rank_p, rot_p = RANK ? ROT : a.rot_p;
   const int D = rank_p + rot_p, LD = D + 8;
-  constexpr int R = 16 * MT, LP = LD_KT + 8, RPW = R / LD_WARPS, NK = LD_KT / 32, RT = LD_KT / LD_WARPS;
+  constexpr int R = 16 * MT, LP = LD_KT + 8, RPW = R / LD_WARPS, NK = LD_KT / 32;
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(ld_smem);        // [2][KT][LD]
   __nv_bfloat16* sP = sK + 2 * LD_KT * LD;                                // [R][LP]
   float* sS = reinterpret_cast<float*>(sP + R * LP);                      // [4][R][LP]  partial scores
   float* sCorr = sS + 4 * R * LP;                                         // [R] rescaling of the accumulators
   float* sM = sCorr + R;                                                  // [R] final maximum
   float* sL = sM + R;                                                     // [R] final sum
+  __shared__ uint64_t full[2];
 
   pdl_wait();
   pdl_launch_dependents();
@@ -68,32 +69,37 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
   const int tiles = len > lo ? (len - lo + LD_KT - 1) / LD_KT : 0;
   const int per = (tiles + a.splits - 1) / a.splits;
   const int t_lo = split * per, t_hi = min(tiles, t_lo + per);
-  const int vec = D >> 3;
   const int* bt = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
 
+  // A tile arrives as one bulk copy per key row, completion on the buffer's mbarrier; every warp issues an eighth of the
+  // copies (a warp issues them one by one).  The rows are looked up in the block table one tile ahead, so that the copies
+  // wait for nothing.  Keys past the end repeat the last one (finite values; their scores are masked).
+  constexpr int PW = LD_KT / LD_WARPS;
+  int blk = 0;
+  auto key_of = [&](int tile) { return min(lo + tile * LD_KT + warp * PW + lane, len - 1); };
+  auto look_up = [&](int tile) {
+    if (lane < PW) blk = bt[key_of(tile) / a.block_size];
+  };
   auto load_tile = [&](int tile, int buf) {
-    const int k0 = lo + tile * LD_KT;
-    // the rows of the warp's RT keys, looked up by one lane each
-    int mine = -1;
-    if (lane < RT) {
-      const int j = k0 + warp + lane * LD_WARPS;
-      if (j < len) {
-        const int blk = bt[j / a.block_size];
-        if (index_ok(blk, a.num_blocks, a.status)) mine = blk * a.block_size + j % a.block_size;
-      }
+    if (lane < PW) {
+      size_t row = 0;
+      if (index_ok(blk, a.num_blocks, a.status)) row = static_cast<size_t>(blk) * a.block_size + key_of(tile) % a.block_size;
+      bulk_load(sK + (buf * LD_KT + warp * PW + lane) * LD, a.cache + row * a.ldc, D * 2, &full[buf]);
     }
-#pragma unroll
-    for (int i = 0; i < RT; ++i) {                       // a warp copies a key's row
-      const int row = __shfl_sync(0xffffffffu, mine, i);
-      const __nv_bfloat16* src = a.cache + static_cast<size_t>(max(row, 0)) * a.ldc;
-      __nv_bfloat16* dst = sK + (buf * LD_KT + warp + i * LD_WARPS) * LD;
-#pragma unroll
-      for (int c = lane; c < vec; c += 32) copy16_async(dst + c * 8, src + c * 8, row >= 0);
-    }
-    copy_commit();
   };
 
-  if (t_lo < t_hi) load_tile(t_lo, 0);
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    fence_mbar_init();
+    if (t_lo < t_hi) mbar_expect_tx(&full[0], LD_KT * D * 2);
+  }
+  __syncthreads();
+  if (t_lo < t_hi) {
+    look_up(t_lo);
+    load_tile(t_lo, 0);
+    look_up(t_lo + 1);
+  }
   // query fragments of this warp's channels: steps dq * KS .. of the concatenated [q~ | q_rot]
   const int ks0 = dq * KS, ks_n = min(KS, (D >> 4) - ks0);              // may be <= 0 for the last quarters
   uint32_t qf[MT][KS][4];
@@ -126,9 +132,17 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
 
   for (int tile = t_lo; tile < t_hi; ++tile) {
     const int buf = (tile - t_lo) & 1, k0 = lo + tile * LD_KT;
-    copy_wait<0>();
-    __syncthreads();                   // the tile has landed and everyone is done with the other buffer
-    if (tile + 1 < t_hi) load_tile(tile + 1, buf ^ 1);
+    const bool landed = mbar_wait(&full[buf], ((tile - t_lo) >> 1) & 1);
+    if (!__syncthreads_and(landed)) {  // also: everyone is done with the other buffer
+      if (tid == 0) atomicMax(a.status, ST_TIMEOUT_FULL);
+      for (int i = 0; i < 2000; ++i) __nanosleep(1000);      // let a copy in flight land before shared memory is released
+      return;                          // the same for every thread
+    }
+    if (tile + 1 < t_hi) {
+      if (tid == 0) mbar_expect_tx(&full[buf ^ 1], LD_KT * D * 2);
+      load_tile(tile + 1, buf ^ 1);
+      look_up(tile + 2);
+    }
     const __nv_bfloat16* K = sK + buf * LD_KT * LD;
     float s[MT][2 * NK][4];
 #pragma unroll
