@@ -110,6 +110,21 @@ __device__ __forceinline__ bool mbar_wait_abortable(uint64_t* bar, uint32_t pari
   }
 }
 
+// Bounded wait by wall time for kernels whose waits depend on nothing outside the CTA: a poll may suspend the thread for a
+// while, so that a limit on the number of polls says little about the time.
+__device__ __forceinline__ bool mbar_wait_timed(uint64_t* bar, uint32_t parity, uint64_t budget_ms = 2000) {
+  uint64_t t0 = 0;
+  for (uint32_t i = 0;; ++i) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if ((i & 63u) == 63u) {
+      uint64_t now;
+      asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(now));
+      if (t0 == 0) t0 = now;
+      if (now - t0 > budget_ms * 1000000ull) return false;
+    }
+  }
+}
+
 // ------------------------------------------------------------------------ TMA
 // Tiled 2-D load global -> shared, completion on an mbarrier (transaction bytes).
 // No multicast qualifier anywhere: each CTA fetches its own tiles.

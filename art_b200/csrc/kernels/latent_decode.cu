@@ -132,7 +132,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
 
   for (int tile = t_lo; tile < t_hi; ++tile) {
     const int buf = (tile - t_lo) & 1, k0 = lo + tile * LD_KT;
-    const bool landed = mbar_wait(&full[buf], ((tile - t_lo) >> 1) & 1);
+    const bool landed = mbar_wait_timed(&full[buf], ((tile - t_lo) >> 1) & 1);
     if (!__syncthreads_and(landed)) {  // also: everyone is done with the other buffer
       if (tid == 0) atomicMax(a.status, ST_TIMEOUT_FULL);
       for (int i = 0; i < 2000; ++i) __nanosleep(1000);      // let a copy in flight land before shared memory is released
@@ -143,6 +143,7 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
       load_tile(tile + 1, buf ^ 1);
       look_up(tile + 2);
     }
+    __syncwarp();                      // the matrix loads below are executed by whole warps
     const __nv_bfloat16* K = sK + buf * LD_KT * LD;
     float s[MT][2 * NK][4];
 #pragma unroll

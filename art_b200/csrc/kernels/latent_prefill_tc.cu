@@ -134,7 +134,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       const int nk = a.dk >> 6;
       for (int it = 0; it < tiles && !*abort_flag; ++it) {
         const int s = it & 1, krow = koff + lo_rel + it * LT_B;
-        if (!mbar_wait(&k_empty[s], ((it >> 1) & 1) ^ 1)) {
+        if (!mbar_wait_timed(&k_empty[s], ((it >> 1) & 1) ^ 1)) {
           atomicMax(a.status, ST_TIMEOUT_EMPTY);
           *abort_flag = 1;
           break;
@@ -146,7 +146,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           if (b < nk) tma_load_2d(sk + b * LT_BLK, &tmK, h * a.dk + b * 64, krow, &k_full[s]);
           else tma_load_2d(sk + b * LT_BLK, &tmC, a.rank_p + (b - nk) * 64, krow, &k_full[s]);
         }
-        if (!mbar_wait(v_empty, (it & 1) ^ 1)) {
+        if (!mbar_wait_timed(v_empty, (it & 1) ^ 1)) {
           atomicMax(a.status, ST_TIMEOUT_EMPTY);
           *abort_flag = 1;
           break;
@@ -161,10 +161,10 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(LT_B, LT_B), idesc_o = umma_idesc_bf16(LT_B, DV);
       const uint32_t sq_ = smem_u32(smem + L::Q), sp = smem_u32(smem + L::P), sv = smem_u32(smem + L::V);
-      bool ok = mbar_wait(q_full, 0);
+      bool ok = mbar_wait_timed(q_full, 0);
       auto issue_pv = [&](int i) -> bool {
         const int s = i & 1;
-        if (!mbar_wait(v_full, i & 1) || !mbar_wait(p_full, i & 1) || !mbar_wait(&pv_empty[s], ((i >> 1) & 1) ^ 1)) return false;
+        if (!mbar_wait_timed(v_full, i & 1) || !mbar_wait_timed(p_full, i & 1) || !mbar_wait_timed(&pv_empty[s], ((i >> 1) & 1) ^ 1)) return false;
         tc_fence_after_sync();
         const uint32_t d = tmem + 256 + s * 128;
 #pragma unroll
@@ -180,7 +180,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       for (; it < tiles && ok && !*abort_flag; ++it) {
         const int s = it & 1;
         const uint32_t ph = (it >> 1) & 1;
-        if (!mbar_wait(&k_full[s], ph) || !mbar_wait(&s_empty[s], ph ^ 1)) {
+        if (!mbar_wait_timed(&k_full[s], ph) || !mbar_wait_timed(&s_empty[s], ph ^ 1)) {
           ok = false;
           break;
         }
@@ -232,7 +232,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       slot[hf * 128 + r] = mine;
       __syncwarp();
       if (lane == 0) mbar_arrive(&x_bar[q]);
-      const int okw = mbar_wait(&x_bar[q], xph & 1) ? 1 : 0;
+      const int okw = mbar_wait_timed(&x_bar[q], xph & 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okw)) return false;
       other = slot[(hf ^ 1) * 128 + r];
       ++xph;
@@ -240,7 +240,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     };
     auto add_pv = [&](int i, float ms_i) -> bool {
       const int s = i & 1;
-      const int okw = mbar_wait(&pv_full[s], (i >> 1) & 1) ? 1 : 0;
+      const int okw = mbar_wait_timed(&pv_full[s], (i >> 1) & 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okw)) return false;
       tc_fence_after_sync();
       const float f = lt_ex2(m_o - ms_i);
@@ -267,7 +267,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       const int s = it & 1;
       const int k0 = kp0 + lo_rel + it * LT_B;                         // position of the tile's first key
       const bool inside = k0 + LT_B - 1 <= p0 && (a.window <= 0 || k0 > p0 + LT_B - 1 - a.window);
-      const int okw = mbar_wait(&s_full[s], (it >> 1) & 1) ? 1 : 0;
+      const int okw = mbar_wait_timed(&s_full[s], (it >> 1) & 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okw)) {
         fail(ST_TIMEOUT_TMEM_FULL);
         break;
@@ -308,7 +308,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       l *= lt_ex2(m - ms);
       m = mn;
       // the previous tile's product has left shared memory P free once it was consumed
-      const int okp = mbar_wait(p_empty, (it & 1) ^ 1) ? 1 : 0;
+      const int okp = mbar_wait_timed(p_empty, (it & 1) ^ 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okp)) {
         fail(ST_TIMEOUT_EMPTY);
         break;

@@ -54,8 +54,8 @@ struct ScanArgs {
 };
 
 struct ScanOut {
-  float* o;             // fp32 [M, ldo] (linear_scan_kernel)
-  int ldo;
+  float* o;             // fp32 [rows, ldo] (linear_scan_kernel)
+  int ldo, rows;
 };
 
 struct DecodeOut {
@@ -125,9 +125,14 @@ __device__ __forceinline__ void scan_gates(float qr, float kr, float g, float au
   }
 }
 
-// all compute and loader warps; a named barrier because the two roles wait at different places of the code
+// All compute and loader warps; a named barrier because the two roles wait at different places of the code.  The
+// instruction wants whole warps: lanes that took different ways through the code before it (a store that only some of them
+// do) come together first.
 template <int THREADS>
-__device__ __forceinline__ void stage_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory"); }
+__device__ __forceinline__ void stage_barrier() {
+  __syncwarp();
+  asm volatile("bar.sync 1, %0;" ::"n"(THREADS) : "memory");
+}
 
 // A CTA's column slice is CW = NC * CPT wide: thread (rg, cg) holds rows {4 rg + 32 i} of columns {cg + NC j}.
 template <int NR, int MODE, int CPT, int NC, typename T>
@@ -146,6 +151,10 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
   const int seq = blockIdx.y, h = blockIdx.x % a.H, c0 = (blockIdx.x / a.H) * CW;
   const int row0 = a.cu_q[seq], len = a.cu_q[seq + 1] - row0;
   if (len <= 0) return;
+  if (row0 < 0 || len > so.rows - row0) {      // not a portion of this batch
+    if (threadIdx.x == 0) atomicMax(a.status, ST_BAD_ARGS);
+    return;
+  }
   int slot = a.state_slot[seq];
   if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
   const bool comp = static_cast<int>(threadIdx.x) < COMP;
@@ -479,18 +488,18 @@ static bool scan_args_ok(const ScanArgs& a, int mode) {
          a.cu_q && a.ctx && a.state_slot;
 }
 
-// Portions of n_seqs sequences (rows cu_q[i] .. cu_q[i + 1] - 1); o fp32 [M, ldo] gets H * vdim columns.
+// Portions of n_seqs sequences (rows cu_q[i] .. cu_q[i + 1] - 1); o fp32 [rows, ldo] gets H * vdim columns.
 // q, k, v bf16 or fp32, g fp32; not ROW_F32_TAKE (several CTAs read them).
 ARTB_EXPORT int artb_linear_scan(int mode, void* q, int ldq, void* k, int ldk, void* v, int ldv, int qkv_kind, void* g, int ldg,
                                  int g_kind, const float* bias, const float* aux, float* state, long slot_stride, int ld_dim,
                                  long num_slots, const int* cu_q, const int* ctx, const int* state_slot, int n_seqs, int H,
-                                 int dim, int vdim, float* o, int ldo, int* status, cudaStream_t st) {
+                                 int dim, int vdim, float* o, int ldo, int rows, int* status, cudaStream_t st) {
   if (n_seqs <= 0) return 0;
   const ScanArgs a{q, k, v, g, ldq, ldk, ldv, ldg, qkv_kind, g_kind, bias, aux, state, slot_stride, ld_dim, num_slots, cu_q, ctx,
                    state_slot, H, dim, vdim, status};
   if (!scan_args_ok(a, mode) || qkv_kind == ROW_F32_TAKE || g_kind != ROW_F32 || n_seqs > 65535 || ldo < H * vdim)
     return ERR_BAD_SHAPE;
-  const ScanOut so{o, ldo};
+  const ScanOut so{o, ldo, rows};
   const int nr = scan_rows(dim);
 #define ARTB_SC(NR_) return mode == SCAN_WKV ? launch_scan<NR_, SCAN_WKV>(a, so, n_seqs, st) : launch_scan<NR_, SCAN_HGRN2>(a, so, n_seqs, st)
   ARTB_BY_ROWS(nr, ARTB_SC)

@@ -41,25 +41,21 @@ def dense_twin(cfg):
                        qkv_bias=False, rope_theta=5e5)
 
 
-def engine_rows(names: list[str], batches: list[int], prompt_len: int = 1024, new_tokens: int = 64, layers: int = 0) -> list[dict]:
+def engine_rows(names: list[str], batches: list[int], prompt_len: int = 1024, new_tokens: int = 64, layers: int = 0):
     from ..models.config import resolve_config
     from .bench_decode import measure_decode
 
-    rows = []
     for name in names:
         cfg = resolve_config(name)
         if layers:
             cfg.layers = cfg.layers[:layers]
         for seqs in batches:
-            pair = {}
             for c in (cfg, dense_twin(cfg)):
                 r = measure_decode(c, "cuda", seqs=seqs, prompt_len=prompt_len, new_tokens=new_tokens, loras=0)
-                pair[c.name] = r
                 torch.cuda.empty_cache()
-                rows.append({"model": r["model"], "layers": c.num_layers, "params_b": round(c.num_params() / 1e9, 2), "seqs": seqs,
-                             "prompt_len": prompt_len, "new_tokens": new_tokens, "prefill_tok_s": r["prefill_tok_s"],
-                             "decode_tok_s": r["decode_tok_s"], "decode_ms_per_step": r["decode_ms_per_step"]})
-    return rows
+                yield {"model": r["model"], "layers": c.num_layers, "params_b": round(c.num_params() / 1e9, 2), "seqs": seqs,
+                       "prompt_len": prompt_len, "new_tokens": new_tokens, "prefill_tok_s": r["prefill_tok_s"],
+                       "decode_tok_s": r["decode_tok_s"], "decode_ms_per_step": r["decode_ms_per_step"]}
 
 
 def _time(fn, flush: torch.Tensor, reps: int = 12) -> float:

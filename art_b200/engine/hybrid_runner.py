@@ -66,6 +66,9 @@ PREFILL_VALUE_MAX, PREFILL_KEY_MAX = 128, 320
 
 class HybridRunner(DeviceRunner):
     mixed_steps = True
+    # One-CTA and CTA-pair products follow one another directly here (per-head products in front of an output projection);
+    # with overlapping launches their tensor-memory allocations would meet on an SM.  Full stream order between kernels.
+    overlap_launches = False
 
     def __init__(self, cfg: HybridConfig, kv, base: dict[str, torch.Tensor], *, device="cuda", dtype: torch.dtype = torch.bfloat16,
                  max_loras: int = 0):

@@ -359,6 +359,7 @@ class DeviceRunner:
 
     tp, tp_group, tp_rank = 1, None, 0
     exact32 = False            # operands are fp32 (no bf16 anywhere)
+    overlap_launches = True    # decode kernels may start their prologue while the kernel before them drains
     mixed_steps = False        # prompt portions and single decoded tokens may share one batch
     table_width: int | None = None
 
@@ -516,7 +517,7 @@ class DeviceRunner:
     def _decode_body(self, st, n_steps: int, any_lora: bool, splits: int, ws, restricted: bool = False, procs=None):
         from ..ops import paged
 
-        prev_pdl = paged.set_pdl(os.environ.get("ARTB_PDL", "1") != "0")
+        prev_pdl = paged.set_pdl(self.overlap_launches and os.environ.get("ARTB_PDL", "1") != "0")
         try:
             self._decode_steps(st, n_steps, any_lora, splits, ws, restricted, procs)
         finally:

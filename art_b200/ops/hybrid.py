@@ -24,7 +24,7 @@ _sigs = {
     "artb_split_tanh": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
     "artb_head_norm": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, cf, vp],
     "artb_gather_norm": [ci, vp, ci, vp, ci, vp, vp, ci, ci, ci, cf, cl, vp, vp],
-    "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, vp, vp],
+    "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
     "artb_linear_decode": [ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci,
                            vp, ci, ci, vp, ci, ci, cf, vp, vp],
     "artb_latent_finish": [ci, vp, ci, ci, vp, vp, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
@@ -141,7 +141,8 @@ def linear_scan(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, sta
     """Portions of ``n_seqs`` sequences through the recurrence; ``state`` fp32 ``[slots, H, vdim, ld]``; ``o`` fp32."""
     _lib.check_rc(_f("artb_linear_scan")(
         mode, *_scan_in(mode, q, k, v, g), _lib.ptr(bias), _lib.ptr(aux), _lib.ptr(state), state.stride(0), state.shape[3],
-        state.shape[0], _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, H, dim, vdim, _lib.ptr(o), o.stride(0), _st(o),
+        state.shape[0], _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, H, dim, vdim, _lib.ptr(o), o.stride(0),
+        o.shape[0], _st(o),
         _lib.stream_ptr()), "linear_scan")
     return o
 
