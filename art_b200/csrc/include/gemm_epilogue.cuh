@@ -4,7 +4,9 @@
 
 namespace artb {
 
-enum GemmEpilogue : int { EPI_BF16 = 0, EPI_BF16_RESID = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_SWIGLU_BWD = 4 };
+// EPI_RELUGLU: as EPI_SWIGLU with relu as the gate's activation
+enum GemmEpilogue : int { EPI_BF16 = 0, EPI_BF16_RESID = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_SWIGLU_BWD = 4, EPI_RELUGLU = 5 };
+__host__ __device__ inline bool epi_is_glu(int e) { return e == EPI_SWIGLU || e == EPI_RELUGLU; }
 
 // Tiles are visited with the M index fastest inside bands of group_m tile rows (see raster_tile), so the CTAs that
 // run concurrently share a band of the activation matrix that stays L2-resident and a handful of weight (B) tiles.
@@ -52,7 +54,8 @@ struct SchedSplitK {
 };
 
 // acc (+ bias) (+ residual on the first res_cols columns) -> C as bf16 or fp32; optional SwiGLU
-// output H for gate|up-interleaved columns (blocks of 16).
+// output H for gate|up-interleaved columns (blocks of 16), with relu instead of silu when relu_gate is set; with H given, C
+// may be null (the pre-activation is not stored).
 // swiglu_bwd: acc is d(silu(gate) * up) [M, N]; H holds the forward's gate|up pre-activations [M, 2N] (interleaved in
 // blocks of 16) and C receives d(gate|up) [M, 2N] in the same layout, so the activation gradient never exists in
 // memory as a separate tensor.
@@ -68,6 +71,7 @@ struct EpiStore {
   int out_f32;
   int res_cols;
   int swiglu_bwd = 0;
+  int relu_gate = 0;
   // Global operands of the NEXT 32-column chunk, loaded while the current chunk is converted and stored.
   // Residual (4 pieces): each thread reads its own row.  SwiGLU backward (8 pieces = 128 bytes of gate|up per row):
   // read cooperatively, 8 lanes per row, so that a warp-wide load touches 4 rows x 128 contiguous bytes instead of 32
@@ -217,7 +221,8 @@ struct EpiStore {
       return;
     }
     __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(C) + static_cast<size_t>(gr) * ldc + gc;
-    if (full) {
+    if (!C) {
+    } else if (full) {
 #pragma unroll
       for (int j = 0; j < 32; j += 8) {
         uint4 v;
@@ -243,8 +248,8 @@ struct EpiStore {
         float g1 = __bfloat162float(__float2bfloat16(__uint_as_float(acc[j + 1])));
         float u0 = __bfloat162float(__float2bfloat16(__uint_as_float(acc[16 + j])));
         float u1 = __bfloat162float(__float2bfloat16(__uint_as_float(acc[16 + j + 1])));
-        float h0 = g0 * rcp_approx(1.f + __expf(-g0)) * u0;
-        float h1 = g1 * rcp_approx(1.f + __expf(-g1)) * u1;
+        float h0 = (relu_gate ? fmaxf(g0, 0.f) : g0 * rcp_approx(1.f + __expf(-g0))) * u0;
+        float h1 = (relu_gate ? fmaxf(g1, 0.f) : g1 * rcp_approx(1.f + __expf(-g1))) * u1;
         hv[j >> 1] = pack_bf16x2(h0, h1);
       }
       *reinterpret_cast<uint4*>(h) = make_uint4(hv[0], hv[1], hv[2], hv[3]);

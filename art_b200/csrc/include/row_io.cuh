@@ -8,6 +8,7 @@
 
 namespace artb {
 
+enum GatedAct : int { ACT_SILU = 0, ACT_RELU = 1 };      // act(gate) * up
 enum RowKind : int { ROW_BF16 = 0, ROW_F32 = 1, ROW_F32_TAKE = 2 };
 
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }

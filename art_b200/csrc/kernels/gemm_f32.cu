@@ -1,5 +1,8 @@
 // fp32 GEMM  C_b[m, n] = A_b[m, :] . B_b[n, :]  (+ batch strides), fp32 multiply-adds in K order.
 //
+// With `tile_expert` the rows of A and C are sorted by expert in segments of 128-row tiles and expert e's matrix is the e-th
+// batch member of B; tiles of expert -1 are left alone.
+//
 // The 32-bit mode of the hybrid decoder: a reference for the bf16 kernels on the device, not a fast path, so a plain
 // 64 x 64 register-tiled kernel.  The reduction order of an element depends on nothing but K.
 #include <cuda_runtime.h>
@@ -13,8 +16,13 @@ constexpr int GF_T = 64, GF_K = 16;
 
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ A, int lda, long sa, const float* __restrict__ B, int ldb, long sb, float* __restrict__ C,
-                int ldc, long sc, int M, int N, int K) {
+                int ldc, long sc, int M, int N, int K, const int* __restrict__ tile_expert) {
   __shared__ float As[GF_K][GF_T + 4], Bs[GF_K][GF_T + 4];
+  if (tile_expert) {
+    const int e = tile_expert[blockIdx.y * GF_T / 128];
+    if (e < 0) return;
+    B += e * sb;
+  }
   A += blockIdx.z * sa;
   B += blockIdx.z * sb;
   C += blockIdx.z * sc;
@@ -59,6 +67,16 @@ ARTB_EXPORT int artb_gemm_f32_tn(const float* A, int lda, long sa, const float* 
   if (batch <= 0 || batch > 65535 || M <= 0 || N <= 0 || K <= 0) return ERR_BAD_SHAPE;
   if ((M + GF_T - 1) / GF_T > 65535) return ERR_TOO_LARGE;
   gemm_f32_kernel<<<dim3((N + GF_T - 1) / GF_T, (M + GF_T - 1) / GF_T, batch), 256, 0, stream>>>(A, lda, sa, B, ldb, sb, C, ldc, sc,
-                                                                                              M, N, K);
+                                                                                              M, N, K, nullptr);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// A [m_tiles * 128, K], B [experts * N, K], C [m_tiles * 128, N]; tile_expert int32 [m_tiles]
+ARTB_EXPORT int artb_gemm_f32_grouped_tn(const float* A, int lda, const float* B, int ldb, float* C, int ldc, const int* tile_expert,
+                                         int m_tiles, int N, int K, cudaStream_t stream) {
+  if (m_tiles <= 0 || N <= 0 || K <= 0 || !tile_expert) return ERR_BAD_SHAPE;
+  if (m_tiles * (128 / GF_T) > 65535) return ERR_TOO_LARGE;
+  gemm_f32_kernel<<<dim3((N + GF_T - 1) / GF_T, m_tiles * (128 / GF_T), 1), 256, 0, stream>>>(
+      A, lda, 0, B, ldb, static_cast<long>(N) * ldb, C, ldc, 0, m_tiles * 128, N, K, tile_expert);
   return static_cast<int>(cudaGetLastError());
 }

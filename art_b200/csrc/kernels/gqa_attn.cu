@@ -1,0 +1,525 @@
+// Grouped-query attention over a paged cache with a key mask (window or chunk) and value heads of their own size.
+//
+// A token's cache row is [ keys of the Hkv heads: dk_p each | values of the Hkv heads: dv_p each ], padded with zeros.
+//
+//   gqa_finish_kernel    what follows the q | k | v projection, one CTA per token: biases, cache write, padded queries
+//   gqa_gather_kernel    the cache rows a batch's portions see, contiguous: keys row by row, values transposed, as the
+//                        tcgen05 kernel of latent_prefill_tc.cu wants them (sizes that do not suit it: latent_gather and
+//                        latent_prefill)
+//   gqa_decode_kernel    rows with few new tokens: a CTA owns (row, key head, split); the query heads of the key head are the
+//                        rows of one m16 tile, four warps walk 32-key tiles through their own staging areas
+//   gqa_attend_kernel    the same in scalar fp32 arithmetic, any sizes: the 32-bit mode runs on it
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <math.h>
+#include <stdint.h>
+
+#include "bounds_check.cuh"
+#include "host_utils.h"
+#include "key_mask.cuh"
+#include "mma_tile.cuh"
+#include "row_io.cuh"
+
+namespace artb {
+
+struct GqaFinish {
+  void* p;                  // [M, ldp] of kind `kind`: q (H heads of dim) | k (Hkv heads of dim) | v (Hkv heads of vdim)
+  int ldp, kind;
+  const float* bias;        // fp32 over the same columns, or null
+  const int* slot;          // cache row of every token, < 0: not written
+  void* cache;              // T [num_slots, ldc]
+  int ldc;
+  long num_slots;
+  void* q;                  // T [M, ldq], heads of dk_p
+  int ldq;
+  int H, Hkv, dim, dk_p, vdim, dv_p;
+  int* status;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gqa_finish_kernel(const GqaFinish a) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x;
+  int slot = a.slot[m];
+  if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
+  T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
+  T* qrow = reinterpret_cast<T*>(a.q) + static_cast<size_t>(m) * a.ldq;
+  const int nq = a.H * a.dim, nk = a.Hkv * a.dim, n = nq + nk + a.Hkv * a.vdim;
+  for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
+    float x[V];
+    if (V == 4) {
+      const float4 v = take4(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+      x[0] = v.x, x[1 % V] = v.y, x[2 % V] = v.z, x[3 % V] = v.w;
+    } else {
+      x[0] = take1(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e)
+      if (a.bias) x[e] += a.bias[c + e];
+    T* dst;
+    if (c < nq) {
+      dst = qrow + c / a.dim * a.dk_p + c % a.dim;
+    } else if (slot < 0) {
+      continue;
+    } else if (c < nq + nk) {
+      dst = crow + (c - nq) / a.dim * a.dk_p + (c - nq) % a.dim;
+    } else {
+      dst = crow + a.Hkv * a.dk_p + (c - nq - nk) / a.vdim * a.dv_p + (c - nq - nk) % a.vdim;
+    }
+    if (V == 4) st4(dst, make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]));
+    else st1(dst, x[0]);
+  }
+  const int np = a.dk_p - a.dim;
+  for (int j = threadIdx.x; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
+}
+
+struct GqaGather {
+  const __nv_bfloat16* cache;
+  int ldc;
+  const int* block_table;
+  int max_blocks, block_size;
+  long num_blocks;
+  const int *seq_of, *key_off, *key_pos0, *key_cnt;
+  int n_seqs, n_keys;
+  __nv_bfloat16* k;         // [n_keys, kcols]
+  __nv_bfloat16* vt;        // [vcols, n_keys]
+  int kcols, vcols;         // multiples of 64
+  int* status;
+};
+
+// blockIdx.x: 64 keys; blockIdx.y: 64 columns, the key columns first
+__global__ void __launch_bounds__(256) gqa_gather_kernel(const GqaGather a) {
+  __shared__ long src[64];
+  __shared__ __align__(16) __nv_bfloat16 tile[64][72];
+  const int k0 = blockIdx.x * 64, c0 = blockIdx.y * 64, tid = threadIdx.x;
+  if (tid < 64) {
+    const int r = k0 + tid;
+    long s = -1;
+    if (r < a.n_keys) {
+      int lo = 0, hi = a.n_seqs - 1;
+      while (lo < hi) {
+        const int mid = (lo + hi + 1) >> 1;
+        if (a.key_off[mid] <= r) lo = mid;
+        else hi = mid - 1;
+      }
+      const int i = r - a.key_off[lo];
+      if (i < a.key_cnt[lo]) {
+        const int j = a.key_pos0[lo] + i;
+        const int blk = a.block_table[static_cast<size_t>(a.seq_of[lo]) * a.max_blocks + j / a.block_size];
+        if (index_ok(blk, a.num_blocks, a.status)) s = static_cast<long>(blk) * a.block_size + j % a.block_size;
+      }
+    }
+    src[tid] = s;
+  }
+  __syncthreads();
+  for (int v = tid; v < 512; v += 256) {
+    const int r = v >> 3, c = (v & 7) * 8;
+    const uint4 x = src[r] >= 0 ? *reinterpret_cast<const uint4*>(a.cache + src[r] * a.ldc + c0 + c) : make_uint4(0, 0, 0, 0);
+    if (c0 < a.kcols) {
+      if (k0 + r < a.n_keys) *reinterpret_cast<uint4*>(a.k + static_cast<size_t>(k0 + r) * a.kcols + c0 + c) = x;
+    } else {
+      *reinterpret_cast<uint4*>(&tile[r][c]) = x;
+    }
+  }
+  if (c0 < a.kcols) return;
+  __syncthreads();
+  for (int v = tid; v < 512; v += 256) {
+    const int c = v & 63, r = (v >> 6) * 8;          // eight keys of one column
+    if (k0 + r >= a.n_keys) continue;                // n_keys is a multiple of 8
+    __align__(16) __nv_bfloat16 y[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = tile[r + i][c];
+    *reinterpret_cast<uint4*>(a.vt + static_cast<size_t>(c0 - a.kcols + c) * a.n_keys + k0 + r) = *reinterpret_cast<const uint4*>(y);
+  }
+}
+
+struct GqaAttend {
+  const void* q;            // T [M, ldq], heads of dk_p
+  int ldq;
+  const void* cache;        // T [num_blocks * block_size, ldc]
+  int ldc;
+  const int* block_table;
+  int max_blocks, block_size;
+  long num_blocks;
+  const int* row_seq;
+  const int* pos;
+  const int* ctx;           // tokens of the sequence; 0: padding sequence
+  KeyMask mask;
+  float scale, out_scale;
+  void* o;                  // T [M, ldo], heads of vp; padding columns zero
+  int ldo, vp;
+  float* ws;                // [M][H][splits][dv_p + 2]
+  int splits;
+  int H, Hkv, dk_p, vdim, dv_p;
+  int* status;
+};
+
+constexpr int GD_KT = 32;   // keys per warp tile
+
+template <int DK, int DV>
+constexpr int gqa_decode_smem() { return (16 * (DK + 8) + 4 * GD_KT * (DK + 8 + DV + 8)) * 2 + 2 * 4 * 16 * 4; }
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
+  constexpr int LK = DK + 8, LV = DV + 8, WARP_ELEMS = GD_KT * (LK + LV);
+  static_assert(16 * DV * 4 <= WARP_ELEMS * 2, "a warp's accumulators must fit its staging area");
+  extern __shared__ __align__(16) uint8_t gd_smem[];
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(gd_smem);      // [16][LK]
+  __nv_bfloat16* sKV = sQ + 16 * LK;                                   // [4 warps][keys | values]
+  float* sM = reinterpret_cast<float*>(sKV + 4 * WARP_ELEMS);          // [4][16] maxima, [4][16] sums
+  pdl_wait();
+  pdl_launch_dependents();
+  const int G = a.H / a.Hkv, groups = (G + 15) / 16;
+  const int m = blockIdx.x, hk = blockIdx.y / groups, g0 = (blockIdx.y % groups) * 16, split = blockIdx.z;
+  const int ng = min(16, G - g0), h0 = hk * G + g0;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t = lane & 3, jm = lane >> 3, rr = lane & 7;
+  const int seq = a.row_seq[m], p = a.pos[m];
+  const int len = a.ctx[seq] > 0 ? p + 1 : 0, first = a.mask.first(p);
+  const int* bt = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
+  const int bs_shift = (a.block_size & (a.block_size - 1)) == 0 ? 31 - __clz(a.block_size) : -1;
+  const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(a.q) + static_cast<size_t>(m) * a.ldq;
+
+  for (int v = tid; v < 16 * (DK / 8); v += 128) {
+    const int r = v / (DK / 8), c = (v % (DK / 8)) * 8;
+    uint4 val = make_uint4(0, 0, 0, 0);
+    if (r < ng && c < a.dk_p) val = *reinterpret_cast<const uint4*>(q + (h0 + r) * a.dk_p + c);
+    *reinterpret_cast<uint4*>(sQ + r * LK + c) = val;
+  }
+  __syncthreads();
+  uint32_t qf[DK / 16][4];
+#pragma unroll
+  for (int ks = 0; ks < DK / 16; ++ks) ldmat_x4(qf[ks], sQ + ((jm & 1) * 8 + rr) * LK + ks * 16 + (jm >> 1) * 8);
+
+  // the splits share [first, len) in whole tiles, the warps of a split take its tiles in turn
+  const int tiles = (len - first + GD_KT - 1) / GD_KT, per = (tiles + a.splits - 1) / a.splits;
+  const int tile_hi = min(tiles, (split + 1) * per);
+  float acc[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  __nv_bfloat16 *wK = sKV + warp * WARP_ELEMS, *wV = wK + GD_KT * LK;
+  const float scale_log2 = a.scale * 1.4426950408889634f;
+  const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + hk * a.dk_p;
+  const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + a.Hkv * a.dk_p + hk * a.dv_p;
+
+  for (int tile = split * per + warp; tile < tile_hi; tile += 4) {
+    const int k0 = first + tile * GD_KT;
+    // lane i looks up key i of the tile, the copies take the row from it
+    long my_row = -1;
+    {
+      const int kt = k0 + lane;
+      if (kt < len) {
+        const int blk = bt[bs_shift >= 0 ? kt >> bs_shift : kt / a.block_size];
+        if (index_ok(blk, a.num_blocks, a.status))
+          my_row = static_cast<long>(blk) * a.block_size + (bs_shift >= 0 ? kt & (a.block_size - 1) : kt % a.block_size);
+      }
+    }
+    auto load = [&](__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int width, auto tag) {
+      constexpr int W = decltype(tag)::value, CPR = W / 8, RPI = CPR >= 32 ? 1 : 32 / CPR;
+      const int c = (lane % CPR) * 8;
+#pragma unroll 4
+      for (int r0 = 0; r0 < GD_KT; r0 += RPI) {
+        const int r = r0 + lane / CPR;
+        const long row = __shfl_sync(0xffffffffu, my_row, r);
+        const bool ok = row >= 0 && c < width;
+        copy16_async(dst + r * ld + c, src + (ok ? row * a.ldc + c : 0), ok);
+      }
+    };
+    load(wK, LK, kc, a.dk_p, std::integral_constant<int, DK>());
+    load(wV, LV, vc, a.dv_p, std::integral_constant<int, DV>());
+    copy_commit();
+    copy_wait<0>();
+    __syncwarp();
+    float s[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks)
+#pragma unroll
+      for (int np = 0; np < 2; ++np) {
+        uint32_t b[4];
+        ldmat_x4(b, wK + (np * 16 + (jm >> 1) * 8 + rr) * LK + ks * 16 + (jm & 1) * 8);
+        mma_bf16(s[np * 2], qf[ks], b[0], b[1]);
+        mma_bf16(s[np * 2 + 1], qf[ks], b[2], b[3]);
+      }
+    uint32_t pf[2][4];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float mn = mx[e];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          float& x = s[i][2 * e + j];
+          x = k0 + i * 8 + 2 * t + j < len ? x * scale_log2 : -INFINITY;
+          mn = fmaxf(mn, x);
+        }
+      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
+      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));
+      const float ms = mn == -INFINITY ? 0.f : mn, corr = exp2f(mx[e] - ms);
+      mx[e] = mn;
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float p0 = exp2f(s[i][2 * e] - ms), p1 = exp2f(s[i][2 * e + 1] - ms);
+        sum += p0 + p1;
+        pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(p0, p1);
+      }
+      l[e] = l[e] * corr + sum;
+#pragma unroll
+      for (int i = 0; i < DV / 8; ++i) {
+        acc[i][2 * e] *= corr;
+        acc[i][2 * e + 1] *= corr;
+      }
+    }
+#pragma unroll
+    for (int ks = 0; ks < 2; ++ks)
+#pragma unroll
+      for (int dp = 0; dp < DV / 16; ++dp) {
+        uint32_t b[4];
+        ldmat_x4_t(b, wV + (ks * 16 + (jm & 1) * 8 + rr) * LV + dp * 16 + (jm >> 1) * 8);
+        mma_bf16(acc[dp * 2], pf[ks], b[0], b[1]);
+        mma_bf16(acc[dp * 2 + 1], pf[ks], b[2], b[3]);
+      }
+    __syncwarp();
+  }
+  auto warp_acc = [&](int w) { return reinterpret_cast<float*>(sKV + w * WARP_ELEMS); };
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+    if (t == 0) {
+      sM[warp * 16 + g + 8 * e] = mx[e];
+      sM[64 + warp * 16 + g + 8 * e] = l[e];
+    }
+#pragma unroll
+    for (int i = 0; i < DV / 8; ++i)
+      *reinterpret_cast<float2*>(warp_acc(warp) + (g + 8 * e) * DV + i * 8 + 2 * t) = make_float2(acc[i][2 * e], acc[i][2 * e + 1]);
+  }
+  __syncthreads();
+  for (int idx = tid; idx < ng * a.vp; idx += 128) {
+    const int r = idx / a.vp, d = idx % a.vp;
+    float mm = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) mm = fmaxf(mm, sM[w * 16 + r]);
+    float ls = 0.f, o = 0.f;
+    if (mm != -INFINITY) {
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float sc = exp2f(sM[w * 16 + r] - mm);
+        ls += sM[64 + w * 16 + r] * sc;
+        o += warp_acc(w)[r * DV + d] * sc;
+      }
+    }
+    if (a.splits == 1) {
+      __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.o) + static_cast<size_t>(m) * a.ldo + (h0 + r) * a.vp;
+      out[d] = __float2bfloat16(ls > 0.f ? o / ls * a.out_scale : 0.f);
+    } else {
+      float* w = a.ws + ((static_cast<size_t>(m) * a.H + h0 + r) * a.splits + split) * (a.vp + 2);
+      w[d] = o;
+      if (d == 0) {
+        w[a.vp] = mm;
+        w[a.vp + 1] = ls;
+      }
+    }
+  }
+}
+
+__global__ void __launch_bounds__(128) gqa_merge_kernel(const GqaAttend a) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, h = blockIdx.y;
+  const float* base = a.ws + (static_cast<size_t>(m) * a.H + h) * a.splits * (a.vp + 2);
+  float mm = -INFINITY;
+  for (int s = 0; s < a.splits; ++s) mm = fmaxf(mm, base[s * (a.vp + 2) + a.vp]);
+  for (int d = threadIdx.x; d < a.vp; d += 128) {
+    float ls = 0.f, o = 0.f;
+    if (mm != -INFINITY)
+      for (int s = 0; s < a.splits; ++s) {
+        const float* w = base + s * (a.vp + 2);
+        const float sc = exp2f(w[a.vp] - mm);
+        ls += w[a.vp + 1] * sc;
+        o += w[d] * sc;
+      }
+    reinterpret_cast<__nv_bfloat16*>(a.o)[static_cast<size_t>(m) * a.ldo + h * a.vp + d] = __float2bfloat16(ls > 0.f ? o / ls * a.out_scale : 0.f);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_attend_kernel(const GqaAttend a) {
+  constexpr int KT = 128, OV = 8;            // up to 1024 value columns
+  extern __shared__ float ga_q[];            // [dk_p]
+  __shared__ float sp[KT];
+  __shared__ long srow[KT];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, h = blockIdx.y, hk = h / (a.H / a.Hkv), tid = threadIdx.x;
+  const int seq = a.row_seq[m], p = a.pos[m], len = a.ctx[seq] > 0 ? p + 1 : 0;
+  const T* q = reinterpret_cast<const T*>(a.q) + static_cast<size_t>(m) * a.ldq + h * a.dk_p;
+  for (int i = tid; i < a.dk_p; i += 128) ga_q[i] = ld1(q + i);
+  float acc[OV];
+#pragma unroll
+  for (int i = 0; i < OV; ++i) acc[i] = 0.f;
+  float mx = -INFINITY, sum = 0.f;
+  const T* keys = reinterpret_cast<const T*>(a.cache) + hk * a.dk_p;
+  const T* vals = reinterpret_cast<const T*>(a.cache) + a.Hkv * a.dk_p + hk * a.dv_p;
+  for (int k0 = a.mask.first(p); k0 < len; k0 += KT) {
+    __syncthreads();
+    const int j = k0 + tid;
+    float s = -INFINITY;
+    long cr = -1;
+    if (j < len) {
+      const int blk = a.block_table[static_cast<size_t>(seq) * a.max_blocks + j / a.block_size];
+      if (index_ok(blk, a.num_blocks, a.status)) {
+        cr = static_cast<long>(blk) * a.block_size + j % a.block_size;
+        const T* k = keys + cr * a.ldc;
+        float d = 0.f;
+        for (int i = 0; i < a.dk_p; i += 4) {
+          const float4 x = ld4(k + i);
+          d = fmaf(x.x, ga_q[i], d);
+          d = fmaf(x.y, ga_q[i + 1], d);
+          d = fmaf(x.z, ga_q[i + 2], d);
+          d = fmaf(x.w, ga_q[i + 3], d);
+        }
+        s = d * a.scale;
+      }
+    }
+    float tm = s;
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, x));
+    if ((tid & 31) == 0) red[tid >> 5] = tm;
+    __syncthreads();
+    tm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+    const float mn = fmaxf(mx, tm);
+    if (mn == -INFINITY) continue;           // uniform: no usable key so far
+    const float corr = mx == -INFINITY ? 0.f : expf(mx - mn);
+    const float e = s == -INFINITY ? 0.f : expf(s - mn);
+    mx = mn;
+    sp[tid] = e;
+    srow[tid] = cr;
+    sum = sum * corr + cta_sum(e, red);      // its barriers publish sp / srow
+    const int nk = min(KT, len - k0);
+#pragma unroll
+    for (int i = 0; i < OV; ++i) {
+      const int d = tid + i * 128;
+      if (d < a.vdim) {
+        float x = acc[i] * corr;
+        for (int k = 0; k < nk; ++k)
+          if (srow[k] >= 0) x = fmaf(sp[k], ld1(vals + srow[k] * a.ldc + d), x);
+        acc[i] = x;
+      }
+    }
+  }
+  const float inv = sum > 0.f ? a.out_scale / sum : 0.f;
+  T* o = reinterpret_cast<T*>(a.o) + static_cast<size_t>(m) * a.ldo + h * a.vp;
+#pragma unroll
+  for (int i = 0; i < OV; ++i) {
+    const int d = tid + i * 128;
+    if (d < a.vp) st1(o + d, acc[i] * inv);
+  }
+}
+
+template <int DK, int DV>
+static int launch_gqa_decode(const GqaAttend& a, int M, cudaStream_t st) {
+  constexpr int smem = gqa_decode_smem<DK, DV>();
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!configured[dev & 63]) {
+    cudaError_t e = cudaFuncSetAttribute(gqa_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured[dev & 63] = true;
+  }
+  const int groups = (a.H / a.Hkv + 15) / 16;
+  cudaError_t e = launch_kernel(gqa_decode_kernel<DK, DV>, dim3(M, a.Hkv * groups, a.splits), dim3(128), smem, st, a);
+  if (e == cudaSuccess && a.splits > 1) e = launch_kernel(gqa_merge_kernel, dim3(M, a.H), dim3(128), 0, st, a);
+  return static_cast<int>(e);
+}
+
+static bool gqa_ok(const GqaAttend& a, int M) {
+  return a.H > 0 && a.H <= 65535 && a.Hkv > 0 && a.H % a.Hkv == 0 && a.block_size > 0 && a.ldc >= a.Hkv * (a.dk_p + a.dv_p) && a.vp >= a.vdim &&
+         a.dv_p >= a.vp && a.ldo >= a.H * a.vp && a.ldq >= a.H * a.dk_p;
+}
+
+}  // namespace artb
+
+using namespace artb;
+
+ARTB_EXPORT int artb_gqa_finish(int f32, void* p, int ldp, int kind, const float* bias, const int* slot, void* cache, int ldc,
+                                long num_slots, void* q, int ldq, int M, int H, int Hkv, int dim, int dk_p, int vdim, int dv_p,
+                                int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (H <= 0 || Hkv <= 0 || H % Hkv || dk_p < dim || dv_p < vdim || ldc < Hkv * (dk_p + dv_p) || ldq < H * dk_p || ((dk_p | dv_p | ldc | ldq) & 3))
+    return ERR_BAD_SHAPE;
+  const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status};
+  const bool v4 = !((dim | vdim | ldp) & 3) && !(reinterpret_cast<uintptr_t>(p) & 15);
+#define ARTB_GF(T_, V_) return static_cast<int>(launch_kernel(gqa_finish_kernel<T_, V_>, dim3(M), dim3(256), 0, st, a))
+  if (f32) {
+    if (v4) ARTB_GF(float, 4);
+    ARTB_GF(float, 1);
+  }
+  if (v4) ARTB_GF(__nv_bfloat16, 4);
+  ARTB_GF(__nv_bfloat16, 1);
+#undef ARTB_GF
+}
+
+// k [n_keys, kcols] and vt [vcols, n_keys] of the gathered rows (see artb_latent_gather); kcols and vcols multiples of 64,
+// n_keys a multiple of 8
+ARTB_EXPORT int artb_gqa_gather(const void* cache, int ldc, const int* block_table, int max_blocks, int block_size, long num_blocks,
+                                const int* seq_of, const int* key_off, const int* key_pos0, const int* key_cnt, int n_seqs, int n_keys,
+                                void* k, void* vt, int kcols, int vcols, int* status, cudaStream_t st) {
+  if (n_keys <= 0 || n_seqs <= 0) return 0;
+  if ((ldc & 7) || (kcols & 63) || (vcols & 63) || (n_keys & 7) || kcols <= 0 || vcols <= 0 || ldc < kcols + vcols || block_size <= 0 ||
+      (kcols + vcols) / 64 > 65535)
+    return ERR_BAD_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(vt) | reinterpret_cast<uintptr_t>(cache)) & 15) return ERR_BAD_ALIGN;
+  const GqaGather a{reinterpret_cast<const __nv_bfloat16*>(cache), ldc, block_table, max_blocks, block_size, num_blocks, seq_of, key_off,
+                    key_pos0, key_cnt, n_seqs, n_keys, reinterpret_cast<__nv_bfloat16*>(k), reinterpret_cast<__nv_bfloat16*>(vt), kcols,
+                    vcols, status};
+  gqa_gather_kernel<<<dim3((n_keys + 63) / 64, (kcols + vcols) / 64), 256, 0, st>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// Rows 0 .. M - 1, each its own query; bf16, dk_p and dv_p multiples of 8 up to 256.  splits > 1: ws fp32 [M * H * splits * (vp + 2)].
+ARTB_EXPORT int artb_gqa_decode(const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
+                                int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
+                                int chunk, float scale, float out_scale, void* o, int ldo, int vp, float* ws, int splits, int M, int H,
+                                int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale,
+                    out_scale, o, ldo, vp, ws, splits, H, Hkv, dk_p, vdim, dv_p, status};
+  if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc | ldq) & 7) || splits < 1 || splits > 65535 || (splits > 1 && !ws)) return ERR_BAD_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return ERR_BAD_ALIGN;
+#define ARTB_GD(K_)                                                   \
+  do {                                                                \
+    if (dv_p <= 64) return launch_gqa_decode<K_, 64>(a, M, st);       \
+    if (dv_p <= 128) return launch_gqa_decode<K_, 128>(a, M, st);     \
+    if (dv_p <= 256) return launch_gqa_decode<K_, 256>(a, M, st);     \
+    return ERR_TOO_LARGE;                                             \
+  } while (0)
+  if (dk_p <= 64) ARTB_GD(64);
+  if (dk_p <= 128) ARTB_GD(128);
+  if (dk_p <= 256) ARTB_GD(256);
+#undef ARTB_GD
+  return ERR_TOO_LARGE;
+}
+
+ARTB_EXPORT int artb_gqa_attend(int f32, const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
+                                int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
+                                int chunk, float scale, float out_scale, void* o, int ldo, int vp, int M, int H, int Hkv, int dk_p,
+                                int vdim, int dv_p, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale,
+                    out_scale, o, ldo, vp, nullptr, 1, H, Hkv, dk_p, vdim, dv_p, status};
+  if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc) & 3) || vp > 1024 || dk_p > 8192) return ERR_BAD_SHAPE;
+  const size_t smem = static_cast<size_t>(dk_p) * 4;
+  return static_cast<int>(f32 ? launch_kernel(gqa_attend_kernel<float>, dim3(M, H), dim3(128), smem, st, a)
+                              : launch_kernel(gqa_attend_kernel<__nv_bfloat16>, dim3(M, H), dim3(128), smem, st, a));
+}

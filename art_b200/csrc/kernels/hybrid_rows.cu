@@ -2,13 +2,17 @@
 //
 //   residual_step      the fp32 residual stream across a sublayer boundary, one pass:
 //                        x = x + mult * RMSNorm(y) w_post          (or x = RMSNorm(table[token]) w_post at the input)
+//                        without w_post: x = x + mult * y          (or x = mult * table[token] + position vector)
+//                        y may have a bias and the weighted rows of a token's experts added to it
 //                        depth average: x <- sum_j weight[j] X_j over the results X_j of all layers so far
 //                        h = RMSNorm(x) w_next                     (operand of the next matrix product)
 //   norm_shift_mix     h = RMSNorm(x) w; the inputs h + (h' - h) mu_s of a token-shifted mixer, h' being the h of the
 //                      token before (from the sequence's state at the start of a portion)
 //   poly_norm          a N(z) + b N(z^2) + c N(z^3) + e, N(v) = v / rms(v)
+//   gated_act          act(gate) * up of a gate|up projection, gate and up columns interleaved in blocks of 16
 //   split_tanh         tanh(z) as a bf16 pair (high part, remainder), so that a product with it loses no 16-bit digits
-//   head_norm          per-head RMSNorm of a mixer's fp32 output, with an optional silu gate
+//   head_norm          per-head RMSNorm of a mixer's fp32 output, with an optional silu or sigmoid gate
+//   row_norm           the same over a whole row of heads
 //   gather_norm        RMSNorm of chosen rows (inputs of the LM head)
 //
 // The residual stream, its history, norms and states are fp32; GEMM operands are written as bf16 (or fp32 in the 32-bit
@@ -25,6 +29,8 @@
 
 namespace artb {
 
+enum GateAct : int { GATE_SILU = 0, GATE_SIGMOID = 1 };
+
 struct ResidualArgs {
   const int64_t* tokens;   // embedding lookup instead of y when set
   const void* table;       // T [vocab, ldt]
@@ -35,8 +41,16 @@ struct ResidualArgs {
   const float* x_in;
   float* x_out;            // may alias x_in
   int ldx;
-  const float* w_post;     // fp32 [dp]
+  const float* w_post;     // fp32 [dp], or null: y is not normalised
   float mult;
+  const float* y_bias;     // fp32 [dp] added to y, or null
+  const void* ex;          // T [.., ldex] rows of experts: y += sum_s ex_w[row, s] * ex[ex_pos[row, s]], or null
+  int ldex, ex_k;
+  const int* ex_pos;
+  const float* ex_w;
+  long ex_rows;
+  const double* freq;      // sinusoidal position vector added at the input: angle of column pair i is pos * freq[i]
+  const int* pos;
   float* hist;             // fp32 [.., rows, ldx] results of the layers, or null
   long hist_stride;
   int hist_n;              // earlier results 0 .. hist_n - 1 are in hist; this one is stored as hist_n
@@ -48,6 +62,15 @@ struct ResidualArgs {
   float eps;
   int* status;
 };
+
+// sine and cosine of pos * freq; the angle is reduced in double so that far positions lose nothing
+__device__ __forceinline__ float2 position_pair(int pos, double freq) {
+  constexpr double TWO_PI = 6.283185307179586476925;
+  const double ang = pos * freq;
+  float2 r;
+  sincosf(static_cast<float>(ang - rint(ang / TWO_PI) * TWO_PI), &r.x, &r.y);
+  return r;
+}
 
 template <typename T, int MAXV>
 __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a) {
@@ -67,21 +90,58 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
     const int v = threadIdx.x + i * blockDim.x;
     y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (v < nv) {
-      y[i] = a.tokens ? ld4(reinterpret_cast<const T*>(a.table) + static_cast<size_t>(tok) * a.ldt + v * 4)
-                      : take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, a.y_kind);
-      ss += sq4(y[i]);
+      if (a.tokens) y[i] = ld4(reinterpret_cast<const T*>(a.table) + static_cast<size_t>(tok) * a.ldt + v * 4);
+      else if (a.y) y[i] = take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, a.y_kind);
+      if (a.y_bias) {
+        const float4 b = ld4(a.y_bias + v * 4);
+        y[i] = make_float4(y[i].x + b.x, y[i].y + b.y, y[i].z + b.z, y[i].w + b.w);
+      }
     }
   }
-  ss = cta_sum(ss, red);
-  const float r = 1.f / sqrtf(ss / a.d + a.eps);
+  if (a.ex) {
+    for (int s = 0; s < a.ex_k; ++s) {
+      const int er = a.ex_pos[static_cast<size_t>(row) * a.ex_k + s];
+      const float ew = a.ex_w[static_cast<size_t>(row) * a.ex_k + s];
+      if (!index_ok(er, a.ex_rows, a.status)) continue;
+      const T* ep = reinterpret_cast<const T*>(a.ex) + static_cast<size_t>(er) * a.ldex;
+#pragma unroll
+      for (int i = 0; i < MAXV; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v < nv) {
+          const float4 e = ld4(ep + v * 4);
+          y[i] = make_float4(fmaf(ew, e.x, y[i].x), fmaf(ew, e.y, y[i].y), fmaf(ew, e.z, y[i].z), fmaf(ew, e.w, y[i].w));
+        }
+      }
+    }
+  }
+  float r = 1.f;
+  if (a.w_post) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) ss += sq4(y[i]);        // columns past the row are zero
+    ss = cta_sum(ss, red);
+    r = 1.f / sqrtf(ss / a.d + a.eps);
+  }
   const size_t xo = static_cast<size_t>(row) * a.ldx;
   ss = 0.f;
 #pragma unroll
   for (int i = 0; i < MAXV; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
     if (v < nv) {
-      const float4 w = ld4(a.w_post + v * 4);
-      float4 x = make_float4(y[i].x * r * w.x, y[i].y * r * w.y, y[i].z * r * w.z, y[i].w * r * w.w);
+      float4 x = y[i];
+      if (a.w_post) {
+        const float4 w = ld4(a.w_post + v * 4);
+        x = make_float4(x.x * r * w.x, x.y * r * w.y, x.z * r * w.z, x.w * r * w.w);
+      } else if (a.tokens) {
+        x = make_float4(a.mult * x.x, a.mult * x.y, a.mult * x.z, a.mult * x.w);
+      }
+      if (a.tokens && a.freq) {
+        const float2 p0 = position_pair(a.pos[row], a.freq[v * 2]), p1 = position_pair(a.pos[row], a.freq[v * 2 + 1]);
+        const int c = v * 4;
+        if (c < a.d) x.x += p0.x;
+        if (c + 1 < a.d) x.y += p0.y;
+        if (c + 2 < a.d) x.z += p1.x;
+        if (c + 3 < a.d) x.w += p1.y;
+      }
       if (!a.tokens) {
         const float4 x0 = ld4(a.x_in + xo + v * 4);
         x = make_float4(fmaf(a.mult, x.x, x0.x), fmaf(a.mult, x.y, x0.y), fmaf(a.mult, x.z, x0.z), fmaf(a.mult, x.w, x0.w));
@@ -284,10 +344,12 @@ __global__ void split_tanh_kernel(void* z, int ldz, int kind, T* out, int ldo, i
 // --------------------------------------------------------------------------------------------- per-head norm
 // out[row, h * vp + j] = rms(o[row, h, :])_j * w  (* silu(gate)), padding columns zero.  LPH lanes share a (row, head);
 // with V4 a lane handles four neighbouring elements (vdim, vp and all strides multiples of 4).
+__device__ __forceinline__ float gate_f(float z, int act) { return act == GATE_SIGMOID ? 1.f / (1.f + expf(-z)) : silu_f(z); }
+
 template <typename T, int LPH, bool V4>
 __global__ void __launch_bounds__(256)
 head_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__ w, int w_per_head, void* gate, int ldg,
-                 int gate_kind, T* out, int ldo, int M, int H, int vdim, int vp, float eps) {
+                 int gate_kind, int gate_act, T* out, int ldo, int M, int H, int vdim, int vp, float eps) {
   pdl_wait();
   pdl_launch_dependents();
   const int u = static_cast<int>(blockIdx.x * (256u / LPH) + threadIdx.x / LPH);     // M * H < 2^31
@@ -317,7 +379,7 @@ head_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__
         v = make_float4(a.x * r * b.x, a.y * r * b.y, a.z * r * b.z, a.w * r * b.w);
         if (gate) {
           const float4 g = take4(gate, go + j, gate_kind);
-          v = make_float4(v.x * silu_f(g.x), v.y * silu_f(g.y), v.z * silu_f(g.z), v.w * silu_f(g.w));
+          v = make_float4(v.x * gate_f(g.x, gate_act), v.y * gate_f(g.y, gate_act), v.z * gate_f(g.z, gate_act), v.w * gate_f(g.w, gate_act));
         }
       }
       st4(y + j, v);
@@ -327,11 +389,65 @@ head_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__
       float v = 0.f;
       if (j < vdim) {
         v = x[j] * r * wh[j];
-        if (gate) v *= silu_f(take1(gate, go + j, gate_kind));
+        if (gate) v *= gate_f(take1(gate, go + j, gate_kind), gate_act);
       }
       st1(y + j, v);
     }
   }
+}
+
+// One norm over the n columns of a row (all heads together); a CTA per row, columns n .. np - 1 of out are zero.
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(256)
+row_norm_kernel(const float* __restrict__ o, int ldi, const float* __restrict__ w, void* gate, int ldg, int gate_kind, int gate_act,
+                T* out, int ldo, int n, int np, float eps) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x;
+  const float* x = o + static_cast<size_t>(row) * ldi;
+  float4 v[MAXV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    v[i] = c < n ? ld4(x + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += sq4(v[i]);
+  }
+  const float r = 1.f / sqrtf(cta_sum(ss, red) / n + eps);
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    if (c >= np) continue;
+    float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < n) {
+      const float4 b = ld4(w + c);
+      y = make_float4(v[i].x * r * b.x, v[i].y * r * b.y, v[i].z * r * b.z, v[i].w * r * b.w);
+      if (gate) {
+        const float4 g = take4(gate, static_cast<size_t>(row) * ldg + c, gate_kind);
+        y = make_float4(y.x * gate_f(g.x, gate_act), y.y * gate_f(g.y, gate_act), y.z * gate_f(g.z, gate_act), y.w * gate_f(g.w, gate_act));
+      }
+    }
+    st4(out + static_cast<size_t>(row) * ldo + c, y);
+  }
+}
+
+// z [M, 2 np]: blocks of 16 gate columns and their 16 up columns in turn -> out [M, np] = act(gate) * up.  Eight columns a thread.
+template <typename T>
+__global__ void __launch_bounds__(256) gated_act_kernel(void* z, int ldz, int kind, T* out, int ldo, long units, int nv, int act) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long u = blockIdx.x * 256L + threadIdx.x;
+  if (u >= units) return;
+  const long m = u / nv;
+  const int c = static_cast<int>(u - m * nv) * 8;
+  const size_t zo = static_cast<size_t>(m) * ldz + (c >> 4) * 32 + (c & 15);
+  float g[8], x[8];
+  take8(z, zo, kind, g);
+  take8(z, zo + 16, kind, x);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) x[i] *= act == ACT_RELU ? fmaxf(g[i], 0.f) : silu_f(g[i]);
+  put8(out + static_cast<size_t>(m) * ldo + c, x);
 }
 
 template <typename T, int MAXV>
@@ -383,13 +499,15 @@ using namespace artb;
 // f32: operands (table, h) are fp32 instead of bf16.  See ResidualArgs; y_kind is a RowKind.
 ARTB_EXPORT int artb_residual_step(int f32, const int64_t* tokens, const void* table, int ldt, long vocab, void* y, int ldy,
                                    int y_kind, const float* x_in, float* x_out, int ldx, const float* w_post, float mult,
-                                   float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
+                                   const float* y_bias, const void* ex, int ldex, int ex_k, const int* ex_pos,
+                                   const float* ex_w, long ex_rows, const double* freq, const int* pos, float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
                                    int ldh, int M, int d, int dp, float eps, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
-  if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || !w_post || !x_out) return ERR_BAD_SHAPE;
-  if (!tokens && (!y || !x_in)) return ERR_BAD_SHAPE;
-  const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, hist, hist_stride, hist_n,
-                       avg, w_next, h, ldh, d, dp, eps, status};
+  if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || (ldex & 3) || !x_out) return ERR_BAD_SHAPE;
+  if (!tokens && ((!y && !ex) || !x_in)) return ERR_BAD_SHAPE;
+  if ((ex && (ex_k <= 0 || !ex_pos || !ex_w)) || (freq && (!tokens || !pos))) return ERR_BAD_SHAPE;
+  const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, y_bias, ex, ldex, ex_k, ex_pos, ex_w,
+                       ex_rows, freq, pos, hist, hist_stride, hist_n, avg, w_next, h, ldh, d, dp, eps, status};
   const int th = row_threads(dp);
   cudaError_t e = cudaSuccess;
 #define ARTB_RS(V)                                                                                                     \
@@ -445,17 +563,42 @@ ARTB_EXPORT int artb_split_tanh(int f32, void* z, int ldz, int kind, void* out, 
                                               reinterpret_cast<__nv_bfloat16*>(out), ldo, M, r, rp));
 }
 
+// z [M, 2 np] of `kind` in gate|up blocks of 16 columns -> out [M, np] (np a multiple of 16)
+ARTB_EXPORT int artb_gated_act(int f32, void* z, int ldz, int kind, void* out, int ldo, int M, int np, int act, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if ((np & 15) || (ldz & 7) || (ldo & 7) || (act != ACT_SILU && act != ACT_RELU)) return ERR_BAD_SHAPE;
+  const long units = static_cast<long>(M) * (np >> 3);
+  const dim3 grid(static_cast<unsigned>((units + 255) / 256));
+  return static_cast<int>(f32 ? launch_kernel(gated_act_kernel<float>, grid, dim3(256), 0, st, z, ldz, kind, reinterpret_cast<float*>(out),
+                                              ldo, units, np >> 3, act)
+                              : launch_kernel(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, z, ldz, kind,
+                                              reinterpret_cast<__nv_bfloat16*>(out), ldo, units, np >> 3, act));
+}
+
 // o fp32 [M, H * vdim]; w [vdim] or, with w_per_head, [H * vdim]; gate [M, H * vdim] of kind gate_kind or null
 ARTB_EXPORT int artb_head_norm(int f32, const float* o, int ldi, const float* w, int w_per_head, void* gate, int ldg,
-                               int gate_kind, void* out, int ldo, int M, int H, int vdim, int vp, float eps, cudaStream_t st) {
+                               int gate_kind, int gate_act, void* out, int ldo, int M, int H, int vdim, int vp, float eps,
+                               cudaStream_t st) {
   if (M <= 0) return 0;
   if (H <= 0 || vdim <= 0 || vp < vdim || ldo < H * vp || static_cast<long>(M) * H >= (1L << 31)) return ERR_BAD_SHAPE;
   const bool v4 = !((vdim | vp | ldi | ldo | (gate ? ldg : 0)) & 3) && !(reinterpret_cast<uintptr_t>(gate) & 15);
+  if (H == 1 && v4 && vp > 256) {      // one norm per row: a CTA each
+    const int th = row_threads(vp);
+    cudaError_t e = cudaSuccess;
+#define ARTB_RN(V)                                                                                                         \
+  e = f32 ? launch_kernel(row_norm_kernel<float, V>, dim3(M), dim3(th), 0, st, o, ldi, w, gate, ldg, gate_kind, gate_act,   \
+                          reinterpret_cast<float*>(out), ldo, vdim, vp, eps)                                               \
+          : launch_kernel(row_norm_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, o, ldi, w, gate, ldg, gate_kind,     \
+                          gate_act, reinterpret_cast<__nv_bfloat16*>(out), ldo, vdim, vp, eps)
+    ARTB_BY_VECS(row_vecs(vp, th), ARTB_RN)
+#undef ARTB_RN
+    return static_cast<int>(e);
+  }
   const int lph = !v4 ? 32 : vdim <= 16 ? 4 : vdim <= 64 ? 16 : 32;
   const dim3 grid(static_cast<unsigned>((static_cast<long>(M) * H * lph + 255) / 256));
 #define ARTB_HN(T_, L_, V_)                                                                                             \
   return static_cast<int>(launch_kernel(head_norm_kernel<T_, L_, V_>, grid, dim3(256), 0, st, o, ldi, w, w_per_head, gate, ldg, \
-                                        gate_kind, reinterpret_cast<T_*>(out), ldo, M, H, vdim, vp, eps))
+                                        gate_kind, gate_act, reinterpret_cast<T_*>(out), ldo, M, H, vdim, vp, eps))
   if (f32) {
     if (lph == 4) ARTB_HN(float, 4, true);
     if (lph == 16) ARTB_HN(float, 16, true);

@@ -4,6 +4,7 @@
 //                           sequence (a GEMM then expands their latents into every head's keys and values)
 //   latent_prefill_kernel   windowed flash attention for any sizes (whole 64-column blocks: latent_prefill_tc.cu); a head's key is [ expanded part: dk | rotated part: rot_p ], the
 //                           rotated part coming from the gathered rows all heads share
+// Without a rotated part, and with G query heads per key head, the same kernel is grouped-query attention.
 //
 // A CTA owns 128 query rows of one sequence and one head: four warps with 32 rows each, key tiles of 32, keys and values
 // double-buffered with asynchronous copies.  Scores, softmax and accumulators are fp32; only the probabilities enter the
@@ -12,6 +13,7 @@
 
 #include "bounds_check.cuh"
 #include "host_utils.h"
+#include "key_mask.cuh"
 #include "mma_tile.cuh"
 
 namespace artb {
@@ -57,11 +59,11 @@ struct LatentPrefill {
   const int* row_pos0;           // per sequence: position of row 0 of q if it belonged to the sequence (position - row)
   const int* key_off;            // per sequence: first gathered row
   const int* key_pos0;           // per sequence: position of that row
-  int window;
-  float scale_log2;
+  KeyMask mask;
+  float scale_log2, out_scale;   // out_scale multiplies the result
   __nv_bfloat16* o;              // [rows][ldo]: heads of vp columns
   int ldo, vp, vdim;
-  int H, dk, dv, rot_p;          // dk, dv, rot_p multiples of 16
+  int H, G, dk, dv, rot_p;       // G heads share a key head; dk, dv, rot_p multiples of 16
 };
 
 // DV: value columns held in registers (dv <= DV)
@@ -76,12 +78,12 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
   const int r0 = a.tile_row[blockIdx.y], nrow = min(LP_BM, a.row_end[sq] - r0);
   const int p0 = r0 + a.row_pos0[sq], p1 = p0 + nrow - 1;                 // positions of the tile's first and last row
   const int kp0 = a.key_pos0[sq];
-  const int lo = a.window > 0 ? max(kp0, p0 - a.window + 1) : kp0;
+  const int lo = max(kp0, a.mask.first(p0));
   const int tiles = (p1 - lo) / LP_BN + 1;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3, jm = lane >> 3, rr = lane & 7;
-  const __nv_bfloat16* kbase = a.kv + static_cast<size_t>(h) * a.dk;
-  const __nv_bfloat16* vbase = a.kv + static_cast<size_t>(a.H) * a.dk + static_cast<size_t>(h) * a.dv;
+  const __nv_bfloat16* kbase = a.kv + static_cast<size_t>(h / a.G) * a.dk;
+  const __nv_bfloat16* vbase = a.kv + static_cast<size_t>(a.H / a.G) * a.dk + static_cast<size_t>(h / a.G) * a.dv;
   const __nv_bfloat16* rbase = a.c + a.rank_p;
   const int kv8 = a.dk >> 3, rv8 = a.rot_p >> 3, vv8 = a.dv >> 3, row8 = kv8 + rv8 + vv8;
 
@@ -125,9 +127,9 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
       copy_wait<0>();
     }
     __syncthreads();
-    // rows of this warp see positions (p - window, p]: skip a tile none of them sees
+    // a row at p sees positions first(p) .. p, first() never falls: skip a tile no row of the warp sees
     const int wp0 = p0 + w0, wp1 = min(p0 + w0 + 31, p1);
-    const bool any = w0 < nrow && k0 <= wp1 && (a.window <= 0 || k0 + LP_BN - 1 > wp0 - a.window);
+    const bool any = w0 < nrow && k0 <= wp1 && k0 + LP_BN - 1 >= a.mask.first(wp0);
     if (any) {
       const __nv_bfloat16* K = sK + buf * LP_BN * LQ;
       float s[2][4][4];
@@ -152,13 +154,13 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
           }
       }
       // no masking needed when every row of the warp sees the whole tile
-      const bool inside = k0 + LP_BN - 1 <= wp0 && (a.window <= 0 || k0 > wp1 - a.window);
+      const bool inside = k0 + LP_BN - 1 <= wp0 && k0 >= a.mask.first(wp1);
       uint32_t pf[2][2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int p = p0 + w0 + i * 16 + g + 8 * e;
+          const int p = p0 + w0 + i * 16 + g + 8 * e, first = a.mask.first(p);
           float mx = mrow[i][e];
 #pragma unroll
           for (int j = 0; j < 4; ++j)
@@ -167,7 +169,7 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
               float& x = s[i][j][2 * e + k];
               const int kp = k0 + j * 8 + 2 * t + k;
               x *= a.scale_log2;
-              if (!inside && (kp > p || (a.window > 0 && kp <= p - a.window))) x = -INFINITY;
+              if (!inside && (kp > p || kp < first)) x = -INFINITY;
               mx = fmaxf(mx, x);
             }
           mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -215,7 +217,7 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int r = w0 + i * 16 + g + 8 * e;
       if (r >= nrow) continue;
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = l > 0.f ? a.out_scale / l : 0.f;
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp;
 #pragma unroll
       for (int n = 0; n < DV / 8; ++n) {
@@ -264,15 +266,15 @@ ARTB_EXPORT int artb_latent_gather(const void* cache, int ldc, const int* block_
 
 ARTB_EXPORT int artb_latent_prefill(const void* q, int ldq, const void* kv, int ldkv, const void* c, int ldc, int rank_p, const int* tile_seq,
                                     const int* tile_row, int n_tiles, const int* row_end, const int* row_pos0, const int* key_off,
-                                    const int* key_pos0, int window, float scale, void* o, int ldo, int vp, int vdim, int H, int dk, int dv,
-                                    int rot_p, cudaStream_t st) {
+                                    const int* key_pos0, int window, int chunk, float scale, float out_scale, void* o, int ldo, int vp, int vdim, int H, int G,
+                                    int dk, int dv, int rot_p, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
-  if (H <= 0 || (dk & 15) || (dv & 15) || (rot_p & 15) || (ldq & 7) || (ldkv & 7) || (ldc & 7) || (rank_p & 7) || (ldo & 1) || (vp & 1) ||
+  if (H <= 0 || G <= 0 || H % G || (dk & 15) || (dv & 15) || (rot_p & 15) || (ldq & 7) || (ldkv & 7) || (ldc & 7) || (rank_p & 7) || (ldo & 1) || (vp & 1) ||
       vp > dv || vdim > vp || n_tiles > 65535)
     return ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(c)) & 15) return ERR_BAD_ALIGN;
   const LatentPrefill a{(const bf16*)q, ldq, (const bf16*)kv, ldkv, (const bf16*)c, ldc, rank_p, tile_seq, tile_row, row_end, row_pos0,
-                        key_off, key_pos0, window, scale * 1.4426950408889634f, (bf16*)o, ldo, vp, vdim, H, dk, dv, rot_p};
+                        key_off, key_pos0, {window, chunk}, scale * 1.4426950408889634f, out_scale, (bf16*)o, ldo, vp, vdim, H, G, dk, dv, rot_p};
   if (dv <= 32) return launch_latent_prefill<32>(a, n_tiles, st);
   if (dv <= 64) return launch_latent_prefill<64>(a, n_tiles, st);
   if (dv <= 96) return launch_latent_prefill<96>(a, n_tiles, st);

@@ -3,6 +3,8 @@
 // The same operation as latent_prefill_kernel (expanded keys of dk columns, a rotated part of rot_p columns shared by all
 // heads, values of dv columns), with S = Q K^T and O = P V as tcgen05.mma with accumulators in TMEM:
 //
+// With G query heads per key head and no rotated part it is grouped-query attention.
+//
 //   warp 0      TMA producer: Q once; per tile of 128 keys the key blocks (expanded part from k, rotated part from the
 //               gathered cache rows) and the value block, which a GEMM has written transposed ([H * dv, keys])
 //   warp 1      MMA issuer: S of tile i, then P V of tile i - 1; S and P V accumulators are double-buffered in TMEM
@@ -15,6 +17,7 @@
 #include <math.h>
 
 #include "host_utils.h"
+#include "key_mask.cuh"
 #include "ptx_sm100.cuh"
 
 namespace artb {
@@ -30,11 +33,11 @@ struct LatentTc {
   const int* row_pos0;
   const int* key_off;
   const int* key_pos0;
-  int window;
-  float scale_log2;
+  KeyMask mask;
+  float scale_log2, out_scale;
   __nv_bfloat16* o;
   int ldo, vp;
-  int rank_p, dk, rot_p;
+  int rank_p, dk, rot_p, G;
   int* status;
 };
 
@@ -81,12 +84,12 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* xch = reinterpret_cast<float*>(smem + L::XCH);
 
-  const int h = blockIdx.y, sq = a.tile_seq[blockIdx.x];
+  const int h = blockIdx.y, hk = h / a.G, sq = a.tile_seq[blockIdx.x];
   const int r0 = a.tile_row[blockIdx.x], nrow = min(LT_B, a.row_end[sq] - r0);
   const int p0 = r0 + a.row_pos0[sq], p1 = p0 + nrow - 1;
   const int kp0 = a.key_pos0[sq], koff = a.key_off[sq];
   // first tile: down to a multiple of 8 keys, where the value load may start
-  const int lo_rel = (a.window > 0 ? max(0, p0 - a.window + 1 - kp0) : 0) & ~7;
+  const int lo_rel = max(0, a.mask.first(p0) - kp0) & ~7;
   const int tiles = (p1 - kp0 - lo_rel) / LT_B + 1;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (koff & 7) {                            // the value loads would not start on a 16-byte boundary
@@ -143,7 +146,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         mbar_expect_tx(&k_full[s], NQ * LT_BLK);
 #pragma unroll
         for (int b = 0; b < NQ; ++b) {
-          if (b < nk) tma_load_2d(sk + b * LT_BLK, &tmK, h * a.dk + b * 64, krow, &k_full[s]);
+          if (b < nk) tma_load_2d(sk + b * LT_BLK, &tmK, hk * a.dk + b * 64, krow, &k_full[s]);
           else tma_load_2d(sk + b * LT_BLK, &tmC, a.rank_p + (b - nk) * 64, krow, &k_full[s]);
         }
         if (!mbar_wait_timed(v_empty, (it & 1) ^ 1)) {
@@ -152,8 +155,8 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           break;
         }
         mbar_expect_tx(v_full, 2 * L::VBLK);
-        tma_load_2d(smem + L::V, &tmVt, krow, h * DV, v_full);
-        tma_load_2d(smem + L::V + L::VBLK, &tmVt, krow + 64, h * DV, v_full);
+        tma_load_2d(smem + L::V, &tmVt, krow, hk * DV, v_full);
+        tma_load_2d(smem + L::V + L::VBLK, &tmVt, krow + 64, hk * DV, v_full);
       }
     }
   } else if (warp == 1) {
@@ -208,7 +211,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const int q = warp & 3;                 // TMEM lane quarter of this warp
     const int hf = (warp - 2) >> 2;         // which half of the columns
     const int r = q * 32 + lane;            // query row inside the tile
-    const int qpos = p0 + r;
+    const int qpos = p0 + r, first = a.mask.first(qpos);
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
     uint8_t* prow = smem + L::P + hf * LT_BLK + r * 128;
     const int sw = r & 7;
@@ -243,7 +246,8 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       const int okw = mbar_wait_timed(&pv_full[s], (i >> 1) & 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okw)) return false;
       tc_fence_after_sync();
-      const float f = lt_ex2(m_o - ms_i);
+      // maxima only grow, but a row that has seen no key yet stands at 0: nothing to rescale then
+      const float f = lt_ex2(fminf(m_o - ms_i, 0.f));
       m_o = ms_i;
 #pragma unroll
       for (int c = 0; c < OC; c += 32) {
@@ -266,7 +270,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       }
       const int s = it & 1;
       const int k0 = kp0 + lo_rel + it * LT_B;                         // position of the tile's first key
-      const bool inside = k0 + LT_B - 1 <= p0 && (a.window <= 0 || k0 > p0 + LT_B - 1 - a.window);
+      const bool inside = k0 + LT_B - 1 <= p0 && k0 >= a.mask.first(p0 + LT_B - 1);
       const int okw = mbar_wait_timed(&s_full[s], (it >> 1) & 1) ? 1 : 0;
       if (!__all_sync(0xffffffffu, okw)) {
         fail(ST_TIMEOUT_TMEM_FULL);
@@ -289,10 +293,10 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[s]);
       if (!inside) {
-        const int hi = qpos - (k0 + hf * 64), lo = a.window > 0 ? hi - a.window : -1;      // visible: lo < j <= hi
+        const int hi = qpos - (k0 + hf * 64), lo = first - (k0 + hf * 64);      // visible: lo <= j <= hi
 #pragma unroll
         for (int j = 0; j < 64; ++j)
-          if (j > hi || j <= lo) x[j] = -INFINITY;
+          if (j > hi || j < lo) x[j] = -INFINITY;
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -344,7 +348,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     if (!dead && !swap_with_partner(l, l_other)) fail(ST_TIMEOUT_PEER);
     if (!dead && r < nrow) {
       const float lt = l + l_other;
-      const float inv = lt > 0.f ? 1.f / lt : 0.f;
+      const float inv = lt > 0.f ? a.out_scale / lt : 0.f;
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp + hf * OC;
 #pragma unroll
       for (int c = 0; c < OC; c += 8) {
@@ -394,27 +398,27 @@ static int launch_latent_tc(const CUtensorMap& tQ, const CUtensorMap& tK, const 
 
 using namespace artb;
 
-// As artb_latent_prefill, with keys k [n_keys, H * dk] and values transposed: vt [H * dv, n_keys].  dk and rot_p multiples
+// As artb_latent_prefill, with keys k [n_keys, H / G * dk] and values transposed: vt [H / G * dv, n_keys].  dk and rot_p multiples
 // of 64 (dk + rot_p <= 192), dv 64 or 128, n_keys and every key_off a multiple of 8, scale > 0.  Gathered rows between two
 // sequences must be finite.
 ARTB_EXPORT int artb_latent_prefill_tc(const void* q, int ldq, int rows, const void* k, int ldk, const void* c, int ldc, int rank_p,
                                        const void* vt, int ldvt, int n_keys, const int* tile_seq, const int* tile_row, int n_tiles,
                                        const int* row_end, const int* row_pos0, const int* key_off, const int* key_pos0, int window,
-                                       float scale, void* o, int ldo, int vp, int H, int dk, int dv, int rot_p, int* status,
-                                       cudaStream_t st) {
+                                       int chunk, float scale, float out_scale, void* o, int ldo, int vp, int H, int G, int dk, int dv, int rot_p,
+                                       int* status, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
-  if (H <= 0 || H > 65535 || dk <= 0 || (dk & 63) || (rot_p & 63) || dk + rot_p > 192 || (dv != 64 && dv != 128) || (n_keys & 7) || (ldo & 7) ||
+  if (H <= 0 || H > 65535 || G <= 0 || H % G || dk <= 0 || (dk & 63) || (rot_p & 63) || dk + rot_p > 192 || (dv != 64 && dv != 128) || (n_keys & 7) || (ldo & 7) ||
       (vp & 7) || vp > dv || !(scale > 0.f) || (rank_p & 7))
     return ERR_BAD_SHAPE;
   if (reinterpret_cast<uintptr_t>(o) & 15) return ERR_BAD_ALIGN;
   CUtensorMap tQ, tK, tC, tV;
   int e;
   if ((e = make_tmap_bf16_2d(&tQ, q, rows, static_cast<uint64_t>(H) * (dk + rot_p), ldq, LT_B, 64))) return e;
-  if ((e = make_tmap_bf16_2d(&tK, k, n_keys, static_cast<uint64_t>(H) * dk, ldk, LT_B, 64))) return e;
+  if ((e = make_tmap_bf16_2d(&tK, k, n_keys, static_cast<uint64_t>(H / G) * dk, ldk, LT_B, 64))) return e;
   if ((e = make_tmap_bf16_2d(&tC, c, n_keys, ldc, ldc, LT_B, 64))) return e;
-  if ((e = make_tmap_bf16_2d(&tV, vt, static_cast<uint64_t>(H) * dv, n_keys, ldvt, dv, 64))) return e;
-  const LatentTc a{tile_seq, tile_row, row_end, row_pos0, key_off, key_pos0, window, scale * 1.4426950408889634f,
-                   reinterpret_cast<__nv_bfloat16*>(o), ldo, vp, rank_p, dk, rot_p, status};
+  if ((e = make_tmap_bf16_2d(&tV, vt, static_cast<uint64_t>(H / G) * dv, n_keys, ldvt, dv, 64))) return e;
+  const LatentTc a{tile_seq, tile_row, row_end, row_pos0, key_off, key_pos0, {window, chunk}, scale * 1.4426950408889634f, out_scale,
+                   reinterpret_cast<__nv_bfloat16*>(o), ldo, vp, rank_p, dk, rot_p, G, status};
   const int nq = (dk + rot_p) / 64;
   if (dv == 128) {
     if (nq == 1) return launch_latent_tc<1, 128>(tQ, tK, tC, tV, a, n_tiles, H, st);

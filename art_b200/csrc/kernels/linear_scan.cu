@@ -1,7 +1,9 @@
-// Linear attention with a per-channel decay, carried in an fp32 state S [dim, vdim] per sequence and head.
+// Linear attention with a decay per channel or per head, carried in an fp32 state S [dim, vdim] per sequence and head.
 //
 //   SCAN_HGRN2   f = l + (1 - l) sigmoid(g + b), q = silu(q);   S = f S + (1 - f) v^T ;  o = S^T q        (reads after)
 //   SCAN_WKV     w = exp(-exp(g + b));   o = (S + (u k) v^T)^T r ;  S = w S + k v^T                       (reads before)
+//   SCAN_FIXED   q, k, v = silu(q), silu(k), silu(v);               S = w S + k v^T ;  o = S^T q          (reads after)
+//                w a constant of the head
 //
 // All of it is fp32 arithmetic on CUDA cores: a recurrence multiplies rounding errors, so its operands do not go through
 // 16-bit tensor-core products.  The decay, the gates and the bonus are computed where they are used; q, k, v and g are
@@ -18,7 +20,7 @@
 //                          instead of twelve.
 //   linear_decode_kernel   one new token per sequence.  A CTA owns (sequence, head), streams the state through registers
 //                          once (read, update, write) and finishes the head: RMSNorm over its vdim outputs, norm weight,
-//                          optional silu gate, bf16 store.
+//                          optional silu gate, bf16 store.  Without a norm weight the fp32 outputs are stored as they are.
 //
 // A portion that starts a sequence (ctx == its length) begins with a zero state whatever the slot holds.
 #include <cuda_bf16.h>
@@ -32,16 +34,16 @@
 
 namespace artb {
 
-enum ScanMode : int { SCAN_HGRN2 = 0, SCAN_WKV = 1 };
+enum ScanMode : int { SCAN_HGRN2 = 0, SCAN_WKV = 1, SCAN_FIXED = 2 };
 
 struct ScanArgs {
   void* q;      // q (hgrn2) or r (wkv): [M, ldq], kind qkv_kind
-  void* k;      // wkv only
+  void* k;      // wkv and fixed
   void* v;
   void* g;      // decay projection, kind g_kind
   int ldq, ldk, ldv, ldg, qkv_kind, g_kind;
   const float* bias;    // [H * dim] added to g
-  const float* aux;     // [H * dim] lower bound (hgrn2) or bonus u (wkv)
+  const float* aux;     // [H * dim] lower bound (hgrn2) or bonus u (wkv); [H] decay (fixed)
   float* state;
   long slot_stride;     // floats per slot
   int ld_dim;           // row pitch of a state column (multiple of 4, >= dim)
@@ -59,7 +61,7 @@ struct ScanOut {
 };
 
 struct DecodeOut {
-  const float* w;       // norm weight [vdim] or [H * vdim]
+  const float* w;       // norm weight [vdim] or [H * vdim]; null: out is fp32 [M, ldo], vdim columns per head, not normalised
   int w_per_head;
   void* gate;           // silu gate, kind gate_kind, or null
   int ldgate, gate_kind;
@@ -103,7 +105,7 @@ constexpr int SCAN_RG = 8;              // threads that share a state column
 constexpr int SCAN_LOADERS = 128;
 
 template <int MODE>
-constexpr int scan_arrays() { return MODE == SCAN_WKV ? 3 : 2; }
+constexpr int scan_arrays() { return MODE == SCAN_WKV ? 3 : 2; }      // q, k and decay, as far as they are operands
 template <int MODE>
 constexpr int scan_smem(int DP, int cw) {
   return 2 * SCAN_TC * (scan_arrays<MODE>() * DP + 2 * cw + 1) * 4;
@@ -117,11 +119,16 @@ __device__ __forceinline__ void scan_gates(float qr, float kr, float g, float au
     f = aux + (1.f - aux) * __fdividef(1.f, 1.f + expf(-g));
     k = 1.f - f;
     bonus = 0.f;
-  } else {
+  } else if (MODE == SCAN_WKV) {
     q = qr;
     f = expf(-expf(g));
     k = kr;
     bonus = qr * aux * kr;
+  } else {
+    q = silu_f(qr);
+    f = aux;
+    k = silu_f(kr);
+    bonus = 0.f;
   }
 }
 
@@ -139,11 +146,12 @@ template <int NR, int MODE, int CPT, int NC, typename T>
 __global__ void __launch_bounds__(SCAN_RG * NC + SCAN_LOADERS, CPT * NR <= 64 && NC == 16 ? 2 : 1)
 linear_scan_kernel(const ScanArgs a, const ScanOut so) {
   constexpr int DP = SCAN_RG * NR, CW = NC * CPT, COMP = SCAN_RG * NC, CH = DP / 32;
+  constexpr bool HAS_K = MODE != SCAN_HGRN2, HAS_F = MODE != SCAN_FIXED;      // k as an operand, a decay per channel
   extern __shared__ __align__(16) float scan_s[];
   float* sq = scan_s;                                   // [2][TC][DP]
   float* sf = sq + 2 * SCAN_TC * DP;
-  float* sk = sf + 2 * SCAN_TC * DP;                    // wkv only
-  float* sv = sk + (MODE == SCAN_WKV ? 2 * SCAN_TC * DP : 0);   // [2][TC][CW]
+  float* sk = sf + (HAS_F ? 2 * SCAN_TC * DP : 0);
+  float* sv = sk + (HAS_K ? 2 * SCAN_TC * DP : 0);      // [2][TC][CW]
   float* sout = sv + 2 * SCAN_TC * CW;                  // [2][TC][CW]
   float* sb = sout + 2 * SCAN_TC * CW;                  // [2][TC] bonus
   pdl_wait();
@@ -170,16 +178,16 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
 #pragma unroll
     for (int i = 0; i < CH; ++i) {
       const int c = i * 32 + lane;
-      bias[i] = c < a.dim ? a.bias[h * a.dim + c] : 0.f;
-      aux[i] = c < a.dim ? a.aux[h * a.dim + c] : 0.f;
+      bias[i] = HAS_F && c < a.dim ? a.bias[h * a.dim + c] : 0.f;
+      aux[i] = HAS_F && c < a.dim ? a.aux[h * a.dim + c] : 0.f;
     }
     const T* __restrict__ gq = reinterpret_cast<const T*>(a.q) + h * a.dim;
     const T* __restrict__ gk = reinterpret_cast<const T*>(a.k) + h * a.dim;
     const T* __restrict__ gv = reinterpret_cast<const T*>(a.v) + h * a.vdim + c0;
     const float* __restrict__ gg = reinterpret_cast<const float*>(a.g) + h * a.dim;
     struct Raw {       // as loaded: converting them here would make the warp wait for them here
-      T q[TB][CH], k[TB][MODE == SCAN_WKV ? CH : 1], v[TB][CV];
-      float g[TB][CH];
+      T q[TB][CH], k[TB][HAS_K ? CH : 1], v[TB][CV];
+      float g[TB][HAS_F ? CH : 1];
     };
     const T zero = T(0.f);
     auto fetch = [&](Raw& r, int chunk, int p) {        // raw values of tokens p, p + 1 of the warp's share of a stage
@@ -193,8 +201,8 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
           const int c = i * 32 + lane;
           const bool ok = t < nt && c < a.dim;
           r.q[b][i] = ok ? gq[m * a.ldq + c] : zero;
-          r.g[b][i] = ok ? gg[m * a.ldg + c] : 0.f;
-          if (MODE == SCAN_WKV) r.k[b][MODE == SCAN_WKV ? i : 0] = ok ? gk[m * a.ldk + c] : zero;
+          if (HAS_F) r.g[b][HAS_F ? i : 0] = ok ? gg[m * a.ldg + c] : 0.f;
+          if (HAS_K) r.k[b][HAS_K ? i : 0] = ok ? gk[m * a.ldk + c] : zero;
         }
 #pragma unroll
         for (int i = 0; i < CV; ++i) {
@@ -212,14 +220,12 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
         for (int i = 0; i < CH; ++i) {
           const int c = i * 32 + lane;
           float q, f, k, bo;
-          scan_gates<MODE>(ld1(&r.q[b][i]), ld1(&r.k[b][MODE == SCAN_WKV ? i : 0]), r.g[b][i] + bias[i], aux[i], q, f, k, bo);
+          scan_gates<MODE>(ld1(&r.q[b][i]), ld1(&r.k[b][HAS_K ? i : 0]), r.g[b][HAS_F ? i : 0] + bias[i], aux[i], q, f, k, bo);
           const bool ok = c < a.dim;                    // channels past dim leave the state at zero
           sq[at * DP + c] = ok ? q : 0.f;
-          sf[at * DP + c] = ok ? f : (MODE == SCAN_HGRN2 ? 1.f : 0.f);
-          if (MODE == SCAN_WKV) {
-            sk[at * DP + c] = ok ? k : 0.f;
-            bsum += ok ? bo : 0.f;
-          }
+          if (HAS_F) sf[at * DP + c] = ok ? f : (MODE == SCAN_HGRN2 ? 1.f : 0.f);
+          if (HAS_K) sk[at * DP + c] = ok ? k : 0.f;
+          if (MODE == SCAN_WKV) bsum += ok ? bo : 0.f;
         }
         if (MODE == SCAN_WKV) {
           bsum = lane_sum(bsum);
@@ -227,7 +233,7 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
         }
 #pragma unroll
         for (int i = 0; i < CV; ++i)
-          if (i * 32 + lane < CW) sv[at * CW + i * 32 + lane] = ld1(&r.v[b][i]);
+          if (i * 32 + lane < CW) sv[at * CW + i * 32 + lane] = MODE == SCAN_FIXED ? silu_f(ld1(&r.v[b][i])) : ld1(&r.v[b][i]);
       }
     };
     // two register sets: the next tokens are on their way while the current ones go through their gates
@@ -264,6 +270,8 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
   float* sp = a.state + static_cast<size_t>(slot < 0 ? 0 : slot) * a.slot_stride + static_cast<size_t>(h) * a.vdim * a.ld_dim;
   const bool resume = slot >= 0 && a.ctx[seq] != len;
   const uint64_t minus1 = pack2(-1.f, -1.f);
+  const float head_decay = MODE == SCAN_FIXED ? a.aux[h] : 0.f;
+  const uint64_t fd = pack2(head_decay, head_decay);
   uint64_t S[CPT][NR / 2];
 #pragma unroll
   for (int j = 0; j < CPT; ++j)
@@ -300,14 +308,19 @@ linear_scan_kernel(const ScanArgs a, const ScanOut so) {
 #pragma unroll
           for (int i = 0; i < NR / 4; ++i) {
             const Pair2 q = *reinterpret_cast<const Pair2*>(qp + i * 32);
-            const Pair2 f = *reinterpret_cast<const Pair2*>(fp + i * 32);
-            Pair2 k{0ull, 0ull};
-            if (MODE == SCAN_WKV) k = *reinterpret_cast<const Pair2*>(kp + i * 32);
+            Pair2 f{fd, fd}, k{0ull, 0ull};
+            if (HAS_F) f = *reinterpret_cast<const Pair2*>(fp + i * 32);
+            if (HAS_K) k = *reinterpret_cast<const Pair2*>(kp + i * 32);
 #pragma unroll
             for (int j = 0; j < CPT; ++j) {
               if (MODE == SCAN_HGRN2) {            // f S + (1 - f) v  =  f (S - v) + v
                 S[j][2 * i] = fma2(f.lo, fma2(v2[j], minus1, S[j][2 * i]), v2[j]);
                 S[j][2 * i + 1] = fma2(f.hi, fma2(v2[j], minus1, S[j][2 * i + 1]), v2[j]);
+                o0[j] = fma2(q.lo, S[j][2 * i], o0[j]);
+                o1[j] = fma2(q.hi, S[j][2 * i + 1], o1[j]);
+              } else if (MODE == SCAN_FIXED) {
+                S[j][2 * i] = fma2(f.lo, S[j][2 * i], mul2(k.lo, v2[j]));
+                S[j][2 * i + 1] = fma2(f.hi, S[j][2 * i + 1], mul2(k.hi, v2[j]));
                 o0[j] = fma2(q.lo, S[j][2 * i], o0[j]);
                 o1[j] = fma2(q.hi, S[j][2 * i + 1], o1[j]);
               } else {
@@ -380,16 +393,19 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
     if (i < a.dim) {
       const int c = h * a.dim + i;
       const float qr = take1(a.q, static_cast<size_t>(m) * a.ldq + c, a.qkv_kind);
-      const float g = take1(a.g, static_cast<size_t>(m) * a.ldg + c, a.g_kind) + a.bias[c];
-      const float kr = MODE == SCAN_WKV ? take1(a.k, static_cast<size_t>(m) * a.ldk + c, a.qkv_kind) : 0.f;
-      scan_gates<MODE>(qr, kr, g, a.aux[c], q, f, k, b);
+      const float g = MODE != SCAN_FIXED ? take1(a.g, static_cast<size_t>(m) * a.ldg + c, a.g_kind) + a.bias[c] : 0.f;
+      const float kr = MODE != SCAN_HGRN2 ? take1(a.k, static_cast<size_t>(m) * a.ldk + c, a.qkv_kind) : 0.f;
+      scan_gates<MODE>(qr, kr, g, a.aux[MODE == SCAN_FIXED ? h : c], q, f, k, b);
     }
     sq[i] = q;
     sf[i] = f;
     sk[i] = k;
     bpart += b;
   }
-  for (int j = threadIdx.x; j < a.vdim; j += 256) sv[j] = take1(a.v, static_cast<size_t>(m) * a.ldv + h * a.vdim + j, a.qkv_kind);
+  for (int j = threadIdx.x; j < a.vdim; j += 256) {
+    const float v = take1(a.v, static_cast<size_t>(m) * a.ldv + h * a.vdim + j, a.qkv_kind);
+    sv[j] = MODE == SCAN_FIXED ? silu_f(v) : v;
+  }
   float bonus = 0.f;
   if (MODE == SCAN_WKV) bonus = cta_sum(bpart, red);
   __syncthreads();
@@ -413,7 +429,7 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
         S[i].y = fmaf(f.y, S[i].y, k.y * v);
         S[i].z = fmaf(f.z, S[i].z, k.z * v);
         S[i].w = fmaf(f.w, S[i].w, k.w * v);
-        if (MODE == SCAN_HGRN2) o += q.x * S[i].x + q.y * S[i].y + q.z * S[i].z + q.w * S[i].w;
+        if (MODE != SCAN_WKV) o += q.x * S[i].x + q.y * S[i].y + q.z * S[i].z + q.w * S[i].w;
         if (slot >= 0 && r < a.ld_dim) *reinterpret_cast<float4*>(sp + r) = S[i];
       }
     }
@@ -422,6 +438,10 @@ linear_decode_kernel(const ScanArgs a, const DecodeOut d) {
     if (rg == 0 && c < a.vdim) so[c] = MODE == SCAN_WKV ? fmaf(sv[c], bonus, o) : o;
   }
   __syncthreads();
+  if (!d.w) {
+    for (int j = threadIdx.x; j < a.vdim; j += 256) reinterpret_cast<float*>(d.out)[static_cast<size_t>(m) * d.ldo + h * a.vdim + j] = so[j];
+    return;
+  }
   float ss = 0.f;
   for (int j = threadIdx.x; j < a.vdim; j += 256) ss += so[j] * so[j];
   const float r = 1.f / sqrtf(cta_sum(ss, red) / a.vdim + d.eps);
@@ -484,7 +504,8 @@ using namespace artb;
 
 static bool scan_args_ok(const ScanArgs& a, int mode) {
   return a.H > 0 && a.dim > 0 && a.vdim > 0 && a.vdim <= 256 && (a.ld_dim & 3) == 0 && a.ld_dim >= a.dim && (a.slot_stride & 3) == 0 &&
-         !(reinterpret_cast<uintptr_t>(a.state) & 15) && a.q && a.v && a.g && a.bias && a.aux && (mode != SCAN_WKV || a.k) &&
+         !(reinterpret_cast<uintptr_t>(a.state) & 15) && a.q && a.v && a.aux && (mode == SCAN_FIXED || (a.g && a.bias)) &&
+         (mode == SCAN_HGRN2 || a.k) && mode >= SCAN_HGRN2 && mode <= SCAN_FIXED &&
          a.cu_q && a.ctx && a.state_slot;
 }
 
@@ -497,17 +518,20 @@ ARTB_EXPORT int artb_linear_scan(int mode, void* q, int ldq, void* k, int ldk, v
   if (n_seqs <= 0) return 0;
   const ScanArgs a{q, k, v, g, ldq, ldk, ldv, ldg, qkv_kind, g_kind, bias, aux, state, slot_stride, ld_dim, num_slots, cu_q, ctx,
                    state_slot, H, dim, vdim, status};
-  if (!scan_args_ok(a, mode) || qkv_kind == ROW_F32_TAKE || g_kind != ROW_F32 || n_seqs > 65535 || ldo < H * vdim)
+  if (!scan_args_ok(a, mode) || qkv_kind == ROW_F32_TAKE || (mode != SCAN_FIXED && g_kind != ROW_F32) || n_seqs > 65535 || ldo < H * vdim)
     return ERR_BAD_SHAPE;
   const ScanOut so{o, ldo, rows};
   const int nr = scan_rows(dim);
-#define ARTB_SC(NR_) return mode == SCAN_WKV ? launch_scan<NR_, SCAN_WKV>(a, so, n_seqs, st) : launch_scan<NR_, SCAN_HGRN2>(a, so, n_seqs, st)
+#define ARTB_SC(NR_)                                                              \
+  return mode == SCAN_WKV     ? launch_scan<NR_, SCAN_WKV>(a, so, n_seqs, st)     \
+         : mode == SCAN_FIXED ? launch_scan<NR_, SCAN_FIXED>(a, so, n_seqs, st)   \
+                              : launch_scan<NR_, SCAN_HGRN2>(a, so, n_seqs, st)
   ARTB_BY_ROWS(nr, ARTB_SC)
 #undef ARTB_SC
   return 0;
 }
 
-// One token of each of M sequences; out T [M, ldo] with vp >= vdim columns per head (padding zero).
+// One token of each of M sequences; out T [M, ldo] with vp >= vdim columns per head (padding zero), or fp32 without w.
 ARTB_EXPORT int artb_linear_decode(int f32, int mode, void* q, int ldq, void* k, int ldk, void* v, int ldv, int qkv_kind, void* g,
                                    int ldg, int g_kind, const float* bias, const float* aux, float* state, long slot_stride,
                                    int ld_dim, long num_slots, const int* cu_q, const int* ctx, const int* state_slot, int M, int H,
@@ -516,7 +540,7 @@ ARTB_EXPORT int artb_linear_decode(int f32, int mode, void* q, int ldq, void* k,
   if (M <= 0) return 0;
   const ScanArgs a{q, k, v, g, ldq, ldk, ldv, ldg, qkv_kind, g_kind, bias, aux, state, slot_stride, ld_dim, num_slots, cu_q, ctx,
                    state_slot, H, dim, vdim, status};
-  if (!scan_args_ok(a, mode) || M > 65535 || vp < vdim || ldo < H * vp || !w || !out) return ERR_BAD_SHAPE;
+  if (!scan_args_ok(a, mode) || M > 65535 || vp < vdim || ldo < H * (w ? vp : vdim) || !out) return ERR_BAD_SHAPE;
   const DecodeOut d{w, w_per_head, gate, ldgate, gate_kind, out, ldo, vp, eps};
   const dim3 grid(H, M);
   cudaError_t e = cudaSuccess;
@@ -525,6 +549,7 @@ ARTB_EXPORT int artb_linear_decode(int f32, int mode, void* q, int ldq, void* k,
           : launch_kernel(linear_decode_kernel<NR_, MODE_, __nv_bfloat16>, grid, dim3(256), 0, st, a, d)
 #define ARTB_LD(NR_)                                                                                              \
   if (mode == SCAN_WKV) ARTB_LD2(NR_, SCAN_WKV);                                                                   \
+  else if (mode == SCAN_FIXED) ARTB_LD2(NR_, SCAN_FIXED);                                                          \
   else ARTB_LD2(NR_, SCAN_HGRN2)
   ARTB_BY_ROWS(scan_rows(dim), ARTB_LD)
 #undef ARTB_LD

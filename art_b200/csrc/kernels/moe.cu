@@ -15,6 +15,8 @@
 #include <stdint.h>
 
 #include "host_utils.h"
+#include "ptx_sm100.cuh"
+#include "row_io.cuh"
 
 namespace artb {
 
@@ -31,56 +33,64 @@ __device__ __forceinline__ float warp_pick(const float (&a)[MOE_MAX_E_PER_LANE],
   return __shfl_sync(0xffffffffu, v, e & 31);
 }
 
-// One warp per token.
-__global__ void moe_router_kernel(const float* __restrict__ logits, int ld, int M, int E, int k, int norm,
-                                  int* __restrict__ topi, float* __restrict__ topw, int* __restrict__ counts) {
+// One warp per token.  The k largest logits (+ bias) are chosen, the lower index on a tie; weights are the softmax over all
+// experts or, with `norm`, over the chosen ones.  Logits of kind ROW_F32_TAKE are cleared once read.
+__global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, const float* __restrict__ bias, int M, int E, int k,
+                                  int norm, int* __restrict__ topi, float* __restrict__ topw, int* __restrict__ counts) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  pdl_wait();
+  pdl_launch_dependents();
   if (warp >= M) return;
-  const float* row = logits + static_cast<size_t>(warp) * ld;
+  float* row = logits + static_cast<size_t>(warp) * ld;
   float v[MOE_MAX_E_PER_LANE];
   float mx = -INFINITY;
 #pragma unroll
   for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j) {
     const int e = j * 32 + lane;
-    v[j] = e < E ? row[e] : -INFINITY;
+    v[j] = -INFINITY;
+    if (e < E) {
+      v[j] = take1(row, e, kind);
+      if (bias) v[j] += bias[e];
+    }
     mx = fmaxf(mx, v[j]);
   }
 #pragma unroll
   for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float sum = 0.f;
-#pragma unroll
-  for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j) {
-    v[j] = (j * 32 + lane) < E ? __expf(v[j] - mx) : -1.f;   // probabilities are >= 0; -1 marks "taken / absent"
-    if (v[j] > 0.f) sum += v[j];
-  }
-#pragma unroll
-  for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-  const float inv = 1.f / sum;
-  float wsel = 0.f, wtot = 0.f;
-  int isel = 0;
-  for (int s = 0; s < k; ++s) {
-    float best = -2.f;
-    int bi = 0x7fffffff;
+  if (!norm) {
 #pragma unroll
     for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j)
-      if (v[j] > best) {
+      if (j * 32 + lane < E) sum += expf(v[j] - mx);
+#pragma unroll
+    for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  }
+  float wsel = 0.f;
+  int isel = 0;
+  uint32_t taken = 0;                            // entries of this lane that are chosen already
+  for (int s = 0; s < k; ++s) {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+#pragma unroll
+    for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j) {
+      const int e = j * 32 + lane;
+      if (e < E && !(taken >> j & 1) && (v[j] > best || bi == 0x7fffffff)) {
         best = v[j];
-        bi = j * 32 + lane;
+        bi = e;
       }
+    }
 #pragma unroll
     for (int o = 16; o; o >>= 1) {
       const float ob = __shfl_xor_sync(0xffffffffu, best, o);
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > best || (ob == best && oi < bi)) {
+      if (ob > best || (ob == best && oi < bi) || bi == 0x7fffffff) {
         best = ob;
         bi = oi;
       }
     }
-#pragma unroll
-    for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j)
-      if (j == (bi >> 5) && (bi & 31) == lane) v[j] = -1.f;
-    const float p = best * inv;
-    wtot += p;
+    if (bi >= E) bi = 0;                         // logits that are no numbers: stay inside the experts
+    if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
+    const float p = expf(best - mx);
+    if (norm) sum += p;
     if (lane == s) {
       wsel = p;
       isel = bi;
@@ -88,7 +98,7 @@ __global__ void moe_router_kernel(const float* __restrict__ logits, int ld, int 
   }
   if (lane < k) {
     topi[static_cast<size_t>(warp) * k + lane] = isel;
-    topw[static_cast<size_t>(warp) * k + lane] = norm ? wsel / wtot : wsel;
+    topw[static_cast<size_t>(warp) * k + lane] = wsel / sum;
     atomicAdd(counts + isel, 1);
   }
 }
@@ -145,6 +155,17 @@ __global__ void moe_assign_kernel(const int* __restrict__ topi, const float* __r
 }
 
 // xp[r] = (use_w ? row_w[r] : 1) * x[row_token[r]], zeros for padding rows; rows >= seg_off[E] untouched.
+// fp32 rows of the 32-bit mode
+__global__ void __launch_bounds__(128)
+moe_gather_f32_kernel(const float* __restrict__ x, int ldx, const int* __restrict__ row_token, const int* __restrict__ total_rows,
+                      float* __restrict__ xp, int ldp, int D) {
+  const int r = blockIdx.x;
+  if (r >= *total_rows) return;
+  const int t = row_token[r];
+  for (int i = threadIdx.x; i < D; i += blockDim.x)
+    xp[static_cast<size_t>(r) * ldp + i] = t < 0 ? 0.f : x[static_cast<size_t>(t) * ldx + i];
+}
+
 __global__ void __launch_bounds__(128)
 moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const int* __restrict__ row_token,
                   const float* __restrict__ row_w, int use_w, const int* __restrict__ total_rows,
@@ -339,13 +360,14 @@ __global__ void moe_router_bwd_kernel(const float* __restrict__ logits, int ld, 
 
 using namespace artb;
 
-// logits fp32 [M, E] (E <= 256, k <= 16); counts int32 [E] must be zero on entry.
-ARTB_EXPORT int artb_moe_router(const float* logits, int ld, int M, int E, int k, int norm, int* topi, float* topw,
-                                int* counts, cudaStream_t st) {
+// logits fp32 [M, E] (E <= 256, k <= 16) of kind ROW_F32 or ROW_F32_TAKE; bias fp32 [E] or null; counts int32 [E] must be
+// zero on entry.
+ARTB_EXPORT int artb_moe_router(float* logits, int ld, int kind, const float* bias, int M, int E, int k, int norm, int* topi,
+                                float* topw, int* counts, cudaStream_t st) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E) return ERR_BAD_SHAPE;
+  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E || kind == ROW_BF16) return ERR_BAD_SHAPE;
   const int threads = 256, warps = threads / 32;
-  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, M, E, k, norm, topi, topw, counts);
+  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, kind, bias, M, E, k, norm, topi, topw, counts);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -372,6 +394,14 @@ ARTB_EXPORT int artb_moe_gather(const void* x, int ldx, const int* row_token, co
   if ((D & 7) || (ldx & 7) || (ldp & 7)) return ERR_BAD_SHAPE;
   moe_gather_kernel<<<cap_rows, 128, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx, row_token, row_w, use_w,
                                              total_rows, reinterpret_cast<__nv_bfloat16*>(xp), ldp, D);
+  return static_cast<int>(cudaGetLastError());
+}
+
+ARTB_EXPORT int artb_moe_gather_f32(const float* x, int ldx, const int* row_token, const int* total_rows, float* xp, int ldp, int D,
+                                    int cap_rows, cudaStream_t st) {
+  if (cap_rows <= 0) return 0;
+  if (D <= 0 || ldx < D || ldp < D) return ERR_BAD_SHAPE;
+  moe_gather_f32_kernel<<<cap_rows, 128, 0, st>>>(x, ldx, row_token, total_rows, xp, ldp, D);
   return static_cast<int>(cudaGetLastError());
 }
 

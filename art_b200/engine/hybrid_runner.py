@@ -3,14 +3,16 @@
 One batch is ragged: every sequence brings its next tokens, whether one decoded token or a portion of its prompt, and all
 of them go through the layers together.  ``Ragged`` describes it to the kernels: rows of the sequences one after another
 (``cu_q``), positions, cache rows, block tables, state slots.  Sequences with few new tokens come first, so that a row
-range tells which form of attention a row takes: short ones attend to the cached latents themselves (absorbed form), longer
-portions to keys and values expanded for their window.
+range tells which form of attention a row takes: short ones read the cache where it lies (latent attention: the absorbed
+form), longer portions gather what they see and run on prompt kernels (latent attention: expanded keys and values).
 
 A batch of single tokens (decoding) leaves its projections as split-K partial sums in fp32 workspaces, which the kernel
 that follows finishes and clears, as the engine's other models do.
 
-Every sublayer is ``norm -> mixer or feed-forward -> norm -> residual``; the step from one to the next (post-norm, residual
-multiplier, depth average, next input norm) is one kernel over the fp32 residual stream (``ops.hybrid.residual_step``).
+Every sublayer is ``norm -> mixer or feed-forward -> (norm ->) residual``; the step from one to the next (a mixture's weighted
+sum, bias, post-norm, residual multiplier, depth average, next input norm: what the design has of them) is one kernel over
+the fp32 residual stream (``ops.hybrid.residual_step``).  Mixers side by side share one input and one output product: their
+factors scale what enters the latter.
 Operands of the matrix products are bf16; with ``dtype=torch.float32`` everything is fp32, products included, through the
 same layer code.
 
@@ -23,9 +25,9 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..models.hybrid import SHIFT_MIXES, HybridConfig, check_weights
+from ..models.hybrid import PART_NAMES, SHIFT_MIXES, HybridConfig, LayerSpec, check_weights
 from ..ops import hybrid as hy
-from ..ops.hybrid import Out, as_out, pad
+from ..ops.hybrid import Out, Sublayer, as_out, pad
 from .runner import DeviceRunner, SeqView
 
 
@@ -49,15 +51,15 @@ class Ragged:
     reach: int = 0              # upper bound of the tokens a short row may attend to
     plans: dict = field(default_factory=dict)
 
-    def plan(self, window: int) -> hy.PrefillPlan:
-        p = self.plans.get(window)
+    def plan(self, window: int, chunk: int = 0) -> hy.PrefillPlan:
+        p = self.plans.get((window, chunk))
         if p is None:
-            p = self.plans[window] = hy.plan_prefill(self.portions, window, self.tokens.device)
+            p = self.plans[window, chunk] = hy.plan_prefill(self.portions, window, self.tokens.device, chunk)
         return p
 
 
-# Portions up to this many tokens attend in latent space: expanding a window's keys and values for them would cost more
-# than the wider products of the absorbed form.
+# Portions up to this many tokens read the cache row by row: gathering (and, of latents, expanding) a window's keys and values
+# for them would cost more.
 ABSORB_MAX = 16
 # Sizes the tensor-core kernels hold in shared memory and registers; beyond them the scalar absorbed form serves.
 LATENT_TC_MAX = 768         # cached row: latent + rotated part
@@ -79,8 +81,8 @@ class HybridRunner(DeviceRunner):
         self.exact32 = dtype == torch.float32
         self.max_loras = max_loras
         self.dp = pad(cfg.hidden_size)
-        wide = any(s.type == "latent_attention" and (s.vdim > PREFILL_VALUE_MAX or pad(s.dim, 16) + pad(s.rot_dim, 16) > PREFILL_KEY_MAX)
-                   for s in cfg.layers)
+        wide = any(m.type in ("latent_attention", "attention") and
+                   (m.vdim > PREFILL_VALUE_MAX or pad(m.dim, 16) + pad(m.rot_dim, 16) > PREFILL_KEY_MAX) for s in cfg.layers for m in s.mixers())
         self.absorb_max = 1 << 30 if self.exact32 or wide else ABSORB_MAX
         self._load(base)
         self._buf: dict = {}
@@ -105,57 +107,142 @@ class HybridRunner(DeviceRunner):
         out[:d, :, :vdim] = w.to(self.device).view(d, heads, vdim)
         return out.view(self.dp, heads * vp)
 
+    def _glu(self, gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+        """gate | up as one operand, rows interleaved in blocks of 16; the width is padded to a multiple of 16."""
+        ff = pad(gate.shape[0], 16)
+        g, u = self._mat(gate, ff, self.dp), self._mat(up, ff, self.dp)
+        return torch.stack([g.view(-1, 16, self.dp), u.view(-1, 16, self.dp)], 1).reshape(2 * ff, self.dp)
+
     def _load(self, base: dict[str, torch.Tensor]) -> None:
         cfg, dp = self.cfg, self.dp
-        V = cfg.vocab_size
-        self._head = self._mat(base["embed"], pad(V), dp)          # embedding and output table are one
-        self.embed = self.lm_head = self._head[:V]
-        self.embed_norm, self.final_norm = self._vec(base["embed.norm"], dp), self._vec(base["final.norm"], dp)
+        V, d = cfg.vocab_size, cfg.hidden_size
+        table = self._mat(base["embed"], pad(V), dp)
+        self._head = table if cfg.tie_word_embeddings else self._mat(base["head"], pad(V), dp)
+        self.embed, self.lm_head = table[:V], self._head[:V]
+
+        def norm(w: torch.Tensor) -> torch.Tensor:
+            out = self._vec(w, dp)
+            out[:d] += cfg.norm_offset
+            return out
+
+        self.embed_norm = norm(base["embed.norm"]) if cfg.embed_norm else None
+        self.final_norm = norm(base["final.norm"])
+        self.pos_freq = None
+        if cfg.position_base > 0:
+            self.pos_freq = torch.tensor([cfg.position_base ** (-2.0 * i / d) for i in range(dp // 2)], dtype=torch.float64).to(self.device)
         self.layers = []
         for i, s in enumerate(cfg.layers):
             w = {k[len(f"l{i}."):]: t for k, t in base.items() if k.startswith(f"l{i}.")}
             m = {k[4:]: t for k, t in w.items() if k.startswith("mix.")}
-            L: dict = {"norm1": self._vec(w["norm1"], dp), "norm1b": self._vec(w["norm1b"], dp), "dwa": self._vec(w["dwa"])}
-            if s.type == "latent_attention":
-                rank_p = pad(s.kv_rank, 16)
-                L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, dp)
-                L["tc_dv"] = hy.prefill_tc_values(s.dim, s.rot_dim, s.vdim, s.scale)
-                dk, dv = pad(s.dim, 16), L["tc_dv"] or pad(s.vdim, 16)
-                L["c_norm"] = self._vec(m["dkv.norm"])
-                uk, uv = m["uk"].view(s.heads, s.dim, s.kv_rank), m["uv"].view(s.heads, s.vdim, s.kv_rank)
-                L["uk_t"] = torch.zeros(s.heads, rank_p, pad(s.dim, 16), dtype=self.dtype, device=self.device)
-                L["uk_t"][:, :s.kv_rank, :s.dim] = uk.transpose(1, 2).to(self.device)
-                L["uv"] = torch.zeros(s.heads, pad(s.vdim), rank_p, dtype=self.dtype, device=self.device)
-                L["uv"][:, :s.vdim, :s.kv_rank] = uv.to(self.device)
-                if not self.exact32:       # keys of all heads, then values of all heads, from a latent
-                    kv = torch.zeros(s.heads * (dk + dv), rank_p, dtype=self.dtype, device=self.device)
-                    kv[:s.heads * dk].view(s.heads, dk, rank_p)[:, :s.dim, :s.kv_rank] = uk.to(self.device)
-                    kv[s.heads * dk:].view(s.heads, dv, rank_p)[:, :s.vdim, :s.kv_rank] = uv.to(self.device)
-                    L["ukv"] = kv
-                L["inv_freq"] = torch.tensor([s.rope_base ** (-2.0 * j / s.rot_dim) for j in range(s.rot_dim // 2)], dtype=torch.float64
-                                             ).to(self.device, torch.float32)
-            elif s.type == "hgrn2":
-                qv, f = self._mat(torch.cat([m["q"], m["v"]], 0), None, dp), self._mat(m["f"], None, dp)
-                L["qvf"] = torch.cat([qv, f], 0)
-                L["qv"], L["f"] = L["qvf"][:qv.shape[0]], L["qvf"][qv.shape[0]:]
-                L["f_b"], L["lower"] = self._vec(m["f.b"]), self._vec(m["lower"])
-                L["o_norm"] = self._vec(m["norm"])
-            else:
-                n = pad(s.heads * s.dim)
-                L["mu"] = torch.stack([self._vec(m["mu." + x], dp) for x in SHIFT_MIXES])
-                L["rkvg"] = torch.stack([self._mat(m[x], n, dp) for x in "rkvg"])
-                rp = pad(s.decay_rank)
-                L["w1"] = self._mat(m["w1"], rp, dp)
-                w2 = self._mat(m["w2"], n, rp)
-                # bf16: tanh arrives as a pair (high part, remainder), both halves against the same matrix
-                L["w2"] = w2 if self.exact32 else torch.cat([w2, w2], 1).contiguous()
-                L["w0"], L["u"], L["o_norm"] = self._vec(m["w0"]), self._vec(m["u"]), self._vec(m["norm"])
-            L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
-            if s.ff:
-                L["norm2"], L["norm2b"] = self._vec(w["norm2"], dp), self._vec(w["norm2b"], dp)
-                L["up"], L["down"] = self._mat(w["mlp.up"], None, dp), self._mat(w["mlp.down"], dp, pad(s.ff))
-                L["act"] = self._vec(w["mlp.act"])
+            L: dict = {n: norm(w[n]) for n in ("norm1", "norm1b", "norm2", "norm2b") if n in w}
+            L["dwa"] = self._vec(w["dwa"]) if cfg.depth_average else None
+            getattr(self, "_load_" + s.type)(s, m, L)
+            if s.has_mlp:
+                getattr(self, "_load_mlp_" + s.mlp)(s, {k[4:]: t for k, t in w.items() if k.startswith("mlp.")}, L)
             self.layers.append(L)
+
+    def _load_latent_attention(self, s: LayerSpec, m: dict, L: dict) -> None:
+        rank_p = pad(s.kv_rank, 16)
+        L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, self.dp)
+        L["tc_dv"] = hy.prefill_tc_values(s.dim, s.rot_dim, s.vdim, s.scale)
+        dk, dv = pad(s.dim, 16), L["tc_dv"] or pad(s.vdim, 16)
+        L["c_norm"] = self._vec(m["dkv.norm"])
+        uk, uv = m["uk"].view(s.heads, s.dim, s.kv_rank), m["uv"].view(s.heads, s.vdim, s.kv_rank)
+        L["uk_t"] = torch.zeros(s.heads, rank_p, pad(s.dim, 16), dtype=self.dtype, device=self.device)
+        L["uk_t"][:, :s.kv_rank, :s.dim] = uk.transpose(1, 2).to(self.device)
+        L["uv"] = torch.zeros(s.heads, pad(s.vdim), rank_p, dtype=self.dtype, device=self.device)
+        L["uv"][:, :s.vdim, :s.kv_rank] = uv.to(self.device)
+        if not self.exact32:       # keys of all heads, then values of all heads, from a latent
+            kv = torch.zeros(s.heads * (dk + dv), rank_p, dtype=self.dtype, device=self.device)
+            kv[:s.heads * dk].view(s.heads, dk, rank_p)[:, :s.dim, :s.kv_rank] = uk.to(self.device)
+            kv[s.heads * dk:].view(s.heads, dv, rank_p)[:, :s.vdim, :s.kv_rank] = uv.to(self.device)
+            L["ukv"] = kv
+        L["inv_freq"] = torch.tensor([s.rope_base ** (-2.0 * j / s.rot_dim) for j in range(s.rot_dim // 2)], dtype=torch.float64
+                                     ).to(self.device, torch.float32)
+        L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
+
+    def _load_hgrn2(self, s: LayerSpec, m: dict, L: dict) -> None:
+        qv, f = self._mat(torch.cat([m["q"], m["v"]], 0), None, self.dp), self._mat(m["f"], None, self.dp)
+        L["qvf"] = torch.cat([qv, f], 0)
+        L["qv"], L["f"] = L["qvf"][:qv.shape[0]], L["qvf"][qv.shape[0]:]
+        L["f_b"], L["lower"] = self._vec(m["f.b"]), self._vec(m["lower"])
+        L["o_norm"] = self._vec(m["norm"])
+        L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
+
+    def _load_wkv(self, s: LayerSpec, m: dict, L: dict) -> None:
+        n = pad(s.heads * s.dim)
+        L["mu"] = torch.stack([self._vec(m["mu." + x], self.dp) for x in SHIFT_MIXES])
+        L["rkvg"] = torch.stack([self._mat(m[x], n, self.dp) for x in "rkvg"])
+        rp = pad(s.decay_rank)
+        L["w1"] = self._mat(m["w1"], rp, self.dp)
+        w2 = self._mat(m["w2"], n, rp)
+        # bf16: tanh arrives as a pair (high part, remainder), both halves against the same matrix
+        L["w2"] = w2 if self.exact32 else torch.cat([w2, w2], 1).contiguous()
+        L["w0"], L["u"], L["o_norm"] = self._vec(m["w0"]), self._vec(m["u"]), self._vec(m["norm"])
+        L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
+
+    def _load_lightning(self, s: LayerSpec, m: dict, L: dict) -> None:
+        L["qkvg"] = self._mat(torch.cat([m["q"], m["k"], m["v"], m["g"]], 0), None, self.dp)
+        L["decay"] = torch.tensor(s.decay, dtype=torch.float64).to(self.device, torch.float32)
+        L["o_norm"] = self._vec(m["norm"])
+        L["o"] = self._heads_in(m["o"], 1, s.heads * s.vdim)
+
+    def _load_parts(self, s: LayerSpec, m: dict, L: dict) -> None:
+        """Mixers side by side: their input matrices one below the other (each from a multiple of 8 rows on), their output
+        matrices side by side."""
+        scales = s.part_scales or (1.0,)
+        rows, cols, bias = [], [], torch.zeros(self.dp, dtype=torch.float32, device=self.device)
+        L["parts"] = []
+        for p, name, scale in zip(s.mixers(), PART_NAMES, scales):
+            w = {k[len(name) + 1:]: t for k, t in m.items() if k.startswith(name + ".")} if s.parts else m
+            P: dict = {"in": sum(r.shape[0] for r in rows), "out": sum(c.shape[1] for c in cols), "scale": scale}
+            r, c = getattr(self, "_load_part_" + p.type)(p, w, P)
+            rows.append(r)
+            cols.append(c)
+            if "o.b" in w:
+                bias[:self.cfg.hidden_size] += scale * self._vec(w["o.b"])
+            L["parts"].append(P)
+        L["in"], L["o"] = torch.cat(rows, 0), torch.cat(cols, 1)
+        L["o_bias"] = bias if any(p.biases for p in s.mixers()) else None
+
+    _load_parallel = _load_attention = _load_rglru = _load_parts
+
+    def _load_part_attention(self, s: LayerSpec, w: dict, P: dict):
+        P["bias"] = self._vec(torch.cat([w[k + ".b"] for k in "qkv"])) if s.biases else None
+        P["tc_dv"] = hy.prefill_tc_values(s.dim, 0, s.vdim, s.scale)
+        P["dvp"] = hy.gqa_value_columns(s.dim, s.vdim, s.scale)
+        return self._mat(torch.cat([w[k] for k in "qkv"], 0), None, self.dp), self._heads_in(w["o"], s.heads, s.vdim)
+
+    def _load_part_rglru(self, s: LayerSpec, w: dict, P: dict):
+        n, bp = s.heads * s.dim, pad(s.dim)
+        gates = torch.zeros(s.heads, 2, bp, bp, dtype=self.dtype, device=self.device)
+        for j, k in enumerate(("ra", "ri")):
+            gates[:, j, :s.dim, :s.dim] = w[k].to(self.device)
+        gates = gates.view(s.heads, 2 * bp, bp)
+        # bf16: the convolution's output arrives as a pair (high part, remainder), both halves against the same matrix
+        P["gates"] = gates if self.exact32 else torch.cat([gates, gates], 2).contiguous()
+        P["y_b"], P["x_b"], P["r_b"], P["i_b"] = (self._vec(w[k]) for k in ("y.b", "x.b", "ra.b", "ri.b"))
+        P["conv"], P["conv_b"] = w["conv"].to(self.device, torch.float32).contiguous(), self._vec(w["conv.b"])
+        P["decay"] = (8.0 * torch.nn.functional.softplus(self._vec(w["lam"]).double())).float()
+        P["x_col"] = pad(n)
+        return torch.cat([self._mat(w["y"], pad(n), self.dp), self._mat(w["x"], pad(n), self.dp)], 0), self._mat(w["o"], self.dp, pad(n))
+
+    def _load_mlp_poly(self, s: LayerSpec, w: dict, L: dict) -> None:
+        L["up"], L["down"], L["act"] = self._mat(w["up"], None, self.dp), self._mat(w["down"], self.dp, pad(s.ff)), self._vec(w["act"])
+
+    def _load_mlp_gated(self, s: LayerSpec, w: dict, L: dict) -> None:
+        L["gu"], L["down"] = self._glu(w["gate"], w["up"]), self._mat(w["down"], self.dp, pad(s.ff, 16))
+
+    def _load_mlp_moe(self, s: LayerSpec, w: dict, L: dict) -> None:
+        ffp = pad(s.expert_ff, 16)
+        L["router"], L["router_b"] = self._mat(w["router"], None, self.dp), self._vec(w["router.b"])
+        L["e_gu"] = torch.empty(s.experts * 2 * ffp, self.dp, dtype=self.dtype, device=self.device)
+        L["e_down"] = torch.empty(s.experts * self.dp, ffp, dtype=self.dtype, device=self.device)
+        for e in range(s.experts):
+            L["e_gu"][e * 2 * ffp:(e + 1) * 2 * ffp] = self._glu(w[f"e{e}.gate"], w[f"e{e}.up"])
+            L["e_down"][e * self.dp:(e + 1) * self.dp] = self._mat(w[f"e{e}.down"], self.dp, ffp)
+        if s.shared_ff:
+            L["gu"], L["down"] = self._glu(w["shared.gate"], w["shared.up"]), self._mat(w["shared.down"], self.dp, pad(s.shared_ff, 16))
 
     def set_adapter(self, slot: int, state) -> None:
         if state is not None:
@@ -178,22 +265,32 @@ class HybridRunner(DeviceRunner):
     def _mm_take(self, b: Ragged, name: str, x, W, f32: bool = False) -> Out:
         """``x W^T`` for a consumer that accepts a split-K workspace: with few rows the product streams the weights from
         all SMs and adds partial sums into the fp32 workspace ``name``, which the consumer reads once and leaves zero."""
-        from ..ops.gemm import gemm_splitk_, gemm_tn, plan_small_m
+        from ..ops.gemm import gemm_splitk_, gemm_tn
 
-        M, N, K = b.M, W.shape[0], W.shape[1]
-        if not b.single or self.exact32 or M > 512:
+        M, N = b.M, W.shape[0]
+        bn, splits, pair = self._small_plan(b, W)
+        if bn == 0 and not pair:
             return self._mm(x, W, f32)
-        pair = M % 256 == 0 and N >= 256
-        bn, splits = plan_small_m(M, N, K, pair=pair)
         if splits == 1:
-            return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16, bn=0 if pair else bn, two_cta=pair))
+            return as_out(gemm_tn(x, W, out_dtype=torch.float32 if f32 else torch.bfloat16, bn=bn, two_cta=pair))
         rows = next(n for n in self.BUCKETS if n >= M)
         key = ("ws", name, N, rows)
         ws = self._buf.get(key)
         if ws is None:
             ws = self._buf[key] = torch.zeros((rows, N), dtype=torch.float32, device=self.device)
-        gemm_splitk_(ws, x, W, bn, splits, two_cta=pair)
+        gemm_splitk_(ws, x, W, bn, splits, two_cta=bool(pair))
         return Out(ws[:M], hy.KIND_TAKE)
+
+    def _small_plan(self, b: Ragged, W) -> tuple[int, int, bool | None]:
+        """``(tile width, splits, CTA pairs)`` of a decode batch's product; ``(0, 1, None)``: the plain product's own choice."""
+        from ..ops.gemm import plan_small_m
+
+        M, N, K = b.M, W.shape[0], W.shape[1]
+        if not b.single or self.exact32 or M > 512:
+            return 0, 1, None
+        pair = M % 256 == 0 and N >= 256
+        bn, splits = plan_small_m(M, N, K, pair=pair)
+        return 0 if pair and splits == 1 else bn, splits, pair
 
     def _logits(self, hidden) -> torch.Tensor:
         y = self._mm(hidden, self._head, f32=True).t
@@ -249,25 +346,60 @@ class HybridRunner(DeviceRunner):
         cfg, dp, d, eps, m = self.cfg, self.dp, self.cfg.hidden_size, self.cfg.norm_eps, self.cfg.residual_mult
         M, dev = b.M, self.device
         x, h = self._new(M, dp, torch.float32), self._new(M, dp)
-        hist = torch.empty((len(self.layers) + 1, M if M <= 1024 else pad(M, 1024), dp), dtype=torch.float32, device=dev)
+        hist = None
+        if cfg.depth_average:
+            hist = torch.empty((len(self.layers) + 1, M if M <= 1024 else pad(M, 1024), dp), dtype=torch.float32, device=dev)
         first_norm = lambda i: (self.layers[i]["norm1"] if cfg.layers[i].type != "wkv" else None) if i < len(self.layers) \
             else (self.final_norm if want_hidden else None)      # noqa: E731  (a token-shift mixer norms its own input)
-        hy.residual_step(x, self.embed_norm, d, eps, tokens=b.tokens, table=self.embed, hist=hist, hist_n=0, w_next=first_norm(0), h=h)
+        hy.residual_step(x, self.embed_norm, d, eps, mult=cfg.embed_scale, tokens=b.tokens, table=self.embed, freq=self.pos_freq, pos=b.pos,
+                         hist=hist, hist_n=0, w_next=first_norm(0), h=h)
         for i, (s, L) in enumerate(zip(cfg.layers, self.layers)):
-            y = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b)
-            post = L["norm1b"]
-            if s.ff:
-                hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
-                z = self._mm_take(b, "up", h, L["up"])
-                a = self._new(M, pad(s.ff))
-                y = self._mm_take(b, "down", hy.poly_norm(z, L["act"], a, s.ff, eps), L["down"])
-                post = L["norm2b"]
-            hy.residual_step(x, post, d, eps, y=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
+            y, post = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b), L.get("norm1b")
+            if s.has_mlp:
+                hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
+                y, post = getattr(self, "_mlp_" + s.mlp)(s, L, h, b), L.get("norm2b")
+            hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
             if capture is not None:
                 capture.append(x[:, :d].clone())
         return x, h
 
-    def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Out:
+    # -- feed-forwards ----------------------------------------------------------------------------------------
+    def _mlp_poly(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+        z = self._mm_take(b, "up", h, L["up"])
+        a = self._new(b.M, pad(s.ff))
+        return Sublayer(self._mm_take(b, "down", hy.poly_norm(z, L["act"], a, s.ff, self.cfg.norm_eps), L["down"]))
+
+    def _glu_product(self, b: Ragged, name: str, h, W, act: str) -> torch.Tensor:
+        """``act(h gate^T) * (h up^T)``: the activation in the product's epilogue where the product is not split."""
+        a = self._new(b.M, W.shape[0] // 2)
+        if not self.exact32 and self._small_plan(b, W)[1] == 1:
+            from ..ops.gemm import gemm_tn
+
+            bn, _, pair = self._small_plan(b, W)
+            gemm_tn(h, W, swiglu_out=a, gate_act=act, keep_preact=False, bn=bn, two_cta=pair)
+            return a
+        return hy.gated_act(self._mm_take(b, name, h, W), a, act)
+
+    def _mlp_gated(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+        return Sublayer(self._mm_take(b, "down", self._glu_product(b, "gu", h, L["gu"], s.act), L["down"]))
+
+    def _mlp_moe(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+        from ..ops import moe
+
+        z = self._mm_take(b, "router", h, L["router"], f32=True)
+        plan = moe.route(z.t[:, :s.experts], s.top, True, L["router_b"], take=z.kind == hy.KIND_TAKE)
+        xp, n = moe.gather(h, plan), L["e_down"].shape[1]
+        a = torch.empty((plan.cap_rows, n), dtype=self.dtype, device=self.device)
+        if self.exact32:
+            hy.gated_act(as_out(moe.grouped_gemm(xp, L["e_gu"], plan, 2 * n)), a, "silu")
+        else:
+            moe.grouped_gemm(xp, L["e_gu"], plan, 2 * n, swiglu_out=a, keep_preact=False)
+        rows = moe.grouped_gemm(a, L["e_down"], plan, self.dp)
+        y = self._mm_take(b, "down", self._glu_product(b, "gu", h, L["gu"], "silu"), L["down"]) if s.shared_ff else None
+        return Sublayer(y, rows=rows, pos=plan.pos, weight=plan.topw)
+
+    # -- mixers -------------------------------------------------------------------------------------------------
+    def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Sublayer:
         M, H, n_abs = b.M, s.heads, b.n_abs
         cache = self.kv.layers[i]["latent"]
         p = self._mm_take(b, "qkv", h, L["qkv"])
@@ -296,12 +428,12 @@ class HybridRunner(DeviceRunner):
             if L["tc_dv"]:
                 k, vt = self._mm(c[:, :rank_p], L["ukv"][:H * dk]).t, self._mm(L["ukv"][H * dk:], c[:, :rank_p]).t
                 hy.latent_prefill_tc(qe, k, vt, c, plan, s.window, s.scale, o[n_abs:], H, dk, L["tc_dv"], rank_p, rot_p, s.vdim)
-                return self._mm_take(b, "o", o, L["o"])
+                return Sublayer(self._mm_take(b, "o", o, L["o"]))
             kv = self._mm(c[:, :rank_p], L["ukv"]).t
             hy.latent_prefill(qe, kv, c, plan, s.window, s.scale, o[n_abs:], H, dk, dv, rank_p, rot_p, s.vdim)
-        return self._mm_take(b, "o", o, L["o"])
+        return Sublayer(self._mm_take(b, "o", o, L["o"]))
 
-    def _scan(self, mode, i, s, L, q, k, v, g, aux, bias, gate, b: Ragged) -> Out:
+    def _scan(self, mode, i, s, L, q, k, v, g, aux, bias, gate, b: Ragged) -> Sublayer:
         """Recurrence, per-head norm and gate, output projection."""
         M, H, vp, eps = b.M, s.heads, pad(s.vdim), self.cfg.norm_eps
         state = self.kv.layers[i]["state"]
@@ -314,9 +446,9 @@ class HybridRunner(DeviceRunner):
             o = self._new(M, H * s.vdim, torch.float32)
             hy.linear_scan(mode, q, k, v, g, bias, aux, state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, H, s.dim, s.vdim, o)
             hy.head_norm(o, L["o_norm"], per_head, H, s.vdim, vp, out, eps, gate)
-        return self._mm_take(b, "o", out, L["o"])
+        return Sublayer(self._mm_take(b, "o", out, L["o"]))
 
-    def _mix_hgrn2(self, i, s, L, x, h, b: Ragged) -> Out:
+    def _mix_hgrn2(self, i, s, L, x, h, b: Ragged) -> Sublayer:
         if b.single:        # one product, its outputs are taken where they lie
             p = self._mm_take(b, "qvf", h, L["qvf"], f32=True)
             qv, g = p, p.col(L["qv"].shape[0])
@@ -324,7 +456,7 @@ class HybridRunner(DeviceRunner):
             qv, g = self._mm(h, L["qv"]), self._mm(h, L["f"], f32=True)
         return self._scan(hy.SCAN_HGRN2, i, s, L, qv, None, qv.col(s.heads * s.dim), g, L["lower"], L["f_b"], None, b)
 
-    def _mix_wkv(self, i, s, L, x, h, b: Ragged) -> Out:
+    def _mix_wkv(self, i, s, L, x, h, b: Ragged) -> Sublayer:
         M, n = b.M, L["rkvg"].shape[1]
         mixes = self._heads_buf("mix", len(SHIFT_MIXES), M, b, self.dp)
         hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
@@ -343,6 +475,65 @@ class HybridRunner(DeviceRunner):
         g = self._mm(hy.split_tanh(z, s.decay_rank, rp, t), L["w2"], f32=True)
         y = as_out(y)
         return self._scan(hy.SCAN_WKV, i, s, L, y, y.col(n), y.col(2 * n), g, L["u"], L["w0"], y.col(3 * n), b)
+
+    def _mix_lightning(self, i, s, L, x, h, b: Ragged) -> Sublayer:
+        M, n, nv = b.M, s.heads * s.dim, s.heads * s.vdim
+        p = self._mm_take(b, "qkvg", h, L["qkvg"])
+        q, k, v, gate = p, p.col(n), p.col(2 * n), p.col(2 * n + nv)
+        state = self.kv.layers[i]["state"]
+        o, out = self._new(M, nv, torch.float32), self._new(M, pad(nv))
+        if b.single:
+            hy.linear_decode(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, s.heads, s.dim, s.vdim, None, False,
+                             None, o, s.vdim, 0.0)
+        else:
+            hy.linear_scan(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, s.heads, s.dim, s.vdim, o)
+        hy.head_norm(o, L["o_norm"], False, 1, nv, pad(nv), out, self.cfg.norm_eps, gate, hy.GATE_SIGMOID)
+        return Sublayer(self._mm_take(b, "o", out, L["o"]))
+
+    def _mix_parts(self, i, s, L, x, h, b: Ragged) -> Sublayer:
+        p = self._mm_take(b, "in", h, L["in"])
+        o = self._new(b.M, L["o"].shape[1])
+        for j, (spec, P) in enumerate(zip(s.mixers(), L["parts"])):
+            getattr(self, "_part_" + spec.type)(spec, P, p.col(P["in"]), o[:, P["out"]:], self.kv.part(i, j), b)
+        return Sublayer(self._mm_take(b, "o", o, L["o"]), bias=L["o_bias"])
+
+    _mix_parallel = _mix_attention = _mix_rglru = _mix_parts
+
+    def _part_attention(self, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
+        M, n_abs, kv = b.M, b.n_abs, cache["kv"]
+        H, G, dk, dvp = s.heads, s.heads // s.kv_heads, pad(s.dim, 16), P["dvp"]
+        q = self._new(M, H * dk)
+        hy.gqa_finish(p, P["bias"], b.slot, kv, q, H, s.kv_heads, s.dim, s.vdim, dvp)
+        if n_abs:
+            args = (q, kv, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.chunk, s.scale, P["scale"], o, n_abs, H, s.kv_heads, s.dim, s.vdim, dvp)
+            if self.exact32 or max(dk, dvp) > hy.GQA_DECODE_MAX:
+                hy.gqa_attend(*args)
+            else:
+                reach = min([b.reach] + [w for w in (s.window, s.chunk) if w > 0])
+                hy.gqa_decode(*args, splits=hy.gqa_decode_splits(n_abs, s.kv_heads * ((G + 15) // 16), reach))
+        if n_abs < M:
+            plan = b.plan(s.window, s.chunk)
+            rest = dict(chunk=s.chunk, G=G, out_scale=P["scale"])
+            if P["tc_dv"]:
+                k, vt = hy.gqa_gather(kv, b.bt, plan, s.kv_heads, dk, dvp)
+                hy.latent_prefill_tc(q[n_abs:], k, vt, k, plan, s.window, s.scale, o[n_abs:], H, dk, dvp, 0, 0, s.vdim, **rest)
+            else:
+                c = hy.latent_gather(kv, b.bt, plan)
+                hy.latent_prefill(q[n_abs:], c, c, plan, s.window, s.scale, o[n_abs:], H, dk, dvp, 0, 0, s.vdim, **rest)
+
+    def _part_rglru(self, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
+        M, bp = b.M, pad(s.dim)
+        # a buffer of its own per block size: padding columns are written by nobody
+        u = self._heads_buf(f"u{s.dim}", s.heads, M, b, P["gates"].shape[2])
+        hy.short_conv(p.col(P["x_col"]), P["x_b"], P["conv"], P["conv_b"], cache["conv"], b.row_seq, b.cu_q, b.ctx, b.state_slot, b.n_seqs,
+                      b.single, u, s.dim, bp)
+        z = self._new(M, s.heads * 2 * bp, torch.float32)
+        hy.gemm_batched(u, P["gates"], z, M, c_batch=2 * bp)
+        n = s.heads * s.dim
+        if n % 8:      # columns between this part and the next: zero weights, but they must be numbers
+            o[:, n:pad(n)].zero_()
+        hy.rglru(u, z, P["r_b"], P["i_b"], P["decay"], p, P["y_b"], cache["state"], b.cu_q, b.ctx, b.state_slot, b.n_seqs, b.single, o, P["scale"],
+                 s.dim, bp)
 
     # -- the shared loops' hooks ------------------------------------------------------------------------------
     def _prompt_forward(self, seqs: list[SeqView], write_kv: bool = True):
@@ -381,9 +572,9 @@ class HybridRunner(DeviceRunner):
         st["state_slot"].copy_(torch.tensor([s.state_slot for s in seqs] + [-1] * (nb - len(seqs)), dtype=torch.int32), non_blocking=True)
 
     def _attn_splits(self, nb: int, max_ctx: int) -> int:
-        """Stands for how far the batch's tokens reach back (a power of two): the latent layers plan their splits by it.
-        Contexts beyond every window change nothing, so that they share one captured graph."""
-        windows = [s.window for s in self.cfg.layers if s.type == "latent_attention"]
+        """Stands for how far the batch's tokens reach back (a power of two): the attention layers plan their splits by it.
+        Contexts beyond every window and chunk change nothing, so that they share one captured graph."""
+        windows = [s.window or s.chunk for L in self.cfg.layers for s in L.mixers() if s.type in ("latent_attention", "attention")]
         if not windows:
             return 1
         bound = max_ctx if any(w <= 0 for w in windows) else min(max_ctx, max(windows))

@@ -276,13 +276,19 @@ class HybridCache:
 
     * latent attention: ``latent`` ``[num_blocks, block_size, rank_p + rot_p]``, paged, in the operand dtype; a row is the
       normed latent and the rotated key part, each padded with zeros to a multiple of 16;
-    * recurrent mixers: ``state`` fp32 ``[num_slots, heads, vdim, dim padded to 4]`` (a value column's channels are
-      contiguous), and for token-shift mixers ``shift`` fp32 ``[num_slots, width padded to 8]``, the last token's input.
+    * grouped-query attention: ``kv`` ``[num_blocks, block_size, kv_heads * (dim_p + vdim_p)]``, paged, in the operand dtype; a
+      row is the keys of all heads, then their values, each padded with zeros;
+    * linear attention: ``state`` fp32 ``[num_slots, heads, vdim, dim padded to 4]`` (a value column's channels are
+      contiguous), and for token-shift mixers ``shift`` fp32 ``[num_slots, width padded to 8]``, the last token's input;
+    * gated linear recurrent units: ``state`` fp32 ``[num_slots, channels]`` and ``conv`` fp32 ``[num_slots, taps - 1, channels]``,
+      the last inputs of the convolution.
 
-    ``state_slots`` hands out the slots; ``None`` for a model without recurrent layers.
+    A layer of several mixers holds the tensors of each, with the mixer's number in front (``0.kv``, ``1.state``); ``part``
+    picks one mixer's.  ``state_slots`` hands out the slots; ``None`` for a model without recurrent layers.
     """
 
     arena = None
+    PAGED = ("latent", "kv")
 
     def __init__(self, cfg, num_blocks: int, block_size: int, num_slots: int, device: torch.device,
                  dtype: torch.dtype = torch.bfloat16):
@@ -297,29 +303,49 @@ class HybridCache:
     @staticmethod
     def layer_shapes(cfg, spec, num_blocks: int, block_size: int, num_slots: int, dtype) -> dict[str, tuple[tuple[int, ...], torch.dtype]]:
         up = lambda n, m: (n + m - 1) // m * m      # noqa: E731
+        if spec.parts:
+            return {f"{j}.{k}": v for j, p in enumerate(spec.parts)
+                    for k, v in HybridCache.layer_shapes(cfg, p, num_blocks, block_size, num_slots, dtype).items()}
         if spec.type == "latent_attention":
             return {"latent": ((num_blocks, block_size, up(spec.kv_rank, 16) + up(spec.rot_dim, 16)), dtype)}
+        if spec.type == "attention":
+            from ..ops.hybrid import gqa_value_columns
+
+            return {"kv": ((num_blocks, block_size, spec.kv_heads * (up(spec.dim, 16) + gqa_value_columns(spec.dim, spec.vdim, spec.scale))), dtype)}
+        if spec.type == "rglru":
+            n = spec.heads * spec.dim
+            return {"state": ((num_slots, n), torch.float32), "conv": ((num_slots, max(1, spec.conv - 1), n), torch.float32)}
         out = {"state": ((num_slots, spec.heads, spec.vdim, up(spec.dim, 4)), torch.float32)}
         if spec.type == "wkv":
             out["shift"] = ((num_slots, up(cfg.hidden_size, 8)), torch.float32)
         return out
 
-    @classmethod
-    def bytes_per_block(cls, cfg, block_size: int, elem: int = 2) -> int:
-        return sum(block_size * shape[2] * elem for s in cfg.layers if not s.recurrent
-                   for shape, _ in cls.layer_shapes(cfg, s, 1, block_size, 1, None).values())
+    def part(self, layer: int, j: int) -> dict[str, torch.Tensor]:
+        """The tensors of mixer ``j`` of a layer."""
+        L = self.layers[layer]
+        if not self.cfg.layers[layer].parts:
+            return L
+        return {k.split(".", 1)[1]: t for k, t in L.items() if k.startswith(f"{j}.")}
 
     @classmethod
-    def bytes_per_slot(cls, cfg) -> int:
+    def _bytes(cls, cfg, block_size: int, paged: bool, elem: int) -> int:
         n = 0
         for s in cfg.layers:
-            if s.recurrent:
-                for shape, _ in cls.layer_shapes(cfg, s, 1, 1, 1, None).values():
-                    k = 4
+            for name, (shape, dt) in cls.layer_shapes(cfg, s, 1, block_size, 1, None).items():
+                if (name.split(".")[-1] in cls.PAGED) == paged:
+                    k = elem if dt is None else 4
                     for d in shape:
                         k *= d
                     n += k
         return n
+
+    @classmethod
+    def bytes_per_block(cls, cfg, block_size: int, elem: int = 2) -> int:
+        return cls._bytes(cfg, block_size, True, elem)
+
+    @classmethod
+    def bytes_per_slot(cls, cfg) -> int:
+        return cls._bytes(cfg, 1, False, 4)
 
     def _allocate(self) -> None:
         nb, bs = self.shape

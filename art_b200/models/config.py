@@ -14,7 +14,7 @@ import json
 import os
 from dataclasses import asdict, dataclass, field
 
-from .hybrid import ARCHITECTURES, HYBRID_PRESETS, HybridConfig
+from .hybrid import HYBRID_PRESETS, HybridConfig
 
 
 @dataclass
@@ -243,10 +243,7 @@ PRESETS: dict[str, ModelConfig] = {
 def config_from_dict(d: dict, name: str = "hf") -> "ModelConfig | HybridConfig":
     """The configuration class a ``config.json`` asks for."""
     if "architecture" in d:
-        make = ARCHITECTURES.get(d["architecture"])
-        if make is None:
-            raise ValueError(f"architecture {d['architecture']!r} is not supported (supported: {', '.join(ARCHITECTURES)})")
-        return make(d, name)
+        return HybridConfig.from_design_dict(d, name)
     return ModelConfig.from_hf_dict(d, name)
 
 

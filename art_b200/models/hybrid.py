@@ -1,9 +1,15 @@
-"""Hybrid decoders: models whose layers are listed one by one, each with its own sequence mixer.
+"""Hybrid decoders: models whose layers are listed one by one, each with its own sequence mixer and feed-forward.
 
-A hybrid configuration names, per layer, a mixer (latent attention with a sliding window, HGRN2 linear attention,
-RWKV-style time mixing) with its sizes, and a feed-forward (dense PolyNorm, or none).  The frame around the sublayers is
-fixed by the design: RMS norms before and after each sublayer, a residual multiplier, a weighted average over the results
-of all earlier layers, a normalised embedding, tied output.
+A configuration consists of layers and of the frame around them.  A layer (``LayerSpec``) names
+
+* a mixer: latent attention with a sliding window, grouped-query attention with a window or in chunks, HGRN2 or lightning
+  linear attention, RWKV-style time mixing, a gated linear recurrent unit behind a short convolution, or several of these
+  side by side on the same input, each with a factor (``parts``);
+* a feed-forward: PolyNorm, gated (``act(gate) * up``), a mixture of gated experts with an optional shared expert, or none.
+
+The frame (fields of ``HybridConfig``) is the design's: norms before, or before and after each sublayer, norm weights stored
+as they are or around zero, a residual multiplier, a weighted average over the results of all earlier layers, an embedding
+that is normalised, or scaled and given sinusoidal position vectors, an output table of its own or the embedding's.
 
 ``HybridConfig`` answers the questions the engine asks of any configuration (``vocab_size``, ``hidden_size``,
 ``num_layers``, ``is_moe`` ...); ``from_design_dict`` reads a ``config.json`` whose ``architecture`` key names a design of
@@ -12,34 +18,59 @@ it.  The reference serves library models only (src/art/local/state.py); designs 
 """
 from __future__ import annotations
 
+import dataclasses
 from dataclasses import dataclass, field
 
 import torch
 
-MIXERS = ("latent_attention", "hgrn2", "wkv")
 SHIFT_MIXES = ("r", "k", "v", "g", "w")        # inputs of the token-shift mixer, in the order its kernels use
+PART_NAMES = ("left", "right")                 # tensors of a parallel mixer's parts
+RECURRENT = ("hgrn2", "wkv", "lightning", "rglru")
+MAX_EXPERTS, MAX_TOP = 256, 16                 # what the router kernel holds
 
 
 @dataclass
 class LayerSpec:
-    """One layer: mixer type, the mixer's sizes and constants, width of the feed-forward (0: none)."""
+    """One layer: mixer type, the mixer's sizes and constants, and its feed-forward."""
     type: str
-    heads: int
-    dim: int
+    heads: int                                 # rglru: blocks of its gate matrices
+    dim: int                                   # rglru: channels per block
     vdim: int
-    ff: int = 0
-    # latent attention
+    ff: int = 0                                # width of a dense feed-forward, 0: none
+    # attention
     rot_dim: int = 0
     kv_rank: int = 0
+    kv_heads: int = 0
     scale: float = 1.0
     rope_base: float = 10000.0
     window: int = 0                            # keys seen, the token itself included; 0: all earlier ones
+    chunk: int = 0                             # keys of the same chunk of the sequence only; 0: all earlier ones
+    biases: bool = False                       # q, k, v and output projections have biases
     # wkv: width of the low-rank decay projection (given by its tensors, not by the configuration)
     decay_rank: int = 0
+    decay: tuple[float, ...] = ()              # lightning: one factor per head
+    conv: int = 1                              # rglru: taps of the short convolution
+    parts: tuple["LayerSpec", ...] = ()        # parallel: mixers side by side, and the factor of each one's result
+    part_scales: tuple[float, ...] = ()
+    # feed-forward: "poly" (up, PolyNorm, down), "gated" (act(gate) * up, down) or "moe" (gated experts)
+    mlp: str = "poly"
+    act: str = "silu"
+    experts: int = 0
+    top: int = 0
+    expert_ff: int = 0
+    shared_ff: int = 0                         # gated shared expert, 0: none
 
     @property
     def recurrent(self) -> bool:
-        return self.type != "latent_attention"
+        return self.type in RECURRENT or any(p.recurrent for p in self.parts)
+
+    @property
+    def has_mlp(self) -> bool:
+        return self.ff > 0 or self.experts > 0
+
+    def mixers(self) -> tuple["LayerSpec", ...]:
+        """The single mixers of the layer."""
+        return self.parts or (self,)
 
 
 @dataclass
@@ -52,9 +83,16 @@ class HybridConfig:
     residual_mult: float = 1.0
     family: str = "nikelix"
     max_position_embeddings: int = 1 << 20
+    # the frame
+    post_norms: bool = True                    # a norm behind each sublayer, too
+    depth_average: bool = True                 # layer results are averaged with all earlier ones
+    norm_offset: float = 0.0                   # added to the weights of the frame's norms
+    embed_norm: bool = True
+    embed_scale: float = 1.0
+    position_base: float = 0.0                 # sinusoidal position vectors of this base are added to the embedding; 0: none
+    tie_word_embeddings: bool = True
 
-    is_moe = False
-    tie_word_embeddings = True
+    is_moe = False                             # of the trainable families
 
     @property
     def num_layers(self) -> int:
@@ -76,62 +114,148 @@ class HybridConfig:
 
     @classmethod
     def from_design_dict(cls, d: dict, name: str = "hybrid") -> "HybridConfig":
-        layers = []
-        for i, e in enumerate(d["layers"]):
-            kind, m, mlp = e["type"], e["mixer"], e.get("mlp")
-            if kind not in MIXERS:
-                raise ValueError(f"layer {i}: mixer {kind!r} is not supported (supported: {', '.join(MIXERS)})")
-            if mlp is not None and mlp.get("kind", "dense") != "dense":
-                raise ValueError(f"layer {i}: feed-forward kind {mlp.get('kind')!r} is not supported (supported: dense)")
-            spec = LayerSpec(kind, int(m["heads"]), int(m["dim"]), int(m.get("vdim", m["dim"])), int(mlp["ff"]) if mlp else 0)
-            if kind == "latent_attention":
-                rot = m["rot"]
-                spec.rot_dim, spec.kv_rank = int(m["rot_dim"]), int(m["kv_rank"])
-                spec.scale, spec.rope_base = float(m["scale"]), float(rot["base"])
-                spec.window = int((m.get("mask") or {}).get("size", 0))
-                if int(rot.get("dims", spec.rot_dim)) != spec.rot_dim:
-                    raise ValueError(f"layer {i}: rot.dims must equal rot_dim (the whole rotated part turns)")
-                if spec.rot_dim % 2:
-                    raise ValueError(f"layer {i}: rot_dim must be even")
-            layers.append(spec)
-        return cls(name=name, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
-                   norm_eps=float(d["norm"]["eps"]), residual_mult=float(d["residual_mult"]),
-                   family=str(d["architecture"]).lower())
+        design = d["architecture"]
+        if design not in ARCHITECTURES:
+            raise ValueError(f"architecture {design!r} is not supported (supported: {', '.join(ARCHITECTURES)})")
+        cfg = ARCHITECTURES[design](d, name)
+        for i, s in enumerate(cfg.layers):
+            _check_layer(i, s)
+        return cfg
 
 
-ARCHITECTURES = {"Nikelix": HybridConfig.from_design_dict}
+def _check_layer(i: int, s: LayerSpec) -> None:
+    for p in s.mixers():
+        if p.type == "attention" and (p.kv_heads <= 0 or p.heads % p.kv_heads):
+            raise ValueError(f"layer {i}: {p.heads} query heads do not divide over {p.kv_heads} key heads")
+        if p.type == "lightning" and len(p.decay) != p.heads:
+            raise ValueError(f"layer {i}: {len(p.decay)} decay factors for {p.heads} heads")
+        if p.type in ("hgrn2", "wkv", "lightning") and max(p.dim, p.vdim) > 256:
+            raise ValueError(f"layer {i}: {p.type} heads of more than 256 columns are not supported")
+    if s.experts and not (0 < s.top <= min(s.experts, MAX_TOP) and s.experts <= MAX_EXPERTS):
+        raise ValueError(f"layer {i}: {s.top} of {s.experts} experts (at most {MAX_TOP} of {MAX_EXPERTS}) are not supported")
+
+
+def _mixer_kind(i: int, e: dict, supported: tuple[str, ...]) -> str:
+    if e["type"] not in supported:
+        raise ValueError(f"layer {i}: mixer {e['type']!r} is not supported (supported: {', '.join(supported)})")
+    return e["type"]
+
+
+def _mlp_kind(i: int, mlp: dict | None, supported: tuple[str, ...]) -> str | None:
+    if mlp is None:
+        return None
+    kind = mlp.get("kind", "dense")
+    if kind not in supported:
+        raise ValueError(f"layer {i}: feed-forward kind {kind!r} is not supported (supported: {', '.join(supported)})")
+    return kind
+
+
+def _read_nikelix(d: dict, name: str) -> HybridConfig:
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        kind, m, mlp = _mixer_kind(i, e, ("latent_attention", "hgrn2", "wkv")), e["mixer"], e.get("mlp")
+        _mlp_kind(i, mlp, ("dense",))
+        spec = LayerSpec(kind, int(m["heads"]), int(m["dim"]), int(m.get("vdim", m["dim"])), int(mlp["ff"]) if mlp else 0)
+        if kind == "latent_attention":
+            rot = m["rot"]
+            spec.rot_dim, spec.kv_rank = int(m["rot_dim"]), int(m["kv_rank"])
+            spec.scale, spec.rope_base = float(m["scale"]), float(rot["base"])
+            spec.window = int((m.get("mask") or {}).get("size", 0))
+            if int(rot.get("dims", spec.rot_dim)) != spec.rot_dim:
+                raise ValueError(f"layer {i}: rot.dims must equal rot_dim (the whole rotated part turns)")
+            if spec.rot_dim % 2:
+                raise ValueError(f"layer {i}: rot_dim must be even")
+        layers.append(spec)
+    return HybridConfig(name=name, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                        norm_eps=float(d["norm"]["eps"]), residual_mult=float(d["residual_mult"]), family="nikelix")
+
+
+def _read_naselorn(d: dict, name: str) -> HybridConfig:
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        kind, m, mlp = _mixer_kind(i, e, ("parallel", "lightning")), e["mixer"], e.get("mlp")
+        if kind == "lightning":
+            spec = LayerSpec(kind, int(m["heads"]), int(m["dim"]), int(m["vdim"]), decay=tuple(float(x) for x in m["decay"]))
+        else:
+            a, r = m["left"], m["right"]
+            width, blocks = int(r["width"]), int(r["blocks"])
+            if width % blocks:
+                raise ValueError(f"layer {i}: {width} channels do not divide over {blocks} blocks")
+            parts = (LayerSpec("attention", int(a["heads"]), int(a["dim"]), int(a["vdim"]), kv_heads=int(a["kv_heads"]), scale=float(a["scale"]),
+                               chunk=int(a["mask"]["size"]), biases=True),
+                     LayerSpec("rglru", blocks, width // blocks, width // blocks, conv=int(r["conv"])))
+            spec = LayerSpec(kind, 0, 0, 0, parts=parts, part_scales=(float(m["left_scale"]), float(m["right_scale"])))
+        ff = _mlp_kind(i, mlp, ("dense", "moe"))
+        if ff == "dense":
+            spec.mlp, spec.act, spec.ff = "gated", "relu", int(mlp["ff"])
+        elif ff == "moe":
+            spec.mlp, spec.expert_ff = "moe", int(mlp["expert"]["ff"])
+            spec.experts, spec.top = int(mlp["router"]["experts"]), int(mlp["router"]["top"])
+            spec.shared_ff = int(mlp["shared"]["ff"]) if mlp.get("shared") else 0
+        layers.append(spec)
+    return HybridConfig(name=name, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers, norm_eps=float(d["norm"]["eps"]),
+                        embed_scale=float(d["embedding"]["scale"]), **NASELORN_FRAME)
+
+
+NASELORN_FRAME = dict(family="naselorn", post_norms=False, depth_average=False, norm_offset=1.0, embed_norm=False, position_base=10000.0,
+                      tie_word_embeddings=False)
+ARCHITECTURES = {"Nikelix": _read_nikelix, "Naselorn": _read_naselorn}
+
+
+def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
+    qk, v = s.heads * s.dim, s.heads * s.vdim
+    if s.parts:
+        return {f"{n}.{k}": t for n, p in zip(PART_NAMES, s.parts) for k, t in _mixer_shapes(p, d).items()}
+    if s.type == "latent_attention":
+        return {"q": (s.heads * (s.dim + s.rot_dim), d), "dkv": (s.kv_rank + s.rot_dim, d), "dkv.norm": (s.kv_rank,),
+                "uk": (qk, s.kv_rank), "uv": (v, s.kv_rank), "o": (d, v)}
+    if s.type == "hgrn2":
+        return {"q": (qk, d), "f": (qk, d), "f.b": (qk,), "lower": (qk,), "v": (v, d), "norm": (s.vdim,), "o": (d, v)}
+    if s.type == "lightning":
+        return {"q": (qk, d), "k": (qk, d), "v": (v, d), "g": (v, d), "o": (d, v), "norm": (v,)}
+    if s.type == "attention":
+        out = {"q": (qk, d), "k": (s.kv_heads * s.dim, d), "v": (s.kv_heads * s.vdim, d), "o": (d, v)}
+        return {**out, **{k + ".b": (t[0],) for k, t in out.items()}} if s.biases else out
+    if s.type == "rglru":
+        gates = {k: t for g in ("ra", "ri") for k, t in ((g, (s.heads, s.dim, s.dim)), (g + ".b", (s.heads, s.dim)))}
+        return {"y": (qk, d), "y.b": (qk,), "x": (qk, d), "x.b": (qk,), "conv": (qk, s.conv), "conv.b": (qk,), **gates, "lam": (qk,), "o": (d, qk)}
+    out = {"mu." + m: (d,) for m in SHIFT_MIXES}
+    out.update({m: (qk, d) for m in "rkvg"})
+    out.update({"w1": (s.decay_rank, d), "w2": (qk, s.decay_rank), "w0": (qk,), "u": (s.heads, s.dim), "norm": (qk,), "o": (d, qk)})
+    return out
+
+
+def _mlp_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
+    def glu(pre: str, ff: int) -> dict[str, tuple[int, ...]]:
+        return {pre + "gate": (ff, d), pre + "up": (ff, d), pre + "down": (d, ff)}
+
+    if s.mlp == "poly":
+        return {"up": (s.ff, d), "down": (d, s.ff), "act": (4,)}
+    if s.mlp == "gated":
+        return glu("", s.ff)
+    out = {k: t for e in range(s.experts) for k, t in glu(f"e{e}.", s.expert_ff).items()}
+    out.update({"router": (s.experts, d), "router.b": (s.experts,)})
+    return {**out, **(glu("shared.", s.shared_ff) if s.shared_ff else {})}
 
 
 def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
     """Name -> shape of every tensor of a checkpoint.  The decay rank of a wkv layer is taken from its spec."""
     d = cfg.hidden_size
-    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, d), "embed.norm": (d,), "final.norm": (d,)}
+    out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, d), "final.norm": (d,)}
+    if cfg.embed_norm:
+        out["embed.norm"] = (d,)
+    if not cfg.tie_word_embeddings:
+        out["head"] = (cfg.vocab_size, d)
     for i, s in enumerate(cfg.layers):
         p = f"l{i}."
-        out[p + "norm1"] = out[p + "norm1b"] = (d,)
-        x = p + "mix."
-        qk, v = s.heads * s.dim, s.heads * s.vdim
-        if s.type == "latent_attention":
-            out[x + "q"] = (s.heads * (s.dim + s.rot_dim), d)
-            out[x + "dkv"] = (s.kv_rank + s.rot_dim, d)
-            out[x + "dkv.norm"] = (s.kv_rank,)
-            out[x + "uk"], out[x + "uv"] = (qk, s.kv_rank), (v, s.kv_rank)
-            out[x + "o"] = (d, v)
-        elif s.type == "hgrn2":
-            out[x + "q"] = out[x + "f"] = (qk, d)
-            out[x + "f.b"] = out[x + "lower"] = (qk,)
-            out[x + "v"], out[x + "norm"], out[x + "o"] = (v, d), (s.vdim,), (d, v)
-        else:
-            for m in SHIFT_MIXES:
-                out[x + "mu." + m] = (d,)
-            for m in "rkvg":
-                out[x + m] = (qk, d)
-            out[x + "w1"], out[x + "w2"], out[x + "w0"] = (s.decay_rank, d), (qk, s.decay_rank), (qk,)
-            out[x + "u"], out[x + "norm"], out[x + "o"] = (s.heads, s.dim), (qk,), (d, qk)
-        if s.ff:
-            out[p + "norm2"] = out[p + "norm2b"] = (d,)
-            out[p + "mlp.up"], out[p + "mlp.down"], out[p + "mlp.act"] = (s.ff, d), (d, s.ff), (4,)
-        out[p + "dwa"] = (i + 2,)
+        norms = ["norm1"] + (["norm1b"] if cfg.post_norms else [])
+        if s.has_mlp:
+            norms += ["norm2"] + (["norm2b"] if cfg.post_norms else [])
+            out.update({p + "mlp." + k: t for k, t in _mlp_shapes(s, d).items()})
+        out.update({p + n: (d,) for n in norms})
+        out.update({p + "mix." + k: t for k, t in _mixer_shapes(s, d).items()})
+        if cfg.depth_average:
+            out[p + "dwa"] = (i + 2,)
     return out
 
 
@@ -164,10 +288,11 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
         if s.type == "wkv" and not s.decay_rank:
             s.decay_rank = max(8, cfg.hidden_size // 64 // 8 * 8)
     w: dict[str, torch.Tensor] = {}
+    frame = ("norm1", "norm1b", "norm2", "norm2b", "final.norm", "embed.norm")
     for k, shape in tensor_shapes(cfg).items():
         leaf = k.split(".", 2)[-1] if k.startswith("l") else k
         if "norm" in leaf:
-            w[k] = rnd(*shape, std=0.1, mean=1.0)
+            w[k] = rnd(*shape, std=0.1, mean=1.0 - (cfg.norm_offset if leaf in frame or k.split(".")[-1] in frame else 0.0))
         elif k.endswith(".dwa"):
             t = torch.full(shape, 0.3 / max(1, shape[0] - 1), device=device)
             t[-1] = 0.8
@@ -180,7 +305,9 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
             w[k] = uni(*shape, lo=-6.0, hi=0.0)
         elif leaf.startswith("mu."):
             w[k] = uni(*shape)
-        elif leaf in ("u", "f.b"):
+        elif leaf.endswith("lam"):             # memories from a token to some thousand tokens
+            w[k] = uni(*shape, lo=-8.0, hi=1.0)
+        elif leaf in ("u", "f.b") or leaf.endswith(".b"):
             w[k] = rnd(*shape, std=0.5)
         else:
             w[k] = rnd(*shape, std=shape[-1] ** -0.5)
@@ -193,11 +320,24 @@ def _preset(name: str, width: int, ff: int, heads: int, n_layers: int, vocab: in
     la = LayerSpec("latent_attention", heads, 128, 128, ff, rot_dim=64, kv_rank=512, scale=192 ** -0.5, rope_base=5e5, window=window)
     hg = LayerSpec("hgrn2", heads, hd, hd, ff)
     wk = LayerSpec("wkv", width // 64, 64, 64, ff, decay_rank=64)
-    import dataclasses
-
     cycle = (la, hg, wk, hg)
     return HybridConfig(name=name, vocab_size=vocab, hidden_size=width,
                         layers=[dataclasses.replace(cycle[i % 4]) for i in range(n_layers)], residual_mult=0.5)
+
+
+def _naselorn_preset(name: str, width: int, n_layers: int, experts: int, top: int, expert_ff: int, shared_ff: int, dense_ff: int,
+                     vocab: int = 32000, chunk: int = 1024) -> HybridConfig:
+    """``n_layers`` layers, every fourth one parallel, the others lightning; the first has a dense feed-forward."""
+    hd = 128
+    decay = tuple(1 - 2.0 ** (-1 - 7.0 * h / max(1, width // hd - 1)) for h in range(width // hd))
+    li = LayerSpec("lightning", width // hd, hd, hd, decay=decay)
+    parts = (LayerSpec("attention", width // hd, hd, hd, kv_heads=max(1, width // hd // 4), scale=hd ** -0.5, chunk=chunk, biases=True),
+             LayerSpec("rglru", width // 256, 256, 256, conv=4))
+    pa = LayerSpec("parallel", 0, 0, 0, parts=parts, part_scales=(0.5, 0.5))
+    layers = [dataclasses.replace(pa if i % 4 == 3 else li, mlp="moe", experts=experts, top=top, expert_ff=expert_ff, shared_ff=shared_ff)
+              for i in range(n_layers)]
+    layers[0] = dataclasses.replace(li, mlp="gated", act="relu", ff=dense_ff)
+    return HybridConfig(name=name, vocab_size=vocab, hidden_size=width, layers=layers, embed_scale=width ** 0.5, **NASELORN_FRAME)
 
 
 HYBRID_PRESETS: dict[str, HybridConfig] = {
@@ -207,4 +347,11 @@ HYBRID_PRESETS: dict[str, HybridConfig] = {
         LayerSpec("wkv", 4, 16, 16, 0, decay_rank=8)], residual_mult=0.7),
     "nikelix-1b": _preset("nikelix-1b", 2048, 8192, 16, 16),
     "nikelix-7b": _preset("nikelix-7b", 4096, 16384, 32, 32),
+    "naselorn-tiny": HybridConfig("naselorn-tiny", 512, 128, [
+        LayerSpec("lightning", 2, 24, 40, 176, decay=(0.7, 0.97), mlp="gated", act="relu"),
+        LayerSpec("parallel", 0, 0, 0, mlp="moe", experts=6, top=2, expert_ff=48, shared_ff=80, part_scales=(0.7, 0.4), parts=(
+            LayerSpec("attention", 4, 16, 24, kv_heads=2, scale=0.25, chunk=20, biases=True), LayerSpec("rglru", 3, 20, 20, conv=3)))],
+        embed_scale=8.0, **NASELORN_FRAME),
+    "naselorn-2b-a1b": _naselorn_preset("naselorn-2b-a1b", 2048, 16, 64, 8, 512, 1024, 6144),
+    "naselorn-14b-a4b": _naselorn_preset("naselorn-14b-a4b", 4096, 16, 64, 8, 1024, 2048, 12288),
 }

@@ -13,7 +13,7 @@ import torch
 
 from . import _lib
 
-EPI_BF16, EPI_BF16_RESID, EPI_F32, EPI_SWIGLU, EPI_SWIGLU_BWD = 0, 1, 2, 3, 4
+EPI_BF16, EPI_BF16_RESID, EPI_F32, EPI_SWIGLU, EPI_SWIGLU_BWD, EPI_RELUGLU = 0, 1, 2, 3, 4, 5
 _configured = False
 _configured2 = False
 TWO_CTA_DEFAULT = os.environ.get("ARTB_GEMM_2CTA", "1") == "1"
@@ -52,12 +52,14 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
             residual: torch.Tensor | None = None, swiglu_out: torch.Tensor | None = None,
             bias: torch.Tensor | None = None, res_cols: int = 0,
             out_dtype: torch.dtype = torch.bfloat16, bn: int = 0, max_ctas: int = 0,
-            two_cta: bool | None = None, swiglu_bwd_gu: torch.Tensor | None = None) -> torch.Tensor:
+            two_cta: bool | None = None, swiglu_bwd_gu: torch.Tensor | None = None, gate_act: str = "silu",
+            keep_preact: bool = True) -> torch.Tensor | None:
     """``out[M,N] = a[M,K] @ b[N,K].T (+ a2[M,K2] @ b2[N,K2].T) (+ residual)``.
 
     ``swiglu_out`` ([M, N/2] bf16) selects the SwiGLU epilogue: ``b``'s rows must be
     interleaved in blocks of 16 (gate rows, then the matching up rows); ``out`` receives
-    the pre-activation and ``swiglu_out`` receives ``silu(gate) * up``.
+    the pre-activation and ``swiglu_out`` receives ``silu(gate) * up`` (``gate_act="relu"``: ``relu(gate) * up``);
+    with ``keep_preact=False`` only ``swiglu_out`` is written and nothing is returned.
 
     ``swiglu_bwd_gu`` ([M, 2N] bf16, the forward's interleaved gate|up pre-activations) selects the fused
     SwiGLU-backward epilogue: the product is taken as ``d(silu(gate) * up)`` and ``out`` ([M, 2N]) receives
@@ -85,16 +87,17 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
         epi = EPI_SWIGLU_BWD
         swiglu_out = swiglu_bwd_gu          # travels in the H slot of the C entry point
     elif swiglu_out is not None:
-        epi = EPI_SWIGLU
+        epi = EPI_RELUGLU if gate_act == "relu" else EPI_SWIGLU
     elif residual is not None:
         epi = EPI_BF16_RESID
     elif out_dtype == torch.float32:
         epi = EPI_F32
     else:
         epi = EPI_BF16
-    if out is None:
+    drop = epi in (EPI_SWIGLU, EPI_RELUGLU) and not keep_preact
+    if out is None and not drop:
         out = torch.empty((M, N), dtype=torch.float32 if epi == EPI_F32 else torch.bfloat16, device=a.device)
-    if out.stride(1) != 1 or tuple(out.shape) != (M, 2 * N if epi == EPI_SWIGLU_BWD else N):
+    if out is not None and (out.stride(1) != 1 or tuple(out.shape) != (M, 2 * N if epi == EPI_SWIGLU_BWD else N)):
         raise ValueError("out must be [M,N] with unit inner stride")
     if residual is not None:
         _check2d(residual, "residual")
@@ -108,7 +111,7 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
             _lib.ptr(a), a.stride(0), _lib.ptr(b), b.stride(0),
             _lib.ptr(a2), a2.stride(0) if a2 is not None else 0,
             _lib.ptr(b2), b2.stride(0) if b2 is not None else 0, K2,
-            _lib.ptr(out), out.stride(0),
+            _lib.ptr(out), out.stride(0) if out is not None else 0,
             _lib.ptr(residual), residual.stride(0) if residual is not None else 0,
             _lib.ptr(swiglu_out), swiglu_out.stride(0) if swiglu_out is not None else 0,
             _lib.ptr(bias),
@@ -120,7 +123,7 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
         _lib.ptr(a), a.stride(0), _lib.ptr(b), b.stride(0),
         _lib.ptr(a2), a2.stride(0) if a2 is not None else 0,
         _lib.ptr(b2), b2.stride(0) if b2 is not None else 0, K2,
-        _lib.ptr(out), out.stride(0),
+        _lib.ptr(out), out.stride(0) if out is not None else 0,
         _lib.ptr(residual), residual.stride(0) if residual is not None else 0,
         _lib.ptr(swiglu_out), swiglu_out.stride(0) if swiglu_out is not None else 0,
         _lib.ptr(bias),

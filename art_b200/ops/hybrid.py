@@ -1,5 +1,5 @@
-"""Front-ends of the hybrid decoder's kernels (``csrc/kernels/hybrid_rows.cu``, ``linear_scan.cu``, ``latent_attn*.cu``,
-``gemm_batched.cu``, ``gemm_f32.cu``).
+"""Front-ends of the hybrid decoder's kernels (``csrc/kernels/hybrid_rows.cu``, ``linear_scan.cu``, ``latent_*.cu``,
+``gqa_attn.cu``, ``rglru.cu``, ``gemm_batched.cu``, ``gemm_f32.cu``).
 
 GEMM operands are bf16, or fp32 in the 32-bit mode; the residual stream, norms, gates and states are fp32 in both.  A
 projection's output reaches its consumer as bf16, as fp32, or as the fp32 workspace of a split-K GEMM that the consumer
@@ -15,14 +15,17 @@ import torch
 from . import _lib
 
 vp, ci, cl, cf = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
-SCAN_HGRN2, SCAN_WKV = 0, 1
+SCAN_HGRN2, SCAN_WKV, SCAN_FIXED = 0, 1, 2
+GATE_SILU, GATE_SIGMOID = 0, 1
+ACTS = {"silu": 0, "relu": 1}
 KIND_BF16, KIND_F32, KIND_TAKE = 0, 1, 2
 _sigs = {
-    "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, cl, ci, vp, vp, vp, ci, ci, ci, ci, cf, vp, vp],
+    "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, vp, ci, ci, vp, vp, cl, vp, vp, vp, cl, ci, vp, vp, vp, ci, ci, ci, ci, cf, vp, vp],
     "artb_norm_shift_mix": [ci, vp, ci, vp, vp, ci, vp, cl, ci, vp, cl, vp, vp, vp, vp, ci, ci, ci, cf, vp, vp],
     "artb_poly_norm": [ci, vp, ci, ci, vp, vp, ci, ci, ci, ci, cf, vp],
     "artb_split_tanh": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
-    "artb_head_norm": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, cf, vp],
+    "artb_gated_act": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
+    "artb_head_norm": [ci, vp, ci, vp, ci, vp, ci, ci, ci, vp, ci, ci, ci, ci, ci, cf, vp],
     "artb_gather_norm": [ci, vp, ci, vp, ci, vp, vp, ci, ci, ci, cf, cl, vp, vp],
     "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
     "artb_linear_decode": [ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci,
@@ -32,9 +35,15 @@ _sigs = {
     "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
     "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, ci, vp, vp],
     "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, vp, ci, vp, vp],
-    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, ci, ci,
-                               vp, vp],
-    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, ci, ci, ci, vp],
+    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci,
+                               ci, ci, vp, vp],
+    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp],
+    "artb_gqa_finish": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, ci, vp, vp, ci, ci, vp, vp],
+    "artb_gqa_decode": [vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_attend": [ci, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_short_conv": [ci, vp, ci, ci, vp, vp, vp, ci, vp, cl, vp, vp, vp, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_rglru": [ci, ci, vp, ci, ci, vp, ci, vp, vp, vp, vp, ci, ci, vp, vp, cl, vp, vp, vp, ci, vp, ci, cf, ci, ci, ci, ci, vp, vp],
     "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
     "artb_gemm_f32_tn": [vp, ci, cl, vp, ci, cl, vp, ci, cl, ci, ci, ci, ci, vp],
 }
@@ -76,17 +85,37 @@ def _st(t: torch.Tensor):
     return _lib.ptr(_lib.status_word(t.device))
 
 
-def residual_step(x_out: torch.Tensor, w_post: torch.Tensor, d: int, eps: float, *, y: Out | None = None, x_in=None,
-                  mult: float = 1.0, tokens=None, table=None, hist=None, hist_n: int = 0, avg=None, w_next=None, h=None) -> None:
-    """One sublayer boundary of the fp32 residual stream ``[M, dp]``; ``y`` is the sublayer's output, or ``tokens`` /
-    ``table`` the embedding.  ``hist`` fp32 ``[layers + 1, M, dp]``: the result is stored at ``hist_n`` and, with ``avg``,
+@dataclass
+class Sublayer:
+    """What a sublayer hands to the residual stream: ``y`` (may be missing), ``bias`` [dp] and the rows of a token's experts,
+    ``rows`` [cap, dp] weighted by ``weight`` [M, k] at the places ``pos`` [M, k]."""
+    y: Out | None = None
+    bias: torch.Tensor | None = None
+    rows: torch.Tensor | None = None
+    pos: torch.Tensor | None = None
+    weight: torch.Tensor | None = None
+
+
+def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps: float, *, y: Out | None = None, x_in=None,
+                  mult: float = 1.0, tokens=None, table=None, sub: Sublayer | None = None, freq=None, pos=None, hist=None,
+                  hist_n: int = 0, avg=None, w_next=None, h=None) -> None:
+    """One sublayer boundary of the fp32 residual stream ``[M, dp]``; ``y`` (or ``sub``) is the sublayer's output, or
+    ``tokens`` / ``table`` the embedding, to which ``freq`` (fp64 ``[dp / 2]``) and ``pos`` add a sinusoidal position vector.
+    ``w_post``: norm weight of the output; None: it is taken as it is, times ``mult``.  ``hist`` fp32 ``[layers + 1, M, dp]``: the result is stored at ``hist_n`` and, with ``avg``,
     replaced by the weighted average of entries ``0 .. hist_n``.  ``w_next`` / ``h``: the next sublayer's input norm."""
     M, dp = x_out.shape
-    f32 = _is32(table if table is not None else h) if (table is not None or h is not None) else 0
+    s = sub if sub is not None else Sublayer(y)
+    y, ex = s.y, s.rows
+    op = next((t for t in (table, h, ex) if t is not None), None)      # any tensor of the operand dtype
+    f32 = _is32(op) if op is not None else 0
+    if freq is not None and freq.dtype != torch.float64:
+        raise ValueError("position frequencies are fp64")
     _lib.check_rc(_f("artb_residual_step")(
         f32, _lib.ptr(tokens), _lib.ptr(table), table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0,
         _lib.ptr(y.t if y is not None else None), y.t.stride(0) if y is not None else 0, y.kind if y is not None else 0,
-        _lib.ptr(x_in), _lib.ptr(x_out), x_out.stride(0), _lib.ptr(w_post), mult, _lib.ptr(hist),
+        _lib.ptr(x_in), _lib.ptr(x_out), x_out.stride(0), _lib.ptr(w_post), mult, _lib.ptr(s.bias), _lib.ptr(ex),
+        ex.stride(0) if ex is not None else 0, s.pos.shape[1] if ex is not None else 0, _lib.ptr(s.pos), _lib.ptr(s.weight),
+        ex.shape[0] if ex is not None else 0, _lib.ptr(freq), _lib.ptr(pos), _lib.ptr(hist),
         hist.stride(0) if hist is not None else 0, hist_n, _lib.ptr(avg), _lib.ptr(w_next), _lib.ptr(h),
         h.stride(0) if h is not None else 0, M, d, dp, eps, _st(x_out), _lib.stream_ptr()), "residual_step")
 
@@ -114,12 +143,21 @@ def split_tanh(z: Out, r: int, rp: int, out) -> torch.Tensor:
     return out
 
 
-def head_norm(o, w, w_per_head: bool, H: int, vdim: int, vpad: int, out, eps: float, gate: Out | None = None) -> torch.Tensor:
-    """Per-head RMSNorm of ``o`` fp32 [M, H * vdim]; ``w`` [vdim], or [H * vdim] with ``w_per_head``; silu ``gate``."""
+def gated_act(z: Out, out, act: str) -> torch.Tensor:
+    """``act(gate) * up`` of a gate|up projection whose columns are interleaved in blocks of 16."""
+    _lib.check_rc(_f("artb_gated_act")(_is32(out), _lib.ptr(z.t), z.t.stride(0), z.kind, _lib.ptr(out), out.stride(0), out.shape[0],
+                                       out.shape[1], ACTS[act], _lib.stream_ptr()), "gated_act")
+    return out
+
+
+def head_norm(o, w, w_per_head: bool, H: int, vdim: int, vpad: int, out, eps: float, gate: Out | None = None,
+              gate_act: int = GATE_SILU) -> torch.Tensor:
+    """Per-head RMSNorm of ``o`` fp32 [M, H * vdim]; ``w`` [vdim], or [H * vdim] with ``w_per_head``; silu or sigmoid ``gate``.
+    H = 1: one norm over the whole row."""
     _lib.check_rc(_f("artb_head_norm")(
         _is32(out), _lib.ptr(o), o.stride(0), _lib.ptr(w), 1 if w_per_head else 0,
-        _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0, _lib.ptr(out), out.stride(0),
-        out.shape[0], H, vdim, vpad, eps, _lib.stream_ptr()), "head_norm")
+        _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0, gate_act, _lib.ptr(out),
+        out.stride(0), out.shape[0], H, vdim, vpad, eps, _lib.stream_ptr()), "head_norm")
     return out
 
 
@@ -129,14 +167,14 @@ def gather_norm(x, rows, w, h, d: int, eps: float) -> torch.Tensor:
     return h
 
 
-def _scan_in(mode, q: Out, k: Out | None, v: Out, g: Out):
+def _scan_in(mode, q: Out, k: Out | None, v: Out, g: Out | None):
     if q.kind != v.kind or (k is not None and k.kind != q.kind):
         raise ValueError("q, k and v come from one projection and share their kind")
     return (_lib.ptr(q.t), q.t.stride(0), _lib.ptr(k.t if k else None), k.t.stride(0) if k else 0, _lib.ptr(v.t), v.t.stride(0), q.kind,
-            _lib.ptr(g.t), g.t.stride(0), g.kind)
+            _lib.ptr(g.t if g else None), g.t.stride(0) if g else 0, g.kind if g else KIND_F32)
 
 
-def linear_scan(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, state, cu_q, ctx, state_slot, n_seqs: int, H: int,
+def linear_scan(mode: int, q: Out, k: Out | None, v: Out, g: Out | None, bias, aux, state, cu_q, ctx, state_slot, n_seqs: int, H: int,
                 dim: int, vdim: int, o) -> torch.Tensor:
     """Portions of ``n_seqs`` sequences through the recurrence; ``state`` fp32 ``[slots, H, vdim, ld]``; ``o`` fp32."""
     _lib.check_rc(_f("artb_linear_scan")(
@@ -147,12 +185,13 @@ def linear_scan(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, sta
     return o
 
 
-def linear_decode(mode: int, q: Out, k: Out | None, v: Out, g: Out, bias, aux, state, cu_q, ctx, state_slot, H: int, dim: int,
+def linear_decode(mode: int, q: Out, k: Out | None, v: Out, g: Out | None, bias, aux, state, cu_q, ctx, state_slot, H: int, dim: int,
                   vdim: int, w, w_per_head: bool, gate: Out | None, out, vpad: int, eps: float) -> torch.Tensor:
-    """One token of each sequence (row m = sequence m): recurrence, per-head norm, optional gate."""
+    """One token of each sequence (row m = sequence m): recurrence, per-head norm, optional gate.  ``w`` None: the fp32 outputs
+    of the recurrence."""
     M = out.shape[0]
     _lib.check_rc(_f("artb_linear_decode")(
-        _is32(out), mode, *_scan_in(mode, q, k, v, g), _lib.ptr(bias), _lib.ptr(aux), _lib.ptr(state), state.stride(0),
+        _is32(out) if w is not None else 0, mode, *_scan_in(mode, q, k, v, g), _lib.ptr(bias), _lib.ptr(aux), _lib.ptr(state), state.stride(0),
         state.shape[3], state.shape[0], _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), M, H, dim, vdim, _lib.ptr(w),
         1 if w_per_head else 0, _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0,
         _lib.ptr(out), out.stride(0), vpad, eps, _st(out), _lib.stream_ptr()), "linear_decode")
@@ -221,13 +260,19 @@ class PrefillPlan:
     tile_row: torch.Tensor
 
 
-def plan_prefill(portions: list[tuple[int, int, int]], window: int, device) -> PrefillPlan:
+def first_key(p: int, window: int, chunk: int = 0) -> int:
+    """First key position ``p`` sees: of the last ``window`` ones and of its own ``chunk`` (0: no limit)."""
+    lo = max(0, p - window + 1) if window > 0 else 0
+    return max(lo, p - p % chunk) if chunk > 0 else lo
+
+
+def plan_prefill(portions: list[tuple[int, int, int]], window: int, device, chunk: int = 0) -> PrefillPlan:
     """``portions``: ``(sequence, tokens before the portion, tokens of the portion)`` in row order.  Every sequence's
     gathered keys start at a multiple of 8 rows."""
     seq_of, key_off, key_pos0, key_cnt, row_end, row_pos0, tile_seq, tile_row = [], [], [], [], [], [], [], []
     row = keys = 0
     for i, (seq, n0, n) in enumerate(portions):
-        first = max(0, n0 - window + 1) if window > 0 else 0
+        first = first_key(n0, window, chunk)
         seq_of.append(seq)
         key_off.append(keys)
         key_pos0.append(first)
@@ -254,14 +299,14 @@ def latent_gather(cache, block_table, plan: PrefillPlan) -> torch.Tensor:
 
 
 def latent_prefill(q, kv, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                   vdim: int) -> torch.Tensor:
-    """Windowed attention of the portions: ``q`` [rows, H * (dk + rot_p)], ``kv`` [n_keys, H * dk + H * dv] the expanded
-    keys and values, ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)]."""
+                   vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0) -> torch.Tensor:
+    """Masked attention of the portions: ``q`` [rows, H * (dk + rot_p)], ``kv`` [n_keys, H / G * (dk + dv)] the expanded
+    keys and values (``G`` heads share them), ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)]."""
     _lib.check_rc(_f("artb_latent_prefill")(
         _lib.ptr(q), q.stride(0), _lib.ptr(kv), kv.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(plan.tile_seq),
         _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0), _lib.ptr(plan.key_off),
-        _lib.ptr(plan.key_pos0), window, scale, _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, dk, dv, rot_p, _lib.stream_ptr()),
-        "latent_prefill")
+        _lib.ptr(plan.key_pos0), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p,
+        _lib.stream_ptr()), "latent_prefill")
     return o
 
 
@@ -272,15 +317,98 @@ def prefill_tc_values(dim: int, rot: int, vdim: int, scale: float) -> int:
     return 64 if vdim <= 64 else 128
 
 
+def gqa_value_columns(dim: int, vdim: int, scale: float) -> int:
+    """Columns of a value head in the cache of grouped-query attention: what the prefill kernel that suits the sizes reads."""
+    return prefill_tc_values(dim, 0, vdim, scale) or pad(vdim, 16)
+
+
 def latent_prefill_tc(q, k, vt, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                      vdim: int) -> torch.Tensor:
-    """:func:`latent_prefill` on tcgen05: ``k`` [n_keys, H * dk], values transposed ``vt`` [H * dv, n_keys]."""
+                      vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0) -> torch.Tensor:
+    """:func:`latent_prefill` on tcgen05: ``k`` [n_keys, H / G * dk], values transposed ``vt`` [H / G * dv, n_keys]."""
     _lib.check_rc(_f("artb_latent_prefill_tc")(
         _lib.ptr(q), q.stride(0), q.shape[0], _lib.ptr(k), k.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(vt), vt.stride(0),
         plan.n_keys, _lib.ptr(plan.tile_seq), _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0),
-        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, scale, _lib.ptr(o), o.stride(0), pad(vdim), H, dk, dv, rot_p, _st(o),
+        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0), pad(vdim), H, G, dk, dv, rot_p, _st(o),
         _lib.stream_ptr()), "latent_prefill_tc")
     return o
+
+
+def gqa_finish(p: Out, bias, slot, cache, q, H: int, Hkv: int, dim: int, vdim: int, dvp: int) -> None:
+    """Biases, cache write and padded queries behind a q | k | v projection; cache rows hold ``Hkv`` keys of pad(dim, 16), then
+    ``Hkv`` values of ``dvp`` columns."""
+    M = slot.numel()
+    _lib.check_rc(_f("artb_gqa_finish")(
+        _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(bias), _lib.ptr(slot), _lib.ptr(cache), cache.shape[-1],
+        cache.shape[0] * cache.shape[1], _lib.ptr(q), q.stride(0), M, H, Hkv, dim, pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()),
+        "gqa_finish")
+
+
+def gqa_gather(cache, block_table, plan: PrefillPlan, Hkv: int, dk: int, dv: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Keys ``[n_keys, Hkv * dk]`` and transposed values ``[Hkv * dv, n_keys]`` of the cache rows the portions see."""
+    k = torch.empty((plan.n_keys, Hkv * dk), dtype=cache.dtype, device=cache.device)
+    vt = torch.empty((Hkv * dv, plan.n_keys), dtype=cache.dtype, device=cache.device)
+    _lib.check_rc(_f("artb_gqa_gather")(
+        _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1], cache.shape[0],
+        _lib.ptr(plan.seq_of), _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), _lib.ptr(plan.key_cnt), plan.n_seqs, plan.n_keys, _lib.ptr(k),
+        _lib.ptr(vt), Hkv * dk, Hkv * dv, _st(cache), _lib.stream_ptr()), "gqa_gather")
+    return k, vt
+
+
+GQA_TILE = 32           # keys per warp tile of the decode kernel, four warps a CTA
+GQA_DECODE_MAX = 256    # head sizes its tiles hold; beyond them the scalar kernel serves
+
+
+def gqa_decode_splits(M: int, ctas_per_row: int, keys: int, sms: int = 148) -> int:
+    """How many CTAs share a row's keys: enough to cover the machine, one tile per warp each at least."""
+    return max(1, min(2 * sms // max(1, M * ctas_per_row), (keys + 4 * GQA_TILE - 1) // (4 * GQA_TILE), 32))
+
+
+def _gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o):
+    return (_lib.ptr(q), q.stride(0), _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1],
+            cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0))
+
+
+def gqa_decode(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
+               Hkv: int, dim: int, vdim: int, dvp: int, splits: int = 1) -> torch.Tensor:
+    """Rows ``0 .. M - 1`` of ``q`` against their sequences' cached keys; ``o`` [., H * pad(vdim)] gets ``out_scale`` times the
+    result."""
+    vpad = pad(vdim)
+    ws = torch.empty(M * H * splits * (vpad + 2), dtype=torch.float32, device=o.device) if splits > 1 else None
+    _lib.check_rc(_f("artb_gqa_decode")(
+        *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o), vpad, _lib.ptr(ws), splits, M, H, Hkv,
+        pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_decode")
+    return o
+
+
+def gqa_attend(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
+               Hkv: int, dim: int, vdim: int, dvp: int) -> torch.Tensor:
+    """Scalar fp32 form of :func:`gqa_decode`, any head sizes."""
+    _lib.check_rc(_f("artb_gqa_attend")(
+        _is32(cache), *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o), pad(vdim), M, H, Hkv,
+        pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_attend")
+    return o
+
+
+def short_conv(x: Out, x_bias, w, bias, state, row_seq, cu_q, ctx, state_slot, n_seqs: int, single: bool, u, bs: int, bp: int) -> None:
+    """Causal convolution ``w`` [n, taps] of ``x + x_bias``; ``u`` [blocks, pitch, .] receives a bf16 pair (or fp32) per
+    channel, ``state`` fp32 [slots, taps - 1, n] the last inputs."""
+    n, taps = w.shape
+    _lib.check_rc(_f("artb_short_conv")(
+        _is32(u), _lib.ptr(x.t), x.t.stride(0), x.kind, _lib.ptr(x_bias), _lib.ptr(w), _lib.ptr(bias), taps, _lib.ptr(state),
+        state.shape[0], _lib.ptr(row_seq), _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, 1 if single else 0, _lib.ptr(u),
+        u.shape[1], u.shape[2], n, bs, bp, x.t.shape[0], _st(u), _lib.stream_ptr()), "short_conv")
+
+
+def rglru(u, z, r_bias, i_bias, decay, y: Out, y_bias, state, cu_q, ctx, state_slot, n_seqs: int, single: bool, o, out_scale: float,
+          bs: int, bp: int) -> None:
+    """Gated recurrence over ``u`` (see :func:`short_conv`) with gate products ``z`` fp32 [M, blocks * 2 bp]; ``o`` [M, n] gets
+    ``out_scale * S * gelu(y + y_bias)``."""
+    n = decay.numel()
+    _lib.check_rc(_f("artb_rglru")(
+        _is32(u), 1 if single else 0, _lib.ptr(u), u.shape[1], u.shape[2], _lib.ptr(z), z.stride(0), _lib.ptr(r_bias), _lib.ptr(i_bias),
+        _lib.ptr(decay), _lib.ptr(y.t), y.t.stride(0), y.kind, _lib.ptr(y_bias), _lib.ptr(state), state.shape[0], _lib.ptr(cu_q),
+        _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, _lib.ptr(o), o.stride(0), out_scale, n, bs, bp, z.shape[0], _st(u), _lib.stream_ptr()),
+        "rglru")
 
 
 def gemm_batched(a, b, out, M: int, *, c_batch: int) -> torch.Tensor:

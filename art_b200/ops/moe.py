@@ -26,15 +26,17 @@ def _k():
     lib = _lib.kernels()
     if not _configured:
         vp, ci, cl = ctypes.c_void_p, ctypes.c_int, ctypes.c_long
-        lib.artb_moe_router.argtypes = [vp, ci, ci, ci, ci, ci, vp, vp, vp, vp]
+        lib.artb_moe_router.argtypes = [vp, ci, ci, vp, ci, ci, ci, ci, vp, vp, vp, vp]
         lib.artb_moe_plan.argtypes = [vp, ci, vp, vp, cl, ci, vp, vp, ci, vp, vp, vp, vp, vp]
         lib.artb_moe_gather.argtypes = [vp, ci, vp, vp, ci, vp, vp, ci, ci, ci, vp]
+        lib.artb_moe_gather_f32.argtypes = [vp, ci, vp, vp, vp, ci, ci, ci, vp]
+        lib.artb_gemm_f32_grouped_tn.argtypes = [vp, ci, vp, ci, vp, ci, vp, ci, ci, ci, vp]
         lib.artb_moe_combine.argtypes = [vp, ci, vp, vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, vp, vp]
         lib.artb_moe_router_bwd.argtypes = [vp, ci, vp, vp, vp, ci, ci, ci, ci, vp, ci, vp]
         lib.artb_gemm_grouped_bf16_tn.argtypes = [vp, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, vp, ci, vp, ci, ci, ci,
                                                   ci, ci, vp, vp]
         lib.artb_lora_wgrad_grouped.argtypes = [vp, ci, vp, ci, vp, ci, cl, vp, ci, ci, ci, ci, vp]
-        for f in (lib.artb_moe_router, lib.artb_moe_plan, lib.artb_moe_gather, lib.artb_moe_combine,
+        for f in (lib.artb_moe_router, lib.artb_moe_plan, lib.artb_moe_gather, lib.artb_moe_gather_f32, lib.artb_gemm_f32_grouped_tn, lib.artb_moe_combine,
                   lib.artb_moe_router_bwd, lib.artb_gemm_grouped_bf16_tn, lib.artb_lora_wgrad_grouped):
             f.restype = ci
         _configured = True
@@ -70,8 +72,9 @@ def cap_tiles_for(M: int, k: int, E: int) -> int:
     return (M * k + E * 127 + 127) // 128
 
 
-def route(logits: torch.Tensor, k: int, norm_topk: bool) -> RoutePlan:
-    """Softmax over experts, top-k, (optional) renormalisation, and the expert-sorted row plan."""
+def route(logits: torch.Tensor, k: int, norm_topk: bool, bias: torch.Tensor | None = None, take: bool = False) -> RoutePlan:
+    """Softmax over experts, top-k, (optional) renormalisation, and the expert-sorted row plan.  ``bias`` fp32 [E] is added
+    to the logits first; with ``take`` the logits lie in a workspace that is to be left zero."""
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     M, E = logits.shape
     dev = logits.device
@@ -83,7 +86,7 @@ def route(logits: torch.Tensor, k: int, norm_topk: bool) -> RoutePlan:
                      torch.empty(cap * 128, dtype=torch.float32, device=dev))
     cursor = torch.empty(E, **i32)
     st = _lib.stream_ptr()
-    _lib.check_rc(_k().artb_moe_router(_lib.ptr(logits), logits.stride(0), M, E, k, int(norm_topk), _lib.ptr(plan.topi),
+    _lib.check_rc(_k().artb_moe_router(_lib.ptr(logits), logits.stride(0), 2 if take else 1, _lib.ptr(bias), M, E, k, int(norm_topk), _lib.ptr(plan.topi),
                                        _lib.ptr(plan.topw), _lib.ptr(plan.counts), st), "moe_router")
     _lib.check_rc(_k().artb_moe_plan(_lib.ptr(plan.counts), E, _lib.ptr(plan.topi), _lib.ptr(plan.topw), M, k,
                                      _lib.ptr(plan.seg_off), _lib.ptr(plan.tile_expert), cap, _lib.ptr(cursor),
@@ -96,7 +99,13 @@ def gather(x: torch.Tensor, plan: RoutePlan, weighted: bool = False, out: torch.
     """``xp[row] = x[token(row)]`` (times the routing weight if ``weighted``); padding rows are zero."""
     D = x.shape[1]
     if out is None:
-        out = torch.empty((plan.cap_rows, D), dtype=torch.bfloat16, device=x.device)
+        out = torch.empty((plan.cap_rows, D), dtype=x.dtype, device=x.device)
+    if x.dtype == torch.float32:
+        if weighted:
+            raise ValueError("fp32 rows are gathered unweighted")
+        _lib.check_rc(_k().artb_moe_gather_f32(_lib.ptr(x), x.stride(0), _lib.ptr(plan.row_token), _lib.ptr(plan.total_rows), _lib.ptr(out),
+                                               out.stride(0), D, plan.cap_rows, _lib.stream_ptr()), "moe_gather_f32")
+        return out
     _lib.check_rc(_k().artb_moe_gather(_lib.ptr(x), x.stride(0), _lib.ptr(plan.row_token), _lib.ptr(plan.row_w),
                                        int(weighted), _lib.ptr(plan.total_rows), _lib.ptr(out), out.stride(0), D,
                                        plan.cap_rows, _lib.stream_ptr()), "moe_gather")
@@ -135,16 +144,26 @@ def router_bwd(logits: torch.Tensor, plan: RoutePlan, dw: torch.Tensor, norm_top
 
 def grouped_gemm(a: torch.Tensor, b: torch.Tensor, plan: RoutePlan, n_per_expert: int, a2: torch.Tensor | None = None,
                  b2: torch.Tensor | None = None, swiglu_out: torch.Tensor | None = None,
-                 out: torch.Tensor | None = None) -> torch.Tensor:
-    """``out[rows of e] = a[rows of e] @ b[e*N:(e+1)*N].T (+ a2[rows] @ b2[e*N:(e+1)*N].T)``."""
+                 out: torch.Tensor | None = None, keep_preact: bool = True) -> torch.Tensor | None:
+    """``out[rows of e] = a[rows of e] @ b[e*N:(e+1)*N].T (+ a2[rows] @ b2[e*N:(e+1)*N].T)``.  ``keep_preact=False`` with
+    ``swiglu_out``: the pre-activation is not stored.  fp32 operands take the 32-bit product."""
     rows, K = a.shape
     assert rows == plan.cap_rows and b.shape == (plan.E * n_per_expert, K)
-    if out is None:
+    if a.dtype == torch.float32:
+        if a2 is not None or swiglu_out is not None:
+            raise ValueError("the 32-bit grouped product has no extra operand and no activation")
+        if out is None:
+            out = torch.empty((rows, n_per_expert), dtype=torch.float32, device=a.device)
+        _lib.check_rc(_k().artb_gemm_f32_grouped_tn(_lib.ptr(a), a.stride(0), _lib.ptr(b), b.stride(0), _lib.ptr(out), out.stride(0),
+                                                    _lib.ptr(plan.tile_expert), plan.cap_tiles, n_per_expert, K, _lib.stream_ptr()),
+                      "gemm_f32_grouped")
+        return out
+    if out is None and (keep_preact or swiglu_out is None):
         out = torch.empty((rows, n_per_expert), dtype=torch.bfloat16, device=a.device)
     K2 = a2.shape[1] if a2 is not None else 0
     rc = _k().artb_gemm_grouped_bf16_tn(
         _lib.ptr(a), a.stride(0), _lib.ptr(b), b.stride(0), _lib.ptr(a2), a2.stride(0) if a2 is not None else 0,
-        _lib.ptr(b2), b2.stride(0) if b2 is not None else 0, K2, _lib.ptr(out), out.stride(0),
+        _lib.ptr(b2), b2.stride(0) if b2 is not None else 0, K2, _lib.ptr(out), out.stride(0) if out is not None else 0,
         _lib.ptr(swiglu_out), swiglu_out.stride(0) if swiglu_out is not None else 0, _lib.ptr(plan.tile_expert),
         plan.cap_tiles, plan.E, n_per_expert, K, EPI_SWIGLU if swiglu_out is not None else EPI_BF16,
         _lib.ptr(_lib.status_word(a.device)), _lib.stream_ptr())
