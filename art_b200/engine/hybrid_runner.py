@@ -485,6 +485,8 @@ class HybridRunner(DeviceRunner):
         if b.single:
             hy.linear_decode(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, s.heads, s.dim, s.vdim, None, False,
                              None, o, s.vdim, 0.0)
+        elif not self.exact32 and hy.lightning_tc(s.dim, s.vdim):
+            hy.lightning_prefill(q.t, k.t, v.t, L["decay"], state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, s.heads, s.dim, s.vdim, o)
         else:
             hy.linear_scan(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, s.heads, s.dim, s.vdim, o)
         hy.head_norm(o, L["o_norm"], False, 1, nv, pad(nv), out, self.cfg.norm_eps, gate, hy.GATE_SIGMOID)

@@ -1,5 +1,5 @@
-"""Front-ends of the hybrid decoder's kernels (``csrc/kernels/hybrid_rows.cu``, ``linear_scan.cu``, ``latent_*.cu``,
-``gqa_attn.cu``, ``rglru.cu``, ``gemm_batched.cu``, ``gemm_f32.cu``).
+"""Front-ends of the hybrid decoder's kernels (``csrc/kernels/hybrid_rows.cu``, ``linear_scan.cu``, ``lightning_prefill.cu``,
+``latent_*.cu``, ``gqa_attn.cu``, ``rglru.cu``, ``gemm_batched.cu``, ``gemm_f32.cu``).
 
 GEMM operands are bf16, or fp32 in the 32-bit mode; the residual stream, norms, gates and states are fp32 in both.  A
 projection's output reaches its consumer as bf16, as fp32, or as the fp32 workspace of a split-K GEMM that the consumer
@@ -30,6 +30,7 @@ _sigs = {
     "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
     "artb_linear_decode": [ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci,
                            vp, ci, ci, vp, ci, ci, cf, vp, vp],
+    "artb_lightning_prefill": [vp, vp, vp, ci, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
     "artb_latent_finish": [ci, vp, ci, ci, vp, vp, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
                            vp],
     "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
@@ -196,6 +197,22 @@ def linear_decode(mode: int, q: Out, k: Out | None, v: Out, g: Out | None, bias,
         1 if w_per_head else 0, _lib.ptr(gate.t if gate else None), gate.t.stride(0) if gate else 0, gate.kind if gate else 0,
         _lib.ptr(out), out.stride(0), vpad, eps, _st(out), _lib.stream_ptr()), "linear_decode")
     return out
+
+
+def lightning_tc(dim: int, vdim: int) -> bool:
+    """Whether the tensor-core form of lightning attention takes these head sizes."""
+    return dim <= 128 and dim % 8 == 0 and vdim % 8 == 0
+
+
+def lightning_prefill(q, k, v, decay, state, cu_q, ctx, state_slot, n_seqs: int, H: int, dim: int, vdim: int, o) -> torch.Tensor:
+    """``linear_scan(SCAN_FIXED, ...)`` in chunks on tensor cores; ``q``, ``k``, ``v`` bf16 columns of one projection."""
+    if not q.stride(0) == k.stride(0) == v.stride(0):
+        raise ValueError("q, k and v come from one projection")
+    _lib.check_rc(_f("artb_lightning_prefill")(
+        _lib.ptr(q), _lib.ptr(k), _lib.ptr(v), q.stride(0), _lib.ptr(decay), _lib.ptr(state), state.stride(0), state.shape[3], state.shape[0],
+        _lib.ptr(cu_q), _lib.ptr(ctx), _lib.ptr(state_slot), n_seqs, H, dim, vdim, _lib.ptr(o), o.stride(0), o.shape[0], _st(o),
+        _lib.stream_ptr()), "lightning_prefill")
+    return o
 
 
 def latent_finish(p: Out, w, inv_freq, pos, slot, cache, n_abs: int, qn, qr, qe, H: int, dim: int, rot: int, rank: int,

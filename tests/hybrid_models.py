@@ -33,3 +33,39 @@ def aligned_design():
 
 def single_layer(layer):
     return design([layer], vocab=97, width=68)
+
+
+# -- Naselorn -------------------------------------------------------------------------------------------------------------
+def dense(ff=72):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts=7, top=2, ff=28, shared=36):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+
+
+def lightning(heads=3, dim=20, vdim=14, decay=None, mlp=None):
+    return {"type": "lightning", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay or [1 - 0.7 * 0.3 ** h for h in range(heads)])}}
+
+
+def parallel(heads=4, kv_heads=2, dim=12, vdim=20, chunk=19, scale=0.3, width=42, blocks=3, conv=3, left=0.8, right=0.55, mlp=None):
+    return {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": chunk}},
+                      "right": {"width": width, "blocks": blocks, "conv": conv}, "left_scale": left, "right_scale": right}}
+
+
+def naselorn(layers, vocab=211, width=84, eps=2e-5, scale=5.0):
+    return {"architecture": "Naselorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": scale}, "layers": layers}
+
+
+def small_naselorn():
+    return naselorn([parallel(mlp=moe()), lightning(mlp=dense(50)), lightning(heads=1, dim=7, vdim=33), parallel(heads=2, kv_heads=2, dim=64, vdim=24,
+                     chunk=32, width=40, blocks=1, conv=5, left=1.3, right=0.2, mlp=dense()), lightning(heads=2, dim=24, vdim=8, mlp=moe(5, 1, 16, 20))])
+
+
+def aligned_naselorn():
+    """Sizes near a real model's proportions, still small: several tiles of the tensor-core kernels."""
+    return naselorn([lightning(heads=3, dim=128, vdim=72, mlp=dense(304)), parallel(heads=6, kv_heads=2, dim=128, vdim=104, chunk=150, scale=0.09,
+                     width=384, blocks=6, conv=4, mlp=moe(12, 4, 96, 144)), lightning(heads=5, dim=48, vdim=80, mlp=moe(9, 2, 80, 64)),
+                     parallel(heads=4, kv_heads=1, dim=64, vdim=64, chunk=129, scale=0.125, width=96, blocks=4, conv=2)], vocab=536, width=320, eps=1e-6)

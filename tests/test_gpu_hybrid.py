@@ -1,6 +1,5 @@
 """Hybrid decoders on the GPU against the plain oracle: each mixer alone and whole models, in fp32 and bf16, as whole prompts,
 token by token, in portions, in mixed batches and through the engine's own generation."""
-import functools
 import json
 import os
 import subprocess
@@ -11,11 +10,9 @@ import torch
 
 from . import nikelix_oracle as oracle
 from .hybrid_models import aligned_design, design, hgrn2, latent, single_layer, small_design, wkv
+from .hybrid_session import BF16, DEV, F32, check, feed, mixed_session, model, session, tokens, want_logits
 
 pytestmark = pytest.mark.gpu
-DEV = "cuda"
-F32, BF16 = torch.float32, torch.bfloat16
-TOL = {F32: 2e-5, BF16: 4e-2}          # root mean square over the vocabulary, relative to that of the oracle's logits
 
 
 @pytest.fixture(autouse=True)
@@ -25,60 +22,6 @@ def _status_clean():
 
     torch.cuda.synchronize()
     _lib.check_status()
-
-
-def tokens(n, vocab, seed=0):
-    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
-
-
-@functools.lru_cache(maxsize=None)
-def _model(key, seed):
-    from art_b200.models.config import config_from_dict
-    from art_b200.models.hybrid import init_hybrid_weights
-
-    d = json.loads(key)
-    return d, init_hybrid_weights(config_from_dict(d), seed=seed, dtype=BF16)
-
-
-def model(d, seed=0):
-    return _model(json.dumps(d), seed)
-
-
-@functools.lru_cache(maxsize=None)
-def _oracle(key, seed, toks):
-    d, w = _model(key, seed)
-    return oracle.forward(d, w, list(toks), torch.float64).float()
-
-
-def want_logits(d, toks, seed=0):
-    return _oracle(json.dumps(d), seed, tuple(toks))
-
-
-def session(d, dtype, blocks=64, slots=4, seed=0, block_size=16):
-    from art_b200.engine.factory import build_runner
-    from art_b200.engine.kv_cache import BlockManager
-    from art_b200.engine.replay import Replay
-    from art_b200.models.config import config_from_dict
-
-    cfg = config_from_dict(d)
-    runner, kv = build_runner(cfg, model(d, seed)[1], num_blocks=blocks, block_size=block_size, num_slots=slots, dtype=dtype)
-    return Replay(runner, BlockManager(blocks, block_size, False), kv)
-
-
-def feed(rep, toks, cuts, name="a"):
-    """Logits of every position, the tokens cut into portions of the given sizes (the last size repeats)."""
-    out, at, i = [], 0, 0
-    while at < len(toks):
-        n = min(cuts[min(i, len(cuts) - 1)], len(toks) - at)
-        last = at + n == len(toks)
-        out.append(rep.step([{"id": name, "tokens": toks[at:at + n], "want": list(range(n))}], [name] if last else []).cpu())
-        at, i = at + n, i + 1
-    return torch.cat(out)
-
-
-def check(got, want, dtype, scale=1.0):
-    err = (got.float() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
-    assert torch.isfinite(got).all() and float(err.max()) < TOL[dtype] * scale, f"worst {float(err.max()):.2e} at {int(err.argmax())}"
 
 
 LAYERS = {"latent": latent(), "latent-one": latent(heads=1, dim=8, rot=2, rank=8, vdim=8, window=1), "latent-wide": latent(heads=17, dim=40, rot=16, rank=144, vdim=136),
@@ -129,37 +72,7 @@ def test_residual_stream_after_every_layer(dtype):
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
 def test_unequal_requests_in_mixed_batches_reuse_pages_and_slots(dtype):
-    """Portions beside single tokens, requests that pause, end and make room for others; each as if it ran alone."""
-    d = aligned_design()
-    lens = [180, 1, 37, 250, 90, 64, 33, 2]
-    reqs = [tokens(n, d["vocab"], 10 + i) for i, n in enumerate(lens)]
-    rep = session(d, dtype, blocks=40, slots=4)
-    g = torch.Generator().manual_seed(4)
-    at, got, live, nxt, used = [0] * 8, [[] for _ in lens], [], 0, set()
-    while nxt < 8 or live:
-        held = sum((lens[i] + 15) // 16 for i in live)
-        while nxt < 8 and len(live) < 4 and held + (lens[nxt] + 15) // 16 <= 40:
-            held += (lens[nxt] + 15) // 16
-            live.append(nxt)
-            nxt += 1
-        act = [i for i in live if torch.rand(1, generator=g).item() < 0.8] or live[:1]
-        entries, end, rows = [], [], []
-        for i in act:
-            n = min([1, 1, 2, 19, 64, 100][int(torch.randint(0, 6, (1,), generator=g))], lens[i] - at[i])
-            entries.append({"id": str(i), "tokens": reqs[i][at[i]:at[i] + n], "want": list(range(n))})
-            rows.append((i, n))
-            at[i] += n
-            if at[i] == lens[i]:
-                end.append(str(i))
-        out = rep.step(entries, end).cpu()
-        used |= {b for r in rep.live.values() for b in r.blocks}
-        for i, n in rows:
-            got[i].append(out[:n])
-            out = out[n:]
-        live = [i for i in live if at[i] < lens[i]]
-    assert rep.bm.num_free == 40 and rep.state_slots.num_free == 4
-    for i, r in enumerate(reqs):
-        check(torch.cat(got[i]), want_logits(d, r), dtype, 1.5)
+    mixed_session(aligned_design(), dtype, [180, 1, 37, 250, 90, 64, 33, 2], check)
 
 
 def test_far_past_is_kept_by_the_states_and_cut_by_the_window():
