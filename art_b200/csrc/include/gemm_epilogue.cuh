@@ -4,8 +4,8 @@
 
 namespace artb {
 
-// EPI_RELUGLU: as EPI_SWIGLU with relu as the gate's activation
-enum GemmEpilogue : int { EPI_BF16 = 0, EPI_BF16_RESID = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_SWIGLU_BWD = 4, EPI_RELUGLU = 5 };
+// EPI_RELUGLU: as EPI_SWIGLU with relu as the gate's activation.  EPI_SILU: as EPI_BF16, the first res_cols columns through silu.
+enum GemmEpilogue : int { EPI_BF16 = 0, EPI_BF16_RESID = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_SWIGLU_BWD = 4, EPI_RELUGLU = 5, EPI_SILU = 6 };
 __host__ __device__ inline bool epi_is_glu(int e) { return e == EPI_SWIGLU || e == EPI_RELUGLU; }
 
 // Tiles are visited with the M index fastest inside bands of group_m tile rows (see raster_tile), so the CTAs that
@@ -72,6 +72,7 @@ struct EpiStore {
   int res_cols;
   int swiglu_bwd = 0;
   int relu_gate = 0;
+  int silu_cols = 0;     // columns that leave as silu(acc)
   // Global operands of the NEXT 32-column chunk, loaded while the current chunk is converted and stored.
   // Residual (4 pieces): each thread reads its own row.  SwiGLU backward (8 pieces = 128 bytes of gate|up per row):
   // read cooperatively, 8 lanes per row, so that a warp-wide load touches 4 rows x 128 contiguous bytes instead of 32
@@ -205,6 +206,13 @@ struct EpiStore {
 #pragma unroll
         for (int j = 0; j < 32; ++j)
           if (gc + j < res_cols) acc[j] = __float_as_uint(__uint_as_float(acc[j]) + __bfloat162float(r[j]));
+      }
+    }
+    if (gc < silu_cols) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) {
+        const float z = __uint_as_float(acc[j]);
+        if (gc + j < silu_cols) acc[j] = __float_as_uint(__fdividef(z, 1.f + __expf(-z)));
       }
     }
     if (out_f32) {

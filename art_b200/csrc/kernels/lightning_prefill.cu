@@ -1,6 +1,7 @@
 // Lightning attention of prompt portions on tensor cores, in chunks of 64 tokens.
 //
-// With q, k, v = silu of the projections, a head's constant decay w and the state S before a chunk of n tokens
+// With q, k, v (activated: the projection's epilogue applies the silu), a head's constant decay w and the state S before a
+// chunk of n tokens
 //
 //   o_i = w^(i+1) q_i S + sum_{j <= i} w^(i-j) (q_i . k_j) v_j          S' = w^n S + sum_j k_j (w^(n-1-j) v_j)^T
 //
@@ -10,8 +11,8 @@
 // too; q, k and v themselves are bf16, as projections are.  The next chunk's rows are loaded while the current one is worked
 // on; two CTAs share an SM.
 //
-// Warp-level tiles: operands are made by the CUDA cores (activation, decay, splitting) chunk by chunk in a serial chain, which
-// leaves no long product to feed to the asynchronous tensor path.
+// Warp-level tiles: operands are made by the CUDA cores (decay, splitting) chunk by chunk in a serial chain, which leaves no
+// long product to feed to the asynchronous tensor path.
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
@@ -27,7 +28,7 @@ namespace artb {
 constexpr int LF_C = 64, LF_V = 64, LF_THREADS = 256;
 
 struct Lightning {
-  const __nv_bfloat16 *q, *k, *v;      // raw projections, [M, ld]: heads of dim (q, k) and vdim (v) columns
+  const __nv_bfloat16 *q, *k, *v;      // [M, ld]: heads of dim (q, k) and vdim (v) columns
   int ld;
   const float* decay;                  // [H]
   float* state;                        // [slots][H][vdim][ld_dim]
@@ -49,7 +50,6 @@ struct LfSmem {
   static constexpr int BYTES = ELEMS * 2 + (LF_C + 1) * 4;
 };
 
-__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pair_bf16(a, b);
   const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
@@ -118,16 +118,6 @@ __global__ void __launch_bounds__(LF_THREADS, 2) lightning_prefill_kernel(const 
       rv[i] = r < n && v0 + c < a.vdim ? *reinterpret_cast<const uint4*>(gv + static_cast<size_t>(row0 + t0 + r) * a.ld + c) : zero;
     }
   };
-  auto silu8 = [](uint4 r) -> uint4 {
-    uint32_t* p = reinterpret_cast<uint32_t*>(&r);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&p[i]));
-      p[i] = pair_bf16(silu_fast(f.x), silu_fast(f.y));
-    }
-    return r;
-  };
-
   fetch(0);
   __syncthreads();
   for (int t0 = 0; t0 < len; t0 += LF_C) {
@@ -136,14 +126,14 @@ __global__ void __launch_bounds__(LF_THREADS, 2) lightning_prefill_kernel(const 
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int x = tid + i * LF_THREADS, r = x / (D / 8), c = x % (D / 8) * 8;
-      *reinterpret_cast<uint4*>(sQ + r * LD + c) = silu8(rq[i]);
-      *reinterpret_cast<uint4*>(sK + r * LD + c) = silu8(rk[i]);
+      *reinterpret_cast<uint4*>(sQ + r * LD + c) = rq[i];
+      *reinterpret_cast<uint4*>(sK + r * LD + c) = rk[i];
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int x = tid + i * LF_THREADS, r = x / (LF_V / 8), c = x % (LF_V / 8) * 8;
       const float w = r < n ? pw[n - 1 - r] : 0.f;
-      const uint4 y = silu8(rv[i]);
+      const uint4 y = rv[i];
       uint4 hi, lo;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -290,7 +280,7 @@ static int launch_lightning(const Lightning& a, int n_seqs, cudaStream_t st) {
 
 using namespace artb;
 
-// q, k, v bf16 [M, ld] (raw projections, 16-byte aligned; dim, vdim and ld multiples of 8, dim <= 128); o fp32 [rows, ldo]
+// q, k, v bf16 [M, ld] (after the silu, 16-byte aligned; dim, vdim and ld multiples of 8, dim <= 128); o fp32 [rows, ldo]
 // gets H * vdim columns.  State and sequence arguments as artb_linear_scan.
 ARTB_EXPORT int artb_lightning_prefill(const void* q, const void* k, const void* v, int ld, const float* decay, float* state,
                                        long slot_stride, int ld_dim, long num_slots, const int* cu_q, const int* ctx,

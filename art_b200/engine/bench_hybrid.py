@@ -3,10 +3,12 @@
 Two parts, random weights throughout:
 
 * ``engine_rows``: prefill and decode tokens/s of whole models through :class:`~art_b200.engine.engine.Engine`, a hybrid
-  preset and a dense Llama-style model of the same width, depth and parameter count per layer, no adapters.
-* ``kernel_rows``: every kernel of the hybrid path at the layer sizes of a model, timed alone with CUDA events (L2 flushed
+  preset and a twin of the same width, depth and feed-forward parameters per layer, no adapters: a dense Llama-style model,
+  or a Qwen3-style mixture of experts where the preset has experts.
+* ``kernel_rows``, ``naselorn_kernel_rows``: every kernel of the hybrid path at the layer sizes of a model, timed alone with CUDA events (L2 flushed
   between calls), with its algorithmic bytes and FLOPs and the fraction of its roofline (the slower of bytes at the
-  measured copy bandwidth and FLOPs at the measured tensor or nominal fp32 rate), and the like kernels of the dense model.
+  measured copy bandwidth and FLOPs at the measured tensor or nominal fp32 rate), and the like kernels of the dense model
+  or of the other design.
 """
 from __future__ import annotations
 
@@ -30,12 +32,19 @@ def peaks() -> tuple[float, float]:
         return 6650.0, 1590.0
 
 
-def dense_twin(cfg):
+def twin(cfg):
     """A Llama-style dense model of the same width and depth whose feed-forward (three matrices) has the hybrid's
-    parameters (two matrices)."""
+    parameters (two matrices), or a Qwen3-style mixture of experts whose experts stand for the hybrid's shared one, too."""
     from ..models.config import ModelConfig
 
-    d, ff = cfg.hidden_size, max(s.ff for s in cfg.layers)
+    d = cfg.hidden_size
+    moe = next((s for s in cfg.layers if s.experts), None)
+    if moe is not None:
+        extra = moe.shared_ff // moe.expert_ff
+        return ModelConfig(name=f"moe-{cfg.name}", family="qwen3_moe", vocab_size=cfg.vocab_size, hidden_size=d, num_layers=cfg.num_layers,
+                           num_heads=d // 128, num_kv_heads=max(1, d // 128 // 4), head_dim=128, intermediate_size=0, qkv_bias=False, qk_norm=True,
+                           num_experts=moe.experts + extra, num_experts_per_tok=moe.top + extra, moe_intermediate_size=moe.expert_ff)
+    ff = max(s.ff for s in cfg.layers)
     return ModelConfig(name=f"dense-{cfg.name}", family="llama", vocab_size=cfg.vocab_size, hidden_size=d, num_layers=cfg.num_layers,
                        num_heads=d // 128, num_kv_heads=max(1, d // 128 // 4), head_dim=128, intermediate_size=(ff * 2 // 3 + 127) // 128 * 128,
                        qkv_bias=False, rope_theta=5e5)
@@ -50,7 +59,7 @@ def engine_rows(names: list[str], batches: list[int], prompt_len: int = 1024, ne
         if layers:
             cfg.layers = cfg.layers[:layers]
         for seqs in batches:
-            for c in (cfg, dense_twin(cfg)):
+            for c in (cfg, twin(cfg)):
                 r = measure_decode(c, "cuda", seqs=seqs, prompt_len=prompt_len, new_tokens=new_tokens, loras=0)
                 torch.cuda.empty_cache()
                 yield {"model": r["model"], "layers": c.num_layers, "params_b": round(c.num_params() / 1e9, 2), "seqs": seqs,
@@ -75,6 +84,21 @@ def _time(fn, flush: torch.Tensor, reps: int = 12) -> float:
     return sorted(ts)[len(ts) // 2]
 
 
+class _Rows:
+    """Timed kernels of one layer size."""
+
+    def __init__(self):
+        self.gbs, self.tf = peaks()
+        self.flush = torch.empty(64 << 20, dtype=torch.float32, device="cuda")
+        self.rows: list[dict] = []
+
+    def add(self, name: str, phase: str, fn, bytes_: float, tc_flops: float = 0.0, f32_flops: float = 0.0) -> None:
+        us = _time(fn, self.flush)
+        floor = max(bytes_ / self.gbs / 1e3, tc_flops / self.tf / 1e6, f32_flops / FP32_TFLOPS / 1e6)
+        self.rows.append({"kernel": name, "phase": phase, "us": round(us, 1), "floor_us": round(floor, 1), "of_roofline": round(floor / us, 3),
+                          "gb_s": round(bytes_ / us / 1e3, 0), "tflop_s": round((tc_flops + f32_flops) / us / 1e6, 1)})
+
+
 def kernel_rows(width: int = 4096, ff: int = 16384, prefill: int = 8192, decode: int = 256, window: int = 1024, ctx: int = 2048,
                 hist: int = 16) -> list[dict]:
     from ..ops import attention as attn_ops
@@ -84,18 +108,11 @@ def kernel_rows(width: int = 4096, ff: int = 16384, prefill: int = 8192, decode:
     from ..ops.gemm import gemm_tn
 
     dev, bf = "cuda", torch.bfloat16
-    gbs, tf = peaks()
-    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
-    rows: list[dict] = []
+    bench = _Rows()
+    rows, add = bench.rows, bench.add
     g = torch.Generator(device=dev).manual_seed(0)
     rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, generator=g) * sc).to(dt)      # noqa: E731
     i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
-
-    def add(name: str, phase: str, fn, bytes_: float, tc_flops: float = 0.0, f32_flops: float = 0.0) -> None:
-        us = _time(fn, flush)
-        floor = max(bytes_ / gbs / 1e3, tc_flops / tf / 1e6, f32_flops / FP32_TFLOPS / 1e6)
-        rows.append({"kernel": name, "phase": phase, "us": round(us, 1), "floor_us": round(floor, 1), "of_roofline": round(floor / us, 3),
-                     "gb_s": round(bytes_ / us / 1e3, 0), "tflop_s": round((tc_flops + f32_flops) / us / 1e6, 1)})
 
     d = width
     for phase, M in (("decode", decode), ("prefill", prefill)):
@@ -204,6 +221,141 @@ def kernel_rows(width: int = 4096, ff: int = 16384, prefill: int = 8192, decode:
     return rows
 
 
+def naselorn_kernel_rows(width: int = 4096, prefill: int = 8192, decode: int = 256, chunk: int = 1024, ctx: int = 2048, experts: int = 64,
+                         top: int = 8, expert_ff: int = 1024, dense_ff: int = 12288, block: int = 256) -> list[dict]:
+    """The kernels of Naselorn layers, each beside the like kernel of another design where there is one ("like: ...")."""
+    from ..ops import attention as attn_ops
+    from ..ops import elementwise as ew
+    from ..ops import hybrid as hy
+    from ..ops import moe, paged
+    from ..ops.gemm import gemm_tn
+
+    dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
+    bench = _Rows()
+    add = bench.add
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, generator=g) * sc).to(dt)      # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
+    d, H, hd, bs = width, width // 128, 128, 16
+    Hkv, G = H // 4, 4
+    for phase, M in (("decode", decode), ("prefill", prefill)):
+        one = phase == "decode"
+        n_seqs = M if one else M // 2048
+        cu = i32(list(range(M + 1)) if one else [i * 2048 for i in range(n_seqs + 1)])
+        row_seq = i32(list(range(M)) if one else [i // 2048 for i in range(M)])
+        c_len, slots = i32([ctx] * n_seqs), i32(list(range(n_seqs)))
+        pos = i32([ctx - 1] * M if one else [i % 2048 for i in range(M)])
+        x, w, h, y = rnd(M, d, dt=f32), rnd(d, dt=f32), rnd(M, d), rnd(M, d)
+        add("residual_step (pre-norm frame)", phase, lambda: hy.residual_step(x, None, d, 1e-5, y=hy.as_out(y), x_in=x, w_next=w, h=h), M * d * 12)
+        add("like: residual_step with post-norm", phase, lambda: hy.residual_step(x, w, d, 1e-5, y=hy.as_out(y), x_in=x, mult=0.5, w_next=w, h=h), M * d * 12)
+        # lightning attention
+        n = H * hd
+        p, st = rnd(M, 4 * n), torch.zeros(n_seqs, H, hd, hd, dtype=f32, device=dev)
+        P = hy.as_out(p)
+        decay = torch.rand(H, device=dev, generator=g)
+        o, o16, nw = torch.empty(M, n, dtype=f32, device=dev), torch.empty(M, n, dtype=bf, device=dev), rnd(n, dt=f32)
+        gr, aux = rnd(M, n, dt=f32), torch.rand(n, device=dev, generator=g)
+        scan = (decay, st, cu, c_len, slots)
+        in_bytes, flops = M * n * 6, 5.0 * M * H * hd * hd
+        if one:
+            add(f"linear_decode fixed {H} x {hd}^2", phase, lambda: hy.linear_decode(hy.SCAN_FIXED, P, P.col(n), P.col(2 * n), None, None, *scan, H, hd, hd, None,
+                                                                                 False, None, o, hd, 0.0), in_bytes + M * n * 4 + 8.0 * st.numel(), f32_flops=flops)
+            add(f"like: linear_decode hgrn2 {H} x {hd}^2", phase, lambda: hy.linear_decode(
+                hy.SCAN_HGRN2, P, None, P.col(2 * n), hy.as_out(gr), aux, aux, st, cu, c_len, slots, H, hd, hd, nw[:hd], False, None, o16, hd, 1e-5),
+                M * n * 10 + 8.0 * st.numel(), f32_flops=flops)
+        else:
+            # chunked form: q k^T, its product with v, q S and the state's update, the latter two with split operands
+            tc = 2.0 * M * H * (64 * hd + 2 * 64 * hd + 4 * hd * hd)
+            add(f"lightning_prefill {H} x {hd}^2", phase, lambda: hy.lightning_prefill(p[:, :n], p[:, n:2 * n], p[:, 2 * n:3 * n], *scan, n_seqs, H, hd, hd, o),
+                in_bytes + M * n * 4 + 8.0 * st.numel(), tc_flops=tc)
+            add(f"linear_scan fixed {H} x {hd}^2 (odd sizes, fp32)", phase, lambda: hy.linear_scan(
+                hy.SCAN_FIXED, P, P.col(n), P.col(2 * n), None, None, *scan, n_seqs, H, hd, hd, o), in_bytes + M * n * 4 + 8.0 * st.numel(), f32_flops=flops)
+            add(f"like: linear_scan hgrn2 {H} x {hd}^2", phase, lambda: hy.linear_scan(
+                hy.SCAN_HGRN2, P, None, P.col(2 * n), hy.as_out(gr), aux, aux, st, cu, c_len, slots, n_seqs, H, hd, hd, o),
+                M * n * 12 + 8.0 * st.numel(), f32_flops=flops)
+        add("row_norm with sigmoid gate", phase, lambda: hy.head_norm(o, nw, False, 1, n, n, o16, 1e-5, P.col(3 * n), hy.GATE_SIGMOID), M * n * 8)
+        add("like: head_norm with silu gate", phase, lambda: hy.head_norm(o, nw, True, H, hd, hd, o16, 1e-5, P.col(3 * n)), M * n * 8)
+        del st, gr, p, P
+        # chunked grouped-query attention
+        ld = Hkv * 2 * hd
+        nb = n_seqs * (ctx // bs)
+        cache = rnd(nb, bs, ld)
+        bt = torch.randperm(nb, device=dev, generator=g).to(torch.int32).view(n_seqs, ctx // bs)
+        qkv, bias = rnd(M, (H + 2 * Hkv) * hd), rnd((H + 2 * Hkv) * hd, dt=f32)
+        q, slot = torch.empty(M, H * hd, dtype=bf, device=dev), i32([i % (nb * bs) for i in range(M)])
+        add("gqa_finish", phase, lambda: hy.gqa_finish(hy.as_out(qkv), bias, slot, cache, q, H, Hkv, hd, hd, hd), 2 * qkv.numel() * 2)
+        ao = torch.empty(M, H * hd, dtype=bf, device=dev)
+        if one:
+            sp = hy.gqa_decode_splits(M, Hkv, chunk)
+            keys = (ctx - 1) % chunk + 1
+            add(f"gqa_decode chunk {chunk}", phase, lambda: hy.gqa_decode(q, cache, bt, row_seq, pos, c_len, 0, chunk, hd ** -0.5, 0.5, ao, M, H, Hkv, hd, hd, hd, sp),
+                M * keys * ld * 2 + M * H * hd * 4, 4.0 * M * H * keys * hd)
+            kc, vc = rnd(n_seqs * chunk // bs, bs, Hkv, hd), rnd(n_seqs * chunk // bs, bs, Hkv, hd)
+            btd = torch.arange(n_seqs * chunk // bs, dtype=torch.int32, device=dev).view(n_seqs, -1)
+            cd = i32([chunk] * M)
+            add(f"like: paged_decode ctx {chunk}", phase, lambda: paged.paged_decode(q, kc, vc, btd, cd, H, Hkv, hd, ao), M * chunk * ld * 2 + M * H * hd * 4,
+                4.0 * M * H * chunk * hd)
+        else:
+            plan = hy.plan_prefill([(i, 0, 2048) for i in range(n_seqs)], 0, dev, chunk)
+            add("gqa_gather", phase, lambda: hy.gqa_gather(cache, bt, plan, Hkv, hd, hd), plan.n_keys * ld * 4)
+            add("like: latent_gather", phase, lambda: hy.latent_gather(cache, bt, plan), plan.n_keys * ld * 4)
+            k, vt = hy.gqa_gather(cache, bt, plan, Hkv, hd, hd)
+            pairs = n_seqs * sum(i % chunk + 1 for i in range(2048))
+            add(f"latent_prefill_tc chunk {chunk}", phase, lambda: hy.latent_prefill_tc(q, k, vt, k, plan, 0, hd ** -0.5, ao, H, hd, hd, 0, 0, hd, chunk=chunk, G=G),
+                (q.numel() + k.numel() + vt.numel() + ao.numel()) * 2, 4.0 * H * pairs * hd)
+            ids = torch.arange(M // chunk, dtype=torch.int32, device=dev).repeat_interleave(chunk)
+            ap = attn_ops.make_plan(ids, ids, M, "native")
+            add(f"like: tree attention fwd, causal, {chunk} tokens", phase, lambda: attn_ops.forward(qkv, H, Hkv, hd, ap, need_grad=False),
+                qkv.numel() * 2 + M * H * hd * 2, 4.0 * H * pairs * hd)
+        # gated linear recurrent unit
+        nblk, bp = d // block, block
+        xy = hy.as_out(rnd(M, 2 * d))
+        u = torch.zeros(nblk, hy.pad(M, 128), 2 * bp, dtype=bf, device=dev)
+        cw, cst, rst = rnd(d, 4, dt=f32), torch.zeros(n_seqs, 3, d, device=dev), torch.zeros(n_seqs, d, device=dev)
+        add("short_conv", phase, lambda: hy.short_conv(xy.col(d), w, cw, w, cst, row_seq, cu, c_len, slots, n_seqs, one, u, block, bp), M * d * 6 + cst.numel() * 8)
+        gates, z = rnd(nblk, 2 * bp, 2 * bp, sc=block ** -0.5), torch.empty(M, 2 * d, dtype=f32, device=dev)
+        add("gemm_batched gates", phase, lambda: hy.gemm_batched(u, gates, z, M, c_batch=2 * bp), gates.numel() * 2 + M * d * 12, 2.0 * M * d * 4 * bp)
+        dec = torch.rand(d, device=dev, generator=g)
+        add("rglru", phase, lambda: hy.rglru(u, z, w, w, dec, xy, w, rst, cu, c_len, slots, n_seqs, one, o16, 0.5, block, bp), M * d * 16 + rst.numel() * 8)
+        del u, z, xy
+        # feed-forwards
+        gu = rnd(M, 2 * dense_ff)
+        a = torch.empty(M, dense_ff, dtype=bf, device=dev)
+        add("gated_act", phase, lambda: hy.gated_act(hy.as_out(gu), a, "relu"), M * dense_ff * 6)
+        add("like: swiglu_fwd", phase, lambda: ew.swiglu_fwd(gu, out=a), M * dense_ff * 6)
+        Wg = rnd(2 * dense_ff, d, sc=d ** -0.5)
+        pf = 4.0 * M * d * dense_ff
+        if not one:
+            add("gemm_tn gate|up, relu epilogue", phase, lambda: gemm_tn(h, Wg, swiglu_out=a, gate_act="relu", keep_preact=False),
+                (Wg.numel() + M * d + a.numel()) * 2, pf)
+            add("like: gemm_tn gate|up, silu epilogue", phase, lambda: gemm_tn(h, Wg, out=gu, swiglu_out=a), (Wg.numel() + M * d + 3 * a.numel()) * 2, pf)
+            Wp, qp = Wg[:4 * n], torch.empty(M, 4 * n, dtype=bf, device=dev)
+            qf = 2.0 * M * d * 4 * n
+            add("gemm_tn q|k|v|g, silu epilogue", phase, lambda: gemm_tn(h, Wp, out=qp, silu_cols=3 * n), (Wp.numel() + M * d + qp.numel()) * 2, qf)
+            add("like: gemm_tn, same product", phase, lambda: gemm_tn(h, Wp, out=qp), (Wp.numel() + M * d + qp.numel()) * 2, qf)
+            del qp, Wp
+        del gu, a, Wg
+        logits, rb = rnd(M, experts, dt=f32), rnd(experts, dt=f32)
+        add("moe.route (router, plan)", phase, lambda: moe.route(logits, top, True, rb), M * (experts * 4 + top * 8))
+        add("like: moe.route without bias", phase, lambda: moe.route(logits, top, True), M * (experts * 4 + top * 8))
+        rp = moe.route(logits, top, True, rb)
+        xp = moe.gather(h, rp)
+        add("moe.gather", phase, lambda: moe.gather(h, rp, out=xp), M * d * 2 * (1 + top))
+        eg, ed = rnd(experts * 2 * expert_ff, d, sc=d ** -0.5), rnd(experts * d, expert_ff, sc=expert_ff ** -0.5)
+        ea = torch.empty(rp.cap_rows, expert_ff, dtype=bf, device=dev)
+        yp = torch.empty(rp.cap_rows, d, dtype=bf, device=dev)
+        ef = 2.0 * M * top * d * expert_ff
+        add("grouped_gemm gate|up, silu epilogue", phase, lambda: moe.grouped_gemm(xp, eg, rp, 2 * expert_ff, swiglu_out=ea, keep_preact=False),
+            (eg.numel() + M * top * (d + expert_ff)) * 2, 2 * ef)
+        add("grouped_gemm down", phase, lambda: moe.grouped_gemm(ea, ed, rp, d, out=yp), (ed.numel() + M * top * (d + expert_ff)) * 2, ef)
+        sub = hy.Sublayer(hy.as_out(y), rows=yp, pos=rp.pos, weight=rp.topw)
+        add("residual_step with experts' rows", phase, lambda: hy.residual_step(x, None, d, 1e-5, sub=sub, x_in=x, w_next=w, h=h), M * d * (12 + 2 * top))
+        add("like: moe.combine", phase, lambda: moe.combine(yp, rp, residual=y), M * d * 2 * (2 + top))
+        del eg, ed, ea, yp, xp, cache, qkv, q, ao, o, o16
+        torch.cuda.empty_cache()
+    return bench.rows
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--models", default="nikelix-1b,nikelix-7b")
@@ -219,8 +371,10 @@ def report(models: list[str], batches: list[int], layers: int, part: str = "both
     from ..ops import _lib
 
     if part != "engine":
-        yield from ({"part": "kernel", **r} for r in kernel_rows())
-        torch.cuda.empty_cache()
+        for design, fn in (("nikelix", kernel_rows), ("naselorn", naselorn_kernel_rows)):
+            if any(m.startswith(design) for m in models):
+                yield from ({"part": "kernel", "design": design, **r} for r in fn())
+                torch.cuda.empty_cache()
     if part != "kernels":
         yield from ({"part": "engine", **r} for r in engine_rows(models, batches, layers=layers))
     _lib.check_status()

@@ -262,6 +262,12 @@ class HybridRunner(DeviceRunner):
 
         return as_out(gemm_tn(x, W, out=out, out_dtype=out.dtype))
 
+    def _mm_silu(self, x, W, cols: int) -> Out:
+        """``x W^T``, the first ``cols`` columns through silu in the product's epilogue (bf16)."""
+        from ..ops.gemm import gemm_tn
+
+        return as_out(gemm_tn(x, W, out=self._new(x.shape[0], W.shape[0]), silu_cols=cols))
+
     def _mm_take(self, b: Ragged, name: str, x, W, f32: bool = False) -> Out:
         """``x W^T`` for a consumer that accepts a split-K workspace: with few rows the product streams the weights from
         all SMs and adds partial sums into the fp32 workspace ``name``, which the consumer reads once and leaves zero."""
@@ -478,14 +484,15 @@ class HybridRunner(DeviceRunner):
 
     def _mix_lightning(self, i, s, L, x, h, b: Ragged) -> Sublayer:
         M, n, nv = b.M, s.heads * s.dim, s.heads * s.vdim
-        p = self._mm_take(b, "qkvg", h, L["qkvg"])
+        chunked = not b.single and not self.exact32 and hy.lightning_tc(s.dim, s.vdim)
+        p = self._mm_silu(h, L["qkvg"], 2 * n + nv) if chunked else self._mm_take(b, "qkvg", h, L["qkvg"])
         q, k, v, gate = p, p.col(n), p.col(2 * n), p.col(2 * n + nv)
         state = self.kv.layers[i]["state"]
         o, out = self._new(M, nv, torch.float32), self._new(M, pad(nv))
         if b.single:
             hy.linear_decode(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, s.heads, s.dim, s.vdim, None, False,
                              None, o, s.vdim, 0.0)
-        elif not self.exact32 and hy.lightning_tc(s.dim, s.vdim):
+        elif chunked:
             hy.lightning_prefill(q.t, k.t, v.t, L["decay"], state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, s.heads, s.dim, s.vdim, o)
         else:
             hy.linear_scan(hy.SCAN_FIXED, q, k, v, None, None, L["decay"], state, b.cu_q, b.ctx, b.state_slot, b.n_seqs, s.heads, s.dim, s.vdim, o)

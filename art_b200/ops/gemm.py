@@ -13,7 +13,7 @@ import torch
 
 from . import _lib
 
-EPI_BF16, EPI_BF16_RESID, EPI_F32, EPI_SWIGLU, EPI_SWIGLU_BWD, EPI_RELUGLU = 0, 1, 2, 3, 4, 5
+EPI_BF16, EPI_BF16_RESID, EPI_F32, EPI_SWIGLU, EPI_SWIGLU_BWD, EPI_RELUGLU, EPI_SILU = 0, 1, 2, 3, 4, 5, 6
 _configured = False
 _configured2 = False
 TWO_CTA_DEFAULT = os.environ.get("ARTB_GEMM_2CTA", "1") == "1"
@@ -53,13 +53,15 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
             bias: torch.Tensor | None = None, res_cols: int = 0,
             out_dtype: torch.dtype = torch.bfloat16, bn: int = 0, max_ctas: int = 0,
             two_cta: bool | None = None, swiglu_bwd_gu: torch.Tensor | None = None, gate_act: str = "silu",
-            keep_preact: bool = True) -> torch.Tensor | None:
+            keep_preact: bool = True, silu_cols: int = 0) -> torch.Tensor | None:
     """``out[M,N] = a[M,K] @ b[N,K].T (+ a2[M,K2] @ b2[N,K2].T) (+ residual)``.
 
     ``swiglu_out`` ([M, N/2] bf16) selects the SwiGLU epilogue: ``b``'s rows must be
     interleaved in blocks of 16 (gate rows, then the matching up rows); ``out`` receives
     the pre-activation and ``swiglu_out`` receives ``silu(gate) * up`` (``gate_act="relu"``: ``relu(gate) * up``);
     with ``keep_preact=False`` only ``swiglu_out`` is written and nothing is returned.
+
+    ``silu_cols``: the first columns of the product leave through silu (bf16 output, no other epilogue).
 
     ``swiglu_bwd_gu`` ([M, 2N] bf16, the forward's interleaved gate|up pre-activations) selects the fused
     SwiGLU-backward epilogue: the product is taken as ``d(silu(gate) * up)`` and ``out`` ([M, 2N]) receives
@@ -88,6 +90,10 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
         swiglu_out = swiglu_bwd_gu          # travels in the H slot of the C entry point
     elif swiglu_out is not None:
         epi = EPI_RELUGLU if gate_act == "relu" else EPI_SWIGLU
+    elif silu_cols > 0:
+        if residual is not None or out_dtype != torch.bfloat16:
+            raise ValueError("silu_cols: a plain bf16 product")
+        epi, res_cols = EPI_SILU, silu_cols
     elif residual is not None:
         epi = EPI_BF16_RESID
     elif out_dtype == torch.float32:

@@ -205,7 +205,8 @@ def lightning_tc(dim: int, vdim: int) -> bool:
 
 
 def lightning_prefill(q, k, v, decay, state, cu_q, ctx, state_slot, n_seqs: int, H: int, dim: int, vdim: int, o) -> torch.Tensor:
-    """``linear_scan(SCAN_FIXED, ...)`` in chunks on tensor cores; ``q``, ``k``, ``v`` bf16 columns of one projection."""
+    """``linear_scan(SCAN_FIXED, ...)`` in chunks on tensor cores; ``q``, ``k``, ``v`` bf16 columns of one projection that have
+    been through the silu already."""
     if not q.stride(0) == k.stride(0) == v.stride(0):
         raise ValueError("q, k and v come from one projection")
     _lib.check_rc(_f("artb_lightning_prefill")(

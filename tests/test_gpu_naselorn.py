@@ -272,21 +272,21 @@ def test_lightning_kernels_against_the_recurrence(n_seqs, H, dim, vdim):
     fresh = [i % 3 == 1 for i in range(n_seqs)]
     ctx = [n if f else n + 5 for n, f in zip(lens, fresh)]
     silu = lambda t, w: oracle.silu(t.double()).view(-1, H, w)      # noqa: E731
-    forms = [("scan", F32, 3e-6), ("scan", BF16, 3e-6)] + ([("tiles", BF16, 4e-3)] if hy.lightning_tc(dim, vdim) else [])
+    forms = [("scan", F32, 3e-6), ("scan", BF16, 3e-6)] + ([("tiles", BF16, 2e-5)] if hy.lightning_tc(dim, vdim) else [])
     for form, dt, tol in forms:
         state, o = init.clone(), torch.zeros(M, nv, device=DEV)
         as_ = lambda t: hy.as_out(t.to(dt))      # noqa: E731
         if form == "tiles":
-            hy.lightning_prefill(q, k, v, decay, state, i32(cu), i32(ctx), i32(slots), n_seqs, H, dim, vdim, o)
+            act = oracle.silu(p.float()).to(BF16)
+            hy.lightning_prefill(act[:, :nk], act[:, nk:2 * nk], act[:, 2 * nk:], decay, state, i32(cu), i32(ctx), i32(slots), n_seqs, H, dim, vdim, o)
         else:
             hy.linear_scan(hy.SCAN_FIXED, as_(q), as_(k), as_(v), None, None, decay, state, i32(cu), i32(ctx), i32(slots), n_seqs, H, dim, vdim, o)
         for i in sorted(set(list(range(min(n_seqs, 5))) + [n_seqs - 1])):
             r = slice(cu[i], cu[i + 1])
             qq, kk, vv = silu(q[r], dim), silu(k[r], dim), silu(v[r], vdim)
             S0 = torch.zeros(H, dim, vdim, dtype=torch.float64, device=DEV) if fresh[i] else init[slots[i], ..., :dim].double().transpose(1, 2)
-            if form == "tiles":       # activations as the kernel rounds them: what remains must be fp32 accurate
-                qq, kk, vv = (t.to(BF16).double() for t in (qq, kk, vv))
-                tol = 3e-3
+            if form == "tiles":       # with activations that are bf16 numbers the chunked form keeps fp32 accuracy
+                qq, kk, vv = (t[r].double().view(-1, H, w) for t, w in ((act[:, :nk], dim), (act[:, nk:2 * nk], dim), (act[:, 2 * nk:], vdim)))
             ref, S = lightning_reference(qq, kk, vv, decay.double(), S0)
             assert ((o[r].view(-1, H, vdim).double() - ref).norm() / ref.norm()).item() < tol
             got = state[slots[i], ..., :dim].transpose(1, 2).double()
@@ -307,26 +307,6 @@ def test_lightning_kernels_against_the_recurrence(n_seqs, H, dim, vdim):
                                      init[sl[i], ..., :dim].double().transpose(1, 2))
         assert ((o[i].view(1, H, vdim).double() - ref).norm() / ref.norm()).item() < 3e-6
         assert ((state[sl[i], ..., :dim].transpose(1, 2).double() - S).norm() / S.norm()).item() < 3e-6
-
-
-def test_lightning_tiles_round_nothing_that_enters_the_state():
-    """With activations that are bf16 numbers the chunked form must agree with the recurrence to fp32 accuracy."""
-    from art_b200.ops import hybrid as hy
-
-    H, dim, vdim, M = 2, 64, 64, 700
-    z = torch.tensor([-30.0, 0.0, 30.0, 60.0], device=DEV)       # silu: 0 (below fp32 resolution), 0, 30, 60
-    g = torch.Generator(device=DEV).manual_seed(3)
-    p = z[torch.randint(0, 4, (M, 3 * H * dim), device=DEV, generator=g)].to(BF16)
-    p[:, 2 * H * dim:] = (torch.randint(20, 64, (M, H * vdim), device=DEV, generator=g)).to(BF16)
-    decay = torch.tensor([0.999, 0.7], device=DEV)
-    state, o = torch.zeros(1, H, vdim, dim, device=DEV), torch.zeros(M, H * vdim, device=DEV)
-    n = H * dim
-    hy.lightning_prefill(p[:, :n], p[:, n:2 * n], p[:, 2 * n:], decay, state, i32([0, M]), i32([M]), i32([0]), 1, H, dim, vdim, o)
-    sil = lambda t, w: oracle.silu(t.double()).view(-1, H, w)      # noqa: E731
-    ref, S = lightning_reference(sil(p[:, :n], dim), sil(p[:, n:2 * n], dim), sil(p[:, 2 * n:], vdim), decay.double(),
-                                 torch.zeros(H, dim, vdim, dtype=torch.float64, device=DEV))
-    assert ((o.view(M, H, vdim).double() - ref).norm(dim=-1) / ref.norm(dim=-1).clamp(min=1e-9)).max().item() < 3e-5
-    assert ((state[0].transpose(1, 2).double() - S).norm() / S.norm()).item() < 1e-5
 
 
 @DTYPES
@@ -530,6 +510,18 @@ def test_relu_gate_in_the_product_epilogue(M, pairs):
         assert gemm_tn(a, W, swiglu_out=out, gate_act=act, keep_preact=False, two_cta=pairs) is None
         ref = f(a.double() @ wg.double().T) * (a.double() @ wu.double().T)
         assert ((out.double() - ref).norm() / ref.norm()).item() < 1e-2
+
+
+@pytest.mark.parametrize("M,N,cols,pairs", [(40, 136, 72, False), (300, 264, 264, False), (1030, 520, 392, True)])
+def test_silu_of_the_first_columns_in_the_product_epilogue(M, N, cols, pairs):
+    from art_b200.ops.gemm import gemm_tn
+
+    rnd = rand(N)
+    a, W = rnd(M, 128).to(BF16), rnd(N, 128).mul(0.2).to(BF16)
+    out = gemm_tn(a, W, silu_cols=cols, two_cta=pairs)
+    ref = a.double() @ W.double().T
+    ref[:, :cols] = oracle.silu(ref[:, :cols])
+    assert torch.allclose(out.double(), ref, atol=1e-2, rtol=1e-2)
 
 
 @DTYPES
