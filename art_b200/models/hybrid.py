@@ -182,7 +182,7 @@ def _read_naselorn(d: dict, name: str) -> HybridConfig:
             if width % blocks:
                 raise ValueError(f"layer {i}: {width} channels do not divide over {blocks} blocks")
             parts = (LayerSpec("attention", int(a["heads"]), int(a["dim"]), int(a["vdim"]), kv_heads=int(a["kv_heads"]), scale=float(a["scale"]),
-                               chunk=int(a["mask"]["size"]), biases=True),
+                               chunk=int((a.get("mask") or {}).get("size", 0)), biases=True),
                      LayerSpec("rglru", blocks, width // blocks, width // blocks, conv=int(r["conv"])))
             spec = LayerSpec(kind, 0, 0, 0, parts=parts, part_scales=(float(m["left_scale"]), float(m["right_scale"])))
         ff = _mlp_kind(i, mlp, ("dense", "moe"))

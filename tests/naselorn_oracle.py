@@ -68,7 +68,7 @@ def short_conv(x, taps, bias):
 
 
 def rglru(h, w, p):
-    """Recurrent block with a real-gated linear recurrent unit."""
+    """Gated recurrence per channel behind a short convolution, times a gelu branch."""
     T, n, blocks = h.shape[0], p["width"], p["blocks"]
     y = gelu_tanh(h @ w["y"].T + w["y.b"])
     u = short_conv(h @ w["x"].T + w["x.b"], w["conv"], w["conv.b"])
