@@ -10,6 +10,9 @@ Two shared objects are produced under ``art_b200/_native``:
 * ``libartb_runtime.so``  the host runtime (paged-KV block manager, continuous-batching
   scheduler, packer) from ``csrc/engine/*.cpp``, compiled by g++.
 
+A process that needs few kernels (the replay of a trace) may ask for a library of just those sources where the complete one
+has not been built: ``build_part``.
+
 ``python -m art_b200.build`` rebuilds what is out of date; ``build_all(force=True)``
 rebuilds everything.  Object files are cached under ``art_b200/_native/obj``.
 """
@@ -85,6 +88,45 @@ def runtime_sources() -> list[Path]:
     return sorted(p for p in (CSRC / "engine").glob("*.cpp") if not p.name.endswith("_selftest.cpp"))
 
 
+def _compile(sources: list[Path], cmd_prefix: list[str], flags: list[str], verbose: bool = False, obj_dir: Path | None = None) -> list[Path]:
+    (obj_dir or OBJ).mkdir(parents=True, exist_ok=True)
+    with cf.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as pool:
+        return list(pool.map(lambda s: _compile_one(s, cmd_prefix, flags, verbose, obj_dir), sources))
+
+
+def _link(lib: Path, objs: list[Path], cmd: list[str], force: bool = False) -> None:
+    if not objs:
+        return
+    if lib.exists() and not force and all(lib.stat().st_mtime >= o.stat().st_mtime for o in objs):
+        return
+    tmp = lib.with_suffix(f".so.{os.getpid()}.tmp")
+    res = subprocess.run(cmd + [str(o) for o in objs] + ["-o", str(tmp)], capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link failed: {lib}\n{res.stdout}\n{res.stderr}")
+    os.replace(tmp, lib)
+
+
+def _link_kernels(nvcc: str) -> list[str]:
+    return [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"]
+
+
+def build_runtime(verbose: bool = False, force: bool = False) -> Path:
+    """The host runtime library alone."""
+    _link(RUNTIME_LIB, _compile(runtime_sources(), ["g++"], CXX_FLAGS, verbose), ["g++", "-shared", "-fPIC", "-pthread"], force)
+    return RUNTIME_LIB
+
+
+def build_part(stems) -> Path:
+    """A kernel library of the named sources alone (``csrc/kernels/<stem>.cu``); its name follows from their contents."""
+    sources = [CSRC / "kernels" / f"{s}.cu" for s in sorted(stems)]
+    h = hashlib.sha256("".join(s.stem + _digest(s, NVCC_FLAGS) for s in sources).encode()).hexdigest()[:16]
+    lib = OUT / f"libartb_part_{h}.so"
+    if not lib.exists():
+        nvcc = _nvcc()
+        _link(lib, _compile(sources, [nvcc], NVCC_FLAGS), _link_kernels(nvcc))
+    return lib
+
+
 def build_all(force: bool = False, verbose: bool = False, ptxas_info: bool = False, checked: bool = False) -> None:
     OBJ.mkdir(parents=True, exist_ok=True)
     if force:
@@ -98,19 +140,8 @@ def build_all(force: bool = False, verbose: bool = False, ptxas_info: bool = Fal
         kobjs = [j.result() for j in kjobs]
         robjs = [j.result() for j in rjobs]
 
-    def _link(lib: Path, objs: list[Path], cmd: list[str]) -> None:
-        if not objs:
-            return
-        if lib.exists() and not force and all(lib.stat().st_mtime >= o.stat().st_mtime for o in objs):
-            return
-        tmp = lib.with_suffix(".so.tmp")
-        res = subprocess.run(cmd + [str(o) for o in objs] + ["-o", str(tmp)], capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed: {lib}\n{res.stdout}\n{res.stderr}")
-        os.replace(tmp, lib)
-
-    _link(KERNEL_LIB, kobjs, [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"])
-    _link(RUNTIME_LIB, robjs, ["g++", "-shared", "-fPIC", "-pthread"])
+    _link(KERNEL_LIB, kobjs, _link_kernels(nvcc), force)
+    _link(RUNTIME_LIB, robjs, ["g++", "-shared", "-fPIC", "-pthread"], force)
     if checked:
         # the same kernels with device-side index checks compiled in (csrc/include/bounds_check.cuh); loaded instead of
         # the normal library when ARTB_BOUNDS_CHECK=1 is set in the environment
@@ -120,7 +151,7 @@ def build_all(force: bool = False, verbose: bool = False, ptxas_info: bool = Fal
             cjobs = [pool.submit(_compile_one, s, [nvcc], nv_flags + ["-DARTB_BOUNDS_CHECK"], verbose, cdir)
                      for s in kernel_sources()]
             cobjs = [j.result() for j in cjobs]
-        _link(CHECKED_KERNEL_LIB, cobjs, [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"])
+        _link(CHECKED_KERNEL_LIB, cobjs, _link_kernels(nvcc), force)
 
 
 if __name__ == "__main__":

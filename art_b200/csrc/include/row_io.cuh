@@ -8,7 +8,7 @@
 
 namespace artb {
 
-enum GatedAct : int { ACT_SILU = 0, ACT_RELU = 1 };      // act(gate) * up
+enum RowAct : int { ACT_SILU = 0, ACT_RELU = 1, ACT_RELU2 = 2 };      // ACT_RELU2: the square of relu
 enum RowKind : int { ROW_BF16 = 0, ROW_F32 = 1, ROW_F32_TAKE = 2 };
 
 __device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -89,7 +89,17 @@ __device__ __forceinline__ float cta_sum(float v, float* red) {
   return lane_sum(t);
 }
 
+// sine and cosine of pos * freq; the angle is reduced in double so that far positions lose nothing
+__device__ __forceinline__ float2 position_pair(int pos, double freq) {
+  constexpr double TWO_PI = 6.283185307179586476925;
+  const double ang = pos * freq;
+  float2 r;
+  sincosf(static_cast<float>(ang - rint(ang / TWO_PI) * TWO_PI), &r.x, &r.y);
+  return r;
+}
+
 __device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+__device__ __forceinline__ float logistic_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
 }  // namespace artb

@@ -49,7 +49,7 @@ ARTB_EXPORT int artb_gemm_grouped_bf16_tn(const void* A, int lda, const void* B,
                                           int epilogue, int* status, cudaStream_t stream) {
   if (m_tiles <= 0 || num_experts <= 0 || N <= 0 || K <= 0 || K2 < 0) return ERR_BAD_SHAPE;
   if ((K & 7) || (K2 & 7) || (N & 7) || (ldc & 7)) return ERR_BAD_SHAPE;
-  if (epilogue != EPI_BF16 && !epi_is_glu(epilogue)) return ERR_BAD_SHAPE;
+  if (epilogue != EPI_BF16 && epilogue != EPI_RELU2 && !epi_is_glu(epilogue)) return ERR_BAD_SHAPE;
   if (epi_is_glu(epilogue) && (!H || (ldh & 7) || (N & 31))) return ERR_BAD_ALIGN;
   if (!epi_is_glu(epilogue)) H = nullptr;
   if (!C && !H) return ERR_BAD_SHAPE;
@@ -71,7 +71,7 @@ ARTB_EXPORT int artb_gemm_grouped_bf16_tn(const void* A, int lda, const void* B,
   {                                                                                                            \
     SchedGrouped sched{tile_expert, m_tiles, (N + BN_ - 1) / BN_, N};                                          \
     EpiGrouped<BN_> epi{EpiStore<BN_, 1>{C, nullptr, reinterpret_cast<__nv_bfloat16*>(H), nullptr, ldc, 0, ldh,   \
-                                      M, N, 0, N, 0, epilogue == EPI_RELUGLU ? 1 : 0}};                                                            \
+                                      M, N, 0, N, 0, epilogue == EPI_RELUGLU ? 1 : 0, 0, epilogue == EPI_RELU2 ? 1 : 0}};                       \
     return launch_grouped<BN_, ST_>(tA, tB, tA2, tB2, kb_main, kb_extra, sched, epi, status, stream);          \
   }
   if (bn == 256) ARTB_LAUNCH(256, 4)

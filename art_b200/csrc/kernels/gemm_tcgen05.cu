@@ -109,7 +109,7 @@ ARTB_EXPORT int artb_gemm_bf16_tn(const void* A, int lda, const void* B, int ldb
                       reinterpret_cast<__nv_bfloat16*>(H), bias, ldc, ldr, ldh, M, N,              \
                       epilogue == EPI_F32 ? 1 : 0, res_cols > 0 ? res_cols : N,                   \
                       epilogue == EPI_SWIGLU_BWD ? 1 : 0, epilogue == EPI_RELUGLU ? 1 : 0,        \
-                      epilogue == EPI_SILU ? res_cols : 0};                                       \
+                      epilogue == EPI_SILU ? res_cols : 0, epilogue == EPI_RELU2 ? 1 : 0};        \
     return launch_gemm<BN_, ST_>(tA, tB, tA2, tB2, kb_main, kb_extra, M, N, epi, status, max_ctas, \
                                  stream);                                                         \
   }

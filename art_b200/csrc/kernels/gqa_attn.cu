@@ -1,8 +1,11 @@
-// Grouped-query attention over a paged cache with a key mask (window or chunk) and value heads of their own size.
+// Grouped-query attention over a paged cache with a key mask (window or chunk), value heads of their own size, optionally
+// squashed scores and a factor per row and head.
 //
 // A token's cache row is [ keys of the Hkv heads: dk_p each | values of the Hkv heads: dv_p each ], padded with zeros.
 //
 //   gqa_finish_kernel    what follows the q | k | v projection, one CTA per token: biases, cache write, padded queries
+//   gqa_finish_norm_kernel   the same with a norm over all heads of q, and of k, a rotation of the first columns of every head
+//                        (angles reduced in fp64, as for position vectors) and the heads' gates
 //   gqa_gather_kernel    the cache rows a batch's portions see, contiguous: keys row by row, values transposed, as the
 //                        tcgen05 kernel of latent_prefill_tc.cu wants them (sizes that do not suit it: latent_gather and
 //                        latent_prefill)
@@ -19,6 +22,7 @@
 #include "key_mask.cuh"
 #include "mma_tile.cuh"
 #include "row_io.cuh"
+#include "softcap.cuh"
 
 namespace artb {
 
@@ -32,8 +36,16 @@ struct GqaFinish {
   long num_slots;
   void* q;                  // T [M, ldq], heads of dk_p
   int ldq;
-  int H, Hkv, dim, dk_p, vdim, dv_p;
+  int H, Hkv, dim, dk_p, vdim, dv_p;      // Hkv = 0: q alone (keys and values are another layer's)
   int* status;
+  // gqa_finish_norm_kernel alone
+  const float *wq, *wk;     // fp32 norm weights over all heads of q and of k, or null
+  float eps;
+  const double* freq;       // angle of pair i of position p: p * freq[i], rot / 2 pairs
+  float rot_scale;          // factor of sine and cosine
+  int rot, next;            // rotated columns of a head; partner: the neighbour (next) or rot / 2 columns further
+  const int* pos;
+  float* gate;              // fp32 [M, H]: the sigmoid of the columns behind v, or null
 };
 
 template <typename T, int V>
@@ -72,6 +84,124 @@ __global__ void __launch_bounds__(256) gqa_finish_kernel(const GqaFinish a) {
   }
   const int np = a.dk_p - a.dim;
   for (int j = threadIdx.x; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
+}
+
+// V = 4: dim, vdim and the projection's pitch are multiples of 4, rot of 8
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gqa_finish_norm_kernel(const GqaFinish a) {
+  extern __shared__ __align__(16) float gn_smem[];      // [nq + nk] columns times their norm weights, then [rot / 2] (cos, sin)
+  __shared__ float red[2][8];
+  constexpr int B = 4;                                  // loads of a thread in flight
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, tid = threadIdx.x;
+  int slot = a.slot[m];
+  if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
+  T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
+  T* qrow = reinterpret_cast<T*>(a.q) + static_cast<size_t>(m) * a.ldq;
+  const int nq = a.H * a.dim, nqk = nq + a.Hkv * a.dim, n = nqk + a.Hkv * a.vdim, half = a.rot >> 1;
+  const size_t row = static_cast<size_t>(m) * a.ldp;
+  float2* turn = reinterpret_cast<float2*>(gn_smem + ((nqk + 3) & ~3));
+  float ssq = 0.f, ssk = 0.f;
+  for (int c0 = tid * V; c0 < n; c0 += blockDim.x * V * B) {
+    float x[B][V];
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = c0 + u * blockDim.x * V;
+      if (c >= n) continue;
+      if (V == 4) {
+        const float4 v = take4(a.p, row + c, a.kind);
+        x[u][0] = v.x, x[u][1 % V] = v.y, x[u][2 % V] = v.z, x[u][3 % V] = v.w;
+      } else {
+        x[u][0] = take1(a.p, row + c, a.kind);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = c0 + u * blockDim.x * V;
+      if (c >= n) continue;
+#pragma unroll
+      for (int e = 0; e < V; ++e)
+        if (a.bias) x[u][e] += a.bias[c + e];
+      if (c >= nqk) {
+        if (slot < 0) continue;
+        T* dst = crow + a.Hkv * a.dk_p + (c - nqk) / a.vdim * a.dv_p + (c - nqk) % a.vdim;
+        if (V == 4) st4(dst, make_float4(x[u][0], x[u][1 % V], x[u][2 % V], x[u][3 % V]));
+        else st1(dst, x[u][0]);
+        continue;
+      }
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < V; ++e) s = fmaf(x[u][e], x[u][e], s);
+      if (c < nq) ssq += s;
+      else ssk += s;
+      const float* w = c < nq ? a.wq : a.wk;
+      if (w) {
+        w += c < nq ? c : c - nq;
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[u][e] *= w[e];
+      }
+      if (V == 4) st4(gn_smem + c, make_float4(x[u][0], x[u][1 % V], x[u][2 % V], x[u][3 % V]));
+      else gn_smem[c] = x[u][0];
+    }
+  }
+  if (a.gate)
+    for (int h = tid; h < a.H; h += blockDim.x) a.gate[static_cast<size_t>(m) * a.H + h] = logistic_f(take1(a.p, row + n + h, a.kind));
+  for (int i = tid; i < half; i += blockDim.x) {
+    const float2 t = position_pair(a.pos[m], a.freq[i]);
+    turn[i] = make_float2(a.rot_scale * t.y, a.rot_scale * t.x);
+  }
+  ssq = lane_sum(ssq);
+  ssk = lane_sum(ssk);
+  const int warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
+  if (lane == 0) red[0][warp] = ssq, red[1][warp] = ssk;
+  __syncthreads();
+  ssq = lane_sum(lane < nw ? red[0][lane] : 0.f);
+  ssk = lane_sum(lane < nw ? red[1][lane] : 0.f);
+  const float rq = a.wq ? 1.f / sqrtf(ssq / nq + a.eps) : 1.f;
+  const float rk = a.wk ? 1.f / sqrtf(ssk / max(1, nqk - nq) + a.eps) : 1.f;
+  for (int c = tid * V; c < (slot < 0 ? nq : nqk); c += blockDim.x * V) {
+    const bool isq = c < nq;
+    const int cc = isq ? c : c - nq, hd = cc / a.dim, d = cc - hd * a.dim;
+    const float r = isq ? rq : rk;
+    float y[V];
+    if (V == 4) {
+      const float4 x = ld4(gn_smem + c);
+      if (d >= a.rot) {
+        y[0] = x.x, y[1 % V] = x.y, y[2 % V] = x.z, y[3 % V] = x.w;
+      } else if (a.next) {
+        const float2 t0 = turn[d >> 1], t1 = turn[(d >> 1) + 1];
+        y[0] = x.x * t0.x - x.y * t0.y;
+        y[1 % V] = x.y * t0.x + x.x * t0.y;
+        y[2 % V] = x.z * t1.x - x.w * t1.y;
+        y[3 % V] = x.w * t1.x + x.z * t1.y;
+      } else {
+        const bool lo = d < half;
+        const float4 z = ld4(gn_smem + (lo ? c + half : c - half));
+        const int i = lo ? d : d - half;
+        const float sg = lo ? -1.f : 1.f;
+        const float2 t0 = turn[i], t1 = turn[i + 1], t2 = turn[i + 2], t3 = turn[i + 3];
+        y[0] = fmaf(sg * z.x, t0.y, x.x * t0.x);
+        y[1 % V] = fmaf(sg * z.y, t1.y, x.y * t1.x);
+        y[2 % V] = fmaf(sg * z.z, t2.y, x.z * t2.x);
+        y[3 % V] = fmaf(sg * z.w, t3.y, x.w * t3.x);
+      }
+    } else {
+      const float x = gn_smem[c];
+      y[0] = x;
+      if (d < a.rot) {
+        const bool lo = a.next ? !(d & 1) : d < half;
+        const int step = a.next ? 1 : half, i = a.next ? d >> 1 : lo ? d : d - half;
+        const float z = gn_smem[lo ? c + step : c - step];
+        y[0] = fmaf(lo ? -z : z, turn[i].y, x * turn[i].x);
+      }
+    }
+    T* dst = (isq ? qrow : crow) + hd * a.dk_p + d;
+    if (V == 4) st4(dst, make_float4(y[0] * r, y[1 % V] * r, y[2 % V] * r, y[3 % V] * r));
+    else st1(dst, y[0] * r);
+  }
+  const int np = a.dk_p - a.dim;
+  for (int j = tid; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
 }
 
 struct GqaGather {
@@ -146,13 +276,19 @@ struct GqaAttend {
   const int* pos;
   const int* ctx;           // tokens of the sequence; 0: padding sequence
   KeyMask mask;
-  float scale, out_scale;
+  float scale, softcap;
+  ScoreScale score;         // the same for base-2 exponents
+  float out_scale;
+  const float* gate;        // fp32 [M][ldg] factor per row and head, or null
+  int ldg;
   void* o;                  // T [M, ldo], heads of vp; padding columns zero
   int ldo, vp;
   float* ws;                // [M][H][splits][dv_p + 2]
   int splits;
   int H, Hkv, dk_p, vdim, dv_p;
   int* status;
+
+  __device__ __forceinline__ float factor(int m, int h) const { return gate ? out_scale * gate[static_cast<size_t>(m) * ldg + h] : out_scale; }
 };
 
 constexpr int GD_KT = 32;   // keys per warp tile
@@ -202,7 +338,6 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   __nv_bfloat16 *wK = sKV + warp * WARP_ELEMS, *wV = wK + GD_KT * LK;
-  const float scale_log2 = a.scale * 1.4426950408889634f;
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + hk * a.dk_p;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + a.Hkv * a.dk_p + hk * a.dv_p;
 
@@ -257,7 +392,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           float& x = s[i][2 * e + j];
-          x = k0 + i * 8 + 2 * t + j < len ? x * scale_log2 : -INFINITY;
+          x = k0 + i * 8 + 2 * t + j < len ? a.score(x) : -INFINITY;
           mn = fmaxf(mn, x);
         }
       mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
@@ -319,7 +454,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
     }
     if (a.splits == 1) {
       __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.o) + static_cast<size_t>(m) * a.ldo + (h0 + r) * a.vp;
-      out[d] = __float2bfloat16(ls > 0.f ? o / ls * a.out_scale : 0.f);
+      out[d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h0 + r) : 0.f);
     } else {
       float* w = a.ws + ((static_cast<size_t>(m) * a.H + h0 + r) * a.splits + split) * (a.vp + 2);
       w[d] = o;
@@ -347,7 +482,7 @@ __global__ void __launch_bounds__(128) gqa_merge_kernel(const GqaAttend a) {
         ls += w[a.vp + 1] * sc;
         o += w[d] * sc;
       }
-    reinterpret_cast<__nv_bfloat16*>(a.o)[static_cast<size_t>(m) * a.ldo + h * a.vp + d] = __float2bfloat16(ls > 0.f ? o / ls * a.out_scale : 0.f);
+    reinterpret_cast<__nv_bfloat16*>(a.o)[static_cast<size_t>(m) * a.ldo + h * a.vp + d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h) : 0.f);
   }
 }
 
@@ -389,6 +524,7 @@ __global__ void __launch_bounds__(128) gqa_attend_kernel(const GqaAttend a) {
           d = fmaf(x.w, ga_q[i + 3], d);
         }
         s = d * a.scale;
+        if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       }
     }
     float tm = s;
@@ -417,7 +553,7 @@ __global__ void __launch_bounds__(128) gqa_attend_kernel(const GqaAttend a) {
       }
     }
   }
-  const float inv = sum > 0.f ? a.out_scale / sum : 0.f;
+  const float inv = sum > 0.f ? a.factor(m, h) / sum : 0.f;
   T* o = reinterpret_cast<T*>(a.o) + static_cast<size_t>(m) * a.ldo + h * a.vp;
 #pragma unroll
   for (int i = 0; i < OV; ++i) {
@@ -458,7 +594,8 @@ ARTB_EXPORT int artb_gqa_finish(int f32, void* p, int ldp, int kind, const float
   if (M <= 0) return 0;
   if (H <= 0 || Hkv <= 0 || H % Hkv || dk_p < dim || dv_p < vdim || ldc < Hkv * (dk_p + dv_p) || ldq < H * dk_p || ((dk_p | dv_p | ldc | ldq) & 3))
     return ERR_BAD_SHAPE;
-  const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status};
+  const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status,
+                    nullptr, nullptr, 0.f, nullptr, 1.f, 0, 0, nullptr, nullptr};
   const bool v4 = !((dim | vdim | ldp) & 3) && !(reinterpret_cast<uintptr_t>(p) & 15);
 #define ARTB_GF(T_, V_) return static_cast<int>(launch_kernel(gqa_finish_kernel<T_, V_>, dim3(M), dim3(256), 0, st, a))
   if (f32) {
@@ -468,6 +605,40 @@ ARTB_EXPORT int artb_gqa_finish(int f32, void* p, int ldp, int kind, const float
   if (v4) ARTB_GF(__nv_bfloat16, 4);
   ARTB_GF(__nv_bfloat16, 1);
 #undef ARTB_GF
+}
+
+// As artb_gqa_finish, with norms (wq, wk), the rotation of the first `rot` columns of every head of q and k, and gates; Hkv = 0: the
+// projection holds q (and gate) columns alone and the cache is not touched.
+ARTB_EXPORT int artb_gqa_finish_norm(int f32, void* p, int ldp, int kind, const float* bias, const int* slot, void* cache, int ldc,
+                                     long num_slots, void* q, int ldq, int M, int H, int Hkv, int dim, int dk_p, int vdim, int dv_p,
+                                     const float* wq, const float* wk, float eps, const double* freq, float rot_scale, int rot, int next,
+                                     const int* pos, float* gate, int* status, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if (H <= 0 || Hkv < 0 || (Hkv && H % Hkv) || dim <= 0 || vdim <= 0 || dk_p < dim || dv_p < vdim || (Hkv && ldc < Hkv * (dk_p + dv_p)) ||
+      ldq < H * dk_p || ((dk_p | dv_p | ldc | ldq) & 3) || (rot & 1) || rot < 0 || rot > dim || (rot && (!freq || !pos)) ||
+      ldp < H * dim + Hkv * (dim + vdim) + (gate ? H : 0))
+    return ERR_BAD_SHAPE;
+  const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status,
+                    wq, wk, eps, freq, rot_scale, rot, next, pos, gate};
+  const size_t smem = (static_cast<size_t>((H + Hkv) * dim + 3) / 4 * 4 + rot) * 4;
+  if (smem > 224 * 1024) return ERR_TOO_LARGE;
+  const bool v4 = !((dim | vdim | ldp) & 3) && !(rot & 7) && !(reinterpret_cast<uintptr_t>(p) & 15);
+#define ARTB_GN(T_, V_)                                                                                                        \
+  do {                                                                                                                         \
+    if (smem > 48 * 1024) {                                                                                                    \
+      const cudaError_t e = cudaFuncSetAttribute(gqa_finish_norm_kernel<T_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
+                                                 static_cast<int>(smem));                                                      \
+      if (e != cudaSuccess) return static_cast<int>(e);                                                                        \
+    }                                                                                                                          \
+    return static_cast<int>(launch_kernel(gqa_finish_norm_kernel<T_, V_>, dim3(M), dim3(256), smem, st, a));                   \
+  } while (0)
+  if (f32) {
+    if (v4) ARTB_GN(float, 4);
+    ARTB_GN(float, 1);
+  }
+  if (v4) ARTB_GN(__nv_bfloat16, 4);
+  ARTB_GN(__nv_bfloat16, 1);
+#undef ARTB_GN
 }
 
 // k [n_keys, kcols] and vt [vcols, n_keys] of the gathered rows (see artb_latent_gather); kcols and vcols multiples of 64,
@@ -490,11 +661,12 @@ ARTB_EXPORT int artb_gqa_gather(const void* cache, int ldc, const int* block_tab
 // Rows 0 .. M - 1, each its own query; bf16, dk_p and dv_p multiples of 8 up to 256.  splits > 1: ws fp32 [M * H * splits * (vp + 2)].
 ARTB_EXPORT int artb_gqa_decode(const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
                                 int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
-                                int chunk, float scale, float out_scale, void* o, int ldo, int vp, float* ws, int splits, int M, int H,
+                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp,
+                                float* ws, int splits, int M, int H,
                                 int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
-  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale,
-                    out_scale, o, ldo, vp, ws, splits, H, Hkv, dk_p, vdim, dv_p, status};
+  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale, softcap,
+                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, o, ldo, vp, ws, splits, H, Hkv, dk_p, vdim, dv_p, status};
   if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc | ldq) & 7) || splits < 1 || splits > 65535 || (splits > 1 && !ws)) return ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return ERR_BAD_ALIGN;
 #define ARTB_GD(K_)                                                   \
@@ -513,11 +685,11 @@ ARTB_EXPORT int artb_gqa_decode(const void* q, int ldq, const void* cache, int l
 
 ARTB_EXPORT int artb_gqa_attend(int f32, const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
                                 int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
-                                int chunk, float scale, float out_scale, void* o, int ldo, int vp, int M, int H, int Hkv, int dk_p,
-                                int vdim, int dv_p, int* status, cudaStream_t st) {
+                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp,
+                                int M, int H, int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
-  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale,
-                    out_scale, o, ldo, vp, nullptr, 1, H, Hkv, dk_p, vdim, dv_p, status};
+  const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale, softcap,
+                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, o, ldo, vp, nullptr, 1, H, Hkv, dk_p, vdim, dv_p, status};
   if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc) & 3) || vp > 1024 || dk_p > 8192) return ERR_BAD_SHAPE;
   const size_t smem = static_cast<size_t>(dk_p) * 4;
   return static_cast<int>(f32 ? launch_kernel(gqa_attend_kernel<float>, dim3(M, H), dim3(128), smem, st, a)

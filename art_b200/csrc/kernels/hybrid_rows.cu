@@ -3,13 +3,15 @@
 //   residual_step      the fp32 residual stream across a sublayer boundary, one pass:
 //                        x = x + mult * RMSNorm(y) w_post          (or x = RMSNorm(table[token]) w_post at the input)
 //                        without w_post: x = x + mult * y          (or x = mult * table[token] + position vector)
-//                        y may have a bias and the weighted rows of a token's experts added to it
+//                        y may have a factor per row, a bias and the weighted rows of a token's experts (or of the
+//                        sublayer's input, for experts that are the identity) added to it
 //                        depth average: x <- sum_j weight[j] X_j over the results X_j of all layers so far
-//                        h = RMSNorm(x) w_next                     (operand of the next matrix product)
+//                        h = RMSNorm(x) w_next, or x               (operand of the next matrix product)
 //   norm_shift_mix     h = RMSNorm(x) w; the inputs h + (h' - h) mu_s of a token-shifted mixer, h' being the h of the
 //                      token before (from the sequence's state at the start of a portion)
 //   poly_norm          a N(z) + b N(z^2) + c N(z^3) + e, N(v) = v / rms(v)
 //   gated_act          act(gate) * up of a gate|up projection, gate and up columns interleaved in blocks of 16
+//   plain_act          act(z)
 //   split_tanh         tanh(z) as a bf16 pair (high part, remainder), so that a product with it loses no 16-bit digits
 //   head_norm          per-head RMSNorm of a mixer's fp32 output, with an optional silu or sigmoid gate
 //   row_norm           the same over a whole row of heads
@@ -43,34 +45,28 @@ struct ResidualArgs {
   int ldx;
   const float* w_post;     // fp32 [dp], or null: y is not normalised
   float mult;
+  const float* y_gate;     // fp32 [rows] factor of y (before the bias), or null
   const float* y_bias;     // fp32 [dp] added to y, or null
   const void* ex;          // T [.., ldex] rows of experts: y += sum_s ex_w[row, s] * ex[ex_pos[row, s]], or null
   int ldex, ex_k;
-  const int* ex_pos;
+  const int* ex_pos;       // < 0: the identity, row `row` of idn
   const float* ex_w;
   long ex_rows;
+  void* idn;               // [rows, ldidn] of idn_kind, or null; may alias x_in, x_out or h
+  int ldidn, idn_kind;
   const double* freq;      // sinusoidal position vector added at the input: angle of column pair i is pos * freq[i]
   const int* pos;
   float* hist;             // fp32 [.., rows, ldx] results of the layers, or null
   long hist_stride;
   int hist_n;              // earlier results 0 .. hist_n - 1 are in hist; this one is stored as hist_n
   const float* avg;        // fp32 [hist_n + 1], or null: store without averaging
-  const float* w_next;     // fp32 [dp], or null
-  void* h;                 // T [rows, ldh]
+  const float* w_next;     // fp32 [dp], or null: h is x itself
+  void* h;                 // T [rows, ldh], or null
   int ldh;
   int d, dp;
   float eps;
   int* status;
 };
-
-// sine and cosine of pos * freq; the angle is reduced in double so that far positions lose nothing
-__device__ __forceinline__ float2 position_pair(int pos, double freq) {
-  constexpr double TWO_PI = 6.283185307179586476925;
-  const double ang = pos * freq;
-  float2 r;
-  sincosf(static_cast<float>(ang - rint(ang / TWO_PI) * TWO_PI), &r.x, &r.y);
-  return r;
-}
 
 template <typename T, int MAXV>
 __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a) {
@@ -92,6 +88,10 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
     if (v < nv) {
       if (a.tokens) y[i] = ld4(reinterpret_cast<const T*>(a.table) + static_cast<size_t>(tok) * a.ldt + v * 4);
       else if (a.y) y[i] = take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, a.y_kind);
+      if (a.y_gate) {
+        const float g = __ldg(a.y_gate + row);
+        y[i] = make_float4(y[i].x * g, y[i].y * g, y[i].z * g, y[i].w * g);
+      }
       if (a.y_bias) {
         const float4 b = ld4(a.y_bias + v * 4);
         y[i] = make_float4(y[i].x + b.x, y[i].y + b.y, y[i].z + b.z, y[i].w + b.w);
@@ -102,13 +102,14 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
     for (int s = 0; s < a.ex_k; ++s) {
       const int er = a.ex_pos[static_cast<size_t>(row) * a.ex_k + s];
       const float ew = a.ex_w[static_cast<size_t>(row) * a.ex_k + s];
-      if (!index_ok(er, a.ex_rows, a.status)) continue;
-      const T* ep = reinterpret_cast<const T*>(a.ex) + static_cast<size_t>(er) * a.ldex;
+      const bool self = er < 0 && a.idn;                    // uniform for the CTA
+      if (!self && !index_ok(er, a.ex_rows, a.status)) continue;
+      const T* ep = reinterpret_cast<const T*>(a.ex) + static_cast<size_t>(self ? 0 : er) * a.ldex;
 #pragma unroll
       for (int i = 0; i < MAXV; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
         if (v < nv) {
-          const float4 e = ld4(ep + v * 4);
+          const float4 e = self ? take4(a.idn, static_cast<size_t>(row) * a.ldidn + v * 4, a.idn_kind) : ld4(ep + v * 4);
           y[i] = make_float4(fmaf(ew, e.x, y[i].x), fmaf(ew, e.y, y[i].y), fmaf(ew, e.z, y[i].z), fmaf(ew, e.w, y[i].w));
         }
       }
@@ -169,10 +170,18 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
       ss += sq4(x);
     }
   }
-  if (!a.w_next) return;       // uniform for the grid
+  if (!a.h) return;            // uniform for the grid
+  T* h = reinterpret_cast<T*>(a.h) + static_cast<size_t>(row) * a.ldh;
+  if (!a.w_next) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nv) st4(h + v * 4, y[i]);
+    }
+    return;
+  }
   ss = cta_sum(ss, red);
   const float r2 = 1.f / sqrtf(ss / a.d + a.eps);
-  T* h = reinterpret_cast<T*>(a.h) + static_cast<size_t>(row) * a.ldh;
 #pragma unroll
   for (int i = 0; i < MAXV; ++i) {
     const int v = threadIdx.x + i * blockDim.x;
@@ -450,6 +459,25 @@ __global__ void __launch_bounds__(256) gated_act_kernel(void* z, int ldz, int ki
   put8(out + static_cast<size_t>(m) * ldo + c, x);
 }
 
+// z [M, np] -> out [M, np] = act(z).  Eight columns a thread.
+template <typename T>
+__global__ void __launch_bounds__(256) plain_act_kernel(void* z, int ldz, int kind, T* out, int ldo, long units, int nv, int act) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long u = blockIdx.x * 256L + threadIdx.x;
+  if (u >= units) return;
+  const long m = u / nv;
+  const int c = static_cast<int>(u - m * nv) * 8;
+  float x[8];
+  take8(z, static_cast<size_t>(m) * ldz + c, kind, x);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const float p = fmaxf(x[i], 0.f);
+    x[i] = act == ACT_RELU2 ? p * p : act == ACT_RELU ? p : silu_f(x[i]);
+  }
+  put8(out + static_cast<size_t>(m) * ldo + c, x);
+}
+
 template <typename T, int MAXV>
 __global__ void __launch_bounds__(256)
 gather_norm_kernel(const float* __restrict__ x, int ldx, const int64_t* __restrict__ rows, const float* __restrict__ w, T* h,
@@ -499,15 +527,15 @@ using namespace artb;
 // f32: operands (table, h) are fp32 instead of bf16.  See ResidualArgs; y_kind is a RowKind.
 ARTB_EXPORT int artb_residual_step(int f32, const int64_t* tokens, const void* table, int ldt, long vocab, void* y, int ldy,
                                    int y_kind, const float* x_in, float* x_out, int ldx, const float* w_post, float mult,
-                                   const float* y_bias, const void* ex, int ldex, int ex_k, const int* ex_pos,
-                                   const float* ex_w, long ex_rows, const double* freq, const int* pos, float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
+                                   const float* y_gate, const float* y_bias, const void* ex, int ldex, int ex_k, const int* ex_pos,
+                                   const float* ex_w, long ex_rows, void* idn, int ldidn, int idn_kind, const double* freq, const int* pos, float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
                                    int ldh, int M, int d, int dp, float eps, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
-  if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || (ldex & 3) || !x_out) return ERR_BAD_SHAPE;
+  if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || (ldex & 3) || (ldidn & 3) || !x_out || (w_next && !h)) return ERR_BAD_SHAPE;
   if (!tokens && ((!y && !ex) || !x_in)) return ERR_BAD_SHAPE;
-  if ((ex && (ex_k <= 0 || !ex_pos || !ex_w)) || (freq && (!tokens || !pos))) return ERR_BAD_SHAPE;
-  const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, y_bias, ex, ldex, ex_k, ex_pos, ex_w,
-                       ex_rows, freq, pos, hist, hist_stride, hist_n, avg, w_next, h, ldh, d, dp, eps, status};
+  if ((ex && (ex_k <= 0 || !ex_pos || !ex_w)) || (idn && (!ex || idn_kind == ROW_F32_TAKE)) || (freq && (!tokens || !pos))) return ERR_BAD_SHAPE;
+  const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, y_gate, y_bias, ex, ldex, ex_k, ex_pos, ex_w,
+                       ex_rows, idn, ldidn, idn_kind, freq, pos, hist, hist_stride, hist_n, avg, w_next, h, ldh, d, dp, eps, status};
   const int th = row_threads(dp);
   cudaError_t e = cudaSuccess;
 #define ARTB_RS(V)                                                                                                     \
@@ -572,6 +600,18 @@ ARTB_EXPORT int artb_gated_act(int f32, void* z, int ldz, int kind, void* out, i
   return static_cast<int>(f32 ? launch_kernel(gated_act_kernel<float>, grid, dim3(256), 0, st, z, ldz, kind, reinterpret_cast<float*>(out),
                                               ldo, units, np >> 3, act)
                               : launch_kernel(gated_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, z, ldz, kind,
+                                              reinterpret_cast<__nv_bfloat16*>(out), ldo, units, np >> 3, act));
+}
+
+// z [M, np] of `kind` -> out [M, np] = act(z) (np a multiple of 8)
+ARTB_EXPORT int artb_plain_act(int f32, void* z, int ldz, int kind, void* out, int ldo, int M, int np, int act, cudaStream_t st) {
+  if (M <= 0) return 0;
+  if ((np & 7) || (ldz & 7) || (ldo & 7) || (act != ACT_SILU && act != ACT_RELU && act != ACT_RELU2)) return ERR_BAD_SHAPE;
+  const long units = static_cast<long>(M) * (np >> 3);
+  const dim3 grid(static_cast<unsigned>((units + 255) / 256));
+  return static_cast<int>(f32 ? launch_kernel(plain_act_kernel<float>, grid, dim3(256), 0, st, z, ldz, kind, reinterpret_cast<float*>(out),
+                                              ldo, units, np >> 3, act)
+                              : launch_kernel(plain_act_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, z, ldz, kind,
                                               reinterpret_cast<__nv_bfloat16*>(out), ldo, units, np >> 3, act));
 }
 

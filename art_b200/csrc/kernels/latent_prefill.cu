@@ -15,6 +15,7 @@
 #include "host_utils.h"
 #include "key_mask.cuh"
 #include "mma_tile.cuh"
+#include "softcap.cuh"
 
 namespace artb {
 
@@ -60,7 +61,10 @@ struct LatentPrefill {
   const int* key_off;            // per sequence: first gathered row
   const int* key_pos0;           // per sequence: position of that row
   KeyMask mask;
-  float scale_log2, out_scale;   // out_scale multiplies the result
+  ScoreScale score;
+  float out_scale;               // multiplies the result
+  const float* gate;             // [rows][ldg] factor per row and head, or null
+  int ldg;
   __nv_bfloat16* o;              // [rows][ldo]: heads of vp columns
   int ldo, vp, vdim;
   int H, G, dk, dv, rot_p;       // G heads share a key head; dk, dv, rot_p multiples of 16
@@ -168,7 +172,7 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
             for (int k = 0; k < 2; ++k) {
               float& x = s[i][j][2 * e + k];
               const int kp = k0 + j * 8 + 2 * t + k;
-              x *= a.scale_log2;
+              x = a.score(x);
               if (!inside && (kp > p || kp < first)) x = -INFINITY;
               mx = fmaxf(mx, x);
             }
@@ -217,7 +221,8 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int r = w0 + i * 16 + g + 8 * e;
       if (r >= nrow) continue;
-      const float inv = l > 0.f ? a.out_scale / l : 0.f;
+      float inv = l > 0.f ? a.out_scale / l : 0.f;
+      if (a.gate) inv *= a.gate[static_cast<size_t>(r0 + r) * a.ldg + h];
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp;
 #pragma unroll
       for (int n = 0; n < DV / 8; ++n) {
@@ -266,7 +271,7 @@ ARTB_EXPORT int artb_latent_gather(const void* cache, int ldc, const int* block_
 
 ARTB_EXPORT int artb_latent_prefill(const void* q, int ldq, const void* kv, int ldkv, const void* c, int ldc, int rank_p, const int* tile_seq,
                                     const int* tile_row, int n_tiles, const int* row_end, const int* row_pos0, const int* key_off,
-                                    const int* key_pos0, int window, int chunk, float scale, float out_scale, void* o, int ldo, int vp, int vdim, int H, int G,
+                                    const int* key_pos0, int window, int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp, int vdim, int H, int G,
                                     int dk, int dv, int rot_p, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || (dk & 15) || (dv & 15) || (rot_p & 15) || (ldq & 7) || (ldkv & 7) || (ldc & 7) || (rank_p & 7) || (ldo & 1) || (vp & 1) ||
@@ -274,7 +279,7 @@ ARTB_EXPORT int artb_latent_prefill(const void* q, int ldq, const void* kv, int 
     return ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(c)) & 15) return ERR_BAD_ALIGN;
   const LatentPrefill a{(const bf16*)q, ldq, (const bf16*)kv, ldkv, (const bf16*)c, ldc, rank_p, tile_seq, tile_row, row_end, row_pos0,
-                        key_off, key_pos0, {window, chunk}, scale * 1.4426950408889634f, out_scale, (bf16*)o, ldo, vp, vdim, H, G, dk, dv, rot_p};
+                        key_off, key_pos0, {window, chunk}, ScoreScale::of(scale, softcap), out_scale, gate, ldg, (bf16*)o, ldo, vp, vdim, H, G, dk, dv, rot_p};
   if (dv <= 32) return launch_latent_prefill<32>(a, n_tiles, st);
   if (dv <= 64) return launch_latent_prefill<64>(a, n_tiles, st);
   if (dv <= 96) return launch_latent_prefill<96>(a, n_tiles, st);

@@ -19,6 +19,7 @@
 #include "host_utils.h"
 #include "key_mask.cuh"
 #include "ptx_sm100.cuh"
+#include "softcap.cuh"
 
 namespace artb {
 
@@ -34,7 +35,10 @@ struct LatentTc {
   const int* key_off;
   const int* key_pos0;
   KeyMask mask;
-  float scale_log2, out_scale;
+  ScoreScale score;
+  float out_scale;
+  const float* gate;      // [rows][ldg] factor per row and head, or null
+  int ldg;
   __nv_bfloat16* o;
   int ldo, vp;
   int rank_p, dk, rot_p, G;
@@ -292,6 +296,10 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       tc_fence_before_sync();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_empty[s]);
+      if (a.score.capped()) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) x[j] = a.score.squash(x[j]);
+      }
       if (!inside) {
         const int hi = qpos - (k0 + hf * 64), lo = first - (k0 + hf * 64);      // visible: lo <= j <= hi
 #pragma unroll
@@ -301,7 +309,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
       for (int j = 0; j < 64; ++j) mx4[j & 3] = fmaxf(mx4[j & 3], x[j]);
-      const float mx_mine = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * a.scale_log2;   // scale > 0
+      const float mx_mine = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * a.score.scale_log2;   // scale > 0
       float mx_other;
       if (!swap_with_partner(mx_mine, mx_other)) {
         fail(ST_TIMEOUT_PEER);
@@ -323,7 +331,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
         float pe[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-          pe[e] = lt_ex2(fmaf(x[8 * i + e], a.scale_log2, -ms));
+          pe[e] = lt_ex2(fmaf(x[8 * i + e], a.score.scale_log2, -ms));
           rs4[e & 3] += pe[e];
         }
         uint4 w;
@@ -348,7 +356,8 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     if (!dead && !swap_with_partner(l, l_other)) fail(ST_TIMEOUT_PEER);
     if (!dead && r < nrow) {
       const float lt = l + l_other;
-      const float inv = lt > 0.f ? a.out_scale / lt : 0.f;
+      float inv = lt > 0.f ? a.out_scale / lt : 0.f;
+      if (a.gate) inv *= a.gate[static_cast<size_t>(r0 + r) * a.ldg + h];
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp + hf * OC;
 #pragma unroll
       for (int c = 0; c < OC; c += 8) {
@@ -404,7 +413,7 @@ using namespace artb;
 ARTB_EXPORT int artb_latent_prefill_tc(const void* q, int ldq, int rows, const void* k, int ldk, const void* c, int ldc, int rank_p,
                                        const void* vt, int ldvt, int n_keys, const int* tile_seq, const int* tile_row, int n_tiles,
                                        const int* row_end, const int* row_pos0, const int* key_off, const int* key_pos0, int window,
-                                       int chunk, float scale, float out_scale, void* o, int ldo, int vp, int H, int G, int dk, int dv, int rot_p,
+                                       int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp, int H, int G, int dk, int dv, int rot_p,
                                        int* status, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (H <= 0 || H > 65535 || G <= 0 || H % G || dk <= 0 || (dk & 63) || (rot_p & 63) || dk + rot_p > 192 || (dv != 64 && dv != 128) || (n_keys & 7) || (ldo & 7) ||
@@ -417,7 +426,7 @@ ARTB_EXPORT int artb_latent_prefill_tc(const void* q, int ldq, int rows, const v
   if ((e = make_tmap_bf16_2d(&tK, k, n_keys, static_cast<uint64_t>(H / G) * dk, ldk, LT_B, 64))) return e;
   if ((e = make_tmap_bf16_2d(&tC, c, n_keys, ldc, ldc, LT_B, 64))) return e;
   if ((e = make_tmap_bf16_2d(&tV, vt, static_cast<uint64_t>(H / G) * dv, n_keys, ldvt, dv, 64))) return e;
-  const LatentTc a{tile_seq, tile_row, row_end, row_pos0, key_off, key_pos0, {window, chunk}, scale * 1.4426950408889634f, out_scale,
+  const LatentTc a{tile_seq, tile_row, row_end, row_pos0, key_off, key_pos0, {window, chunk}, ScoreScale::of(scale, softcap), out_scale, gate, ldg,
                    reinterpret_cast<__nv_bfloat16*>(o), ldo, vp, rank_p, dk, rot_p, G, status};
   const int nq = (dk + rot_p) / 64;
   if (dv == 128) {

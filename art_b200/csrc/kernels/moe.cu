@@ -3,7 +3,7 @@
 //
 //   router   logits[M, E] -> top-k expert ids and weights per token (+ per-expert counts)
 //   plan     counts -> segment offsets padded to 128 rows, tile -> expert map for the grouped GEMM
-//   assign   (token, slot) -> row position inside its expert's segment
+//   assign   (token, slot) -> row position inside its expert's segment, -1 for outputs without rows (identity experts)
 //   gather   xp[pos] = scale * x[token]                       (rows sorted by expert)
 //   combine  out[token] = residual[token] + sum_slot w * yp[pos(token, slot)]   (fixed order)
 //   router_bwd  d(top-k weights) -> d(logits)
@@ -34,9 +34,13 @@ __device__ __forceinline__ float warp_pick(const float (&a)[MOE_MAX_E_PER_LANE],
 }
 
 // One warp per token.  The k largest logits (+ bias) are chosen, the lower index on a tie; weights are the softmax over all
-// experts or, with `norm`, over the chosen ones.  Logits of kind ROW_F32_TAKE are cleared once read.
-__global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, const float* __restrict__ bias, int M, int E, int k,
-                                  int norm, int* __restrict__ topi, float* __restrict__ topw, int* __restrict__ counts) {
+// experts or, with `norm`, over the chosen ones.  With `correction` the softmax over all outputs is taken first, the largest
+// of its entries + correction are chosen, and with `norm` their weights are divided by their sum (+ 1e-20).  Outputs from
+// `real` on have no rows of their own (counts end there).  `gate`: the sigmoid of the column behind the outputs.  Logits of kind
+// ROW_F32_TAKE are cleared once read.
+__global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, const float* __restrict__ bias,
+                                  const float* __restrict__ correction, int M, int E, int real, int k, int norm, int* __restrict__ topi,
+                                  float* __restrict__ topw, int* __restrict__ counts, float* __restrict__ gate) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   pdl_launch_dependents();
@@ -56,14 +60,26 @@ __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, 
   }
 #pragma unroll
   for (int o = 16; o; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+  if (gate && lane == 0) gate[warp] = logistic_f(take1(row, E, kind));
   float sum = 0.f;
-  if (!norm) {
+  if (!norm || correction) {
 #pragma unroll
     for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j)
       if (j * 32 + lane < E) sum += expf(v[j] - mx);
 #pragma unroll
     for (int o = 16; o; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   }
+  float p[MOE_MAX_E_PER_LANE];                   // weights before the division, v: what the choice goes by
+#pragma unroll
+  for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j) {
+    const int e = j * 32 + lane;
+    p[j] = e < E ? expf(v[j] - mx) : 0.f;
+    if (correction && e < E) {
+      p[j] /= sum;
+      v[j] = p[j] + correction[e];
+    }
+  }
+  if (correction) sum = norm ? 1e-20f : 1.f;
   float wsel = 0.f;
   int isel = 0;
   uint32_t taken = 0;                            // entries of this lane that are chosen already
@@ -89,17 +105,17 @@ __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, 
     }
     if (bi >= E) bi = 0;                         // logits that are no numbers: stay inside the experts
     if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
-    const float p = expf(best - mx);
-    if (norm) sum += p;
+    const float pb = warp_pick(p, bi);
+    if (norm) sum += pb;
     if (lane == s) {
-      wsel = p;
+      wsel = pb;
       isel = bi;
     }
   }
   if (lane < k) {
     topi[static_cast<size_t>(warp) * k + lane] = isel;
     topw[static_cast<size_t>(warp) * k + lane] = wsel / sum;
-    atomicAdd(counts + isel, 1);
+    if (isel < real) atomicAdd(counts + isel, 1);
   }
 }
 
@@ -143,11 +159,15 @@ __global__ void moe_fill_kernel(int* __restrict__ row_token, float* __restrict__
 }
 
 __global__ void moe_assign_kernel(const int* __restrict__ topi, const float* __restrict__ topw, long n /* M*k */, int k,
-                                  const int* __restrict__ seg_off, int* __restrict__ cursor, int* __restrict__ pos,
+                                  const int* __restrict__ seg_off, int E, int* __restrict__ cursor, int* __restrict__ pos,
                                   int* __restrict__ row_token, float* __restrict__ row_w) {
   const long i = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x;
   if (i >= n) return;
   const int e = topi[i];
+  if (e >= E) {                                  // an output without rows
+    pos[i] = -1;
+    return;
+  }
   const int p = seg_off[e] + atomicAdd(cursor + e, 1);
   pos[i] = p;
   row_token[p] = static_cast<int>(i / k);
@@ -360,14 +380,15 @@ __global__ void moe_router_bwd_kernel(const float* __restrict__ logits, int ld, 
 
 using namespace artb;
 
-// logits fp32 [M, E] (E <= 256, k <= 16) of kind ROW_F32 or ROW_F32_TAKE; bias fp32 [E] or null; counts int32 [E] must be
-// zero on entry.
-ARTB_EXPORT int artb_moe_router(float* logits, int ld, int kind, const float* bias, int M, int E, int k, int norm, int* topi,
-                                float* topw, int* counts, cudaStream_t st) {
+// logits fp32 [M, E] (E <= 256, k <= 16) of kind ROW_F32 or ROW_F32_TAKE; bias, correction fp32 [E] or null; real <= E outputs
+// have rows; counts int32 [real] must be zero on entry; gate fp32 [M] (logits then have E + 1 columns) or null.
+ARTB_EXPORT int artb_moe_router(float* logits, int ld, int kind, const float* bias, const float* correction, int M, int E, int real, int k,
+                                int norm, int* topi, float* topw, int* counts, float* gate, cudaStream_t st) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E || kind == ROW_BF16) return ERR_BAD_SHAPE;
+  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E || real <= 0 || real > E || ld < E + (gate ? 1 : 0) || kind == ROW_BF16)
+    return ERR_BAD_SHAPE;
   const int threads = 256, warps = threads / 32;
-  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, kind, bias, M, E, k, norm, topi, topw, counts);
+  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, kind, bias, correction, M, E, real, k, norm, topi, topw, counts, gate);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -383,7 +404,7 @@ ARTB_EXPORT int artb_moe_plan(const int* counts, int E, const int* topi, const f
   moe_fill_kernel<<<static_cast<unsigned>((rows + 255) / 256), 256, 0, st>>>(row_token, row_w, rows);
   const long n = M * k;
   if (n > 0)
-    moe_assign_kernel<<<static_cast<unsigned>((n + 255) / 256), 256, 0, st>>>(topi, topw, n, k, seg_off, cursor, pos,
+    moe_assign_kernel<<<static_cast<unsigned>((n + 255) / 256), 256, 0, st>>>(topi, topw, n, k, seg_off, E, cursor, pos,
                                                                               row_token, row_w);
   return static_cast<int>(cudaGetLastError());
 }

@@ -5,7 +5,7 @@ Two parts, random weights throughout:
 * ``engine_rows``: prefill and decode tokens/s of whole models through :class:`~art_b200.engine.engine.Engine`, a hybrid
   preset and a twin of the same width, depth and feed-forward parameters per layer, no adapters: a dense Llama-style model,
   or a Qwen3-style mixture of experts where the preset has experts.
-* ``kernel_rows``, ``naselorn_kernel_rows``: every kernel of the hybrid path at the layer sizes of a model, timed alone with CUDA events (L2 flushed
+* ``kernel_rows``, ``naselorn_kernel_rows``, ``gaborax_kernel_rows``: every kernel of the hybrid path at the layer sizes of a model, timed alone with CUDA events (L2 flushed
   between calls), with its algorithmic bytes and FLOPs and the fraction of its roofline (the slower of bytes at the
   measured copy bandwidth and FLOPs at the measured tensor or nominal fp32 rate), and the like kernels of the dense model
   or of the other design.
@@ -34,7 +34,8 @@ def peaks() -> tuple[float, float]:
 
 def twin(cfg):
     """A Llama-style dense model of the same width and depth whose feed-forward (three matrices) has the hybrid's
-    parameters (two matrices), or a Qwen3-style mixture of experts whose experts stand for the hybrid's shared one, too."""
+    parameters (two matrices), or a Qwen3-style mixture of experts whose experts stand for the hybrid's shared one, too
+    (experts of two matrices count as gated ones of two thirds the width)."""
     from ..models.config import ModelConfig
 
     d = cfg.hidden_size
@@ -43,7 +44,7 @@ def twin(cfg):
         extra = moe.shared_ff // moe.expert_ff
         return ModelConfig(name=f"moe-{cfg.name}", family="qwen3_moe", vocab_size=cfg.vocab_size, hidden_size=d, num_layers=cfg.num_layers,
                            num_heads=d // 128, num_kv_heads=max(1, d // 128 // 4), head_dim=128, intermediate_size=0, qkv_bias=False, qk_norm=True,
-                           num_experts=moe.experts + extra, num_experts_per_tok=moe.top + extra, moe_intermediate_size=moe.expert_ff)
+                           num_experts=moe.experts + extra, num_experts_per_tok=moe.top + extra, moe_intermediate_size=moe.expert_ff if moe.glu else (moe.expert_ff * 2 // 3 + 15) // 16 * 16)
     ff = max(s.ff for s in cfg.layers)
     return ModelConfig(name=f"dense-{cfg.name}", family="llama", vocab_size=cfg.vocab_size, hidden_size=d, num_layers=cfg.num_layers,
                        num_heads=d // 128, num_kv_heads=max(1, d // 128 // 4), head_dim=128, intermediate_size=(ff * 2 // 3 + 127) // 128 * 128,
@@ -356,6 +357,112 @@ def naselorn_kernel_rows(width: int = 4096, prefill: int = 8192, decode: int = 2
     return bench.rows
 
 
+def gaborax_kernel_rows(width: int = 4096, prefill: int = 8192, decode: int = 256, ctx: int = 2048, experts: int = 64, identity: int = 8,
+                        top: int = 8, expert_ff: int = 1536, shared_ff: int = 3072, softcap: float = 50.0) -> list[dict]:
+    """The kernels of Gaborax layers, each beside the like kernel of another design ("like: ...")."""
+    from ..ops import attention as attn_ops
+    from ..ops import hybrid as hy
+    from ..ops import moe, paged
+    from ..ops.gemm import gemm_tn
+
+    dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
+    bench = _Rows()
+    add = bench.add
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, generator=g) * sc).to(dt)      # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
+    d, H, hd, bs = width, width // 128, 128, 16
+    Hkv, G = H // 4, 4
+    freq = torch.tensor([5e5 ** (-2 * i / hd) for i in range(hd // 2)], dtype=torch.float64, device=dev)
+    for phase, M in (("decode", decode), ("prefill", prefill)):
+        one = phase == "decode"
+        n_seqs = M if one else M // 2048
+        row_seq = i32(list(range(M)) if one else [i // 2048 for i in range(M)])
+        c_len = i32([ctx] * n_seqs)
+        pos = i32([ctx - 1] * M if one else [i % 2048 for i in range(M)])
+        x, w, h, y = rnd(M, d, dt=f32), rnd(d, dt=f32), rnd(M, d), rnd(M, d)
+        add("residual_step, post-norm, stream as operand", phase, lambda: hy.residual_step(x, w, d, 1e-5, y=hy.as_out(y), x_in=x, h=h), M * d * 12)
+        add("like: residual_step with both norms", phase, lambda: hy.residual_step(x, w, d, 1e-5, y=hy.as_out(y), x_in=x, w_next=w, h=h), M * d * 12)
+        # attention
+        ld = Hkv * 2 * hd
+        nb = n_seqs * (ctx // bs)
+        cache = rnd(nb, bs, ld)
+        bt = torch.randperm(nb, device=dev, generator=g).to(torch.int32).view(n_seqs, ctx // bs)
+        n = (H + 2 * Hkv) * hd
+        qkvg, bias, wn = rnd(M, n + H), rnd(n, dt=f32), rnd(n, dt=f32)
+        q, slot = torch.empty(M, H * hd, dtype=bf, device=dev), i32([i % (nb * bs) for i in range(M)])
+        gate = torch.empty(M, H, dtype=f32, device=dev)
+        P = hy.as_out(qkvg)
+        for nxt, gt, b_ in ((False, gate, None), (True, None, bias)):
+            add("gqa_finish_norm, " + ("neighbours, biases" if nxt else "halves, gates"), phase, lambda: hy.gqa_finish_norm(
+                P, b_, slot, cache, q, H, Hkv, hd, hd, hd, wn, wn, 1e-5, hy.Rotation(hd, freq, 1.1, nxt), pos, gt), M * n * 4)
+        add("gqa_finish_norm, queries alone", phase, lambda: hy.gqa_finish_norm(P, None, slot, cache, q, H, 0, hd, hd, hd, wn, None, 1e-5, hy.Rotation(hd, freq), pos, gate),
+            M * H * hd * 4)
+        add("like: gqa_finish (no norm, no rotation)", phase, lambda: hy.gqa_finish(P, bias, slot, cache, q, H, Hkv, hd, hd, hd), M * n * 4)
+        ao = torch.empty(M, H * hd, dtype=bf, device=dev)
+        forms = (("gate", dict(gate=gate)), (f"softcap {softcap:.0f}", dict(softcap=softcap)))
+        if one:
+            sp = hy.gqa_decode_splits(M, Hkv, ctx)
+            b_, f_ = M * ctx * ld * 2 + M * H * hd * 4, 4.0 * M * H * ctx * hd
+            for name, kw in forms:
+                add(f"gqa_decode ctx {ctx}, {name}", phase, lambda: hy.gqa_decode(q, cache, bt, row_seq, pos, c_len, 0, 0, hd ** -0.5, 1.0, ao, M, H, Hkv, hd, hd, hd, sp,
+                                                                               **kw), b_, f_)
+            kc, vc = rnd(nb, bs, Hkv, hd), rnd(nb, bs, Hkv, hd)
+            add(f"like: paged_decode ctx {ctx}", phase, lambda: paged.paged_decode(q, kc, vc, bt, c_len, H, Hkv, hd, ao), b_, f_)
+            del kc, vc
+        else:
+            plan = hy.plan_prefill([(i, 0, 2048) for i in range(n_seqs)], 0, dev)
+            add("gqa_gather", phase, lambda: hy.gqa_gather(cache, bt, plan, Hkv, hd, hd), plan.n_keys * ld * 4)
+            add("like: latent_gather", phase, lambda: hy.latent_gather(cache, bt, plan), plan.n_keys * ld * 4)
+            k, vt = hy.gqa_gather(cache, bt, plan, Hkv, hd, hd)
+            pairs = n_seqs * 2048 * 2049 // 2
+            b_, f_ = (q.numel() + k.numel() + vt.numel() + ao.numel()) * 2, 4.0 * H * pairs * hd
+            for name, kw in (("plain", {}),) + forms:
+                add(f"latent_prefill_tc causal 2048, {name}", phase, lambda: hy.latent_prefill_tc(q, k, vt, k, plan, 0, hd ** -0.5, ao, H, hd, hd, 0, 0, hd, G=G, **kw), b_, f_)
+            c = hy.latent_gather(cache, bt, plan)
+            for name, kw in (("plain", {}), forms[1]):
+                add(f"latent_prefill (any sizes) causal 2048, {name}", phase, lambda: hy.latent_prefill(q, c, c, plan, 0, hd ** -0.5, ao, H, hd, hd, 0, 0, hd, G=G, **kw), b_, f_)
+            ids = torch.arange(n_seqs, dtype=torch.int32, device=dev).repeat_interleave(2048)
+            ap = attn_ops.make_plan(ids, ids, M, "native")
+            qkv = qkvg[:, :n].contiguous()
+            add("like: tree attention fwd, causal, 2048 tokens", phase, lambda: attn_ops.forward(qkv, H, Hkv, hd, ap, need_grad=False), b_, f_)
+            del qkv, k, vt, c
+        # feed-forward
+        a, Wu = torch.empty(M, shared_ff, dtype=bf, device=dev), rnd(shared_ff, d, sc=d ** -0.5)
+        wb, wf = (Wu.numel() + M * d + a.numel()) * 2, 2.0 * M * d * shared_ff
+        add("gemm_tn up, squared relu epilogue", phase, lambda: gemm_tn(h, Wu, out=a, relu2=True), wb, wf)
+        add("like: gemm_tn, same product", phase, lambda: gemm_tn(h, Wu, out=a), wb, wf)
+        z = rnd(M, shared_ff, dt=f32)
+        add("plain_act (split products)", phase, lambda: hy.plain_act(hy.Out(z, hy.KIND_TAKE), a, "relu2"), M * shared_ff * 10)
+        z2 = rnd(M, 2 * shared_ff, dt=f32)
+        add("like: gated_act", phase, lambda: hy.gated_act(hy.Out(z2, hy.KIND_TAKE), a, "silu"), M * shared_ff * 18)
+        del z, z2, a, Wu
+        outputs = experts + identity
+        logits, corr = rnd(M, outputs + 1, dt=f32), rnd(outputs, dt=f32, sc=1e-3)
+        add("moe.route by corrected scores", phase, lambda: moe.route(logits, top, True, correction=corr, identity=identity, gate=True), M * (outputs * 4 + top * 8))
+        add("like: moe.route by logits", phase, lambda: moe.route(logits[:, :experts], top, True, corr), M * (outputs * 4 + top * 8))
+        rp = moe.route(logits, top, True, correction=corr, identity=identity, gate=True)
+        real = int((rp.topi < experts).sum())
+        xp = moe.gather(h, rp)
+        add("moe.gather", phase, lambda: moe.gather(h, rp, out=xp), d * 2 * (M + real))
+        eu, ed = rnd(experts * expert_ff, d, sc=d ** -0.5), rnd(experts * d, expert_ff, sc=expert_ff ** -0.5)
+        ea, yp = torch.empty(rp.cap_rows, expert_ff, dtype=bf, device=dev), torch.empty(rp.cap_rows, d, dtype=bf, device=dev)
+        eb, ef = (eu.numel() + real * (d + expert_ff)) * 2, 2.0 * real * d * expert_ff
+        add("grouped_gemm up, squared relu epilogue", phase, lambda: moe.grouped_gemm(xp, eu, rp, expert_ff, out=ea, relu2=True), eb, ef)
+        eg = eu[:experts * (expert_ff // 32 * 32)]
+        sw = torch.empty(rp.cap_rows, expert_ff // 2, dtype=bf, device=dev)
+        add("like: grouped_gemm gate|up, silu epilogue, same product", phase, lambda: moe.grouped_gemm(xp, eg, rp, expert_ff, swiglu_out=sw, keep_preact=False),
+            (eu.numel() + real * (d + expert_ff // 2)) * 2, ef)
+        add("grouped_gemm down", phase, lambda: moe.grouped_gemm(ea, ed, rp, d, out=yp), eb, ef)
+        sub = hy.Sublayer(hy.as_out(y), rows=yp, pos=rp.pos, weight=rp.topw, gate=rp.gate, identity=hy.as_out(x))
+        add("residual_step with experts' rows, gate, identity", phase, lambda: hy.residual_step(x, w, d, 1e-5, sub=sub, x_in=x, h=h), M * d * 12 + real * d * 2)
+        plain = hy.Sublayer(hy.as_out(y), rows=yp, pos=rp.pos.clamp(min=0), weight=rp.topw)
+        add("like: residual_step with experts' rows", phase, lambda: hy.residual_step(x, None, d, 1e-5, sub=plain, x_in=x, w_next=w, h=h), M * d * (12 + 2 * top))
+        del eu, ed, ea, eg, sw, yp, xp, cache, qkvg, q, ao, P
+        torch.cuda.empty_cache()
+    return bench.rows
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--models", default="nikelix-1b,nikelix-7b")
@@ -371,7 +478,7 @@ def report(models: list[str], batches: list[int], layers: int, part: str = "both
     from ..ops import _lib
 
     if part != "engine":
-        for design, fn in (("nikelix", kernel_rows), ("naselorn", naselorn_kernel_rows)):
+        for design, fn in (("nikelix", kernel_rows), ("naselorn", naselorn_kernel_rows), ("gaborax", gaborax_kernel_rows)):
             if any(m.startswith(design) for m in models):
                 yield from ({"part": "kernel", "design": design, **r} for r in fn())
                 torch.cuda.empty_cache()

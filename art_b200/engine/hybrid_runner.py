@@ -9,9 +9,9 @@ form), longer portions gather what they see and run on prompt kernels (latent at
 A batch of single tokens (decoding) leaves its projections as split-K partial sums in fp32 workspaces, which the kernel
 that follows finishes and clears, as the engine's other models do.
 
-Every sublayer is ``norm -> mixer or feed-forward -> (norm ->) residual``; the step from one to the next (a mixture's weighted
-sum, bias, post-norm, residual multiplier, depth average, next input norm: what the design has of them) is one kernel over
-the fp32 residual stream (``ops.hybrid.residual_step``).  Mixers side by side share one input and one output product: their
+Every sublayer is ``(norm ->) mixer or feed-forward -> (norm ->) residual``; the step from one to the next (a mixture's weighted
+sum, bias, post-norm and factors, residual multiplier, depth average, next input norm: what the design has of them) is one
+kernel over the fp32 residual stream (``ops.hybrid.residual_step``).  Mixers side by side share one input and one output product: their
 factors scale what enters the latter.
 Operands of the matrix products are bf16; with ``dtype=torch.float32`` everything is fp32, products included, through the
 same layer code.
@@ -25,7 +25,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..models.hybrid import PART_NAMES, SHIFT_MIXES, HybridConfig, LayerSpec, check_weights
+from ..models.hybrid import PART_NAMES, SHIFT_MIXES, HybridConfig, LayerSpec, check_weights, rope_frequencies
 from ..ops import hybrid as hy
 from ..ops.hybrid import Out, Sublayer, as_out, pad
 from .runner import DeviceRunner, SeqView
@@ -50,6 +50,7 @@ class Ragged:
     n_abs: int = 0
     reach: int = 0              # upper bound of the tokens a short row may attend to
     plans: dict = field(default_factory=dict)
+    kept: dict = field(default_factory=dict)      # gathered keys and values that a later layer reads, too
 
     def plan(self, window: int, chunk: int = 0) -> hy.PrefillPlan:
         p = self.plans.get((window, chunk))
@@ -64,6 +65,21 @@ ABSORB_MAX = 16
 # Sizes the tensor-core kernels hold in shared memory and registers; beyond them the scalar absorbed form serves.
 LATENT_TC_MAX = 768         # cached row: latent + rotated part
 PREFILL_VALUE_MAX, PREFILL_KEY_MAX = 128, 320
+
+
+# Kernel sources of each mechanism (what a fresh checkout has to compile before it can run a model's layers)
+_GEMM = {"gemm_tcgen05", "gemm_tcgen05_2cta", "gemm_splitk", "gemm_f32"}
+_SCAN = {"linear_scan"}
+KERNEL_SOURCES = {
+    "latent_attention": {"latent_attn", "latent_decode", "latent_prefill", "latent_prefill_tc", "gemm_batched"},
+    "attention": {"gqa_attn", "latent_prefill", "latent_prefill_tc"}, "hgrn2": _SCAN, "wkv": _SCAN | {"gemm_batched"},
+    "lightning": _SCAN | {"lightning_prefill"}, "rglru": {"rglru", "gemm_batched"}, "moe": {"moe", "gemm_grouped", "lora_wgrad"}}
+
+
+def kernel_sources(cfg: HybridConfig) -> set[str]:
+    """The kernel sources that the layers of a model run on."""
+    kinds = {m.type for s in cfg.layers for m in s.mixers()} | {s.mlp for s in cfg.layers if s.has_mlp}
+    return _GEMM | {"hybrid_rows"} | {f for k in kinds for f in KERNEL_SOURCES.get(k, ())}
 
 
 class HybridRunner(DeviceRunner):
@@ -83,6 +99,7 @@ class HybridRunner(DeviceRunner):
         self.dp = pad(cfg.hidden_size)
         wide = any(m.type in ("latent_attention", "attention") and
                    (m.vdim > PREFILL_VALUE_MAX or pad(m.dim, 16) + pad(m.rot_dim, 16) > PREFILL_KEY_MAX) for s in cfg.layers for m in s.mixers())
+        self.shared_kv = {s.kv_from for s in cfg.layers if s.kv_from >= 0}
         self.absorb_max = 1 << 30 if self.exact32 or wide else ABSORB_MAX
         self._load(base)
         self._buf: dict = {}
@@ -134,7 +151,12 @@ class HybridRunner(DeviceRunner):
         for i, s in enumerate(cfg.layers):
             w = {k[len(f"l{i}."):]: t for k, t in base.items() if k.startswith(f"l{i}.")}
             m = {k[4:]: t for k, t in w.items() if k.startswith("mix.")}
-            L: dict = {n: norm(w[n]) for n in ("norm1", "norm1b", "norm2", "norm2b") if n in w}
+            L: dict = {}
+            for k in (1, 2) if s.has_mlp else (1,):
+                pre, post = cfg.norm_names(k)
+                L[f"pre{k}"], L[f"post{k}"] = norm(w[pre]) if pre else None, norm(w[post]) if post else None
+                if cfg.layer_scale:
+                    L[f"post{k}"] *= self._vec(w[f"ls{k}"], dp)
             L["dwa"] = self._vec(w["dwa"]) if cfg.depth_average else None
             getattr(self, "_load_" + s.type)(s, m, L)
             if s.has_mlp:
@@ -157,8 +179,7 @@ class HybridRunner(DeviceRunner):
             kv[:s.heads * dk].view(s.heads, dk, rank_p)[:, :s.dim, :s.kv_rank] = uk.to(self.device)
             kv[s.heads * dk:].view(s.heads, dv, rank_p)[:, :s.vdim, :s.kv_rank] = uv.to(self.device)
             L["ukv"] = kv
-        L["inv_freq"] = torch.tensor([s.rope_base ** (-2.0 * j / s.rot_dim) for j in range(s.rot_dim // 2)], dtype=torch.float64
-                                     ).to(self.device, torch.float32)
+        L["inv_freq"] = torch.tensor(rope_frequencies(s)[0], dtype=torch.float64).to(self.device, torch.float32)
         L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
 
     def _load_hgrn2(self, s: LayerSpec, m: dict, L: dict) -> None:
@@ -203,15 +224,24 @@ class HybridRunner(DeviceRunner):
                 bias[:self.cfg.hidden_size] += scale * self._vec(w["o.b"])
             L["parts"].append(P)
         L["in"], L["o"] = torch.cat(rows, 0), torch.cat(cols, 1)
-        L["o_bias"] = bias if any(p.biases for p in s.mixers()) else None
+        L["o_bias"] = bias if any(p.out_bias for p in s.mixers()) else None
 
     _load_parallel = _load_attention = _load_rglru = _load_parts
 
     def _load_part_attention(self, s: LayerSpec, w: dict, P: dict):
-        P["bias"] = self._vec(torch.cat([w[k + ".b"] for k in "qkv"])) if s.biases else None
-        P["tc_dv"] = hy.prefill_tc_values(s.dim, 0, s.vdim, s.scale)
-        P["dvp"] = hy.gqa_value_columns(s.dim, s.vdim, s.scale)
-        return self._mat(torch.cat([w[k] for k in "qkv"], 0), None, self.dp), self._heads_in(w["o"], s.heads, s.vdim)
+        own = "qkv" if s.kv_from < 0 else "q"
+        src = self.cfg.layers[s.kv_from] if s.kv_from >= 0 else s
+        P["bias"] = self._vec(torch.cat([w[k + ".b"] for k in own])) if s.biases else None
+        P["dvp"] = hy.gqa_value_columns(src.dim, src.vdim, src.scale)      # as the cache holds them
+        P["tc"] = hy.prefill_tc_values(s.dim, 0, s.vdim, s.scale) == P["dvp"]
+        P["kv_heads"] = s.kv_heads if s.kv_from < 0 else 0
+        P["q_norm"], P["k_norm"] = (self._vec(w[k + ".norm"]) if s.qk_norm and k in own else None for k in "qk")
+        P["rot"] = None
+        if s.rot_dim:
+            freq, scale = rope_frequencies(s)
+            P["rot"] = hy.Rotation(s.rot_dim, torch.tensor(freq, dtype=torch.float64).to(self.device), scale, s.rot_pairs == "next")
+        rows = [w[k] for k in own] + ([w["g"]] if s.head_gate else [])
+        return self._mat(torch.cat(rows, 0), None, self.dp), self._heads_in(w["o"], s.heads, s.vdim)
 
     def _load_part_rglru(self, s: LayerSpec, w: dict, P: dict):
         n, bp = s.heads * s.dim, pad(s.dim)
@@ -235,14 +265,21 @@ class HybridRunner(DeviceRunner):
 
     def _load_mlp_moe(self, s: LayerSpec, w: dict, L: dict) -> None:
         ffp = pad(s.expert_ff, 16)
-        L["router"], L["router_b"] = self._mat(w["router"], None, self.dp), self._vec(w["router.b"])
-        L["e_gu"] = torch.empty(s.experts * 2 * ffp, self.dp, dtype=self.dtype, device=self.device)
+
+        def inner(name: str, ff: int) -> torch.Tensor:
+            return self._glu(w[name + ".gate"], w[name + ".up"]) if s.glu else self._mat(w[name + ".up"], pad(ff, 16), self.dp)
+
+        # the gate of the shared expert is one more row of the router's matrix
+        L["router"] = self._mat(torch.cat([w["router"], w["shared.sg"]], 0) if s.shared_gate else w["router"], None, self.dp)
+        L["router_b"], L["correction"] = (self._vec(w[k]) if k in w else None for k in ("router.b", "correction"))
+        n = (2 if s.glu else 1) * ffp
+        L["e_in"] = torch.empty(s.experts * n, self.dp, dtype=self.dtype, device=self.device)
         L["e_down"] = torch.empty(s.experts * self.dp, ffp, dtype=self.dtype, device=self.device)
         for e in range(s.experts):
-            L["e_gu"][e * 2 * ffp:(e + 1) * 2 * ffp] = self._glu(w[f"e{e}.gate"], w[f"e{e}.up"])
+            L["e_in"][e * n:(e + 1) * n] = inner(f"e{e}", s.expert_ff)
             L["e_down"][e * self.dp:(e + 1) * self.dp] = self._mat(w[f"e{e}.down"], self.dp, ffp)
         if s.shared_ff:
-            L["gu"], L["down"] = self._glu(w["shared.gate"], w["shared.up"]), self._mat(w["shared.down"], self.dp, pad(s.shared_ff, 16))
+            L["s_in"], L["down"] = inner("shared", s.shared_ff), self._mat(w["shared.down"], self.dp, pad(s.shared_ff, 16))
 
     def set_adapter(self, slot: int, state) -> None:
         if state is not None:
@@ -355,22 +392,27 @@ class HybridRunner(DeviceRunner):
         hist = None
         if cfg.depth_average:
             hist = torch.empty((len(self.layers) + 1, M if M <= 1024 else pad(M, 1024), dp), dtype=torch.float32, device=dev)
-        first_norm = lambda i: (self.layers[i]["norm1"] if cfg.layers[i].type != "wkv" else None) if i < len(self.layers) \
-            else (self.final_norm if want_hidden else None)      # noqa: E731  (a token-shift mixer norms its own input)
+
+        def feed(i: int) -> dict:
+            """What the stream leaves for layer ``i``'s mixer, or for the output product behind the last layer."""
+            if i == len(self.layers):
+                return dict(w_next=self.final_norm, h=h) if want_hidden else {}
+            return {} if cfg.layers[i].type == "wkv" else dict(w_next=self.layers[i]["pre1"], h=h)      # a token-shift mixer norms its own input
+
         hy.residual_step(x, self.embed_norm, d, eps, mult=cfg.embed_scale, tokens=b.tokens, table=self.embed, freq=self.pos_freq, pos=b.pos,
-                         hist=hist, hist_n=0, w_next=first_norm(0), h=h)
+                         hist=hist, hist_n=0, **feed(0))
         for i, (s, L) in enumerate(zip(cfg.layers, self.layers)):
-            y, post = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b), L.get("norm1b")
+            y, post = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b), L["post1"]
             if s.has_mlp:
-                hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, w_next=L["norm2"], h=h)
-                y, post = getattr(self, "_mlp_" + s.mlp)(s, L, h, b), L.get("norm2b")
-            hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], w_next=first_norm(i + 1), h=h)
+                hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, w_next=L["pre2"], h=h)
+                y, post = getattr(self, "_mlp_" + s.mlp)(s, L, x, h, b), L["post2"]
+            hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], **feed(i + 1))
             if capture is not None:
                 capture.append(x[:, :d].clone())
         return x, h
 
     # -- feed-forwards ----------------------------------------------------------------------------------------
-    def _mlp_poly(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+    def _mlp_poly(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
         z = self._mm_take(b, "up", h, L["up"])
         a = self._new(b.M, pad(s.ff))
         return Sublayer(self._mm_take(b, "down", hy.poly_norm(z, L["act"], a, s.ff, self.cfg.norm_eps), L["down"]))
@@ -386,23 +428,41 @@ class HybridRunner(DeviceRunner):
             return a
         return hy.gated_act(self._mm_take(b, name, h, W), a, act)
 
-    def _mlp_gated(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+    def _act_product(self, b: Ragged, name: str, h, W, act: str) -> torch.Tensor:
+        """``act(h W^T)``, likewise."""
+        a = self._new(b.M, W.shape[0])
+        if not self.exact32 and self._small_plan(b, W)[1] == 1 and act == "relu2":
+            from ..ops.gemm import gemm_tn
+
+            bn, _, pair = self._small_plan(b, W)
+            return gemm_tn(h, W, out=a, relu2=True, bn=bn, two_cta=pair)
+        return hy.plain_act(self._mm_take(b, name, h, W), a, act)
+
+    def _mlp_gated(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
         return Sublayer(self._mm_take(b, "down", self._glu_product(b, "gu", h, L["gu"], s.act), L["down"]))
 
-    def _mlp_moe(self, s: LayerSpec, L, h, b: Ragged) -> Sublayer:
+    def _mlp_moe(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
         from ..ops import moe
 
         z = self._mm_take(b, "router", h, L["router"], f32=True)
-        plan = moe.route(z.t[:, :s.experts], s.top, True, L["router_b"], take=z.kind == hy.KIND_TAKE)
+        plan = moe.route(z.t[:, :s.experts + s.identity + s.shared_gate], s.top, True, L["router_b"], take=z.kind == hy.KIND_TAKE,
+                         correction=L["correction"], identity=s.identity, gate=s.shared_gate)
         xp, n = moe.gather(h, plan), L["e_down"].shape[1]
         a = torch.empty((plan.cap_rows, n), dtype=self.dtype, device=self.device)
         if self.exact32:
-            hy.gated_act(as_out(moe.grouped_gemm(xp, L["e_gu"], plan, 2 * n)), a, "silu")
+            z = as_out(moe.grouped_gemm(xp, L["e_in"], plan, (2 if s.glu else 1) * n))
+            (hy.gated_act if s.glu else hy.plain_act)(z, a, s.act)
+        elif s.glu:
+            moe.grouped_gemm(xp, L["e_in"], plan, 2 * n, swiglu_out=a, keep_preact=False)
         else:
-            moe.grouped_gemm(xp, L["e_gu"], plan, 2 * n, swiglu_out=a, keep_preact=False)
+            moe.grouped_gemm(xp, L["e_in"], plan, n, out=a, relu2=True)
         rows = moe.grouped_gemm(a, L["e_down"], plan, self.dp)
-        y = self._mm_take(b, "down", self._glu_product(b, "gu", h, L["gu"], "silu"), L["down"]) if s.shared_ff else None
-        return Sublayer(y, rows=rows, pos=plan.pos, weight=plan.topw)
+        y = None
+        if s.shared_ff:
+            y = self._mm_take(b, "down", (self._glu_product if s.glu else self._act_product)(b, "s_in", h, L["s_in"], s.act), L["down"])
+        # experts that are the identity take the sublayer's input, in 32-bit where that is the stream itself
+        return Sublayer(y, rows=rows, pos=plan.pos, weight=plan.topw, gate=plan.gate,
+                        identity=as_out(h if self.cfg.pre_norms else x) if s.identity else None)
 
     # -- mixers -------------------------------------------------------------------------------------------------
     def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Sublayer:
@@ -465,7 +525,7 @@ class HybridRunner(DeviceRunner):
     def _mix_wkv(self, i, s, L, x, h, b: Ragged) -> Sublayer:
         M, n = b.M, L["rkvg"].shape[1]
         mixes = self._heads_buf("mix", len(SHIFT_MIXES), M, b, self.dp)
-        hy.norm_shift_mix(x, L["norm1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
+        hy.norm_shift_mix(x, L["pre1"], L["mu"], mixes, self.kv.layers[i]["shift"], b.row_seq, b.cu_q, b.ctx, b.state_slot,
                           self.cfg.hidden_size, self.cfg.norm_eps)
         y = self._new(M, 4 * n)
         if M >= 1024 and not self.exact32:      # four products that each fill the machine: CTA-pair tiles
@@ -503,34 +563,45 @@ class HybridRunner(DeviceRunner):
         p = self._mm_take(b, "in", h, L["in"])
         o = self._new(b.M, L["o"].shape[1])
         for j, (spec, P) in enumerate(zip(s.mixers(), L["parts"])):
-            getattr(self, "_part_" + spec.type)(spec, P, p.col(P["in"]), o[:, P["out"]:], self.kv.part(i, j), b)
+            getattr(self, "_part_" + spec.type)(i, spec, P, p.col(P["in"]), o[:, P["out"]:], self.kv.part(i, j), b)
         return Sublayer(self._mm_take(b, "o", o, L["o"]), bias=L["o_bias"])
 
     _mix_parallel = _mix_attention = _mix_rglru = _mix_parts
 
-    def _part_attention(self, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
+    def _part_attention(self, i, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
         M, n_abs, kv = b.M, b.n_abs, cache["kv"]
         H, G, dk, dvp = s.heads, s.heads // s.kv_heads, pad(s.dim, 16), P["dvp"]
-        q = self._new(M, H * dk)
-        hy.gqa_finish(p, P["bias"], b.slot, kv, q, H, s.kv_heads, s.dim, s.vdim, dvp)
+        q, gate = self._new(M, H * dk), None
+        if s.qk_norm or P["rot"] or s.head_gate or s.kv_from >= 0:
+            gate = torch.empty((M, H), dtype=torch.float32, device=self.device) if s.head_gate else None
+            hy.gqa_finish_norm(p, P["bias"], b.slot, kv, q, H, P["kv_heads"], s.dim, s.vdim, dvp, P["q_norm"], P["k_norm"], self.cfg.norm_eps, P["rot"],
+                               b.pos, gate)
+        else:
+            hy.gqa_finish(p, P["bias"], b.slot, kv, q, H, s.kv_heads, s.dim, s.vdim, dvp)
         if n_abs:
             args = (q, kv, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.chunk, s.scale, P["scale"], o, n_abs, H, s.kv_heads, s.dim, s.vdim, dvp)
             if self.exact32 or max(dk, dvp) > hy.GQA_DECODE_MAX:
-                hy.gqa_attend(*args)
+                hy.gqa_attend(*args, softcap=s.softcap, gate=gate)
             else:
                 reach = min([b.reach] + [w for w in (s.window, s.chunk) if w > 0])
-                hy.gqa_decode(*args, splits=hy.gqa_decode_splits(n_abs, s.kv_heads * ((G + 15) // 16), reach))
+                hy.gqa_decode(*args, splits=hy.gqa_decode_splits(n_abs, s.kv_heads * ((G + 15) // 16), reach), softcap=s.softcap, gate=gate)
         if n_abs < M:
             plan = b.plan(s.window, s.chunk)
-            rest = dict(chunk=s.chunk, G=G, out_scale=P["scale"])
-            if P["tc_dv"]:
-                k, vt = hy.gqa_gather(kv, b.bt, plan, s.kv_heads, dk, dvp)
+            rest = dict(chunk=s.chunk, G=G, out_scale=P["scale"], softcap=s.softcap, gate=gate[n_abs:] if gate is not None else None)
+            src = self.cfg.kv_layer(i)
+            key = (src, s.window, s.chunk, P["tc"])
+            got = b.kept.get(key)
+            if got is None:
+                got = hy.gqa_gather(kv, b.bt, plan, s.kv_heads, dk, dvp) if P["tc"] else hy.latent_gather(kv, b.bt, plan)
+                if src in self.shared_kv:
+                    b.kept[key] = got
+            if P["tc"]:
+                k, vt = got
                 hy.latent_prefill_tc(q[n_abs:], k, vt, k, plan, s.window, s.scale, o[n_abs:], H, dk, dvp, 0, 0, s.vdim, **rest)
             else:
-                c = hy.latent_gather(kv, b.bt, plan)
-                hy.latent_prefill(q[n_abs:], c, c, plan, s.window, s.scale, o[n_abs:], H, dk, dvp, 0, 0, s.vdim, **rest)
+                hy.latent_prefill(q[n_abs:], got, got, plan, s.window, s.scale, o[n_abs:], H, dk, dvp, 0, 0, s.vdim, **rest)
 
-    def _part_rglru(self, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
+    def _part_rglru(self, i, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
         M, bp = b.M, pad(s.dim)
         # a buffer of its own per block size: padding columns are written by nobody
         u = self._heads_buf(f"u{s.dim}", s.heads, M, b, P["gates"].shape[2])

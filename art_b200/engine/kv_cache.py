@@ -277,7 +277,8 @@ class HybridCache:
     * latent attention: ``latent`` ``[num_blocks, block_size, rank_p + rot_p]``, paged, in the operand dtype; a row is the
       normed latent and the rotated key part, each padded with zeros to a multiple of 16;
     * grouped-query attention: ``kv`` ``[num_blocks, block_size, kv_heads * (dim_p + vdim_p)]``, paged, in the operand dtype; a
-      row is the keys of all heads, then their values, each padded with zeros;
+      row is the keys of all heads (as the scores take them: normed and rotated), then their values, each padded with zeros; a
+      layer that reads another one's keys and values holds none;
     * linear attention: ``state`` fp32 ``[num_slots, heads, vdim, dim padded to 4]`` (a value column's channels are
       contiguous), and for token-shift mixers ``shift`` fp32 ``[num_slots, width padded to 8]``, the last token's input;
     * gated linear recurrent units: ``state`` fp32 ``[num_slots, channels]`` and ``conv`` fp32 ``[num_slots, taps - 1, channels]``,
@@ -308,6 +309,8 @@ class HybridCache:
                     for k, v in HybridCache.layer_shapes(cfg, p, num_blocks, block_size, num_slots, dtype).items()}
         if spec.type == "latent_attention":
             return {"latent": ((num_blocks, block_size, up(spec.kv_rank, 16) + up(spec.rot_dim, 16)), dtype)}
+        if spec.kv_from >= 0:
+            return {}
         if spec.type == "attention":
             from ..ops.hybrid import gqa_value_columns
 
@@ -321,7 +324,8 @@ class HybridCache:
         return out
 
     def part(self, layer: int, j: int) -> dict[str, torch.Tensor]:
-        """The tensors of mixer ``j`` of a layer."""
+        """The tensors of mixer ``j`` of a layer, or of the layer whose keys and values it reads."""
+        layer = self.cfg.kv_layer(layer)
         L = self.layers[layer]
         if not self.cfg.layers[layer].parts:
             return L

@@ -81,6 +81,7 @@ class Replay:
 
 def main(argv: list[str] | None = None) -> int:
     from ..models.config import ModelConfig
+    from ..models.hybrid import HybridConfig
     from ..models.weights import load_base_weights
     from ..ops import _lib
     from .factory import UnsupportedPrecision, build_runner
@@ -93,6 +94,10 @@ def main(argv: list[str] | None = None) -> int:
     ap.add_argument("--slots", type=int, default=4, help="live requests (state slots)")
     a = ap.parse_args(argv)
     cfg = ModelConfig.from_pretrained_dir(a.model)
+    if isinstance(cfg, HybridConfig):
+        from .hybrid_runner import kernel_sources
+
+        _lib.require(kernel_sources(cfg))
     blocks = (a.max_tokens + BLOCK_SIZE - 1) // BLOCK_SIZE
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)

@@ -4,12 +4,15 @@ A configuration consists of layers and of the frame around them.  A layer (``Lay
 
 * a mixer: latent attention with a sliding window, grouped-query attention with a window or in chunks, HGRN2 or lightning
   linear attention, RWKV-style time mixing, a gated linear recurrent unit behind a short convolution, or several of these
-  side by side on the same input, each with a factor (``parts``);
-* a feed-forward: PolyNorm, gated (``act(gate) * up``), a mixture of gated experts with an optional shared expert, or none.
+  side by side on the same input, each with a factor (``parts``).  Grouped-query attention may rotate its queries and keys
+  (either pairing, scaled frequencies), norm them, squash its scores, gate its heads and read another layer's keys and values;
+* a feed-forward: PolyNorm, gated (``act(gate) * up``), a mixture of experts (gated or not, some of them the identity) with an
+  optional shared expert, or none.
 
-The frame (fields of ``HybridConfig``) is the design's: norms before, or before and after each sublayer, norm weights stored
-as they are or around zero, a residual multiplier, a weighted average over the results of all earlier layers, an embedding
-that is normalised, or scaled and given sinusoidal position vectors, an output table of its own or the embedding's.
+The frame (fields of ``HybridConfig``) is the design's: norms before, after, or before and after each sublayer, norm weights
+stored as they are or around zero, a factor per column on each sublayer's result, a residual multiplier, a weighted average
+over the results of all earlier layers, an embedding that is normalised, or scaled and given sinusoidal position vectors, an
+output table of its own or the embedding's.
 
 ``HybridConfig`` answers the questions the engine asks of any configuration (``vocab_size``, ``hidden_size``,
 ``num_layers``, ``is_moe`` ...); ``from_design_dict`` reads a ``config.json`` whose ``architecture`` key names a design of
@@ -19,6 +22,7 @@ it.  The reference serves library models only (src/art/local/state.py); designs 
 from __future__ import annotations
 
 import dataclasses
+import math
 from dataclasses import dataclass, field
 
 import torch
@@ -38,27 +42,38 @@ class LayerSpec:
     vdim: int
     ff: int = 0                                # width of a dense feed-forward, 0: none
     # attention
-    rot_dim: int = 0
+    rot_dim: int = 0                           # rotated dimensions of a head, 0: no rotation
+    rot_pairs: str = "half"                    # a dimension's partner: half the rotated ones further ("half") or its neighbour ("next")
+    rope_scaling: tuple[float, float, float, float] | None = None      # factor, original context, fast and slow turns (YaRN)
     kv_rank: int = 0
     kv_heads: int = 0
     scale: float = 1.0
     rope_base: float = 10000.0
     window: int = 0                            # keys seen, the token itself included; 0: all earlier ones
     chunk: int = 0                             # keys of the same chunk of the sequence only; 0: all earlier ones
-    biases: bool = False                       # q, k, v and output projections have biases
+    biases: bool = False                       # q, k and v projections have biases
+    out_bias: bool = False                     # ... and the output projection
+    qk_norm: bool = False                      # RMS norm over all heads of q together, and of k, before the rotation
+    softcap: float = 0.0                       # scores pass softcap * tanh(score / softcap); 0: as they are
+    head_gate: bool = False                    # heads are multiplied by the sigmoid of a projection of the input
+    kv_from: int = -1                          # layer whose keys and values this one reads; -1: its own
     # wkv: width of the low-rank decay projection (given by its tensors, not by the configuration)
     decay_rank: int = 0
     decay: tuple[float, ...] = ()              # lightning: one factor per head
     conv: int = 1                              # rglru: taps of the short convolution
     parts: tuple["LayerSpec", ...] = ()        # parallel: mixers side by side, and the factor of each one's result
     part_scales: tuple[float, ...] = ()
-    # feed-forward: "poly" (up, PolyNorm, down), "gated" (act(gate) * up, down) or "moe" (gated experts)
+    # feed-forward: "poly" (up, PolyNorm, down), "gated" (act(gate) * up, down) or "moe" (experts)
     mlp: str = "poly"
     act: str = "silu"
+    glu: bool = True                           # experts are act(gate) * up, down; else act(up), down
     experts: int = 0
     top: int = 0
     expert_ff: int = 0
-    shared_ff: int = 0                         # gated shared expert, 0: none
+    identity: int = 0                          # further outputs of the router that hand the input on
+    router: str = "logits"                     # chooses by "logits" (+ bias, softmax over the chosen) or "scores" (softmax over all, + correction)
+    shared_ff: int = 0                         # shared expert, 0: none
+    shared_gate: bool = False                  # the shared expert is multiplied by the sigmoid of a projection of the input
 
     @property
     def recurrent(self) -> bool:
@@ -84,7 +99,9 @@ class HybridConfig:
     family: str = "nikelix"
     max_position_embeddings: int = 1 << 20
     # the frame
-    post_norms: bool = True                    # a norm behind each sublayer, too
+    pre_norms: bool = True                     # a norm before each sublayer; without, sublayers read the residual stream itself
+    post_norms: bool = True                    # a norm behind each sublayer
+    layer_scale: bool = False                  # each sublayer's result (behind its norm) has a factor per column
     depth_average: bool = True                 # layer results are averaged with all earlier ones
     norm_offset: float = 0.0                   # added to the weights of the frame's norms
     embed_norm: bool = True
@@ -103,6 +120,16 @@ class HybridConfig:
         """True when some layer carries a state from token to token (no prefix of a sequence can then be shared)."""
         return any(s.recurrent for s in self.layers)
 
+    def kv_layer(self, i: int) -> int:
+        """The layer whose keys and values layer ``i`` reads: its own, or the one it shares with."""
+        return self.layers[i].kv_from if self.layers[i].kv_from >= 0 else i
+
+    def norm_names(self, k: int) -> tuple[str | None, str | None]:
+        """Tensors of sublayer ``k``'s (1: mixer, 2: feed-forward) norms before and behind it."""
+        if not self.pre_norms:
+            return None, f"norm{k}"
+        return f"norm{k}", f"norm{k}b" if self.post_norms else None
+
     def num_params(self) -> int:
         n = 0
         for shape in tensor_shapes(self).values():
@@ -120,6 +147,8 @@ class HybridConfig:
         cfg = ARCHITECTURES[design](d, name)
         for i, s in enumerate(cfg.layers):
             _check_layer(i, s)
+            if s.kv_from >= 0:
+                _check_shared(cfg, i, s)
         return cfg
 
 
@@ -127,12 +156,49 @@ def _check_layer(i: int, s: LayerSpec) -> None:
     for p in s.mixers():
         if p.type == "attention" and (p.kv_heads <= 0 or p.heads % p.kv_heads):
             raise ValueError(f"layer {i}: {p.heads} query heads do not divide over {p.kv_heads} key heads")
+        if p.type == "attention" and (p.rot_dim % 2 or p.rot_dim > p.dim):
+            raise ValueError(f"layer {i}: rot.dims must be even and at most the head's {p.dim} dimensions, not {p.rot_dim}")
         if p.type == "lightning" and len(p.decay) != p.heads:
             raise ValueError(f"layer {i}: {len(p.decay)} decay factors for {p.heads} heads")
         if p.type in ("hgrn2", "wkv", "lightning") and max(p.dim, p.vdim) > 256:
             raise ValueError(f"layer {i}: {p.type} heads of more than 256 columns are not supported")
-    if s.experts and not (0 < s.top <= min(s.experts, MAX_TOP) and s.experts <= MAX_EXPERTS):
-        raise ValueError(f"layer {i}: {s.top} of {s.experts} experts (at most {MAX_TOP} of {MAX_EXPERTS}) are not supported")
+    outputs = s.experts + s.identity
+    if s.experts and not (0 < s.top <= min(outputs, MAX_TOP) and outputs <= MAX_EXPERTS):
+        raise ValueError(f"layer {i}: {s.top} of {outputs} experts (at most {MAX_TOP} of {MAX_EXPERTS}) are not supported")
+
+
+def _check_shared(cfg: HybridConfig, i: int, s: LayerSpec) -> None:
+    src = cfg.layers[s.kv_from] if s.kv_from < i else None
+    if src is None or src.type != "attention" or src.parts or src.kv_from >= 0:
+        raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys and values of its own")
+    if (src.kv_heads, src.dim, src.vdim) != (s.kv_heads, s.dim, s.vdim):
+        raise ValueError(f"layer {i}: its key heads differ from those of layer {s.kv_from}, whose keys and values it reads")
+
+
+def rope_frequencies(s: LayerSpec) -> tuple[list[float], float]:
+    """One frequency per rotated pair and the factor of sine and cosine.  Scaled (YaRN; Peng et al., "YaRN: Efficient Context
+    Window Extension of Large Language Models"): pairs that make few turns over the original context are slowed by the factor,
+    those that make many are kept, with a linear ramp over the pairs in between."""
+    n = s.rot_dim
+    freq = [s.rope_base ** (-2.0 * j / n) for j in range(n // 2)]
+    if s.rope_scaling is None:
+        return freq, 1.0
+    factor, original, fast, slow = s.rope_scaling
+
+    def pair(turns: float) -> float:
+        return n * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(s.rope_base))
+
+    lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), n - 1)
+    for j in range(n // 2):
+        ramp = min(1.0, max(0.0, (j - lo) / max(hi - lo, 0.001)))
+        freq[j] = freq[j] / factor * ramp + freq[j] * (1.0 - ramp)
+    return freq, 0.1 * math.log(factor) + 1.0
+
+
+def _known(i: int, what: str, d: dict, keys: tuple[str, ...]) -> None:
+    extra = sorted(set(d) - set(keys))
+    if extra:
+        raise ValueError(f"layer {i}: {what} key{'s' if len(extra) > 1 else ''} {', '.join(map(repr, extra))} not supported")
 
 
 def _mixer_kind(i: int, e: dict, supported: tuple[str, ...]) -> str:
@@ -182,7 +248,7 @@ def _read_naselorn(d: dict, name: str) -> HybridConfig:
             if width % blocks:
                 raise ValueError(f"layer {i}: {width} channels do not divide over {blocks} blocks")
             parts = (LayerSpec("attention", int(a["heads"]), int(a["dim"]), int(a["vdim"]), kv_heads=int(a["kv_heads"]), scale=float(a["scale"]),
-                               chunk=int((a.get("mask") or {}).get("size", 0)), biases=True),
+                               chunk=int((a.get("mask") or {}).get("size", 0)), biases=True, out_bias=True),
                      LayerSpec("rglru", blocks, width // blocks, width // blocks, conv=int(r["conv"])))
             spec = LayerSpec(kind, 0, 0, 0, parts=parts, part_scales=(float(m["left_scale"]), float(m["right_scale"])))
         ff = _mlp_kind(i, mlp, ("dense", "moe"))
@@ -197,9 +263,36 @@ def _read_naselorn(d: dict, name: str) -> HybridConfig:
                         embed_scale=float(d["embedding"]["scale"]), **NASELORN_FRAME)
 
 
+def _read_gaborax(d: dict, name: str) -> HybridConfig:
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        kind, m, mlp = _mixer_kind(i, e, ("attention", "attention_2")), e["mixer"], e.get("mlp")
+        _known(i, "mixer", m, ("heads", "kv_heads", "dim", "vdim", "rot", "scale", "softcap", "kv_from"))
+        first, rot = kind == "attention", m["rot"]
+        _known(i, "rot", rot, ("base", "dims", "scaling"))
+        spec = LayerSpec("attention", int(m["heads"]), int(m["dim"]), int(m["vdim"]), kv_heads=int(m["kv_heads"]), scale=float(m["scale"]),
+                         rot_dim=int(rot["dims"]), rope_base=float(rot["base"]), rot_pairs="half" if first else "next", qk_norm=True,
+                         biases=not first, head_gate=first, softcap=float(m.get("softcap") or 0.0))
+        if rot.get("scaling"):
+            spec.rope_scaling = tuple(float(rot["scaling"][k]) for k in ("factor", "original", "fast", "slow"))
+        if m.get("kv_from") is not None:
+            spec.kv_from = int(m["kv_from"])
+            if spec.kv_from < 0:
+                raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys and values of its own")
+        if _mlp_kind(i, mlp, ("moe",)):
+            r, shared = mlp["router"], mlp.get("shared")
+            spec.mlp, spec.act, spec.glu, spec.router = "moe", "relu2", False, "scores"
+            spec.expert_ff, spec.experts, spec.top, spec.identity = int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"]), int(r.get("identity") or 0)
+            spec.shared_ff, spec.shared_gate = (int(shared["ff"]), True) if shared else (0, False)
+        layers.append(spec)
+    return HybridConfig(name=name, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers, norm_eps=float(d["norm"]["eps"]),
+                        **GABORAX_FRAME)
+
+
 NASELORN_FRAME = dict(family="naselorn", post_norms=False, depth_average=False, norm_offset=1.0, embed_norm=False, position_base=10000.0,
                       tie_word_embeddings=False)
-ARCHITECTURES = {"Nikelix": _read_nikelix, "Naselorn": _read_naselorn}
+GABORAX_FRAME = dict(family="gaborax", pre_norms=False, post_norms=True, layer_scale=True, depth_average=False, norm_offset=1.0, embed_norm=False)
+ARCHITECTURES = {"Nikelix": _read_nikelix, "Naselorn": _read_naselorn, "Gaborax": _read_gaborax}
 
 
 def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
@@ -214,8 +307,19 @@ def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
     if s.type == "lightning":
         return {"q": (qk, d), "k": (qk, d), "v": (v, d), "g": (v, d), "o": (d, v), "norm": (v,)}
     if s.type == "attention":
-        out = {"q": (qk, d), "k": (s.kv_heads * s.dim, d), "v": (s.kv_heads * s.vdim, d), "o": (d, v)}
-        return {**out, **{k + ".b": (t[0],) for k, t in out.items()}} if s.biases else out
+        own = {"q": (qk, d)}
+        if s.kv_from < 0:
+            own.update({"k": (s.kv_heads * s.dim, d), "v": (s.kv_heads * s.vdim, d)})
+        out = {**own, "o": (d, v)}
+        if s.biases:
+            out.update({k + ".b": (t[0],) for k, t in own.items()})
+        if s.out_bias:
+            out["o.b"] = (d,)
+        if s.qk_norm:
+            out.update({k + ".norm": (own[k][0],) for k in "qk" if k in own})
+        if s.head_gate:
+            out["g"] = (s.heads, d)
+        return out
     if s.type == "rglru":
         gates = {k: t for g in ("ra", "ri") for k, t in ((g, (s.heads, s.dim, s.dim)), (g + ".b", (s.heads, s.dim)))}
         return {"y": (qk, d), "y.b": (qk,), "x": (qk, d), "x.b": (qk,), "conv": (qk, s.conv), "conv.b": (qk,), **gates, "lam": (qk,), "o": (d, qk)}
@@ -233,9 +337,15 @@ def _mlp_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
         return {"up": (s.ff, d), "down": (d, s.ff), "act": (4,)}
     if s.mlp == "gated":
         return glu("", s.ff)
-    out = {k: t for e in range(s.experts) for k, t in glu(f"e{e}.", s.expert_ff).items()}
-    out.update({"router": (s.experts, d), "router.b": (s.experts,)})
-    return {**out, **(glu("shared.", s.shared_ff) if s.shared_ff else {})}
+    form = glu if s.glu else lambda pre, ff: {pre + "up": (ff, d), pre + "down": (d, ff)}
+    out = {k: t for e in range(s.experts) for k, t in form(f"e{e}.", s.expert_ff).items()}
+    n = s.experts + s.identity
+    out.update({"router": (n, d), "router.b" if s.router == "logits" else "correction": (n,)})
+    if s.shared_ff:
+        out.update(form("shared.", s.shared_ff))
+        if s.shared_gate:
+            out["shared.sg"] = (1, d)
+    return out
 
 
 def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
@@ -248,11 +358,12 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
         out["head"] = (cfg.vocab_size, d)
     for i, s in enumerate(cfg.layers):
         p = f"l{i}."
-        norms = ["norm1"] + (["norm1b"] if cfg.post_norms else [])
+        for k in (1, 2) if s.has_mlp else (1,):
+            out.update({p + n: (d,) for n in cfg.norm_names(k) if n})
+            if cfg.layer_scale:
+                out[f"{p}ls{k}"] = (d,)
         if s.has_mlp:
-            norms += ["norm2"] + (["norm2b"] if cfg.post_norms else [])
             out.update({p + "mlp." + k: t for k, t in _mlp_shapes(s, d).items()})
-        out.update({p + n: (d,) for n in norms})
         out.update({p + "mix." + k: t for k, t in _mixer_shapes(s, d).items()})
         if cfg.depth_average:
             out[p + "dwa"] = (i + 2,)
@@ -307,6 +418,10 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
             w[k] = uni(*shape)
         elif leaf.endswith("lam"):             # memories from a token to some thousand tokens
             w[k] = uni(*shape, lo=-8.0, hi=1.0)
+        elif leaf in ("ls1", "ls2"):
+            w[k] = rnd(*shape, std=0.2, mean=0.8)
+        elif leaf == "correction":             # moves a choice now and then
+            w[k] = rnd(*shape, std=0.3 / shape[0])
         elif leaf in ("u", "f.b") or leaf.endswith(".b"):
             w[k] = rnd(*shape, std=0.5)
         else:
@@ -331,13 +446,34 @@ def _naselorn_preset(name: str, width: int, n_layers: int, experts: int, top: in
     hd = 128
     decay = tuple(1 - 2.0 ** (-1 - 7.0 * h / max(1, width // hd - 1)) for h in range(width // hd))
     li = LayerSpec("lightning", width // hd, hd, hd, decay=decay)
-    parts = (LayerSpec("attention", width // hd, hd, hd, kv_heads=max(1, width // hd // 4), scale=hd ** -0.5, chunk=chunk, biases=True),
+    parts = (LayerSpec("attention", width // hd, hd, hd, kv_heads=max(1, width // hd // 4), scale=hd ** -0.5, chunk=chunk, biases=True, out_bias=True),
              LayerSpec("rglru", width // 256, 256, 256, conv=4))
     pa = LayerSpec("parallel", 0, 0, 0, parts=parts, part_scales=(0.5, 0.5))
     layers = [dataclasses.replace(pa if i % 4 == 3 else li, mlp="moe", experts=experts, top=top, expert_ff=expert_ff, shared_ff=shared_ff)
               for i in range(n_layers)]
     layers[0] = dataclasses.replace(li, mlp="gated", act="relu", ff=dense_ff)
     return HybridConfig(name=name, vocab_size=vocab, hidden_size=width, layers=layers, embed_scale=width ** 0.5, **NASELORN_FRAME)
+
+
+def _gaborax_preset(name: str, width: int, n_layers: int, experts: int, identity: int, top: int, expert_ff: int, shared_ff: int,
+                    vocab: int = 32000) -> HybridConfig:
+    """``n_layers`` layers that alternate between the two kinds of attention; every fourth one reads the keys and values of the
+    layer two before it."""
+    hd, heads = 128, width // 128
+    one = LayerSpec("attention", heads, hd, hd, kv_heads=max(1, heads // 4), scale=hd ** -0.5, rot_dim=hd, rope_base=5e5, qk_norm=True, mlp="moe",
+                    act="relu2", glu=False, router="scores", experts=experts, identity=identity, top=top, expert_ff=expert_ff, shared_ff=shared_ff,
+                    shared_gate=True)
+    a, b = dataclasses.replace(one, head_gate=True), dataclasses.replace(one, rot_pairs="next", biases=True, softcap=50.0, rope_scaling=(4.0, 8192, 32, 1))
+    layers = [dataclasses.replace(b if i % 2 else a, kv_from=i - 2 if i % 4 == 2 else -1) for i in range(n_layers)]
+    return HybridConfig(name=name, vocab_size=vocab, hidden_size=width, layers=layers, **GABORAX_FRAME)
+
+
+def _gaborax_tiny() -> HybridConfig:
+    moe = dict(mlp="moe", act="relu2", glu=False, router="scores", experts=6, identity=3, top=2, expert_ff=48, shared_ff=80, shared_gate=True)
+    a = LayerSpec("attention", 4, 32, 24, kv_heads=2, scale=0.2, rot_dim=16, qk_norm=True, head_gate=True, **moe)
+    b = LayerSpec("attention", 6, 24, 40, kv_heads=3, scale=0.25, rot_dim=24, rot_pairs="next", rope_scaling=(2.0, 256, 16, 1), qk_norm=True, biases=True,
+                  softcap=20.0, **moe)
+    return HybridConfig("gaborax-tiny", 512, 128, [a, b, dataclasses.replace(a, kv_from=0)], **GABORAX_FRAME)
 
 
 HYBRID_PRESETS: dict[str, HybridConfig] = {
@@ -350,8 +486,11 @@ HYBRID_PRESETS: dict[str, HybridConfig] = {
     "naselorn-tiny": HybridConfig("naselorn-tiny", 512, 128, [
         LayerSpec("lightning", 2, 24, 40, 176, decay=(0.7, 0.97), mlp="gated", act="relu"),
         LayerSpec("parallel", 0, 0, 0, mlp="moe", experts=6, top=2, expert_ff=48, shared_ff=80, part_scales=(0.7, 0.4), parts=(
-            LayerSpec("attention", 4, 16, 24, kv_heads=2, scale=0.25, chunk=20, biases=True), LayerSpec("rglru", 3, 20, 20, conv=3)))],
+            LayerSpec("attention", 4, 16, 24, kv_heads=2, scale=0.25, chunk=20, biases=True, out_bias=True), LayerSpec("rglru", 3, 20, 20, conv=3)))],
         embed_scale=8.0, **NASELORN_FRAME),
     "naselorn-2b-a1b": _naselorn_preset("naselorn-2b-a1b", 2048, 16, 64, 8, 512, 1024, 6144),
     "naselorn-14b-a4b": _naselorn_preset("naselorn-14b-a4b", 4096, 16, 64, 8, 1024, 2048, 12288),
+    "gaborax-tiny": _gaborax_tiny(),
+    "gaborax-2b-a1b": _gaborax_preset("gaborax-2b-a1b", 2048, 16, 64, 8, 8, 768, 1536),
+    "gaborax-14b-a4b": _gaborax_preset("gaborax-14b-a4b", 4096, 16, 64, 8, 8, 1536, 3072),
 }

@@ -22,7 +22,7 @@ import torch
 
 _NATIVE = Path(__file__).resolve().parent.parent / "_native"
 _lock = threading.Lock()
-_kernels: ctypes.CDLL | None = None
+_kernels: "ctypes.CDLL | _Part | None" = None
 _runtime: ctypes.CDLL | None = None
 _status: dict[int, torch.Tensor] = {}
 
@@ -56,13 +56,48 @@ def _load(name: str) -> ctypes.CDLL:
         from .. import build as _build
 
         try:
-            _build.build_all(checked=name.endswith("_checked.so"))
+            if path == _build.RUNTIME_LIB:
+                _build.build_runtime()
+            else:
+                _build.build_all(checked=name.endswith("_checked.so"))
         except Exception as e:  # pragma: no cover - depends on toolchain
             raise NativeLibraryError(f"{path} is missing and could not be built: {e}") from e
     try:
         return ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
     except OSError as e:
         raise NativeLibraryError(f"cannot load {path}: {e}") from e
+
+
+class _Part:
+    """A library of some kernels; a kernel that it lacks builds and loads the complete one."""
+
+    def __init__(self, lib: ctypes.CDLL):
+        self._lib = lib
+
+    def __getattr__(self, name: str):
+        try:
+            f = getattr(self._lib, name)
+        except AttributeError:
+            if not name.startswith("artb_"):
+                raise
+            f = getattr(_load("libartb_kernels.so"), name)
+        setattr(self, name, f)
+        return f
+
+
+def require(stems) -> None:
+    """Says, before the first kernel call, which kernel sources this process will use.  Where the complete library has not
+    been built yet (a fresh checkout), only those are compiled."""
+    global _kernels
+    from .. import build as _build
+
+    with _lock:
+        if _kernels is not None or bounds_checked() or _build.KERNEL_LIB.exists():
+            return
+        try:
+            _kernels = _Part(ctypes.CDLL(str(_build.build_part(stems)), mode=ctypes.RTLD_GLOBAL))
+        except Exception as e:  # pragma: no cover - depends on toolchain
+            raise NativeLibraryError(f"the kernels of {', '.join(sorted(stems))} could not be built: {e}") from e
 
 
 def kernels() -> ctypes.CDLL:

@@ -17,14 +17,16 @@ from . import _lib
 vp, ci, cl, cf = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
 SCAN_HGRN2, SCAN_WKV, SCAN_FIXED = 0, 1, 2
 GATE_SILU, GATE_SIGMOID = 0, 1
-ACTS = {"silu": 0, "relu": 1}
+ACTS = {"silu": 0, "relu": 1, "relu2": 2}       # relu2: the square of relu
 KIND_BF16, KIND_F32, KIND_TAKE = 0, 1, 2
 _sigs = {
-    "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, vp, ci, ci, vp, vp, cl, vp, vp, vp, cl, ci, vp, vp, vp, ci, ci, ci, ci, cf, vp, vp],
+    "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, vp, vp, ci, ci, vp, vp, cl, vp, ci, ci, vp, vp, vp, cl, ci, vp, vp,
+                           vp, ci, ci, ci, ci, cf, vp, vp],
     "artb_norm_shift_mix": [ci, vp, ci, vp, vp, ci, vp, cl, ci, vp, cl, vp, vp, vp, vp, ci, ci, ci, cf, vp, vp],
     "artb_poly_norm": [ci, vp, ci, ci, vp, vp, ci, ci, ci, ci, cf, vp],
     "artb_split_tanh": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
     "artb_gated_act": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
+    "artb_plain_act": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
     "artb_head_norm": [ci, vp, ci, vp, ci, vp, ci, ci, ci, vp, ci, ci, ci, ci, ci, cf, vp],
     "artb_gather_norm": [ci, vp, ci, vp, ci, vp, vp, ci, ci, ci, cf, cl, vp, vp],
     "artb_linear_scan": [ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
@@ -36,13 +38,15 @@ _sigs = {
     "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
     "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, ci, vp, vp],
     "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, vp, ci, vp, vp],
-    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci,
+    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci,
                                ci, ci, vp, vp],
-    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp],
+    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci, ci,
+                            ci, ci, vp],
     "artb_gqa_finish": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_finish_norm": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp, cf, vp, cf, ci, ci, vp, vp, vp, vp],
     "artb_gqa_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, ci, vp, vp, ci, ci, vp, vp],
-    "artb_gqa_decode": [vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, vp, vp],
-    "artb_gqa_attend": [ci, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_decode": [vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_attend": [ci, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
     "artb_short_conv": [ci, vp, ci, ci, vp, vp, vp, ci, vp, cl, vp, vp, vp, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, vp, vp],
     "artb_rglru": [ci, ci, vp, ci, ci, vp, ci, vp, vp, vp, vp, ci, ci, vp, vp, cl, vp, vp, vp, ci, vp, ci, cf, ci, ci, ci, ci, vp, vp],
     "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
@@ -88,13 +92,16 @@ def _st(t: torch.Tensor):
 
 @dataclass
 class Sublayer:
-    """What a sublayer hands to the residual stream: ``y`` (may be missing), ``bias`` [dp] and the rows of a token's experts,
-    ``rows`` [cap, dp] weighted by ``weight`` [M, k] at the places ``pos`` [M, k]."""
+    """What a sublayer hands to the residual stream: ``y`` (may be missing) times ``gate`` [M], ``bias`` [dp] and the rows of a
+    token's experts, ``rows`` [cap, dp] weighted by ``weight`` [M, k] at the places ``pos`` [M, k]; a place of -1 is the token's
+    row of ``identity``."""
     y: Out | None = None
     bias: torch.Tensor | None = None
     rows: torch.Tensor | None = None
     pos: torch.Tensor | None = None
     weight: torch.Tensor | None = None
+    gate: torch.Tensor | None = None
+    identity: Out | None = None
 
 
 def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps: float, *, y: Out | None = None, x_in=None,
@@ -103,10 +110,12 @@ def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps:
     """One sublayer boundary of the fp32 residual stream ``[M, dp]``; ``y`` (or ``sub``) is the sublayer's output, or
     ``tokens`` / ``table`` the embedding, to which ``freq`` (fp64 ``[dp / 2]``) and ``pos`` add a sinusoidal position vector.
     ``w_post``: norm weight of the output; None: it is taken as it is, times ``mult``.  ``hist`` fp32 ``[layers + 1, M, dp]``: the result is stored at ``hist_n`` and, with ``avg``,
-    replaced by the weighted average of entries ``0 .. hist_n``.  ``w_next`` / ``h``: the next sublayer's input norm."""
+    replaced by the weighted average of entries ``0 .. hist_n``.  ``w_next`` / ``h``: the next sublayer's input norm; without
+    ``w_next``, ``h`` is the stream itself in the operand dtype."""
     M, dp = x_out.shape
     s = sub if sub is not None else Sublayer(y)
     y, ex = s.y, s.rows
+    idn = s.identity
     op = next((t for t in (table, h, ex) if t is not None), None)      # any tensor of the operand dtype
     f32 = _is32(op) if op is not None else 0
     if freq is not None and freq.dtype != torch.float64:
@@ -114,9 +123,10 @@ def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps:
     _lib.check_rc(_f("artb_residual_step")(
         f32, _lib.ptr(tokens), _lib.ptr(table), table.stride(0) if table is not None else 0, table.shape[0] if table is not None else 0,
         _lib.ptr(y.t if y is not None else None), y.t.stride(0) if y is not None else 0, y.kind if y is not None else 0,
-        _lib.ptr(x_in), _lib.ptr(x_out), x_out.stride(0), _lib.ptr(w_post), mult, _lib.ptr(s.bias), _lib.ptr(ex),
+        _lib.ptr(x_in), _lib.ptr(x_out), x_out.stride(0), _lib.ptr(w_post), mult, _lib.ptr(s.gate), _lib.ptr(s.bias), _lib.ptr(ex),
         ex.stride(0) if ex is not None else 0, s.pos.shape[1] if ex is not None else 0, _lib.ptr(s.pos), _lib.ptr(s.weight),
-        ex.shape[0] if ex is not None else 0, _lib.ptr(freq), _lib.ptr(pos), _lib.ptr(hist),
+        ex.shape[0] if ex is not None else 0, _lib.ptr(idn.t if idn is not None else None), idn.t.stride(0) if idn is not None else 0,
+        idn.kind if idn is not None else 0, _lib.ptr(freq), _lib.ptr(pos), _lib.ptr(hist),
         hist.stride(0) if hist is not None else 0, hist_n, _lib.ptr(avg), _lib.ptr(w_next), _lib.ptr(h),
         h.stride(0) if h is not None else 0, M, d, dp, eps, _st(x_out), _lib.stream_ptr()), "residual_step")
 
@@ -148,6 +158,13 @@ def gated_act(z: Out, out, act: str) -> torch.Tensor:
     """``act(gate) * up`` of a gate|up projection whose columns are interleaved in blocks of 16."""
     _lib.check_rc(_f("artb_gated_act")(_is32(out), _lib.ptr(z.t), z.t.stride(0), z.kind, _lib.ptr(out), out.stride(0), out.shape[0],
                                        out.shape[1], ACTS[act], _lib.stream_ptr()), "gated_act")
+    return out
+
+
+def plain_act(z: Out, out, act: str) -> torch.Tensor:
+    """``act(z)``, for a consumer behind a split product."""
+    _lib.check_rc(_f("artb_plain_act")(_is32(out), _lib.ptr(z.t), z.t.stride(0), z.kind, _lib.ptr(out), out.stride(0), out.shape[0],
+                                       out.shape[1], ACTS[act], _lib.stream_ptr()), "plain_act")
     return out
 
 
@@ -316,14 +333,19 @@ def latent_gather(cache, block_table, plan: PrefillPlan) -> torch.Tensor:
     return out
 
 
+def _gate(gate):
+    return _lib.ptr(gate), gate.stride(0) if gate is not None else 0
+
+
 def latent_prefill(q, kv, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                   vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0) -> torch.Tensor:
+                   vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None) -> torch.Tensor:
     """Masked attention of the portions: ``q`` [rows, H * (dk + rot_p)], ``kv`` [n_keys, H / G * (dk + dv)] the expanded
-    keys and values (``G`` heads share them), ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)]."""
+    keys and values (``G`` heads share them), ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)].  ``softcap`` > 0 squashes
+    the scores; ``gate`` fp32 [rows, H] multiplies the heads."""
     _lib.check_rc(_f("artb_latent_prefill")(
         _lib.ptr(q), q.stride(0), _lib.ptr(kv), kv.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(plan.tile_seq),
         _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0), _lib.ptr(plan.key_off),
-        _lib.ptr(plan.key_pos0), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p,
+        _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p,
         _lib.stream_ptr()), "latent_prefill")
     return o
 
@@ -341,12 +363,13 @@ def gqa_value_columns(dim: int, vdim: int, scale: float) -> int:
 
 
 def latent_prefill_tc(q, k, vt, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                      vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0) -> torch.Tensor:
+                      vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None) -> torch.Tensor:
     """:func:`latent_prefill` on tcgen05: ``k`` [n_keys, H / G * dk], values transposed ``vt`` [H / G * dv, n_keys]."""
     _lib.check_rc(_f("artb_latent_prefill_tc")(
         _lib.ptr(q), q.stride(0), q.shape[0], _lib.ptr(k), k.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(vt), vt.stride(0),
         plan.n_keys, _lib.ptr(plan.tile_seq), _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0),
-        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0), pad(vdim), H, G, dk, dv, rot_p, _st(o),
+        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(o), o.stride(0),
+        pad(vdim), H, G, dk, dv, rot_p, _st(o),
         _lib.stream_ptr()), "latent_prefill_tc")
     return o
 
@@ -359,6 +382,32 @@ def gqa_finish(p: Out, bias, slot, cache, q, H: int, Hkv: int, dim: int, vdim: i
         _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(bias), _lib.ptr(slot), _lib.ptr(cache), cache.shape[-1],
         cache.shape[0] * cache.shape[1], _lib.ptr(q), q.stride(0), M, H, Hkv, dim, pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()),
         "gqa_finish")
+
+
+@dataclass
+class Rotation:
+    """The rotation of the first ``dims`` columns of a head: ``freq`` fp64 [dims / 2] per pair (on the device), ``scale`` the factor of
+    sine and cosine; a column's partner is its neighbour (``next``) or ``dims / 2`` columns further."""
+    dims: int
+    freq: torch.Tensor
+    scale: float = 1.0
+    next: bool = False
+
+
+def gqa_finish_norm(p: Out, bias, slot, cache, q, H: int, Hkv: int, dim: int, vdim: int, dvp: int, wq, wk, eps: float, rot: Rotation | None, pos,
+                    gate=None) -> None:
+    """:func:`gqa_finish` with norms over all heads of q (``wq``) and of k (``wk``), a rotation behind them, and ``gate`` fp32 [M, H]
+    receiving the sigmoids of the columns behind v.  ``Hkv`` = 0: the projection has no k and v and the cache stays as it is."""
+    M = slot.numel()
+    if rot is not None and (rot.freq.dtype != torch.float64 or rot.freq.numel() != rot.dims // 2):
+        raise ValueError("rotation frequencies are fp64, one per pair")
+    if gate is not None and gate.stride(0) != H:
+        raise ValueError("gate: a dense [M, H] tensor")
+    _lib.check_rc(_f("artb_gqa_finish_norm")(
+        _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(bias), _lib.ptr(slot), _lib.ptr(cache), cache.shape[-1],
+        cache.shape[0] * cache.shape[1], _lib.ptr(q), q.stride(0), M, H, Hkv, dim, pad(dim, 16), vdim, dvp, _lib.ptr(wq), _lib.ptr(wk), eps,
+        _lib.ptr(rot.freq if rot else None), rot.scale if rot else 1.0, rot.dims if rot else 0, 1 if rot and rot.next else 0, _lib.ptr(pos),
+        _lib.ptr(gate), _st(cache), _lib.stream_ptr()), "gqa_finish_norm")
 
 
 def gqa_gather(cache, block_table, plan: PrefillPlan, Hkv: int, dk: int, dv: int) -> tuple[torch.Tensor, torch.Tensor]:
@@ -381,28 +430,29 @@ def gqa_decode_splits(M: int, ctas_per_row: int, keys: int, sms: int = 148) -> i
     return max(1, min(2 * sms // max(1, M * ctas_per_row), (keys + 4 * GQA_TILE - 1) // (4 * GQA_TILE), 32))
 
 
-def _gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o):
+def _gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate):
     return (_lib.ptr(q), q.stride(0), _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1],
-            cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, chunk, scale, out_scale, _lib.ptr(o), o.stride(0))
+            cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, chunk, scale, softcap, out_scale, *_gate(gate),
+            _lib.ptr(o), o.stride(0))
 
 
 def gqa_decode(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
-               Hkv: int, dim: int, vdim: int, dvp: int, splits: int = 1) -> torch.Tensor:
+               Hkv: int, dim: int, vdim: int, dvp: int, splits: int = 1, softcap: float = 0.0, gate=None) -> torch.Tensor:
     """Rows ``0 .. M - 1`` of ``q`` against their sequences' cached keys; ``o`` [., H * pad(vdim)] gets ``out_scale`` times the
-    result."""
+    result, and times ``gate`` fp32 [M, H]; ``softcap`` > 0 squashes the scores."""
     vpad = pad(vdim)
     ws = torch.empty(M * H * splits * (vpad + 2), dtype=torch.float32, device=o.device) if splits > 1 else None
     _lib.check_rc(_f("artb_gqa_decode")(
-        *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o), vpad, _lib.ptr(ws), splits, M, H, Hkv,
+        *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate), vpad, _lib.ptr(ws), splits, M, H, Hkv,
         pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_decode")
     return o
 
 
 def gqa_attend(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
-               Hkv: int, dim: int, vdim: int, dvp: int) -> torch.Tensor:
+               Hkv: int, dim: int, vdim: int, dvp: int, softcap: float = 0.0, gate=None) -> torch.Tensor:
     """Scalar fp32 form of :func:`gqa_decode`, any head sizes."""
     _lib.check_rc(_f("artb_gqa_attend")(
-        _is32(cache), *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o), pad(vdim), M, H, Hkv,
+        _is32(cache), *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate), pad(vdim), M, H, Hkv,
         pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_attend")
     return o
 

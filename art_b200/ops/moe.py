@@ -16,7 +16,7 @@ from dataclasses import dataclass
 import torch
 
 from . import _lib
-from .gemm import EPI_BF16, EPI_SWIGLU
+from .gemm import EPI_BF16, EPI_RELU2, EPI_SWIGLU
 
 _configured = False
 
@@ -26,7 +26,7 @@ def _k():
     lib = _lib.kernels()
     if not _configured:
         vp, ci, cl = ctypes.c_void_p, ctypes.c_int, ctypes.c_long
-        lib.artb_moe_router.argtypes = [vp, ci, ci, vp, ci, ci, ci, ci, vp, vp, vp, vp]
+        lib.artb_moe_router.argtypes = [vp, ci, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp, vp, vp, vp]
         lib.artb_moe_plan.argtypes = [vp, ci, vp, vp, cl, ci, vp, vp, ci, vp, vp, vp, vp, vp]
         lib.artb_moe_gather.argtypes = [vp, ci, vp, vp, ci, vp, vp, ci, ci, ci, vp]
         lib.artb_moe_gather_f32.argtypes = [vp, ci, vp, vp, vp, ci, ci, ci, vp]
@@ -55,9 +55,10 @@ class RoutePlan:
     counts: torch.Tensor      # int32 [E]
     seg_off: torch.Tensor     # int32 [E + 1]   padded segment offsets (multiples of 128)
     tile_expert: torch.Tensor  # int32 [cap_tiles]
-    pos: torch.Tensor         # int32 [M, k]    row of (token, slot) in the expert-sorted order
+    pos: torch.Tensor         # int32 [M, k]    row of (token, slot) in the expert-sorted order, -1: an output without rows
     row_token: torch.Tensor   # int32 [cap_rows] token of each row, -1 for padding
     row_w: torch.Tensor       # fp32  [cap_rows]
+    gate: torch.Tensor | None = None      # fp32 [M]  sigmoid of the column behind the router's outputs
 
     @property
     def cap_rows(self) -> int:
@@ -72,22 +73,30 @@ def cap_tiles_for(M: int, k: int, E: int) -> int:
     return (M * k + E * 127 + 127) // 128
 
 
-def route(logits: torch.Tensor, k: int, norm_topk: bool, bias: torch.Tensor | None = None, take: bool = False) -> RoutePlan:
+def route(logits: torch.Tensor, k: int, norm_topk: bool, bias: torch.Tensor | None = None, take: bool = False,
+          correction: torch.Tensor | None = None, identity: int = 0, gate: bool = False) -> RoutePlan:
     """Softmax over experts, top-k, (optional) renormalisation, and the expert-sorted row plan.  ``bias`` fp32 [E] is added
-    to the logits first; with ``take`` the logits lie in a workspace that is to be left zero."""
+    to the logits first; with ``take`` the logits lie in a workspace that is to be left zero.
+
+    ``correction`` fp32 [outputs]: the choice goes by softmax + correction, the weights by the softmax (its share of the
+    chosen ones' sum + 1e-20 with ``norm_topk``).  The last ``identity`` outputs have no rows (``pos`` is -1).  ``gate``: one
+    more column, whose sigmoid is ``plan.gate``."""
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
-    M, E = logits.shape
+    M, outputs = logits.shape[0], logits.shape[1] - int(gate)
+    E = outputs - identity
     dev = logits.device
     i32 = dict(dtype=torch.int32, device=dev)
     cap = cap_tiles_for(M, k, E)
     plan = RoutePlan(M, k, E, cap, torch.empty((M, k), **i32), torch.empty((M, k), dtype=torch.float32, device=dev),
                      torch.zeros(E, **i32), torch.empty(E + 1, **i32), torch.empty(cap, **i32),
                      torch.empty((M, k), **i32), torch.empty(cap * 128, **i32),
-                     torch.empty(cap * 128, dtype=torch.float32, device=dev))
+                     torch.empty(cap * 128, dtype=torch.float32, device=dev),
+                     torch.empty(M, dtype=torch.float32, device=dev) if gate else None)
     cursor = torch.empty(E, **i32)
     st = _lib.stream_ptr()
-    _lib.check_rc(_k().artb_moe_router(_lib.ptr(logits), logits.stride(0), 2 if take else 1, _lib.ptr(bias), M, E, k, int(norm_topk), _lib.ptr(plan.topi),
-                                       _lib.ptr(plan.topw), _lib.ptr(plan.counts), st), "moe_router")
+    _lib.check_rc(_k().artb_moe_router(_lib.ptr(logits), logits.stride(0), 2 if take else 1, _lib.ptr(bias), _lib.ptr(correction), M, outputs, E, k,
+                                       int(norm_topk), _lib.ptr(plan.topi), _lib.ptr(plan.topw), _lib.ptr(plan.counts), _lib.ptr(plan.gate), st),
+                  "moe_router")
     _lib.check_rc(_k().artb_moe_plan(_lib.ptr(plan.counts), E, _lib.ptr(plan.topi), _lib.ptr(plan.topw), M, k,
                                      _lib.ptr(plan.seg_off), _lib.ptr(plan.tile_expert), cap, _lib.ptr(cursor),
                                      _lib.ptr(plan.pos), _lib.ptr(plan.row_token), _lib.ptr(plan.row_w), st),
@@ -144,13 +153,14 @@ def router_bwd(logits: torch.Tensor, plan: RoutePlan, dw: torch.Tensor, norm_top
 
 def grouped_gemm(a: torch.Tensor, b: torch.Tensor, plan: RoutePlan, n_per_expert: int, a2: torch.Tensor | None = None,
                  b2: torch.Tensor | None = None, swiglu_out: torch.Tensor | None = None,
-                 out: torch.Tensor | None = None, keep_preact: bool = True) -> torch.Tensor | None:
+                 out: torch.Tensor | None = None, keep_preact: bool = True, relu2: bool = False) -> torch.Tensor | None:
     """``out[rows of e] = a[rows of e] @ b[e*N:(e+1)*N].T (+ a2[rows] @ b2[e*N:(e+1)*N].T)``.  ``keep_preact=False`` with
-    ``swiglu_out``: the pre-activation is not stored.  fp32 operands take the 32-bit product."""
+    ``swiglu_out``: the pre-activation is not stored.  ``relu2``: the product leaves through the square of relu.  fp32 operands
+    take the 32-bit product."""
     rows, K = a.shape
     assert rows == plan.cap_rows and b.shape == (plan.E * n_per_expert, K)
     if a.dtype == torch.float32:
-        if a2 is not None or swiglu_out is not None:
+        if a2 is not None or swiglu_out is not None or relu2:
             raise ValueError("the 32-bit grouped product has no extra operand and no activation")
         if out is None:
             out = torch.empty((rows, n_per_expert), dtype=torch.float32, device=a.device)
@@ -165,7 +175,7 @@ def grouped_gemm(a: torch.Tensor, b: torch.Tensor, plan: RoutePlan, n_per_expert
         _lib.ptr(a), a.stride(0), _lib.ptr(b), b.stride(0), _lib.ptr(a2), a2.stride(0) if a2 is not None else 0,
         _lib.ptr(b2), b2.stride(0) if b2 is not None else 0, K2, _lib.ptr(out), out.stride(0) if out is not None else 0,
         _lib.ptr(swiglu_out), swiglu_out.stride(0) if swiglu_out is not None else 0, _lib.ptr(plan.tile_expert),
-        plan.cap_tiles, plan.E, n_per_expert, K, EPI_SWIGLU if swiglu_out is not None else EPI_BF16,
+        plan.cap_tiles, plan.E, n_per_expert, K, EPI_SWIGLU if swiglu_out is not None else EPI_RELU2 if relu2 else EPI_BF16,
         _lib.ptr(_lib.status_word(a.device)), _lib.stream_ptr())
     _lib.check_rc(rc, "gemm_grouped")
     return out

@@ -69,3 +69,45 @@ def aligned_naselorn():
     return naselorn([lightning(heads=3, dim=128, vdim=72, mlp=dense(304)), parallel(heads=6, kv_heads=2, dim=128, vdim=104, chunk=150, scale=0.09,
                      width=384, blocks=6, conv=4, mlp=moe(12, 4, 96, 144)), lightning(heads=5, dim=48, vdim=80, mlp=moe(9, 2, 80, 64)),
                      parallel(heads=4, kv_heads=1, dim=64, vdim=64, chunk=129, scale=0.125, width=96, blocks=4, conv=2)], vocab=536, width=320, eps=1e-6)
+
+
+# -- Gaborax --------------------------------------------------------------------------------------------------------------
+def relu2_moe(experts=5, identity=3, top=2, ff=28, shared=36):
+    return {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+
+
+def gated_heads(heads=4, kv_heads=2, dim=20, vdim=12, rot=12, base=700.0, scale=0.3, kv_from=None, mlp=None, scaling=None):
+    """Rotate-half attention with a gate per head."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "rot": {"base": base, "dims": rot}, "scale": scale}
+    if scaling:
+        m["rot"]["scaling"] = scaling
+    return {"type": "attention", "mlp": mlp, "mixer": m if kv_from is None else {**m, "kv_from": kv_from}}
+
+
+def yarn(factor=3.0, original=64, fast=12.0, slow=0.8):
+    return {"factor": factor, "original": original, "fast": fast, "slow": slow}
+
+
+def capped(heads=3, kv_heads=3, dim=14, vdim=22, rot=10, base=300.0, scale=0.4, softcap=6.0, scaling=yarn(), kv_from=None, mlp=None):
+    """Attention with neighbouring pairs, biases and squashed scores."""
+    e = gated_heads(heads, kv_heads, dim, vdim, rot, base, scale, kv_from, mlp, scaling)
+    e["mixer"]["softcap"] = softcap
+    return {**e, "type": "attention_2"}
+
+
+def gaborax(layers, vocab=199, width=92, eps=4e-5):
+    return {"architecture": "Gaborax", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
+
+
+def small_gaborax():
+    return gaborax([capped(mlp=relu2_moe()), gated_heads(mlp=relu2_moe(3, 0, 1, 16, 20)), gated_heads(heads=6, mlp=relu2_moe(2, 5, 4, 7, 33), kv_from=1),
+                    capped(heads=2, kv_heads=1, dim=64, vdim=40, rot=64, softcap=3.0), gated_heads(kv_from=1, scale=0.11, base=50.0),
+                    capped(heads=4, kv_heads=1, dim=64, vdim=40, rot=24, kv_from=3, scaling=None, mlp=relu2_moe(4, 1, 3, 24, 8))])
+
+
+def aligned_gaborax():
+    """Sizes near a real model's proportions, still small: several tiles of the tensor-core kernels."""
+    return gaborax([gated_heads(heads=6, kv_heads=2, dim=128, vdim=104, rot=96, scale=0.09, mlp=relu2_moe(12, 4, 4, 96, 144)),
+                    capped(heads=4, kv_heads=4, dim=64, vdim=64, rot=64, scale=0.125, softcap=15.0, mlp=relu2_moe(9, 2, 2, 80, 64)),
+                    gated_heads(heads=6, kv_heads=2, dim=128, vdim=104, rot=96, scale=0.09, kv_from=0, mlp=relu2_moe(6, 1, 3, 64, 80)),
+                    capped(heads=8, kv_heads=1, dim=80, vdim=96, rot=48, scale=0.11, softcap=30.0)], vocab=528, width=304, eps=1e-6)

@@ -408,7 +408,7 @@ def test_mixture_of_experts_alone(experts, top, ff, shared, dtype):
     h = h.to(dtype)
     x = torch.zeros(75, run.dp, device=DEV)
     b = run._pack([_view(tokens(75, 97))])[0]
-    hy.residual_step(x, None, 68, 1e-5, sub=run._mlp_moe(run.cfg.layers[0], run.layers[0], h, b), x_in=torch.zeros_like(x))
+    hy.residual_step(x, None, 68, 1e-5, sub=run._mlp_moe(run.cfg.layers[0], run.layers[0], None, h, b), x_in=torch.zeros_like(x))
     hh = h[:, :68].double().cpu()
     W = {k: t.double() for k, t in w.items()}
     ref = oracle.moe(hh, W, d["layers"][0]["mlp"])

@@ -279,3 +279,37 @@ def test_prefill_plan_covers_every_row_and_window():
         rows += range(r, min(r + PREFILL_ROWS, plan.row_end.tolist()[s]))
     assert rows == list(range(434))
     assert plan_prefill(portions, window=0, device="cpu").key_pos0.tolist() == [0, 0, 0]
+
+
+def test_a_process_that_needs_few_kernels_compiles_few(tmp_path, monkeypatch):
+    """Every kernel a design's front-ends may call lies in the sources its layers ask for; one that is missing all the same
+    is taken from the complete library."""
+    import re
+
+    from art_b200 import build
+    from art_b200.engine.hybrid_runner import KERNEL_SOURCES, kernel_sources
+    from art_b200.models.config import resolve_config
+    from art_b200.ops import _lib
+
+    everything = {p.stem for p in build.kernel_sources()}
+    assert all(v <= everything for v in KERNEL_SOURCES.values())
+    for name in ("nikelix-tiny", "naselorn-tiny", "gaborax-tiny"):
+        assert {"hybrid_rows", "gemm_tcgen05"} <= kernel_sources(resolve_config(name)) < everything
+    assert "linear_scan" not in kernel_sources(resolve_config("gaborax-tiny")) and "linear_scan" in kernel_sources(resolve_config("naselorn-tiny"))
+    exported = {s: p.stem for p in build.kernel_sources() for s in re.findall(r"ARTB_EXPORT \w+ (artb_\w+)\(", p.read_text())}
+    from art_b200.ops import hybrid as hy
+
+    everyone = set().union(*(kernel_sources(resolve_config(n)) for n in ("nikelix-tiny", "naselorn-tiny", "gaborax-tiny")))
+    assert {exported[s] for s in hy._sigs} <= everyone
+
+    class Lib:
+        artb_one = 1
+
+    class Full:
+        artb_two = 2
+
+    monkeypatch.setattr(_lib, "_load", lambda name: Full)
+    part = _lib._Part(Lib)
+    assert part.artb_one == 1 and part.artb_two == 2
+    with pytest.raises(AttributeError):
+        part.artb_three
