@@ -94,7 +94,7 @@ __device__ __forceinline__ float2 position_pair(int pos, double freq) {
   constexpr double TWO_PI = 6.283185307179586476925;
   const double ang = pos * freq;
   float2 r;
-  sincosf(static_cast<float>(ang - rint(ang / TWO_PI) * TWO_PI), &r.x, &r.y);
+  sincosf(static_cast<float>(ang - rint(ang * (1.0 / TWO_PI)) * TWO_PI), &r.x, &r.y);
   return r;
 }
 

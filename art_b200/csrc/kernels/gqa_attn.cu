@@ -86,10 +86,32 @@ __global__ void __launch_bounds__(256) gqa_finish_kernel(const GqaFinish a) {
   for (int j = threadIdx.x; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
 }
 
-// V = 4: dim, vdim and the projection's pitch are multiples of 4, rot of 8
+// n / d without a division, for n * d < 2^32
+struct QuickDiv {
+  unsigned d, m;
+  static QuickDiv by(int d) { return {static_cast<unsigned>(d), d > 1 ? 0xffffffffu / d + 1 : 0u}; }
+  __device__ __forceinline__ int operator()(int n) const { return d > 1 ? static_cast<int>(__umulhi(static_cast<unsigned>(n), m)) : n; }
+};
+
 template <typename T, int V>
-__global__ void __launch_bounds__(256) gqa_finish_norm_kernel(const GqaFinish a) {
-  extern __shared__ __align__(16) float gn_smem[];      // [nq + nk] columns times their norm weights, then [rot / 2] (cos, sin)
+__device__ __forceinline__ void put_vec(T* dst, const float (&y)[V]) {
+  if (V == 4) st4(dst, make_float4(y[0], y[1 % V], y[2 % V], y[3 % V]));
+  else st1(dst, y[0]);
+}
+template <int V>
+__device__ __forceinline__ void get_vec(const float* src, float (&y)[V]) {
+  if (V == 4) {
+    const float4 v = ld4(src);
+    y[0] = v.x, y[1 % V] = v.y, y[2 % V] = v.z, y[3 % V] = v.w;
+  } else {
+    y[0] = *src;
+  }
+}
+
+// V = 4: dim, vdim and the projection's pitch are multiples of 4, rot of 8; everything 16-byte aligned
+template <typename T, int V>
+__global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish a, const QuickDiv by_dim, const QuickDiv by_vdim, const QuickDiv by_units) {
+  extern __shared__ __align__(16) float gn_smem[];      // [nq + nk] columns times their norm weights, then cos [rot / 2], sin [rot / 2]
   __shared__ float red[2][8];
   constexpr int B = 4;                                  // loads of a thread in flight
   pdl_wait();
@@ -101,7 +123,7 @@ __global__ void __launch_bounds__(256) gqa_finish_norm_kernel(const GqaFinish a)
   T* qrow = reinterpret_cast<T*>(a.q) + static_cast<size_t>(m) * a.ldq;
   const int nq = a.H * a.dim, nqk = nq + a.Hkv * a.dim, n = nqk + a.Hkv * a.vdim, half = a.rot >> 1;
   const size_t row = static_cast<size_t>(m) * a.ldp;
-  float2* turn = reinterpret_cast<float2*>(gn_smem + ((nqk + 3) & ~3));
+  float *cosine = gn_smem + ((nqk + 3) & ~3), *sine = cosine + ((half + 3) & ~3);
   float ssq = 0.f, ssk = 0.f;
   for (int c0 = tid * V; c0 < n; c0 += blockDim.x * V * B) {
     float x[B][V];
@@ -120,36 +142,39 @@ __global__ void __launch_bounds__(256) gqa_finish_norm_kernel(const GqaFinish a)
     for (int u = 0; u < B; ++u) {
       const int c = c0 + u * blockDim.x * V;
       if (c >= n) continue;
+      float t[V];
+      if (a.bias) {
+        get_vec(a.bias + c, t);
 #pragma unroll
-      for (int e = 0; e < V; ++e)
-        if (a.bias) x[u][e] += a.bias[c + e];
+        for (int e = 0; e < V; ++e) x[u][e] += t[e];
+      }
       if (c >= nqk) {
         if (slot < 0) continue;
-        T* dst = crow + a.Hkv * a.dk_p + (c - nqk) / a.vdim * a.dv_p + (c - nqk) % a.vdim;
-        if (V == 4) st4(dst, make_float4(x[u][0], x[u][1 % V], x[u][2 % V], x[u][3 % V]));
-        else st1(dst, x[u][0]);
+        const int hd = by_vdim(c - nqk);
+        put_vec(crow + a.Hkv * a.dk_p + hd * (a.dv_p - a.vdim) + c - nqk, x[u]);
         continue;
       }
+      const bool isq = c < nq;
       float s = 0.f;
 #pragma unroll
       for (int e = 0; e < V; ++e) s = fmaf(x[u][e], x[u][e], s);
-      if (c < nq) ssq += s;
-      else ssk += s;
-      const float* w = c < nq ? a.wq : a.wk;
+      ssq += isq ? s : 0.f;
+      ssk += isq ? 0.f : s;
+      const float* w = isq ? a.wq : a.wk;
       if (w) {
-        w += c < nq ? c : c - nq;
+        get_vec(w + (isq ? c : c - nq), t);
 #pragma unroll
-        for (int e = 0; e < V; ++e) x[u][e] *= w[e];
+        for (int e = 0; e < V; ++e) x[u][e] *= t[e];
       }
-      if (V == 4) st4(gn_smem + c, make_float4(x[u][0], x[u][1 % V], x[u][2 % V], x[u][3 % V]));
-      else gn_smem[c] = x[u][0];
+      put_vec(gn_smem + c, x[u]);
     }
   }
   if (a.gate)
     for (int h = tid; h < a.H; h += blockDim.x) a.gate[static_cast<size_t>(m) * a.H + h] = logistic_f(take1(a.p, row + n + h, a.kind));
   for (int i = tid; i < half; i += blockDim.x) {
     const float2 t = position_pair(a.pos[m], a.freq[i]);
-    turn[i] = make_float2(a.rot_scale * t.y, a.rot_scale * t.x);
+    cosine[i] = a.rot_scale * t.y;
+    sine[i] = a.rot_scale * t.x;
   }
   ssq = lane_sum(ssq);
   ssk = lane_sum(ssk);
@@ -160,46 +185,48 @@ __global__ void __launch_bounds__(256) gqa_finish_norm_kernel(const GqaFinish a)
   ssk = lane_sum(lane < nw ? red[1][lane] : 0.f);
   const float rq = a.wq ? 1.f / sqrtf(ssq / nq + a.eps) : 1.f;
   const float rk = a.wk ? 1.f / sqrtf(ssk / max(1, nqk - nq) + a.eps) : 1.f;
-  for (int c = tid * V; c < (slot < 0 ? nq : nqk); c += blockDim.x * V) {
-    const bool isq = c < nq;
-    const int cc = isq ? c : c - nq, hd = cc / a.dim, d = cc - hd * a.dim;
-    const float r = isq ? rq : rk;
-    float y[V];
-    if (V == 4) {
-      const float4 x = ld4(gn_smem + c);
-      if (d >= a.rot) {
-        y[0] = x.x, y[1 % V] = x.y, y[2 % V] = x.z, y[3 % V] = x.w;
-      } else if (a.next) {
-        const float2 t0 = turn[d >> 1], t1 = turn[(d >> 1) + 1];
-        y[0] = x.x * t0.x - x.y * t0.y;
-        y[1 % V] = x.y * t0.x + x.x * t0.y;
-        y[2 % V] = x.z * t1.x - x.w * t1.y;
-        y[3 % V] = x.w * t1.x + x.z * t1.y;
-      } else {
-        const bool lo = d < half;
-        const float4 z = ld4(gn_smem + (lo ? c + half : c - half));
-        const int i = lo ? d : d - half;
-        const float sg = lo ? -1.f : 1.f;
-        const float2 t0 = turn[i], t1 = turn[i + 1], t2 = turn[i + 2], t3 = turn[i + 3];
-        y[0] = fmaf(sg * z.x, t0.y, x.x * t0.x);
-        y[1 % V] = fmaf(sg * z.y, t1.y, x.y * t1.x);
-        y[2 % V] = fmaf(sg * z.z, t2.y, x.z * t2.x);
-        y[3 % V] = fmaf(sg * z.w, t3.y, x.w * t3.x);
+  const int heads = slot < 0 ? a.H : a.H + a.Hkv;       // the heads of q, then those of k
+  auto out = [&](int hd) { return hd < a.H ? qrow + hd * a.dk_p : crow + (hd - a.H) * a.dk_p; };
+  // rotated columns, a unit being V pairs (halves) or the pairs of V columns (neighbours), then the others
+  const int units = a.next ? a.rot / (V == 4 ? 4 : 2) : half / V;
+  for (int j = tid; j < heads * units; j += blockDim.x) {
+    const int hd = by_units(j), i = j - hd * units;
+    const float r = hd < a.H ? rq : rk;
+    const float* src = gn_smem + hd * a.dim;
+    T* dst = out(hd);
+    if (!a.next) {
+      float x[V], z[V], c[V], s[V], y0[V], y1[V];
+      get_vec(src + i * V, x);
+      get_vec(src + half + i * V, z);
+      get_vec(cosine + i * V, c);
+      get_vec(sine + i * V, s);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        y0[e] = (x[e] * c[e] - z[e] * s[e]) * r;
+        y1[e] = (z[e] * c[e] + x[e] * s[e]) * r;
       }
+      put_vec(dst + i * V, y0);
+      put_vec(dst + half + i * V, y1);
+    } else if (V == 4) {
+      const float4 x = ld4(src + i * 4);
+      const float2 c = *reinterpret_cast<const float2*>(cosine + i * 2), s = *reinterpret_cast<const float2*>(sine + i * 2);
+      st4(dst + i * 4, make_float4((x.x * c.x - x.y * s.x) * r, (x.y * c.x + x.x * s.x) * r, (x.z * c.y - x.w * s.y) * r, (x.w * c.y + x.z * s.y) * r));
     } else {
-      const float x = gn_smem[c];
-      y[0] = x;
-      if (d < a.rot) {
-        const bool lo = a.next ? !(d & 1) : d < half;
-        const int step = a.next ? 1 : half, i = a.next ? d >> 1 : lo ? d : d - half;
-        const float z = gn_smem[lo ? c + step : c - step];
-        y[0] = fmaf(lo ? -z : z, turn[i].y, x * turn[i].x);
-      }
+      const float x = src[2 * i], z = src[2 * i + 1], c = cosine[i], s = sine[i];
+      st1(dst + 2 * i, (x * c - z * s) * r);
+      st1(dst + 2 * i + 1, (z * c + x * s) * r);
     }
-    T* dst = (isq ? qrow : crow) + hd * a.dk_p + d;
-    if (V == 4) st4(dst, make_float4(y[0] * r, y[1 % V] * r, y[2 % V] * r, y[3 % V] * r));
-    else st1(dst, y[0] * r);
   }
+  if (a.rot < a.dim)
+    for (int c = tid * V; c < heads * a.dim; c += blockDim.x * V) {
+      const int hd = by_dim(c), d = c - hd * a.dim;
+      if (d < a.rot) continue;
+      float x[V];
+      get_vec(gn_smem + c, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] *= hd < a.H ? rq : rk;
+      put_vec(out(hd) + d, x);
+    }
   const int np = a.dk_p - a.dim;
   for (int j = tid; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
 }
@@ -620,9 +647,12 @@ ARTB_EXPORT int artb_gqa_finish_norm(int f32, void* p, int ldp, int kind, const 
     return ERR_BAD_SHAPE;
   const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status,
                     wq, wk, eps, freq, rot_scale, rot, next, pos, gate};
-  const size_t smem = (static_cast<size_t>((H + Hkv) * dim + 3) / 4 * 4 + rot) * 4;
+  const size_t smem = (static_cast<size_t>((H + Hkv) * dim + 3) / 4 * 4 + (rot / 2 + 3) / 4 * 8) * 4;
   if (smem > 224 * 1024) return ERR_TOO_LARGE;
-  const bool v4 = !((dim | vdim | ldp) & 3) && !(rot & 7) && !(reinterpret_cast<uintptr_t>(p) & 15);
+  const auto aligned = [](const void* x) { return !(reinterpret_cast<uintptr_t>(x) & 15); };
+  const bool v4 = !((dim | vdim | ldp) & 3) && !(rot & 7) && aligned(p) && aligned(bias) && aligned(wq) && aligned(wk);
+  const QuickDiv by_dim = QuickDiv::by(dim), by_vdim = QuickDiv::by(vdim),
+                 by_units = QuickDiv::by(rot ? (next ? rot / (v4 ? 4 : 2) : rot / 2 / (v4 ? 4 : 1)) : 1);
 #define ARTB_GN(T_, V_)                                                                                                        \
   do {                                                                                                                         \
     if (smem > 48 * 1024) {                                                                                                    \
@@ -630,7 +660,8 @@ ARTB_EXPORT int artb_gqa_finish_norm(int f32, void* p, int ldp, int kind, const 
                                                  static_cast<int>(smem));                                                      \
       if (e != cudaSuccess) return static_cast<int>(e);                                                                        \
     }                                                                                                                          \
-    return static_cast<int>(launch_kernel(gqa_finish_norm_kernel<T_, V_>, dim3(M), dim3(256), smem, st, a));                   \
+    return static_cast<int>(launch_kernel(gqa_finish_norm_kernel<T_, V_>, dim3(M), dim3(256), smem, st, a, by_dim, by_vdim,    \
+                                          by_units));                                                                     \
   } while (0)
   if (f32) {
     if (v4) ARTB_GN(float, 4);

@@ -99,19 +99,24 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
     }
   }
   if (a.ex) {
-    for (int s = 0; s < a.ex_k; ++s) {
-      const int er = a.ex_pos[static_cast<size_t>(row) * a.ex_k + s];
-      const float ew = a.ex_w[static_cast<size_t>(row) * a.ex_k + s];
-      const bool self = er < 0 && a.idn;                    // uniform for the CTA
-      if (!self && !index_ok(er, a.ex_rows, a.status)) continue;
-      const T* ep = reinterpret_cast<const T*>(a.ex) + static_cast<size_t>(self ? 0 : er) * a.ldex;
+    auto add = [&](float ew, auto&& row4) {
 #pragma unroll
       for (int i = 0; i < MAXV; ++i) {
         const int v = threadIdx.x + i * blockDim.x;
         if (v < nv) {
-          const float4 e = self ? take4(a.idn, static_cast<size_t>(row) * a.ldidn + v * 4, a.idn_kind) : ld4(ep + v * 4);
+          const float4 e = row4(v * 4);
           y[i] = make_float4(fmaf(ew, e.x, y[i].x), fmaf(ew, e.y, y[i].y), fmaf(ew, e.z, y[i].z), fmaf(ew, e.w, y[i].w));
         }
+      }
+    };
+    for (int s = 0; s < a.ex_k; ++s) {
+      const int er = a.ex_pos[static_cast<size_t>(row) * a.ex_k + s];
+      const float ew = a.ex_w[static_cast<size_t>(row) * a.ex_k + s];
+      if (er < 0 && a.idn) {                                // uniform for the CTA
+        add(ew, [&](int c) { return take4(a.idn, static_cast<size_t>(row) * a.ldidn + c, a.idn_kind); });
+      } else if (index_ok(er, a.ex_rows, a.status)) {
+        const T* ep = reinterpret_cast<const T*>(a.ex) + static_cast<size_t>(er) * a.ldex;
+        add(ew, [&](int c) { return ld4(ep + c); });
       }
     }
   }
