@@ -650,11 +650,11 @@ class Engine:
         return True
 
     def _score(self, toks: list[int], n_prompt: int, adapter: int) -> list[float]:
-        if self.state_slots is None:
+        if not hasattr(self.runner, "score_view"):
             return self.runner.score(toks, n_prompt, adapter)
-        # a recurrent model scores through the cache and the state like any prompt: lend it blocks and a slot
+        # a hybrid model scores through the cache (and the state) like any prompt: lend it blocks (and a slot)
         seq = Sequence(toks, SamplingParams(), adapter, None)
-        blocks, slot = self.bm.alloc(self._blocks_needed(len(toks))), self.state_slots.alloc()
+        blocks, slot = self.bm.alloc(self._blocks_needed(len(toks))), self.state_slots.alloc() if self.state_slots is not None else -1
         seq.blocks, seq.state_slot = blocks or [], -1 if slot is None else slot
         try:
             if blocks is None or slot is None:

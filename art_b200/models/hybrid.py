@@ -196,7 +196,7 @@ def rope_frequencies(s: LayerSpec) -> tuple[list[float], float]:
 
 
 def _known(i: int, what: str, d: dict, keys: tuple[str, ...]) -> None:
-    extra = sorted(set(d) - set(keys))
+    extra = sorted(k for k in set(d) - set(keys) if d[k] is not None)
     if extra:
         raise ValueError(f"layer {i}: {what} key{'s' if len(extra) > 1 else ''} {', '.join(map(repr, extra))} not supported")
 

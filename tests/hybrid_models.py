@@ -73,7 +73,7 @@ def aligned_naselorn():
 
 # -- Gaborax --------------------------------------------------------------------------------------------------------------
 def relu2_moe(experts=5, identity=3, top=2, ff=28, shared=36):
-    return {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+    return {"kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared} if shared else None}
 
 
 def gated_heads(heads=4, kv_heads=2, dim=20, vdim=12, rot=12, base=700.0, scale=0.3, kv_from=None, mlp=None, scaling=None):

@@ -1,5 +1,6 @@
 """Gaborax decoders on the GPU against the plain oracle: each mechanism alone and whole models, in fp32 and bf16, as whole
 prompts, token by token, in portions, in mixed batches and through the engine's own generation."""
+import asyncio
 import json
 import math
 import os
@@ -273,7 +274,7 @@ def test_norms_rotation_gates_and_cache_write_behind_the_projection(H, Hkv, dim,
 
 
 @DTYPES
-@pytest.mark.parametrize("experts,identity,top,ff,shared", [(1, 0, 1, 16, 16), (1, 4, 2, 16, 20), (5, 3, 8, 7, 40), (9, 2, 1, 64, 24), (40, 24, 6, 33, 64), (200, 56, 16, 16, 48)])
+@pytest.mark.parametrize("experts,identity,top,ff,shared", [(1, 0, 1, 16, 16), (1, 4, 2, 16, 20), (5, 3, 8, 7, 40), (9, 2, 1, 64, 24), (40, 24, 6, 33, 64), (200, 56, 16, 16, 48), (6, 2, 3, 20, None)])
 def test_mixture_of_experts_alone(experts, identity, top, ff, shared, dtype):
     """The feed-forward of a layer against the equations; bf16 rows are compared where the choice of experts is no close call."""
     from art_b200.ops import hybrid as hy
@@ -423,6 +424,8 @@ def test_greedy_generation_through_the_engine(dtype):
                 assert float((lp.amax(-1) - mine).max()) < 0.3       # the token taken is the best one or a near-tie
                 assert torch.allclose(torch.tensor(s.logprobs, dtype=torch.float64), mine, atol=0.2)
     assert len(eng.runner._dgraphs) >= 1 and eng.bm.stats()["prefix_hits"] > 0
+    got = asyncio.run(eng.score(prompts[1], seqs[1].output_ids[:6]))
+    assert all(abs(a - b) < (1e-3 if dtype == F32 else 0.1) for a, b in zip(got, seqs[1].logprobs[:6])) and eng.bm.num_free == 40
     sampled = eng.generate_sync(prompts[0], SamplingParams(max_tokens=8, temperature=0.9, top_k=5, top_logprobs=3, seed=1))
     assert len(sampled.output_ids) == 8 and all(len(t) == 3 for t in sampled.top_logprobs)
     eng.runner.close()
