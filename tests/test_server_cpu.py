@@ -281,7 +281,7 @@ def test_health_probe_restarts_a_stopped_engine_until_the_budget_is_spent(long_s
     eng.max_recoveries = 1
 
     async def main():
-        body = {"model": "tiny-base", "messages": [{"role": "user", "content": "hi"}], "max_tokens": 4}
+        body = {"model": "tiny-base", "messages": [{"role": "user", "content": "hi"}], "max_tokens": 4, "min_tokens": 4}
         transport = httpx.ASGITransport(app=srv.app, raise_app_exceptions=False)
         async with httpx.AsyncClient(transport=transport, base_url="http://t",
                                      headers={"Authorization": "Bearer default"}) as c:
