@@ -5,7 +5,7 @@
 namespace artb {
 
 // EPI_RELUGLU: as EPI_SWIGLU with relu as the gate's activation.  EPI_SILU: as EPI_BF16, the first res_cols columns through silu.
-// EPI_RELU2: as EPI_BF16, every column through the square of relu.
+// EPI_RELU2: as EPI_BF16, the first res_cols columns through the square of relu.
 enum GemmEpilogue : int {
   EPI_BF16 = 0, EPI_BF16_RESID = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_SWIGLU_BWD = 4, EPI_RELUGLU = 5, EPI_SILU = 6, EPI_RELU2 = 7
 };
@@ -76,7 +76,7 @@ struct EpiStore {
   int swiglu_bwd = 0;
   int relu_gate = 0;
   int silu_cols = 0;     // columns that leave as silu(acc)
-  int relu2 = 0;         // all columns leave as max(acc, 0)^2
+  int relu2_cols = 0;    // columns that leave as max(acc, 0)^2
   // Global operands of the NEXT 32-column chunk, loaded while the current chunk is converted and stored.
   // Residual (4 pieces): each thread reads its own row.  SwiGLU backward (8 pieces = 128 bytes of gate|up per row):
   // read cooperatively, 8 lanes per row, so that a warp-wide load touches 4 rows x 128 contiguous bytes instead of 32
@@ -219,11 +219,11 @@ struct EpiStore {
         if (gc + j < silu_cols) acc[j] = __float_as_uint(__fdividef(z, 1.f + __expf(-z)));
       }
     }
-    if (relu2) {
+    if (gc < relu2_cols) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         const float z = fmaxf(__uint_as_float(acc[j]), 0.f);
-        acc[j] = __float_as_uint(z * z);
+        if (gc + j < relu2_cols) acc[j] = __float_as_uint(z * z);
       }
     }
     if (out_f32) {

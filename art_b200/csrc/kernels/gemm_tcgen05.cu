@@ -64,7 +64,7 @@ ARTB_EXPORT int artb_pick_bn(int M, int N, int ctas) {
 //   A, B, A2, B2 : bf16 row-major, leading dimensions in elements (multiples of 8), 16-B aligned
 //   K2 == 0      : no extra-K operand (A2/B2 ignored)
 //   epilogue     : GemmEpilogue (EPI_SWIGLU_BWD: H = forward gate|up [M,2N] input, C = d(gate|up) [M,2N] output); R (bf16 [M,res_cols]) is added for EPI_BF16_RESID and, when given, for EPI_SWIGLU;
-//                  H (bf16 [M,N/2]) receives silu(gate)*up for EPI_SWIGLU, relu(gate)*up for EPI_RELUGLU (C may then be null);  res_cols 0 = all N columns; EPI_SILU: its columns
+//                  H (bf16 [M,N/2]) receives silu(gate)*up for EPI_SWIGLU, relu(gate)*up for EPI_RELUGLU (C may then be null);  res_cols 0 = all N columns; EPI_SILU, EPI_RELU2: their columns
 //   bias         : optional fp32 [N], added to the accumulator before any other epilogue step
 //   bn           : tile width 64 / 128 / 192 / 224 / 256 (0 = choose, see artb_pick_bn)
 //   status       : device int32, receives a KernelStatus on a bounded-wait expiry (0 otherwise)
@@ -109,7 +109,8 @@ ARTB_EXPORT int artb_gemm_bf16_tn(const void* A, int lda, const void* B, int ldb
                       reinterpret_cast<__nv_bfloat16*>(H), bias, ldc, ldr, ldh, M, N,              \
                       epilogue == EPI_F32 ? 1 : 0, res_cols > 0 ? res_cols : N,                   \
                       epilogue == EPI_SWIGLU_BWD ? 1 : 0, epilogue == EPI_RELUGLU ? 1 : 0,        \
-                      epilogue == EPI_SILU ? res_cols : 0, epilogue == EPI_RELU2 ? 1 : 0};        \
+                      epilogue == EPI_SILU ? res_cols : 0,                                        \
+                      epilogue == EPI_RELU2 ? (res_cols > 0 ? res_cols : N) : 0};                 \
     return launch_gemm<BN_, ST_>(tA, tB, tA2, tB2, kb_main, kb_extra, M, N, epi, status, max_ctas, \
                                  stream);                                                         \
   }

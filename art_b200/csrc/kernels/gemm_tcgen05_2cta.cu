@@ -43,7 +43,7 @@ static int launch_2cta(const void* A, int lda, const void* B, int ldb, const voi
   EpiStore<BN2> epi{C, reinterpret_cast<const __nv_bfloat16*>(R), reinterpret_cast<__nv_bfloat16*>(H), bias, ldc, ldr,
                       ldh, M, N, epilogue == EPI_F32 ? 1 : 0, res_cols > 0 ? res_cols : N,
                      epilogue == EPI_SWIGLU_BWD ? 1 : 0, epilogue == EPI_RELUGLU ? 1 : 0, epilogue == EPI_SILU ? res_cols : 0,
-                     epilogue == EPI_RELU2 ? 1 : 0};
+                     epilogue == EPI_RELU2 ? (res_cols > 0 ? res_cols : N) : 0};
   SchedPair sched{m_tiles2, n_tiles, pick_group_m(m_tiles2, 2 * GEMM_BM, K), 1, kb_main, kb_main};
   return static_cast<int>(launch_kernel(kern, dim3(2 * clusters), dim3(gemm_pipe_threads<EpiStore<BN2>>()), L::TOTAL, stream,
                                         tA, tB, tA2, tB2, kb_main, kb_extra, sched, epi, status, NoComm{}));

@@ -1,11 +1,13 @@
 // Grouped-query attention over a paged cache with a key mask (window or chunk), value heads of their own size, optionally
-// squashed scores and a factor per row and head.
+// squashed scores, a bias by distance with sigmoid weights instead of a softmax (key_weights.cuh), a factor per row and head
+// or per row and column.
 //
 // A token's cache row is [ keys of the Hkv heads: dk_p each | values of the Hkv heads: dv_p each ], padded with zeros.
 //
 //   gqa_finish_kernel    what follows the q | k | v projection, one CTA per token: biases, cache write, padded queries
-//   gqa_finish_norm_kernel   the same with a norm over all heads of q, and of k, a rotation of the first columns of every head
-//                        (angles reduced in fp64, as for position vectors) and the heads' gates
+//   gqa_finish_norm_kernel   the same with a norm over all heads of q, and of k, or over each head, a rotation of the first
+//                        columns of every head (angles reduced in fp64, as for position vectors) and the heads' or columns'
+//                        gates
 //   gqa_gather_kernel    the cache rows a batch's portions see, contiguous: keys row by row, values transposed, as the
 //                        tcgen05 kernel of latent_prefill_tc.cu wants them (sizes that do not suit it: latent_gather and
 //                        latent_prefill)
@@ -20,6 +22,7 @@
 #include "bounds_check.cuh"
 #include "host_utils.h"
 #include "key_mask.cuh"
+#include "key_weights.cuh"
 #include "mma_tile.cuh"
 #include "row_io.cuh"
 #include "softcap.cuh"
@@ -39,13 +42,17 @@ struct GqaFinish {
   int H, Hkv, dim, dk_p, vdim, dv_p;      // Hkv = 0: q alone (keys and values are another layer's)
   int* status;
   // gqa_finish_norm_kernel alone
-  const float *wq, *wk;     // fp32 norm weights over all heads of q and of k, or null
+  const float *wq, *wk;     // fp32 norm weights over all heads of q and of k, or null; per_head: one head's, shared by all
+  int per_head;             // a norm over each head instead
+  const float* q_scale;     // fp32 [H] factor of every query head (per_head alone), or null
   float eps;
   const double* freq;       // angle of pair i of position p: p * freq[i], rot / 2 pairs
   float rot_scale;          // factor of sine and cosine
   int rot, next;            // rotated columns of a head; partner: the neighbour (next) or rot / 2 columns further
   const int* pos;
   float* gate;              // fp32 [M, H]: the sigmoid of the columns behind v, or null
+  void* cols;               // T [M, ldcols], heads of colp: the H * vdim columns behind v, or null
+  int ldcols, colp;
 };
 
 template <typename T, int V>
@@ -161,12 +168,25 @@ __global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish
       ssq += isq ? s : 0.f;
       ssk += isq ? 0.f : s;
       const float* w = isq ? a.wq : a.wk;
-      if (w) {
+      if (w && !a.per_head) {
         get_vec(w + (isq ? c : c - nq), t);
 #pragma unroll
         for (int e = 0; e < V; ++e) x[u][e] *= t[e];
       }
       put_vec(gn_smem + c, x[u]);
+    }
+  }
+  if (a.cols) {
+    T* g = reinterpret_cast<T*>(a.cols) + static_cast<size_t>(m) * a.ldcols;
+    for (int c = tid * V; c < a.H * a.vdim; c += blockDim.x * V) {
+      float x[V];
+      if (V == 4) {
+        const float4 v = take4(a.p, row + n + c, a.kind);
+        x[0] = v.x, x[1 % V] = v.y, x[2 % V] = v.z, x[3 % V] = v.w;
+      } else {
+        x[0] = take1(a.p, row + n + c, a.kind);
+      }
+      put_vec(g + by_vdim(c) * (a.colp - a.vdim) + c, x);
     }
   }
   if (a.gate)
@@ -176,16 +196,43 @@ __global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish
     cosine[i] = a.rot_scale * t.y;
     sine[i] = a.rot_scale * t.x;
   }
-  ssq = lane_sum(ssq);
-  ssk = lane_sum(ssk);
   const int warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
-  if (lane == 0) red[0][warp] = ssq, red[1][warp] = ssk;
-  __syncthreads();
-  ssq = lane_sum(lane < nw ? red[0][lane] : 0.f);
-  ssk = lane_sum(lane < nw ? red[1][lane] : 0.f);
-  const float rq = a.wq ? 1.f / sqrtf(ssq / nq + a.eps) : 1.f;
-  const float rk = a.wk ? 1.f / sqrtf(ssk / max(1, nqk - nq) + a.eps) : 1.f;
   const int heads = slot < 0 ? a.H : a.H + a.Hkv;       // the heads of q, then those of k
+  float rq = 1.f, rk = 1.f;
+  if (a.per_head) {                                     // a warp norms a head where it lies
+    __syncthreads();
+    for (int hd = warp; hd < heads; hd += nw) {
+      float* x = gn_smem + hd * a.dim;
+      const float* w = hd < a.H ? a.wq : a.wk;
+      float ss = 0.f;
+      for (int c = lane * V; c < a.dim; c += 32 * V) {
+        float y[V];
+        get_vec(x + c, y);
+#pragma unroll
+        for (int e = 0; e < V; ++e) ss = fmaf(y[e], y[e], ss);
+      }
+      float r = 1.f / sqrtf(lane_sum(ss) / a.dim + a.eps);
+      if (hd < a.H && a.q_scale) r *= a.q_scale[hd];
+      for (int c = lane * V; c < a.dim; c += 32 * V) {
+        float y[V], g[V];
+        get_vec(x + c, y);
+        get_vec(w + c, g);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] *= r * g[e];
+        put_vec(x + c, y);
+      }
+    }
+    __syncthreads();
+  } else {
+    ssq = lane_sum(ssq);
+    ssk = lane_sum(ssk);
+    if (lane == 0) red[0][warp] = ssq, red[1][warp] = ssk;
+    __syncthreads();
+    ssq = lane_sum(lane < nw ? red[0][lane] : 0.f);
+    ssk = lane_sum(lane < nw ? red[1][lane] : 0.f);
+    if (a.wq) rq = 1.f / sqrtf(ssq / nq + a.eps);
+    if (a.wk) rk = 1.f / sqrtf(ssk / max(1, nqk - nq) + a.eps);
+  }
   auto out = [&](int hd) { return hd < a.H ? qrow + hd * a.dk_p : crow + (hd - a.H) * a.dk_p; };
   // rotated columns, a unit being V pairs (halves) or the pairs of V columns (neighbours), then the others
   const int units = a.next ? a.rot / (V == 4 ? 4 : 2) : half / V;
@@ -308,6 +355,10 @@ struct GqaAttend {
   float out_scale;
   const float* gate;        // fp32 [M][ldg] factor per row and head, or null
   int ldg;
+  int sigmoid;              // weights are sigmoids of score + bias, not a softmax
+  DistanceBias bias;        // of every query head (sigmoid weights)
+  const void* cols;         // T [M][ldcols] gate logits of the result's columns, heads of colp, or null
+  int ldcols, colp;
   void* o;                  // T [M, ldo], heads of vp; padding columns zero
   int ldo, vp;
   float* ws;                // [M][H][splits][dv_p + 2]
@@ -323,7 +374,8 @@ constexpr int GD_KT = 32;   // keys per warp tile
 template <int DK, int DV>
 constexpr int gqa_decode_smem() { return (16 * (DK + 8) + 4 * GD_KT * (DK + 8 + DV + 8)) * 2 + 2 * 4 * 16 * 4; }
 
-template <int DK, int DV>
+// SIG: sigmoid weights
+template <int DK, int DV, bool SIG>
 __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
   constexpr int LK = DK + 8, LV = DV + 8, WARP_ELEMS = GD_KT * (LK + LV);
   static_assert(16 * DV * 4 <= WARP_ELEMS * 2, "a warp's accumulators must fit its staging area");
@@ -364,6 +416,15 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
   float mx[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  const float* tab[2];                                 // bias of the thread's two heads, and what it is far away
+  float far[2];
+  if (SIG) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      tab[e] = a.bias.head(h0 + min(g + 8 * e, ng - 1));
+      far[e] = a.bias.last(tab[e]);
+    }
+  }
   __nv_bfloat16 *wK = sKV + warp * WARP_ELEMS, *wV = wK + GD_KT * LK;
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + hk * a.dk_p;
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(a.cache) + a.Hkv * a.dk_p + hk * a.dv_p;
@@ -411,33 +472,49 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
         mma_bf16(s[np * 2 + 1], qf[ks], b[2], b[3]);
       }
     uint32_t pf[2][4];
+    if (SIG) {
+      const bool near = !a.bias.beyond(p, min(k0 + GD_KT, len) - 1);
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      float mn = mx[e];
+      for (int e = 0; e < 2; ++e)
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+        for (int i = 0; i < 4; ++i) {
+          float w[2];
 #pragma unroll
-        for (int j = 0; j < 2; ++j) {
-          float& x = s[i][2 * e + j];
-          x = k0 + i * 8 + 2 * t + j < len ? a.score(x) : -INFINITY;
-          mn = fmaxf(mn, x);
+          for (int j = 0; j < 2; ++j) {
+            const int kt = k0 + i * 8 + 2 * t + j;
+            w[j] = kt < len ? sigmoid_base2(a.score(s[i][2 * e + j]) + (near ? a.bias.at(tab[e], p - kt) : far[e])) : 0.f;
+          }
+          pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(w[0], w[1]);
         }
-      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
-      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));
-      const float ms = mn == -INFINITY ? 0.f : mn, corr = exp2f(mx[e] - ms);
-      mx[e] = mn;
-      float sum = 0.f;
+    } else {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const float p0 = exp2f(s[i][2 * e] - ms), p1 = exp2f(s[i][2 * e + 1] - ms);
-        sum += p0 + p1;
-        pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(p0, p1);
-      }
-      l[e] = l[e] * corr + sum;
+      for (int e = 0; e < 2; ++e) {
+        float mn = mx[e];
 #pragma unroll
-      for (int i = 0; i < DV / 8; ++i) {
-        acc[i][2 * e] *= corr;
-        acc[i][2 * e + 1] *= corr;
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 2; ++j) {
+            float& x = s[i][2 * e + j];
+            x = k0 + i * 8 + 2 * t + j < len ? a.score(x) : -INFINITY;
+            mn = fmaxf(mn, x);
+          }
+        mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
+        mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));
+        const float ms = mn == -INFINITY ? 0.f : mn, corr = exp2f(mx[e] - ms);
+        mx[e] = mn;
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float p0 = exp2f(s[i][2 * e] - ms), p1 = exp2f(s[i][2 * e + 1] - ms);
+          sum += p0 + p1;
+          pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(p0, p1);
+        }
+        l[e] = l[e] * corr + sum;
+#pragma unroll
+        for (int i = 0; i < DV / 8; ++i) {
+          acc[i][2 * e] *= corr;
+          acc[i][2 * e + 1] *= corr;
+        }
       }
     }
 #pragma unroll
@@ -451,6 +528,11 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
       }
     __syncwarp();
   }
+  if (SIG) {                                           // nothing to rescale; the first part alone counts as the sum
+#pragma unroll
+    for (int e = 0; e < 2; ++e) mx[e] = 0.f, l[e] = split == 0 && warp == 0 && t == 0 ? 1.f : 0.f;
+  }
+  const auto cols = ColumnGate<__nv_bfloat16>::of(a.cols, a.ldcols, a.colp, a.vdim);
   auto warp_acc = [&](int w) { return reinterpret_cast<float*>(sKV + w * WARP_ELEMS); };
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
@@ -481,7 +563,7 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
     }
     if (a.splits == 1) {
       __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.o) + static_cast<size_t>(m) * a.ldo + (h0 + r) * a.vp;
-      out[d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h0 + r) : 0.f);
+      out[d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h0 + r) * cols(m, h0 + r, d) : 0.f);
     } else {
       float* w = a.ws + ((static_cast<size_t>(m) * a.H + h0 + r) * a.splits + split) * (a.vp + 2);
       w[d] = o;
@@ -497,6 +579,7 @@ __global__ void __launch_bounds__(128) gqa_merge_kernel(const GqaAttend a) {
   pdl_wait();
   pdl_launch_dependents();
   const int m = blockIdx.x, h = blockIdx.y;
+  const auto cols = ColumnGate<__nv_bfloat16>::of(a.cols, a.ldcols, a.colp, a.vdim);
   const float* base = a.ws + (static_cast<size_t>(m) * a.H + h) * a.splits * (a.vp + 2);
   float mm = -INFINITY;
   for (int s = 0; s < a.splits; ++s) mm = fmaxf(mm, base[s * (a.vp + 2) + a.vp]);
@@ -509,7 +592,7 @@ __global__ void __launch_bounds__(128) gqa_merge_kernel(const GqaAttend a) {
         ls += w[a.vp + 1] * sc;
         o += w[d] * sc;
       }
-    reinterpret_cast<__nv_bfloat16*>(a.o)[static_cast<size_t>(m) * a.ldo + h * a.vp + d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h) : 0.f);
+    reinterpret_cast<__nv_bfloat16*>(a.o)[static_cast<size_t>(m) * a.ldo + h * a.vp + d] = __float2bfloat16(ls > 0.f ? o / ls * a.factor(m, h) * cols(m, h, d) : 0.f);
   }
 }
 
@@ -554,20 +637,28 @@ __global__ void __launch_bounds__(128) gqa_attend_kernel(const GqaAttend a) {
         if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       }
     }
-    float tm = s;
+    float corr = 1.f, e;
+    if (a.sigmoid) {
+      e = s == -INFINITY ? 0.f : 1.f / (1.f + exp2f(-fmaf(s, KW_LOG2E, a.bias.at(a.bias.head(h), p - j))));
+      sp[tid] = e;
+      srow[tid] = cr;
+      __syncthreads();
+    } else {
+      float tm = s;
 #pragma unroll
-    for (int x = 16; x > 0; x >>= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, x));
-    if ((tid & 31) == 0) red[tid >> 5] = tm;
-    __syncthreads();
-    tm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-    const float mn = fmaxf(mx, tm);
-    if (mn == -INFINITY) continue;           // uniform: no usable key so far
-    const float corr = mx == -INFINITY ? 0.f : expf(mx - mn);
-    const float e = s == -INFINITY ? 0.f : expf(s - mn);
-    mx = mn;
-    sp[tid] = e;
-    srow[tid] = cr;
-    sum = sum * corr + cta_sum(e, red);      // its barriers publish sp / srow
+      for (int x = 16; x > 0; x >>= 1) tm = fmaxf(tm, __shfl_xor_sync(0xffffffffu, tm, x));
+      if ((tid & 31) == 0) red[tid >> 5] = tm;
+      __syncthreads();
+      tm = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+      const float mn = fmaxf(mx, tm);
+      if (mn == -INFINITY) continue;           // uniform: no usable key so far
+      corr = mx == -INFINITY ? 0.f : expf(mx - mn);
+      e = s == -INFINITY ? 0.f : expf(s - mn);
+      mx = mn;
+      sp[tid] = e;
+      srow[tid] = cr;
+      sum = sum * corr + cta_sum(e, red);      // its barriers publish sp / srow
+    }
     const int nk = min(KT, len - k0);
 #pragma unroll
     for (int i = 0; i < OV; ++i) {
@@ -580,35 +671,37 @@ __global__ void __launch_bounds__(128) gqa_attend_kernel(const GqaAttend a) {
       }
     }
   }
-  const float inv = sum > 0.f ? a.factor(m, h) / sum : 0.f;
+  const float inv = a.sigmoid ? a.factor(m, h) : sum > 0.f ? a.factor(m, h) / sum : 0.f;
+  const auto cols = ColumnGate<T>::of(a.cols, a.ldcols, a.colp, a.vdim);
   T* o = reinterpret_cast<T*>(a.o) + static_cast<size_t>(m) * a.ldo + h * a.vp;
 #pragma unroll
   for (int i = 0; i < OV; ++i) {
     const int d = tid + i * 128;
-    if (d < a.vp) st1(o + d, acc[i] * inv);
+    if (d < a.vp) st1(o + d, acc[i] * inv * cols(m, h, d));
   }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool SIG>
 static int launch_gqa_decode(const GqaAttend& a, int M, cudaStream_t st) {
   constexpr int smem = gqa_decode_smem<DK, DV>();
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(gqa_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(gqa_decode_kernel<DK, DV, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = true;
   }
   const int groups = (a.H / a.Hkv + 15) / 16;
-  cudaError_t e = launch_kernel(gqa_decode_kernel<DK, DV>, dim3(M, a.Hkv * groups, a.splits), dim3(128), smem, st, a);
+  cudaError_t e = launch_kernel(gqa_decode_kernel<DK, DV, SIG>, dim3(M, a.Hkv * groups, a.splits), dim3(128), smem, st, a);
   if (e == cudaSuccess && a.splits > 1) e = launch_kernel(gqa_merge_kernel, dim3(M, a.H), dim3(128), 0, st, a);
   return static_cast<int>(e);
 }
 
 static bool gqa_ok(const GqaAttend& a, int M) {
   return a.H > 0 && a.H <= 65535 && a.Hkv > 0 && a.H % a.Hkv == 0 && a.block_size > 0 && a.ldc >= a.Hkv * (a.dk_p + a.dv_p) && a.vp >= a.vdim &&
-         a.dv_p >= a.vp && a.ldo >= a.H * a.vp && a.ldq >= a.H * a.dk_p;
+         a.dv_p >= a.vp && a.ldo >= a.H * a.vp && a.ldq >= a.H * a.dk_p && (!a.sigmoid || (a.bias.tab && a.bias.n > 0)) &&
+         (!a.cols || (a.colp >= a.vdim && a.ldcols >= a.H * a.colp - (a.colp - a.vdim)));
 }
 
 }  // namespace artb
@@ -622,7 +715,7 @@ ARTB_EXPORT int artb_gqa_finish(int f32, void* p, int ldp, int kind, const float
   if (H <= 0 || Hkv <= 0 || H % Hkv || dk_p < dim || dv_p < vdim || ldc < Hkv * (dk_p + dv_p) || ldq < H * dk_p || ((dk_p | dv_p | ldc | ldq) & 3))
     return ERR_BAD_SHAPE;
   const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status,
-                    nullptr, nullptr, 0.f, nullptr, 1.f, 0, 0, nullptr, nullptr};
+                    nullptr, nullptr, 0, nullptr, 0.f, nullptr, 1.f, 0, 0, nullptr, nullptr, nullptr, 0, 0};
   const bool v4 = !((dim | vdim | ldp) & 3) && !(reinterpret_cast<uintptr_t>(p) & 15);
 #define ARTB_GF(T_, V_) return static_cast<int>(launch_kernel(gqa_finish_kernel<T_, V_>, dim3(M), dim3(256), 0, st, a))
   if (f32) {
@@ -634,23 +727,27 @@ ARTB_EXPORT int artb_gqa_finish(int f32, void* p, int ldp, int kind, const float
 #undef ARTB_GF
 }
 
-// As artb_gqa_finish, with norms (wq, wk), the rotation of the first `rot` columns of every head of q and k, and gates; Hkv = 0: the
+// As artb_gqa_finish, with norms (wq, wk; per_head: over each head, q_scale its factor), the rotation of the first `rot` columns
+// of every head of q and k, and gates: of the heads, or the column gates' logits (cols), one or the other; Hkv = 0: the
 // projection holds q (and gate) columns alone and the cache is not touched.
 ARTB_EXPORT int artb_gqa_finish_norm(int f32, void* p, int ldp, int kind, const float* bias, const int* slot, void* cache, int ldc,
                                      long num_slots, void* q, int ldq, int M, int H, int Hkv, int dim, int dk_p, int vdim, int dv_p,
-                                     const float* wq, const float* wk, float eps, const double* freq, float rot_scale, int rot, int next,
-                                     const int* pos, float* gate, int* status, cudaStream_t st) {
+                                     const float* wq, const float* wk, int per_head, const float* q_scale, float eps, const double* freq,
+                                     float rot_scale, int rot, int next, const int* pos, float* gate, void* cols, int ldcols, int colp,
+                                     int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   if (H <= 0 || Hkv < 0 || (Hkv && H % Hkv) || dim <= 0 || vdim <= 0 || dk_p < dim || dv_p < vdim || (Hkv && ldc < Hkv * (dk_p + dv_p)) ||
       ldq < H * dk_p || ((dk_p | dv_p | ldc | ldq) & 3) || (rot & 1) || rot < 0 || rot > dim || (rot && (!freq || !pos)) ||
-      ldp < H * dim + Hkv * (dim + vdim) + (gate ? H : 0))
+      ldp < H * dim + Hkv * (dim + vdim) + (gate ? H : cols ? H * vdim : 0) || (gate && cols) || (cols && (colp < vdim || ldcols < H * colp)) ||
+      (per_head && (!wq || (Hkv && !wk))) || (q_scale && !per_head))
     return ERR_BAD_SHAPE;
   const GqaFinish a{p, ldp, kind, bias, slot, cache, ldc, num_slots, q, ldq, H, Hkv, dim, dk_p, vdim, dv_p, status,
-                    wq, wk, eps, freq, rot_scale, rot, next, pos, gate};
+                    wq, wk, per_head, q_scale, eps, freq, rot_scale, rot, next, pos, gate, cols, ldcols, colp};
   const size_t smem = (static_cast<size_t>((H + Hkv) * dim + 3) / 4 * 4 + (rot / 2 + 3) / 4 * 8) * 4;
   if (smem > 224 * 1024) return ERR_TOO_LARGE;
   const auto aligned = [](const void* x) { return !(reinterpret_cast<uintptr_t>(x) & 15); };
-  const bool v4 = !((dim | vdim | ldp) & 3) && !(rot & 7) && aligned(p) && aligned(bias) && aligned(wq) && aligned(wk);
+  const bool v4 = !((dim | vdim | ldp) & 3) && !(rot & 7) && aligned(p) && aligned(bias) && aligned(wq) && aligned(wk) &&
+                  !((ldcols | colp) & 3) && aligned(cols);
   const QuickDiv by_dim = QuickDiv::by(dim), by_vdim = QuickDiv::by(vdim),
                  by_units = QuickDiv::by(rot ? (next ? rot / (v4 ? 4 : 2) : rot / 2 / (v4 ? 4 : 1)) : 1);
 #define ARTB_GN(T_, V_)                                                                                                        \
@@ -689,38 +786,45 @@ ARTB_EXPORT int artb_gqa_gather(const void* cache, int ldc, const int* block_tab
   return static_cast<int>(cudaGetLastError());
 }
 
+// sigmoid: weights sigmoid(score + bias) with bias fp32 [H][n_bias + 2 * DistanceBias::PAD]; cols: column gates (key_weights.cuh).
 // Rows 0 .. M - 1, each its own query; bf16, dk_p and dv_p multiples of 8 up to 256.  splits > 1: ws fp32 [M * H * splits * (vp + 2)].
 ARTB_EXPORT int artb_gqa_decode(const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
                                 int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
-                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp,
-                                float* ws, int splits, int M, int H,
+                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, int sigmoid,
+                                const float* bias, int n_bias, const void* cols, int ldcols, int colp, void* o, int ldo, int vp, float* ws, int splits, int M, int H,
                                 int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale, softcap,
-                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, o, ldo, vp, ws, splits, H, Hkv, dk_p, vdim, dv_p, status};
+                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, sigmoid, {bias, n_bias}, cols, ldcols, colp, o, ldo, vp, ws, splits, H, Hkv, dk_p, vdim, dv_p, status};
   if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc | ldq) & 7) || splits < 1 || splits > 65535 || (splits > 1 && !ws)) return ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return ERR_BAD_ALIGN;
-#define ARTB_GD(K_)                                                   \
+#define ARTB_GD(K_, S_)                                               \
   do {                                                                \
-    if (dv_p <= 64) return launch_gqa_decode<K_, 64>(a, M, st);       \
-    if (dv_p <= 128) return launch_gqa_decode<K_, 128>(a, M, st);     \
-    if (dv_p <= 256) return launch_gqa_decode<K_, 256>(a, M, st);     \
+    if (dv_p <= 64) return launch_gqa_decode<K_, 64, S_>(a, M, st);   \
+    if (dv_p <= 128) return launch_gqa_decode<K_, 128, S_>(a, M, st); \
+    if (dv_p <= 256) return launch_gqa_decode<K_, 256, S_>(a, M, st); \
     return ERR_TOO_LARGE;                                             \
   } while (0)
-  if (dk_p <= 64) ARTB_GD(64);
-  if (dk_p <= 128) ARTB_GD(128);
-  if (dk_p <= 256) ARTB_GD(256);
+  if (sigmoid) {
+    if (dk_p <= 64) ARTB_GD(64, true);
+    if (dk_p <= 128) ARTB_GD(128, true);
+    if (dk_p <= 256) ARTB_GD(256, true);
+    return ERR_TOO_LARGE;
+  }
+  if (dk_p <= 64) ARTB_GD(64, false);
+  if (dk_p <= 128) ARTB_GD(128, false);
+  if (dk_p <= 256) ARTB_GD(256, false);
 #undef ARTB_GD
   return ERR_TOO_LARGE;
 }
 
 ARTB_EXPORT int artb_gqa_attend(int f32, const void* q, int ldq, const void* cache, int ldc, const int* block_table, int max_blocks,
                                 int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx, int window,
-                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp,
-                                int M, int H, int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
+                                int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, int sigmoid,
+                                const float* bias, int n_bias, const void* cols, int ldcols, int colp, void* o, int ldo, int vp, int M, int H, int Hkv, int dk_p, int vdim, int dv_p, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   const GqaAttend a{q, ldq, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, {window, chunk}, scale, softcap,
-                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, o, ldo, vp, nullptr, 1, H, Hkv, dk_p, vdim, dv_p, status};
+                    ScoreScale::of(scale, softcap), out_scale, gate, ldg, sigmoid, {bias, n_bias}, cols, ldcols, colp, o, ldo, vp, nullptr, 1, H, Hkv, dk_p, vdim, dv_p, status};
   if (!gqa_ok(a, M) || ((dk_p | dv_p | ldc) & 3) || vp > 1024 || dk_p > 8192) return ERR_BAD_SHAPE;
   const size_t smem = static_cast<size_t>(dk_p) * 4;
   return static_cast<int>(f32 ? launch_kernel(gqa_attend_kernel<float>, dim3(M, H), dim3(128), smem, st, a)

@@ -5,8 +5,12 @@
 //                        without w_post: x = x + mult * y          (or x = mult * table[token] + position vector)
 //                        y may have a factor per row, a bias and the weighted rows of a token's experts (or of the
 //                        sublayer's input, for experts that are the identity) added to it
+//                        and the sum a gate per column, sigmoid(logits + bias)
 //                        depth average: x <- sum_j weight[j] X_j over the results X_j of all layers so far
 //                        h = RMSNorm(x) w_next, or x               (operand of the next matrix product)
+//   stream_step        the same with hyper-connections: the residual stream has several copies x_s, and a boundary mixes them
+//                        x_t <- sum_s mix[s][t] x_s + out[t] * y   (all at once from the old ones)
+//                        h = RMSNorm(sum_t in[t] x_t) w_next
 //   norm_shift_mix     h = RMSNorm(x) w; the inputs h + (h' - h) mu_s of a token-shifted mixer, h' being the h of the
 //                      token before (from the sequence's state at the start of a portion)
 //   poly_norm          a N(z) + b N(z^2) + c N(z^3) + e, N(v) = v / rms(v)
@@ -66,16 +70,18 @@ struct ResidualArgs {
   int d, dp;
   float eps;
   int* status;
+  void* rg;                // logits [rows, ldrg] of rg_kind of a gate on the result's columns, or null
+  int ldrg, rg_kind;
+  const float* rg_b;       // fp32 [dp] added to them
+  // stream_step_kernel alone
+  const float* coef;       // mix [n_in][n_out] | out [n_out] | in of the next sublayer [n_out]
+  int n_in, n_out;         // copies of the stream before (x_in: rows of n_in * dp columns) and behind the step (x_out)
+  int ldxi;
 };
 
+// The sublayer's result (or the embedding row) of row `row`, four columns per thread and vector; `y` of columns past the row is zero.
 template <typename T, int MAXV>
-__global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a) {
-  __shared__ float red[32];
-  pdl_wait();
-  pdl_launch_dependents();
-  const int row = blockIdx.x, nv = a.dp >> 2;
-  float4 y[MAXV];
-  float ss = 0.f;
+__device__ __forceinline__ void sublayer_result(const ResidualArgs& a, int row, int nv, float4 (&y)[MAXV]) {
   long tok = 0;
   if (a.tokens) {
     tok = a.tokens[row];
@@ -120,6 +126,51 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
       }
     }
   }
+  if (a.rg) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nv) {
+        const float4 z = take4(a.rg, static_cast<size_t>(row) * a.ldrg + v * 4, a.rg_kind), b = ld4(a.rg_b + v * 4);
+        y[i] = make_float4(y[i].x * logistic_f(z.x + b.x), y[i].y * logistic_f(z.y + b.y), y[i].z * logistic_f(z.z + b.z), y[i].w * logistic_f(z.w + b.w));
+      }
+    }
+  }
+}
+
+// h = RMSNorm(x) w_next, or x
+template <typename T, int MAXV>
+__device__ __forceinline__ void write_operand(const ResidualArgs& a, int row, int nv, const float4 (&x)[MAXV], float ss, float* red) {
+  T* h = reinterpret_cast<T*>(a.h) + static_cast<size_t>(row) * a.ldh;
+  if (!a.w_next) {
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nv) st4(h + v * 4, x[i]);
+    }
+    return;
+  }
+  ss = cta_sum(ss, red);
+  const float r = 1.f / sqrtf(ss / a.d + a.eps);
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nv) {
+      const float4 w = ld4(a.w_next + v * 4);
+      st4(h + v * 4, make_float4(x[i].x * r * w.x, x[i].y * r * w.y, x[i].z * r * w.z, x[i].w * r * w.w));
+    }
+  }
+}
+
+template <typename T, int MAXV>
+__global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, nv = a.dp >> 2;
+  float4 y[MAXV];
+  float ss = 0.f;
+  sublayer_result<T, MAXV>(a, row, nv, y);
   float r = 1.f;
   if (a.w_post) {
 #pragma unroll
@@ -175,26 +226,68 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
       ss += sq4(x);
     }
   }
-  if (!a.h) return;            // uniform for the grid
-  T* h = reinterpret_cast<T*>(a.h) + static_cast<size_t>(row) * a.ldh;
-  if (!a.w_next) {
-#pragma unroll
-    for (int i = 0; i < MAXV; ++i) {
-      const int v = threadIdx.x + i * blockDim.x;
-      if (v < nv) st4(h + v * 4, y[i]);
+  if (a.h) write_operand<T, MAXV>(a, row, nv, y, ss, red);      // uniform for the grid
+}
+
+// Hyper-connections.  NS: the most copies on either side; the copies of a vector are read together, several vectors in flight.
+template <typename T, int MAXV, int NS>
+__global__ void __launch_bounds__(256) stream_step_kernel(const ResidualArgs a) {
+  constexpr int B = MAXV * NS <= 16 ? MAXV : NS >= 16 ? 1 : 16 / NS;
+  __shared__ float red[32];
+  __shared__ float sc[NS * NS + 2 * NS];     // mix [NS][NS] (zeros where there is no copy) | out | in
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row = blockIdx.x, nv = a.dp >> 2;
+  for (int i = threadIdx.x; i < NS * NS + 2 * NS; i += blockDim.x) {
+    const int s = i / NS, t = i % NS;
+    float c = 0.f;
+    if (t < a.n_out) {
+      if (s < a.n_in) c = a.coef[s * a.n_out + t];
+      else if (s >= NS) c = a.coef[(a.n_in + s - NS) * a.n_out + t];
     }
-    return;
+    sc[i] = c;
   }
-  ss = cta_sum(ss, red);
-  const float r2 = 1.f / sqrtf(ss / a.d + a.eps);
+  float4 y[MAXV];
+  float ss = 0.f;
+  sublayer_result<T, MAXV>(a, row, nv, y);
+  __syncthreads();
+  const float* xi = a.x_in + static_cast<size_t>(row) * a.ldxi;
+  float* xo = a.x_out + static_cast<size_t>(row) * a.ldx;
 #pragma unroll
-  for (int i = 0; i < MAXV; ++i) {
-    const int v = threadIdx.x + i * blockDim.x;
-    if (v < nv) {
-      const float4 w = ld4(a.w_next + v * 4);
-      st4(h + v * 4, make_float4(y[i].x * r2 * w.x, y[i].y * r2 * w.y, y[i].z * r2 * w.z, y[i].w * r2 * w.w));
+  for (int i0 = 0; i0 < MAXV; i0 += B) {
+    float4 x[B][NS];
+#pragma unroll
+    for (int i = 0; i < B; ++i) {
+      const int v = threadIdx.x + (i0 + i) * blockDim.x;
+#pragma unroll
+      for (int s = 0; s < NS; ++s)
+        x[i][s] = v < nv && s < a.n_in ? ld4(xi + s * a.dp + v * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < B; ++i) {
+      const int v = threadIdx.x + (i0 + i) * blockDim.x;
+      float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (v < nv) {
+        const float4 yv = y[i0 + i];
+#pragma unroll
+        for (int t = 0; t < NS; ++t)
+          if (t < a.n_out) {
+            const float o = sc[NS * NS + t], in = sc[NS * NS + NS + t];
+            float4 n = make_float4(o * yv.x, o * yv.y, o * yv.z, o * yv.w);
+#pragma unroll
+            for (int s = 0; s < NS; ++s) {
+              const float m = sc[s * NS + t];
+              n = make_float4(fmaf(m, x[i][s].x, n.x), fmaf(m, x[i][s].y, n.y), fmaf(m, x[i][s].z, n.z), fmaf(m, x[i][s].w, n.w));
+            }
+            st4(xo + t * a.dp + v * 4, n);
+            u = make_float4(fmaf(in, n.x, u.x), fmaf(in, n.y, u.y), fmaf(in, n.z, u.z), fmaf(in, n.w, u.w));
+          }
+      }
+      y[i0 + i] = u;
+      ss += sq4(u);
     }
   }
+  if (a.h) write_operand<T, MAXV>(a, row, nv, y, ss, red);
 }
 
 // ---------------------------------------------------------------------------------------------- token shift
@@ -499,6 +592,7 @@ gather_norm_kernel(const float* __restrict__ x, int ldx, const int64_t* __restri
   }
 }
 
+constexpr int MAX_STREAMS = 8;
 static int row_threads(int dp) { return dp <= 512 ? 128 : 256; }
 // vectors of four per thread, rounded up to the instantiated counts; 0: too wide
 static int row_vecs(int dp, int threads) {
@@ -529,20 +623,43 @@ using namespace artb;
     default: return ERR_TOO_LARGE; \
   }
 
-// f32: operands (table, h) are fp32 instead of bf16.  See ResidualArgs; y_kind is a RowKind.
+// f32: operands (table, h) are fp32 instead of bf16.  See ResidualArgs; y_kind, rg_kind are RowKinds.  coef: a step of hyper-connected
+// streams (stream_step_kernel; n_in = 0: the embedding, of which every copy is the same).
 ARTB_EXPORT int artb_residual_step(int f32, const int64_t* tokens, const void* table, int ldt, long vocab, void* y, int ldy,
                                    int y_kind, const float* x_in, float* x_out, int ldx, const float* w_post, float mult,
                                    const float* y_gate, const float* y_bias, const void* ex, int ldex, int ex_k, const int* ex_pos,
                                    const float* ex_w, long ex_rows, void* idn, int ldidn, int idn_kind, const double* freq, const int* pos, float* hist, long hist_stride, int hist_n, const float* avg, const float* w_next, void* h,
-                                   int ldh, int M, int d, int dp, float eps, int* status, cudaStream_t st) {
+                                   int ldh, int M, int d, int dp, float eps, int* status, void* rg, int ldrg, int rg_kind, const float* rg_b,
+                                   const float* coef, int n_in, int n_out, int ldxi, cudaStream_t st) {
   if (M <= 0) return 0;
   if ((dp & 3) || dp < d || (ldx & 3) || (ldy & 3) || (ldh & 3) || (ldt & 3) || (ldex & 3) || (ldidn & 3) || !x_out || (w_next && !h)) return ERR_BAD_SHAPE;
   if (!tokens && ((!y && !ex) || !x_in)) return ERR_BAD_SHAPE;
+  if (rg && ((rg_kind == ROW_BF16 ? 7 : 15) & reinterpret_cast<uintptr_t>(rg))) return ERR_BAD_ALIGN;
   if ((ex && (ex_k <= 0 || !ex_pos || !ex_w)) || (idn && (!ex || idn_kind == ROW_F32_TAKE)) || (freq && (!tokens || !pos))) return ERR_BAD_SHAPE;
   const ResidualArgs a{tokens, table, ldt, vocab, y, ldy, y_kind, x_in, x_out, ldx, w_post, mult, y_gate, y_bias, ex, ldex, ex_k, ex_pos, ex_w,
-                       ex_rows, idn, ldidn, idn_kind, freq, pos, hist, hist_stride, hist_n, avg, w_next, h, ldh, d, dp, eps, status};
+                       ex_rows, idn, ldidn, idn_kind, freq, pos, hist, hist_stride, hist_n, avg, w_next, h, ldh, d, dp, eps, status, rg, ldrg, rg_kind,
+                       rg_b, coef, n_in, n_out, ldxi};
+  if (rg && (!rg_b || tokens || w_post || (ldrg & 3))) return ERR_BAD_SHAPE;
   const int th = row_threads(dp);
   cudaError_t e = cudaSuccess;
+  if (coef) {
+    if (n_in < 0 || n_out < 1 || n_in > MAX_STREAMS || n_out > MAX_STREAMS || (n_in == 0) != (tokens != nullptr) || (tokens && mult != 1.f) || w_post ||
+        hist || freq || idn || (ldxi & 3) || ldxi < n_in * dp || ldx < n_out * dp || (n_in != n_out && x_in == x_out))
+      return ERR_BAD_SHAPE;
+    const int ns = n_in > n_out ? n_in : n_out;
+#define ARTB_SS_N(V, N)                                                                                                \
+  e = f32 ? launch_kernel(stream_step_kernel<float, V, N>, dim3(M), dim3(th), 0, st, a)                                 \
+          : launch_kernel(stream_step_kernel<__nv_bfloat16, V, N>, dim3(M), dim3(th), 0, st, a)
+#define ARTB_SS(V)              \
+  if (ns <= 1) ARTB_SS_N(V, 1); \
+  else if (ns <= 2) ARTB_SS_N(V, 2); \
+  else if (ns <= 4) ARTB_SS_N(V, 4); \
+  else ARTB_SS_N(V, 8)
+    ARTB_BY_VECS(row_vecs(dp, th), ARTB_SS)
+#undef ARTB_SS
+#undef ARTB_SS_N
+    return static_cast<int>(e);
+  }
 #define ARTB_RS(V)                                                                                                     \
   e = f32 ? launch_kernel(residual_step_kernel<float, V>, dim3(M), dim3(th), 0, st, a)                                  \
           : launch_kernel(residual_step_kernel<__nv_bfloat16, V>, dim3(M), dim3(th), 0, st, a)

@@ -4,9 +4,9 @@
 // that every head expands into its keys and values, and one rotated key part that all heads share.  Position i sees the
 // keys j with 0 <= i - j < window.
 //
-//   latent_finish_kernel   what follows the q | latent projection, one CTA per token: RMSNorm of the latent, interleaved
-//                          rotation of the shared key part and of every head's rotated query part, cache write, and the
-//                          queries in the layout the attention form of the row reads
+//   latent_finish_kernel   what follows the q | latent projection, one CTA per token: RMSNorm of the latent, rotation of the
+//                          shared key part and of every head's rotated query part (angles reduced in fp64), cache write, and
+//                          the queries in the layout the attention form of the row reads
 //   latent_attend_kernel   attention in latent space ("absorbed" form): q~ = W_uk^T q per head is taken against the cached
 //                          latents themselves, the weighted latents are expanded by W_uv afterwards.  Scalar fp32
 //                          arithmetic: the 32-bit mode runs on it (bf16: latent_decode.cu, latent_prefill.cu).
@@ -17,6 +17,7 @@
 
 #include "bounds_check.cuh"
 #include "host_utils.h"
+#include "key_weights.cuh"
 #include "row_io.cuh"
 
 namespace artb {
@@ -25,7 +26,9 @@ struct LatentFinish {
   void* p;                  // [M, ldp] of kind `kind`: q (H heads of dim | rot) | latent (rank) | rotated part (rot)
   int ldp, kind;
   const float* w;           // latent norm weight [rank]
-  const float* inv_freq;    // [rot / 2]
+  const double* freq;       // angle of pair i of position p: p * freq[i], rot / 2 pairs
+  float rot_scale;          // factor of sine and cosine
+  int next;                 // a dimension's partner: its neighbour, or (0) rot / 2 dimensions further
   const int* pos;
   const int* slot;          // cache row of every token, < 0: not written
   void* cache;              // T [num_slots, ldc]
@@ -73,7 +76,11 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
   const int m = blockIdx.x, tid = threadIdx.x, hp = a.rot >> 1, hq = a.dim + a.rot;
   float *cc = cs, *sn = cs + hp;
   const size_t row = static_cast<size_t>(m) * a.ldp;
-  for (int i = tid; i < hp; i += blockDim.x) sincosf(static_cast<float>(a.pos[m]) * a.inv_freq[i], &sn[i], &cc[i]);
+  for (int i = tid; i < hp; i += blockDim.x) {
+    const float2 t = position_pair(a.pos[m], a.freq[i]);
+    sn[i] = a.rot_scale * t.x;
+    cc[i] = a.rot_scale * t.y;
+  }
   int slot = a.slot[m];
   if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
   T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
@@ -108,7 +115,31 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
     if (slot >= 0) put_v(crow + i, x);
   }
   // rotated parts: heads 0 .. H - 1 of the query, then the shared key part as "head" H
-  const int ru = a.rot / RW;
+  auto rotated = [&](int h) {              // where its part goes, null: nowhere
+    if (h < a.H) return absorbed ? qr + static_cast<size_t>(h) * a.pitch * a.rot_p : erow + h * he + a.dim_p;
+    return slot >= 0 ? crow + a.rank_p : static_cast<T*>(nullptr);
+  };
+  if (!a.next) {                           // a unit: W neighbours and their partners half the dimensions further
+    const int ru = hp / W;
+    for (int j = tid; j < (a.H + 1) * ru; j += blockDim.x) {
+      const int h = j / ru, i = (j - h * ru) * W;
+      const size_t src = row + (h < a.H ? h * hq + a.dim : c0 + a.rank) + i;
+      float x[W], z[W], y0[W], y1[W];
+      take_v<W>(a.p, src, a.kind, x);
+      take_v<W>(a.p, src + hp, a.kind, z);
+#pragma unroll
+      for (int e = 0; e < W; ++e) {
+        y0[e] = x[e] * cc[i + e] - z[e] * sn[i + e];
+        y1[e] = z[e] * cc[i + e] + x[e] * sn[i + e];
+      }
+      T* dst = rotated(h);
+      if (dst) {
+        put_v(dst + i, y0);
+        put_v(dst + hp + i, y1);
+      }
+    }
+  }
+  const int ru = a.next ? a.rot / RW : 0;
   for (int j = tid; j < (a.H + 1) * ru; j += blockDim.x) {
     const int h = j / ru, i = (j - h * ru) * RW;
     float x[RW], y[RW];
@@ -119,8 +150,8 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
       y[e] = x[e] * c - x[e + 1] * s;
       y[e + 1] = x[e + 1] * c + x[e] * s;
     }
-    if (h < a.H) put_v(absorbed ? qr + static_cast<size_t>(h) * a.pitch * a.rot_p + i : erow + h * he + a.dim_p + i, y);
-    else if (slot >= 0) put_v(crow + a.rank_p + i, y);
+    T* dst = rotated(h);
+    if (dst) put_v(dst + i, y);
   }
   if (!absorbed) {
     const int np = he - a.dim - a.rot;       // padding columns of a head: behind the first part, behind the rotated part
@@ -145,6 +176,7 @@ struct LatentAttend {
   const int* ctx;           // tokens of the sequence; 0: padding sequence
   int window;               // <= 0: every earlier key
   float scale;
+  const float* sink;        // fp32 [H] sinks of the softmax, or null
   void* o;                  // T [H][pitch][rank_p]   weighted latents
   int rank_p, rot_p;
   int* status;
@@ -172,7 +204,7 @@ __global__ void __launch_bounds__(128) latent_attend_kernel(const LatentAttend a
   float acc[OV];
 #pragma unroll
   for (int i = 0; i < OV; ++i) acc[i] = 0.f;
-  float mx = -INFINITY, sum = 0.f;
+  float mx = a.sink ? a.sink[h] : -INFINITY, sum = a.sink ? 1.f : 0.f;
   const T* cache = reinterpret_cast<const T*>(a.cache);
   for (int k0 = lo; k0 < len; k0 += KT) {
     __syncthreads();
@@ -233,17 +265,17 @@ __global__ void __launch_bounds__(128) latent_attend_kernel(const LatentAttend a
 
 using namespace artb;
 
-ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const float* w, const float* inv_freq, const int* pos,
-                                   const int* slot, void* cache, int ldc, long num_slots, int n_abs, void* qn, void* qr, int pitch,
+ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const float* w, const double* freq, float rot_scale, int next,
+                                   const int* pos, const int* slot, void* cache, int ldc, long num_slots, int n_abs, void* qn, void* qr, int pitch,
                                    void* qe, int ldqe, int M, int H, int dim, int dim_p, int rot, int rot_p, int rank, int rank_p,
                                    float eps, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
-  if (H <= 0 || (rot & 1) || dim_p < dim || rot_p < rot || rank_p < rank || ldc < rank_p + rot_p) return ERR_BAD_SHAPE;
+  if (H <= 0 || (rot & 1) || (rot && !freq) || dim_p < dim || rot_p < rot || rank_p < rank || ldc < rank_p + rot_p) return ERR_BAD_SHAPE;
   if ((n_abs > 0 && (!qn || !qr || pitch < n_abs)) || (n_abs < M && (!qe || ldqe < H * (dim_p + rot_p)))) return ERR_BAD_SHAPE;
-  const LatentFinish a{p, ldp, kind, w, inv_freq, pos, slot, cache, ldc, num_slots, n_abs, qn, qr, pitch, qe, ldqe, H, dim, dim_p,
+  const LatentFinish a{p, ldp, kind, w, freq, rot_scale, next, pos, slot, cache, ldc, num_slots, n_abs, qn, qr, pitch, qe, ldqe, H, dim, dim_p,
                        rot, rot_p, rank, rank_p, eps, status};
   const size_t smem = static_cast<size_t>(rot) * 4;
-  const bool v4 = !((dim | rot | rank | ldp) & 3) && !(reinterpret_cast<uintptr_t>(p) & 15);
+  const bool v4 = !((dim | rot | rank | ldp) & 3) && (next || !(rot & 7)) && !(reinterpret_cast<uintptr_t>(p) & 15);
 #define ARTB_LF(T_, W_, R_) return static_cast<int>(launch_kernel(latent_finish_kernel<T_, W_, R_>, dim3(M), dim3(256), smem, st, a))
   if (f32) {
     if (v4) ARTB_LF(float, 4, 4);
@@ -256,13 +288,13 @@ ARTB_EXPORT int artb_latent_finish(int f32, void* p, int ldp, int kind, const fl
 
 ARTB_EXPORT int artb_latent_attend(int f32, const void* ql, const void* qr, int pitch, const void* cache, int ldc,
                                    const int* block_table, int max_blocks, int block_size, long num_blocks, const int* row_seq,
-                                   const int* pos, const int* ctx, int window, float scale, void* o, int M, int H, int rank_p,
-                                   int rot_p, int* status, cudaStream_t st) {
+                                   const int* pos, const int* ctx, int window, float scale, const float* sink, void* o, int M, int H,
+                                   int rank_p, int rot_p, int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   if (H <= 0 || H > 65535 || rank_p > 1024 || (rank_p & 3) || (rot_p & 3) || (ldc & 3) || ldc < rank_p + rot_p || pitch < M ||
       block_size <= 0)
     return ERR_BAD_SHAPE;
-  const LatentAttend a{ql, qr, pitch, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, window, scale,
+  const LatentAttend a{ql, qr, pitch, cache, ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos, ctx, window, scale, sink,
                        o, rank_p, rot_p, status};
   const size_t smem = static_cast<size_t>(rank_p + rot_p) * 4;
   return static_cast<int>(f32 ? launch_kernel(latent_attend_kernel<float>, dim3(M, H), dim3(128), smem, st, a)

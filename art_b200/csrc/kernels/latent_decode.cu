@@ -14,6 +14,7 @@
 
 #include "bounds_check.cuh"
 #include "host_utils.h"
+#include "key_weights.cuh"
 #include "mma_tile.cuh"
 
 namespace artb {
@@ -34,6 +35,7 @@ struct LatentDecode {
   const int* ctx;
   int window;
   float scale_log2;
+  const float* sink;               // fp32 [H] sinks of the softmax, or null
   __nv_bfloat16* o;                // [H][pitch][rank_p]
   float* ws;                       // [M][H][splits][rank_p + 2]
   int splits, H, rank_p, rot_p;
@@ -128,7 +130,12 @@ __global__ void __launch_bounds__(32 * LD_WARPS, LD_KT == 32 && KS < 17 ? 2 : 1)
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
   float mrow[RPW], lrow[RPW];          // of rows warp * RPW + j, the same in every lane
 #pragma unroll
-  for (int j = 0; j < RPW; ++j) mrow[j] = -INFINITY, lrow[j] = 0.f;
+  for (int j = 0; j < RPW; ++j) {
+    const int h = h0 + warp * RPW + j;
+    const bool sink = a.sink && split == 0 && h < a.H;      // counted by one split
+    mrow[j] = sink ? a.sink[h] * KW_LOG2E : -INFINITY;
+    lrow[j] = sink ? 1.f : 0.f;
+  }
 
   for (int tile = t_lo; tile < t_hi; ++tile) {
     const int buf = (tile - t_lo) & 1, k0 = lo + tile * LD_KT;
@@ -329,7 +336,7 @@ using namespace artb;
 // splits > 1.  rank_p, rot_p multiples of 16; rank_p <= 1024.
 ARTB_EXPORT int artb_latent_decode(const void* ql, const void* qr, int pitch, const void* cache, int ldc, const int* block_table,
                                    int max_blocks, int block_size, long num_blocks, const int* row_seq, const int* pos, const int* ctx,
-                                   int window, float scale, void* o, float* ws, int splits, int M, int H, int rank_p, int rot_p,
+                                   int window, float scale, const float* sink, void* o, float* ws, int splits, int M, int H, int rank_p, int rot_p,
                                    int* status, cudaStream_t st) {
   if (M <= 0) return 0;
   if (H <= 0 || (rank_p & 15) || (rot_p & 15) || rank_p <= 0 || (ldc & 7) || ldc < rank_p + rot_p || pitch < M || splits < 1 ||
@@ -338,7 +345,7 @@ ARTB_EXPORT int artb_latent_decode(const void* ql, const void* qr, int pitch, co
   if ((reinterpret_cast<uintptr_t>(ql) | reinterpret_cast<uintptr_t>(qr) | reinterpret_cast<uintptr_t>(cache)) & 15) return ERR_BAD_ALIGN;
   const LatentDecode a{reinterpret_cast<const __nv_bfloat16*>(ql), reinterpret_cast<const __nv_bfloat16*>(qr), pitch,
                        reinterpret_cast<const __nv_bfloat16*>(cache), ldc, block_table, max_blocks, block_size, num_blocks, row_seq, pos,
-                       ctx, window, scale * 1.4426950408889634f, reinterpret_cast<__nv_bfloat16*>(o), ws, splits, H, rank_p, rot_p,
+                       ctx, window, scale * KW_LOG2E, sink, reinterpret_cast<__nv_bfloat16*>(o), ws, splits, H, rank_p, rot_p,
                        status};
   const int D = rank_p + rot_p;
   if (M > 65535) return ERR_BAD_SHAPE;

@@ -4,7 +4,8 @@
 //                           sequence (a GEMM then expands their latents into every head's keys and values)
 //   latent_prefill_kernel   windowed flash attention for any sizes (whole 64-column blocks: latent_prefill_tc.cu); a head's key is [ expanded part: dk | rotated part: rot_p ], the
 //                           rotated part coming from the gathered rows all heads share
-// Without a rotated part, and with G query heads per key head, the same kernel is grouped-query attention.
+// Without a rotated part, and with G query heads per key head, the same kernel is grouped-query attention.  Sigmoid weights
+// with a bias by distance, sinks and column gates: key_weights.cuh.
 //
 // A CTA owns 128 query rows of one sequence and one head: four warps with 32 rows each, key tiles of 32, keys and values
 // double-buffered with asynchronous copies.  Scores, softmax and accumulators are fp32; only the probabilities enter the
@@ -14,6 +15,7 @@
 #include "bounds_check.cuh"
 #include "host_utils.h"
 #include "key_mask.cuh"
+#include "key_weights.cuh"
 #include "mma_tile.cuh"
 #include "softcap.cuh"
 
@@ -65,13 +67,16 @@ struct LatentPrefill {
   float out_scale;               // multiplies the result
   const float* gate;             // [rows][ldg] factor per row and head, or null
   int ldg;
+  const float* sink;             // fp32 [H] sinks of the softmax, or null
+  DistanceBias bias;             // of every query head (sigmoid weights)
+  ColumnGate<__nv_bfloat16> cols;
   __nv_bfloat16* o;              // [rows][ldo]: heads of vp columns
   int ldo, vp, vdim;
   int H, G, dk, dv, rot_p;       // G heads share a key head; dk, dv, rot_p multiples of 16
 };
 
-// DV: value columns held in registers (dv <= DV)
-template <int DV>
+// DV: value columns held in registers (dv <= DV); SIG: sigmoid weights
+template <int DV, bool SIG>
 __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefill_kernel(const LatentPrefill a) {
   extern __shared__ __align__(16) uint8_t lp_smem[];
   const int DQ = a.dk + a.rot_p, LQ = DQ + 8, LV = a.dv + 8;
@@ -120,6 +125,13 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
   float mrow[2][2], lrow[2][2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) mrow[i][0] = mrow[i][1] = -INFINITY, lrow[i][0] = lrow[i][1] = 0.f;
+  if (!SIG && a.sink) {                           // counted by one of the four lanes of a row
+    const float sk = a.sink[h] * KW_LOG2E;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) mrow[i][0] = mrow[i][1] = sk, lrow[i][0] = lrow[i][1] = t == 0 ? 1.f : 0.f;
+  }
+  const float* tab = SIG ? a.bias.head(h) : nullptr;
+  const float far = SIG ? a.bias.last(tab) : 0.f;
   const int w0 = warp * 32;                       // first row of the warp inside the tile
 
   for (int tile = 0; tile < tiles; ++tile) {
@@ -159,12 +171,27 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
       }
       // no masking needed when every row of the warp sees the whole tile
       const bool inside = k0 + LP_BN - 1 <= wp0 && k0 >= a.mask.first(wp1);
+      const bool near = SIG && !a.bias.beyond(wp0, k0 + LP_BN - 1);
       uint32_t pf[2][2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int p = p0 + w0 + i * 16 + g + 8 * e, first = a.mask.first(p);
+          if (SIG) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+              float w[2];
+#pragma unroll
+              for (int k = 0; k < 2; ++k) {
+                const int kp = k0 + j * 8 + 2 * t + k;
+                w[k] = sigmoid_base2(a.score(s[i][j][2 * e + k]) + (near ? a.bias.at(tab, p - kp) : far));
+                if (!inside && (kp > p || kp < first)) w[k] = 0.f;
+              }
+              pf[i][j >> 1][(j & 1) * 2 + e] = pair_bf16(w[0], w[1]);
+            }
+            continue;
+          }
           float mx = mrow[i][e];
 #pragma unroll
           for (int j = 0; j < 4; ++j)
@@ -221,20 +248,21 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
       l += __shfl_xor_sync(0xffffffffu, l, 2);
       const int r = w0 + i * 16 + g + 8 * e;
       if (r >= nrow) continue;
-      float inv = l > 0.f ? a.out_scale / l : 0.f;
+      float inv = SIG ? a.out_scale : l > 0.f ? a.out_scale / l : 0.f;
       if (a.gate) inv *= a.gate[static_cast<size_t>(r0 + r) * a.ldg + h];
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp;
 #pragma unroll
       for (int n = 0; n < DV / 8; ++n) {
         const int d = n * 8 + 2 * t;
-        if (d < a.vp) *reinterpret_cast<uint32_t*>(o + d) = pair_bf16(acc[i][n][2 * e] * inv, acc[i][n][2 * e + 1] * inv);
+        if (d < a.vp)
+          *reinterpret_cast<uint32_t*>(o + d) = pair_bf16(acc[i][n][2 * e] * inv * a.cols(r0 + r, h, d), acc[i][n][2 * e + 1] * inv * a.cols(r0 + r, h, d + 1));
       }
     }
 }
 
 static size_t latent_prefill_smem(int DQ, int dv) { return (static_cast<size_t>(LP_BM + 2 * LP_BN) * (DQ + 8) + 2ull * LP_BN * (dv + 8)) * 2; }
 
-template <int DV>
+template <int DV, bool SIG>
 static int launch_latent_prefill(const LatentPrefill& a, int n_tiles, cudaStream_t st) {
   const size_t smem = latent_prefill_smem(a.dk + a.rot_p, a.dv);
   if (smem > 225 * 1024) return ERR_TOO_LARGE;
@@ -242,11 +270,11 @@ static int launch_latent_prefill(const LatentPrefill& a, int n_tiles, cudaStream
   int dev = 0;
   cudaGetDevice(&dev);
   if (configured[dev & 63] < smem) {
-    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<DV, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = smem;
   }
-  latent_prefill_kernel<DV><<<dim3(a.H, n_tiles), 32 * LP_WARPS, smem, st>>>(a);
+  latent_prefill_kernel<DV, SIG><<<dim3(a.H, n_tiles), 32 * LP_WARPS, smem, st>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -271,18 +299,22 @@ ARTB_EXPORT int artb_latent_gather(const void* cache, int ldc, const int* block_
 
 ARTB_EXPORT int artb_latent_prefill(const void* q, int ldq, const void* kv, int ldkv, const void* c, int ldc, int rank_p, const int* tile_seq,
                                     const int* tile_row, int n_tiles, const int* row_end, const int* row_pos0, const int* key_off,
-                                    const int* key_pos0, int window, int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp, int vdim, int H, int G,
-                                    int dk, int dv, int rot_p, cudaStream_t st) {
+                                    const int* key_pos0, int window, int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, const float* sink, int sigmoid, const float* bias, int n_bias, const void* cols, int ldcols, int colp,
+                                    void* o, int ldo, int vp, int vdim, int H, int G, int dk, int dv, int rot_p, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G || (dk & 15) || (dv & 15) || (rot_p & 15) || (ldq & 7) || (ldkv & 7) || (ldc & 7) || (rank_p & 7) || (ldo & 1) || (vp & 1) ||
-      vp > dv || vdim > vp || n_tiles > 65535)
+      vp > dv || vdim > vp || n_tiles > 65535 || (sigmoid && (!bias || n_bias <= 0 || sink)) || (cols && colp < vdim))
     return ERR_BAD_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(c)) & 15) return ERR_BAD_ALIGN;
   const LatentPrefill a{(const bf16*)q, ldq, (const bf16*)kv, ldkv, (const bf16*)c, ldc, rank_p, tile_seq, tile_row, row_end, row_pos0,
-                        key_off, key_pos0, {window, chunk}, ScoreScale::of(scale, softcap), out_scale, gate, ldg, (bf16*)o, ldo, vp, vdim, H, G, dk, dv, rot_p};
-  if (dv <= 32) return launch_latent_prefill<32>(a, n_tiles, st);
-  if (dv <= 64) return launch_latent_prefill<64>(a, n_tiles, st);
-  if (dv <= 96) return launch_latent_prefill<96>(a, n_tiles, st);
-  if (dv <= 128) return launch_latent_prefill<128>(a, n_tiles, st);
+                        key_off, key_pos0, {window, chunk}, ScoreScale::of(scale, softcap), out_scale, gate, ldg, sink, {bias, n_bias},
+                        ColumnGate<bf16>::of(cols, ldcols, colp, vdim), (bf16*)o, ldo, vp, vdim, H, G, dk, dv, rot_p};
+#define ARTB_LP(V_)                                                                                                          \
+  if (dv <= V_) return sigmoid ? launch_latent_prefill<V_, true>(a, n_tiles, st) : launch_latent_prefill<V_, false>(a, n_tiles, st)
+  ARTB_LP(32);
+  ARTB_LP(64);
+  ARTB_LP(96);
+  ARTB_LP(128);
+#undef ARTB_LP
   return ERR_TOO_LARGE;
 }

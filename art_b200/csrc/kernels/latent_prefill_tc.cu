@@ -3,7 +3,8 @@
 // The same operation as latent_prefill_kernel (expanded keys of dk columns, a rotated part of rot_p columns shared by all
 // heads, values of dv columns), with S = Q K^T and O = P V as tcgen05.mma with accumulators in TMEM:
 //
-// With G query heads per key head and no rotated part it is grouped-query attention.
+// With G query heads per key head and no rotated part it is grouped-query attention.  With sigmoid weights (key_weights.cuh)
+// nothing is rescaled: P V of all tiles adds up in one TMEM accumulator, and the warps of a row need not agree on a maximum.
 //
 //   warp 0      TMA producer: Q once; per tile of 128 keys the key blocks (expanded part from k, rotated part from the
 //               gathered cache rows) and the value block, which a GEMM has written transposed ([H * dv, keys])
@@ -18,6 +19,7 @@
 
 #include "host_utils.h"
 #include "key_mask.cuh"
+#include "key_weights.cuh"
 #include "ptx_sm100.cuh"
 #include "softcap.cuh"
 
@@ -39,6 +41,9 @@ struct LatentTc {
   float out_scale;
   const float* gate;      // [rows][ldg] factor per row and head, or null
   int ldg;
+  const float* sink;      // fp32 [H] sinks of the softmax, or null
+  DistanceBias bias;      // of every query head (sigmoid weights)
+  ColumnGate<__nv_bfloat16> cols;
   __nv_bfloat16* o;
   int ldo, vp;
   int rank_p, dk, rot_p, G;
@@ -57,13 +62,10 @@ struct LtSmem {
   static constexpr int TOTAL = BAR + 28 * 8 + 1024;
 };
 
-__device__ __forceinline__ float lt_ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+__device__ __forceinline__ float lt_ex2(float x) { return exp2_approx(x); }
 
-template <int NQ, int DV>
+// SIG: sigmoid weights
+template <int NQ, int DV, bool SIG>
 __global__ void __launch_bounds__(LT_THREADS, 1)
 latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                          const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmVt, const LatentTc a) {
@@ -171,14 +173,16 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       bool ok = mbar_wait_timed(q_full, 0);
       auto issue_pv = [&](int i) -> bool {
         const int s = i & 1;
-        if (!mbar_wait_timed(v_full, i & 1) || !mbar_wait_timed(p_full, i & 1) || !mbar_wait_timed(&pv_empty[s], ((i >> 1) & 1) ^ 1)) return false;
+        if (!mbar_wait_timed(v_full, i & 1) || !mbar_wait_timed(p_full, i & 1)) return false;
+        if (!SIG && !mbar_wait_timed(&pv_empty[s], ((i >> 1) & 1) ^ 1)) return false;
         tc_fence_after_sync();
-        const uint32_t d = tmem + 256 + s * 128;
+        const uint32_t d = tmem + 256 + (SIG ? 0 : s * 128);
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)
           tc_mma_f16(d, umma_smem_desc_k128(sp + (kk >> 2) * LT_BLK) + 2 * (kk & 3),
-                     umma_smem_desc_k128(sv + (kk >> 2) * L::VBLK) + 2 * (kk & 3), idesc_o, kk != 0);
-        tc_commit(&pv_full[s]);
+                     umma_smem_desc_k128(sv + (kk >> 2) * L::VBLK) + 2 * (kk & 3), idesc_o, kk != 0 || (SIG && i > 0));
+        if (!SIG) tc_commit(&pv_full[s]);
+        else if (i == tiles - 1) tc_commit(&pv_full[0]);
         tc_commit(v_empty);
         tc_commit(p_empty);
         return true;
@@ -223,6 +227,12 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 #pragma unroll
     for (int i = 0; i < OC; ++i) O[i] = 0.f;
     float m = -INFINITY, l = 0.f, m_o = 0.f, ms_prev = 0.f;
+    if (!SIG && a.sink) {                   // counted by one warp of the pair
+      m = a.sink[h] * KW_LOG2E;
+      l = hf == 0 ? 1.f : 0.f;
+    }
+    const float* tab = SIG ? a.bias.head(h) : nullptr;
+    const float far = SIG ? a.bias.last(tab) : 0.f;
     bool dead = false;
     uint32_t xph = 0;
 
@@ -300,6 +310,40 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
 #pragma unroll
         for (int j = 0; j < 64; ++j) x[j] = a.score.squash(x[j]);
       }
+      if (SIG) {
+        if (a.bias.beyond(p0, k0 + LT_B - 1)) {
+#pragma unroll
+          for (int j = 0; j < 64; ++j) x[j] = sigmoid_base2(fmaf(x[j], a.score.scale_log2, far));
+        } else {                              // distances of the tile stay within the table's padding
+          const float* td = tab + qpos - (k0 + hf * 64);
+#pragma unroll
+          for (int j = 0; j < 64; ++j) x[j] = sigmoid_base2(fmaf(x[j], a.score.scale_log2, __ldg(td - j)));
+        }
+        if (!inside) {
+          const int hi = qpos - (k0 + hf * 64), lo = first - (k0 + hf * 64);
+#pragma unroll
+          for (int j = 0; j < 64; ++j)
+            if (j > hi || j < lo) x[j] = 0.f;
+        }
+        const int okp = mbar_wait_timed(p_empty, (it & 1) ^ 1) ? 1 : 0;
+        if (!__all_sync(0xffffffffu, okp)) {
+          fail(ST_TIMEOUT_EMPTY);
+          break;
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          uint4 w;
+          w.x = pack_bf16x2(x[8 * i], x[8 * i + 1]);
+          w.y = pack_bf16x2(x[8 * i + 2], x[8 * i + 3]);
+          w.z = pack_bf16x2(x[8 * i + 4], x[8 * i + 5]);
+          w.w = pack_bf16x2(x[8 * i + 6], x[8 * i + 7]);
+          *reinterpret_cast<uint4*>(prow + ((i ^ sw) << 4)) = w;
+        }
+        fence_proxy_async_smem();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(p_full);
+        continue;
+      }
       if (!inside) {
         const int hi = qpos - (k0 + hf * 64), lo = first - (k0 + hf * 64);      // visible: lo <= j <= hi
 #pragma unroll
@@ -351,22 +395,43 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       }
       ms_prev = ms;
     }
-    if (!dead && tiles > 0 && !add_pv(tiles - 1, ms_prev)) fail(ST_TIMEOUT_TMEM_FULL);
     float l_other = 0.f;
-    if (!dead && !swap_with_partner(l, l_other)) fail(ST_TIMEOUT_PEER);
+    if (SIG) {
+      const int okw = !dead && mbar_wait_timed(&pv_full[0], 0) ? 1 : 0;
+      if (!__all_sync(0xffffffffu, okw)) {
+        if (!dead) fail(ST_TIMEOUT_TMEM_FULL);
+      } else {
+        tc_fence_after_sync();
+#pragma unroll
+        for (int c = 0; c < OC; c += 32) {
+          uint32_t v[32];
+          tmem_ld_32x32(tmem + lane_off + 256 + hf * OC + c, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int j = 0; j < 32; ++j) O[c + j] = __uint_as_float(v[j]);
+        }
+      }
+    } else {
+      if (!dead && tiles > 0 && !add_pv(tiles - 1, ms_prev)) fail(ST_TIMEOUT_TMEM_FULL);
+      if (!dead && !swap_with_partner(l, l_other)) fail(ST_TIMEOUT_PEER);
+    }
     if (!dead && r < nrow) {
       const float lt = l + l_other;
-      float inv = lt > 0.f ? a.out_scale / lt : 0.f;
+      float inv = SIG ? a.out_scale : lt > 0.f ? a.out_scale / lt : 0.f;
       if (a.gate) inv *= a.gate[static_cast<size_t>(r0 + r) * a.ldg + h];
       __nv_bfloat16* o = a.o + static_cast<size_t>(r0 + r) * a.ldo + static_cast<size_t>(h) * a.vp + hf * OC;
 #pragma unroll
       for (int c = 0; c < OC; c += 8) {
         if (hf * OC + c < a.vp) {
+          float y[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[j] = O[c + j] * inv;
+          a.cols.scale8(r0 + r, h, hf * OC + c, y);
           uint4 w;
-          w.x = pack_bf16x2(O[c] * inv, O[c + 1] * inv);
-          w.y = pack_bf16x2(O[c + 2] * inv, O[c + 3] * inv);
-          w.z = pack_bf16x2(O[c + 4] * inv, O[c + 5] * inv);
-          w.w = pack_bf16x2(O[c + 6] * inv, O[c + 7] * inv);
+          w.x = pack_bf16x2(y[0], y[1]);
+          w.y = pack_bf16x2(y[2], y[3]);
+          w.z = pack_bf16x2(y[4], y[5]);
+          w.w = pack_bf16x2(y[6], y[7]);
           *reinterpret_cast<uint4*>(o + c) = w;
         }
       }
@@ -386,8 +451,8 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
   }
 }
 
-template <int NQ, int DV>
-static int launch_latent_tc(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tC, const CUtensorMap& tV, const LatentTc& a,
+template <int NQ, int DV, bool SIG>
+static int launch_latent_tc_form(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tC, const CUtensorMap& tV, const LatentTc& a,
                             int n_tiles, int H, cudaStream_t st) {
   using L = LtSmem<NQ, DV>;
   static_assert(L::TOTAL <= 227 * 1024, "shared memory");
@@ -395,12 +460,19 @@ static int launch_latent_tc(const CUtensorMap& tQ, const CUtensorMap& tK, const 
   int dev = 0;
   cudaGetDevice(&dev);
   if (!configured[dev & 63]) {
-    cudaError_t e = cudaFuncSetAttribute(latent_prefill_tc_kernel<NQ, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+    cudaError_t e = cudaFuncSetAttribute(latent_prefill_tc_kernel<NQ, DV, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
     if (e != cudaSuccess) return static_cast<int>(e);
     configured[dev & 63] = true;
   }
-  latent_prefill_tc_kernel<NQ, DV><<<dim3(n_tiles, H), LT_THREADS, L::TOTAL, st>>>(tQ, tK, tC, tV, a);
+  latent_prefill_tc_kernel<NQ, DV, SIG><<<dim3(n_tiles, H), LT_THREADS, L::TOTAL, st>>>(tQ, tK, tC, tV, a);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <int NQ, int DV>
+static int launch_latent_tc(const CUtensorMap& tQ, const CUtensorMap& tK, const CUtensorMap& tC, const CUtensorMap& tV, const LatentTc& a,
+                            int n_tiles, int H, cudaStream_t st) {
+  return a.bias.tab ? launch_latent_tc_form<NQ, DV, true>(tQ, tK, tC, tV, a, n_tiles, H, st)
+                    : launch_latent_tc_form<NQ, DV, false>(tQ, tK, tC, tV, a, n_tiles, H, st);
 }
 
 }  // namespace artb
@@ -413,11 +485,13 @@ using namespace artb;
 ARTB_EXPORT int artb_latent_prefill_tc(const void* q, int ldq, int rows, const void* k, int ldk, const void* c, int ldc, int rank_p,
                                        const void* vt, int ldvt, int n_keys, const int* tile_seq, const int* tile_row, int n_tiles,
                                        const int* row_end, const int* row_pos0, const int* key_off, const int* key_pos0, int window,
-                                       int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, void* o, int ldo, int vp, int H, int G, int dk, int dv, int rot_p,
+                                       int chunk, float scale, float softcap, float out_scale, const float* gate, int ldg, const float* sink, int sigmoid, const float* bias, int n_bias, const void* cols, int ldcols, int colp,
+                                       void* o, int ldo, int vp, int vdim, int H, int G, int dk, int dv, int rot_p,
                                        int* status, cudaStream_t st) {
   if (n_tiles <= 0) return 0;
   if (H <= 0 || H > 65535 || G <= 0 || H % G || dk <= 0 || (dk & 63) || (rot_p & 63) || dk + rot_p > 192 || (dv != 64 && dv != 128) || (n_keys & 7) || (ldo & 7) ||
-      (vp & 7) || vp > dv || !(scale > 0.f) || (rank_p & 7))
+      (vp & 7) || vp > dv || vdim > vp || !(scale > 0.f) || (rank_p & 7) || (sigmoid ? !bias || n_bias <= 0 || sink : bias != nullptr) ||
+      (cols && colp < vdim))
     return ERR_BAD_SHAPE;
   if (reinterpret_cast<uintptr_t>(o) & 15) return ERR_BAD_ALIGN;
   CUtensorMap tQ, tK, tC, tV;
@@ -427,7 +501,7 @@ ARTB_EXPORT int artb_latent_prefill_tc(const void* q, int ldq, int rows, const v
   if ((e = make_tmap_bf16_2d(&tC, c, n_keys, ldc, ldc, LT_B, 64))) return e;
   if ((e = make_tmap_bf16_2d(&tV, vt, static_cast<uint64_t>(H / G) * dv, n_keys, ldvt, dv, 64))) return e;
   const LatentTc a{tile_seq, tile_row, row_end, row_pos0, key_off, key_pos0, {window, chunk}, ScoreScale::of(scale, softcap), out_scale, gate, ldg,
-                   reinterpret_cast<__nv_bfloat16*>(o), ldo, vp, rank_p, dk, rot_p, G, status};
+                   sink, {bias, n_bias}, ColumnGate<__nv_bfloat16>::of(cols, ldcols, colp, vdim), reinterpret_cast<__nv_bfloat16*>(o), ldo, vp, rank_p, dk, rot_p, G, status};
   const int nq = (dk + rot_p) / 64;
   if (dv == 128) {
     if (nq == 1) return launch_latent_tc<1, 128>(tQ, tK, tC, tV, a, n_tiles, H, st);

@@ -35,12 +35,13 @@ __device__ __forceinline__ float warp_pick(const float (&a)[MOE_MAX_E_PER_LANE],
 
 // One warp per token.  The k largest logits (+ bias) are chosen, the lower index on a tie; weights are the softmax over all
 // experts or, with `norm`, over the chosen ones.  With `correction` the softmax over all outputs is taken first, the largest
-// of its entries + correction are chosen, and with `norm` their weights are divided by their sum (+ 1e-20).  Outputs from
-// `real` on have no rows of their own (counts end there).  `gate`: the sigmoid of the column behind the outputs.  Logits of kind
+// of its entries + correction are chosen, and with `norm` their weights are divided by their sum (+ 1e-20).  With `keep` > 0 the
+// outputs form groups of `group` neighbours, and only those of the `keep` groups with the largest single entries can be chosen.
+// `scale` multiplies the weights.  Outputs from `real` on have no rows of their own (counts end there).  `gate`: the sigmoid of the column behind the outputs.  Logits of kind
 // ROW_F32_TAKE are cleared once read.
 __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, const float* __restrict__ bias,
-                                  const float* __restrict__ correction, int M, int E, int real, int k, int norm, int* __restrict__ topi,
-                                  float* __restrict__ topw, int* __restrict__ counts, float* __restrict__ gate) {
+                                  const float* __restrict__ correction, int M, int E, int real, int k, int norm, int group, int keep,
+                                  float scale, int* __restrict__ topi, float* __restrict__ topw, int* __restrict__ counts, float* __restrict__ gate) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   pdl_wait();
   pdl_launch_dependents();
@@ -82,8 +83,8 @@ __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, 
   if (correction) sum = norm ? 1e-20f : 1.f;
   float wsel = 0.f;
   int isel = 0;
-  uint32_t taken = 0;                            // entries of this lane that are chosen already
-  for (int s = 0; s < k; ++s) {
+  uint32_t taken = 0;                            // entries of this lane that are chosen already, or cannot be
+  auto largest = [&]() {                         // of the others
     float best = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
@@ -103,7 +104,19 @@ __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, 
         bi = oi;
       }
     }
-    if (bi >= E) bi = 0;                         // logits that are no numbers: stay inside the experts
+    return bi < E ? bi : 0;                      // logits that are no numbers: stay inside the experts
+  };
+  if (keep > 0) {                                // the best group holds the largest entry, the next one the largest outside it
+    for (int s = 0; s < keep; ++s) {
+      const int g = largest() / group;
+#pragma unroll
+      for (int j = 0; j < MOE_MAX_E_PER_LANE; ++j)
+        if ((j * 32 + lane) / group == g) taken |= 1u << j;
+    }
+    taken = ~taken;
+  }
+  for (int s = 0; s < k; ++s) {
+    const int bi = largest();
     if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
     const float pb = warp_pick(p, bi);
     if (norm) sum += pb;
@@ -114,7 +127,7 @@ __global__ void moe_router_kernel(float* __restrict__ logits, int ld, int kind, 
   }
   if (lane < k) {
     topi[static_cast<size_t>(warp) * k + lane] = isel;
-    topw[static_cast<size_t>(warp) * k + lane] = wsel / sum;
+    topw[static_cast<size_t>(warp) * k + lane] = wsel / sum * scale;
     if (isel < real) atomicAdd(counts + isel, 1);
   }
 }
@@ -381,14 +394,16 @@ __global__ void moe_router_bwd_kernel(const float* __restrict__ logits, int ld, 
 using namespace artb;
 
 // logits fp32 [M, E] (E <= 256, k <= 16) of kind ROW_F32 or ROW_F32_TAKE; bias, correction fp32 [E] or null; real <= E outputs
-// have rows; counts int32 [real] must be zero on entry; gate fp32 [M] (logits then have E + 1 columns) or null.
+// have rows; keep > 0: the outputs form `groups` groups (see the kernel); counts int32 [real] must be zero on entry; gate fp32 [M] (logits then have E + 1 columns) or null.
 ARTB_EXPORT int artb_moe_router(float* logits, int ld, int kind, const float* bias, const float* correction, int M, int E, int real, int k,
-                                int norm, int* topi, float* topw, int* counts, float* gate, cudaStream_t st) {
+                                int norm, int groups, int keep, float scale, int* topi, float* topw, int* counts, float* gate, cudaStream_t st) {
   if (M <= 0) return 0;
-  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E || real <= 0 || real > E || ld < E + (gate ? 1 : 0) || kind == ROW_BF16)
+  if (E <= 0 || E > 32 * MOE_MAX_E_PER_LANE || k <= 0 || k > MOE_MAX_K || k > E || real <= 0 || real > E || ld < E + (gate ? 1 : 0) || kind == ROW_BF16 ||
+      (keep > 0 && (groups <= 0 || E % groups || keep > groups || keep * (E / groups) < k)))
     return ERR_BAD_SHAPE;
   const int threads = 256, warps = threads / 32;
-  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, kind, bias, correction, M, E, real, k, norm, topi, topw, counts, gate);
+  moe_router_kernel<<<(M + warps - 1) / warps, threads, 0, st>>>(logits, ld, kind, bias, correction, M, E, real, k, norm, groups > 0 ? E / groups : E,
+                                                                   keep < groups ? keep : 0, scale, topi, topw, counts, gate);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -175,12 +175,12 @@ def kernel_rows(width: int = 4096, ff: int = 16384, prefill: int = 8192, decode:
         cache = rnd(nb, bs, ldc)
         bt = torch.randperm(nb, device=dev, generator=g).to(torch.int32).view(n_seqs, ctx // bs)
         pq = rnd(M, H * (dk + rot) + rank + rot)
-        inv = rnd(rot // 2, dt=torch.float32)
+        turn = hy.Rotation(rot, rnd(rot // 2, dt=torch.float64), next=True)
         cn = rnd(rank, dt=torch.float32)
         slot = i32([-1] * M)
         qn, qr = torch.zeros(H, hy.pad(M, 128), dk, dtype=bf, device=dev), torch.zeros(H, hy.pad(M, 128), rot, dtype=bf, device=dev)
         qe = torch.zeros(M, H * (dk + rot), dtype=bf, device=dev)
-        add("latent_finish", phase, lambda: hy.latent_finish(hy.as_out(pq), cn, inv, pos, slot, cache, M if one else 0, qn, qr, qe, H, dk, rot, rank, 1e-5),
+        add("latent_finish", phase, lambda: hy.latent_finish(hy.as_out(pq), cn, turn, pos, slot, cache, M if one else 0, qn, qr, qe, H, dk, rank, 1e-5),
             M * (2 * H * (dk + rot) + rank + rot) * 2)
         if one:
             ql, ol = rnd(H, hy.pad(M, 128), rank), torch.zeros(H, hy.pad(M, 128), rank, dtype=bf, device=dev)

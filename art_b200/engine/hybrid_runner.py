@@ -10,8 +10,9 @@ A batch of single tokens (decoding) leaves its projections as split-K partial su
 that follows finishes and clears, as the engine's other models do.
 
 Every sublayer is ``(norm ->) mixer or feed-forward -> (norm ->) residual``; the step from one to the next (a mixture's weighted
-sum, bias, post-norm and factors, residual multiplier, depth average, next input norm: what the design has of them) is one
-kernel over the fp32 residual stream (``ops.hybrid.residual_step``).  Mixers side by side share one input and one output product: their
+sum, bias, gate, post-norm and factors, residual multiplier, depth average or mixing of hyper-connected streams, next input norm:
+what the design has of them) is one kernel over the fp32 residual stream (``ops.hybrid.residual_step``).  A gate on a sublayer's
+result is further rows of the sublayer's input product.  Mixers side by side share one input and one output product: their
 factors scale what enters the latter.
 Operands of the matrix products are bf16; with ``dtype=torch.float32`` everything is fp32, products included, through the
 same layer code.
@@ -25,7 +26,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from ..models.hybrid import PART_NAMES, SHIFT_MIXES, HybridConfig, LayerSpec, check_weights, rope_frequencies
+from ..models.hybrid import PART_NAMES, SHIFT_MIXES, HybridConfig, LayerSpec, check_weights, distance_buckets, rope_frequencies
 from ..ops import hybrid as hy
 from ..ops.hybrid import Out, Sublayer, as_out, pad
 from .runner import DeviceRunner, SeqView
@@ -158,14 +159,55 @@ class HybridRunner(DeviceRunner):
                 if cfg.layer_scale:
                     L[f"post{k}"] *= self._vec(w[f"ls{k}"], dp)
             L["dwa"] = self._vec(w["dwa"]) if cfg.depth_average else None
+            if cfg.residual_gate:
+                for k in (1, 2) if s.has_mlp else (1,):
+                    L[f"rg{k}"], L[f"rg{k}_b"] = self._mat(w[f"rg{k}"], dp, dp), self._vec(w[f"rg{k}.b"], dp)
             getattr(self, "_load_" + s.type)(s, m, L)
             if s.has_mlp:
                 getattr(self, "_load_mlp_" + s.mlp)(s, {k[4:]: t for k, t in w.items() if k.startswith("mlp.")}, L)
             self.layers.append(L)
+        if cfg.streams:
+            self._load_streams(base)
+
+    def _load_streams(self, base: dict[str, torch.Tensor]) -> None:
+        """The boundaries of hyper-connected streams.  All copies are equal before the first sublayer and only their sum is read
+        behind the last one, so that one copy stands for all at either end."""
+        subs = [(i, k) for i, s in enumerate(self.cfg.layers) for k in ((1, 2) if s.has_mlp else (1,))]
+        get = lambda i, k, what: base[f"l{i}.hc{k}.{what}"].to(self.device, torch.float64)      # noqa: E731
+        for n, (i, k) in enumerate(subs):
+            mix, out = get(i, k, "mix"), get(i, k, "out")
+            if n == 0:
+                mix = mix.sum(0, keepdim=True)
+            if n == len(subs) - 1:
+                mix, out = mix.sum(1, keepdim=True), out.sum(0, keepdim=True)
+                nxt = torch.ones_like(out)
+            else:
+                nxt = get(*subs[n + 1], "in")
+            self.layers[i][f"hc{k}"] = hy.Streams(mix.shape[0], mix.shape[1], torch.cat([mix.flatten(), out, nxt]).float())
+        first = get(*subs[0], "in").sum(0, keepdim=True)
+        self._embed_streams = hy.Streams(0, 1, torch.cat([torch.ones_like(first), first]).float())
+
+    def _with_gate(self, k: int, W: torch.Tensor, L: dict) -> torch.Tensor:
+        """An input matrix with the rows of sublayer ``k``'s residual gate below it; their place is ``L["rg<k>_at"]``."""
+        rg = L.pop(f"rg{k}", None)
+        if rg is None:
+            return W
+        L[f"rg{k}_at"] = W.shape[0]
+        return torch.cat([W, rg], 0)
+
+    def _gate_of(self, k: int, p: Out, L: dict) -> dict:
+        """The residual gate of sublayer ``k`` in its input product's output."""
+        at = L.get(f"rg{k}_at")
+        return {} if at is None else dict(col_gate=p.col(at), col_bias=L[f"rg{k}_b"])
+
+    def _rotation(self, s: LayerSpec) -> hy.Rotation:
+        freq, scale = rope_frequencies(s)
+        return hy.Rotation(s.rot_dim, torch.tensor(freq, dtype=torch.float64).to(self.device), scale, s.rot_pairs == "next")
 
     def _load_latent_attention(self, s: LayerSpec, m: dict, L: dict) -> None:
         rank_p = pad(s.kv_rank, 16)
-        L["qkv"] = self._mat(torch.cat([m["q"], m["dkv"]], 0), None, self.dp)
+        L["qkv"] = self._with_gate(1, self._mat(torch.cat([m["q"], m["dkv"]], 0), None, self.dp), L)
+        L["sink"] = self._vec(m["sink"]) if s.sink else None
         L["tc_dv"] = hy.prefill_tc_values(s.dim, s.rot_dim, s.vdim, s.scale)
         dk, dv = pad(s.dim, 16), L["tc_dv"] or pad(s.vdim, 16)
         L["c_norm"] = self._vec(m["dkv.norm"])
@@ -179,7 +221,7 @@ class HybridRunner(DeviceRunner):
             kv[:s.heads * dk].view(s.heads, dk, rank_p)[:, :s.dim, :s.kv_rank] = uk.to(self.device)
             kv[s.heads * dk:].view(s.heads, dv, rank_p)[:, :s.vdim, :s.kv_rank] = uv.to(self.device)
             L["ukv"] = kv
-        L["inv_freq"] = torch.tensor(rope_frequencies(s)[0], dtype=torch.float64).to(self.device, torch.float32)
+        L["rot"] = self._rotation(s)
         L["o"] = self._heads_in(m["o"], s.heads, s.vdim)
 
     def _load_hgrn2(self, s: LayerSpec, m: dict, L: dict) -> None:
@@ -223,7 +265,7 @@ class HybridRunner(DeviceRunner):
             if "o.b" in w:
                 bias[:self.cfg.hidden_size] += scale * self._vec(w["o.b"])
             L["parts"].append(P)
-        L["in"], L["o"] = torch.cat(rows, 0), torch.cat(cols, 1)
+        L["in"], L["o"] = self._with_gate(1, torch.cat(rows, 0), L), torch.cat(cols, 1)
         L["o_bias"] = bias if any(p.out_bias for p in s.mixers()) else None
 
     _load_parallel = _load_attention = _load_rglru = _load_parts
@@ -236,11 +278,13 @@ class HybridRunner(DeviceRunner):
         P["tc"] = hy.prefill_tc_values(s.dim, 0, s.vdim, s.scale) == P["dvp"]
         P["kv_heads"] = s.kv_heads if s.kv_from < 0 else 0
         P["q_norm"], P["k_norm"] = (self._vec(w[k + ".norm"]) if s.qk_norm and k in own else None for k in "qk")
-        P["rot"] = None
-        if s.rot_dim:
-            freq, scale = rope_frequencies(s)
-            P["rot"] = hy.Rotation(s.rot_dim, torch.tensor(freq, dtype=torch.float64).to(self.device), scale, s.rot_pairs == "next")
-        rows = [w[k] for k in own] + ([w["g"]] if s.head_gate else [])
+        P["temp"] = self._vec(w["temp"]) if s.head_temp else None
+        P["table"] = None
+        if s.sigmoid:
+            P["table"] = hy.distance_table(w["rel"].to(self.device, torch.float32), distance_buckets(s.bias_rows, s.bias_max, s.chunk), self._vec(w["pb"]))
+        P["rot"] = self._rotation(s) if s.rot_dim else None
+        rows = [w[k] for k in own] + ([w["g"]] if s.head_gate or s.out_gate else [])
+        P["g_at"] = sum(r.shape[0] for r in rows) - rows[-1].shape[0] if s.out_gate else 0
         return self._mat(torch.cat(rows, 0), None, self.dp), self._heads_in(w["o"], s.heads, s.vdim)
 
     def _load_part_rglru(self, s: LayerSpec, w: dict, P: dict):
@@ -260,6 +304,9 @@ class HybridRunner(DeviceRunner):
     def _load_mlp_poly(self, s: LayerSpec, w: dict, L: dict) -> None:
         L["up"], L["down"], L["act"] = self._mat(w["up"], None, self.dp), self._mat(w["down"], self.dp, pad(s.ff)), self._vec(w["act"])
 
+    def _load_mlp_plain(self, s: LayerSpec, w: dict, L: dict) -> None:
+        L["up"], L["down"] = self._with_gate(2, self._mat(w["up"], None, self.dp), L), self._mat(w["down"], self.dp, pad(s.ff))
+
     def _load_mlp_gated(self, s: LayerSpec, w: dict, L: dict) -> None:
         L["gu"], L["down"] = self._glu(w["gate"], w["up"]), self._mat(w["down"], self.dp, pad(s.ff, 16))
 
@@ -270,7 +317,7 @@ class HybridRunner(DeviceRunner):
             return self._glu(w[name + ".gate"], w[name + ".up"]) if s.glu else self._mat(w[name + ".up"], pad(ff, 16), self.dp)
 
         # the gate of the shared expert is one more row of the router's matrix
-        L["router"] = self._mat(torch.cat([w["router"], w["shared.sg"]], 0) if s.shared_gate else w["router"], None, self.dp)
+        L["router"] = self._with_gate(2, self._mat(torch.cat([w["router"], w["shared.sg"]], 0) if s.shared_gate else w["router"], None, self.dp), L)
         L["router_b"], L["correction"] = (self._vec(w[k]) if k in w else None for k in ("router.b", "correction"))
         n = (2 if s.glu else 1) * ffp
         L["e_in"] = torch.empty(s.experts * n, self.dp, dtype=self.dtype, device=self.device)
@@ -389,6 +436,7 @@ class HybridRunner(DeviceRunner):
         cfg, dp, d, eps, m = self.cfg, self.dp, self.cfg.hidden_size, self.cfg.norm_eps, self.cfg.residual_mult
         M, dev = b.M, self.device
         x, h = self._new(M, dp, torch.float32), self._new(M, dp)
+        wide = self._new(M, cfg.streams * dp, torch.float32) if cfg.streams > 1 else x
         hist = None
         if cfg.depth_average:
             hist = torch.empty((len(self.layers) + 1, M if M <= 1024 else pad(M, 1024), dp), dtype=torch.float32, device=dev)
@@ -399,17 +447,25 @@ class HybridRunner(DeviceRunner):
                 return dict(w_next=self.final_norm, h=h) if want_hidden else {}
             return {} if cfg.layers[i].type == "wkv" else dict(w_next=self.layers[i]["pre1"], h=h)      # a token-shift mixer norms its own input
 
+        def boundary(k: int, L: dict, cur, sub: Sublayer, **kw):
+            """The stream (or its copies) behind sublayer ``k``."""
+            st = L.get(f"hc{k}")
+            out = cur if st is None else x if st.n_out == 1 else wide
+            hy.residual_step(out, L[f"post{k}"], d, eps, sub=sub, x_in=cur, mult=m, streams=st, **kw)
+            return out
+
         hy.residual_step(x, self.embed_norm, d, eps, mult=cfg.embed_scale, tokens=b.tokens, table=self.embed, freq=self.pos_freq, pos=b.pos,
-                         hist=hist, hist_n=0, **feed(0))
+                         hist=hist, hist_n=0, streams=self._embed_streams if cfg.streams else None, **feed(0))
+        cur = x
         for i, (s, L) in enumerate(zip(cfg.layers, self.layers)):
-            y, post = getattr(self, "_mix_" + s.type)(i, s, L, x, h, b), L["post1"]
+            y, k = getattr(self, "_mix_" + s.type)(i, s, L, cur, h, b), 1
             if s.has_mlp:
-                hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, w_next=L["pre2"], h=h)
-                y, post = getattr(self, "_mlp_" + s.mlp)(s, L, x, h, b), L["post2"]
-            hy.residual_step(x, post, d, eps, sub=y, x_in=x, mult=m, hist=hist, hist_n=i + 1, avg=L["dwa"], **feed(i + 1))
+                cur = boundary(1, L, cur, y, w_next=L["pre2"], h=h)
+                y, k = getattr(self, "_mlp_" + s.mlp)(s, L, cur, h, b), 2
+            cur = boundary(k, L, cur, y, hist=hist, hist_n=i + 1, avg=L["dwa"], **feed(i + 1))
             if capture is not None:
-                capture.append(x[:, :d].clone())
-        return x, h
+                capture.append(cur.view(M, -1, dp)[..., :d].sum(1))
+        return cur, h
 
     # -- feed-forwards ----------------------------------------------------------------------------------------
     def _mlp_poly(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
@@ -428,15 +484,22 @@ class HybridRunner(DeviceRunner):
             return a
         return hy.gated_act(self._mm_take(b, name, h, W), a, act)
 
-    def _act_product(self, b: Ragged, name: str, h, W, act: str) -> torch.Tensor:
-        """``act(h W^T)``, likewise."""
-        a = self._new(b.M, W.shape[0])
+    def _act_product(self, b: Ragged, name: str, h, W, act: str, n: int = 0) -> tuple[torch.Tensor, Out | None]:
+        """``act`` of the first ``n`` columns of ``h W^T`` (0: all), likewise, and the product itself where the columns behind them
+        are to be taken from."""
+        n = n or W.shape[0]
         if not self.exact32 and self._small_plan(b, W)[1] == 1 and act == "relu2":
             from ..ops.gemm import gemm_tn
 
             bn, _, pair = self._small_plan(b, W)
-            return gemm_tn(h, W, out=a, relu2=True, bn=bn, two_cta=pair)
-        return hy.plain_act(self._mm_take(b, name, h, W), a, act)
+            z = gemm_tn(h, W, out=self._new(b.M, W.shape[0]), relu2=True, relu2_cols=n, bn=bn, two_cta=pair)
+            return z[:, :n], as_out(z)
+        z = self._mm_take(b, name, h, W)
+        return hy.plain_act(z, self._new(b.M, n), act), z
+
+    def _mlp_plain(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
+        a, z = self._act_product(b, "up", h, L["up"], s.act, pad(s.ff))
+        return Sublayer(self._mm_take(b, "down", a, L["down"]), **self._gate_of(2, z, L))
 
     def _mlp_gated(self, s: LayerSpec, L, x, h, b: Ragged) -> Sublayer:
         return Sublayer(self._mm_take(b, "down", self._glu_product(b, "gu", h, L["gu"], s.act), L["down"]))
@@ -445,9 +508,9 @@ class HybridRunner(DeviceRunner):
         from ..ops import moe
 
         z = self._mm_take(b, "router", h, L["router"], f32=True)
-        plan = moe.route(z.t[:, :s.experts + s.identity + s.shared_gate], s.top, True, L["router_b"], take=z.kind == hy.KIND_TAKE,
-                         correction=L["correction"], identity=s.identity, gate=s.shared_gate)
-        xp, n = moe.gather(h, plan), L["e_down"].shape[1]
+        plan = moe.route(z.t[:, :s.experts + s.identity + s.shared_gate], s.top, s.router != "softmax", L["router_b"], take=z.kind == hy.KIND_TAKE,
+                         correction=L["correction"], identity=s.identity, gate=s.shared_gate, groups=s.groups, keep=s.group_keep, scale=s.router_scale)
+        xp, n, gate = moe.gather(h, plan), L["e_down"].shape[1], self._gate_of(2, z, L)
         a = torch.empty((plan.cap_rows, n), dtype=self.dtype, device=self.device)
         if self.exact32:
             z = as_out(moe.grouped_gemm(xp, L["e_in"], plan, (2 if s.glu else 1) * n))
@@ -459,10 +522,11 @@ class HybridRunner(DeviceRunner):
         rows = moe.grouped_gemm(a, L["e_down"], plan, self.dp)
         y = None
         if s.shared_ff:
-            y = self._mm_take(b, "down", (self._glu_product if s.glu else self._act_product)(b, "s_in", h, L["s_in"], s.act), L["down"])
+            a = self._glu_product(b, "s_in", h, L["s_in"], s.act) if s.glu else self._act_product(b, "s_in", h, L["s_in"], s.act)[0]
+            y = self._mm_take(b, "down", a, L["down"])
         # experts that are the identity take the sublayer's input, in 32-bit where that is the stream itself
         return Sublayer(y, rows=rows, pos=plan.pos, weight=plan.topw, gate=plan.gate,
-                        identity=as_out(h if self.cfg.pre_norms else x) if s.identity else None)
+                        identity=as_out(h if self.cfg.pre_norms else x) if s.identity else None, **gate)
 
     # -- mixers -------------------------------------------------------------------------------------------------
     def _mix_latent_attention(self, i, s, L, x, h, b: Ragged) -> Sublayer:
@@ -475,29 +539,29 @@ class HybridRunner(DeviceRunner):
             qn, qr = self._heads_buf("qn", H, n_abs, b, dk), self._heads_buf("qr", H, n_abs, b, rot_p)
         if n_abs < M:
             qe = self._new(M - n_abs, H * (dk + rot_p))
-        hy.latent_finish(p, L["c_norm"], L["inv_freq"], b.pos, b.slot, cache, n_abs, qn, qr, qe, H, s.dim, s.rot_dim, s.kv_rank,
-                         self.cfg.norm_eps)
+        hy.latent_finish(p, L["c_norm"], L["rot"], b.pos, b.slot, cache, n_abs, qn, qr, qe, H, s.dim, s.kv_rank, self.cfg.norm_eps)
+        gate, weights = self._gate_of(1, p, L), hy.KeyWeights(sink=L["sink"])
         o = self._new(M, H * vp)
         if n_abs:
             ql, ol = self._heads_buf("ql", H, n_abs, b, rank_p), self._heads_buf("ol", H, n_abs, b, rank_p)
             hy.gemm_batched(qn, L["uk_t"], ql.view(-1, rank_p), n_abs, c_batch=ql.stride(0))
             if self.exact32 or rank_p + rot_p > LATENT_TC_MAX:
-                hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs)
+                hy.latent_attend(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs, sink=L["sink"])
             else:
                 keys = min(b.reach, s.window) if s.window > 0 else b.reach
                 hy.latent_decode(ql, qr, cache, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.scale, ol, n_abs,
-                                 hy.latent_decode_splits(n_abs, H, keys))
+                                 hy.latent_decode_splits(n_abs, H, keys), sink=L["sink"])
             hy.gemm_batched(ol, L["uv"], o, n_abs, c_batch=vp)
         if n_abs < M:
             plan = b.plan(s.window)
             c = hy.latent_gather(cache, b.bt, plan)
             if L["tc_dv"]:
                 k, vt = self._mm(c[:, :rank_p], L["ukv"][:H * dk]).t, self._mm(L["ukv"][H * dk:], c[:, :rank_p]).t
-                hy.latent_prefill_tc(qe, k, vt, c, plan, s.window, s.scale, o[n_abs:], H, dk, L["tc_dv"], rank_p, rot_p, s.vdim)
-                return Sublayer(self._mm_take(b, "o", o, L["o"]))
+                hy.latent_prefill_tc(qe, k, vt, c, plan, s.window, s.scale, o[n_abs:], H, dk, L["tc_dv"], rank_p, rot_p, s.vdim, weights=weights)
+                return Sublayer(self._mm_take(b, "o", o, L["o"]), **gate)
             kv = self._mm(c[:, :rank_p], L["ukv"]).t
-            hy.latent_prefill(qe, kv, c, plan, s.window, s.scale, o[n_abs:], H, dk, dv, rank_p, rot_p, s.vdim)
-        return Sublayer(self._mm_take(b, "o", o, L["o"]))
+            hy.latent_prefill(qe, kv, c, plan, s.window, s.scale, o[n_abs:], H, dk, dv, rank_p, rot_p, s.vdim, weights=weights)
+        return Sublayer(self._mm_take(b, "o", o, L["o"]), **gate)
 
     def _scan(self, mode, i, s, L, q, k, v, g, aux, bias, gate, b: Ragged) -> Sublayer:
         """Recurrence, per-head norm and gate, output projection."""
@@ -564,30 +628,37 @@ class HybridRunner(DeviceRunner):
         o = self._new(b.M, L["o"].shape[1])
         for j, (spec, P) in enumerate(zip(s.mixers(), L["parts"])):
             getattr(self, "_part_" + spec.type)(i, spec, P, p.col(P["in"]), o[:, P["out"]:], self.kv.part(i, j), b)
-        return Sublayer(self._mm_take(b, "o", o, L["o"]), bias=L["o_bias"])
+        return Sublayer(self._mm_take(b, "o", o, L["o"]), bias=L["o_bias"], **self._gate_of(1, p, L))
 
     _mix_parallel = _mix_attention = _mix_rglru = _mix_parts
 
     def _part_attention(self, i, s: LayerSpec, P, p: Out, o, cache, b: Ragged) -> None:
         M, n_abs, kv = b.M, b.n_abs, cache["kv"]
         H, G, dk, dvp = s.heads, s.heads // s.kv_heads, pad(s.dim, 16), P["dvp"]
-        q, gate = self._new(M, H * dk), None
-        if s.qk_norm or P["rot"] or s.head_gate or s.kv_from >= 0:
+        q, gate, cols, weights = self._new(M, H * dk), None, None, None
+        if s.out_gate:                       # the gate's logits stay in the projection, or leave its workspace with the rest
+            cols = self._new(M, H * pad(s.vdim)) if p.kind == hy.KIND_TAKE else None
+            weights = hy.KeyWeights(P["table"], cols=p.t[:, P["g_at"]:P["g_at"] + H * s.vdim] if cols is None else cols, pitch=s.vdim if cols is None else pad(s.vdim))
+        elif s.sigmoid:
+            weights = hy.KeyWeights(P["table"])
+        if s.out_gate or s.qk_norm or P["rot"] or s.head_gate or s.kv_from >= 0:
             gate = torch.empty((M, H), dtype=torch.float32, device=self.device) if s.head_gate else None
             hy.gqa_finish_norm(p, P["bias"], b.slot, kv, q, H, P["kv_heads"], s.dim, s.vdim, dvp, P["q_norm"], P["k_norm"], self.cfg.norm_eps, P["rot"],
-                               b.pos, gate)
+                               b.pos, gate, s.qk_norm_heads, P["temp"], cols, pad(s.vdim) if cols is not None else 0)
         else:
             hy.gqa_finish(p, P["bias"], b.slot, kv, q, H, s.kv_heads, s.dim, s.vdim, dvp)
         if n_abs:
             args = (q, kv, b.bt, b.row_seq, b.pos, b.ctx, s.window, s.chunk, s.scale, P["scale"], o, n_abs, H, s.kv_heads, s.dim, s.vdim, dvp)
             if self.exact32 or max(dk, dvp) > hy.GQA_DECODE_MAX:
-                hy.gqa_attend(*args, softcap=s.softcap, gate=gate)
+                hy.gqa_attend(*args, softcap=s.softcap, gate=gate, weights=weights)
             else:
                 reach = min([b.reach] + [w for w in (s.window, s.chunk) if w > 0])
-                hy.gqa_decode(*args, splits=hy.gqa_decode_splits(n_abs, s.kv_heads * ((G + 15) // 16), reach), softcap=s.softcap, gate=gate)
+                hy.gqa_decode(*args, splits=hy.gqa_decode_splits(n_abs, s.kv_heads * ((G + 15) // 16), reach), softcap=s.softcap, gate=gate,
+                              weights=weights)
         if n_abs < M:
             plan = b.plan(s.window, s.chunk)
-            rest = dict(chunk=s.chunk, G=G, out_scale=P["scale"], softcap=s.softcap, gate=gate[n_abs:] if gate is not None else None)
+            rest = dict(chunk=s.chunk, G=G, out_scale=P["scale"], softcap=s.softcap, gate=gate[n_abs:] if gate is not None else None,
+                        weights=weights.rows_from(n_abs) if weights is not None else None)
             src = self.cfg.kv_layer(i)
             key = (src, s.window, s.chunk, P["tc"])
             got = b.kept.get(key)

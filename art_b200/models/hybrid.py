@@ -2,17 +2,20 @@
 
 A configuration consists of layers and of the frame around them.  A layer (``LayerSpec``) names
 
-* a mixer: latent attention with a sliding window, grouped-query attention with a window or in chunks, HGRN2 or lightning
-  linear attention, RWKV-style time mixing, a gated linear recurrent unit behind a short convolution, or several of these
-  side by side on the same input, each with a factor (``parts``).  Grouped-query attention may rotate its queries and keys
-  (either pairing, scaled frequencies), norm them, squash its scores, gate its heads and read another layer's keys and values;
-* a feed-forward: PolyNorm, gated (``act(gate) * up``), a mixture of experts (gated or not, some of them the identity) with an
-  optional shared expert, or none.
+* a mixer: latent attention with a sliding window or a sink, grouped-query attention with a window or in chunks, HGRN2 or
+  lightning linear attention, RWKV-style time mixing, a gated linear recurrent unit behind a short convolution, or several of
+  these side by side on the same input, each with a factor (``parts``).  Grouped-query attention may rotate its queries and keys
+  (either pairing, scaled frequencies), norm them (all heads together or each), squash its scores, weigh keys by sigmoids of
+  scores with a bias by distance instead of a softmax, gate its heads or its result's columns and read another layer's keys and
+  values;
+* a feed-forward: PolyNorm, plain (``act(up)``), gated (``act(gate) * up``), a mixture of experts (gated or not, some of them the
+  identity, chosen among all or among the best groups) with an optional shared expert, or none.
 
 The frame (fields of ``HybridConfig``) is the design's: norms before, after, or before and after each sublayer, norm weights
-stored as they are or around zero, a factor per column on each sublayer's result, a residual multiplier, a weighted average
-over the results of all earlier layers, an embedding that is normalised, or scaled and given sinusoidal position vectors, an
-output table of its own or the embedding's.
+stored as they are or around zero, a factor per column or a gate on each sublayer's result, a residual multiplier, a weighted
+average over the results of all earlier layers, hyper-connections (several copies of the residual stream that every sublayer
+reads and mixes), an embedding that is normalised, or scaled and given sinusoidal position vectors, an output table of its own
+or the embedding's.
 
 ``HybridConfig`` answers the questions the engine asks of any configuration (``vocab_size``, ``hidden_size``,
 ``num_layers``, ``is_moe`` ...); ``from_design_dict`` reads a ``config.json`` whose ``architecture`` key names a design of
@@ -31,6 +34,8 @@ SHIFT_MIXES = ("r", "k", "v", "g", "w")        # inputs of the token-shift mixer
 PART_NAMES = ("left", "right")                 # tensors of a parallel mixer's parts
 RECURRENT = ("hgrn2", "wkv", "lightning", "rglru")
 MAX_EXPERTS, MAX_TOP = 256, 16                 # what the router kernel holds
+MAX_STREAMS = 8                                # ... and the one that mixes the copies of the residual stream
+GATED_SUBLAYERS = ("latent_attention", "attention", "rglru", "parallel", "plain", "moe")      # whose input product takes a residual gate's rows, too
 
 
 @dataclass
@@ -54,8 +59,15 @@ class LayerSpec:
     biases: bool = False                       # q, k and v projections have biases
     out_bias: bool = False                     # ... and the output projection
     qk_norm: bool = False                      # RMS norm over all heads of q together, and of k, before the rotation
+    qk_norm_heads: bool = False                # ... over each head instead, with one head's weights
+    head_temp: bool = False                    # scores have a learned factor per head (with qk_norm_heads)
     softcap: float = 0.0                       # scores pass softcap * tanh(score / softcap); 0: as they are
+    sigmoid: bool = False                      # a key weighs sigmoid(score + its distance's bias + the head's), without normalisation
+    bias_max: float = 0.0                      # distance at which the logarithmic buckets of the bias end
+    bias_rows: int = 0                         # ... and their number (given by the tensor, not by the configuration)
+    sink: bool = False                         # the softmax's denominator has a learned term per head (latent attention)
     head_gate: bool = False                    # heads are multiplied by the sigmoid of a projection of the input
+    out_gate: bool = False                     # all columns of the heads are
     kv_from: int = -1                          # layer whose keys and values this one reads; -1: its own
     # wkv: width of the low-rank decay projection (given by its tensors, not by the configuration)
     decay_rank: int = 0
@@ -63,7 +75,7 @@ class LayerSpec:
     conv: int = 1                              # rglru: taps of the short convolution
     parts: tuple["LayerSpec", ...] = ()        # parallel: mixers side by side, and the factor of each one's result
     part_scales: tuple[float, ...] = ()
-    # feed-forward: "poly" (up, PolyNorm, down), "gated" (act(gate) * up, down) or "moe" (experts)
+    # feed-forward: "poly" (up, PolyNorm, down), "plain" (act(up), down), "gated" (act(gate) * up, down) or "moe" (experts)
     mlp: str = "poly"
     act: str = "silu"
     glu: bool = True                           # experts are act(gate) * up, down; else act(up), down
@@ -71,7 +83,11 @@ class LayerSpec:
     top: int = 0
     expert_ff: int = 0
     identity: int = 0                          # further outputs of the router that hand the input on
-    router: str = "logits"                     # chooses by "logits" (+ bias, softmax over the chosen) or "scores" (softmax over all, + correction)
+    router: str = "logits"                     # chooses by "logits" (+ bias, softmax over the chosen) or "scores" (softmax over all, + correction);
+                                               # "softmax": by the softmax over all, which are the weights
+    groups: int = 1                            # experts form equal groups of neighbours, of which the best ones can be chosen from
+    group_keep: int = 1
+    router_scale: float = 1.0                  # factor of the weights
     shared_ff: int = 0                         # shared expert, 0: none
     shared_gate: bool = False                  # the shared expert is multiplied by the sigmoid of a projection of the input
 
@@ -102,6 +118,8 @@ class HybridConfig:
     pre_norms: bool = True                     # a norm before each sublayer; without, sublayers read the residual stream itself
     post_norms: bool = True                    # a norm behind each sublayer
     layer_scale: bool = False                  # each sublayer's result (behind its norm) has a factor per column
+    residual_gate: bool = False                # each sublayer's result is multiplied by sigmoid(W h + b), h being its input
+    streams: int = 0                           # hyper-connections: copies of the residual stream; 0: one stream, plain sums
     depth_average: bool = True                 # layer results are averaged with all earlier ones
     norm_offset: float = 0.0                   # added to the weights of the frame's norms
     embed_norm: bool = True
@@ -149,6 +167,7 @@ class HybridConfig:
             _check_layer(i, s)
             if s.kv_from >= 0:
                 _check_shared(cfg, i, s)
+        _check_frame(cfg)
         return cfg
 
 
@@ -162,6 +181,14 @@ def _check_layer(i: int, s: LayerSpec) -> None:
             raise ValueError(f"layer {i}: {len(p.decay)} decay factors for {p.heads} heads")
         if p.type in ("hgrn2", "wkv", "lightning") and max(p.dim, p.vdim) > 256:
             raise ValueError(f"layer {i}: {p.type} heads of more than 256 columns are not supported")
+        if p.head_temp and not p.qk_norm_heads:
+            raise ValueError(f"layer {i}: a factor per head goes with a norm of each head")
+        if p.sigmoid and p.bias_max <= 0:
+            raise ValueError(f"layer {i}: bias_max must be positive, not {p.bias_max}")
+    if s.groups < 1 or (s.experts and ((s.experts + s.identity) % s.groups or not 1 <= s.group_keep <= s.groups)):
+        raise ValueError(f"layer {i}: {s.group_keep} of {s.groups} groups of {s.experts + s.identity} experts are not supported")
+    if s.experts and s.top > (s.experts + s.identity) // s.groups * s.group_keep:
+        raise ValueError(f"layer {i}: {s.group_keep} groups have fewer than {s.top} experts")
     outputs = s.experts + s.identity
     if s.experts and not (0 < s.top <= min(outputs, MAX_TOP) and outputs <= MAX_EXPERTS):
         raise ValueError(f"layer {i}: {s.top} of {outputs} experts (at most {MAX_TOP} of {MAX_EXPERTS}) are not supported")
@@ -173,6 +200,31 @@ def _check_shared(cfg: HybridConfig, i: int, s: LayerSpec) -> None:
         raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys and values of its own")
     if (src.kv_heads, src.dim, src.vdim) != (s.kv_heads, s.dim, s.vdim):
         raise ValueError(f"layer {i}: its key heads differ from those of layer {s.kv_from}, whose keys and values it reads")
+
+
+def _check_frame(cfg: HybridConfig) -> None:
+    if not 0 <= cfg.streams <= MAX_STREAMS:
+        raise ValueError(f"{cfg.streams} streams are not supported (at most {MAX_STREAMS})")
+    plain = cfg.pre_norms and not (cfg.post_norms or cfg.depth_average or cfg.embed_norm or cfg.layer_scale or cfg.position_base)
+    if cfg.streams and not (plain and cfg.embed_scale == 1.0 and cfg.residual_mult == 1.0 and not any(s.type == "wkv" for s in cfg.layers)):
+        raise ValueError("hyper-connections go with norms before the sublayers and nothing else around them")
+    for i, s in enumerate(cfg.layers if cfg.residual_gate else ()):
+        bad = [k for k in (s.type, s.mlp if s.has_mlp else "plain") if k not in GATED_SUBLAYERS]
+        if bad or not cfg.pre_norms or cfg.post_norms:
+            raise ValueError(f"layer {i}: a residual gate is not supported with {bad[0] if bad else 'these norms'}")
+
+
+def distance_buckets(rows: int, reach: float, chunk: int = 0) -> list[int]:
+    """Row of a distance bias's table for every distance from 0 on, up to the first one that has the row of all farther ones
+    (or to the end of a chunk): a row per distance in the near half of the rows, then logarithmic up to ``reach``."""
+    half = rows // 2
+    if half < 1 or reach <= half:
+        raise ValueError(f"a distance bias of {rows} rows up to distance {reach} is not supported")
+    out: list[int] = []
+    while not (out and (out[-1] == rows - 1 or len(out) in (chunk, 1 << 20))):
+        n = len(out)
+        out.append(n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / math.log(reach / half) * (rows - half))))
+    return out
 
 
 def rope_frequencies(s: LayerSpec) -> tuple[list[float], float]:
@@ -216,6 +268,10 @@ def _mlp_kind(i: int, mlp: dict | None, supported: tuple[str, ...]) -> str | Non
     return kind
 
 
+def _scaling(rot: dict) -> tuple[float, float, float, float] | None:
+    return tuple(float(rot["scaling"][k]) for k in ("factor", "original", "fast", "slow")) if rot.get("scaling") else None
+
+
 def _read_nikelix(d: dict, name: str) -> HybridConfig:
     layers = []
     for i, e in enumerate(d["layers"]):
@@ -224,7 +280,7 @@ def _read_nikelix(d: dict, name: str) -> HybridConfig:
         spec = LayerSpec(kind, int(m["heads"]), int(m["dim"]), int(m.get("vdim", m["dim"])), int(mlp["ff"]) if mlp else 0)
         if kind == "latent_attention":
             rot = m["rot"]
-            spec.rot_dim, spec.kv_rank = int(m["rot_dim"]), int(m["kv_rank"])
+            spec.rot_dim, spec.kv_rank, spec.rot_pairs = int(m["rot_dim"]), int(m["kv_rank"]), "next"
             spec.scale, spec.rope_base = float(m["scale"]), float(rot["base"])
             spec.window = int((m.get("mask") or {}).get("size", 0))
             if int(rot.get("dims", spec.rot_dim)) != spec.rot_dim:
@@ -273,8 +329,7 @@ def _read_gaborax(d: dict, name: str) -> HybridConfig:
         spec = LayerSpec("attention", int(m["heads"]), int(m["dim"]), int(m["vdim"]), kv_heads=int(m["kv_heads"]), scale=float(m["scale"]),
                          rot_dim=int(rot["dims"]), rope_base=float(rot["base"]), rot_pairs="half" if first else "next", qk_norm=True,
                          biases=not first, head_gate=first, softcap=float(m.get("softcap") or 0.0))
-        if rot.get("scaling"):
-            spec.rope_scaling = tuple(float(rot["scaling"][k]) for k in ("factor", "original", "fast", "slow"))
+        spec.rope_scaling = _scaling(rot)
         if m.get("kv_from") is not None:
             spec.kv_from = int(m["kv_from"])
             if spec.kv_from < 0:
@@ -289,10 +344,46 @@ def _read_gaborax(d: dict, name: str) -> HybridConfig:
                         **GABORAX_FRAME)
 
 
+def _read_gaparax(d: dict, name: str) -> HybridConfig:
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        kind, m, mlp = _mixer_kind(i, e, ("attention", "latent_attention")), e["mixer"], e.get("mlp")
+        spec = LayerSpec(kind, int(m["heads"]), int(m["dim"]), int(m["vdim"]), scale=float(m["scale"]))
+        if kind == "attention":
+            _known(i, "mixer", m, ("heads", "kv_heads", "dim", "vdim", "scale", "softcap", "bias_max", "mask"))
+            _known(i, "mask", m.get("mask") or {}, ("size",))
+            spec.kv_heads, spec.chunk = int(m["kv_heads"]), int((m.get("mask") or {}).get("size", 0))
+            spec.softcap, spec.bias_max, spec.sigmoid = float(m.get("softcap") or 0.0), float(m["bias_max"]), True
+            spec.qk_norm = spec.qk_norm_heads = spec.head_temp = spec.out_gate = True
+        else:
+            _known(i, "mixer", m, ("heads", "dim", "rot_dim", "kv_rank", "vdim", "rot", "scale"))
+            rot = m["rot"]
+            _known(i, "rot", rot, ("base", "dims", "scaling"))
+            spec.rot_dim, spec.kv_rank, spec.rope_base, spec.rope_scaling = int(m["rot_dim"]), int(m["kv_rank"]), float(rot["base"]), _scaling(rot)
+            spec.sink = True
+            if int(rot.get("dims", spec.rot_dim)) != spec.rot_dim or spec.rot_dim % 2:
+                raise ValueError(f"layer {i}: rot.dims must equal rot_dim, an even number (the whole rotated part turns)")
+        ff = _mlp_kind(i, mlp, ("dense", "moe"))
+        if ff == "dense":
+            spec.mlp, spec.act, spec.ff = "plain", "relu2", int(mlp["ff"])
+        elif ff == "moe":
+            _known(i, "mlp", mlp, ("kind", "expert", "router"))
+            r = mlp["router"]
+            _known(i, "router", r, ("experts", "top", "groups", "scale"))
+            spec.mlp, spec.router, spec.expert_ff, spec.experts, spec.top = "moe", "softmax", int(mlp["expert"]["ff"]), int(r["experts"]), int(r["top"])
+            spec.router_scale = float(r.get("scale", 1.0))
+            if r.get("groups"):
+                spec.groups, spec.group_keep = int(r["groups"]["count"]), int(r["groups"]["keep"])
+        layers.append(spec)
+    return HybridConfig(name=name, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers, norm_eps=float(d["norm"]["eps"]),
+                        streams=int(d["streams"]), **GAPARAX_FRAME)
+
+
 NASELORN_FRAME = dict(family="naselorn", post_norms=False, depth_average=False, norm_offset=1.0, embed_norm=False, position_base=10000.0,
                       tie_word_embeddings=False)
 GABORAX_FRAME = dict(family="gaborax", pre_norms=False, post_norms=True, layer_scale=True, depth_average=False, norm_offset=1.0, embed_norm=False)
-ARCHITECTURES = {"Nikelix": _read_nikelix, "Naselorn": _read_naselorn, "Gaborax": _read_gaborax}
+GAPARAX_FRAME = dict(family="gaparax", post_norms=False, depth_average=False, embed_norm=False, residual_gate=True, tie_word_embeddings=False)
+ARCHITECTURES = {"Nikelix": _read_nikelix, "Naselorn": _read_naselorn, "Gaborax": _read_gaborax, "Gaparax": _read_gaparax}
 
 
 def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
@@ -301,7 +392,7 @@ def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
         return {f"{n}.{k}": t for n, p in zip(PART_NAMES, s.parts) for k, t in _mixer_shapes(p, d).items()}
     if s.type == "latent_attention":
         return {"q": (s.heads * (s.dim + s.rot_dim), d), "dkv": (s.kv_rank + s.rot_dim, d), "dkv.norm": (s.kv_rank,),
-                "uk": (qk, s.kv_rank), "uv": (v, s.kv_rank), "o": (d, v)}
+                "uk": (qk, s.kv_rank), "uv": (v, s.kv_rank), "o": (d, v), **({"sink": (s.heads,)} if s.sink else {})}
     if s.type == "hgrn2":
         return {"q": (qk, d), "f": (qk, d), "f.b": (qk,), "lower": (qk,), "v": (v, d), "norm": (s.vdim,), "o": (d, v)}
     if s.type == "lightning":
@@ -316,9 +407,13 @@ def _mixer_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
         if s.out_bias:
             out["o.b"] = (d,)
         if s.qk_norm:
-            out.update({k + ".norm": (own[k][0],) for k in "qk" if k in own})
-        if s.head_gate:
-            out["g"] = (s.heads, d)
+            out.update({k + ".norm": (s.dim if s.qk_norm_heads else own[k][0],) for k in "qk" if k in own})
+        if s.head_gate or s.out_gate:
+            out["g"] = (v if s.out_gate else s.heads, d)
+        if s.head_temp:
+            out["temp"] = (s.heads,)
+        if s.sigmoid:
+            out.update({"rel": (s.bias_rows, s.heads), "pb": (s.heads,)})
         return out
     if s.type == "rglru":
         gates = {k: t for g in ("ra", "ri") for k, t in ((g, (s.heads, s.dim, s.dim)), (g + ".b", (s.heads, s.dim)))}
@@ -335,12 +430,16 @@ def _mlp_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
 
     if s.mlp == "poly":
         return {"up": (s.ff, d), "down": (d, s.ff), "act": (4,)}
+    if s.mlp == "plain":
+        return {"up": (s.ff, d), "down": (d, s.ff)}
     if s.mlp == "gated":
         return glu("", s.ff)
     form = glu if s.glu else lambda pre, ff: {pre + "up": (ff, d), pre + "down": (d, ff)}
     out = {k: t for e in range(s.experts) for k, t in form(f"e{e}.", s.expert_ff).items()}
     n = s.experts + s.identity
-    out.update({"router": (n, d), "router.b" if s.router == "logits" else "correction": (n,)})
+    out["router"] = (n, d)
+    if s.router != "softmax":
+        out["router.b" if s.router == "logits" else "correction"] = (n,)
     if s.shared_ff:
         out.update(form("shared.", s.shared_ff))
         if s.shared_gate:
@@ -349,7 +448,8 @@ def _mlp_shapes(s: LayerSpec, d: int) -> dict[str, tuple[int, ...]]:
 
 
 def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
-    """Name -> shape of every tensor of a checkpoint.  The decay rank of a wkv layer is taken from its spec."""
+    """Name -> shape of every tensor of a checkpoint.  The decay rank of a wkv layer and the rows of a distance bias are taken
+    from the layer's spec."""
     d = cfg.hidden_size
     out: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, d), "final.norm": (d,)}
     if cfg.embed_norm:
@@ -362,6 +462,11 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
             out.update({p + n: (d,) for n in cfg.norm_names(k) if n})
             if cfg.layer_scale:
                 out[f"{p}ls{k}"] = (d,)
+            if cfg.residual_gate:
+                out.update({f"{p}rg{k}": (d, d), f"{p}rg{k}.b": (d,)})
+            if cfg.streams:
+                n = cfg.streams
+                out.update({f"{p}hc{k}.in": (n,), f"{p}hc{k}.out": (n,), f"{p}hc{k}.mix": (n, n)})
         if s.has_mlp:
             out.update({p + "mlp." + k: t for k, t in _mlp_shapes(s, d).items()})
         out.update({p + "mix." + k: t for k, t in _mixer_shapes(s, d).items()})
@@ -371,11 +476,16 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple[int, ...]]:
 
 
 def check_weights(cfg: HybridConfig, w: dict[str, torch.Tensor]) -> None:
-    """Fills in the decay ranks from the tensors and raises when a tensor is missing or has another shape."""
+    """Fills in the sizes that only the tensors give and raises when a tensor is missing or has another shape."""
     for i, s in enumerate(cfg.layers):
         w1 = w.get(f"l{i}.mix.w1")
         if s.type == "wkv" and w1 is not None:
             s.decay_rank = int(w1.shape[0])
+        for p, pre in zip(s.mixers(), PART_NAMES if s.parts else ("",)):
+            rel = w.get(f"l{i}.mix.{pre + '.' if pre else ''}rel")
+            if p.sigmoid and rel is not None:
+                p.bias_rows = int(rel.shape[0])
+                distance_buckets(p.bias_rows, p.bias_max)
     for k, shape in tensor_shapes(cfg).items():
         if k not in w:
             raise ValueError(f"checkpoint of {cfg.name} lacks tensor {k!r}")
@@ -398,6 +508,9 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
     for s in cfg.layers:
         if s.type == "wkv" and not s.decay_rank:
             s.decay_rank = max(8, cfg.hidden_size // 64 // 8 * 8)
+        for p in s.mixers():
+            if p.sigmoid and not p.bias_rows:
+                p.bias_rows = max(2, min(32, int(p.bias_max) // 2 * 2))
     w: dict[str, torch.Tensor] = {}
     frame = ("norm1", "norm1b", "norm2", "norm2b", "final.norm", "embed.norm")
     for k, shape in tensor_shapes(cfg).items():
@@ -422,7 +535,15 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
             w[k] = rnd(*shape, std=0.2, mean=0.8)
         elif leaf == "correction":             # moves a choice now and then
             w[k] = rnd(*shape, std=0.3 / shape[0])
-        elif leaf in ("u", "f.b") or leaf.endswith(".b"):
+        elif leaf in ("in", "out") and ".hc" in k:      # streams stay of one size: about their mean goes in, a share comes out
+            w[k] = rnd(*shape, std=0.3 / shape[0], mean=1.0 / shape[0] if leaf == "in" else 0.8)
+        elif leaf == "mix":
+            w[k] = (torch.eye(shape[0], device=device) * 0.8 + 0.2 / shape[0]).to(dtype) + rnd(*shape, std=0.05)
+        elif leaf == "temp":
+            w[k] = rnd(*shape, std=0.2, mean=1.0)
+        elif leaf in ("rel", "pb", "sink"):
+            w[k] = rnd(*shape, std=0.7)
+        elif leaf in ("u", "f.b", "b") or leaf.endswith(".b"):
             w[k] = rnd(*shape, std=0.5)
         else:
             w[k] = rnd(*shape, std=shape[-1] ** -0.5)
@@ -432,7 +553,7 @@ def init_hybrid_weights(cfg: HybridConfig, seed: int = 0, dtype: torch.dtype = t
 def _preset(name: str, width: int, ff: int, heads: int, n_layers: int, vocab: int = 32000, window: int = 1024) -> HybridConfig:
     """``n_layers`` layers that repeat (latent attention, hgrn2, wkv, hgrn2) at the proportions of a model this wide."""
     hd = width // heads
-    la = LayerSpec("latent_attention", heads, 128, 128, ff, rot_dim=64, kv_rank=512, scale=192 ** -0.5, rope_base=5e5, window=window)
+    la = LayerSpec("latent_attention", heads, 128, 128, ff, rot_dim=64, kv_rank=512, scale=192 ** -0.5, rope_base=5e5, rot_pairs="next", window=window)
     hg = LayerSpec("hgrn2", heads, hd, hd, ff)
     wk = LayerSpec("wkv", width // 64, 64, 64, ff, decay_rank=64)
     cycle = (la, hg, wk, hg)
@@ -476,10 +597,32 @@ def _gaborax_tiny() -> HybridConfig:
     return HybridConfig("gaborax-tiny", 512, 128, [a, b, dataclasses.replace(a, kv_from=0)], **GABORAX_FRAME)
 
 
+def _gaparax_preset(name: str, width: int, n_layers: int, experts: int, top: int, expert_ff: int, dense_ff: int, vocab: int = 32000,
+                    chunk: int = 1024) -> HybridConfig:
+    """``n_layers`` layers, every fourth one latent attention, the others chunked attention; the first has a dense feed-forward."""
+    hd, heads = 128, width // 128
+    la = LayerSpec("latent_attention", heads, 128, 128, rot_dim=64, kv_rank=512, scale=192 ** -0.5, rope_base=5e5, rope_scaling=(4.0, 8192, 32, 1), sink=True)
+    at = LayerSpec("attention", heads, hd, hd, kv_heads=max(1, heads // 4), scale=hd ** -0.5, chunk=chunk, qk_norm=True, qk_norm_heads=True, head_temp=True,
+                   softcap=30.0, sigmoid=True, bias_max=256, out_gate=True)
+    moe = dict(mlp="moe", router="softmax", experts=experts, top=top, groups=8, group_keep=4, router_scale=2.5, expert_ff=expert_ff)
+    layers = [dataclasses.replace(la if i % 4 == 3 else at, **moe) for i in range(n_layers)]
+    layers[0] = dataclasses.replace(at, mlp="plain", act="relu2", ff=dense_ff)
+    return HybridConfig(name=name, vocab_size=vocab, hidden_size=width, layers=layers, streams=2, **GAPARAX_FRAME)
+
+
+def _gaparax_tiny() -> HybridConfig:
+    moe = dict(mlp="moe", router="softmax", experts=6, top=3, groups=3, group_keep=2, router_scale=1.5, expert_ff=48)
+    at = LayerSpec("attention", 4, 32, 24, kv_heads=2, scale=0.2, chunk=40, qk_norm=True, qk_norm_heads=True, head_temp=True, softcap=15.0, sigmoid=True,
+                   bias_max=60, out_gate=True)
+    la = LayerSpec("latent_attention", 3, 24, 40, rot_dim=16, kv_rank=56, scale=0.15, rope_scaling=(3.0, 128, 16, 1), sink=True)
+    return HybridConfig("gaparax-tiny", 512, 128, [dataclasses.replace(at, mlp="plain", act="relu2", ff=200), dataclasses.replace(la, **moe), at], streams=3,
+                        **GAPARAX_FRAME)
+
+
 HYBRID_PRESETS: dict[str, HybridConfig] = {
     "nikelix-tiny": HybridConfig("nikelix-tiny", 512, 128, [
         LayerSpec("hgrn2", 2, 24, 40, 192), LayerSpec("latent_attention", 3, 16, 24, 256, rot_dim=8, kv_rank=48, scale=0.2,
-                                                       rope_base=1e4, window=24),
+                                                       rope_base=1e4, rot_pairs="next", window=24),
         LayerSpec("wkv", 4, 16, 16, 0, decay_rank=8)], residual_mult=0.7),
     "nikelix-1b": _preset("nikelix-1b", 2048, 8192, 16, 16),
     "nikelix-7b": _preset("nikelix-7b", 4096, 16384, 32, 32),
@@ -493,4 +636,7 @@ HYBRID_PRESETS: dict[str, HybridConfig] = {
     "gaborax-tiny": _gaborax_tiny(),
     "gaborax-2b-a1b": _gaborax_preset("gaborax-2b-a1b", 2048, 16, 64, 8, 8, 768, 1536),
     "gaborax-14b-a4b": _gaborax_preset("gaborax-14b-a4b", 4096, 16, 64, 8, 8, 1536, 3072),
+    "gaparax-tiny": _gaparax_tiny(),
+    "gaparax-2b-a1b": _gaparax_preset("gaparax-2b-a1b", 2048, 16, 64, 8, 512, 8192),
+    "gaparax-14b-a4b": _gaparax_preset("gaparax-14b-a4b", 4096, 16, 64, 8, 1024, 16384),
 }

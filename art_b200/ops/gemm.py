@@ -53,7 +53,7 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
             bias: torch.Tensor | None = None, res_cols: int = 0,
             out_dtype: torch.dtype = torch.bfloat16, bn: int = 0, max_ctas: int = 0,
             two_cta: bool | None = None, swiglu_bwd_gu: torch.Tensor | None = None, gate_act: str = "silu",
-            keep_preact: bool = True, silu_cols: int = 0, relu2: bool = False) -> torch.Tensor | None:
+            keep_preact: bool = True, silu_cols: int = 0, relu2: bool = False, relu2_cols: int = 0) -> torch.Tensor | None:
     """``out[M,N] = a[M,K] @ b[N,K].T (+ a2[M,K2] @ b2[N,K2].T) (+ residual)``.
 
     ``swiglu_out`` ([M, N/2] bf16) selects the SwiGLU epilogue: ``b``'s rows must be
@@ -62,7 +62,7 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
     with ``keep_preact=False`` only ``swiglu_out`` is written and nothing is returned.
 
     ``silu_cols``: the first columns of the product leave through silu (bf16 output, no other epilogue); ``relu2``: all of
-    them through the square of relu.
+    them (with ``relu2_cols``: the first ones) through the square of relu.
 
     ``swiglu_bwd_gu`` ([M, 2N] bf16, the forward's interleaved gate|up pre-activations) selects the fused
     SwiGLU-backward epilogue: the product is taken as ``d(silu(gate) * up)`` and ``out`` ([M, 2N]) receives
@@ -105,7 +105,7 @@ def gemm_tn(a: torch.Tensor, b: torch.Tensor, *, a2: torch.Tensor | None = None,
     if relu2:
         if epi != EPI_BF16:
             raise ValueError("relu2: a plain bf16 product")
-        epi = EPI_RELU2
+        epi, res_cols = EPI_RELU2, relu2_cols
     if out is None and not drop:
         out = torch.empty((M, N), dtype=torch.float32 if epi == EPI_F32 else torch.bfloat16, device=a.device)
     if out is not None and (out.stride(1) != 1 or tuple(out.shape) != (M, 2 * N if epi == EPI_SWIGLU_BWD else N)):

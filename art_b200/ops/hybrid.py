@@ -8,6 +8,7 @@ leaves zero: ``Out`` carries the tensor together with that kind.
 from __future__ import annotations
 
 import ctypes
+import math
 from dataclasses import dataclass
 
 import torch
@@ -21,7 +22,7 @@ ACTS = {"silu": 0, "relu": 1, "relu2": 2}       # relu2: the square of relu
 KIND_BF16, KIND_F32, KIND_TAKE = 0, 1, 2
 _sigs = {
     "artb_residual_step": [ci, vp, vp, ci, cl, vp, ci, ci, vp, vp, ci, vp, cf, vp, vp, vp, ci, ci, vp, vp, cl, vp, ci, ci, vp, vp, vp, cl, ci, vp, vp,
-                           vp, ci, ci, ci, ci, cf, vp, vp],
+                           vp, ci, ci, ci, ci, cf, vp, vp, ci, ci, vp, vp, ci, ci, ci, vp],
     "artb_norm_shift_mix": [ci, vp, ci, vp, vp, ci, vp, cl, ci, vp, cl, vp, vp, vp, vp, ci, ci, ci, cf, vp, vp],
     "artb_poly_norm": [ci, vp, ci, ci, vp, vp, ci, ci, ci, ci, cf, vp],
     "artb_split_tanh": [ci, vp, ci, ci, vp, ci, ci, ci, ci, vp],
@@ -33,20 +34,21 @@ _sigs = {
     "artb_linear_decode": [ci, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci,
                            vp, ci, ci, vp, ci, ci, cf, vp, vp],
     "artb_lightning_prefill": [vp, vp, vp, ci, vp, vp, cl, ci, cl, vp, vp, vp, ci, ci, ci, ci, vp, ci, ci, vp, vp],
-    "artb_latent_finish": [ci, vp, ci, ci, vp, vp, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
+    "artb_latent_finish": [ci, vp, ci, ci, vp, vp, cf, ci, vp, vp, vp, ci, cl, ci, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf, vp,
                            vp],
-    "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, ci, ci, ci, ci, vp, vp],
-    "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, ci, vp, vp],
+    "artb_latent_attend": [ci, vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, ci, ci, ci, ci, vp, vp],
+    "artb_latent_decode": [vp, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, cf, vp, vp, vp, ci, ci, ci, ci, ci, vp, vp],
     "artb_latent_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, vp, ci, vp, vp],
-    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci,
-                               ci, ci, vp, vp],
-    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci, ci,
-                            ci, ci, vp],
+    "artb_latent_prefill_tc": [vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, vp, ci, vp, ci, ci,
+                               vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_latent_prefill": [vp, ci, vp, ci, vp, ci, ci, vp, vp, ci, vp, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, vp, ci, vp, ci, ci, vp, ci,
+                            ci, ci, ci, ci, ci, ci, ci, vp],
     "artb_gqa_finish": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
-    "artb_gqa_finish_norm": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp, cf, vp, cf, ci, ci, vp, vp, vp, vp],
+    "artb_gqa_finish_norm": [ci, vp, ci, ci, vp, vp, vp, ci, cl, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp, ci, vp, cf, vp, cf, ci, ci, vp, vp, vp, ci, ci, vp,
+                             vp],
     "artb_gqa_gather": [vp, ci, vp, ci, ci, cl, vp, vp, vp, vp, ci, ci, vp, vp, ci, ci, vp, vp],
-    "artb_gqa_decode": [vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, vp, vp],
-    "artb_gqa_attend": [ci, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_decode": [vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, vp, vp],
+    "artb_gqa_attend": [ci, vp, ci, vp, ci, vp, ci, ci, cl, vp, vp, vp, ci, ci, cf, cf, cf, vp, ci, ci, vp, ci, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp, vp],
     "artb_short_conv": [ci, vp, ci, ci, vp, vp, vp, ci, vp, cl, vp, vp, vp, vp, ci, ci, vp, ci, ci, ci, ci, ci, ci, vp, vp],
     "artb_rglru": [ci, ci, vp, ci, ci, vp, ci, vp, vp, vp, vp, ci, ci, vp, vp, cl, vp, vp, vp, ci, vp, ci, cf, ci, ci, ci, ci, vp, vp],
     "artb_gemm_batched_bf16_tn": [vp, ci, ci, vp, ci, vp, ci, cl, ci, ci, ci, ci, ci, vp, vp],
@@ -94,7 +96,7 @@ def _st(t: torch.Tensor):
 class Sublayer:
     """What a sublayer hands to the residual stream: ``y`` (may be missing) times ``gate`` [M], ``bias`` [dp] and the rows of a
     token's experts, ``rows`` [cap, dp] weighted by ``weight`` [M, k] at the places ``pos`` [M, k]; a place of -1 is the token's
-    row of ``identity``."""
+    row of ``identity``.  The sum is multiplied by the sigmoid of ``col_gate`` + ``col_bias`` [dp]."""
     y: Out | None = None
     bias: torch.Tensor | None = None
     rows: torch.Tensor | None = None
@@ -102,17 +104,35 @@ class Sublayer:
     weight: torch.Tensor | None = None
     gate: torch.Tensor | None = None
     identity: Out | None = None
+    col_gate: Out | None = None
+    col_bias: torch.Tensor | None = None
+
+
+@dataclass
+class Streams:
+    """A boundary between hyper-connected sublayers: ``coef`` fp32 [(n_in + 2) * n_out] holds mix [n_in][n_out] (from, to), what each
+    copy gets of the sublayer's result, and what the next sublayer takes of each copy.  ``n_in`` = 0: the embedding, all copies
+    being equal to it."""
+    n_in: int
+    n_out: int
+    coef: torch.Tensor
 
 
 def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps: float, *, y: Out | None = None, x_in=None,
                   mult: float = 1.0, tokens=None, table=None, sub: Sublayer | None = None, freq=None, pos=None, hist=None,
-                  hist_n: int = 0, avg=None, w_next=None, h=None) -> None:
+                  hist_n: int = 0, avg=None, w_next=None, h=None, streams: Streams | None = None) -> None:
     """One sublayer boundary of the fp32 residual stream ``[M, dp]``; ``y`` (or ``sub``) is the sublayer's output, or
     ``tokens`` / ``table`` the embedding, to which ``freq`` (fp64 ``[dp / 2]``) and ``pos`` add a sinusoidal position vector.
     ``w_post``: norm weight of the output; None: it is taken as it is, times ``mult``.  ``hist`` fp32 ``[layers + 1, M, dp]``: the result is stored at ``hist_n`` and, with ``avg``,
     replaced by the weighted average of entries ``0 .. hist_n``.  ``w_next`` / ``h``: the next sublayer's input norm; without
-    ``w_next``, ``h`` is the stream itself in the operand dtype."""
+    ``w_next``, ``h`` is the stream itself in the operand dtype.  ``streams``: ``x_in`` and ``x_out`` hold several copies of the
+    stream side by side, which the step mixes; ``h`` then comes from their weighted sum."""
     M, dp = x_out.shape
+    if streams is not None:
+        dp //= streams.n_out
+        if streams.coef.numel() != (streams.n_in + 2) * streams.n_out or (x_in is not None and x_in.shape[1] != streams.n_in * dp):
+            raise ValueError("streams: the tensors do not hold as many copies as the boundary has")
+    cg = sub.col_gate if sub is not None else None
     s = sub if sub is not None else Sublayer(y)
     y, ex = s.y, s.rows
     idn = s.identity
@@ -128,7 +148,9 @@ def residual_step(x_out: torch.Tensor, w_post: torch.Tensor | None, d: int, eps:
         ex.shape[0] if ex is not None else 0, _lib.ptr(idn.t if idn is not None else None), idn.t.stride(0) if idn is not None else 0,
         idn.kind if idn is not None else 0, _lib.ptr(freq), _lib.ptr(pos), _lib.ptr(hist),
         hist.stride(0) if hist is not None else 0, hist_n, _lib.ptr(avg), _lib.ptr(w_next), _lib.ptr(h),
-        h.stride(0) if h is not None else 0, M, d, dp, eps, _st(x_out), _lib.stream_ptr()), "residual_step")
+        h.stride(0) if h is not None else 0, M, d, dp, eps, _st(x_out), _lib.ptr(cg.t if cg is not None else None), cg.t.stride(0) if cg is not None else 0,
+        cg.kind if cg is not None else 0, _lib.ptr(s.col_bias), _lib.ptr(streams.coef if streams else None), streams.n_in if streams else 0,
+        streams.n_out if streams else 0, x_in.stride(0) if streams and x_in is not None else 0, _lib.stream_ptr()), "residual_step")
 
 
 def norm_shift_mix(x, w, mu, out, state, row_seq, cu_q, ctx, state_slot, d: int, eps: float) -> None:
@@ -233,25 +255,41 @@ def lightning_prefill(q, k, v, decay, state, cu_q, ctx, state_slot, n_seqs: int,
     return o
 
 
-def latent_finish(p: Out, w, inv_freq, pos, slot, cache, n_abs: int, qn, qr, qe, H: int, dim: int, rot: int, rank: int,
-                  eps: float) -> None:
+@dataclass
+class Rotation:
+    """The rotation of the first ``dims`` columns of a head (or of its rotated part): ``freq`` fp64 [dims / 2] per pair (on the device),
+    ``scale`` the factor of sine and cosine; a column's partner is its neighbour (``next``) or ``dims / 2`` columns further."""
+    dims: int
+    freq: torch.Tensor
+    scale: float = 1.0
+    next: bool = False
+
+
+def _rotation(rot: Rotation | None) -> None:
+    if rot is not None and (rot.freq.dtype != torch.float64 or rot.freq.numel() != rot.dims // 2):
+        raise ValueError("rotation frequencies are fp64, one per pair")
+
+
+def latent_finish(p: Out, w, rotation: Rotation, pos, slot, cache, n_abs: int, qn, qr, qe, H: int, dim: int, rank: int, eps: float) -> None:
     """Norm, rotation and cache write behind the q | latent projection.  Rows below ``n_abs`` leave their queries in
     ``qn`` [H, pitch, dim_p] / ``qr`` [H, pitch, rot_p], the others in ``qe`` [M - n_abs, H * (dim_p + rot_p)]."""
-    M = pos.numel()
+    M, rot = pos.numel(), rotation.dims
+    _rotation(rotation)
     _lib.check_rc(_f("artb_latent_finish")(
-        _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(w), _lib.ptr(inv_freq), _lib.ptr(pos), _lib.ptr(slot),
+        _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(w), _lib.ptr(rotation.freq), rotation.scale, int(rotation.next), _lib.ptr(pos), _lib.ptr(slot),
         _lib.ptr(cache), cache.shape[-1], cache.shape[0] * cache.shape[1], n_abs, _lib.ptr(qn), _lib.ptr(qr),
         qn.shape[1] if qn is not None else 0, _lib.ptr(qe), qe.stride(0) if qe is not None else 0, M, H, dim, pad(dim, 16), rot,
         pad(rot, 16), rank, pad(rank, 16), eps, _st(cache), _lib.stream_ptr()), "latent_finish")
 
 
-def latent_attend(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int) -> torch.Tensor:
-    """Windowed attention in latent space over the paged cache, scalar fp32 form; everything head-major [H, pitch, .]."""
+def latent_attend(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int, sink=None) -> torch.Tensor:
+    """Windowed attention in latent space over the paged cache, scalar fp32 form; everything head-major [H, pitch, .].  ``sink`` fp32
+    [H]: one more term of the softmax's denominator."""
     H, pitch, rank_p = ql.shape
     _lib.check_rc(_f("artb_latent_attend")(
         _is32(cache), _lib.ptr(ql), _lib.ptr(qr), pitch, _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table),
         block_table.stride(0), cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale,
-        _lib.ptr(o), M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_attend")
+        _lib.ptr(sink), _lib.ptr(o), M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_attend")
     return o
 
 
@@ -266,14 +304,14 @@ def latent_decode_splits(M: int, H: int, keys: int, sms: int = 148) -> int:
 
 
 def latent_decode(ql, qr, cache, block_table, row_seq, pos, ctx, window: int, scale: float, o, M: int, splits: int = 1,
-                  ws=None) -> torch.Tensor:
+                  ws=None, sink=None) -> torch.Tensor:
     """Tensor-core form of :func:`latent_attend` for rows ``0 .. M - 1`` (bf16)."""
     H, pitch, rank_p = ql.shape
     if splits > 1 and ws is None:
         ws = torch.empty(M * H * splits * (rank_p + 2), dtype=torch.float32, device=o.device)
     _lib.check_rc(_f("artb_latent_decode")(
         _lib.ptr(ql), _lib.ptr(qr), pitch, _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0),
-        cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale, _lib.ptr(o), _lib.ptr(ws), splits,
+        cache.shape[1], cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, scale, _lib.ptr(sink), _lib.ptr(o), _lib.ptr(ws), splits,
         M, H, rank_p, qr.shape[2], _st(cache), _lib.stream_ptr()), "latent_decode")
     return o
 
@@ -337,15 +375,57 @@ def _gate(gate):
     return _lib.ptr(gate), gate.stride(0) if gate is not None else 0
 
 
+BIAS_PAD = 256          # entries in front of and behind a distance table (key_weights.cuh)
+
+
+@dataclass
+class KeyWeights:
+    """What an attention kernel makes of scores besides a softmax, and of its result.  ``bias`` fp32 [H, n + 2 BIAS_PAD] (see
+    :func:`distance_table`): a key weighs sigmoid(score + bias of its distance), without normalisation.  ``sink`` fp32 [H]: one
+    more term of the softmax's denominator.  ``cols`` [rows, .], operand dtype: logits of a gate of the result's columns, a head's
+    ``pitch`` columns after the one before it."""
+    bias: torch.Tensor | None = None
+    sink: torch.Tensor | None = None
+    cols: torch.Tensor | None = None
+    pitch: int = 0
+
+    def rows_from(self, n: int) -> "KeyWeights":
+        """The same for the rows from ``n`` on."""
+        return KeyWeights(self.bias, self.sink, self.cols[n:] if self.cols is not None else None, self.pitch)
+
+
+def distance_table(rel: torch.Tensor, buckets: list[int], head_bias: torch.Tensor) -> torch.Tensor:
+    """The kernels' table of ``rel`` fp32 [rows, H] by distance plus ``head_bias`` [H], in base-2 units; ``buckets[t]`` is the row of
+    distance t, the last one that of all farther ones."""
+    idx = torch.tensor([buckets[0]] * BIAS_PAD + list(buckets) + [buckets[-1]] * BIAS_PAD, device=rel.device)
+    return ((rel.double()[idx] + head_bias.double()) * math.log2(math.e)).t().float().contiguous()
+
+
+def _bias(kw: "KeyWeights | None", H: int):
+    b = kw.bias if kw is not None else None
+    if b is not None and (b.dtype != torch.float32 or b.shape[0] != H or not b.is_contiguous() or b.shape[1] <= 2 * BIAS_PAD):
+        raise ValueError("a distance table is fp32 [heads, distances + padding]")
+    return (1, _lib.ptr(b), b.shape[1] - 2 * BIAS_PAD) if b is not None else (0, _lib.ptr(None), 0)
+
+
+def _cols(kw: "KeyWeights | None", like: torch.Tensor):
+    c = kw.cols if kw is not None else None
+    if c is not None and (c.dtype != like.dtype or c.stride(1) != 1):
+        raise ValueError("a column gate has the operand dtype and unit inner stride")
+    return _lib.ptr(c), c.stride(0) if c is not None else 0, kw.pitch if kw is not None else 0
+
+
 def latent_prefill(q, kv, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                   vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None) -> torch.Tensor:
+                   vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None,
+                   weights: KeyWeights | None = None) -> torch.Tensor:
     """Masked attention of the portions: ``q`` [rows, H * (dk + rot_p)], ``kv`` [n_keys, H / G * (dk + dv)] the expanded
     keys and values (``G`` heads share them), ``c`` the gathered cache rows; ``o`` [rows, H * pad(vdim)].  ``softcap`` > 0 squashes
     the scores; ``gate`` fp32 [rows, H] multiplies the heads."""
     _lib.check_rc(_f("artb_latent_prefill")(
         _lib.ptr(q), q.stride(0), _lib.ptr(kv), kv.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(plan.tile_seq),
         _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0), _lib.ptr(plan.key_off),
-        _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p,
+        _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(weights.sink if weights else None), *_bias(weights, H),
+        *_cols(weights, o), _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p,
         _lib.stream_ptr()), "latent_prefill")
     return o
 
@@ -363,13 +443,14 @@ def gqa_value_columns(dim: int, vdim: int, scale: float) -> int:
 
 
 def latent_prefill_tc(q, k, vt, c, plan: PrefillPlan, window: int, scale: float, o, H: int, dk: int, dv: int, rank_p: int, rot_p: int,
-                      vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None) -> torch.Tensor:
+                      vdim: int, chunk: int = 0, G: int = 1, out_scale: float = 1.0, softcap: float = 0.0, gate=None,
+                      weights: KeyWeights | None = None) -> torch.Tensor:
     """:func:`latent_prefill` on tcgen05: ``k`` [n_keys, H / G * dk], values transposed ``vt`` [H / G * dv, n_keys]."""
     _lib.check_rc(_f("artb_latent_prefill_tc")(
         _lib.ptr(q), q.stride(0), q.shape[0], _lib.ptr(k), k.stride(0), _lib.ptr(c), c.stride(0), rank_p, _lib.ptr(vt), vt.stride(0),
         plan.n_keys, _lib.ptr(plan.tile_seq), _lib.ptr(plan.tile_row), plan.n_tiles, _lib.ptr(plan.row_end), _lib.ptr(plan.row_pos0),
-        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(o), o.stride(0),
-        pad(vdim), H, G, dk, dv, rot_p, _st(o),
+        _lib.ptr(plan.key_off), _lib.ptr(plan.key_pos0), window, chunk, scale, softcap, out_scale, *_gate(gate), _lib.ptr(weights.sink if weights else None),
+        *_bias(weights, H), *_cols(weights, o), _lib.ptr(o), o.stride(0), pad(vdim), vdim, H, G, dk, dv, rot_p, _st(o),
         _lib.stream_ptr()), "latent_prefill_tc")
     return o
 
@@ -384,30 +465,26 @@ def gqa_finish(p: Out, bias, slot, cache, q, H: int, Hkv: int, dim: int, vdim: i
         "gqa_finish")
 
 
-@dataclass
-class Rotation:
-    """The rotation of the first ``dims`` columns of a head: ``freq`` fp64 [dims / 2] per pair (on the device), ``scale`` the factor of
-    sine and cosine; a column's partner is its neighbour (``next``) or ``dims / 2`` columns further."""
-    dims: int
-    freq: torch.Tensor
-    scale: float = 1.0
-    next: bool = False
-
-
 def gqa_finish_norm(p: Out, bias, slot, cache, q, H: int, Hkv: int, dim: int, vdim: int, dvp: int, wq, wk, eps: float, rot: Rotation | None, pos,
-                    gate=None) -> None:
+                    gate=None, per_head: bool = False, q_scale=None, cols=None, pitch: int = 0) -> None:
     """:func:`gqa_finish` with norms over all heads of q (``wq``) and of k (``wk``), a rotation behind them, and ``gate`` fp32 [M, H]
-    receiving the sigmoids of the columns behind v.  ``Hkv`` = 0: the projection has no k and v and the cache stays as it is."""
+    receiving the sigmoids of the columns behind v.  ``Hkv`` = 0: the projection has no k and v and the cache stays as it is.
+
+    ``per_head``: a norm over each head with the weights of one; ``q_scale`` fp32 [H] then multiplies the query heads.  ``cols``
+    [M, H * pitch], operand dtype: receives the ``H * vdim`` columns behind v."""
     M = slot.numel()
-    if rot is not None and (rot.freq.dtype != torch.float64 or rot.freq.numel() != rot.dims // 2):
-        raise ValueError("rotation frequencies are fp64, one per pair")
+    _rotation(rot)
+    if per_head and any(w is not None and w.numel() != dim for w in (wq, wk)):
+        raise ValueError("per_head: norm weights of one head")
+    if cols is not None and cols.dtype != q.dtype:
+        raise ValueError("cols: a tensor of the operand dtype")
     if gate is not None and gate.stride(0) != H:
         raise ValueError("gate: a dense [M, H] tensor")
     _lib.check_rc(_f("artb_gqa_finish_norm")(
         _is32(cache), _lib.ptr(p.t), p.t.stride(0), p.kind, _lib.ptr(bias), _lib.ptr(slot), _lib.ptr(cache), cache.shape[-1],
-        cache.shape[0] * cache.shape[1], _lib.ptr(q), q.stride(0), M, H, Hkv, dim, pad(dim, 16), vdim, dvp, _lib.ptr(wq), _lib.ptr(wk), eps,
-        _lib.ptr(rot.freq if rot else None), rot.scale if rot else 1.0, rot.dims if rot else 0, 1 if rot and rot.next else 0, _lib.ptr(pos),
-        _lib.ptr(gate), _st(cache), _lib.stream_ptr()), "gqa_finish_norm")
+        cache.shape[0] * cache.shape[1], _lib.ptr(q), q.stride(0), M, H, Hkv, dim, pad(dim, 16), vdim, dvp, _lib.ptr(wq), _lib.ptr(wk), int(per_head),
+        _lib.ptr(q_scale), eps, _lib.ptr(rot.freq if rot else None), rot.scale if rot else 1.0, rot.dims if rot else 0, 1 if rot and rot.next else 0, _lib.ptr(pos),
+        _lib.ptr(gate), _lib.ptr(cols), cols.stride(0) if cols is not None else 0, pitch, _st(cache), _lib.stream_ptr()), "gqa_finish_norm")
 
 
 def gqa_gather(cache, block_table, plan: PrefillPlan, Hkv: int, dk: int, dv: int) -> tuple[torch.Tensor, torch.Tensor]:
@@ -430,29 +507,32 @@ def gqa_decode_splits(M: int, ctas_per_row: int, keys: int, sms: int = 148) -> i
     return max(1, min(2 * sms // max(1, M * ctas_per_row), (keys + 4 * GQA_TILE - 1) // (4 * GQA_TILE), 32))
 
 
-def _gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate):
+def _gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate, weights, H):
+    if weights is not None and weights.sink is not None:
+        raise ValueError("sinks are not supported by this form of attention")
     return (_lib.ptr(q), q.stride(0), _lib.ptr(cache), cache.shape[-1], _lib.ptr(block_table), block_table.stride(0), cache.shape[1],
             cache.shape[0], _lib.ptr(row_seq), _lib.ptr(pos), _lib.ptr(ctx), window, chunk, scale, softcap, out_scale, *_gate(gate),
-            _lib.ptr(o), o.stride(0))
+            *_bias(weights, H), *_cols(weights, o), _lib.ptr(o), o.stride(0))
 
 
 def gqa_decode(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
-               Hkv: int, dim: int, vdim: int, dvp: int, splits: int = 1, softcap: float = 0.0, gate=None) -> torch.Tensor:
+               Hkv: int, dim: int, vdim: int, dvp: int, splits: int = 1, softcap: float = 0.0, gate=None,
+               weights: KeyWeights | None = None) -> torch.Tensor:
     """Rows ``0 .. M - 1`` of ``q`` against their sequences' cached keys; ``o`` [., H * pad(vdim)] gets ``out_scale`` times the
     result, and times ``gate`` fp32 [M, H]; ``softcap`` > 0 squashes the scores."""
     vpad = pad(vdim)
     ws = torch.empty(M * H * splits * (vpad + 2), dtype=torch.float32, device=o.device) if splits > 1 else None
     _lib.check_rc(_f("artb_gqa_decode")(
-        *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate), vpad, _lib.ptr(ws), splits, M, H, Hkv,
+        *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate, weights, H), vpad, _lib.ptr(ws), splits, M, H, Hkv,
         pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_decode")
     return o
 
 
 def gqa_attend(q, cache, block_table, row_seq, pos, ctx, window: int, chunk: int, scale: float, out_scale: float, o, M: int, H: int,
-               Hkv: int, dim: int, vdim: int, dvp: int, softcap: float = 0.0, gate=None) -> torch.Tensor:
+               Hkv: int, dim: int, vdim: int, dvp: int, softcap: float = 0.0, gate=None, weights: KeyWeights | None = None) -> torch.Tensor:
     """Scalar fp32 form of :func:`gqa_decode`, any head sizes."""
     _lib.check_rc(_f("artb_gqa_attend")(
-        _is32(cache), *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate), pad(vdim), M, H, Hkv,
+        _is32(cache), *_gqa(q, cache, block_table, row_seq, pos, ctx, window, chunk, scale, out_scale, o, softcap, gate, weights, H), pad(vdim), M, H, Hkv,
         pad(dim, 16), vdim, dvp, _st(cache), _lib.stream_ptr()), "gqa_attend")
     return o
 

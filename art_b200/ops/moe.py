@@ -26,7 +26,7 @@ def _k():
     lib = _lib.kernels()
     if not _configured:
         vp, ci, cl = ctypes.c_void_p, ctypes.c_int, ctypes.c_long
-        lib.artb_moe_router.argtypes = [vp, ci, ci, vp, vp, ci, ci, ci, ci, ci, vp, vp, vp, vp, vp]
+        lib.artb_moe_router.argtypes = [vp, ci, ci, vp, vp, ci, ci, ci, ci, ci, ci, ci, ctypes.c_float, vp, vp, vp, vp, vp]
         lib.artb_moe_plan.argtypes = [vp, ci, vp, vp, cl, ci, vp, vp, ci, vp, vp, vp, vp, vp]
         lib.artb_moe_gather.argtypes = [vp, ci, vp, vp, ci, vp, vp, ci, ci, ci, vp]
         lib.artb_moe_gather_f32.argtypes = [vp, ci, vp, vp, vp, ci, ci, ci, vp]
@@ -74,13 +74,17 @@ def cap_tiles_for(M: int, k: int, E: int) -> int:
 
 
 def route(logits: torch.Tensor, k: int, norm_topk: bool, bias: torch.Tensor | None = None, take: bool = False,
-          correction: torch.Tensor | None = None, identity: int = 0, gate: bool = False) -> RoutePlan:
+          correction: torch.Tensor | None = None, identity: int = 0, gate: bool = False, groups: int = 1, keep: int = 1,
+          scale: float = 1.0) -> RoutePlan:
     """Softmax over experts, top-k, (optional) renormalisation, and the expert-sorted row plan.  ``bias`` fp32 [E] is added
     to the logits first; with ``take`` the logits lie in a workspace that is to be left zero.
 
     ``correction`` fp32 [outputs]: the choice goes by softmax + correction, the weights by the softmax (its share of the
     chosen ones' sum + 1e-20 with ``norm_topk``).  The last ``identity`` outputs have no rows (``pos`` is -1).  ``gate``: one
-    more column, whose sigmoid is ``plan.gate``."""
+    more column, whose sigmoid is ``plan.gate``.
+
+    The outputs form ``groups`` equal groups of neighbours; only those of the ``keep`` groups with the largest single outputs can
+    be chosen.  ``scale`` multiplies the weights."""
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     M, outputs = logits.shape[0], logits.shape[1] - int(gate)
     E = outputs - identity
@@ -95,7 +99,7 @@ def route(logits: torch.Tensor, k: int, norm_topk: bool, bias: torch.Tensor | No
     cursor = torch.empty(E, **i32)
     st = _lib.stream_ptr()
     _lib.check_rc(_k().artb_moe_router(_lib.ptr(logits), logits.stride(0), 2 if take else 1, _lib.ptr(bias), _lib.ptr(correction), M, outputs, E, k,
-                                       int(norm_topk), _lib.ptr(plan.topi), _lib.ptr(plan.topw), _lib.ptr(plan.counts), _lib.ptr(plan.gate), st),
+                                       int(norm_topk), groups, keep, scale, _lib.ptr(plan.topi), _lib.ptr(plan.topw), _lib.ptr(plan.counts), _lib.ptr(plan.gate), st),
                   "moe_router")
     _lib.check_rc(_k().artb_moe_plan(_lib.ptr(plan.counts), E, _lib.ptr(plan.topi), _lib.ptr(plan.topw), M, k,
                                      _lib.ptr(plan.seg_off), _lib.ptr(plan.tile_expert), cap, _lib.ptr(cursor),
