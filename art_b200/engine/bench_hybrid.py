@@ -5,8 +5,8 @@ Two parts, random weights throughout:
 * ``engine_rows``: prefill and decode tokens/s of whole models through :class:`~art_b200.engine.engine.Engine`, a hybrid
   preset and a twin of the same width, depth and feed-forward parameters per layer, no adapters: a dense Llama-style model,
   or a Qwen3-style mixture of experts where the preset has experts.
-* ``kernel_rows``, ``naselorn_kernel_rows``, ``gaborax_kernel_rows``: every kernel of the hybrid path at the layer sizes of a model, timed alone with CUDA events (L2 flushed
-  between calls), with its algorithmic bytes and FLOPs and the fraction of its roofline (the slower of bytes at the
+* ``kernel_rows``, ``naselorn_kernel_rows``, ``gaborax_kernel_rows``, ``gaparax_kernel_rows``: every kernel of the hybrid path at the
+  layer sizes of a model, timed alone with CUDA events (L2 flushed between calls), with its algorithmic bytes and FLOPs and the fraction of its roofline (the slower of bytes at the
   measured copy bandwidth and FLOPs at the measured tensor or nominal fp32 rate), and the like kernels of the dense model
   or of the other design.
 """
@@ -463,6 +463,146 @@ def gaborax_kernel_rows(width: int = 4096, prefill: int = 8192, decode: int = 25
     return bench.rows
 
 
+def gaparax_kernel_rows(width: int = 4096, prefill: int = 8192, decode: int = 256, ctx: int = 2048, chunk: int = 1024, streams: tuple[int, ...] = (2, 4),
+                        experts: int = 64, top: int = 8, expert_ff: int = 1024, dense_ff: int = 16384, softcap: float = 30.0, reach: int = 256) -> list[dict]:
+    """The kernels of Gaparax layers, each beside the like kernel of another design ("like: ...")."""
+    from ..models.hybrid import distance_buckets
+    from ..ops import attention as attn_ops
+    from ..ops import hybrid as hy
+    from ..ops import moe, paged
+    from ..ops.gemm import gemm_tn
+
+    dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
+    bench = _Rows()
+    add = bench.add
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, generator=g) * sc).to(dt)      # noqa: E731
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)      # noqa: E731
+    d, H, hd, bs = width, width // 128, 128, 16
+    Hkv, G = H // 4, 4
+    table = hy.distance_table(rnd(32, H, dt=f32), distance_buckets(32, reach, chunk), rnd(H, dt=f32) - 4.0)
+    for phase, M in (("decode", decode), ("prefill", prefill)):
+        one = phase == "decode"
+        n_seqs = M if one else M // 2048
+        row_seq = i32(list(range(M)) if one else [i // 2048 for i in range(M)])
+        c_len = i32([ctx] * n_seqs)
+        pos = i32([ctx - 1] * M if one else [i % 2048 for i in range(M)])
+        # boundaries of streams: the copies read and written, the result, its gate, the next operand
+        w, h, y, gl = rnd(d, dt=f32), rnd(M, d), rnd(M, d), rnd(M, d)
+        for n in streams:
+            x, coef = rnd(M, n * d, dt=f32), rnd((n + 2) * n, dt=f32, sc=0.3)
+            sub = hy.Sublayer(hy.as_out(y), col_gate=hy.as_out(gl), col_bias=w)
+            add(f"stream_step, {n} streams, gate", phase, lambda: hy.residual_step(x, None, d, 1e-5, sub=sub, x_in=x, w_next=w, h=h, streams=hy.Streams(n, n, coef)),
+                M * d * (6 + 8 * n))
+        x = rnd(M, d, dt=f32)
+        add("residual_step with gate", phase, lambda: hy.residual_step(x, None, d, 1e-5, sub=sub, x_in=x, w_next=w, h=h), M * d * 14)
+        add("like: residual_step (pre-norm frame)", phase, lambda: hy.residual_step(x, None, d, 1e-5, y=hy.as_out(y), x_in=x, w_next=w, h=h), M * d * 12)
+        # sigmoid attention in chunks
+        ld = Hkv * 2 * hd
+        nb = n_seqs * (ctx // bs)
+        cache = rnd(nb, bs, ld)
+        bt = torch.randperm(nb, device=dev, generator=g).to(torch.int32).view(n_seqs, ctx // bs)
+        n = (H + 2 * Hkv) * hd
+        P32, wn, temp = rnd(M, n + H * hd, dt=f32), rnd(n, dt=f32), torch.rand(H, device=dev) + 0.5
+        P = P32.to(bf)
+        q, slot = torch.empty(M, H * hd, dtype=bf, device=dev), i32([i % (nb * bs) for i in range(M)])
+        add("gqa_finish_norm, norm of each head", phase, lambda: hy.gqa_finish_norm(hy.as_out(P), None, slot, cache, q, H, Hkv, hd, hd, hd, wn[:hd], wn[:hd], 1e-5, None,
+                                                                                   pos, per_head=True, q_scale=temp), M * n * 4)
+        if one:
+            cols = torch.empty(M, H * hd, dtype=bf, device=dev)
+            add("gqa_finish_norm, norm of each head, workspace and gates", phase, lambda: hy.gqa_finish_norm(
+                hy.Out(P32, hy.KIND_TAKE), None, slot, cache, q, H, Hkv, hd, hd, hd, wn[:hd], wn[:hd], 1e-5, None, pos, None, True, temp, cols, hd), M * (n + H * hd) * 10)
+        freq = torch.tensor([5e5 ** (-2 * i / hd) for i in range(hd // 2)], dtype=torch.float64, device=dev)
+        add("like: gqa_finish_norm, norm of all heads, rotation", phase, lambda: hy.gqa_finish_norm(hy.as_out(P), None, slot, cache, q, H, Hkv, hd, hd, hd, wn, wn, 1e-5,
+                                                                                                    hy.Rotation(hd, freq), pos), M * n * 4)
+        ao, kw = torch.empty(M, H * hd, dtype=bf, device=dev), hy.KeyWeights(table, cols=P[:, n:], pitch=hd)
+        if one:
+            keys = (ctx - 1) % chunk + 1
+            sp = hy.gqa_decode_splits(M, Hkv, chunk)
+            args = (q, cache, bt, row_seq, pos, c_len, 0, chunk, hd ** -0.5, 1.0, ao, M, H, Hkv, hd, hd, hd, sp)
+            b_, f_ = M * keys * ld * 2 + M * H * hd * 4, 4.0 * M * H * keys * hd
+            add(f"gqa_decode chunk {chunk}, sigmoid weights, gates", phase, lambda: hy.gqa_decode(*args, softcap=softcap, weights=kw), b_ + M * H * hd * 2, f_)
+            add("like: gqa_decode, softmax, capped", phase, lambda: hy.gqa_decode(*args, softcap=softcap), b_, f_)
+            kc, vc = rnd(n_seqs * chunk // bs, bs, Hkv, hd), rnd(n_seqs * chunk // bs, bs, Hkv, hd)
+            btd = torch.arange(n_seqs * chunk // bs, dtype=torch.int32, device=dev).view(n_seqs, -1)
+            cd = i32([chunk] * M)
+            add(f"like: paged_decode ctx {chunk}", phase, lambda: paged.paged_decode(q, kc, vc, btd, cd, H, Hkv, hd, ao), b_, f_)
+            del kc, vc
+        else:
+            plan = hy.plan_prefill([(i, 0, 2048) for i in range(n_seqs)], 0, dev, chunk)
+            k, vt = hy.gqa_gather(cache, bt, plan, Hkv, hd, hd)
+            pairs = n_seqs * sum(i % chunk + 1 for i in range(2048))
+            b_, f_ = (q.numel() + k.numel() + vt.numel() + ao.numel()) * 2, 4.0 * H * pairs * hd
+            args = (q, k, vt, k, plan, 0, hd ** -0.5, ao, H, hd, hd, 0, 0, hd)
+            add(f"latent_prefill_tc chunk {chunk}, sigmoid weights, gates", phase, lambda: hy.latent_prefill_tc(*args, chunk=chunk, G=G, softcap=softcap, weights=kw),
+                b_ + M * H * hd * 2, f_)
+            add("the same, not capped", phase, lambda: hy.latent_prefill_tc(*args, chunk=chunk, G=G, weights=kw), b_ + M * H * hd * 2, f_)
+            add("like: latent_prefill_tc, softmax, capped", phase, lambda: hy.latent_prefill_tc(*args, chunk=chunk, G=G, softcap=softcap), b_, f_)
+            add("like: latent_prefill_tc, softmax", phase, lambda: hy.latent_prefill_tc(*args, chunk=chunk, G=G), b_, f_)
+            c = hy.latent_gather(cache, bt, plan)
+            args = (q, c, c, plan, 0, hd ** -0.5, ao, H, hd, hd, 0, 0, hd)
+            add(f"latent_prefill (any sizes) chunk {chunk}, sigmoid weights, gates", phase, lambda: hy.latent_prefill(*args, chunk=chunk, G=G, softcap=softcap, weights=kw),
+                b_ + M * H * hd * 2, f_)
+            add("like: latent_prefill (any sizes), softmax, capped", phase, lambda: hy.latent_prefill(*args, chunk=chunk, G=G, softcap=softcap), b_, f_)
+            ids = torch.arange(M // chunk, dtype=torch.int32, device=dev).repeat_interleave(chunk)
+            ap = attn_ops.make_plan(ids, ids, M, "native")
+            qkv = P[:, :n].contiguous()
+            add(f"like: tree attention fwd, causal, {chunk} tokens", phase, lambda: attn_ops.forward(qkv, H, Hkv, hd, ap, need_grad=False), b_, f_)
+            del qkv, k, vt, c
+        del P, P32, cache
+        # latent attention without a window, with a sink: d / 128 heads of 128 + 64, latent 512, values 128
+        dk, rot, rank, dv = 128, 64, 512, 128
+        cache = rnd(nb, bs, rank + rot)
+        pq, cn, none = rnd(M, H * (dk + rot) + rank + rot), rnd(rank, dt=f32), i32([-1] * M)
+        qn, qr = torch.zeros(H, hy.pad(M, 128), dk, dtype=bf, device=dev), torch.zeros(H, hy.pad(M, 128), rot, dtype=bf, device=dev)
+        qe = torch.zeros(M, H * (dk + rot), dtype=bf, device=dev)
+        turn = torch.tensor([5e5 ** (-2 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=dev)
+        for nxt in (False, True):
+            add("like: latent_finish, neighbours" if nxt else "latent_finish, halves", phase, lambda: hy.latent_finish(
+                hy.as_out(pq), cn, hy.Rotation(rot, turn, 1.1, nxt), pos, none, cache, M if one else 0, qn, qr, qe, H, dk, rank, 1e-5), M * (2 * H * (dk + rot) + rank + rot) * 2)
+        sink = rnd(H, dt=f32)
+        if one:
+            ql, ol = rnd(H, hy.pad(M, 128), rank), torch.zeros(H, hy.pad(M, 128), rank, dtype=bf, device=dev)
+            sp = hy.latent_decode_splits(M, H, ctx)
+            for s_ in (sink, None):
+                add(f"latent_decode ctx {ctx}, sink" if s_ is not None else "like: latent_decode without sink", phase, lambda: hy.latent_decode(
+                    ql, qr, cache, bt, row_seq, pos, c_len, 0, 0.07, ol, M, sp, sink=s_), M * ctx * (rank + rot) * 2 + M * H * (2 * rank + rot) * 2,
+                    2.0 * M * H * ctx * (2 * rank + rot))
+        else:
+            plan = hy.plan_prefill([(i, 0, 2048) for i in range(n_seqs)], 0, dev)
+            c = hy.latent_gather(cache, bt, plan)
+            k, vt = rnd(plan.n_keys, H * dk), rnd(H * dv, plan.n_keys)
+            pairs = n_seqs * 2048 * 2049 // 2
+            for s_ in (sink, None):
+                add("latent_prefill_tc causal 2048, sink" if s_ is not None else "like: latent_prefill_tc without sink", phase, lambda: hy.latent_prefill_tc(
+                    qe, k, vt, c, plan, 0, 0.07, ao, H, dk, dv, rank, rot, dv, weights=hy.KeyWeights(sink=s_)),
+                    (qe.numel() + k.numel() + vt.numel() + ao.numel()) * 2, 2.0 * H * pairs * (dk + rot + dv))
+            del k, vt, c
+        del cache, pq, qn, qr, qe
+        # feed-forwards, the residual gate's rows in their input products
+        Wu, z = rnd(dense_ff + d, d, sc=d ** -0.5), torch.empty(M, dense_ff + d, dtype=bf, device=dev)
+        wb, wf = (Wu.numel() + M * d + z.numel()) * 2, 2.0 * M * d * (dense_ff + d)
+        add("gemm_tn up | gate, squared relu of the first columns", phase, lambda: gemm_tn(h, Wu, out=z, relu2=True, relu2_cols=dense_ff), wb, wf)
+        add("like: gemm_tn, same product", phase, lambda: gemm_tn(h, Wu, out=z), wb, wf)
+        del Wu, z
+        logits = rnd(M, experts + d, dt=f32)[:, :experts]
+        add("moe.route, best groups", phase, lambda: moe.route(logits, top, False, groups=8, keep=4, scale=2.5), M * (experts * 4 + top * 8))
+        add("like: moe.route by logits", phase, lambda: moe.route(logits, top, True), M * (experts * 4 + top * 8))
+        rp = moe.route(logits, top, False, groups=8, keep=4, scale=2.5)
+        yp = torch.empty(rp.cap_rows, d, dtype=bf, device=dev).normal_()
+        gf = rnd(M, d, dt=f32)
+        n = streams[0]
+        x2, coef = rnd(M, n * d, dt=f32), rnd((n + 2) * n, dt=f32, sc=0.3)
+        sub = hy.Sublayer(rows=yp, pos=rp.pos, weight=rp.topw, col_gate=hy.as_out(gf), col_bias=w)
+        add(f"stream_step with experts' rows, {n} streams, gate", phase, lambda: hy.residual_step(x2, None, d, 1e-5, sub=sub, x_in=x2, w_next=w, h=h,
+                                                                                                 streams=hy.Streams(n, n, coef)), M * d * (6 + 8 * n + 2 * top))
+        plain = hy.Sublayer(hy.as_out(y), rows=yp, pos=rp.pos, weight=rp.topw)
+        add("like: residual_step with experts' rows", phase, lambda: hy.residual_step(x, None, d, 1e-5, sub=plain, x_in=x, w_next=w, h=h), M * d * (12 + 2 * top))
+        del yp, logits
+        torch.cuda.empty_cache()
+    return bench.rows
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
     ap.add_argument("--models", default="nikelix-1b,nikelix-7b")
@@ -478,7 +618,8 @@ def report(models: list[str], batches: list[int], layers: int, part: str = "both
     from ..ops import _lib
 
     if part != "engine":
-        for design, fn in (("nikelix", kernel_rows), ("naselorn", naselorn_kernel_rows), ("gaborax", gaborax_kernel_rows)):
+        for design, fn in (("nikelix", kernel_rows), ("naselorn", naselorn_kernel_rows), ("gaborax", gaborax_kernel_rows),
+                           ("gaparax", gaparax_kernel_rows)):
             if any(m.startswith(design) for m in models):
                 yield from ({"part": "kernel", "design": design, **r} for r in fn())
                 torch.cuda.empty_cache()

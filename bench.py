@@ -69,7 +69,7 @@ def parse_args():
     ap.add_argument("--hybrid", action="store_true",
                     help="instead of the headline benchmark: prefill / decode throughput and per-kernel timings of the hybrid "
                          "decoders beside a model of equal size of the other families, one JSON line per measurement (one GPU)")
-    ap.add_argument("--hybrid-models", default="nikelix-1b,nikelix-7b,naselorn-2b-a1b,naselorn-14b-a4b,gaborax-2b-a1b,gaborax-14b-a4b")
+    ap.add_argument("--hybrid-models", default="nikelix-1b,nikelix-7b,naselorn-2b-a1b,naselorn-14b-a4b,gaborax-2b-a1b,gaborax-14b-a4b,gaparax-2b-a1b,gaparax-14b-a4b")
     ap.add_argument("--hybrid-batches", default="1,64,256")
     ap.add_argument("--hybrid-layers", type=int, default=8, help="layers of each preset to run (0: all)")
     return ap.parse_args()

@@ -63,8 +63,8 @@ def attention(h, w, p, eps):
     for n in range(H):
         g = n // (H // G)
         s = q[:, n] @ k[:, g].T * p["scale"] * w["temp"][n]
-        s = p["softcap"] * torch.tanh(s / p["softcap"]) + bias[:, :, n]
-        out[:, n] = (sigmoid(s + w["pb"][n]) * seen) @ v[:, g]
+        s = p["softcap"] * torch.tanh(s / p["softcap"]) if p["softcap"] else s
+        out[:, n] = (sigmoid(s + bias[:, :, n] + w["pb"][n]) * seen) @ v[:, g]
     return (out.reshape(T, -1) * sigmoid(h @ w["g"].T)) @ w["o"].T
 
 

@@ -111,3 +111,40 @@ def aligned_gaborax():
                     capped(heads=4, kv_heads=4, dim=64, vdim=64, rot=64, scale=0.125, softcap=15.0, mlp=relu2_moe(9, 2, 2, 80, 64)),
                     gated_heads(heads=6, kv_heads=2, dim=128, vdim=104, rot=96, scale=0.09, kv_from=0, mlp=relu2_moe(6, 1, 3, 64, 80)),
                     capped(heads=8, kv_heads=1, dim=80, vdim=96, rot=48, scale=0.11, softcap=30.0)], vocab=528, width=304, eps=1e-6)
+
+
+# -- Gaparax --------------------------------------------------------------------------------------------------------------
+def relu2_dense(ff=70):
+    return {"kind": "dense", "ff": ff}
+
+
+def group_moe(experts=6, groups=3, keep=2, top=3, ff=28, scale=1.7):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}, "scale": scale}}
+
+
+def sigmoid_heads(heads=4, kv_heads=2, dim=20, vdim=12, chunk=23, scale=0.3, softcap=6.0, bias_max=15, mlp=None):
+    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "softcap": softcap,
+                                                      "bias_max": bias_max, "mask": {"size": chunk}}}
+
+
+def sink_latent(heads=3, dim=20, rot=6, rank=36, vdim=28, scale=0.19, base=300.0, scaling=yarn(), mlp=None):
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "kv_rank": rank, "vdim": vdim, "scale": scale,
+                                                             "rot": {"base": base, "dims": rot, "scaling": scaling}}}
+
+
+def gaparax(layers, vocab=193, width=84, eps=4e-5, streams=3):
+    return {"architecture": "Gaparax", "vocab": vocab, "width": width, "norm": {"eps": eps}, "streams": streams, "layers": layers}
+
+
+def small_gaparax():
+    return gaparax([sigmoid_heads(mlp=group_moe()), sink_latent(mlp=relu2_dense()), sigmoid_heads(heads=3, kv_heads=3, dim=7, vdim=33, chunk=50, softcap=2.0,
+                    bias_max=120, mlp=relu2_dense(33)), sink_latent(heads=1, dim=16, rot=2, rank=16, vdim=8, scaling=None), sigmoid_heads(heads=5, kv_heads=1, dim=64,
+                    vdim=40, chunk=7, bias_max=4), sink_latent(heads=4, dim=64, rot=64, rank=40, vdim=24, scale=0.1, mlp=group_moe(8, 4, 1, 2, 16, 0.6))])
+
+
+def aligned_gaparax():
+    """Sizes near a real model's proportions, still small: several tiles of the tensor-core kernels."""
+    return gaparax([sink_latent(heads=6, dim=128, rot=64, rank=160, vdim=96, scale=0.08, base=5e4, scaling=yarn(4.0, 256, 16.0, 1.0), mlp=relu2_dense(520)),
+                    sigmoid_heads(heads=8, kv_heads=2, dim=128, vdim=104, chunk=200, scale=0.09, softcap=15.0, bias_max=90, mlp=group_moe(12, 4, 2, 4, 96)),
+                    sigmoid_heads(heads=4, kv_heads=4, dim=64, vdim=64, chunk=131, scale=0.2, softcap=30.0, bias_max=200, mlp=group_moe(10, 5, 4, 6, 80, 2.5)),
+                    sink_latent(heads=17, dim=48, rot=32, rank=96, vdim=40, scale=0.12, mlp=group_moe(8, 2, 1, 3, 64))], vocab=544, width=312, eps=1e-6, streams=2)

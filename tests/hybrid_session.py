@@ -4,12 +4,12 @@ import json
 
 import torch
 
-from . import gaborax_oracle, naselorn_oracle, nikelix_oracle
+from . import gaborax_oracle, gaparax_oracle, naselorn_oracle, nikelix_oracle
 
 DEV = "cuda"
 F32, BF16 = torch.float32, torch.bfloat16
 TOL = {F32: 2e-5, BF16: 4e-2}          # root mean square over the vocabulary, relative to that of the oracle's logits
-ORACLES = {"Nikelix": nikelix_oracle, "Naselorn": naselorn_oracle, "Gaborax": gaborax_oracle}
+ORACLES = {"Nikelix": nikelix_oracle, "Naselorn": naselorn_oracle, "Gaborax": gaborax_oracle, "Gaparax": gaparax_oracle}
 
 
 def tokens(n, vocab, seed=0):
