@@ -38,6 +38,19 @@ __device__ __forceinline__ float4 take4(void* p, size_t off, int kind) {
   if (kind == ROW_F32_TAKE) st4(f, make_float4(0.f, 0.f, 0.f, 0.f));
   return v;
 }
+// The two halves of take4 / take1: where several loads are in flight, the workspace is cleared once they have arrived (a store
+// behind a load of the same line that is still under way holds up the loads behind it).
+__device__ __forceinline__ int peek_kind(int kind) { return kind == ROW_BF16 ? ROW_BF16 : ROW_F32; }
+__device__ __forceinline__ void clear4(void* p, size_t off, int kind) {
+  if (kind == ROW_F32_TAKE) st4(reinterpret_cast<float*>(p) + off, make_float4(0.f, 0.f, 0.f, 0.f));
+}
+__device__ __forceinline__ void clear1(void* p, size_t off, int kind) {
+  if (kind == ROW_F32_TAKE) reinterpret_cast<float*>(p)[off] = 0.f;
+}
+__device__ __forceinline__ void clear8(void* p, size_t off, int kind) {
+  clear4(p, off, kind);
+  clear4(p, off + 4, kind);
+}
 // eight elements (16-byte aligned)
 __device__ __forceinline__ void take8(void* p, size_t off, int kind, float (&f)[8]) {
   if (kind == ROW_BF16) {

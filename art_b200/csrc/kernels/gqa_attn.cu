@@ -68,10 +68,10 @@ __global__ void __launch_bounds__(256) gqa_finish_kernel(const GqaFinish a) {
   for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
     float x[V];
     if (V == 4) {
-      const float4 v = take4(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+      const float4 v = take4(a.p, static_cast<size_t>(m) * a.ldp + c, peek_kind(a.kind));
       x[0] = v.x, x[1 % V] = v.y, x[2 % V] = v.z, x[3 % V] = v.w;
     } else {
-      x[0] = take1(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+      x[0] = take1(a.p, static_cast<size_t>(m) * a.ldp + c, peek_kind(a.kind));
     }
 #pragma unroll
     for (int e = 0; e < V; ++e)
@@ -89,6 +89,11 @@ __global__ void __launch_bounds__(256) gqa_finish_kernel(const GqaFinish a) {
     if (V == 4) st4(dst, make_float4(x[0], x[1 % V], x[2 % V], x[3 % V]));
     else st1(dst, x[0]);
   }
+  if (a.kind == ROW_F32_TAKE)
+    for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
+      if (V == 4) clear4(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+      else clear1(a.p, static_cast<size_t>(m) * a.ldp + c, a.kind);
+    }
   const int np = a.dk_p - a.dim;
   for (int j = threadIdx.x; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
 }
@@ -132,23 +137,28 @@ __global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish
   const size_t row = static_cast<size_t>(m) * a.ldp;
   float *cosine = gn_smem + ((nqk + 3) & ~3), *sine = cosine + ((half + 3) & ~3);
   float ssq = 0.f, ssk = 0.f;
-  for (int c0 = tid * V; c0 < n; c0 += blockDim.x * V * B) {
+  const int n_cols = a.cols ? a.H * a.vdim : 0, pk = peek_kind(a.kind);
+  for (int c0 = tid * V; c0 < n + n_cols; c0 += blockDim.x * V * B) {
     float x[B][V];
 #pragma unroll
     for (int u = 0; u < B; ++u) {
       const int c = c0 + u * blockDim.x * V;
-      if (c >= n) continue;
+      if (c >= n + n_cols) continue;
       if (V == 4) {
-        const float4 v = take4(a.p, row + c, a.kind);
+        const float4 v = take4(a.p, row + c, pk);
         x[u][0] = v.x, x[u][1 % V] = v.y, x[u][2 % V] = v.z, x[u][3 % V] = v.w;
       } else {
-        x[u][0] = take1(a.p, row + c, a.kind);
+        x[u][0] = take1(a.p, row + c, pk);
       }
     }
 #pragma unroll
     for (int u = 0; u < B; ++u) {
       const int c = c0 + u * blockDim.x * V;
-      if (c >= n) continue;
+      if (c >= n + n_cols) continue;
+      if (c >= n) {
+        put_vec(reinterpret_cast<T*>(a.cols) + static_cast<size_t>(m) * a.ldcols + by_vdim(c - n) * (a.colp - a.vdim) + c - n, x[u]);
+        continue;
+      }
       float t[V];
       if (a.bias) {
         get_vec(a.bias + c, t);
@@ -175,18 +185,14 @@ __global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish
       }
       put_vec(gn_smem + c, x[u]);
     }
-  }
-  if (a.cols) {
-    T* g = reinterpret_cast<T*>(a.cols) + static_cast<size_t>(m) * a.ldcols;
-    for (int c = tid * V; c < a.H * a.vdim; c += blockDim.x * V) {
-      float x[V];
-      if (V == 4) {
-        const float4 v = take4(a.p, row + n + c, a.kind);
-        x[0] = v.x, x[1 % V] = v.y, x[2 % V] = v.z, x[3 % V] = v.w;
-      } else {
-        x[0] = take1(a.p, row + n + c, a.kind);
+    if (a.kind == ROW_F32_TAKE) {
+#pragma unroll
+      for (int u = 0; u < B; ++u) {
+        const int c = c0 + u * blockDim.x * V;
+        if (c >= n + n_cols) continue;
+        if (V == 4) clear4(a.p, row + c, a.kind);
+        else clear1(a.p, row + c, a.kind);
       }
-      put_vec(g + by_vdim(c) * (a.colp - a.vdim) + c, x);
     }
   }
   if (a.gate)

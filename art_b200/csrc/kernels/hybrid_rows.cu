@@ -79,7 +79,8 @@ struct ResidualArgs {
   int ldxi;
 };
 
-// The sublayer's result (or the embedding row) of row `row`, four columns per thread and vector; `y` of columns past the row is zero.
+// The sublayer's result (or the embedding row) of row `row`, four columns per thread and vector; `y` of columns past the row is
+// zero.  Workspaces are cleared by clear_inputs at the end of a kernel.
 template <typename T, int MAXV>
 __device__ __forceinline__ void sublayer_result(const ResidualArgs& a, int row, int nv, float4 (&y)[MAXV]) {
   long tok = 0;
@@ -93,7 +94,7 @@ __device__ __forceinline__ void sublayer_result(const ResidualArgs& a, int row, 
     y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (v < nv) {
       if (a.tokens) y[i] = ld4(reinterpret_cast<const T*>(a.table) + static_cast<size_t>(tok) * a.ldt + v * 4);
-      else if (a.y) y[i] = take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, a.y_kind);
+      else if (a.y) y[i] = take4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, peek_kind(a.y_kind));
       if (a.y_gate) {
         const float g = __ldg(a.y_gate + row);
         y[i] = make_float4(y[i].x * g, y[i].y * g, y[i].z * g, y[i].w * g);
@@ -131,10 +132,22 @@ __device__ __forceinline__ void sublayer_result(const ResidualArgs& a, int row, 
     for (int i = 0; i < MAXV; ++i) {
       const int v = threadIdx.x + i * blockDim.x;
       if (v < nv) {
-        const float4 z = take4(a.rg, static_cast<size_t>(row) * a.ldrg + v * 4, a.rg_kind), b = ld4(a.rg_b + v * 4);
+        const float4 z = take4(a.rg, static_cast<size_t>(row) * a.ldrg + v * 4, peek_kind(a.rg_kind)), b = ld4(a.rg_b + v * 4);
         y[i] = make_float4(y[i].x * logistic_f(z.x + b.x), y[i].y * logistic_f(z.y + b.y), y[i].z * logistic_f(z.z + b.z), y[i].w * logistic_f(z.w + b.w));
       }
     }
+  }
+}
+
+template <int MAXV>
+__device__ __forceinline__ void clear_inputs(const ResidualArgs& a, int row, int nv) {
+  const bool y = a.y && a.y_kind == ROW_F32_TAKE, rg = a.rg && a.rg_kind == ROW_F32_TAKE;
+  if (!y && !rg) return;
+#pragma unroll
+  for (int i = 0; i < MAXV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nv && y) clear4(a.y, static_cast<size_t>(row) * a.ldy + v * 4, ROW_F32_TAKE);
+    if (v < nv && rg) clear4(a.rg, static_cast<size_t>(row) * a.ldrg + v * 4, ROW_F32_TAKE);
   }
 }
 
@@ -227,6 +240,7 @@ __global__ void __launch_bounds__(256) residual_step_kernel(const ResidualArgs a
     }
   }
   if (a.h) write_operand<T, MAXV>(a, row, nv, y, ss, red);      // uniform for the grid
+  clear_inputs<MAXV>(a, row, nv);
 }
 
 // Hyper-connections.  NS: the most copies on either side; the copies of a vector are read together, several vectors in flight.
@@ -288,6 +302,7 @@ __global__ void __launch_bounds__(256) stream_step_kernel(const ResidualArgs a) 
     }
   }
   if (a.h) write_operand<T, MAXV>(a, row, nv, y, ss, red);
+  clear_inputs<MAXV>(a, row, nv);
 }
 
 // ---------------------------------------------------------------------------------------------- token shift
@@ -397,7 +412,7 @@ poly_norm_kernel(void* z, int ldz, int kind, const float* __restrict__ act, T* o
     const int c = threadIdx.x + i * blockDim.x;
 #pragma unroll
     for (int j = 0; j < 8; ++j) v[i][j] = 0.f;
-    if (c < nv) take8(z, static_cast<size_t>(row) * ldz + c * 8, kind, v[i]);
+    if (c < nv) take8(z, static_cast<size_t>(row) * ldz + c * 8, peek_kind(kind), v[i]);
   }
 #pragma unroll
   for (int i = 0; i < MAXV; ++i)
@@ -429,6 +444,7 @@ poly_norm_kernel(void* z, int ldz, int kind, const float* __restrict__ act, T* o
         v[i][j] = c * 8 + j < n ? fmaf(fmaf(fmaf(c3, x, b), x, a), x, e0) : 0.f;
       }
       put8(out + static_cast<size_t>(row) * ldo + c * 8, v[i]);
+      clear8(z, static_cast<size_t>(row) * ldz + c * 8, kind);
     }
   }
 }
@@ -550,11 +566,13 @@ __global__ void __launch_bounds__(256) gated_act_kernel(void* z, int ldz, int ki
   const int c = static_cast<int>(u - m * nv) * 8;
   const size_t zo = static_cast<size_t>(m) * ldz + (c >> 4) * 32 + (c & 15);
   float g[8], x[8];
-  take8(z, zo, kind, g);
-  take8(z, zo + 16, kind, x);
+  take8(z, zo, peek_kind(kind), g);
+  take8(z, zo + 16, peek_kind(kind), x);
 #pragma unroll
   for (int i = 0; i < 8; ++i) x[i] *= act == ACT_RELU ? fmaxf(g[i], 0.f) : silu_f(g[i]);
   put8(out + static_cast<size_t>(m) * ldo + c, x);
+  clear8(z, zo, kind);
+  clear8(z, zo + 16, kind);
 }
 
 // z [M, np] -> out [M, np] = act(z).  Eight columns a thread.
@@ -567,13 +585,14 @@ __global__ void __launch_bounds__(256) plain_act_kernel(void* z, int ldz, int ki
   const long m = u / nv;
   const int c = static_cast<int>(u - m * nv) * 8;
   float x[8];
-  take8(z, static_cast<size_t>(m) * ldz + c, kind, x);
+  take8(z, static_cast<size_t>(m) * ldz + c, peek_kind(kind), x);
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
     const float p = fmaxf(x[i], 0.f);
     x[i] = act == ACT_RELU2 ? p * p : act == ACT_RELU ? p : silu_f(x[i]);
   }
   put8(out + static_cast<size_t>(m) * ldo + c, x);
+  clear8(z, static_cast<size_t>(m) * ldz + c, kind);
 }
 
 template <typename T, int MAXV>

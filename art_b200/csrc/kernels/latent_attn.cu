@@ -76,6 +76,7 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
   const int m = blockIdx.x, tid = threadIdx.x, hp = a.rot >> 1, hq = a.dim + a.rot;
   float *cc = cs, *sn = cs + hp;
   const size_t row = static_cast<size_t>(m) * a.ldp;
+  const int pk = peek_kind(a.kind);        // a workspace is cleared at the end
   for (int i = tid; i < hp; i += blockDim.x) {
     const float2 t = position_pair(a.pos[m], a.freq[i]);
     sn[i] = a.rot_scale * t.x;
@@ -94,22 +95,22 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
   for (int j = tid; j < a.H * du; j += blockDim.x) {
     const int h = j / du, i = (j - h * du) * W;
     float x[W];
-    take_v<W>(a.p, row + h * hq + i, a.kind, x);
+    take_v<W>(a.p, row + h * hq + i, pk, x);
     put_v(absorbed ? qn + static_cast<size_t>(h) * a.pitch * a.dim_p + i : erow + h * he + i, x);
   }
-  // latent: two passes over the row (the second finds it in L1 / L2; a taken workspace is only cleared then)
-  const int c0 = a.H * hq, rkind = a.kind == ROW_F32_TAKE ? ROW_F32 : a.kind;
+  // latent: two passes over the row (the second finds it in L1 / L2)
+  const int c0 = a.H * hq;
   float ss = 0.f;
   for (int i = tid * W; i < a.rank; i += blockDim.x * W) {
     float x[W];
-    take_v<W>(a.p, row + c0 + i, rkind, x);
+    take_v<W>(a.p, row + c0 + i, pk, x);
 #pragma unroll
     for (int e = 0; e < W; ++e) ss += x[e] * x[e];
   }
   const float r = 1.f / sqrtf(cta_sum(ss, red) / a.rank + a.eps);      // also the barrier behind cos / sin
   for (int i = tid * W; i < a.rank; i += blockDim.x * W) {
     float x[W];
-    take_v<W>(a.p, row + c0 + i, a.kind, x);
+    take_v<W>(a.p, row + c0 + i, pk, x);
 #pragma unroll
     for (int e = 0; e < W; ++e) x[e] = x[e] * r * a.w[i + e];
     if (slot >= 0) put_v(crow + i, x);
@@ -125,8 +126,8 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
       const int h = j / ru, i = (j - h * ru) * W;
       const size_t src = row + (h < a.H ? h * hq + a.dim : c0 + a.rank) + i;
       float x[W], z[W], y0[W], y1[W];
-      take_v<W>(a.p, src, a.kind, x);
-      take_v<W>(a.p, src + hp, a.kind, z);
+      take_v<W>(a.p, src, pk, x);
+      take_v<W>(a.p, src + hp, pk, z);
 #pragma unroll
       for (int e = 0; e < W; ++e) {
         y0[e] = x[e] * cc[i + e] - z[e] * sn[i + e];
@@ -143,7 +144,7 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
   for (int j = tid; j < (a.H + 1) * ru; j += blockDim.x) {
     const int h = j / ru, i = (j - h * ru) * RW;
     float x[RW], y[RW];
-    take_v<RW>(a.p, row + (h < a.H ? h * hq + a.dim : c0 + a.rank) + i, a.kind, x);
+    take_v<RW>(a.p, row + (h < a.H ? h * hq + a.dim : c0 + a.rank) + i, pk, x);
 #pragma unroll
     for (int e = 0; e < RW; e += 2) {
       const float c = cc[(i + e) >> 1], s = sn[(i + e) >> 1];
@@ -158,6 +159,13 @@ __global__ void __launch_bounds__(256) latent_finish_kernel(const LatentFinish a
     for (int j = tid; j < a.H * np; j += blockDim.x) {
       const int h = j / np, i = j - h * np;
       st1(erow + h * he + (i < a.dim_p - a.dim ? a.dim + i : a.dim + i + a.rot), 0.f);
+    }
+  }
+  if (a.kind == ROW_F32_TAKE) {
+    __syncthreads();
+    for (int i = tid * W; i < c0 + a.rank + a.rot; i += blockDim.x * W) {
+      if (W == 4) clear4(a.p, row + i, a.kind);
+      else clear1(a.p, row + i, a.kind);
     }
   }
 }
