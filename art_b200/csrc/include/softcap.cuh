@@ -15,6 +15,18 @@ __device__ __forceinline__ float tanh_from_exp(float u) {
   return fmaf(-2.f, rcp_approx(1.f + e), 1.f);
 }
 
+// of two numbers with one reciprocal: 1 / a = b / (a b).  From |u| = 20 on tanh is 1 in fp32; the product stays finite.
+__device__ __forceinline__ void tanh_pair(float& u, float& v) {
+  float e, f;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(u, 20.f) * 2.885390081777927f));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(f) : "f"(fminf(v, 20.f) * 2.885390081777927f));
+  e += 1.f;
+  f += 1.f;
+  const float r = -2.f * rcp_approx(e * f);
+  u = fmaf(r, f, 1.f);
+  v = fmaf(r, e, 1.f);
+}
+
 struct ScoreScale {
   float in;            // score / softcap = in * (q . k); 0: not squashed
   float scale_log2;    // factor behind it, log2(e) included
@@ -25,6 +37,17 @@ struct ScoreScale {
   }
   __host__ __device__ __forceinline__ bool capped() const { return in != 0.f; }
   __device__ __forceinline__ float squash(float qk) const { return tanh_from_exp(qk * in); }
+  __device__ __forceinline__ void squash(float& a, float& b) const {
+    a *= in;
+    b *= in;
+    tanh_pair(a, b);
+  }
+  // the exponents of two products
+  __device__ __forceinline__ void operator()(float& a, float& b) const {
+    if (capped()) squash(a, b);
+    a *= scale_log2;
+    b *= scale_log2;
+  }
   // the exponent (base 2) of a product q . k
   __device__ __forceinline__ float operator()(float qk) const { return (capped() ? squash(qk) : qk) * scale_log2; }
 };

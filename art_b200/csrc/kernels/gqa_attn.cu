@@ -484,17 +484,26 @@ __global__ void __launch_bounds__(128) gqa_decode_kernel(const GqaAttend a) {
       for (int e = 0; e < 2; ++e)
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          float w[2];
-#pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const int kt = k0 + i * 8 + 2 * t + j;
-            w[j] = kt < len ? sigmoid_base2(a.score(s[i][2 * e + j]) + (near ? a.bias.at(tab[e], p - kt) : far[e])) : 0.f;
+          if (e == 1 && ng <= 8) {                       // rows without a head
+            pf[i >> 1][(i & 1) * 2 + e] = 0;
+            continue;
           }
-          pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(w[0], w[1]);
+          float w[2] = {s[i][2 * e], s[i][2 * e + 1]};
+          const int kt = k0 + i * 8 + 2 * t;
+          a.score(w[0], w[1]);
+          w[0] += near ? a.bias.at(tab[e], p - kt) : far[e];
+          w[1] += near ? a.bias.at(tab[e], p - kt - 1) : far[e];
+          sigmoid_pair(w[0], w[1]);
+          pf[i >> 1][(i & 1) * 2 + e] = pair_bf16(kt < len ? w[0] : 0.f, kt + 1 < len ? w[1] : 0.f);
         }
     } else {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
+        if (e == 1 && ng <= 8) {                         // rows without a head
+#pragma unroll
+          for (int i = 0; i < 4; ++i) pf[i >> 1][(i & 1) * 2 + e] = 0;
+          continue;
+        }
         float mn = mx[e];
 #pragma unroll
         for (int i = 0; i < 4; ++i)

@@ -181,12 +181,15 @@ __global__ void __launch_bounds__(32 * LP_WARPS, DV <= 128 ? 2 : 1) latent_prefi
           if (SIG) {
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-              float w[2];
-#pragma unroll
-              for (int k = 0; k < 2; ++k) {
-                const int kp = k0 + j * 8 + 2 * t + k;
-                w[k] = sigmoid_base2(a.score(s[i][j][2 * e + k]) + (near ? a.bias.at(tab, p - kp) : far));
-                if (!inside && (kp > p || kp < first)) w[k] = 0.f;
+              float w[2] = {s[i][j][2 * e], s[i][j][2 * e + 1]};
+              const int kp = k0 + j * 8 + 2 * t;
+              a.score(w[0], w[1]);
+              w[0] += near ? a.bias.at(tab, p - kp) : far;
+              w[1] += near ? a.bias.at(tab, p - kp - 1) : far;
+              sigmoid_pair(w[0], w[1]);
+              if (!inside) {
+                if (kp > p || kp < first) w[0] = 0.f;
+                if (kp + 1 > p || kp + 1 < first) w[1] = 0.f;
               }
               pf[i][j >> 1][(j & 1) * 2 + e] = pair_bf16(w[0], w[1]);
             }

@@ -308,17 +308,19 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       if (lane == 0) mbar_arrive(&s_empty[s]);
       if (a.score.capped()) {
 #pragma unroll
-        for (int j = 0; j < 64; ++j) x[j] = a.score.squash(x[j]);
+        for (int j = 0; j < 64; j += 2) a.score.squash(x[j], x[j + 1]);
       }
       if (SIG) {
         if (a.bias.beyond(p0, k0 + LT_B - 1)) {
 #pragma unroll
-          for (int j = 0; j < 64; ++j) x[j] = sigmoid_base2(fmaf(x[j], a.score.scale_log2, far));
+          for (int j = 0; j < 64; ++j) x[j] = fmaf(x[j], a.score.scale_log2, far);
         } else {                              // distances of the tile stay within the table's padding
           const float* td = tab + qpos - (k0 + hf * 64);
 #pragma unroll
-          for (int j = 0; j < 64; ++j) x[j] = sigmoid_base2(fmaf(x[j], a.score.scale_log2, __ldg(td - j)));
+          for (int j = 0; j < 64; ++j) x[j] = fmaf(x[j], a.score.scale_log2, __ldg(td - j));
         }
+#pragma unroll
+        for (int j = 0; j < 64; j += 2) sigmoid_pair(x[j], x[j + 1]);
         if (!inside) {
           const int hi = qpos - (k0 + hf * 64), lo = first - (k0 + hf * 64);
 #pragma unroll
