@@ -57,23 +57,28 @@ struct ColumnGate {
     return {g, ld, pitch, vdim, p && !((ld | pitch) & 7) && !(reinterpret_cast<uintptr_t>(p) & 15)};
   }
   __device__ __forceinline__ const T* row(int m, int h) const { return g + static_cast<size_t>(m) * ld + static_cast<size_t>(h) * pitch; }
+  __device__ __forceinline__ void prefetch(int m, int h, int d) const { asm volatile("prefetch.global.L2 [%0];" ::"l"(row(m, h) + d)); }
   // factor of column d (1 for padding columns)
   __device__ __forceinline__ float operator()(int m, int h, int d) const { return g && d < vdim ? logistic_f(ld1(row(m, h) + d)) : 1.f; }
-  // x[0 .. 7] of columns d .. d + 7
-  __device__ __forceinline__ void scale8(int m, int h, int d, float (&x)[8]) const {
-    if (!g) return;
-    if (vec && d + 8 <= vdim) {
-      float z[8];
-      const T* p = row(m, h) + d;
-      const float4 a = ld4(p), b = ld4(p + 4);
-      z[0] = a.x, z[1] = a.y, z[2] = a.z, z[3] = a.w, z[4] = b.x, z[5] = b.y, z[6] = b.z, z[7] = b.w;
+  // logits of columns d .. d + 7 (bf16), and what they make of those columns
+  __device__ __forceinline__ uint4 load8(int m, int h, int d) const {
+    if (vec && d + 8 <= vdim) return *reinterpret_cast<const uint4*>(row(m, h) + d);
+    __align__(16) T z[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) x[i] *= rcp_approx(1.f + exp2_approx(-z[i] * KW_LOG2E));
-      return;
+    for (int i = 0; i < 8; ++i) z[i] = d + i < vdim ? row(m, h)[d + i] : T(0.f);
+    return *reinterpret_cast<const uint4*>(z);
+  }
+  static __device__ __forceinline__ void apply8(const uint4& q, float (&x)[8]) {
+    const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&q);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      float2 z = __bfloat1622float2(b[i]);
+      z.x *= KW_LOG2E;
+      z.y *= KW_LOG2E;
+      sigmoid_pair(z.x, z.y);
+      x[2 * i] *= z.x;
+      x[2 * i + 1] *= z.y;
     }
-#pragma unroll
-    for (int i = 0; i < 8; ++i)
-      if (d + i < vdim) x[i] *= logistic_f(ld1(row(m, h) + d + i));
   }
 };
 

@@ -223,6 +223,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
     uint8_t* prow = smem + L::P + hf * LT_BLK + r * 128;
     const int sw = r & 7;
+    if (a.cols.g && r < nrow && hf * OC < a.cols.vdim) a.cols.prefetch(r0 + r, h, hf * OC);      // the epilogue's loads then hit the L2
     float O[OC];
 #pragma unroll
     for (int i = 0; i < OC; ++i) O[i] = 0.f;
@@ -397,6 +398,12 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
       }
       ms_prev = ms;
     }
+    uint4 gates[OC / 8];                      // they arrive while the last product ends
+    const bool gated = a.cols.g && r < nrow;
+    if (gated) {
+#pragma unroll
+      for (int c = 0; c < OC; c += 8) gates[c / 8] = a.cols.load8(r0 + r, h, hf * OC + c);
+    }
     float l_other = 0.f;
     if (SIG) {
       const int okw = !dead && mbar_wait_timed(&pv_full[0], 0) ? 1 : 0;
@@ -428,7 +435,7 @@ latent_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_c
           float y[8];
 #pragma unroll
           for (int j = 0; j < 8; ++j) y[j] = O[c + j] * inv;
-          a.cols.scale8(r0 + r, h, hf * OC + c, y);
+          if (gated) a.cols.apply8(gates[c / 8], y);
           uint4 w;
           w.x = pack_bf16x2(y[0], y[1]);
           w.y = pack_bf16x2(y[2], y[3]);
