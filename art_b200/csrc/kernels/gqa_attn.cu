@@ -8,6 +8,7 @@
 //   gqa_finish_norm_kernel   the same with a norm over all heads of q, and of k, or over each head, a rotation of the first
 //                        columns of every head (angles reduced in fp64, as for position vectors) and the heads' or columns'
 //                        gates
+//   gqa_finish_heads_kernel  a norm over each head and no rotation, heads of a power of two up to 128: in registers alone
 //   gqa_gather_kernel    the cache rows a batch's portions see, contiguous: keys row by row, values transposed, as the
 //                        tcgen05 kernel of latent_prefill_tc.cu wants them (sizes that do not suit it: latent_gather and
 //                        latent_prefill)
@@ -282,6 +283,66 @@ __global__ void __launch_bounds__(256, 5) gqa_finish_norm_kernel(const GqaFinish
     }
   const int np = a.dk_p - a.dim;
   for (int j = tid; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
+}
+
+// A warp takes 128 columns at a time, a lane four: a head is dim / 4 neighbouring lanes.
+template <typename T>
+__global__ void __launch_bounds__(256) gqa_finish_heads_kernel(const GqaFinish a, const QuickDiv by_vdim) {
+  constexpr int B = 4;                                  // loads of a thread in flight
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x, lane = threadIdx.x & 31, step = blockDim.x * 4;
+  int slot = a.slot[m];
+  if (slot >= 0 && !index_ok(slot, a.num_slots, a.status)) slot = -1;
+  T* crow = reinterpret_cast<T*>(a.cache) + static_cast<size_t>(slot < 0 ? 0 : slot) * a.ldc;
+  T* qrow = reinterpret_cast<T*>(a.q) + static_cast<size_t>(m) * a.ldq;
+  T* grow = reinterpret_cast<T*>(a.cols) + static_cast<size_t>(a.cols ? m : 0) * a.ldcols;
+  const int nq = a.H * a.dim, nqk = nq + a.Hkv * a.dim, n = nqk + a.Hkv * a.vdim, total = n + (a.cols ? a.H * a.vdim : 0);
+  const size_t row = static_cast<size_t>(m) * a.ldp;
+  const int pk = peek_kind(a.kind), shift = 31 - __clz(a.dim), d0 = (lane * 4) & (a.dim - 1);
+  const float4 wq = ld4(a.wq + d0), wk = a.Hkv ? ld4(a.wk + d0) : wq;
+  const float inv_dim = 1.f / a.dim;
+  for (int c0 = (threadIdx.x - lane) * 4; c0 < total; c0 += step * B) {      // the same for a warp
+    float4 x[B];
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = c0 + u * step + lane * 4;
+      x[u] = c < total ? take4(a.p, row + c, pk) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int u = 0; u < B; ++u) {
+      const int c = c0 + u * step + lane * 4;
+      if (a.bias && c < n) {
+        const float4 b = ld4(a.bias + c);
+        x[u] = make_float4(x[u].x + b.x, x[u].y + b.y, x[u].z + b.z, x[u].w + b.w);
+      }
+      float ss = sq4(x[u]);
+      for (int o = a.dim >> 3; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (c < nqk) {
+        const int hd = c >> shift;
+        const bool isq = hd < a.H;
+        float r = rsqrtf(fmaf(ss, inv_dim, a.eps));
+        if (isq && a.q_scale) r *= __ldg(a.q_scale + hd);
+        const float4 w = isq ? wq : wk;
+        x[u] = make_float4(x[u].x * r * w.x, x[u].y * r * w.y, x[u].z * r * w.z, x[u].w * r * w.w);
+        if (isq) st4(qrow + hd * a.dk_p + d0, x[u]);
+        else if (slot >= 0) st4(crow + (hd - a.H) * a.dk_p + d0, x[u]);
+      } else if (c < n) {
+        if (slot >= 0) st4(crow + a.Hkv * a.dk_p + by_vdim(c - nqk) * (a.dv_p - a.vdim) + c - nqk, x[u]);
+      } else if (c < total) {
+        st4(grow + by_vdim(c - n) * (a.colp - a.vdim) + c - n, x[u]);
+      }
+    }
+    if (a.kind == ROW_F32_TAKE) {
+#pragma unroll
+      for (int u = 0; u < B; ++u) {
+        const int c = c0 + u * step + lane * 4;
+        if (c < total) clear4(a.p, row + c, a.kind);
+      }
+    }
+  }
+  const int np = a.dk_p - a.dim;
+  for (int j = threadIdx.x; j < a.H * np; j += blockDim.x) st1(qrow + j / np * a.dk_p + a.dim + j % np, 0.f);
 }
 
 struct GqaGather {
@@ -765,6 +826,9 @@ ARTB_EXPORT int artb_gqa_finish_norm(int f32, void* p, int ldp, int kind, const 
                   !((ldcols | colp) & 3) && aligned(cols);
   const QuickDiv by_dim = QuickDiv::by(dim), by_vdim = QuickDiv::by(vdim),
                  by_units = QuickDiv::by(rot ? (next ? rot / (v4 ? 4 : 2) : rot / 2 / (v4 ? 4 : 1)) : 1);
+  if (per_head && !rot && v4 && !gate && dim <= 128 && !(dim & (dim - 1)))
+    return static_cast<int>(f32 ? launch_kernel(gqa_finish_heads_kernel<float>, dim3(M), dim3(256), 0, st, a, by_vdim)
+                                : launch_kernel(gqa_finish_heads_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, st, a, by_vdim));
 #define ARTB_GN(T_, V_)                                                                                                        \
   do {                                                                                                                         \
     if (smem > 48 * 1024) {                                                                                                    \

@@ -15,7 +15,7 @@ import torch
 
 
 def measure_decode(cfg, device, seqs: int = 256, prompt_len: int = 512, new_tokens: int = 128, loras: int = 4,
-                   runs: int = 3, base=None, tp_group=None, prompt_len_max: int = 0) -> dict:
+                   runs: int = 3, base=None, tp_group=None, prompt_len_max: int = 0, prefill_runs: int = 0) -> dict:
     """Prefill + decode throughput of one engine replica.  ``tp_group``: the replica spans that process group (every
     rank calls this with the same arguments and gets the same numbers).  ``prompt_len_max`` > ``prompt_len`` draws
     prompt lengths uniformly from [prompt_len, prompt_len_max].  The first ``runs - 1`` passes warm every CUDA-graph
@@ -98,6 +98,25 @@ def measure_decode(cfg, device, seqs: int = 256, prompt_len: int = 512, new_toke
         for s in reqs:
             eng._release(s)
         eng.running = []
+    # prompts alone, several times: the first pass behind a decode phase may wait for the allocator
+    times = []
+    for run in range(prefill_runs):
+        reqs = [eng.add_request(torch.randint(0, cfg.vocab_size, (prompt_len,), generator=g).tolist(), SamplingParams(max_tokens=1, temperature=1.0, ignore_eos=True))
+                for _ in range(seqs)]
+        e0, e1 = (torch.cuda.Event(enable_timing=True) for _ in range(2))
+        torch.cuda.synchronize()
+        e0.record()
+        while not all(s.finished for s in reqs):
+            eng.step()
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1) / 1e3)
+        for s in reqs:
+            eng._release(s)
+        eng.running = []
+    if times:
+        t_pre = sorted(times)[len(times) // 2]
+        res.update(prefill_tok_s=round(seqs * prompt_len / t_pre, 1), prefill_s=round(t_pre, 4))
     _lib.check_status(dev)
     runner.close()
     return res

@@ -61,7 +61,7 @@ def engine_rows(names: list[str], batches: list[int], prompt_len: int = 1024, ne
             cfg.layers = cfg.layers[:layers]
         for seqs in batches:
             for c in (cfg, twin(cfg)):
-                r = measure_decode(c, "cuda", seqs=seqs, prompt_len=prompt_len, new_tokens=new_tokens, loras=0)
+                r = measure_decode(c, "cuda", seqs=seqs, prompt_len=prompt_len, new_tokens=new_tokens, loras=0, prefill_runs=7)
                 torch.cuda.empty_cache()
                 yield {"model": r["model"], "layers": c.num_layers, "params_b": round(c.num_params() / 1e9, 2), "seqs": seqs,
                        "prompt_len": prompt_len, "new_tokens": new_tokens, "prefill_tok_s": r["prefill_tok_s"],
