@@ -36,9 +36,8 @@ __device__ __forceinline__ float exp2_approx(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// sigmoid(x ln 2): the weight of a key whose score is x in base-2 units
-__device__ __forceinline__ float sigmoid_base2(float x) { return rcp_approx(1.f + exp2_approx(-x)); }
-// of two numbers with one reciprocal (1 / a = b / (a b)); weights below 2^-60 count as that, so that the product stays finite
+// sigmoid(x ln 2), the weight of a key whose score is x in base-2 units, of two keys with one reciprocal (1 / a = b / (a b));
+// weights below 2^-60 count as that, so that the product stays finite
 __device__ __forceinline__ void sigmoid_pair(float& x, float& y) {
   const float a = 1.f + exp2_approx(fminf(-x, 60.f)), b = 1.f + exp2_approx(fminf(-y, 60.f)), r = rcp_approx(a * b);
   x = r * b;
